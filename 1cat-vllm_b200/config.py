@@ -79,6 +79,35 @@ class QuantConfig:
         raise ValueError(f"unsupported quantization method {m!r}")
 
 
+def _gabisun_fields(hf: dict) -> dict:
+    """``ModelConfig`` fields of a Gabisun config.json: a list of layers with their own attention and feed-forward sizes, an optional run
+    of looped layers, layer norms on both sides of every sub-block, layer scales and tied embeddings. The number of distance buckets is
+    the row count of a checkpoint's bias table; the value here is what random-weight models use."""
+    layers, over = hf["layers"], []
+    for i, l in enumerate(layers):
+        if l.get("type") != "attention":
+            raise ValueError(f"Gabisun layer {i}: mixer {l.get('type')!r} is not known")
+        m, mlp, mask = l["mixer"], l.get("mlp"), l["mixer"].get("mask")
+        if m.get("vdim", m["dim"]) != m["dim"]:
+            raise ValueError(f"Gabisun layer {i}: the values are the keys, so vdim must equal dim")
+        if mlp is not None and mlp.get("kind", "dense") != "dense":
+            raise ValueError(f"Gabisun layer {i}: feed-forward {mlp.get('kind')!r} is not known")
+        over.append(dict(num_attention_heads=int(m["heads"]), num_key_value_heads=int(m["kv_heads"]), head_dim=int(m["dim"]),
+                         attn_scale=float(m["scale"]), attn_rel_max=int(m["bias_max"]), sliding_window=int(mask["size"]) if mask else 0,
+                         attn_window_keep=int(mask.get("keep_first", 0)) if mask else 0, intermediate_size=int(mlp["ff"]) if mlp else 0,
+                         mixer_only_layers=mlp is None))
+    loop, n = hf.get("loop"), len(layers)
+    if loop and not (0 <= loop["start"] < loop["stop"] <= n and loop["times"] >= 1):
+        raise ValueError(f"Gabisun loop {loop} does not fit {n} layers")
+    top = {k: over[0][k] for k in ("num_attention_heads", "num_key_value_heads", "head_dim", "attn_scale")}
+    return dict(architecture="Gabisun", vocab_size=int(hf["vocab"]), hidden_size=int(hf["width"]), num_hidden_layers=n,
+                intermediate_size=max(o["intermediate_size"] for o in over), rms_norm_eps=float(hf["norm"]["eps"]), norm_type="layernorm",
+                norm_bias=True, sandwich_norm=True, layer_scale=True, residual_fp32=True, tie_word_embeddings=True, mlp_gated=False,
+                hidden_act="gelu_tanh", attn_sinks=True, attn_head_gate=True, attn_kv_shared=True, attn_rel_buckets=32,
+                nope_layers=tuple(range(n)), sliding_layers=tuple(i for i, o in enumerate(over) if o["sliding_window"]),
+                layer_overrides=tuple(over), loop=(int(loop["start"]), int(loop["stop"]), int(loop["times"])) if loop else None, **top)
+
+
 @dataclass
 class ModelConfig:
     """Architecture description, normalised from an HF ``config.json`` (or a dict for synthetic models).
@@ -137,6 +166,16 @@ class ModelConfig:
     nope_layers: tuple = ()  # layers whose attention applies no rotary embedding (SmolLM3)
     pre_norm: bool = True  # False: no norm before a sub-block, its output is normalised and added (OLMo-2 / OLMo-3)
     qk_norm_full: bool = False  # q / k RMSNorm over the whole projection instead of per head (OLMo-2 / OLMo-3)
+    # values of single layers that differ from the model's: per layer a dict of ModelConfig fields (``for_layer`` applies it)
+    layer_overrides: tuple = ()
+    attn_window_keep: int = 0  # sliding-window layers: the first tokens of a sequence stay visible to every later position
+    attn_kv_shared: bool = False  # the values are the projected keys: no value projection, one cached tensor per layer
+    attn_head_gate: bool = False  # each head's output is multiplied by sigmoid(g_proj(x)) of that head before the output projection
+    attn_rel_buckets: int = 0  # > 0: a learned bias per (distance bucket, head) is added to the scores; a checkpoint's table sets the row count
+    attn_rel_max: int = 0  # distance at which the last bucket begins
+    layer_scale: bool = False  # a sub-block's (normalised) output is multiplied by a learned vector before it joins the residual
+    residual_fp32: bool = False  # the residual stream is carried in fp32 (fused join kernel); logits are fp32 as well
+    loop: Optional[tuple] = None  # (start, stop, times): layers start..stop-1 run ``times`` times in a row with the same weights
     num_labels: int = 0  # > 0: a *ForSequenceClassification checkpoint (a ``score`` head on the pooled state instead of an LM head)
     # hybrid (Gated-DeltaNet)
     layer_types: Optional[list[str]] = None  # "full_attention" | "linear_attention" (Gated-DeltaNet) | "mamba2" | "mamba1" | "short_conv"
@@ -226,6 +265,25 @@ class ModelConfig:
         """Sliding window of layer ``i`` in tokens, 0 for full attention."""
         return self.sliding_window if i in self.sliding_layers else 0
 
+    def for_layer(self, i: int) -> "ModelConfig":
+        """The configuration layer ``i`` is built from: this one with the layer's own values in place."""
+        ov = self.layer_overrides[i] if i < len(self.layer_overrides) else None
+        return dataclasses.replace(self, layer_overrides=(), **ov) if ov else self
+
+    def layer_runs(self) -> list[tuple[int, int]]:
+        """(layer index, pass) in execution order; the pass is -1 for layers outside the loop. Each entry has its own K/V pages."""
+        n = self.num_hidden_layers
+        if self.loop is None:
+            return [(i, -1) for i in range(n)]
+        a, b, times = self.loop
+        return [(i, -1) for i in range(a)] + [(i, t) for t in range(times) for i in range(a, b)] + [(i, -1) for i in range(b, n)]
+
+    def release_window(self) -> tuple[int, int]:
+        """(window, kept first tokens) outside of which no layer reads a sequence's K/V; (0, 0) when some layer reads all of it."""
+        cfgs = [self.for_layer(i) for i in range(self.num_hidden_layers)]
+        w = [c.layer_window(i) for i, c in enumerate(cfgs)]
+        return (max(w), max(c.attn_window_keep for c in cfgs)) if w and all(w) else (0, 0)
+
     def is_moe_layer(self, i: int) -> bool:
         return self.is_moe and i >= self.first_k_dense_replace and i not in self.dense_layers
 
@@ -251,6 +309,8 @@ class ModelConfig:
     def from_hf_dict(cls, hf: dict, **over) -> "ModelConfig":
         """Normalise an HF config dict. Nested ``text_config`` (Qwen3.5) is flattened."""
         over = dict(over)
+        if hf.get("architecture") == "Gabisun" or "Gabisun" in (hf.get("architectures") or ()):
+            return cls(**{**_gabisun_fields(hf), **over})
         mm_ids = {m: int(hf[k]) for m, k in (("image", "image_token_id"), ("video", "video_token_id"), ("audio", "audio_token_id")) if hf.get(k) is not None}
         if mm_ids:
             over.setdefault("mm_token_ids", mm_ids)

@@ -29,7 +29,7 @@ def cdiv(a: int, b: int) -> int:
 class KVCacheManager:
     def __init__(self, num_blocks: int, block_size: int, max_model_len: int, enable_caching: bool = True,
                  num_state_slots: int = 0, use_eagle: bool = False, dcp_world_size: int = 1, log_stats: bool = True,
-                 sliding_window: int = 0) -> None:
+                 sliding_window: int = 0, window_keep: int = 0) -> None:
         self.block_size = block_size * dcp_world_size  # with decode-CP a logical block spans all ranks
         self.max_model_len = max_model_len
         self.enable_caching = enable_caching and num_state_slots == 0
@@ -46,6 +46,9 @@ class KVCacheManager:
         # the next query are given back while the request runs (reference: single_type_kv_cache_manager.py:570 ``SlidingWindowManager``
         # ``remove_skipped_blocks``). Models that mix windowed and global layers share one block table here and keep every block.
         self.sliding_window = sliding_window
+        # The first `window_keep` tokens stay visible outside the window; their pages (in whole 64-key tiles, as the kernels load them)
+        # are never given back early.
+        self.window_keep_blocks = cdiv(cdiv(window_keep, 64) * 64, self.block_size)
         self.window_slack = 128  # keys kept below the window start: the attention kernels load whole key tiles and mask inside them
 
     def enable_cpu_offload(self, num_cpu_blocks: int, policy: str = "lru") -> None:
@@ -171,7 +174,7 @@ class KVCacheManager:
         blocks they fill (their table entries become the placeholder block, so positions keep their indices)."""
         n = (first_query_pos - self.sliding_window + 1 - self.window_slack) // self.block_size
         gone = []
-        for i in range(min(max(n, 0), len(blocks))):
+        for i in range(self.window_keep_blocks, min(max(n, 0), len(blocks))):
             if not blocks[i].is_null:
                 gone.append(blocks[i])
                 blocks[i] = self.block_pool.null_block

@@ -126,12 +126,13 @@ class KVCacheSpec:
     head_size: int
     dtype_bytes: int
     state_bytes: int = 0  # mamba: bytes of recurrent + conv state per sequence
+    tensors: int = 2  # full: cached tensors per page, keys and values (1: the values are the keys)
 
     @property
     def page_size_bytes(self) -> int:
         if self.kind == "mamba":
             return self.state_bytes
-        coef = 1 if self.kind == "mla" else 2
+        coef = 1 if self.kind == "mla" else self.tensors
         return coef * self.block_size * self.num_kv_heads * self.head_size * self.dtype_bytes
 
 

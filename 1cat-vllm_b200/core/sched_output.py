@@ -56,6 +56,9 @@ class SchedulerOutput:
     scheduled_encoder_inputs: dict[str, list[int]] = field(default_factory=dict)  # request id -> indices of its multimodal items to encode
     free_encoder_mm_hashes: list = field(default_factory=list)  # encoder outputs the workers may drop
 
+    # trace replay: request id -> offsets among its scheduled tokens whose logits are reported; such a step samples nothing
+    logits_for: Optional[dict] = None
+
     @property
     def is_empty(self) -> bool:
         return self.total_num_scheduled_tokens == 0
@@ -79,6 +82,7 @@ class ModelRunnerOutput:
     prompt_logprobs: Optional[dict] = None
     num_nans_in_logits: Optional[dict] = None
     pooler_output: Optional[list] = None  # per request: pooled vector (list of floats) once its prompt is complete, else None
+    logits: Any = None  # fp32 host tensor [rows, vocab] of the positions in SchedulerOutput.logits_for, in their order
     device_time_ms: float = 0.0  # CUDA-event time of the step (0 when not measured)
     status: int = 0  # non-zero: a bounded device wait expired
 

@@ -117,12 +117,12 @@ class Scheduler:
         mc = vllm_config.model_config
         self.num_spec_tokens = spec.num_speculative_tokens if spec.enabled else 0
         self.num_lookahead_tokens = self.num_spec_tokens if spec.method in ("mtp", "eagle", "eagle3", "draft_model") else 0
+        window, window_keep = mc.release_window() if not spec.enabled else (0, 0)
         self.kv_cache_manager = KVCacheManager(num_gpu_blocks, cc.block_size, self.max_model_len, cc.enable_prefix_caching,
                                                num_state_slots, use_eagle=spec.method in ("mtp", "eagle", "eagle3", "draft_model"),
                                                dcp_world_size=vllm_config.parallel_config.decode_context_parallel_size,
                                                log_stats=log_stats,
-                                               sliding_window=(mc.sliding_window if mc.sliding_window and len(mc.sliding_layers) == mc.num_hidden_layers
-                                                               and not spec.enabled else 0))
+                                               sliding_window=window, window_keep=window_keep)
         from onecat_vllm.core.encoder_cache_manager import EncoderCacheManager
         self.max_num_encoder_input_tokens = sc.max_num_encoder_input_tokens
         self.encoder_cache_manager = EncoderCacheManager(sc.encoder_cache_size)
@@ -149,7 +149,9 @@ class Scheduler:
             request = Request.from_engine_core_request(request, self.block_hasher)
         if request.request_id in self.requests:
             raise ValueError(f"duplicate request id {request.request_id}")
-        if request.num_prompt_tokens >= self.max_model_len:
+        # room for one sampled token is needed unless nothing is sampled (trace replay)
+        samples = request.sampling_params is not None or request.pooling_params is not None
+        if request.num_prompt_tokens + samples > self.max_model_len:
             raise ValueError(f"prompt of {request.num_prompt_tokens} tokens does not fit max_model_len={self.max_model_len}")
         if request.num_prompt_tokens == 0:
             raise ValueError("empty prompt")
@@ -334,6 +336,38 @@ class Scheduler:
 
         out.total_num_scheduled_tokens = self.max_num_scheduled_tokens - budget
         assert out.total_num_scheduled_tokens == sum(out.num_scheduled_tokens.values())
+        return self._finish_schedule(out, scheduled_new, scheduled_resumed, scheduled_running, preempted, new_blocks_of)
+
+    def schedule_exact(self, num_tokens: dict[str, int]) -> SchedulerOutput:
+        """A step with exactly these token counts (trace replay): the named requests, waiting ones admitted, run that many of their
+        next tokens together. Pages come from the same manager as for ``schedule``; there is no preemption, running out is an error."""
+        out = SchedulerOutput()
+        scheduled_new: list[Request] = []
+        scheduled_running: list[Request] = []
+        new_blocks_of: dict[str, list[int]] = {}
+        for rid, n in num_tokens.items():
+            r = self.requests[rid]
+            if not 0 < n <= r.num_tokens - r.num_computed_tokens:
+                raise ValueError(f"request {rid} has {r.num_tokens - r.num_computed_tokens} tokens left, not {n}")
+            new_blocks = self.kv_cache_manager.allocate_slots(r, n)
+            if new_blocks is None:
+                raise RuntimeError(f"the KV cache cannot hold {n} more tokens of request {rid}")
+            new_blocks_of[rid] = [b.block_id for b in new_blocks]
+            if r.status == RequestStatus.WAITING:
+                self.waiting.remove(r)
+                self.running.append(r)
+                r.status = RequestStatus.RUNNING
+                scheduled_new.append(r)
+            else:
+                scheduled_running.append(r)
+            out.num_scheduled_tokens[rid] = n
+        out.total_num_scheduled_tokens = sum(num_tokens.values())
+        return self._finish_schedule(out, scheduled_new, [], scheduled_running, [], new_blocks_of, forced=True)
+
+    def _finish_schedule(self, out: SchedulerOutput, scheduled_new: list, scheduled_resumed: list, scheduled_running: list, preempted: list,
+                         new_blocks_of: dict, forced: bool = False) -> SchedulerOutput:
+        """What the workers need for the chosen requests; counts the step's tokens as computed. ``forced``: running requests take their
+        next tokens from the scheduler instead of from sampling."""
         km = self.kv_cache_manager
         out.scheduled_new_reqs = [
             NewRequestData(r.request_id, r.prompt_token_ids, r.sampling_params, new_blocks_of[r.request_id],
@@ -347,7 +381,7 @@ class Scheduler:
             cached.resumed_from_preemption.append(resumed)
             if resumed:
                 cached.new_token_ids.append(list(r.all_token_ids))
-            elif self.use_pp:  # stages that do not sample learn the tokens from here (reference: scheduler.py ``use_pp`` branch)
+            elif self.use_pp or forced:  # stages that do not sample learn the tokens from here (reference: scheduler.py ``use_pp`` branch)
                 cached.new_token_ids.append(list(r.all_token_ids[r.num_computed_tokens:]))
             else:
                 cached.new_token_ids.append([])

@@ -13,6 +13,10 @@
 // joins the softmax denominator only).
 // FP8 KV cache (KV8): pages hold e4m3 bytes in the same layout; tiles stream through a byte-wide cp.async ring and are widened to
 // bf16 into one working tile per operand before the MMAs; the per-tensor scales fold into the softmax scale (K) and the output (V).
+// Extended variants (EXT, bf16 cache): first tokens that stay visible outside the window (their tiles are walked ahead of the window's),
+// a bias by distance added to the scores in fp32, values that are the keys (one tensor per page: the ring holds one tile per stage and
+// both products read it), one output gate per head. The softmax weights enter the value product as two bf16 terms (p and the rest of
+// p after rounding), so that they keep about 16 bits of mantissa.
 // (reference: flash-attention-v100/kernel/fused_mha_forward_paged.cu:364, flash_decode_paged.cu:667,831,1301;
 //  v1/attention/backends/flash_attn_v100.py:2216 for the math)
 #include <cuda_fp8.h>
@@ -70,7 +74,15 @@ __device__ __forceinline__ void widen_fp8x16(const uint4& in, uint4& lo, uint4& 
   hi = make_uint4(widen_fp8_pair(in.z, 0x1404u), widen_fp8_pair(in.z, 0x3424u), widen_fp8_pair(in.w, 0x1404u), widen_fp8_pair(in.w, 0x3424u));
 }
 
-template <int D, int MODE, int MB, bool KV8, int ST = 3>
+constexpr float kLog2e = 1.4426950408889634f;
+
+// sigmoid of the output gate of (token, head); 1 without a gate
+__device__ __forceinline__ float head_gate(const AttnParams& p, size_t tok, int head) {
+  if (p.gate == nullptr) return 1.f;
+  return 1.f / (1.f + __expf(-__bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.gate)[tok * p.gate_st + head])));
+}
+
+template <int D, int MODE, int MB, bool KV8, int ST = 3, bool EXT = false>
 __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
   pdl_trigger();
   pdl_wait();
@@ -85,7 +97,8 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
   constexpr int ESZ = KV8 ? 1 : 2;
   uint8_t* sQ = smem;
   uint8_t* sK = sQ + ROWS * D * 2;
-  uint8_t* sV = sK + STAGES * kKeysPerTile * D * ESZ;
+  const bool shared_kv = EXT && p.kv_shared;    // one tile per stage serves both products
+  uint8_t* sV = shared_kv ? sK : sK + STAGES * kKeysPerTile * D * ESZ;
   uint8_t* sKb = sV + STAGES * kKeysPerTile * D * ESZ;
   uint8_t* sVb = sKb + kKeysPerTile * D * 2;
   __shared__ int s_req, s_tile0;
@@ -131,9 +144,17 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
   const int wlo = p.window > 0 ? p.window : 0x3fffffff;
   const int tile_first = p.window > 0 ? max(0, ctx0 + tq0 - p.window + 1) / kKeysPerTile : 0;
   int tile_lo = tile_first, tile_hi = ntiles;
+  // kept first tokens: their tiles that lie wholly before the window are walked first (tile index - tile_shift for those)
+  int keep_tiles = 0;
+  if (EXT) {
+    keep_tiles = min((p.keep + kKeysPerTile - 1) / kKeysPerTile, tile_first);
+    tile_lo -= keep_tiles;
+  }
+  const int tile_shift = tile_first - keep_tiles, tile_first_v = tile_lo;
+  auto tile_of = [&](int v) { return (EXT && v < tile_first) ? v - tile_shift : v; };
   if (MODE == 1 && p.splits > 1) {
-    int per = (ntiles - tile_first + p.splits - 1) / p.splits;
-    tile_lo = tile_first + blockIdx.z * per;
+    int per = (ntiles - tile_first_v + p.splits - 1) / p.splits;
+    tile_lo = tile_first_v + blockIdx.z * per;
     tile_hi = min(ntiles, tile_lo + per);
   }
   const int* bt = p.block_table + (size_t)r * p.bt_stride;
@@ -147,7 +168,7 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
   const int bs_shift = p.bs_shift, bs_mask = p.bs - 1;
   // byte addressing covers both element sizes
   const uint8_t* kv_head = reinterpret_cast<const uint8_t*>(p.kv_cache) + ((size_t)hkv * page_elems) * ESZ + ld_ch * 16;
-  const size_t blk_stride = (size_t)2 * p.Hkv * page_elems * ESZ, v_off = (size_t)p.Hkv * page_elems * ESZ;
+  const size_t blk_stride = (size_t)(shared_kv ? 1 : 2) * p.Hkv * page_elems * ESZ, v_off = (size_t)p.Hkv * page_elems * ESZ;
   // One block-table lookup per 16-key chunk of the tile: pages are at least 16 keys long and tiles start at multiples of 64, so
   // the 16 / kRowStep rows that a thread copies inside a chunk share a page.
   auto load_tile = [&](int tile, int buf) {
@@ -167,7 +188,7 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
           const uint32_t off = KV8 ? (uint32_t)(row * D + ld_ch * 16) : sw_off<D>(row, ld_ch);
           if (k0 + row < kv_end) {
             cp_async16(dk + off, src + (size_t)j * (kRowStep * D * ESZ));
-            cp_async16(dv + off, src + (size_t)j * (kRowStep * D * ESZ) + v_off);
+            if (!shared_kv) cp_async16(dv + off, src + (size_t)j * (kRowStep * D * ESZ) + v_off);
           } else {
             *reinterpret_cast<uint4*>(dk + off) = make_uint4(0, 0, 0, 0);
             *reinterpret_cast<uint4*>(dv + off) = make_uint4(0, 0, 0, 0);
@@ -184,7 +205,7 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
           const int blk = bt[key >> bs_shift];
           const uint8_t* src = kv_head + (size_t)blk * blk_stride + (size_t)(key & bs_mask) * D * ESZ;
           cp_async16(dk + off, src);
-          cp_async16(dv + off, src + v_off);
+          if (!shared_kv) cp_async16(dv + off, src + v_off);
         } else {
           *reinterpret_cast<uint4*>(dk + off) = make_uint4(0, 0, 0, 0);
           *reinterpret_cast<uint4*>(dv + off) = make_uint4(0, 0, 0, 0);
@@ -211,7 +232,7 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
       const uint32_t off = KV8 ? (uint32_t)((warp * 16 + rl) * D + ch * 16) : sw_off<D>(warp * 16 + rl, ch);
       if (key0 + rl < kv_end) {
         cp_async16(dk + off, src + (size_t)rl * (D * ESZ) + ch * 16);
-        cp_async16(dv + off, src + (size_t)rl * (D * ESZ) + ch * 16 + v_off);
+        if (!shared_kv) cp_async16(dv + off, src + (size_t)rl * (D * ESZ) + ch * 16 + v_off);
       } else {
         *reinterpret_cast<uint4*>(dk + off) = make_uint4(0, 0, 0, 0);
         *reinterpret_cast<uint4*>(dv + off) = make_uint4(0, 0, 0, 0);
@@ -240,8 +261,8 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
 #pragma unroll
   for (int i = 0; i < STAGES - 1; ++i) {
     if (tile_lo + i < tile_hi) {
-      if constexpr (WARP_PIPE) load_tile_w(tile_lo + i, i);
-      else load_tile(tile_lo + i, i);
+      if constexpr (WARP_PIPE) load_tile_w(tile_of(tile_lo + i), i);
+      else load_tile(tile_of(tile_lo + i), i);
     }
     cp_async_commit();
   }
@@ -263,10 +284,10 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
     cp_async_wait<STAGES - 2>();  // the group of this tile has landed (one group is committed per iteration)
     if constexpr (WARP_PIPE) {
       __syncwarp();                // ...for every lane of this warp, whose ldmatrix reads of the buffer refilled below are done
-      if (tile + STAGES - 1 < tile_hi) load_tile_w(tile + STAGES - 1, (tile - tile_lo + STAGES - 1) % STAGES);
+      if (tile + STAGES - 1 < tile_hi) load_tile_w(tile_of(tile + STAGES - 1), (tile - tile_lo + STAGES - 1) % STAGES);
     } else {
       __syncthreads();             // ...for every thread, and everybody has finished the buffer refilled below
-      if (tile + STAGES - 1 < tile_hi) load_tile(tile + STAGES - 1, (tile - tile_lo + STAGES - 1) % STAGES);
+      if (tile + STAGES - 1 < tile_hi) load_tile(tile_of(tile + STAGES - 1), (tile - tile_lo + STAGES - 1) % STAGES);
     }
     cp_async_commit();
     if (KV8) {
@@ -305,7 +326,7 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
     const uint32_t kb = smem_u32(KV8 ? sKb : sK + (size_t)buf * kKeysPerTile * D * 2);
     const uint32_t vb = smem_u32(KV8 ? sVb : sV + (size_t)buf * kKeysPerTile * D * 2);
     const uint32_t qb = smem_u32(sQ);
-    const int k0 = tile * kKeysPerTile + key_base;
+    const int k0 = tile_of(tile) * kKeysPerTile + key_base;
 
     // ---- S = Q K^T
     float s[MBW][NB2 * 2][4];
@@ -335,12 +356,27 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
     }
     // ---- mask, online softmax
     float alpha_r[MBW][2];
+    // whole tiles of this warp that need neither masking nor a per-key bias
+    bool no_mask = false, far_bias = false;
+    if constexpr (EXT) {
+      const int q_lo = ctx0 + tq0 + row_base / G, q_hi = ctx0 + tq0 + (row_base + 16 * MBW - 1) / G, k_hi = k0 + NB2 * 16 - 1;
+      no_mask = k_hi <= q_lo && k_hi < kv_end && (k0 + wlo > q_hi || k_hi < p.keep);
+      far_bias = p.bias != nullptr && q_lo - k_hi >= p.bias_len - 1;
+    }
 #pragma unroll
     for (int b = 0; b < MBW; ++b) {
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
         const int row = row_base + b * 16 + g_ + h * 8;
         const int qpos = ctx0 + tq0 + row / G;  // rows past nrows are never stored
+        const float* bias_row = nullptr;
+        float bias_far = 0.f;
+        if constexpr (EXT) {
+          if (p.bias != nullptr) {
+            bias_row = p.bias + (size_t)(hkv * G + row % G) * p.bias_len;
+            bias_far = __ldg(bias_row + p.bias_len - 1);
+          }
+        }
         float mx = -INFINITY;
 #pragma unroll
         for (int n = 0; n < NB2 * 2; ++n) {
@@ -349,7 +385,12 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
             int key = k0 + n * 8 + tg * 2 + e;
             float v = s[b][n][h * 2 + e] * sc;
             if (capped) v = tanhf(v) * sc_post;
-            v = (key <= qpos && key < kv_end && key + wlo > qpos) ? v : -INFINITY;
+            if constexpr (EXT) {
+              if (p.bias != nullptr) v = fmaf(far_bias ? bias_far : __ldg(bias_row + min(max(qpos - key, 0), p.bias_len - 1)), kLog2e, v);
+              if (!no_mask) v = (key <= qpos && key < kv_end && (key + wlo > qpos || key < p.keep)) ? v : -INFINITY;
+            } else {
+              v = (key <= qpos && key < kv_end && key + wlo > qpos) ? v : -INFINITY;
+            }
             s[b][n][h * 2 + e] = v;
             mx = fmaxf(mx, v);
           }
@@ -400,6 +441,20 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
         a[b][2] = pack_bf16(s[b][n2 * 2 + 1][0], s[b][n2 * 2 + 1][1]);
         a[b][3] = pack_bf16(s[b][n2 * 2 + 1][2], s[b][n2 * 2 + 1][3]);
       }
+      uint32_t lo[MBW][4];   // what rounding took from the weights, as a second bf16 term
+      if constexpr (EXT) {
+        auto rest = [](uint32_t hi, float x, float y) {
+          const float2 f = __bfloat1622float2(*reinterpret_cast<__nv_bfloat162*>(&hi));
+          return pack_bf16(x - f.x, y - f.y);
+        };
+#pragma unroll
+        for (int b = 0; b < MBW; ++b) {
+          lo[b][0] = rest(a[b][0], s[b][n2 * 2][0], s[b][n2 * 2][1]);
+          lo[b][1] = rest(a[b][1], s[b][n2 * 2][2], s[b][n2 * 2][3]);
+          lo[b][2] = rest(a[b][2], s[b][n2 * 2 + 1][0], s[b][n2 * 2 + 1][1]);
+          lo[b][3] = rest(a[b][3], s[b][n2 * 2 + 1][2], s[b][n2 * 2 + 1][3]);
+        }
+      }
 #pragma unroll
       for (int d2 = 0; d2 < D / 16; ++d2) {
         uint32_t bfr[4];
@@ -409,6 +464,10 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
         for (int b = 0; b < MBW; ++b) {
           mma_bf16(o[b][d2 * 2], a[b], bfr[0], bfr[1]);
           mma_bf16(o[b][d2 * 2 + 1], a[b], bfr[2], bfr[3]);
+          if constexpr (EXT) {
+            mma_bf16(o[b][d2 * 2], lo[b], bfr[0], bfr[1]);
+            mma_bf16(o[b][d2 * 2 + 1], lo[b], bfr[2], bfr[3]);
+          }
         }
       }
     }
@@ -422,7 +481,8 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
       if (row >= nrows) continue;
       const int tok = tq0 + row / G, gh = row % G;
       const float den = lrow[0][h] + (p.sinks != nullptr ? exp2f(p.sinks[hkv * G + gh] * 1.4426950408889634f - mrow[0][h]) : 0.f);
-      const float inv = den > 0.f ? (KV8 ? p.v_scale : 1.f) / den : 0.f;
+      float inv = den > 0.f ? (KV8 ? p.v_scale : 1.f) / den : 0.f;
+      if constexpr (EXT) inv *= head_gate(p, (size_t)(qs + tok), hkv * G + gh);
       __nv_bfloat16* dst = p.out + ((size_t)(qs + tok) * p.Hq + hkv * G + gh) * D;
 #pragma unroll
       for (int i = 0; i < D / 8; ++i)
@@ -480,7 +540,8 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
       }
     } else {
       const float den = L + (p.sinks != nullptr ? exp2f(p.sinks[hkv * G + gh] * 1.4426950408889634f - M) : 0.f);
-      const float inv = den > 0.f ? (KV8 ? p.v_scale : 1.f) / den : 0.f;
+      float inv = den > 0.f ? (KV8 ? p.v_scale : 1.f) / den : 0.f;
+      if constexpr (EXT) inv *= head_gate(p, (size_t)(qs + tok), hkv * G + gh);
       __nv_bfloat16* dst = p.out + orow * D + c4;
       *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16(acc[0] * inv, acc[1] * inv), pack_bf16(acc[2] * inv, acc[3] * inv));
       if (p.lse != nullptr && c4 == 0) p.lse[orow] = (M + log2f(L)) * 0.6931471805599453f;
@@ -511,25 +572,30 @@ __global__ void attn_combine_kernel(const AttnParams p) {
     for (int i = 0; i < D / 32; ++i) acc[i] += src[lane + 32 * i] * f;
   }
   const float den = L + (p.sinks != nullptr ? exp2f(p.sinks[warp % p.Hq] * 1.4426950408889634f - M) : 0.f);
-  const float inv = den > 0.f ? (p.kv_fp8 ? p.v_scale : 1.f) / den : 0.f;
+  const float inv = (den > 0.f ? (p.kv_fp8 ? p.v_scale : 1.f) / den : 0.f) * head_gate(p, (size_t)(warp / p.Hq), warp % p.Hq);
 #pragma unroll
   for (int i = 0; i < D / 32; ++i) p.out[(size_t)warp * D + lane + 32 * i] = __float2bfloat16(acc[i] * inv);
   if (p.lse != nullptr && lane == 0) p.lse[warp] = (M + log2f(L)) * 0.6931471805599453f;
 }
 
-template <int D, int MODE, int MB, bool KV8, int ST = 3>
+template <int D, int MODE, int MB, bool KV8, int ST = 3, bool EXT = false>
 int launch_one(const AttnParams& p, cudaStream_t st) {
   constexpr int ROWS = (MODE == 0) ? 64 : 16 * MB;
-  const int smem = ROWS * D * 2 + (KV8 ? 2 * ST * kKeysPerTile * D + 2 * kKeysPerTile * D * 2 : 2 * ST * kKeysPerTile * D * 2);
+  const int smem_max = ROWS * D * 2 + (KV8 ? 2 * ST * kKeysPerTile * D + 2 * kKeysPerTile * D * 2 : 2 * ST * kKeysPerTile * D * 2);
+  int smem = smem_max;
+  if (EXT && p.kv_shared) {  // one ring; the decode kernel's merge of its warps' fp32 partials lies over it
+    const int ring = ST * kKeysPerTile * D * 2, merge = (MODE == 1) ? 4 * ROWS * D * 4 : 0;
+    smem = ROWS * D * 2 + (ring > merge ? ring : merge);
+  }
   static int configured_dev[kMaxDevices] = {};
   int& configured = configured_dev[current_device_slot()];  // the limit is an attribute of (kernel, device)
   if (!configured) {
-    if (cudaFuncSetAttribute(attn_kernel<D, MODE, MB, KV8, ST>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -4;
+    if (cudaFuncSetAttribute(attn_kernel<D, MODE, MB, KV8, ST, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_max) != cudaSuccess) return -4;
     configured = 1;
   }
   dim3 grid(MODE == 0 ? p.num_q_tiles : p.R, p.Hkv, MODE == 0 ? 1 : p.splits);
   if (grid.x == 0) return 0;
-  launch_k(attn_kernel<D, MODE, MB, KV8, ST>, grid, dim3(128), (size_t)smem, st, true, p);
+  launch_k(attn_kernel<D, MODE, MB, KV8, ST, EXT>, grid, dim3(128), (size_t)smem, st, true, p);
   if (MODE == 1 && p.splits > 1) {
     int rows = p.T * p.Hq;
     launch_k(attn_combine_kernel<D>, dim3((rows * 32 + 255) / 256), dim3(256), 0, st, true, p);
@@ -544,6 +610,24 @@ int attention_launch(const AttnParams& p, int mode, cudaStream_t st) {
   const int G = p.Hq / p.Hkv;
   if (G > 64) return -1;
   const bool f8 = p.kv_fp8 != 0;
+  if (p.keep > 0 || p.kv_shared || p.bias != nullptr || p.gate != nullptr) {
+    if (f8 || (p.bias != nullptr && p.bias_len < 1)) return -7;
+    const int rows = p.short_q_len * G;
+    if (mode == 1) {
+      if (p.D == 64) {
+        if (rows <= 16) return launch_one<64, 1, 1, false, 3, true>(p, st);
+        if (rows <= 32) return launch_one<64, 1, 2, false, 3, true>(p, st);
+      } else if (p.D == 128) {
+        if (rows <= 16) return launch_one<128, 1, 1, false, 3, true>(p, st);
+        if (rows <= 32) return launch_one<128, 1, 2, false, 3, true>(p, st);
+      } else if (rows <= 16) {
+        return launch_one<256, 1, 1, false, 3, true>(p, st);
+      }
+      return -6;
+    }
+    return p.D == 64 ? launch_one<64, 0, 1, false, 3, true>(p, st) : p.D == 128 ? launch_one<128, 0, 1, false, 3, true>(p, st)
+                                                                               : launch_one<256, 0, 1, false, 3, true>(p, st);
+  }
   if (mode == 1) {
     const int rows = p.short_q_len * G;
     if (p.D == 64) {

@@ -29,7 +29,13 @@ void gemm(torch::Tensor x, c10::optional<torch::Tensor> w, c10::optional<torch::
           int64_t n_out, int64_t n_pad, int64_t epi, int64_t group_ktiles, int64_t force_splits, int64_t force_tn,
           std::vector<int64_t> push_dst, int64_t push_rows, int64_t wkind, int64_t trace_ptr, int64_t push_sel, int64_t push_sel_stride) {
   check_bf16(x, "x");
-  check_bf16(out, "out");
+  const bool f32_out = out.scalar_type() == torch::kFloat32;
+  if (f32_out) {
+    TORCH_CHECK(out.is_cuda() && w.has_value() && epi == oc::EPI_STORE && push_dst.empty(), "fp32 output is for the plain store of bf16 weights");
+  } else {
+    check_bf16(out, "out");
+  }
+  TORCH_CHECK(epi != oc::EPI_GELU_TANH || w.has_value(), "the GELU epilogue is for bf16 weights");
   TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && out.dim() == 2 && out.stride(1) == 1, "x/out must be row-major 2-D");
   const c10::cuda::CUDAGuard guard(x.device());
   oc::GemmParams p{};
@@ -44,7 +50,8 @@ void gemm(torch::Tensor x, c10::optional<torch::Tensor> w, c10::optional<torch::
   p.n_pad = (int)n_pad;
   p.epi = (int)epi;
   p.group_ktiles = (int)group_ktiles;
-  p.out = (__nv_bfloat16*)out.data_ptr();
+  p.out = f32_out ? nullptr : (__nv_bfloat16*)out.data_ptr();
+  p.out_f32 = f32_out ? out.data_ptr<float>() : nullptr;
   p.ldo = (int)out.stride(0);
   TORCH_CHECK(out.size(0) >= p.T && out.size(1) >= (epi == oc::EPI_SILU_MUL ? n_out : N), "out is too small");
   p.bias = bias.has_value() ? (const __nv_bfloat16*)bias->data_ptr() : nullptr;
@@ -207,14 +214,23 @@ void rope_and_cache(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Te
 void paged_attention(torch::Tensor q, torch::Tensor kv_cache, torch::Tensor out, c10::optional<torch::Tensor> lse, torch::Tensor qsl,
                      torch::Tensor seq_lens, torch::Tensor block_table, double scale, int64_t mode, int64_t num_q_tiles, int64_t splits,
                      int64_t max_q_len, int64_t short_q_len, c10::optional<torch::Tensor> ws_o, c10::optional<torch::Tensor> ws_ml,
-                     int64_t window, double softcap, c10::optional<torch::Tensor> sinks, double k_scale, double v_scale) {
-  check_bf16(q, "q");
-  TORCH_CHECK(kv_cache.is_cuda() && (kv_cache.scalar_type() == torch::kBFloat16 || kv_cache.scalar_type() == torch::kFloat8_e4m3fn),
-              "kv_cache must be a bf16 or float8_e4m3fn CUDA tensor");
-  check_bf16(out, "out");
+                     int64_t window, double softcap, c10::optional<torch::Tensor> sinks, double k_scale, double v_scale, int64_t keep,
+                     c10::optional<torch::Tensor> bias, c10::optional<torch::Tensor> gate) {
+  // mode 3: everything fp32 (attention_f32.cu)
+  if (mode == 3) {
+    TORCH_CHECK(q.is_cuda() && q.scalar_type() == torch::kFloat32 && kv_cache.scalar_type() == torch::kFloat32 && out.scalar_type() == torch::kFloat32,
+                "q, kv_cache and out must be fp32 CUDA tensors");
+  } else {
+    check_bf16(q, "q");
+    TORCH_CHECK(kv_cache.is_cuda() && (kv_cache.scalar_type() == torch::kBFloat16 || kv_cache.scalar_type() == torch::kFloat8_e4m3fn),
+                "kv_cache must be a bf16 or float8_e4m3fn CUDA tensor");
+    check_bf16(out, "out");
+    TORCH_CHECK(((uintptr_t)q.data_ptr() & 15) == 0 && (q.stride(0) % 8) == 0 && (q.stride(1) % 8) == 0, "q must be 16-byte aligned");
+  }
   TORCH_CHECK(q.dim() == 3 && q.stride(2) == 1 && out.is_contiguous(), "q must be [T,Hq,D]; out contiguous");
-  TORCH_CHECK(((uintptr_t)q.data_ptr() & 15) == 0 && (q.stride(0) % 8) == 0 && (q.stride(1) % 8) == 0, "q must be 16-byte aligned");
-  TORCH_CHECK(kv_cache.is_contiguous() && kv_cache.dim() == 5 && kv_cache.size(1) == 2, "kv_cache must be contiguous [blocks,2,Hkv,bs,D]");
+  TORCH_CHECK(kv_cache.is_contiguous() && kv_cache.dim() == 5 && (kv_cache.size(1) == 2 || kv_cache.size(1) == 1) && kv_cache.size(4) == q.size(2),
+              "kv_cache must be contiguous [blocks,2 (or 1: the values are the keys),Hkv,bs,D]");
+  TORCH_CHECK(q.size(0) == out.size(0) && q.size(1) == out.size(1) && q.size(2) == out.size(2) && q.size(1) % kv_cache.size(2) == 0, "q / out / cache heads do not match");
   TORCH_CHECK(qsl.scalar_type() == torch::kInt32 && seq_lens.scalar_type() == torch::kInt32 && block_table.scalar_type() == torch::kInt32,
               "metadata must be int32");
   const c10::cuda::CUDAGuard guard(q.device());
@@ -253,7 +269,23 @@ void paged_attention(torch::Tensor q, torch::Tensor kv_cache, torch::Tensor out,
                 "sinks must be a contiguous fp32 CUDA tensor with one entry per query head");
     p.sinks = sinks->data_ptr<float>();
   }
-  TORCH_CHECK(mode != 2 || (window == 0 && softcap == 0.0 && !sinks.has_value()), "window / softcap / sinks run on the mma.sync kernels");
+  p.keep = (int)keep;
+  p.kv_shared = kv_cache.size(1) == 1;
+  if (bias.has_value()) {
+    TORCH_CHECK(bias->is_cuda() && bias->scalar_type() == torch::kFloat32 && bias->is_contiguous() && bias->dim() == 2 && bias->size(0) == q.size(1) &&
+                bias->size(1) >= 1, "the bias table must be a contiguous fp32 CUDA [Hq, distances] matrix");
+    p.bias = bias->data_ptr<float>();
+    p.bias_len = (int)bias->size(1);
+  }
+  if (gate.has_value()) {
+    TORCH_CHECK(gate->is_cuda() && gate->scalar_type() == q.scalar_type() && gate->dim() == 2 && gate->size(0) == q.size(0) && gate->size(1) == q.size(1) &&
+                gate->stride(1) == 1, "the gate must be [T, Hq] of q's type with unit inner stride");
+    p.gate = gate->data_ptr();
+    p.gate_st = gate->stride(0);
+  }
+  const bool extended = keep > 0 || p.kv_shared || p.bias != nullptr || p.gate != nullptr;
+  TORCH_CHECK(mode != 2 || (window == 0 && softcap == 0.0 && !sinks.has_value() && !extended), "window / softcap / sinks and the like run on the mma.sync kernels");
+  TORCH_CHECK(!(extended && p.kv_fp8), "an fp8 KV cache has no distance bias, kept tokens, output gate or shared keys and values");
   if (mode == 1 && splits > 1) {
     TORCH_CHECK(ws_o.has_value() && ws_ml.has_value(), "split-KV needs workspaces");
     TORCH_CHECK((size_t)ws_o->numel() >= (size_t)splits * p.T * p.Hq * p.D && (size_t)ws_ml->numel() >= (size_t)splits * p.T * p.Hq * 2,
@@ -262,9 +294,89 @@ void paged_attention(torch::Tensor q, torch::Tensor kv_cache, torch::Tensor out,
     p.ws_ml = ws_ml->data_ptr<float>();
   }
   if (p.T == 0 || p.R == 0) return;
-  // mode 0: mma.sync prefill, 1: decode / short verify queries, 2: tcgen05 prefill (D = 128, query tiles of 128 tokens)
-  int rc = mode == 2 ? oc::attention_prefill_tc_launch(p, kv_cache.size(0), cur_stream()) : oc::attention_launch(p, (int)mode, cur_stream());
+  // mode 0: mma.sync prefill, 1: decode / short verify queries, 2: tcgen05 prefill (D = 128, query tiles of 128 tokens), 3: fp32
+  int rc = mode == 3 ? oc::attention_f32_launch(p, cur_stream()) : mode == 2 ? oc::attention_prefill_tc_launch(p, kv_cache.size(0), cur_stream()) : oc::attention_launch(p, (int)mode, cur_stream());
   TORCH_CHECK(rc == 0, "attention launch failed with code ", rc);
+}
+
+// Key (and value) rows [T, H, D] into pages [blocks, 1 or 2, H, block_size, D] of the same element type.
+void kv_insert(torch::Tensor k, c10::optional<torch::Tensor> v, torch::Tensor cache, torch::Tensor slot_mapping) {
+  TORCH_CHECK(k.is_cuda() && cache.is_cuda() && k.scalar_type() == cache.scalar_type() && cache.is_contiguous() && cache.dim() == 5, "k and the cache must be CUDA tensors of one type");
+  auto rows = [&](const torch::Tensor& t) {
+    TORCH_CHECK(t.dim() == 3 && t.size(1) == cache.size(2) && t.size(2) == cache.size(4) && t.stride(2) == 1 && (t.size(1) == 1 || t.stride(1) == t.size(2)),
+                "rows must be [T, H, D] with heads D apart");
+  };
+  rows(k);
+  TORCH_CHECK(cache.size(1) == (v.has_value() ? 2 : 1), "the cache must hold one tensor per page, or two with values");
+  TORCH_CHECK(slot_mapping.scalar_type() == torch::kInt32 && slot_mapping.is_contiguous() && slot_mapping.numel() >= k.size(0), "slot_mapping must be int32 [T]");
+  const c10::cuda::CUDAGuard guard(k.device());
+  const int64_t es = k.element_size();
+  oc::KvInsertParams p{};
+  p.k = (const char*)k.data_ptr();
+  p.k_st = k.stride(0) * es;
+  if (v.has_value()) {
+    rows(*v);
+    TORCH_CHECK(v->scalar_type() == k.scalar_type() && v->size(0) == k.size(0), "v must match k");
+    p.v = (const char*)v->data_ptr();
+    p.v_st = v->stride(0) * es;
+  }
+  p.cache = (char*)cache.data_ptr();
+  p.slot_mapping = slot_mapping.data_ptr<int>();
+  p.T = (int)k.size(0); p.H = (int)k.size(1); p.row_bytes = (int)(k.size(2) * es); p.bs = (int)cache.size(3);
+  TORCH_CHECK(oc::kv_insert_launch(p, cur_stream()) == 0, "kv_insert failed");
+}
+
+// See StreamJoinParams. Norms come as (kind, weight, bias, eps, weight stored minus one).
+void stream_join(torch::Tensor part, c10::optional<torch::Tensor> x_in, torch::Tensor x_out, int64_t post_kind, c10::optional<torch::Tensor> post_w,
+                 c10::optional<torch::Tensor> post_b, double post_eps, bool post_plus, c10::optional<torch::Tensor> scale, int64_t next_kind,
+                 c10::optional<torch::Tensor> next_w, c10::optional<torch::Tensor> next_b, double next_eps, bool next_plus, c10::optional<torch::Tensor> y,
+                 c10::optional<torch::Tensor> add, c10::optional<torch::Tensor> copy_out, bool f32) {
+  const auto et = f32 ? torch::kFloat32 : torch::kBFloat16;
+  TORCH_CHECK(part.is_cuda() && part.dim() == 2 && part.stride(1) == 1, "part must be a CUDA [T, H] matrix with unit inner stride");
+  TORCH_CHECK(part.scalar_type() == torch::kFloat32 || part.scalar_type() == et, "part must be fp32 or of the model's type");
+  const int64_t T = part.size(0), H = part.size(1);
+  const c10::cuda::CUDAGuard guard(part.device());
+  auto vec = [&](const c10::optional<torch::Tensor>& t, const char* name) -> const void* {
+    if (!t.has_value()) return nullptr;
+    TORCH_CHECK(t->is_cuda() && t->scalar_type() == et && t->is_contiguous() && t->numel() == H, name, " must be a contiguous [H] vector of the model's type");
+    return t->data_ptr();
+  };
+  auto mat = [&](const torch::Tensor& t, c10::ScalarType ty, const char* name) {
+    TORCH_CHECK(t.is_cuda() && t.scalar_type() == ty && t.dim() == 2 && t.size(0) == T && t.size(1) == H && t.is_contiguous(), name, " must be contiguous [T, H]");
+  };
+  oc::StreamJoinParams p{};
+  p.part = part.data_ptr();
+  p.ld_part = part.stride(0);
+  p.part_f32 = part.scalar_type() == torch::kFloat32;
+  mat(x_out, torch::kFloat32, "x_out");
+  p.x_out = x_out.data_ptr<float>();
+  if (x_in.has_value()) {
+    mat(*x_in, torch::kFloat32, "x_in");
+    p.x_in = x_in->data_ptr<float>();
+  }
+  p.post = {(int)post_kind, post_plus ? 1 : 0, vec(post_w, "post weight"), vec(post_b, "post bias"), (float)post_eps};
+  p.next = {(int)next_kind, next_plus ? 1 : 0, vec(next_w, "next weight"), vec(next_b, "next bias"), (float)next_eps};
+  p.scale = vec(scale, "scale");
+  p.add = vec(add, "add");
+  if (y.has_value()) {
+    mat(*y, et, "y");
+    p.y = y->data_ptr();
+  }
+  if (copy_out.has_value()) {
+    TORCH_CHECK(copy_out->is_cuda() && copy_out->scalar_type() == et && copy_out->dim() == 2 && copy_out->size(0) == T && copy_out->size(1) == H && copy_out->stride(1) == 1,
+                "copy_out must be [T, H] of the model's type with unit inner stride");
+    p.copy_out = copy_out->data_ptr();
+    p.ld_copy = copy_out->stride(0);
+  }
+  p.T = (int)T; p.H = (int)H; p.f32 = f32 ? 1 : 0;
+  const int rc = oc::stream_join_launch(p, cur_stream());
+  TORCH_CHECK(rc == 0, "stream_join failed: ", rc, " (widths up to 8192)");
+}
+
+void gelu_tanh_f32(torch::Tensor x) {
+  TORCH_CHECK(x.is_cuda() && x.scalar_type() == torch::kFloat32 && x.is_contiguous(), "x must be a contiguous fp32 CUDA tensor");
+  const c10::cuda::CUDAGuard guard(x.device());
+  TORCH_CHECK(oc::gelu_tanh_f32_launch(x.data_ptr<float>(), x.numel(), cur_stream()) == 0, "gelu_tanh_f32 failed");
 }
 
 // LSE-weighted merge of two partial attention results [T, H, D] bf16 with fp32 [T, H] log-sum-exps; returns (merged, merged lse)
@@ -740,7 +852,13 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("rms_norm_gated", &rms_norm_gated);
   m.def("silu_and_mul", &silu_and_mul);
   m.def("rope_and_cache", &rope_and_cache);
-  m.def("paged_attention", &paged_attention);
+  m.def("paged_attention", &paged_attention, py::arg("q"), py::arg("kv_cache"), py::arg("out"), py::arg("lse"), py::arg("qsl"), py::arg("seq_lens"),
+        py::arg("block_table"), py::arg("scale"), py::arg("mode"), py::arg("num_q_tiles"), py::arg("splits"), py::arg("max_q_len"), py::arg("short_q_len"),
+        py::arg("ws_o"), py::arg("ws_ml"), py::arg("window"), py::arg("softcap"), py::arg("sinks"), py::arg("k_scale"), py::arg("v_scale"),
+        py::arg("keep") = 0, py::arg("bias") = py::none(), py::arg("gate") = py::none());
+  m.def("kv_insert", &kv_insert);
+  m.def("stream_join", &stream_join);
+  m.def("gelu_tanh_f32", &gelu_tanh_f32);
   m.def("argmax", &argmax);
   m.def("merge_attn_states", &merge_attn_states);
   m.def("read_status", &read_status);

@@ -274,6 +274,27 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ 
 #pragma unroll
       for (int j = 0; j < 32; ++j) a[j] += bias_v;
     }
+    if constexpr (WKIND == 0) {
+      if (p.epi == EPI_GELU_TANH) {
+#pragma unroll
+        for (int j = 0; j < 32; ++j) {  // 0.5 z (1 + tanh(u)) = z / (1 + e^-2u), u = sqrt(2/pi) (z + 0.044715 z^3)
+          const float z = a[j], u2 = 1.5957691216057308f * (z + 0.044715f * z * z * z);
+          a[j] = z / (1.f + __expf(-u2));
+        }
+      }
+      if (p.out_f32 != nullptr) {
+        // a warp holds 32 neighbouring features of a token: its fp32 stores are whole 128-byte segments as they are
+        const int n = n_base + row;
+        if (n < p.N) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) {
+            const int t = t0 + tok0 + (j >> 2) * tok_gstride + (j & 3);
+            if (j < rows && t < t_end) p.out_f32[(size_t)t * p.ldo + n] = a[j];
+          }
+        }
+        return;
+      }
+    }
     // feature pair (f, f + 1) of staged token j goes to the even lane, of token j + 1 to the odd lane
     const uint32_t col_b = silu ? (uint32_t)(q * 16 + (lane & 14)) * 2u : (uint32_t)(q * 32 + (lane & 30)) * 2u;
 #pragma unroll

@@ -6,7 +6,7 @@
 
 namespace oc {
 
-enum { EPI_STORE = 0, EPI_SILU_MUL = 1 };
+enum { EPI_STORE = 0, EPI_SILU_MUL = 1, EPI_GELU_TANH = 2 };
 
 struct GemmParams {
   int T, N, K;        // tokens, logical output features, reduction length (multiple of 64)
@@ -24,6 +24,7 @@ struct GemmParams {
   int epi;
   int group_ktiles;   // 64-wide k tiles per quantisation group (group 128 -> 2)
   __nv_bfloat16* out;
+  float* out_f32;     // bf16 weights, plain store: when set, the fp32 accumulators go here (row pitch ldo) instead of to `out`
   int ldo;
   const __nv_bfloat16* bias;
   // Tensor-parallel push (row-parallel layers): when n_push > 0 the epilogue stores each output row into peer GPUs' slabs instead

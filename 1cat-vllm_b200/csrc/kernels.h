@@ -30,6 +30,39 @@ int rms_norm_gated_launch(const void* x, const void* z, const void* w, void* y, 
                           float eps, cudaStream_t st);
 int silu_and_mul_launch(const void* x, void* y, int T, int I, cudaStream_t st);
 int rope_cache_launch(const RopeCacheParams& p, cudaStream_t st);
+// k (and v) rows [T][H][D] into pages [blocks][tensors][H][bs][D]; strides and widths in bytes
+struct KvInsertParams {
+  const char *k, *v;            // v null: one cached tensor per page
+  char* cache;
+  const int* slot_mapping;      // negative: skip
+  long long k_st, v_st;         // bytes between tokens (heads are row_bytes apart)
+  int T, H, row_bytes, bs;
+};
+int kv_insert_launch(const KvInsertParams& p, cudaStream_t st);
+
+// fp32 residual stream: x' = x + scale * post(part) (+ add); y = next(x'). Norm kinds: 0 none, 1 RMS, 2 mean-and-variance.
+struct StreamNorm {
+  int kind, plus_one;
+  const void *w, *b;            // null: ones / zeros
+  float eps;
+};
+struct StreamJoinParams {
+  const void* part;             // [T][H], pitch ld_part
+  long long ld_part;
+  int part_f32;                 // part is fp32 (else the model's element type)
+  const float* x_in;            // [T][H] or null: the stream starts from part
+  float* x_out;                 // [T][H], may be x_in
+  StreamNorm post, next;
+  const void *scale, *add;      // [H] or null
+  void* y;                      // [T][H] in the model's element type, or null (next.kind 0)
+  void* copy_out;               // x' in the model's element type, pitch ld_copy, or null
+  long long ld_copy;
+  int T, H;
+  int f32;                      // the model's element type (part, weights, y, copy_out): 1 fp32, 0 bf16
+};
+int stream_join_launch(const StreamJoinParams& p, cudaStream_t st);
+int gelu_tanh_f32_launch(float* x, long long n, cudaStream_t st);  // in place
+
 int argmax_launch(const void* x, int is_fp32, long long* out, unsigned long long* packed, int B, int V, long long ld, cudaStream_t st);
 int merge_attn_states_launch(const void* o1, const float* lse1, const void* o2, const float* lse2, void* out, float* lse_out, int rows, int D,
                              cudaStream_t st);
@@ -59,7 +92,17 @@ struct AttnParams {
   const float* sinks;         // [Hq] attention-sink logits or null; mma.sync kernels only
   int kv_fp8;                 // the cache holds e4m3 bytes (value / scale) instead of bf16; mma.sync kernels only
   float k_scale, v_scale;     // per-tensor scales of an fp8 cache
+  // Extended variants of the mma.sync kernels (and the fp32 kernel), taken when any of these is set; not with an fp8 cache:
+  int keep;                   // keys at positions below it stay visible outside the window
+  int kv_shared;              // the cache is [blocks][1][Hkv][bs][D]: the values are the keys
+  const float* bias;          // [Hq][bias_len] added to the scaled score by distance (the last entry for all distances past it), or null
+  int bias_len;
+  const void* gate;           // [T][Hq] (row pitch gate_st, element type of q): outputs are multiplied by its sigmoid, or null
+  long long gate_st;
 };
+// fp32 queries, cache and outputs (attention_f32.cu): q / kv_cache / out / gate point at floats, num_q_tiles counts tiles of 16
+// (token, query head of the group) rows over all requests; splits, short_q_len and the workspaces are not used.
+int attention_f32_launch(const AttnParams& p, cudaStream_t st);
 // mode 0: rows of a query tile are spread over warps (prefill / long queries); mode 1: keys are spread over warps
 // (decode and short verify queries, with split-KV + combine).
 int attention_launch(const AttnParams& p, int mode, cudaStream_t st);

@@ -1,6 +1,9 @@
 """Self-attention block: fused QKV GEMM → (per-head norm) → RoPE + paged-KV insert → paged flash attention
 → (sigmoid output gate) → o_proj (reference: models/llama.py attention; models/qwen3_next.py:505-626 for the
-gated variant with per-head q/k RMSNorm and partial rotary)."""
+gated variant with per-head q/k RMSNorm and partial rotary).
+
+Further options, each on its own: values that are the keys (one cached tensor), a learned distance bias, first tokens that stay visible
+outside the sliding window, one output gate per head applied inside the attention kernel."""
 from __future__ import annotations
 
 from typing import Optional
@@ -11,7 +14,8 @@ import torch.nn as nn
 from onecat_vllm import ops
 from onecat_vllm.config import ModelConfig
 from onecat_vllm.layers.common import get_rope
-from onecat_vllm.layers.linear import QKVParallelLinear, RowParallelLinear
+from onecat_vllm.layers.linear import QKGParallelLinear, QKVParallelLinear, RowParallelLinear
+from onecat_vllm.ops import ref
 from onecat_vllm.parallel.state import get_state
 
 
@@ -21,11 +25,28 @@ class Attention(nn.Module):
         tp = get_state().tp_size
         self.D = cfg.head_dim
         self.gated = cfg.attn_output_gate
+        self.kv_shared, self.head_gate = cfg.attn_kv_shared, cfg.attn_head_gate
+        if (self.kv_shared or self.head_gate) and (cfg.num_attention_heads % tp or (cfg.num_key_value_heads % tp and tp % cfg.num_key_value_heads)):
+            raise ValueError(f"tensor_parallel_size={tp} does not divide the heads of layer {layer_idx}")
         # qkv_in: width of the projection's input when it is not the hidden size (EAGLE-3 feeds [embedding ; hidden])
-        self.qkv_proj = QKVParallelLinear(qkv_in or cfg.hidden_size, cfg.head_dim, cfg.num_attention_heads, cfg.num_key_value_heads,
-                                          q_mult=2 if self.gated else 1, bias=cfg.attention_bias, quant=cfg.quant,
-                                          prefix=prefix + ".qkv_proj", dtype=cfg.dtype)
-        self.Hq, self.Hkv = self.qkv_proj.num_heads, self.qkv_proj.num_kv_heads
+        if self.kv_shared:
+            if self.gated or cfg.qk_norm or cfg.qk_norm_full or layer_idx not in cfg.nope_layers:
+                raise ValueError("attention whose values are its keys is served without rotary embedding, q / k norms and the elementwise gate")
+            self.qkg_proj = QKGParallelLinear(qkv_in or cfg.hidden_size, cfg.head_dim, cfg.num_attention_heads, cfg.num_key_value_heads,
+                                              head_gate=self.head_gate, bias=cfg.attention_bias, quant=cfg.quant, prefix=prefix + ".qkg_proj",
+                                              dtype=cfg.dtype)
+            self.Hq, self.Hkv = self.qkg_proj.num_heads, self.qkg_proj.num_kv_heads
+        else:
+            if self.head_gate:
+                raise ValueError("the per-head output gate is served for attention whose values are its keys")
+            self.qkv_proj = QKVParallelLinear(qkv_in or cfg.hidden_size, cfg.head_dim, cfg.num_attention_heads, cfg.num_key_value_heads,
+                                              q_mult=2 if self.gated else 1, bias=cfg.attention_bias, quant=cfg.quant,
+                                              prefix=prefix + ".qkv_proj", dtype=cfg.dtype)
+            self.Hq, self.Hkv = self.qkv_proj.num_heads, self.qkv_proj.num_kv_heads
+        self.window_keep = cfg.attn_window_keep
+        self.rel_max, self.bias_table = cfg.attn_rel_max, None
+        self.rel_bias = nn.Parameter(torch.zeros(cfg.attn_rel_buckets, self.Hq, dtype=torch.float32), requires_grad=False) \
+            if cfg.attn_rel_buckets else None
         self.o_proj = RowParallelLinear(cfg.num_attention_heads * cfg.head_dim, cfg.hidden_size, bias=cfg.attn_o_bias, quant=cfg.quant,
                                         prefix=prefix + ".o_proj", dtype=cfg.dtype)
         self.sinks = nn.Parameter(torch.zeros(self.Hq, dtype=torch.float32), requires_grad=False) if cfg.attn_sinks else None
@@ -54,13 +75,53 @@ class Attention(nn.Module):
         self.qkv_clip = cfg.qkv_clip
 
     def load_weight(self, pname: str, w: torch.Tensor, shard_id=None) -> None:
-        """Parameters that belong to the block itself: the per-head sink logits are sharded with the query heads."""
+        """Parameters that belong to the block itself: the per-head sink logits and the columns of the distance-bias table are sharded
+        with the query heads. The table takes as many rows (distance buckets) as the checkpoint has."""
         p = getattr(self, pname)
         if pname == "sinks":
             w = w.narrow(0, self._tp_rank * self.Hq, self.Hq)
+        if pname == "rel_bias":
+            w = w.narrow(1, self._tp_rank * self.Hq, self.Hq)
+            p.data = torch.empty(w.shape, dtype=p.dtype, device=p.device)
         p.data.copy_(w.reshape(p.shape))
 
+    def process_weights_after_loading(self) -> None:
+        if self.rel_bias is not None:
+            idx = torch.tensor(ref.distance_buckets(self.rel_bias.shape[0], self.rel_max), device=self.rel_bias.device)
+            self.bias_table = self.rel_bias.data[idx].t().contiguous()   # [Hq, rel_max + 1]: the bias by distance, last entry for all beyond
+        if self.kv_shared and self.qkg_proj.compute_dtype == torch.bfloat16 and self.o_proj.weight.is_cuda:
+            self._pad_heads()
+
+    def _pad_heads(self) -> None:
+        """The bf16 attention kernels exist for head sizes 64, 128 and 256: other sizes run as the next larger one, with zero rows in the
+        projections and zero columns in the output projection (scores and outputs stay the same numbers)."""
+        D, pad = self.D, next((d for d in (64, 128, 256) if d >= self.D), None)
+        if pad is None:
+            raise ValueError(f"head size {D} is not supported (at most 256)")
+        if pad == D:
+            return
+        Hq, Hkv, proj = self.Hq, self.Hkv, self.qkg_proj
+        w = proj.weight.data
+        q, k, g = w[: Hq * D], w[Hq * D: (Hq + Hkv) * D], w[(Hq + Hkv) * D:]
+        rows = lambda t: torch.nn.functional.pad(t.view(-1, D, t.shape[1]), (0, 0, 0, pad - D)).reshape(-1, t.shape[1])
+        proj.weight.data = torch.cat([rows(q), rows(k), g]).contiguous()
+        o = self.o_proj.weight.data
+        self.o_proj.weight.data = torch.nn.functional.pad(o.view(o.shape[0], Hq, D), (0, pad - D)).reshape(o.shape[0], -1).contiguous()
+        self.D = pad
+
+    def _forward_shared(self, x: torch.Tensor, md, kv_cache: torch.Tensor) -> torch.Tensor:
+        T, D, Hq, Hkv = x.shape[0], self.D, self.Hq, self.Hkv
+        qkg = self.qkg_proj(x)
+        q = qkg[:, : Hq * D].view(T, Hq, D)
+        k = qkg[:, Hq * D: (Hq + Hkv) * D].view(T, Hkv, D)
+        ops.kv_insert(k, kv_cache, md.slot_mapping)
+        o = ops.paged_attention(q, kv_cache, md, self.scale, window=self.window, softcap=self.softcap, sinks=self.sinks, keep=self.window_keep,
+                                bias_table=self.bias_table, gate=qkg[:, (Hq + Hkv) * D:] if self.head_gate else None)
+        return self.o_proj(o.reshape(T, Hq * D))
+
     def forward(self, x: torch.Tensor, md, kv_cache: torch.Tensor) -> torch.Tensor:
+        if self.kv_shared:
+            return self._forward_shared(x, md, kv_cache)
         T = x.shape[0]
         D, Hq, Hkv = self.D, self.Hq, self.Hkv
         qkv = self.qkv_proj(x)
@@ -89,7 +150,8 @@ class Attention(nn.Module):
             ops.rope_and_cache(q, k, v, md.mrope_positions if mrope else md.positions, self.rope.cos_sin, kv_cache, md.slot_mapping, self.rotary_dim,
                                self.q_norm if self.qk_norm else None, self.k_norm if self.qk_norm else None, self.eps, self.gemma,
                                mrope_section=mrope)
-        o = ops.paged_attention(q, kv_cache, md, self.scale, window=self.window, softcap=self.softcap, sinks=self.sinks)
+        o = ops.paged_attention(q, kv_cache, md, self.scale, window=self.window, softcap=self.softcap, sinks=self.sinks, keep=self.window_keep,
+                                bias_table=self.bias_table)
         if gate is not None:
             o = o * torch.sigmoid(gate.float()).to(o.dtype)
         return self.o_proj(o.reshape(T, Hq * D))

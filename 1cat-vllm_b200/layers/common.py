@@ -117,12 +117,13 @@ class VocabParallelEmbedding(nn.Module):
 class ParallelLMHead(VocabParallelEmbedding):
     """Vocab-sharded output projection; ``compute_logits`` gathers the shards."""
 
-    def compute_logits(self, hidden: torch.Tensor) -> torch.Tensor:
+    def compute_logits(self, hidden: torch.Tensor, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
         if hidden.is_cuda:
             from onecat_vllm.ops import cuda as K
-            local = K.gemm_bf16(hidden, self.weight)
+            local = K.dense(hidden, self.weight, out_dtype=out_dtype)
         else:
             local = F.linear(hidden, self.weight)
+            local = local.to(out_dtype) if out_dtype is not None else local
         full = ps.all_gather_last_dim(local)
         return full[..., : self.vocab]
 

@@ -54,7 +54,9 @@ class LinearMethod:
         y = F.linear(x, w, layer.bias if hasattr(layer, "bias") and layer.bias is not None else None)
         if layer.fuse_silu_mul:
             y = ref.silu_and_mul(y)
-        return y
+        elif layer.fuse_gelu_tanh:
+            y = F.gelu(y, approximate="tanh")
+        return y.to(layer.out_dtype) if layer.out_dtype is not None else y
 
 
 class UnquantizedMethod(LinearMethod):
@@ -268,12 +270,14 @@ class LinearBase(nn.Module):
 
     def __init__(self, in_features: int, output_sizes: list[int], parallel: str = "replicated", bias: bool = False,
                  quant: Optional[QuantConfig] = None, prefix: str = "", dtype: torch.dtype = torch.float32,
-                 fuse_silu_mul: bool = False, segment_tp: Optional[list[int]] = None) -> None:
+                 fuse_silu_mul: bool = False, segment_tp: Optional[list[int]] = None, fuse_gelu_tanh: bool = False,
+                 out_dtype: Optional[torch.dtype] = None) -> None:
         super().__init__()
         st = get_state()
         self.tp, self.tp_rank = st.tp_size, st.tp_rank
         self.parallel, self.prefix, self.compute_dtype = parallel, prefix, dtype
-        self.fuse_silu_mul = fuse_silu_mul
+        self.fuse_silu_mul, self.fuse_gelu_tanh = fuse_silu_mul, fuse_gelu_tanh
+        self.out_dtype = out_dtype  # None: the input's dtype; fp32 keeps the accumulator's precision (dense weights only)
         self.in_features_global, self.output_sizes = in_features, list(output_sizes)
         # segment_tp[i]: over how many ranks segment i is split (kv heads may be replicated)
         self.segment_tp = segment_tp or [self.tp if parallel == "column" else 1] * len(output_sizes)
@@ -363,6 +367,18 @@ class QKVParallelLinear(LinearBase):
         self.num_heads, self.num_kv_heads = num_heads // tp, max(num_kv_heads // tp, 1)
         super().__init__(hidden, [num_heads * head_dim * q_mult, num_kv_heads * head_dim, num_kv_heads * head_dim], "column",
                          segment_tp=[tp, kv_tp, kv_tp], **kw)
+
+
+class QKGParallelLinear(LinearBase):
+    """q|k|gate stacked along the output, for attention whose values are its keys: there is no value segment, and the optional third
+    segment holds one gate logit per query head."""
+
+    def __init__(self, hidden, head_dim, num_heads, num_kv_heads, head_gate: bool = False, **kw):
+        tp = get_state().tp_size
+        kv_tp = min(tp, num_kv_heads)
+        self.num_heads, self.num_kv_heads = num_heads // tp, max(num_kv_heads // tp, 1)
+        super().__init__(hidden, [num_heads * head_dim, num_kv_heads * head_dim] + ([num_heads] if head_gate else []), "column",
+                         segment_tp=[tp, kv_tp] + ([tp] if head_gate else []), **kw)
 
 
 class RowParallelLinear(LinearBase):

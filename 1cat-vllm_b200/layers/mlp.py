@@ -29,19 +29,24 @@ class MLP(nn.Module):
 
 class PlainMLP(nn.Module):
     """Feed-forward without a gate: ``down(act(up(x)))`` with ``act`` = squared ReLU (Arcee) or GELU
-    (reference: models/arcee.py ``ArceeMLP``; layers/activation.py ``ReLUSquaredActivation``). The activation is an elementwise
-    PyTorch operation between the two GEMMs."""
+    (reference: models/arcee.py ``ArceeMLP``; layers/activation.py ``ReLUSquaredActivation``). The tanh form of GELU is part of the up
+    projection's epilogue (``fuse_act=False``, for LoRA-enabled models, keeps it apart); the other activations are elementwise
+    PyTorch operations between the two GEMMs."""
 
-    def __init__(self, hidden: int, inter: int, quant, prefix: str, dtype, act: str = "relu2", bias: bool = False):
+    def __init__(self, hidden: int, inter: int, quant, prefix: str, dtype, act: str = "relu2", bias: bool = False, fuse_act: bool = True):
         super().__init__()
         self.act = act
-        self.up_proj = ColumnParallelLinear(hidden, inter, bias=bias, quant=quant, prefix=prefix + ".up_proj", dtype=dtype)
+        self.fuse_act = fuse_act and act == "gelu_tanh"
+        self.up_proj = ColumnParallelLinear(hidden, inter, bias=bias, quant=quant, prefix=prefix + ".up_proj", dtype=dtype,
+                                            fuse_gelu_tanh=self.fuse_act)
         self.down_proj = RowParallelLinear(inter, hidden, bias=bias, quant=quant, prefix=prefix + ".down_proj", dtype=dtype)
 
     def forward(self, x):
         import torch
         import torch.nn.functional as F
         h = self.up_proj(x)
+        if self.fuse_act:
+            return self.down_proj(h)
         if self.act == "relu2":
             h = torch.square(F.relu(h))
         elif self.act == "gelu_tanh":

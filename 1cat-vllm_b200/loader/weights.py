@@ -58,6 +58,28 @@ def _half_split_rows(w: torch.Tensor, head_dim: int, rotary_dim: int) -> torch.T
     return w.reshape(heads, head_dim, -1)[:, perm].reshape(w.shape)
 
 
+# Gabisun checkpoints: ``l<i>.<name>``
+_GABISUN_NAMES = {"norm1": "input_layernorm.weight", "norm1b": "post_attention_layernorm.weight", "norm2": "pre_feedforward_layernorm.weight",
+                  "norm2b": "post_feedforward_layernorm.weight", "ls1": "attn_layer_scale", "ls2": "mlp_layer_scale",
+                  "mix.q": "self_attn.q_proj.weight", "mix.k": "self_attn.k_proj.weight", "mix.g": "self_attn.g_proj.weight",
+                  "mix.o": "self_attn.o_proj.weight", "mix.rel": "self_attn.rel_bias", "mix.sink": "self_attn.sinks",
+                  "mlp.up": "mlp.up_proj.weight", "mlp.down": "mlp.down_proj.weight"}
+_GABISUN_TOP = {"embed": "model.embed_tokens.weight", "final.norm": "model.norm.weight", "final.norm.b": "model.norm.bias",
+                "loop.in": "model.loop_in.weight", "loop.step": "model.loop_step"}
+_GABISUN_RE = re.compile(r"l(\d+)\.(.+?)(\.b)?$")
+
+
+def gabisun_name(name: str) -> str:
+    """Module parameter that a Gabisun checkpoint tensor belongs to (unknown names come back unchanged)."""
+    m = _GABISUN_RE.match(name)
+    if m is None:
+        return _GABISUN_TOP.get(name, name)
+    ours = _GABISUN_NAMES.get(m.group(2))
+    if ours is None or (m.group(3) and not m.group(2).startswith("norm")):
+        return name
+    return f"model.layers.{m.group(1)}." + (ours[: -len("weight")] + "bias" if m.group(3) else ours)
+
+
 _EXPERT_RE = re.compile(r"(.*\.mlp)\.experts\.(\d+)\.(gate_proj|up_proj|down_proj)\.(weight|weight_scale_inv|weight_scale|bias)$")
 
 
@@ -72,8 +94,11 @@ def load_weights(model: nn.Module, weights: Iterable[tuple[str, torch.Tensor]]) 
     mixer_only = cfg is not None and getattr(cfg, "mixer_only_layers", False)
     vault = cfg is not None and cfg.architecture.startswith("VaultGemma")
     nemotron_h = cfg is not None and cfg.architecture.startswith("NemotronH")
+    gabisun = cfg is not None and cfg.architecture == "Gabisun"
     loaded = set()
     for name, w in weights:
+        if gabisun:
+            name = gabisun_name(name)
         if name.startswith("language_model."):
             name = name[len("language_model."):]
         elif name.startswith("model.language_model."):  # text tower of a multimodal checkpoint (Qwen3.5)
@@ -245,7 +270,7 @@ def dummy_init(model: nn.Module, seed: int = 0, std: float = 0.02) -> None:
     for name, p in model.named_parameters():
         g = gen(p.device)
         leaf = name.rsplit(".", 1)[-1]
-        if leaf in ("weight",) and name.endswith(("layernorm.weight", "norm.weight")) or leaf in ("q_norm", "k_norm", "norm_weight"):
+        if leaf in ("weight",) and name.endswith(("layernorm.weight", "norm.weight")) or leaf in ("q_norm", "k_norm", "norm_weight", "attn_layer_scale", "mlp_layer_scale"):
             continue  # keep constructor init (1, or 0 for Gemma-style)
         if p.dtype in (torch.float32, torch.float16, torch.bfloat16):
             if leaf in ("scales",):

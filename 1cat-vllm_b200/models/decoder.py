@@ -13,10 +13,12 @@ from typing import Optional
 import torch
 import torch.nn as nn
 
+from onecat_vllm import ops
 from onecat_vllm.config import ModelConfig
 from onecat_vllm.layers.attention import Attention
 from onecat_vllm.layers.common import ParallelLMHead, RMSNorm, VocabParallelEmbedding, make_norm
 from onecat_vllm.layers.gdn import GatedDeltaNet
+from onecat_vllm.layers.linear import ReplicatedLinear
 from onecat_vllm.layers.mla import MLAAttention
 from onecat_vllm.layers.mlp import MLP
 from onecat_vllm.layers.moe import SparseMoeBlock
@@ -35,6 +37,7 @@ class DecoderLayer(nn.Module):
     def __init__(self, cfg: ModelConfig, idx: int, prefix: str, device):
         super().__init__()
         from onecat_vllm.utils.plugins import layer_class
+        cfg = cfg.for_layer(idx)
         self.kind = cfg.layer_type(idx)
         if cfg.use_mla:
             self.kind = "mla"
@@ -55,16 +58,21 @@ class DecoderLayer(nn.Module):
             self.graph_safe = False          # its convolution and scan read batch geometry on the host
         else:
             self.self_attn = layer_class("Attention", Attention)(cfg, idx, prefix + ".self_attn", device)
+        if cfg.layer_scale:
+            scale = lambda: nn.Parameter(torch.ones(cfg.hidden_size, dtype=cfg.dtype), requires_grad=False)
+            self.attn_layer_scale, self.mlp_layer_scale = scale(), None if cfg.mixer_only_layers else scale()
         if cfg.mixer_only_layers:
             self.mlp = None
             self.input_layernorm = make_norm(cfg)
+            if cfg.sandwich_norm:
+                self.post_attention_layernorm = make_norm(cfg)
             return
         if cfg.is_moe_layer(idx):
             self.mlp = layer_class("SparseMoeBlock", SparseMoeBlock)(cfg, prefix + ".mlp")
         elif not cfg.mlp_gated:
             from onecat_vllm.layers.mlp import PlainMLP
             self.mlp = layer_class("PlainMLP", PlainMLP)(cfg.hidden_size, cfg.intermediate_size, cfg.quant, prefix + ".mlp", cfg.dtype, act=cfg.hidden_act,
-                                                         bias=cfg.mlp_bias)
+                                                         bias=cfg.mlp_bias, fuse_act=not cfg.enable_lora)
         else:
             self.mlp = layer_class("MLP", MLP)(cfg.hidden_size, cfg.intermediate_size, cfg.quant, prefix + ".mlp", cfg.dtype, fuse_act=not cfg.enable_lora,
                            act=cfg.hidden_act, bias=cfg.mlp_bias)
@@ -97,13 +105,29 @@ class DecoderModel(nn.Module):
         self.layers = nn.ModuleList([DecoderLayer(cfg, i, f"model.layers.{i}", device) if self.start <= i < self.end else PPMissingLayer()
                                      for i in range(cfg.num_hidden_layers)])
         self.norm = make_norm(cfg) if self.last_stage else PPMissingLayer()
+        if cfg.residual_fp32 and (self.start != 0 or not self.last_stage):
+            raise ValueError("models with an fp32 residual stream are served without pipeline parallelism")
+        if (cfg.residual_fp32 or cfg.layer_scale) and not (cfg.residual_fp32 and cfg.sandwich_norm) or cfg.loop is not None and not cfg.residual_fp32:
+            raise ValueError("the fp32 residual stream is served for blocks with norms on both sides; looped layers and layer scales need it")
+        if cfg.loop is not None:
+            # ahead of every pass of the looped layers the stream x becomes loop_in([x ; x0]) + loop_step[pass], x0 being the embeddings
+            self.loop_in = ReplicatedLinear(2 * cfg.hidden_size, cfg.hidden_size, quant=None, prefix="model.loop_in", dtype=cfg.dtype,
+                                            out_dtype=torch.float32)
+            self.loop_step = nn.Parameter(torch.zeros(cfg.loop[2], cfg.hidden_size, dtype=cfg.dtype), requires_grad=False)
         # EAGLE-3 drafting reads the residual stream at a few depths: layer indices to record, and what the last forward recorded
         self.aux_hidden_layers: tuple = ()
         self.last_aux: list = []
 
     def local_layers(self):
-        """(global index, layer) of the decoder layers this pipeline stage owns; KV caches are indexed in this order."""
+        """(global index, layer) of the decoder layers this pipeline stage owns."""
         return [(i, self.layers[i]) for i in range(self.start, self.end)]
+
+    def cache_layers(self):
+        """(name, layer) of everything on this stage that owns a cache or a state, in execution order: the layers, with one entry per
+        pass for looped ones (every pass has its own K/V). KV caches are indexed in this order."""
+        if self.cfg.loop is None:
+            return [(f"layers.{i}", layer) for i, layer in self.local_layers()]
+        return [(f"layers.{i}" if t < 0 else f"layers.{i}.{t}", self.layers[i]) for i, t in self.cfg.layer_runs()]
 
     def forward(self, input_ids: torch.Tensor, md, caches: list, inputs_embeds: Optional[torch.Tensor] = None,
                 return_prenorm: bool = False, intermediate: Optional[tuple] = None):
@@ -119,6 +143,8 @@ class DecoderModel(nn.Module):
                     h = h * torch.tensor(cfg.embed_scale, dtype=h.dtype)  # the factor is rounded to the model dtype first, as in the checkpoint's code
             else:
                 h = inputs_embeds
+            if cfg.residual_fp32:
+                return self._forward_stream(h, md, caches, return_prenorm)
             x, residual = layers[self.start].input_layernorm(h, None)
             residual = h
         else:
@@ -161,6 +187,39 @@ class DecoderModel(nn.Module):
         if return_prenorm:
             return x, residual
         return x
+
+    def _forward_stream(self, h, md, caches, return_prenorm: bool = False):
+        """fp32 residual stream: ``x += scale * post_norm(sub-block(pre_norm(x)))``. One fused kernel joins a sub-block's output to the
+        stream and produces the next sub-block's input (``ops.stream_join``). Looped layers: the join ahead of a pass also leaves the
+        stream beside the embeddings as the input of the pass's entry projection, whose fp32 output becomes the new stream."""
+        runs, loop = self.cfg.layer_runs(), self.cfg.loop
+        T, H = h.shape
+        both = None
+        if loop is not None:
+            both = torch.empty(T, 2 * H, dtype=h.dtype, device=h.device)   # [stream ; embeddings]
+            both[:, H:] = h
+
+        def join(part, x, post, scale, at):
+            """Join, then the input of run ``at`` (past the last run: the final norm)."""
+            part = reduce_only(part) if x is not None else part
+            if at < len(runs) and loop is not None and runs[at][0] == loop[0] and runs[at][1] >= 0:
+                ops.stream_join(part, x, post, scale, None, copy_out=both[:, :H])
+                return ops.stream_join(self.loop_in(both), None, None, None, self.layers[loop[0]].input_layernorm, out_dtype=h.dtype,
+                                       add=self.loop_step[runs[at][1]])
+            return ops.stream_join(part, x, post, scale, self.layers[runs[at][0]].input_layernorm if at < len(runs) else self.norm,
+                                   out_dtype=h.dtype)
+
+        y, x = join(h, None, None, None, 0)
+        for r, (i, _) in enumerate(runs):
+            layer = self.layers[i]
+            part = layer.mixer(y, md, caches[r])
+            if layer.mlp is None:
+                y, x = join(part, x, layer.post_attention_layernorm, layer.attn_layer_scale, r + 1)
+                continue
+            y, x = ops.stream_join(reduce_only(part), x, layer.post_attention_layernorm, layer.attn_layer_scale, layer.pre_feedforward_layernorm,
+                                   out_dtype=h.dtype)
+            y, x = join(layer.mlp(y), x, layer.post_feedforward_layernorm, layer.mlp_layer_scale, r + 1)
+        return (y, x) if return_prenorm else y
 
     def _forward_post_norm(self, _x, residual, md, caches):
         """OLMo-2 / OLMo-3 block order: ``h = h + norm(attn(h)); h = h + norm(mlp(h))`` with no norm in front of either sub-block
@@ -205,6 +264,7 @@ class CausalLM(nn.Module):
     # checkpoint name fragment → (our stacked parameter, shard id)
     stacked_params_mapping = [
         (".qkv_proj", ".q_proj", 0), (".qkv_proj", ".k_proj", 1), (".qkv_proj", ".v_proj", 2),
+        (".qkg_proj", ".q_proj", 0), (".qkg_proj", ".k_proj", 1), (".qkg_proj", ".g_proj", 2),
         (".gate_up_proj", ".gate_proj", 0), (".gate_up_proj", ".up_proj", 1),
         (".in_proj_qkvz", ".in_proj_q", 0), (".in_proj_qkvz", ".in_proj_k", 1), (".in_proj_qkvz", ".in_proj_v", 2),
         (".in_proj_qkvz", ".in_proj_z", 3), (".in_proj_ba", ".in_proj_b", 0), (".in_proj_ba", ".in_proj_a", 1),
@@ -254,7 +314,7 @@ class CausalLM(nn.Module):
         head = self.lm_head
         if head is None:
             e = self.model.embed_tokens
-            logits = ParallelLMHead.compute_logits(e, hidden)
+            logits = ParallelLMHead.compute_logits(e, hidden, torch.float32 if self.cfg.residual_fp32 else None)
         else:
             logits = head.compute_logits(hidden)
         c = self.cfg

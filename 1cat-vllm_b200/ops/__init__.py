@@ -46,16 +46,40 @@ def rope_and_cache(q, k, v, positions, cos_sin, kv_cache, slot_mapping, rotary_d
     return ref.rope_and_cache(q, k, v, positions, cos_sin, kv_cache, slot_mapping, rotary_dim, q_norm_w, k_norm_w, eps, gemma, mrope_section)
 
 
-def paged_attention(q, kv_cache, md, scale, out=None, window=0, softcap=0.0, sinks=None):
+def kv_insert(k, kv_cache, slot_mapping, v=None):
+    """Copy key (and value) rows into the paged cache, no rotation or norm (a cache with one tensor per page holds keys that are the values)."""
+    if k.is_cuda:
+        return ext().kv_insert(k, kv_cache, slot_mapping, v)
+    return ref.kv_insert(k, kv_cache, slot_mapping, v)
+
+
+def _norm_spec(norm):
+    """(kind, weight, bias, eps, weight stored minus one) of a norm module: kind 1 RMS, 2 layer norm."""
+    if norm is None:
+        return None
+    return 2 if getattr(norm, "plain", False) else 1, norm.weight, getattr(norm, "bias", None), norm.eps, bool(norm.gemma)
+
+
+def stream_join(part, x, post, scale, nxt, out_dtype=None, add=None, copy_out=None):
+    """Join a sub-block's output to the fp32 residual stream and normalise it for the next one, in one kernel:
+    ``x += scale * post(part) (+ add)``, ``y = nxt(x)``. ``post`` / ``nxt`` are norm modules or None. Returns (y, x); see ``ref.stream_join``."""
+    f = ext().stream_join if part.is_cuda else ref.stream_join
+    return f(part, x, _norm_spec(post), scale, _norm_spec(nxt), out_dtype, add, copy_out)
+
+
+def paged_attention(q, kv_cache, md, scale, out=None, window=0, softcap=0.0, sinks=None, keep=0, bias_table=None, gate=None):
     """``md`` is the step's AttentionMetadata. ``window``: sliding window in tokens (0 = full causal); ``softcap``: tanh soft-capping
-    of the scaled scores (0 = off); ``sinks``: fp32 ``[Hq]`` sink logits that join the softmax denominator."""
+    of the scaled scores (0 = off); ``sinks``: fp32 ``[Hq]`` sink logits that join the softmax denominator; ``keep``: first tokens visible
+    outside the window; ``bias_table``: fp32 ``[Hq, n]`` added by distance; ``gate``: ``[T, Hq]`` logits of the per-head output gate."""
     if q.is_cuda:
-        return ext().paged_attention(q, kv_cache, md, scale, out, window=window, softcap=softcap, sinks=sinks)
+        return ext().paged_attention(q, kv_cache, md, scale, out, window=window, softcap=softcap, sinks=sinks, keep=keep, bias_table=bias_table,
+                                     gate=gate)
     from onecat_vllm import envs
-    if envs.ONECAT_CPU_ATTENTION == "native" and kv_cache.dtype in (torch.float32, torch.bfloat16) and q.dtype in (torch.float32, torch.bfloat16):
+    extended = keep or bias_table is not None or gate is not None or kv_cache.shape[1] == 1   # not in the native CPU kernel
+    if envs.ONECAT_CPU_ATTENTION == "native" and not extended and kv_cache.dtype in (torch.float32, torch.bfloat16) and q.dtype in (torch.float32, torch.bfloat16):
         return cpu_paged_attention(q, kv_cache, md.block_table, md.query_start_loc, md.seq_lens, scale, out, window=window, softcap=softcap, sinks=sinks)
     return ref.paged_attention(q, kv_cache, md.block_table, md.query_start_loc, md.seq_lens, scale, out, window=window, softcap=softcap,
-                               sinks=sinks)
+                               sinks=sinks, keep=keep, bias_table=bias_table, gate=gate)
 
 
 def cpu_paged_attention(q, kv_cache, block_table, query_start_loc, seq_lens, scale, out=None, return_lse=False, window=0, softcap=0.0, sinks=None,

@@ -16,6 +16,8 @@ CSRC = os.path.join(os.path.dirname(HERE), "csrc")
 OUT = os.path.join(HERE, "_C.so")
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "--use_fast_math",
               "-Xcompiler", "-fPIC", "-Xptxas", "-v"] + (["-DONECAT_GEMM_TRACE"] if os.environ.get("ONECAT_GEMM_TRACE") else [])
+# units whose results are fp32: without the approximate division, square root and exponentials
+PRECISE = ("attention_f32.cu", "stream.cu")
 # --use_fast_math only affects __expf/exp2f-style intrinsics used in softmax/SiLU epilogues; accumulation stays fp32
 
 
@@ -45,7 +47,7 @@ def build(force: bool = False, verbose: bool = False) -> str:
         src, obj = os.path.join(CSRC, f), os.path.join(bdir, f + ".o")
         objs.append(obj)
         if force or _newer(src, obj, headers):
-            jobs.append([nvcc] + NVCC_FLAGS + ["-c", src, "-o", obj])
+            jobs.append([nvcc] + [x for x in NVCC_FLAGS if f not in PRECISE or x != "--use_fast_math"] + ["-c", src, "-o", obj])
     inc = [f"-I{p}" for p in ce.include_paths(device_type="cuda")] + [f"-I{sysconfig.get_paths()['include']}"]
     abi = int(torch._C._GLIBCXX_USE_CXX11_ABI)
     for f in cpp:
@@ -71,6 +73,18 @@ def build(force: bool = False, verbose: bool = False) -> str:
         link = ["g++", "-shared", "-o", OUT] + objs + [f"-L{d}" for d in libdirs] + [f"-Wl,-rpath,{d}" for d in libdirs] + \
                ["-lc10", "-lc10_cuda", "-ltorch_cpu", "-ltorch_cuda", "-ltorch", "-ltorch_python", "-lcudart"]
         run(link)
+    return OUT
+
+
+def ensure_built() -> str:
+    """Build the extension where it is missing or older than a source (a fresh checkout); one builder at a time."""
+    import fcntl
+    srcs = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cu", ".cpp", ".h", ".cuh"))]
+    os.makedirs(os.path.join(CSRC, "build"), exist_ok=True)
+    with open(os.path.join(CSRC, "build", ".lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        if _newer(srcs[0], OUT, srcs[1:]):
+            build()
     return OUT
 
 

@@ -18,7 +18,7 @@ except ImportError as e:  # pragma: no cover
     raise ImportError("the CUDA extension onecat_vllm.ops._C is not built; run `python -c 'import __graft_entry__ as g; g.build()'` "
                       f"or `python 1cat-vllm_b200/ops/build.py` ({e})") from e
 
-EPI_STORE, EPI_SILU_MUL = 0, 1
+EPI_STORE, EPI_SILU_MUL, EPI_GELU_TANH = 0, 1, 2
 TORCH_STANDINS: set = set()  # names of ops that ran as device-side PyTorch code in this process
 _LAUNCHES = 0  # launches of our own kernels (for bench accounting)
 _LIB_GEMM = os.environ.get("ONECAT_GEMM_BACKEND", "tcgen05") == "library"  # debug switch only
@@ -134,7 +134,11 @@ def prepare_bf16(layer) -> None:
         w = w[interleave_gate_up(n_rows // 2, w.device)].contiguous()
         layer.weight.data = w
         epi, n_out = EPI_SILU_MUL, n_rows // 2
+    elif getattr(layer, "fuse_gelu_tanh", False):
+        epi = EPI_GELU_TANH
     layer.kernel_state = dict(kind="bf16", n_rows=n_rows, n_out=n_out, epi=epi, K=w.shape[1])
+    if w.shape[1] % 64:   # the GEMM walks whole 64-wide k tiles: zero columns in a copy that only the kernel reads
+        layer.kernel_state["w_pad"] = torch.nn.functional.pad(w, (0, -w.shape[1] % 64)).contiguous()
 
 
 def _bf16_bits(x: torch.Tensor) -> torch.Tensor:
@@ -286,41 +290,81 @@ def _gemm(x, w, w4, sz, out, bias, N, n_rows, n_out, n_pad, epi, gk, force_split
 
 
 def gemm_bf16(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
-              force_splits: int = 0, force_tn: int = 0) -> torch.Tensor:
-    """x ``[T,K]`` @ w ``[N,K]``^T → ``[T,N]`` bf16."""
+              force_splits: int = 0, force_tn: int = 0, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """x ``[T,K]`` @ w ``[N,K]``^T → ``[T,N]`` bf16, or fp32 (the accumulators) with ``out_dtype``."""
     N = w.shape[0]
     if _LIB_GEMM:
-        return torch.nn.functional.linear(x, w, bias)
+        y = torch.nn.functional.linear(x, w, bias)
+        return y if out_dtype is None else y.to(out_dtype)
+    if x.shape[1] % 64:
+        x, w = (torch.nn.functional.pad(t, (0, -x.shape[1] % 64)) for t in (x, w))
     if out is None:
-        out = torch.empty(x.shape[0], N, dtype=torch.bfloat16, device=x.device)
-    if x.stride(-1) != 1 or (x.stride(0) * 2) % 16:
+        out = torch.empty(x.shape[0], N, dtype=out_dtype or torch.bfloat16, device=x.device)
+    if x.stride(-1) != 1 or (x.stride(0) * 2) % 16 or x.data_ptr() % 16:
         x = x.contiguous()
     return _gemm(x, w, None, None, out, bias, N, N, N, 0, EPI_STORE, 1, force_splits, force_tn)
 
 
+def dense(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """x @ w^T in the inputs' precision: the tcgen05 GEMM for bf16, the library's fp32 product (no reduced-precision mode) for fp32."""
+    if x.dtype == torch.float32:
+        return _matmul_f32(x, w)
+    return gemm_bf16(x, w, out_dtype=out_dtype)
+
+
+def _matmul_f32(x, w, bias=None):
+    if torch.backends.cuda.matmul.allow_tf32:
+        raise RuntimeError("fp32 models need torch.backends.cuda.matmul.allow_tf32 = False")
+    return torch.nn.functional.linear(x, w, bias)
+
+
+def _linear_f32(layer, x: torch.Tensor) -> torch.Tensor:
+    """Linear layer of an engine that runs in 32 bits (dense weights)."""
+    global _LAUNCHES
+    w = getattr(layer, "weight", None)
+    if w is None or w.dtype != torch.float32:
+        raise ValueError("quantised weights are served with bf16 activations only")
+    y = _matmul_f32(x, w, layer.bias)
+    if layer.fuse_silu_mul:
+        return ref.silu_and_mul(y)
+    if getattr(layer, "fuse_gelu_tanh", False):
+        _LAUNCHES += 1
+        _C.gelu_tanh_f32(y)
+    return y
+
+
 def linear(layer, x: torch.Tensor, out: Optional[torch.Tensor] = None, push=None) -> torch.Tensor:
+    if x.dtype == torch.float32:
+        return _linear_f32(layer, x)
     ks = layer.kernel_state
     if ks is None:
         prepare_bf16(layer)
         ks = layer.kernel_state
     T = x.shape[0]
-    if x.stride(-1) != 1 or (x.stride(0) * 2) % 16:
+    w = ks.get("w_pad")
+    if w is not None:
+        x = torch.nn.functional.pad(x, (0, w.shape[1] - x.shape[1]))
+    if x.stride(-1) != 1 or (x.stride(0) * 2) % 16 or x.data_ptr() % 16:
         x = x.contiguous()
     if out is None:
-        out = torch.empty(T, ks["n_out"], dtype=torch.bfloat16, device=x.device)
+        n = ks["n_out"]   # row pitches are multiples of 16 bytes, so that column slices of the result are aligned for the next kernel
+        out = torch.empty(T, -(-n // 8) * 8, dtype=getattr(layer, "out_dtype", None) or torch.bfloat16, device=x.device)[:, :n]
     bias = layer.bias
     if ks["kind"] == "w4":
         if _LIB_GEMM:
             raise RuntimeError("the library GEMM debug switch does not cover 4-bit weights")
-        return _gemm(x, None, ks["tiles"], ks["sz"], out, bias, ks["n_rows"], ks["n_rows"], ks["n_out"], ks["n_pad"], ks["epi"], ks["group_ktiles"], push=push,
-                     wkind=ks.get("wkind", 1))
+        y = _gemm(x, None, ks["tiles"], ks["sz"], out, bias, ks["n_rows"], ks["n_rows"], ks["n_out"], ks["n_pad"], ks["epi"], ks["group_ktiles"], push=push,
+                  wkind=ks.get("wkind", 1))
+        return torch.nn.functional.gelu(y, approximate="tanh") if getattr(layer, "fuse_gelu_tanh", False) else y
     if _LIB_GEMM:
-        y = torch.nn.functional.linear(x, layer.weight, bias)
+        y = torch.nn.functional.linear(x, layer.weight if w is None else w, bias)
         if ks["epi"] == EPI_SILU_MUL:  # rows are interleaved in blocks of 16
             y = y.view(T, -1, 2, 16)
             return (torch.nn.functional.silu(y[:, :, 0].float()) * y[:, :, 1].float()).to(x.dtype).reshape(T, -1)
-        return y
-    return _gemm(x, layer.weight, None, None, out, bias, ks["n_rows"], ks["n_rows"], ks["n_out"], 0, ks["epi"], 1, push=push)
+        if ks["epi"] == EPI_GELU_TANH:
+            y = torch.nn.functional.gelu(y, approximate="tanh")
+        return y.to(out.dtype)
+    return _gemm(x, layer.weight if w is None else w, None, None, out, bias, ks["n_rows"], ks["n_rows"], ks["n_out"], 0, ks["epi"], 1, push=push)
 
 
 # ----------------------------------------------------------------------------- elementwise
@@ -357,6 +401,24 @@ def rope_and_cache(q, k, v, positions, cos_sin, kv_cache, slot_mapping, rotary_d
     _LAUNCHES += 1
     s0, s1 = (int(mrope_section[0]), int(mrope_section[0] + mrope_section[1])) if mrope_section is not None and positions.dim() == 2 else (0, 0)
     _C.rope_and_cache(q, k, v, positions, cos_sin, kv_cache, slot_mapping, rotary_dim, q_norm_w, k_norm_w, eps, gemma, 1.0, 1.0, s0, s1)
+
+
+def kv_insert(k, kv_cache, slot_mapping, v=None):
+    global _LAUNCHES
+    _LAUNCHES += 1
+    _C.kv_insert(k, v, kv_cache, slot_mapping)
+
+
+def stream_join(part, x, post, scale, nxt, out_dtype=None, add=None, copy_out=None):
+    global _LAUNCHES
+    _LAUNCHES += 1
+    T, H = part.shape
+    x_out = torch.empty(T, H, dtype=torch.float32, device=part.device) if x is None else x
+    y = torch.empty(T, H, dtype=out_dtype, device=part.device) if nxt is not None else None
+    none = (0, None, None, 0.0, False)
+    _C.stream_join(part, x, x_out, *(post or none), scale, *(nxt or none), y, add, copy_out, (copy_out.dtype if y is None and copy_out is not None
+                   else out_dtype or part.dtype) == torch.float32)
+    return y, x_out
 
 
 def sample(logits, temperature, top_k=None, top_p=None, min_p=None, generators=None, kept=None):
@@ -424,9 +486,10 @@ def choose_decode_splits(base_ctas: int, max_seq: int, num_sms: int) -> int:
     return best
 
 
-def plan_attention(query_lens: list, seq_lens: list, Hq: int, Hkv: int, D: int, num_sms: int, force_splits: int = 0):
+def plan_attention(query_lens: list, seq_lens: list, Hq: int, Hkv: int, D: int, num_sms: int, force_splits: int = 0, span: int = 0):
     """Decide which requests take the decode kernel (rows = q_len * group fit in one 16/32-row tile) and how many KV
-    splits it uses. Returns (short_q_len, num_q_tiles for the prefill kernel, splits)."""
+    splits it uses. Returns (short_q_len, num_q_tiles for the prefill kernel, splits). ``span`` > 0: a decode row reads at most that many
+    keys of its context (window and kept first tokens)."""
     G = Hq // Hkv
     max_rows = 32 if D <= 128 else 16
     short = max_rows // G
@@ -438,23 +501,38 @@ def plan_attention(query_lens: list, seq_lens: list, Hq: int, Hkv: int, D: int, 
     splits = 1
     if n_short:
         max_s = max((s for q, s in zip(query_lens, seq_lens) if q <= short), default=1)
-        splits = choose_decode_splits(n_short * Hkv, max_s, num_sms)
+        splits = choose_decode_splits(n_short * Hkv, min(max_s, span) if span else max_s, num_sms)
     if force_splits:
         splits = force_splits
     return short, tiles, splits
 
 
-def paged_attention(q, kv_cache, md, scale, out=None, lse=None, window=0, softcap=0.0, sinks=None):
-    """``window`` (tokens, 0 = full), ``softcap`` (0 = off) and ``sinks`` (fp32 ``[Hq]``) select the mma.sync kernels; the tcgen05
-    prefill kernel serves plain causal attention with D = 128."""
+def attention_span(window: int, keep: int) -> int:
+    """Most keys that the decode kernel walks for a sliding-window layer, in whole 64-key tiles; 0: the whole context."""
+    return 64 * (-(-window // 64) + 1 + -(-keep // 64)) if window else 0
+
+
+def paged_attention(q, kv_cache, md, scale, out=None, lse=None, window=0, softcap=0.0, sinks=None, keep=0, bias_table=None, gate=None):
+    """``window`` (tokens, 0 = full), ``softcap`` (0 = off), ``sinks`` (fp32 ``[Hq]``), ``keep`` (first tokens visible outside the window),
+    ``bias_table`` (fp32 ``[Hq, n]`` by distance), ``gate`` (``[T, Hq]`` logits) and a cache with one tensor per page select the mma.sync
+    kernels; the tcgen05 prefill kernel serves plain causal attention with D = 128. fp32 queries run the fp32 kernel."""
     global _LAUNCHES
     T, Hq, D = q.shape
     Hkv = kv_cache.shape[2]
     if out is None:
         out = torch.empty(T, Hq, D, dtype=q.dtype, device=q.device)
+    if q.dtype == torch.float32:
+        G = Hq // Hkv
+        tiles = sum(-(-n * G // 16) for n in md.query_lens_cpu)
+        _C.paged_attention(q, kv_cache, out, lse, md.query_start_loc, md.seq_lens, md.block_table, scale, 3, tiles, 1, md.max_query_len, 0, None, None,
+                           window, softcap, sinks, 1.0, 1.0, keep, bias_table, gate)
+        _LAUNCHES += 1
+        return out
+    extended = keep > 0 or bias_table is not None or gate is not None or kv_cache.shape[1] == 1
+    key = (Hq, Hkv, D, attention_span(window, keep)) if extended else (Hq, Hkv, D)
     plan = getattr(md, "attn_plan", None)
-    if plan is None or plan[0] != (Hq, Hkv, D):
-        plan = ((Hq, Hkv, D), plan_attention(md.query_lens_cpu, md.seq_lens_cpu, Hq, Hkv, D, _sms(q.device)))
+    if plan is None or plan[0] != key:
+        plan = (key, plan_attention(md.query_lens_cpu, md.seq_lens_cpu, Hq, Hkv, D, _sms(q.device), span=key[3] if extended else 0))
         md.attn_plan = plan
     short, tiles, splits = plan[1]
     n_short = sum(1 for x in md.query_lens_cpu if 0 < x <= short)
@@ -464,10 +542,10 @@ def paged_attention(q, kv_cache, md, scale, out=None, lse=None, window=0, softca
         ws_o, ws_ml = (w.attn_static if getattr(md, "static_ws", False) else w.attn)(splits * T * Hq * D, splits * T * Hq * 2)
     if n_short:
         _C.paged_attention(q, kv_cache, out, lse, md.query_start_loc, md.seq_lens, md.block_table, scale, 1, 0, splits,
-                           md.max_query_len, short, ws_o, ws_ml, window, softcap, sinks, 1.0, 1.0)
+                           md.max_query_len, short, ws_o, ws_ml, window, softcap, sinks, 1.0, 1.0, keep, bias_table, gate)
         _LAUNCHES += 2 if splits > 1 else 1
     if tiles:
-        if (D == 128 and q.stride(1) == D and _ATTN_PREFILL_TC and not window and not softcap and sinks is None
+        if (D == 128 and q.stride(1) == D and _ATTN_PREFILL_TC and not window and not softcap and sinks is None and not extended
                 and kv_cache.dtype == torch.bfloat16):
             # tcgen05 kernel: 128-token query tiles per (request, head)
             tiles_tc = sum(-(-x // 128) for x in md.query_lens_cpu if x > short)
@@ -475,7 +553,7 @@ def paged_attention(q, kv_cache, md, scale, out=None, lse=None, window=0, softca
                                md.max_query_len, short, None, None, 0, 0.0, None, 1.0, 1.0)
         else:
             _C.paged_attention(q, kv_cache, out, lse, md.query_start_loc, md.seq_lens, md.block_table, scale, 0, tiles, 1,
-                               md.max_query_len, short, None, None, window, softcap, sinks, 1.0, 1.0)
+                               md.max_query_len, short, None, None, window, softcap, sinks, 1.0, 1.0, keep, bias_table, gate)
         _LAUNCHES += 1
     return out
 

@@ -33,6 +33,31 @@ def rms_norm(x: torch.Tensor, w: torch.Tensor, eps: float, residual: Optional[to
     return y.to(x.dtype), new_res
 
 
+def stream_join(part, x, post, scale, nxt, out_dtype=None, add=None, copy_out=None):
+    """fp32 residual stream: ``x' = x + scale * post(part) (+ add)``, ``y = nxt(x')``. ``x`` None starts a stream from ``part``; ``post`` /
+    ``nxt`` are (kind, weight, bias, eps, plus_one) with kind 1 RMS, 2 layer norm, or None; ``copy_out`` receives ``x'`` in its own dtype.
+    Everything is fp32; returns (y in ``out_dtype`` or None, x'), with ``x`` updated in place."""
+    def norm(v, n):
+        kind, w, b, eps, plus = n
+        if kind == 2:
+            v = v - v.mean(-1, keepdim=True)
+        v = v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps)
+        if w is not None:
+            v = v * (w.float() + 1.0 if plus else w.float())
+        return v + b.float() if b is not None else v
+    v = part.float()
+    if post is not None:
+        v = norm(v, post)
+    if scale is not None:
+        v = v * scale.float()
+    if add is not None:
+        v = v + add.float()
+    x = x.add_(v) if x is not None else v.clone()
+    if copy_out is not None:
+        copy_out.copy_(x)
+    return (norm(x, nxt).to(out_dtype) if nxt is not None else None), x
+
+
 def rms_norm_gated(x: torch.Tensor, z: torch.Tensor, w: torch.Tensor, eps: float) -> torch.Tensor:
     """RMSNorm(x) * w * silu(z) per head (reference: layers/layernorm.py:422 ``RMSNormGated``)."""
     xf = x.float()
@@ -174,16 +199,50 @@ def rope_and_cache(q, k, v, positions, cos_sin, kv_cache, slot_mapping, rotary_d
             kv_cache[blk, 1, :, off, :] = v[ok].to(kv_cache.dtype)
 
 
+def kv_insert(k, kv_cache, slot_mapping, v=None) -> None:
+    """Rows of ``k`` (and ``v``) ``[T, Hkv, D]`` into the paged cache ``[blocks, 1 or 2, Hkv, block_size, D]`` at ``slot_mapping`` (negative:
+    skip). One cached tensor: the values are the keys."""
+    bs = kv_cache.shape[3]
+    ok = slot_mapping >= 0
+    sm = slot_mapping[ok].long()
+    kv_cache[sm // bs, 0, :, sm % bs, :] = k[ok].to(kv_cache.dtype)
+    if v is not None:
+        kv_cache[sm // bs, 1, :, sm % bs, :] = v[ok].to(kv_cache.dtype)
+
+
+def distance_buckets(buckets: int, max_dist: int) -> list[int]:
+    """Bucket of every distance 0..max_dist: each distance its own up to half of the buckets, from there on
+    ``half + floor(log(n / half) / log(max_dist / half) * (buckets - half))``, at most the last. The edge of step m is the smallest n with
+    ``n^K >= half^(K - m) * max_dist^m`` (K steps), so the floor is taken in integers and does not depend on how a logarithm rounds."""
+    half = buckets // 2
+    steps = buckets - half
+    if half < 1 or max_dist <= half:
+        raise ValueError(f"a distance bias with {buckets} buckets needs a maximum distance above {max(half, 1)}, got {max_dist}")
+    out, m = [], 0
+    for n in range(max_dist + 1):
+        if n < half:
+            out.append(n)
+            continue
+        while m < steps and n ** steps >= half ** (steps - m - 1) * max_dist ** (m + 1):
+            m += 1
+        out.append(min(buckets - 1, half + m))
+    return out
+
+
 # ----------------------------------------------------------------------------- paged attention
 def paged_attention(q, kv_cache, block_table, query_start_loc, seq_lens, scale: float,
                     out: Optional[torch.Tensor] = None, return_lse: bool = False, window: int = 0, softcap: float = 0.0,
-                    sinks: Optional[torch.Tensor] = None):
+                    sinks: Optional[torch.Tensor] = None, keep: int = 0, bias_table: Optional[torch.Tensor] = None,
+                    gate: Optional[torch.Tensor] = None):
     """Causal varlen attention over a paged cache. Request r owns query rows
     ``query_start_loc[r]:query_start_loc[r+1]`` which are the LAST rows of its ``seq_lens[r]``-token context
     (so decode, chunked prefill with prefix and multi-token verify are the same call).
     q ``[T, Hq, D]``, kv_cache ``[blocks, 2, Hkv, bs, D]``. fp32 math. ``window`` > 0: query i sees keys i-window+1..i
     (reference: Gemma2/3, GPT-OSS, Mistral sliding attention); ``softcap`` > 0: scores become cap·tanh(score/cap) (Gemma2);
-    ``sinks`` ``[Hq]``: one extra logit per head that takes probability mass but contributes no value (GPT-OSS)."""
+    ``sinks`` ``[Hq]``: one extra logit per head that takes probability mass but contributes no value (GPT-OSS). ``keep``: keys at
+    positions below it stay visible outside the window. ``bias_table`` ``[Hq, n]``: added to the scaled score by distance, distances past
+    the end take the last entry. ``gate`` ``[T, Hq]``: outputs are multiplied by its sigmoid. A cache with one tensor per page
+    (``[blocks, 1, ...]``) serves as keys and values."""
     T, Hq, D = q.shape
     Hkv, bs = kv_cache.shape[2], kv_cache.shape[3]
     g = Hq // Hkv
@@ -201,21 +260,26 @@ def paged_attention(q, kv_cache, block_table, query_start_loc, seq_lens, scale: 
         # an fp8 cache is gathered through a byte view (index ops on float8 tensors are not available everywhere)
         pages = kv_cache.view(torch.uint8)[blocks].view(torch.float8_e4m3fn) if kv_cache.dtype == torch.float8_e4m3fn else kv_cache[blocks]
         kk = pages[:, 0].float().permute(1, 0, 2, 3).reshape(Hkv, nb * bs, D)[:, :S]
-        vv = pages[:, 1].float().permute(1, 0, 2, 3).reshape(Hkv, nb * bs, D)[:, :S]
+        vv = pages[:, -1].float().permute(1, 0, 2, 3).reshape(Hkv, nb * bs, D)[:, :S]
         qq = q[q0:q1].float().permute(1, 0, 2).reshape(Hkv, g, nq, D)
         s = torch.einsum("hgqd,hkd->hgqk", qq, kk) * scale
         qpos = torch.arange(S - nq, S, device=q.device).view(1, 1, nq, 1)
         kpos = torch.arange(S, device=q.device).view(1, 1, 1, S)
         if softcap > 0:
             s = torch.tanh(s / softcap) * softcap
+        if bias_table is not None:
+            dist = (qpos - kpos).view(nq, S).clamp(0, bias_table.shape[1] - 1)
+            s = s + bias_table.float()[:, dist].view(Hkv, g, nq, S)
         s = s.masked_fill(kpos > qpos, -float("inf"))
         if window > 0:
-            s = s.masked_fill(kpos <= qpos - window, -float("inf"))
+            s = s.masked_fill((kpos <= qpos - window) & (kpos >= keep), -float("inf"))
         l = torch.logsumexp(s, dim=-1)
         if sinks is not None:
             l = torch.logaddexp(l, sinks.float().view(Hkv, g, 1).expand_as(l))
         p = torch.exp(s - l.unsqueeze(-1))
         oo = torch.einsum("hgqk,hkd->hgqd", p, vv).reshape(Hq, nq, D).permute(1, 0, 2)
+        if gate is not None:
+            oo = oo * torch.sigmoid(gate[q0:q1].float()).unsqueeze(-1)
         o[q0:q1] = oo.to(o.dtype)
         lse[q0:q1] = l.reshape(Hq, nq).t()
     return (o, lse) if return_lse else o

@@ -3,7 +3,9 @@ compilation/cuda_graph.py:147,268; capture sizes config/vllm.py:2084-2200).
 
 A graph is keyed by (padded request count, tokens per request, KV-split count). Batches are padded up to the next
 captured size; the split count follows the live context length in power-of-two buckets, so short contexts never
-launch a grid sized for the longest one (the reference's context-bucketed graphs). All inputs live in the runner's
+launch a grid sized for the longest one (the reference's context-bucketed graphs). Models whose layers differ in attention geometry or
+window have no single split count: their graphs are keyed by the context bucket itself, and every layer plans its splits for that
+bucket (capped by its own window) while it is captured. All inputs live in the runner's
 persistent device buffers, so replay needs no pointer patching."""
 from __future__ import annotations
 
@@ -38,10 +40,16 @@ class DecodeGraphs:
         # geometry that sizes the split-KV grid and workspace: (query heads, KV heads, head size); MLA runs all heads of a request
         # against one latent "head" of 512
         self.geom = None
+        attns = [l.self_attn for l in layers]
+        self.own_plans = any(a.kv_shared or a.window_keep or a.bias_table is not None or (a.Hq, a.Hkv, a.D) != (attns[0].Hq, attns[0].Hkv, attns[0].D)
+                             for a in attns)
+        self.max_span = 0   # the longest stretch of keys that a decode row of any layer walks (0: the whole context)
         if layers:
             a = layers[0].self_attn
             self.geom = (a.Hq, a.Hkv, a.D)
-            K.workspace(runner.device).attn_static(32 * tmax * a.Hq * a.D, 32 * tmax * a.Hq * 2)
+            K.workspace(runner.device).attn_static(32 * tmax * max(a.Hq * a.D for a in attns), 32 * tmax * 2 * max(a.Hq for a in attns))
+            spans = [K.attention_span(a.window, a.window_keep) for a in attns]
+            self.max_span = max(spans) if all(spans) else 0
         elif mla:
             a = mla[0].self_attn
             self.geom = ("mla", a.H, 512)
@@ -59,6 +67,8 @@ class DecodeGraphs:
         if not self.eligible or R > self.sizes[-1] or q > self.max_q:
             return None
         rp = self.sizes[bisect.bisect_left(self.sizes, R)]
+        if self.own_plans:
+            return rp, q, self._context_bucket(max_seq)
         from onecat_vllm.ops.cuda import _sms, choose_decode_splits, choose_kv_splits
         if self.geom[0] == "mla":
             want = choose_kv_splits(rp * (-(-q * self.geom[1] // 16)), max_seq, _sms(self.r.device))
@@ -69,6 +79,14 @@ class DecodeGraphs:
             s *= 2
         return rp, q, min(s, 32)
 
+    def _context_bucket(self, max_seq: int) -> int:
+        """Power of two of at least 512 that covers the keys a decode row walks (contexts beyond every layer's window share one bucket)."""
+        n = min(max_seq, self.max_span) if self.max_span else max_seq
+        b = 512
+        while b < n:
+            b *= 2
+        return b
+
     def _metadata(self, rp: int, q: int, splits: int) -> AttentionMetadata:
         r = self.r
         T = rp * q
@@ -77,7 +95,9 @@ class DecodeGraphs:
                                uniform_query_len=q)
         if r._seg["pos3"]:
             md.mrope_positions = r._view("pos3", 3 * r._tcap).view(3, r._tcap)[:, :T]
-        if self.geom[0] == "mla":
+        if self.own_plans:
+            md.seq_lens_cpu = [splits] * rp   # the context bucket; each layer's plan follows from it
+        elif self.geom[0] == "mla":
             md.attn_plan = (("mla", self.geom[1], 512), (q, 0, splits))
         else:
             Hq, Hkv, D = self.geom
@@ -120,8 +140,9 @@ class DecodeGraphs:
         r.np_pack[o["slot"][0]: o["slot"][0] + o["slot"][1]] = -1
         r.d_pack.copy_(r.h_pack)
         r.d_bt.copy_(r.h_bt)
+        first = self._context_bucket(self.max_span or 1) if self.own_plans else 1
         for s in reversed(self.sizes):
-            self.capture((s, 1, 1))
+            self.capture((s, 1, first))
         log.info_once(f"captured {len(self.graphs)} decode graphs (sizes up to {self.sizes[-1]})")
 
     def run(self, key: tuple, T: int) -> torch.Tensor:

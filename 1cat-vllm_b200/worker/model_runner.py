@@ -186,16 +186,17 @@ class ModelRunner:
         mc, specs = self.mc, {}
         esz = torch.empty(0, dtype=self._kv_dtype()).element_size()
         asz = torch.empty(0, dtype=self._attn_kv_dtype()).element_size()
-        for i, layer in self.model.model.local_layers():
+        for name, layer in self.model.model.cache_layers():
             if layer.kind == "linear_attention":
                 (cd, kw), (hv, k, v) = layer.linear_attn.state_shapes()
                 nspec = self.num_spec + 1
-                specs[f"layers.{i}"] = KVCacheSpec("mamba", self.block_size, 0, 0, 0,
+                specs[name] = KVCacheSpec("mamba", self.block_size, 0, 0, 0,
                                                     state_bytes=(cd * kw * esz + hv * k * v * 4))
             elif layer.kind == "mla":
-                specs[f"layers.{i}"] = KVCacheSpec("mla", self.block_size, 1, mc.kv_lora_rank + mc.qk_rope_head_dim, esz)
+                specs[name] = KVCacheSpec("mla", self.block_size, 1, mc.kv_lora_rank + mc.qk_rope_head_dim, esz)
             else:
-                specs[f"layers.{i}"] = KVCacheSpec("full", self.block_size, layer.self_attn.Hkv, mc.head_dim, asz)
+                a = layer.self_attn
+                specs[name] = KVCacheSpec("full", self.block_size, a.Hkv, a.D, asz, tensors=1 if a.kv_shared else 2)
         for i, layer in (self.draft.model.local_layers() if self.draft is not None else ()):
             specs[f"draft.{i}"] = KVCacheSpec("full", self.block_size, layer.self_attn.Hkv, self.draft.cfg.head_dim, asz)
         if self.mtp is not None:
@@ -217,6 +218,8 @@ class ModelRunner:
         if cd in ("auto", "bfloat16", "bf16"):
             return self.mc.dtype
         if cd in ("fp8", "fp8_e4m3"):
+            if self.mc.attn_kv_shared or self.mc.attn_rel_buckets or any(o.get("attn_window_keep") for o in self.mc.layer_overrides):
+                raise ValueError("an fp8 KV cache is not served for attention with shared keys and values, a distance bias or kept first tokens")
             return torch.float8_e4m3fn
         raise ValueError(f"kv cache dtype {cd!r} is not supported (auto | fp8 | fp8_e4m3)")
 
@@ -236,11 +239,11 @@ class ModelRunner:
                 return None
             if spec.kind == "mla":
                 return torch.zeros(nb, bs, spec.head_size, dtype=dt, device=dev)
-            return torch.zeros(nb, 2, spec.num_kv_heads, bs, spec.head_size, dtype=self._attn_kv_dtype(), device=dev)
+            return torch.zeros(nb, spec.tensors, spec.num_kv_heads, bs, spec.head_size, dtype=self._attn_kv_dtype(), device=dev)
 
         self.kv_caches = []
-        for i, layer in self.model.model.local_layers():
-            spec = kvc.layer_specs[f"layers.{i}"]
+        for name, layer in self.model.model.cache_layers():
+            spec = kvc.layer_specs[name]
             if spec.kind == "mamba":
                 (cd, kw), (hv, k, v) = layer.linear_attn.state_shapes()
                 slots = kvc.num_state_slots
@@ -703,6 +706,12 @@ class ModelRunner:
                 torch.cuda.synchronize()
                 out.device_time_ms = ev0.elapsed_time(ev1)
             return out
+        if so.logits_for is not None:
+            out.logits = self._wanted_logits(so.logits_for, hidden, req_ids, query_lens)
+            if self.use_cuda:
+                from onecat_vllm.ops import cuda as K
+                out.status = K.check_status()
+            return out
         sampled_lists: list[list[int]] = [[] for _ in req_ids]
         if n_l > 0:
             lidx = self._view("lidx", n_l).long()
@@ -779,6 +788,17 @@ class ModelRunner:
             from onecat_vllm.ops import cuda as K
             out.status = K.check_status()
         return out
+
+    def _wanted_logits(self, wanted: dict, hidden: torch.Tensor, req_ids: list, query_lens: list[int]) -> Optional[torch.Tensor]:
+        """fp32 logits of the asked-for positions of a replayed step, in the order of ``wanted``."""
+        start, o = {}, 0
+        for rid, q in zip(req_ids, query_lens):
+            start[rid] = o
+            o += q
+        rows = [start[rid] + j for rid, offs in wanted.items() for j in offs]
+        if not rows:
+            return None
+        return self.model.compute_logits(hidden[torch.tensor(rows, device=hidden.device)]).float().cpu()
 
     def _prompt_logprobs(self, hidden: torch.Tensor, req_ids: list, query_lens: list[int]):
         """Log-probabilities of the prompt tokens that this step's chunk predicts, for requests that asked for them: per request a
@@ -1088,12 +1108,13 @@ class ModelRunner:
         """One-block caches so the profiling forward can run before the real cache exists."""
         out = []
         dt = self._kv_dtype()
-        for _, layer in self.model.model.local_layers():
+        for _, layer in self.model.model.cache_layers():
             if layer.kind == "linear_attention":
                 (cd, kw), (hv, k, v) = layer.linear_attn.state_shapes()
                 out.append((torch.zeros(1, cd, kw, dtype=dt, device=self.device), torch.zeros(1, hv, k, v, dtype=torch.float32, device=self.device)))
             elif layer.kind == "mla":
                 out.append(torch.zeros(1, self.block_size, self.mc.kv_lora_rank + self.mc.qk_rope_head_dim, dtype=dt, device=self.device))
             else:
-                out.append(torch.zeros(1, 2, layer.self_attn.Hkv, self.block_size, self.mc.head_dim, dtype=dt, device=self.device))
+                a = layer.self_attn
+                out.append(torch.zeros(1, 1 if a.kv_shared else 2, a.Hkv, self.block_size, a.D, dtype=dt, device=self.device))
         return out
