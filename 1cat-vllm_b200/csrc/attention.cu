@@ -16,7 +16,8 @@
 // Extended variants (EXT, bf16 cache): first tokens that stay visible outside the window (their tiles are walked ahead of the window's),
 // a bias by distance added to the scores in fp32, values that are the keys (one tensor per page: the ring holds one tile per stage and
 // both products read it), one output gate per head. The softmax weights enter the value product as two bf16 terms (p and the rest of
-// p after rounding), so that they keep about 16 bits of mantissa.
+// p after rounding), so that they keep about 16 bits of mantissa. In a decode tile of at most eight rows the second terms ride in the
+// unused rows 8..15 of the same operand and cost no extra product.
 // (reference: flash-attention-v100/kernel/fused_mha_forward_paged.cu:364, flash_decode_paged.cu:667,831,1301;
 //  v1/attention/backends/flash_attn_v100.py:2216 for the math)
 #include <cuda_fp8.h>
@@ -82,8 +83,17 @@ __device__ __forceinline__ float head_gate(const AttnParams& p, size_t tok, int 
   return 1.f / (1.f + __expf(-__bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.gate)[tok * p.gate_st + head])));
 }
 
+// CTAs per SM that the extended variants are compiled for (0: the compiler's choice)
+template <int D, int MODE, int MB, bool EXT>
+constexpr int ext_min_ctas() {
+  if (!EXT) return 0;
+  if (D == 64) return MODE == 0 ? 4 : (MB == 1 ? 5 : 3);
+  if (D == 128) return MODE == 0 ? 3 : (MB == 1 ? 4 : 2);
+  return 0;
+}
+
 template <int D, int MODE, int MB, bool KV8, int ST = 3, bool EXT = false>
-__global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
+__global__ void __launch_bounds__(128, ext_min_ctas<D, MODE, MB, EXT>()) attn_kernel(const AttnParams p) {
   pdl_trigger();
   pdl_wait();
   constexpr int STAGES = ST;                    // K/V tiles in the cp.async ring (a fourth stage of byte tiles measured no faster)
@@ -220,12 +230,19 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
   constexpr bool WARP_PIPE = (MODE == 1);
   constexpr int WCH = KV8 ? D / 16 : CH;        // 16-byte chunks per cache row
   const uint8_t* kv_warp = reinterpret_cast<const uint8_t*>(p.kv_cache) + ((size_t)hkv * page_elems) * ESZ;
-  auto load_tile_w = [&](int tile, int buf) {
+  // Extended variants read a tile's block-table entry one iteration before its copies are issued, so that its latency is not in the way
+  // of this iteration's products.
+  int next_blk = 0;
+  auto peek_blk = [&](int v) {
+    const int key0 = tile_of(v) * kKeysPerTile + warp * 16;
+    next_blk = (v < tile_hi && key0 < kv_end) ? __ldg(bt + (key0 >> bs_shift)) : 0;
+  };
+  auto load_tile_w = [&](int tile, int buf, int blk) {
     const int key0 = tile * kKeysPerTile + warp * 16;
     uint8_t* dk = sK + (size_t)buf * kKeysPerTile * D * ESZ;
     uint8_t* dv = sV + (size_t)buf * kKeysPerTile * D * ESZ;
     const uint8_t* src = kv_warp;
-    if (key0 < kv_end) src += (size_t)bt[key0 >> bs_shift] * blk_stride + (size_t)(key0 & bs_mask) * (D * ESZ);
+    if (key0 < kv_end) src += (size_t)(EXT ? blk : bt[key0 >> bs_shift]) * blk_stride + (size_t)(key0 & bs_mask) * (D * ESZ);
 #pragma unroll
     for (int i = 0; i < 16 * WCH / 32; ++i) {
       const int idx = lane + 32 * i, rl = idx / WCH, ch = idx % WCH;
@@ -258,10 +275,32 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
   const int key_base = (MODE == 0) ? 0 : warp * 16;
   const int g_ = lane >> 2, tg = lane & 3;
 
+  // extended variants: what the rows of this thread need in every tile
+  int row_pos[MBW][2];
+  const float* row_bias[MBW][2];
+  float row_far[MBW][2];
+  int pos_lo = 0, pos_hi = 0;
+  const bool paired = EXT && MODE == 1 && MB == 1 && nrows <= 8;   // rows 8..15 carry the second terms of rows 0..7
+  if constexpr (EXT) {
+    pos_lo = ctx0 + tq0 + row_base / G;
+    pos_hi = ctx0 + tq0 + (row_base + 16 * MBW - 1) / G;
+#pragma unroll
+    for (int b = 0; b < MBW; ++b)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int row = row_base + b * 16 + g_ + h * 8, tok = row / G;
+        row_pos[b][h] = ctx0 + tq0 + tok;
+        row_bias[b][h] = p.bias != nullptr ? p.bias + (size_t)(hkv * G + row - tok * G) * p.bias_len : nullptr;
+        row_far[b][h] = p.bias != nullptr ? __ldg(row_bias[b][h] + p.bias_len - 1) * kLog2e : 0.f;
+      }
+  }
 #pragma unroll
   for (int i = 0; i < STAGES - 1; ++i) {
     if (tile_lo + i < tile_hi) {
-      if constexpr (WARP_PIPE) load_tile_w(tile_of(tile_lo + i), i);
+      if constexpr (WARP_PIPE) {
+        if constexpr (EXT) peek_blk(tile_lo + i);
+        load_tile_w(tile_of(tile_lo + i), i, next_blk);
+      }
       else load_tile(tile_of(tile_lo + i), i);
     }
     cp_async_commit();
@@ -277,6 +316,7 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
     }
     *reinterpret_cast<uint4*>(sQ + sw_off<D>(row, ch)) = v;
   }
+  if constexpr (WARP_PIPE && EXT) peek_blk(tile_lo + STAGES - 1);
   if constexpr (WARP_PIPE) __syncthreads();  // publishes the Q tile; the loop below has no CTA-wide barrier
 
   for (int tile = tile_lo; tile < tile_hi; ++tile) {
@@ -284,7 +324,8 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
     cp_async_wait<STAGES - 2>();  // the group of this tile has landed (one group is committed per iteration)
     if constexpr (WARP_PIPE) {
       __syncwarp();                // ...for every lane of this warp, whose ldmatrix reads of the buffer refilled below are done
-      if (tile + STAGES - 1 < tile_hi) load_tile_w(tile_of(tile + STAGES - 1), (tile - tile_lo + STAGES - 1) % STAGES);
+      if (tile + STAGES - 1 < tile_hi) load_tile_w(tile_of(tile + STAGES - 1), (tile - tile_lo + STAGES - 1) % STAGES, next_blk);
+      if constexpr (EXT) peek_blk(tile + STAGES);
     } else {
       __syncthreads();             // ...for every thread, and everybody has finished the buffer refilled below
       if (tile + STAGES - 1 < tile_hi) load_tile(tile_of(tile + STAGES - 1), (tile - tile_lo + STAGES - 1) % STAGES);
@@ -359,23 +400,39 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
     // whole tiles of this warp that need neither masking nor a per-key bias
     bool no_mask = false, far_bias = false;
     if constexpr (EXT) {
-      const int q_lo = ctx0 + tq0 + row_base / G, q_hi = ctx0 + tq0 + (row_base + 16 * MBW - 1) / G, k_hi = k0 + NB2 * 16 - 1;
-      no_mask = k_hi <= q_lo && k_hi < kv_end && (k0 + wlo > q_hi || k_hi < p.keep);
-      far_bias = p.bias != nullptr && q_lo - k_hi >= p.bias_len - 1;
+      const int k_hi = k0 + NB2 * 16 - 1;
+      no_mask = k_hi <= pos_lo && k_hi < kv_end && (k0 + wlo > pos_hi || k_hi < p.keep);
+      far_bias = p.bias == nullptr || pos_lo - k_hi >= p.bias_len - 1;   // one value per row (0 without a bias)
     }
 #pragma unroll
     for (int b = 0; b < MBW; ++b) {
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
+        if (paired && h == 1) {
+          alpha_r[b][1] = alpha_r[b][0];
+          continue;
+        }
         const int row = row_base + b * 16 + g_ + h * 8;
-        const int qpos = ctx0 + tq0 + row / G;  // rows past nrows are never stored
-        const float* bias_row = nullptr;
-        float bias_far = 0.f;
+        const int qpos = EXT ? row_pos[b][h] : ctx0 + tq0 + row / G;  // rows past nrows are never stored
         if constexpr (EXT) {
-          if (p.bias != nullptr) {
-            bias_row = p.bias + (size_t)(hkv * G + row % G) * p.bias_len;
-            bias_far = __ldg(bias_row + p.bias_len - 1);
+          // one decision per tile and row instead of one per score
+          auto each = [&](auto f) {
+#pragma unroll
+            for (int n = 0; n < NB2 * 2; ++n)
+#pragma unroll
+              for (int e = 0; e < 2; ++e) s[b][n][h * 2 + e] = f(s[b][n][h * 2 + e], k0 + n * 8 + tg * 2 + e);
+          };
+          const float far = row_far[b][h];
+          if (far_bias && !capped) {
+            each([&](float v, int) { return fmaf(v, sc, far); });
+          } else {
+            if (capped) each([&](float v, int) { return tanhf(v * sc) * sc_post; });
+            else each([&](float v, int) { return v * sc; });
+            if (far_bias) each([&](float v, int) { return v + far; });
+            else each([&](float v, int key) { return fmaf(__ldg(row_bias[b][h] + min(max(qpos - key, 0), p.bias_len - 1)), kLog2e, v); });
           }
+          if (!no_mask)
+            each([&](float v, int key) { return (key <= qpos && key < kv_end && (key + wlo > qpos || key < p.keep)) ? v : -INFINITY; });
         }
         float mx = -INFINITY;
 #pragma unroll
@@ -383,12 +440,10 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
             int key = k0 + n * 8 + tg * 2 + e;
-            float v = s[b][n][h * 2 + e] * sc;
-            if (capped) v = tanhf(v) * sc_post;
-            if constexpr (EXT) {
-              if (p.bias != nullptr) v = fmaf(far_bias ? bias_far : __ldg(bias_row + min(max(qpos - key, 0), p.bias_len - 1)), kLog2e, v);
-              if (!no_mask) v = (key <= qpos && key < kv_end && (key + wlo > qpos || key < p.keep)) ? v : -INFINITY;
-            } else {
+            float v = s[b][n][h * 2 + e];
+            if constexpr (!EXT) {
+              v *= sc;
+              if (capped) v = tanhf(v) * sc_post;
               v = (key <= qpos && key < kv_end && key + wlo > qpos) ? v : -INFINITY;
             }
             s[b][n][h * 2 + e] = v;
@@ -447,12 +502,17 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
           const float2 f = __bfloat1622float2(*reinterpret_cast<__nv_bfloat162*>(&hi));
           return pack_bf16(x - f.x, y - f.y);
         };
+        if (paired) {
+          a[0][1] = rest(a[0][0], s[0][n2 * 2][0], s[0][n2 * 2][1]);
+          a[0][3] = rest(a[0][2], s[0][n2 * 2 + 1][0], s[0][n2 * 2 + 1][1]);
+        } else {
 #pragma unroll
-        for (int b = 0; b < MBW; ++b) {
-          lo[b][0] = rest(a[b][0], s[b][n2 * 2][0], s[b][n2 * 2][1]);
-          lo[b][1] = rest(a[b][1], s[b][n2 * 2][2], s[b][n2 * 2][3]);
-          lo[b][2] = rest(a[b][2], s[b][n2 * 2 + 1][0], s[b][n2 * 2 + 1][1]);
-          lo[b][3] = rest(a[b][3], s[b][n2 * 2 + 1][2], s[b][n2 * 2 + 1][3]);
+          for (int b = 0; b < MBW; ++b) {
+            lo[b][0] = rest(a[b][0], s[b][n2 * 2][0], s[b][n2 * 2][1]);
+            lo[b][1] = rest(a[b][1], s[b][n2 * 2][2], s[b][n2 * 2][3]);
+            lo[b][2] = rest(a[b][2], s[b][n2 * 2 + 1][0], s[b][n2 * 2 + 1][1]);
+            lo[b][3] = rest(a[b][3], s[b][n2 * 2 + 1][2], s[b][n2 * 2 + 1][3]);
+          }
         }
       }
 #pragma unroll
@@ -464,7 +524,7 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
         for (int b = 0; b < MBW; ++b) {
           mma_bf16(o[b][d2 * 2], a[b], bfr[0], bfr[1]);
           mma_bf16(o[b][d2 * 2 + 1], a[b], bfr[2], bfr[3]);
-          if constexpr (EXT) {
+          if (EXT && !paired) {
             mma_bf16(o[b][d2 * 2], lo[b], bfr[0], bfr[1]);
             mma_bf16(o[b][d2 * 2 + 1], lo[b], bfr[2], bfr[3]);
           }
@@ -495,6 +555,13 @@ __global__ void __launch_bounds__(128) attn_kernel(const AttnParams p) {
 
   // ---- mode 1: merge the four warps' partial results (they saw disjoint keys), then store or hand to the split combine
   __syncthreads();  // everyone is done reading K/V tiles; reuse that memory
+  if (paired) {
+#pragma unroll
+    for (int i = 0; i < D / 8; ++i) {
+      o[0][i][0] += o[0][i][2];
+      o[0][i][1] += o[0][i][3];
+    }
+  }
   float* mo = reinterpret_cast<float*>(sK);             // [4][ROWS][D]
   float* mm = reinterpret_cast<float*>(sQ);             // [4][ROWS][2] (the Q tile is no longer needed)
 #pragma unroll

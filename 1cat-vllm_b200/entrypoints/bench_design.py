@@ -1,0 +1,167 @@
+"""Prefill and decode throughput of the Gabisun design beside the closest models of equal size, and its kernels beside theirs.
+
+``python bench.py --design gabisun`` prints one JSON line per size. Random weights and token ids. The models share width, heads, head
+size, window, layer runs, vocabulary and tied embeddings: Starcoder2 (layer norms, ungated GELU feed-forward of the same width; its norms
+are PyTorch operations) and Mistral (every step fused; RMS norms, a gated feed-forward of 2/3 the width, so the same number of weights).
+Model throughput is device time of engine steps (CUDA events); kernels are timed alone with the L2 flushed before every launch."""
+from __future__ import annotations
+
+import gc
+import json
+
+import torch
+
+SIZES = {
+    # width, query heads, kv heads, head size, feed-forward, layers, loop, window, kept tokens, scale
+    "w2048": dict(width=2048, heads=16, kv=4, dim=128, ff=8192, layers=12, loop=(2, 6, 2), window=1024, keep=64),
+    "w4096": dict(width=4096, heads=32, kv=8, dim=128, ff=16384, layers=8, loop=(2, 4, 2), window=4096, keep=128),
+    "w2048d64": dict(width=2048, heads=32, kv=8, dim=64, ff=8192, layers=12, loop=(2, 6, 2), window=1024, keep=64),
+}
+VOCAB, BIAS_MAX = 32000, 128
+PREFILL, DECODE_REQS, DECODE_CTX = 8192, 64, 4096
+
+
+def gabisun_config(s: dict) -> dict:
+    layer = dict(type="attention", mixer=dict(heads=s["heads"], kv_heads=s["kv"], dim=s["dim"], vdim=s["dim"], scale=s["dim"] ** -0.5, bias_max=BIAS_MAX,
+                 mask=dict(size=s["window"], keep_first=s["keep"])), mlp=dict(kind="dense", ff=s["ff"]))
+    return dict(architecture="Gabisun", width=s["width"], vocab=VOCAB, norm=dict(eps=1e-5), layers=[layer] * s["layers"],
+                loop=dict(zip(("start", "stop", "times"), s["loop"])))
+
+
+def like_config(s: dict, arch: str) -> dict:
+    a, b, times = s["loop"]
+    cfg = dict(architectures=[arch], hidden_size=s["width"], num_hidden_layers=s["layers"] + (times - 1) * (b - a), num_attention_heads=s["heads"],
+               num_key_value_heads=s["kv"], head_dim=s["dim"], vocab_size=VOCAB, tie_word_embeddings=True, max_position_embeddings=32768,
+               sliding_window=s["window"], rope_theta=10000.0)
+    if arch.startswith("Starcoder2"):
+        return dict(cfg, intermediate_size=s["ff"], hidden_act="gelu_pytorch_tanh", norm_epsilon=1e-5, use_bias=False)
+    return dict(cfg, intermediate_size=s["ff"] * 2 // 3 // 64 * 64, rms_norm_eps=1e-5)
+
+
+def model_throughput(cfg: dict, steps: int, warmup: int) -> dict:
+    """Device time per step of (a) 8192-token prefill steps, (b) decode steps of 64 requests at a context of about 4096 tokens."""
+    from onecat_vllm.config import EngineArgs
+    from onecat_vllm.engine.llm_engine import LLMEngine
+    from onecat_vllm.sampling_params import SamplingParams
+    eng = LLMEngine.from_engine_args(EngineArgs(hf_config=cfg, dtype="bfloat16", device="cuda", max_model_len=2 * PREFILL, max_num_seqs=DECODE_REQS,
+                                                max_num_batched_tokens=PREFILL, enable_prefix_caching=False, async_scheduling=False, disable_log_stats=False,
+                                                kv_cache_memory_bytes=24 << 30))
+    g, n = torch.Generator().manual_seed(0), [0]
+
+    def add(length, out):
+        n[0] += 1
+        eng.add_request(f"r{n[0]}", torch.randint(0, VOCAB, (length,), generator=g).tolist(),
+                        SamplingParams(temperature=0.0, max_tokens=out, ignore_eos=True, detokenize=False))
+
+    def step():
+        eng.step()
+        st = eng.last_scheduler_stats
+        return st.step_device_ms, st.num_scheduled_tokens
+
+    ms = []
+    for i in range(warmup + max(4, steps // 4)):
+        add(PREFILL, 1)
+        t, tok = step()
+        assert tok == PREFILL
+        if i >= warmup:
+            ms.append(t)
+    out = dict(prefill_ms=sorted(ms)[len(ms) // 2])
+    out["prefill_tokens_per_s"] = PREFILL / out["prefill_ms"] * 1e3
+    for _ in range(DECODE_REQS):
+        add(DECODE_CTX, warmup + steps + 80)
+    ms = []
+    while len(ms) < warmup + steps:
+        t, tok = step()
+        if tok == DECODE_REQS:
+            ms.append(t)
+    ms = sorted(ms[warmup:])
+    out["decode_ms"] = ms[len(ms) // 2]
+    out["decode_tokens_per_s"] = DECODE_REQS / out["decode_ms"] * 1e3
+    eng.shutdown()
+    del eng
+    gc.collect()
+    torch.cuda.empty_cache()
+    return out
+
+
+def _meta(R, q, S):
+    from onecat_vllm.worker.attn_metadata import AttentionMetadata
+    nb = -(-S // 16)
+    bt = (torch.randperm(R * nb, device="cuda").to(torch.int32) + 1).view(R, nb)
+    return AttentionMetadata(R, R * q, torch.arange(R + 1, device="cuda", dtype=torch.int32) * q, torch.full((R,), S, device="cuda", dtype=torch.int32), bt,
+                             None, None, q, S, query_lens_cpu=[q] * R, seq_lens_cpu=[S] * R), R * nb + 1
+
+
+def kernel_rows(s: dict, iters: int) -> list[dict]:
+    """Each kernel of the design beside the like kernel of the dense models, as fractions of the measured peaks."""
+    from onecat_vllm.ops import cuda as K
+    from onecat_vllm.ops.microbench import _peaks, timeit
+    pk, rows = _peaks(), []
+    W, H, G, D, win, keep = s["width"], s["heads"], s["kv"], s["dim"], s["window"], s["keep"]
+
+    def row(kernel, case, who, fn, flops=0.0, nbytes=0.0):
+        ms = timeit(fn, iters)
+        t = max(flops / pk["bf16_tflops"] / 1e9, nbytes / pk["hbm_gbs"] / 1e6)
+        rows.append(dict(kernel=kernel, case=case, model=who, us=ms * 1e3, roofline_us=t * 1e3, frac_of_roofline=t / ms))
+
+    sinks, table = torch.randn(H, device="cuda"), torch.randn(H, BIAS_MAX + 1, device="cuda")
+    for case, R, q, S in (("prefill", 1, PREFILL, PREFILL), ("decode", DECODE_REQS, 1, DECODE_CTX)):
+        md, nblk = _meta(R, q, S)
+        x = (torch.randn(R * q, H * D + G * D + H, device="cuda") * 0.5).bfloat16()
+        qq, gate = x[:, : H * D].view(-1, H, D), x[:, (H + G) * D:]
+        pairs = sum(min(i + 1, win) + max(0, min(keep, i + 1 - win)) for i in range(S - q, S)) * R
+        keys = min(S, win + keep) * R if q == 1 else S * R
+        for who, tensors, kw in (("gabisun", 1, dict(keep=keep, bias_table=table, gate=gate, sinks=sinks)), ("window+sinks", 2, dict(sinks=sinks))):
+            cache = (torch.randn(nblk, tensors, G, 16, D, device="cuda") * 0.5).bfloat16()
+            md.attn_plan = None
+            out = torch.empty(R * q, H, D, dtype=torch.bfloat16, device="cuda")
+            row("attention", case, who, lambda: K.paged_attention(qq, cache, md, D ** -0.5, out=out, window=win, **kw), flops=4.0 * H * D * pairs,
+                nbytes=2.0 * (keys * tensors * G * D + 2 * R * q * H * D))
+            del cache
+    for T in (PREFILL, DECODE_REQS):
+        b = lambda *sh: torch.randn(*sh, device="cuda").bfloat16()
+        part, x32, w, res = b(T, W), torch.randn(T, W, device="cuda"), b(W), b(T, W)
+        norm = (2, w, w, 1e-5, False)
+        row("norm", T, "gabisun join", lambda: K.stream_join(part, x32, norm, w, norm, torch.bfloat16), nbytes=12.0 * T * W)
+        row("norm", T, "add + rms norm", lambda: K.rms_norm(part, w, 1e-5, res, False), nbytes=8.0 * T * W)
+        slot = torch.arange(T, device="cuda", dtype=torch.int32)
+        kk = b(T, (H + 2 * G) * D)
+        ksl = kk[:, H * D: (H + G) * D].view(T, G, D)
+        c1, c2 = b(T // 16 + 1, 1, G, 16, D), b(T // 16 + 1, 2, G, 16, D)
+        row("cache insert", T, "gabisun", lambda: K.kv_insert(ksl, c1, slot), nbytes=4.0 * T * G * D)
+        cs = torch.ones(T, D, device="cuda")
+        row("cache insert", T, "rope + insert", lambda: K.rope_and_cache(kk[:, : H * D].view(T, H, D), ksl, kk[:, (H + G) * D:].view(T, G, D), slot, cs, c2, slot, D,
+                                                                       None, None, 1e-5, False), nbytes=4.0 * T * (H + 2 * G) * D)
+
+        def gemm(name, who, N, Kd, **kw):
+            wt, xx = (torch.randn(N, Kd, device="cuda") * 0.02).bfloat16(), b(T, Kd)
+            out = torch.empty(T, -(-N // 8) * 8, dtype=kw.get("out_dtype", torch.bfloat16), device="cuda")[:, :N]
+            epi = kw.get("epi", K.EPI_STORE)
+            row(f"gemm {name}", T, who, lambda: K._gemm(xx, wt, None, None, out, None, N, N, N // 2 if epi == K.EPI_SILU_MUL else N, 0, epi, 1),
+                flops=2.0 * T * N * Kd, nbytes=2.0 * (N * Kd + T * Kd) + out.element_size() * T * N)
+        gemm("projections", "gabisun q|k|g", H * D + G * D + H, W)
+        gemm("projections", "q|k|v", (H + 2 * G) * D, W)
+        gemm("up", "gabisun, GELU epilogue", s["ff"], W, epi=K.EPI_GELU_TANH)
+        gemm("up", "gate|up, SiLU epilogue", 2 * (s["ff"] * 2 // 3 // 64 * 64), W, epi=K.EPI_SILU_MUL)
+        gemm("loop entry", "gabisun, fp32 output", W, 2 * W, out_dtype=torch.float32)
+        gemm("loop entry", "bf16 output", W, 2 * W)
+    gemm("logits", "gabisun, fp32 output", VOCAB, W, out_dtype=torch.float32)
+    gemm("logits", "bf16 output", VOCAB, W)
+    return rows
+
+
+def run(steps: int, warmup: int, sizes=None, kernels: bool = True, clock_sampler=None) -> None:
+    for name, s in SIZES.items():
+        if sizes and name not in sizes:
+            continue
+        clocks = clock_sampler() if clock_sampler else None
+        models = {"Gabisun": gabisun_config(s), "Starcoder2": like_config(s, "Starcoder2ForCausalLM"), "Mistral": like_config(s, "MistralForCausalLM")}
+        res = {"design": "gabisun", "size": name, "dims": s, "dtype": "bf16", "data": "synthetic: random token ids and weights",
+               "workload": f"prefill: one {PREFILL}-token prompt a step; decode: {DECODE_REQS} requests at a context of about {DECODE_CTX}",
+               "l2": "model steps stream weights and KV larger than L2; kernels: L2 flushed before every launch",
+               "models": {k: model_throughput(c, steps, warmup) for k, c in models.items()}}
+        if kernels:
+            res["kernels"] = kernel_rows(s, max(5, steps // 6))
+        if clocks is not None:
+            res["clocks"] = clocks.stop()
+        print(json.dumps(res), flush=True)

@@ -467,13 +467,13 @@ def choose_kv_splits(base_ctas: int, max_seq: int, num_sms: int) -> int:
     return max(1, min(want, by_ctx, 32))
 
 
-def choose_decode_splits(base_ctas: int, max_seq: int, num_sms: int) -> int:
-    """KV splits of the paged decode kernel from a cost model of its waves. Two CTAs fit per SM; a CTA needs about 1.6 us to start
+def choose_decode_splits(base_ctas: int, max_seq: int, num_sms: int, per_sm: int = 2) -> int:
+    """KV splits of the paged decode kernel from a cost model of its waves. ``per_sm`` CTAs fit per SM; a CTA needs about 1.6 us to start
     and 1.9 us per 64-key tile when the SMs are full, and more than one split adds the combine launch (about 6 us). Measured on
     B200 (64 requests x 8 KV heads x 1150 keys): 71.7 us unsplit against 80.9 us in two splits, whose 1024 CTAs need four waves
     of 296 where 512 need two; 16 requests x 4096 keys: 66 us in two splits (one wave) against 83 us in three (two waves)."""
     nt = max(1, -(-max_seq // 64))
-    slots = 2 * num_sms
+    slots = per_sm * num_sms
     best, best_cost = 1, None
     for s in range(1, min(32, nt) + 1):
         per = -(-nt // s)
@@ -486,10 +486,12 @@ def choose_decode_splits(base_ctas: int, max_seq: int, num_sms: int) -> int:
     return best
 
 
-def plan_attention(query_lens: list, seq_lens: list, Hq: int, Hkv: int, D: int, num_sms: int, force_splits: int = 0, span: int = 0):
+def plan_attention(query_lens: list, seq_lens: list, Hq: int, Hkv: int, D: int, num_sms: int, force_splits: int = 0, span: int = 0,
+                   extended: bool = False):
     """Decide which requests take the decode kernel (rows = q_len * group fit in one 16/32-row tile) and how many KV
     splits it uses. Returns (short_q_len, num_q_tiles for the prefill kernel, splits). ``span`` > 0: a decode row reads at most that many
-    keys of its context (window and kept first tokens)."""
+    keys of its context (window and kept first tokens). ``extended``: the variants of the kernel with one ring of shared keys and values,
+    of which more CTAs fit per SM."""
     G = Hq // Hkv
     max_rows = 32 if D <= 128 else 16
     short = max_rows // G
@@ -501,7 +503,8 @@ def plan_attention(query_lens: list, seq_lens: list, Hq: int, Hkv: int, D: int, 
     splits = 1
     if n_short:
         max_s = max((s for q, s in zip(query_lens, seq_lens) if q <= short), default=1)
-        splits = choose_decode_splits(n_short * Hkv, min(max_s, span) if span else max_s, num_sms)
+        per_sm = {64: 5, 128: 4}.get(D, 2) if extended and short * G <= 16 else 2
+        splits = choose_decode_splits(n_short * Hkv, min(max_s, span) if span else max_s, num_sms, per_sm)
     if force_splits:
         splits = force_splits
     return short, tiles, splits
@@ -532,7 +535,8 @@ def paged_attention(q, kv_cache, md, scale, out=None, lse=None, window=0, softca
     key = (Hq, Hkv, D, attention_span(window, keep)) if extended else (Hq, Hkv, D)
     plan = getattr(md, "attn_plan", None)
     if plan is None or plan[0] != key:
-        plan = (key, plan_attention(md.query_lens_cpu, md.seq_lens_cpu, Hq, Hkv, D, _sms(q.device), span=key[3] if extended else 0))
+        plan = (key, plan_attention(md.query_lens_cpu, md.seq_lens_cpu, Hq, Hkv, D, _sms(q.device), span=key[3] if extended else 0,
+                                    extended=kv_cache.shape[1] == 1))
         md.attn_plan = plan
     short, tiles, splits = plan[1]
     n_short = sum(1 for x in md.query_lens_cpu if 0 < x <= short)
