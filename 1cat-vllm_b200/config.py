@@ -816,6 +816,9 @@ class VllmConfig:
         m, p = self.model_config, self.parallel_config
         if m.num_attention_heads % p.tensor_parallel_size:
             raise ValueError("tensor_parallel_size must divide num_attention_heads")
+        if m.residual_fp32 and (p.pipeline_parallel_size > 1 or self.speculative_config.method in ("mtp", "eagle", "eagle3")):
+            raise ValueError(f"{m.architecture}: models with an fp32 residual stream are served without pipeline parallelism and without draft heads "
+                             "that read the target's hidden states")
         if p.pipeline_parallel_size > 1:
             if p.pipeline_parallel_size > m.num_hidden_layers:
                 raise ValueError("pipeline_parallel_size exceeds the number of decoder layers")

@@ -276,3 +276,69 @@ def test_random_weights_without_a_checkpoint():
     llm = LLM(hf_config=M.CONFIGS["mixed"], dtype="float32", device="cpu", max_model_len=64)
     o = llm.generate([{"prompt_token_ids": [1, 2, 3]}], SamplingParams(temperature=0.0, max_tokens=4, ignore_eos=True, detokenize=False))
     assert len(o[0].outputs[0].token_ids) == 4
+
+
+# ------------------------------------------------------------------------------------------------ what the comparisons would catch
+def _mutate(cfg, w, what):
+    import copy
+    cfg, w = copy.deepcopy(cfg), {k: v.clone() for k, v in w.items()}
+    for i, l in enumerate(cfg["layers"]):
+        m = l["mixer"]
+        if what == "window":
+            m["mask"]["size"] += 1
+        elif what == "keep":
+            m["mask"]["keep_first"] += 1
+        elif what == "scale":
+            m["scale"] *= 1.02
+        elif what == "bias_max":
+            m["bias_max"] += 7
+        elif what in ("sink", "rel", "g"):
+            w[f"l{i}.mix.{what}"].add_(0.25)
+        elif what == "ls1":
+            w[f"l{i}.ls1"].mul_(1.05)
+    if what == "times":
+        cfg["loop"]["times"] -= 1
+    elif what == "step":
+        w["loop.step"] = w["loop.step"].flip(0)
+    elif what == "eps":
+        cfg["norm"]["eps"] *= 100
+    return cfg, w
+
+
+@pytest.mark.parametrize("what", ["window", "keep", "scale", "bias_max", "sink", "rel", "g", "ls1", "times", "step", "eps"])
+def test_mistakes_show_in_the_logits(models, what):
+    """A mistake in the restatement (a window or the kept tokens one token off, a shifted sink, a lost pass, ...) moves the logits by far
+    more than the tolerance, so the comparisons above would find the same mistake in the engine."""
+    cfg, w, _ = models["mixed"]
+    toks = M.tokens(cfg, 110, 7)
+    assert M.error(O.forward(*_mutate(cfg, w, what), toks)[0], O.forward(cfg, w, toks)[0]) > (5 if what == "eps" else 50) * TOL
+
+
+def test_ngram_drafts_keep_the_tokens(models):
+    cfg, w, path = models["plain"]
+    llm = LLM(model=path, dtype="float32", device="cpu", max_model_len=128, speculative_config=dict(method="ngram", num_speculative_tokens=3))
+    p = M.tokens(cfg, 12, 4) * 3
+    o = llm.generate([{"prompt_token_ids": p}], SamplingParams(temperature=0.0, max_tokens=30, ignore_eos=True, detokenize=False))
+    assert list(o[0].outputs[0].token_ids) == O.greedy(cfg, w, p, 30)
+
+
+@pytest.mark.timeout(300)
+def test_two_tensor_parallel_ranks(tmp_path):
+    """Query heads, bias columns, sinks and gates are split over the ranks; keys too, or replicated where a layer has one key head."""
+    cfg = M.config(64, 90, [M.layer(4, 2, 16, 24, 3, 64), M.layer(6, 1, 16, 40, 2, 96), M.layer(2, 2, 8, 9, 0, None)], loop=(0, 2, 2))
+    w = M.make_weights(cfg, 3, sharp=1.5)
+    path = M.save(cfg, w, tmp_path)
+    llm = LLM(model=path, dtype="float32", device="cpu", max_model_len=128, tensor_parallel_size=2, distributed_executor_backend="mp")
+    prompts = [M.tokens(cfg, n, n) for n in (5, 60)]
+    outs = llm.generate([{"prompt_token_ids": p} for p in prompts], SamplingParams(temperature=0.0, max_tokens=12, ignore_eos=True, detokenize=False))
+    llm.shutdown()
+    for p, o in zip(prompts, outs):
+        assert list(o.outputs[0].token_ids) == O.greedy(cfg, w, p, 12)
+
+
+def test_combinations_that_are_not_served_are_refused(models):
+    _, _, path = models["plain"]
+    for kw in (dict(pipeline_parallel_size=2), dict(kv_cache_dtype="fp8"), dict(tensor_parallel_size=2),
+               dict(speculative_config=dict(method="mtp", num_speculative_tokens=1))):
+        with pytest.raises(ValueError):
+            LLM(model=path, dtype="float32", device="cpu", max_model_len=64, **kw)
