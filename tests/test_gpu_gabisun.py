@@ -58,7 +58,7 @@ def attention_oracle(q, k, scale, mask, rel, top, sink, gate):
 
 
 CASES = [  # heads, kv heads, head size, window, keep, (new tokens, context) of each request
-    (4, 1, 64, 136, 20, [(200, 200), (1, 400), (3, 77), (64, 300), (1, 1)]),
+    (6, 2, 64, 150, 37, [(200, 200), (1, 400), (3, 77), (64, 300), (1, 1)]),
     (8, 2, 128, 100, 130, [(1, 1000), (1, 99), (2, 131), (8, 640)]),
     (8, 8, 128, 64, 0, [(33, 33), (1, 64), (1, 65), (130, 513)]),
     (6, 2, 64, 1, 1, [(70, 70), (1, 129), (2, 66)]),
