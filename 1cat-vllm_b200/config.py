@@ -108,6 +108,52 @@ def _gabisun_fields(hf: dict) -> dict:
                 layer_overrides=tuple(over), loop=(int(loop["start"]), int(loop["stop"]), int(loop["times"])) if loop else None, **top)
 
 
+def _sepirax_fields(hf: dict) -> dict:
+    """``ModelConfig`` fields of a Sepirax config.json: a list of layers, each with latent attention or an mLSTM as its mixer and an optional
+    mixture of experts, dynamic-tanh norms ahead of the sub-blocks, an fp32 residual stream whose sub-block outputs are scaled."""
+    over, types = [], []
+    for i, l in enumerate(hf["layers"]):
+        m, mlp = l["mixer"], l.get("mlp")
+        o: dict[str, Any] = dict(mixer_only_layers=mlp is None)
+        if l["type"] == "latent_attention":
+            rot = m["rot"]
+            if int(rot["dims"]) != int(m["rot_dim"]) or int(rot["dims"]) % 2:
+                raise ValueError(f"Sepirax layer {i}: the rotated part has {m['rot_dim']} dimensions, rot.dims is {rot['dims']}")
+            s = rot.get("scaling")
+            o.update(use_mla=True, num_attention_heads=int(m["heads"]), num_key_value_heads=int(m["heads"]), q_lora_rank=int(m["q_rank"]),
+                     kv_lora_rank=int(m["kv_rank"]), qk_nope_head_dim=int(m["dim"]), qk_rope_head_dim=int(m["rot_dim"]), v_head_dim=int(m["vdim"]),
+                     attn_scale=float(m["scale"]), rope_theta=float(rot["base"]),
+                     rope_scaling=dict(rope_type="yarn", factor=float(s["factor"]), original_max_position_embeddings=float(s["original"]),
+                                       beta_fast=float(s["fast"]), beta_slow=float(s["slow"])) if s else None)
+            types.append("full_attention")
+        elif l["type"] == "mlstm":
+            o.update(use_mla=False, mlstm_heads=int(m["heads"]), mlstm_key_dim=int(m["dim"]), mlstm_value_dim=int(m["vdim"]),
+                     mlstm_gate_cap=float(m["gate_cap"]), num_attention_heads=int(m["heads"]), num_key_value_heads=int(m["heads"]))
+            types.append("mlstm")
+        else:
+            raise ValueError(f"Sepirax layer {i}: mixer {l['type']!r} is not known")
+        if mlp is not None:
+            if mlp.get("kind") != "moe":
+                raise ValueError(f"Sepirax layer {i}: feed-forward {mlp.get('kind')!r} is not known")
+            r = mlp["router"]
+            g = r.get("groups") or dict(count=1, keep=1)
+            if r["experts"] % g["count"] or r["top"] > r["experts"] // g["count"] * g["keep"]:
+                raise ValueError(f"Sepirax layer {i}: {r['experts']} experts in {g['count']} groups, {g['keep']} kept, cannot give each token {r['top']}")
+            o.update(num_experts=int(r["experts"]), num_experts_per_tok=int(r["top"]), n_group=int(g["count"]), topk_group=int(g["keep"]),
+                     moe_intermediate_size=int(mlp["expert"]["ff"]))
+        over.append(o)
+    attn = [o for o in over if o["use_mla"]]
+    top: dict[str, Any] = {k: (attn or over)[0][k] for k in ("num_attention_heads", "num_key_value_heads")}
+    for k in ("q_lora_rank", "kv_lora_rank", "qk_nope_head_dim", "qk_rope_head_dim", "v_head_dim"):
+        if attn:
+            top[k] = attn[0][k]
+    return dict(architecture="Sepirax", vocab_size=int(hf["vocab"]), hidden_size=int(hf["width"]), num_hidden_layers=len(over),
+                rms_norm_eps=float(hf["norm"]["eps"]), norm_type="dyt", residual_fp32=True, residual_multiplier=float(hf["residual_mult"]),
+                embed_scale=float(hf["embedding"]["scale"]), final_softcap=float(hf.get("logit_softcap") or 0.0), use_mla=bool(attn),
+                mla_rope_half=True, mla_fused_in=True, attn_output_gate=True, router_fp32=True, norm_topk_prob=True, layer_types=types,
+                num_experts=max((o.get("num_experts", 0) for o in over), default=0), layer_overrides=tuple(over), **top)
+
+
 @dataclass
 class ModelConfig:
     """Architecture description, normalised from an HF ``config.json`` (or a dict for synthetic models).
@@ -152,7 +198,9 @@ class ModelConfig:
     attn_sinks: bool = False  # one learned sink logit per query head joins the softmax denominator (GPT-OSS)
     attn_o_bias: bool = False  # bias on the attention output projection
     mlp_bias: bool = False  # biases on the dense feed-forward projections (Llama / Granite ``mlp_bias``)
-    norm_type: str = "rms"  # rms | layernorm (mean-and-variance normalisation; ``gemma_norm`` then means the weight is stored minus one)
+    # rms | layernorm (mean-and-variance normalisation; ``gemma_norm`` then means the weight is stored minus one) | dyt (dynamic tanh:
+    # tanh(alpha * x) * w + b, no statistics of the row)
+    norm_type: str = "rms"
     norm_affine: bool = True  # False: the layer norm has no learned parameters (OLMo)
     norm_bias: bool = False  # the layer norm has a bias
     parallel_block: bool = False  # h += attn(norm(h)) + mlp(norm(h)) with one norm per block (Cohere)
@@ -174,11 +222,12 @@ class ModelConfig:
     attn_rel_buckets: int = 0  # > 0: a learned bias per (distance bucket, head) is added to the scores; a checkpoint's table sets the row count
     attn_rel_max: int = 0  # distance at which the last bucket begins
     layer_scale: bool = False  # a sub-block's (normalised) output is multiplied by a learned vector before it joins the residual
+    router_fp32: bool = False  # router logits stay in the accumulator's precision
     residual_fp32: bool = False  # the residual stream is carried in fp32 (fused join kernel); logits are fp32 as well
     loop: Optional[tuple] = None  # (start, stop, times): layers start..stop-1 run ``times`` times in a row with the same weights
     num_labels: int = 0  # > 0: a *ForSequenceClassification checkpoint (a ``score`` head on the pooled state instead of an LM head)
     # hybrid (Gated-DeltaNet)
-    layer_types: Optional[list[str]] = None  # "full_attention" | "linear_attention" (Gated-DeltaNet) | "mamba2" | "mamba1" | "short_conv"
+    layer_types: Optional[list[str]] = None  # "full_attention" | "linear_attention" (Gated-DeltaNet) | "mamba2" | "mamba1" | "short_conv" | "mlstm"
     # Mamba-2 mixers (Bamba, Mamba2): heads x head size = inner width; B / C groups of the state size; conv kernel
     mamba_n_heads: int = 0
     mamba_d_head: int = 64
@@ -198,6 +247,11 @@ class ModelConfig:
     linear_key_head_dim: int = 128
     linear_value_head_dim: int = 128
     linear_conv_kernel_dim: int = 4
+    # mLSTM mixers: matrix memory [key size, value size] per head, exponential gates whose logits are soft-capped
+    mlstm_heads: int = 0
+    mlstm_key_dim: int = 0
+    mlstm_value_dim: int = 0
+    mlstm_gate_cap: float = 15.0
     # MoE
     num_experts: int = 0
     num_experts_per_tok: int = 0
@@ -218,6 +272,8 @@ class ModelConfig:
     qk_nope_head_dim: int = 0
     qk_rope_head_dim: int = 0
     v_head_dim: int = 0
+    mla_rope_half: bool = False  # rotary pairs are (i, i + rope/2) instead of (2i, 2i + 1)
+    mla_fused_in: bool = False  # query latent, key/value latent (and output gate) are one projection of the input
     # MTP draft head
     num_nextn_predict_layers: int = 0
     # runtime
@@ -252,7 +308,7 @@ class ModelConfig:
     # ---- derived
     @property
     def is_hybrid(self) -> bool:
-        return bool(self.layer_types) and any(t in ("linear_attention", "mamba2", "mamba1", "short_conv") for t in self.layer_types)
+        return bool(self.layer_types) and any(t in ("linear_attention", "mamba2", "mamba1", "short_conv", "mlstm") for t in self.layer_types)
 
     @property
     def is_moe(self) -> bool:
@@ -311,6 +367,8 @@ class ModelConfig:
         over = dict(over)
         if hf.get("architecture") == "Gabisun" or "Gabisun" in (hf.get("architectures") or ()):
             return cls(**{**_gabisun_fields(hf), **over})
+        if hf.get("architecture") == "Sepirax" or "Sepirax" in (hf.get("architectures") or ()):
+            return cls(**{**_sepirax_fields(hf), **over})
         mm_ids = {m: int(hf[k]) for m, k in (("image", "image_token_id"), ("video", "video_token_id"), ("audio", "audio_token_id")) if hf.get(k) is not None}
         if mm_ids:
             over.setdefault("mm_token_ids", mm_ids)

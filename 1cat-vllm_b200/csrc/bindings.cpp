@@ -330,7 +330,8 @@ void kv_insert(torch::Tensor k, c10::optional<torch::Tensor> v, torch::Tensor ca
 void stream_join(torch::Tensor part, c10::optional<torch::Tensor> x_in, torch::Tensor x_out, int64_t post_kind, c10::optional<torch::Tensor> post_w,
                  c10::optional<torch::Tensor> post_b, double post_eps, bool post_plus, c10::optional<torch::Tensor> scale, int64_t next_kind,
                  c10::optional<torch::Tensor> next_w, c10::optional<torch::Tensor> next_b, double next_eps, bool next_plus, c10::optional<torch::Tensor> y,
-                 c10::optional<torch::Tensor> add, c10::optional<torch::Tensor> copy_out, bool f32) {
+                 c10::optional<torch::Tensor> add, c10::optional<torch::Tensor> copy_out, bool f32, double mul, c10::optional<torch::Tensor> post_alpha,
+                 c10::optional<torch::Tensor> next_alpha) {
   const auto et = f32 ? torch::kFloat32 : torch::kBFloat16;
   TORCH_CHECK(part.is_cuda() && part.dim() == 2 && part.stride(1) == 1, "part must be a CUDA [T, H] matrix with unit inner stride");
   TORCH_CHECK(part.scalar_type() == torch::kFloat32 || part.scalar_type() == et, "part must be fp32 or of the model's type");
@@ -339,6 +340,11 @@ void stream_join(torch::Tensor part, c10::optional<torch::Tensor> x_in, torch::T
   auto vec = [&](const c10::optional<torch::Tensor>& t, const char* name) -> const void* {
     if (!t.has_value()) return nullptr;
     TORCH_CHECK(t->is_cuda() && t->scalar_type() == et && t->is_contiguous() && t->numel() == H, name, " must be a contiguous [H] vector of the model's type");
+    return t->data_ptr();
+  };
+  auto num = [&](const c10::optional<torch::Tensor>& t) -> const void* {
+    if (!t.has_value()) return nullptr;
+    TORCH_CHECK(t->is_cuda() && t->scalar_type() == et && t->numel() == 1, "alpha must be one element of the model's type");
     return t->data_ptr();
   };
   auto mat = [&](const torch::Tensor& t, c10::ScalarType ty, const char* name) {
@@ -354,8 +360,9 @@ void stream_join(torch::Tensor part, c10::optional<torch::Tensor> x_in, torch::T
     mat(*x_in, torch::kFloat32, "x_in");
     p.x_in = x_in->data_ptr<float>();
   }
-  p.post = {(int)post_kind, post_plus ? 1 : 0, vec(post_w, "post weight"), vec(post_b, "post bias"), (float)post_eps};
-  p.next = {(int)next_kind, next_plus ? 1 : 0, vec(next_w, "next weight"), vec(next_b, "next bias"), (float)next_eps};
+  p.post = {(int)post_kind, post_plus ? 1 : 0, vec(post_w, "post weight"), vec(post_b, "post bias"), (float)post_eps, num(post_alpha)};
+  p.next = {(int)next_kind, next_plus ? 1 : 0, vec(next_w, "next weight"), vec(next_b, "next bias"), (float)next_eps, num(next_alpha)};
+  p.mul = (float)mul;
   p.scale = vec(scale, "scale");
   p.add = vec(add, "add");
   if (y.has_value()) {
@@ -556,22 +563,24 @@ torch::Tensor rejection_sample(torch::Tensor draft_ids, torch::Tensor num_draft,
 
 std::tuple<torch::Tensor, torch::Tensor> route(torch::Tensor logits, c10::optional<torch::Tensor> bias, int64_t k, int64_t n_group, int64_t topk_group,
                                                bool sigmoid, bool renormalize, double scaling) {
-  check_bf16(logits, "router logits");
+  TORCH_CHECK(logits.is_cuda() && (logits.scalar_type() == torch::kBFloat16 || logits.scalar_type() == torch::kFloat32), "router logits must be bf16 or fp32");
   TORCH_CHECK(logits.dim() == 2 && logits.stride(1) == 1, "router logits must be [T, E]");
   const c10::cuda::CUDAGuard guard(logits.device());
   const int T = (int)logits.size(0);
   auto w = torch::empty({T, k}, logits.options().dtype(torch::kFloat32));
   auto ids = torch::empty({T, k}, logits.options().dtype(torch::kInt32));
   oc::RouteParams p{};
-  p.logits = (const __nv_bfloat16*)logits.data_ptr();
+  p.logits = logits.data_ptr();
+  p.is_fp32 = logits.scalar_type() == torch::kFloat32;
   p.ld = logits.stride(0);
+  TORCH_CHECK(!bias.has_value() || (bias->scalar_type() == torch::kFloat32 && bias->is_contiguous() && bias->numel() == logits.size(1)), "bias must be fp32 [E]");
   p.bias = bias.has_value() ? bias->data_ptr<float>() : nullptr;
   p.topk_w = w.data_ptr<float>();
   p.topk_ids = ids.data_ptr<int>();
   p.T = T; p.E = (int)logits.size(1); p.k = (int)k; p.n_group = (int)n_group; p.topk_group = (int)topk_group;
   p.sigmoid = sigmoid ? 1 : 0; p.renormalize = renormalize ? 1 : 0; p.scaling = (float)scaling;
   int rc = oc::route_launch(p, cur_stream());
-  TORCH_CHECK(rc == 0, "router launch failed (needs E % 32 == 0, E <= 512, k <= 16)");
+  TORCH_CHECK(rc == 0, "router launch failed (needs E <= 512, k <= 16)");
   return {w, ids};
 }
 
@@ -615,10 +624,11 @@ torch::Tensor fused_moe(torch::Tensor x, torch::Tensor w13, torch::Tensor w2, to
   TORCH_CHECK(topk_ids.scalar_type() == torch::kInt32 && topk_ids.is_contiguous() && topk_w.scalar_type() == torch::kFloat32 && topk_w.is_contiguous(),
               "routing tensors must be contiguous int32 ids / fp32 weights");
   const c10::cuda::CUDAGuard guard(x.device());
-  const int T = (int)x.size(0), H = (int)x.size(1), k = (int)topk_ids.size(1);
+  // expert weights may be padded with zeros to the kernel's tiles: Hp >= H columns of w13 and rows of w2
+  const int T = (int)x.size(0), H = (int)x.size(1), k = (int)topk_ids.size(1), Hp = wkind == 0 ? (int)w13.size(1) : H;
   const int I2 = wkind == 0 ? (int)(w13.size(0) / E_local) : (int)I2_packed, I = I2 / 2;
   if (wkind == 0) {
-    TORCH_CHECK(w13.size(1) == H && w2.size(0) == E_local * H && w2.size(1) == I, "expert weight shapes do not match");
+    TORCH_CHECK(w13.size(1) == Hp && w2.size(0) == E_local * Hp && w2.size(1) == I, "expert weight shapes do not match");
   } else {
     const size_t tb = wkind == 2 ? 8192 : 4096;
     TORCH_CHECK((size_t)w13.numel() * w13.element_size() >= (size_t)(E_local * I2 / 128) * (H / 64) * tb &&
@@ -626,20 +636,20 @@ torch::Tensor fused_moe(torch::Tensor x, torch::Tensor w13, torch::Tensor w2, to
     TORCH_CHECK((size_t)w13_sz->numel() >= (size_t)((H / 64 + group_ktiles - 1) / group_ktiles) * E_local * I2 &&
                 (size_t)w2_sz->numel() >= (size_t)((I / 64 + group_ktiles - 1) / group_ktiles) * E_local * H, "expert scale tables are too small");
   }
-  TORCH_CHECK(I2 % 128 == 0 && H % 128 == 0 && H % 64 == 0 && I % 64 == 0, "expert dims must be multiples of 128 (rows) and 64 (k)");
+  TORCH_CHECK(Hp >= H && I2 % 128 == 0 && Hp % 128 == 0 && I % 64 == 0, "expert dims must be multiples of 128 (rows) and 64 (k)");
   auto y = torch::empty({T, H}, x.options());
   if (T == 0) return y;
   const int n_pairs = T * k;
   const int avg = (n_pairs + (int)E_local - 1) / (int)E_local;
   const int tn = avg <= 32 ? 32 : avg <= 64 ? 64 : (avg <= 128 || wkind != 0) ? 128 : 256;  // packed kinds share TMEM with the weight ring
-  const int n1 = I2 / 128, n2 = H / 128;
+  const int n1 = I2 / 128, n2 = Hp / 128;
   const int max_tt = (n_pairs + tn - 1) / tn + (int)E_local;
   auto iopt = x.options().dtype(torch::kInt32);
   auto meta = torch::empty({3 * E_local + 8 + n_pairs}, iopt);
   auto work = torch::empty({(int64_t)max_tt * (n1 + n2) * 4}, iopt);
-  auto xs = torch::empty({n_pairs, H}, x.options());
+  auto xs = torch::empty({n_pairs, Hp}, x.options());
   auto a1 = torch::empty({n_pairs, I}, x.options());
-  auto a2 = torch::empty({n_pairs, H}, x.options());
+  auto a2 = torch::empty({n_pairs, Hp}, x.options());
   int* mp = meta.data_ptr<int>();
   oc::MoePlanParams pp{};
   pp.counts = mp; pp.offsets = mp + E_local; pp.cursor = mp + 2 * E_local + 1; pp.total_slots = mp + 3 * E_local + 1; pp.work_count = mp + 3 * E_local + 2;
@@ -648,16 +658,48 @@ torch::Tensor fused_moe(torch::Tensor x, torch::Tensor w13, torch::Tensor w2, to
   pp.work2 = pp.work1 + (size_t)max_tt * n1;
   TORCH_CHECK(((uintptr_t)pp.work2 & 15) == 0, "work list alignment");
   pp.E = (int)E_local; pp.tn = tn; pp.n1 = n1; pp.n2 = n2;
-  int rc = oc::moe_prepare_launch(pp, topk_ids.data_ptr<int>(), n_pairs, k, (int)e_off, slot_of, x.data_ptr(), x.stride(0), xs.data_ptr(), H, cur_stream());
+  int rc = oc::moe_prepare_launch(pp, topk_ids.data_ptr<int>(), n_pairs, k, (int)e_off, slot_of, x.data_ptr(), x.stride(0), xs.data_ptr(), H, Hp, 0,
+                                  cur_stream());
   TORCH_CHECK(rc == 0, "moe prepare failed: ", rc);
   auto run = [&](const torch::Tensor& in, const torch::Tensor& w, const c10::optional<torch::Tensor>& sz, int n_rows, torch::Tensor& out, int Kd, int N,
                  int n_out, int epi, const int4* wl, const int* cnt, int cap) {
     moe_gemm_run(in, w, sz, n_rows, out, Kd, N, n_out, epi, wl, cnt, cap, n_pairs, tn, (int)wkind, (int)group_ktiles, counters);
   };
-  run(xs, w13, w13_sz, (int)E_local * I2, a1, H, I2, I, oc::EPI_SILU_MUL, pp.work1, pp.work_count, max_tt * n1);
-  run(a1, w2, w2_sz, (int)E_local * H, a2, I, H, H, oc::EPI_STORE, pp.work2, pp.work_count + 1, max_tt * n2);
-  rc = oc::moe_combine_launch(a2.data_ptr(), slot_of, topk_w.data_ptr<float>(), y.data_ptr(), T, k, H, cur_stream());
+  run(xs, w13, w13_sz, (int)E_local * I2, a1, Hp, I2, I, oc::EPI_SILU_MUL, pp.work1, pp.work_count, max_tt * n1);
+  run(a1, w2, w2_sz, (int)E_local * Hp, a2, I, Hp, Hp, oc::EPI_STORE, pp.work2, pp.work_count + 1, max_tt * n2);
+  rc = oc::moe_combine_launch(a2.data_ptr(), Hp, slot_of, topk_w.data_ptr<float>(), y.data_ptr(), T, k, H, 0, cur_stream());
   TORCH_CHECK(rc == 0, "moe combine failed");
+  return y;
+}
+
+// The same layer in fp32 (engines that run in 32 bits): w13 [E_local, 2I, H] gate rows then up rows, w2 [E_local, H, I], any sizes.
+torch::Tensor fused_moe_f32(torch::Tensor x, torch::Tensor w13, torch::Tensor w2, torch::Tensor topk_w, torch::Tensor topk_ids, int64_t e_off) {
+  for (auto* t : {&x, &w13, &w2, &topk_w}) TORCH_CHECK(t->is_cuda() && t->scalar_type() == torch::kFloat32 && t->is_contiguous(), "contiguous fp32 CUDA tensors");
+  TORCH_CHECK(topk_ids.scalar_type() == torch::kInt32 && topk_ids.is_contiguous() && topk_ids.sizes() == topk_w.sizes(), "routing tensors");
+  const c10::cuda::CUDAGuard guard(x.device());
+  const int T = (int)x.size(0), H = (int)x.size(1), k = (int)topk_ids.size(1), E = (int)w13.size(0), I = (int)w2.size(2), n_pairs = T * k;
+  TORCH_CHECK(w13.dim() == 3 && w2.dim() == 3 && w13.size(1) == 2 * I && w13.size(2) == H && w2.size(0) == E && w2.size(1) == H && topk_ids.size(0) == T,
+              "expert weight shapes do not match");
+  auto y = torch::empty({T, H}, x.options());
+  if (T == 0) return y;
+  const int tn = 64, n1 = (2 * I + 127) / 128, n2 = (H + 127) / 128, max_tt = (n_pairs + tn - 1) / tn + E;
+  auto iopt = x.options().dtype(torch::kInt32);
+  auto meta = torch::empty({3 * E + 8 + n_pairs}, iopt);
+  auto work = torch::empty({(int64_t)max_tt * (n1 + n2) * 4}, iopt);
+  auto xs = torch::empty({n_pairs, H}, x.options()), a1 = torch::empty({n_pairs, 2 * I}, x.options()), a2 = torch::empty({n_pairs, H}, x.options());
+  int* mp = meta.data_ptr<int>();
+  oc::MoePlanParams pp{};
+  pp.counts = mp; pp.offsets = mp + E; pp.cursor = mp + 2 * E + 1; pp.total_slots = mp + 3 * E + 1; pp.work_count = mp + 3 * E + 2;
+  int* slot_of = mp + 3 * E + 8;
+  pp.work1 = (int4*)work.data_ptr<int>();
+  pp.work2 = pp.work1 + (size_t)max_tt * n1;
+  pp.E = E; pp.tn = tn; pp.n1 = n1; pp.n2 = n2;
+  auto st = cur_stream();
+  TORCH_CHECK(oc::moe_prepare_launch(pp, topk_ids.data_ptr<int>(), n_pairs, k, (int)e_off, slot_of, x.data_ptr(), H, xs.data_ptr(), H, H, 1, st) == 0, "moe prepare failed");
+  TORCH_CHECK(oc::moe_gemm_f32_launch(xs.data_ptr<float>(), H, w13.data_ptr<float>(), a1.data_ptr<float>(), 2 * I, H, 0, pp.work1, pp.work_count, n1, sm_count(), st) == 0 &&
+              oc::moe_gemm_f32_launch(a1.data_ptr<float>(), 2 * I, w2.data_ptr<float>(), a2.data_ptr<float>(), H, I, 1, pp.work2, pp.work_count + 1, n2, sm_count(), st) == 0,
+              "fp32 grouped gemm failed");
+  TORCH_CHECK(oc::moe_combine_launch(a2.data_ptr(), H, slot_of, topk_w.data_ptr<float>(), y.data_ptr(), T, k, H, 1, st) == 0, "moe combine failed");
   return y;
 }
 
@@ -726,18 +768,26 @@ torch::Tensor fused_moe_a2a(torch::Tensor x, torch::Tensor w13, torch::Tensor w2
 
 torch::Tensor mla_decode(torch::Tensor q_abs, torch::Tensor q_rope, torch::Tensor cache, torch::Tensor qsl, torch::Tensor seq_lens,
                          torch::Tensor block_table, double scale, int64_t max_q_len, int64_t splits, c10::optional<torch::Tensor> ws_o,
-                         c10::optional<torch::Tensor> ws_ml) {
-  check_bf16(q_abs, "q_abs");
-  check_bf16(q_rope, "q_rope");
-  check_bf16(cache, "latent cache");
-  TORCH_CHECK(q_abs.is_contiguous() && q_rope.is_contiguous() && cache.is_contiguous() && cache.dim() == 3, "q and cache must be contiguous");
+                         c10::optional<torch::Tensor> ws_ml, c10::optional<torch::Tensor> cos_sin, bool interleaved, bool fine) {
+  const auto et = q_abs.scalar_type();
+  TORCH_CHECK(q_abs.is_cuda() && (et == torch::kBFloat16 || et == torch::kFloat32) && q_rope.scalar_type() == et && cache.scalar_type() == et, "bf16 or fp32 throughout");
+  TORCH_CHECK(q_abs.is_contiguous() && cache.is_contiguous() && cache.dim() == 3 && q_rope.dim() == 3 && q_rope.stride(2) == 1, "q and cache layouts");
+  TORCH_CHECK(qsl.scalar_type() == torch::kInt32 && seq_lens.scalar_type() == torch::kInt32 && block_table.scalar_type() == torch::kInt32, "metadata must be int32");
   const c10::cuda::CUDAGuard guard(q_abs.device());
   oc::MlaParams p{};
   p.T = (int)q_abs.size(0); p.H = (int)q_abs.size(1); p.kv_lora = (int)q_abs.size(2); p.rope = (int)q_rope.size(2);
-  TORCH_CHECK(cache.size(2) == p.kv_lora + p.rope, "cache width must be kv_lora + rope");
+  p.rope_pad = (int)cache.size(2) - p.kv_lora;
+  TORCH_CHECK(p.rope_pad >= p.rope && q_rope.size(0) == p.T && q_rope.size(1) == p.H, "a cached row is the latent and the shared key part");
+  p.f32 = et == torch::kFloat32;
   auto out = torch::empty({p.T, p.H, p.kv_lora}, q_abs.options());
-  p.q_abs = (const __nv_bfloat16*)q_abs.data_ptr(); p.q_rope = (const __nv_bfloat16*)q_rope.data_ptr();
-  p.cache = (const __nv_bfloat16*)cache.data_ptr(); p.out = (__nv_bfloat16*)out.data_ptr();
+  p.q_abs = q_abs.data_ptr(); p.q_rope = q_rope.data_ptr(); p.qr_st = q_rope.stride(0); p.qr_sh = q_rope.stride(1);
+  if (cos_sin.has_value()) {
+    TORCH_CHECK(cos_sin->is_cuda() && cos_sin->scalar_type() == torch::kFloat32 && cos_sin->is_contiguous() && cos_sin->size(1) == p.rope && p.rope % 2 == 0, "cos_sin must be fp32 [positions, rope]");
+    p.cos_sin = cos_sin->data_ptr<float>();
+  }
+  p.interleaved = interleaved ? 1 : 0;
+  p.fine = fine ? 1 : 0;
+  p.cache = cache.data_ptr(); p.out = out.data_ptr();
   p.query_start_loc = qsl.data_ptr<int>(); p.seq_lens = seq_lens.data_ptr<int>(); p.block_table = block_table.data_ptr<int>();
   p.bt_stride = (int)block_table.stride(0); p.R = (int)seq_lens.size(0);
   p.bs = (int)cache.size(1); p.bs_shift = 0;
@@ -749,8 +799,109 @@ torch::Tensor mla_decode(torch::Tensor q_abs, torch::Tensor q_rope, torch::Tenso
     p.ws_o = ws_o->data_ptr<float>(); p.ws_ml = ws_ml->data_ptr<float>();
   }
   int rc = oc::mla_decode_launch(p, cur_stream());
-  TORCH_CHECK(rc == 0, "mla decode launch failed: ", rc, " (needs kv_lora 512, rope 64)");
+  TORCH_CHECK(rc == 0, "latent attention launch failed: ", rc, " (latents up to 1024)");
   return out;
+}
+
+bool mla_tensor_core_sizes(int64_t kv_lora, int64_t rope_pad) { return oc::mla_tensor_core_sizes((int)kv_lora, (int)rope_pad); }
+
+// Latent norms, rotation of the shared key part, cache insert; returns the normalised query latent when there is one.
+c10::optional<torch::Tensor> mla_prepare(c10::optional<torch::Tensor> q, torch::Tensor kv, c10::optional<torch::Tensor> q_w, torch::Tensor kv_w, double eps,
+                                         torch::Tensor positions, torch::Tensor cos_sin, torch::Tensor cache, torch::Tensor slots, int64_t lora,
+                                         int64_t lora_pad, bool interleaved) {
+  const auto et = kv.scalar_type();
+  TORCH_CHECK(kv.is_cuda() && (et == torch::kBFloat16 || et == torch::kFloat32) && kv.dim() == 2 && kv.stride(1) == 1 && cache.scalar_type() == et && cache.is_contiguous(),
+              "latents and cache must be bf16 or fp32");
+  const c10::cuda::CUDAGuard guard(kv.device());
+  oc::MlaPrepareParams p{};
+  p.T = (int)kv.size(0); p.lora = (int)lora; p.lora_pad = (int)lora_pad; p.rope = (int)(kv.size(1) - lora); p.width = (int)cache.size(cache.dim() - 1);
+  TORCH_CHECK(lora > 0 && lora_pad >= lora && p.rope >= 2 && p.rope % 2 == 0 && p.width >= lora_pad + p.rope, "latent sizes do not fit the cache rows");
+  TORCH_CHECK(kv_w.scalar_type() == et && kv_w.is_contiguous() && kv_w.numel() == lora, "norm weight of the key/value latent");
+  TORCH_CHECK(positions.scalar_type() == torch::kInt32 && slots.scalar_type() == torch::kInt32 && positions.numel() >= p.T && slots.numel() >= p.T, "positions and slots must be int32 [T]");
+  TORCH_CHECK(cos_sin.scalar_type() == torch::kFloat32 && cos_sin.is_contiguous() && cos_sin.size(1) == p.rope, "cos_sin must be fp32 [positions, rope]");
+  p.kv = kv.data_ptr(); p.ld_kv = kv.stride(0); p.kv_w = kv_w.data_ptr(); p.eps = (float)eps;
+  p.positions = positions.data_ptr<int>(); p.slots = slots.data_ptr<int>(); p.cos_sin = cos_sin.data_ptr<float>(); p.cache = cache.data_ptr();
+  p.interleaved = interleaved ? 1 : 0;
+  p.f32 = et == torch::kFloat32;
+  c10::optional<torch::Tensor> out;
+  if (q.has_value()) {
+    TORCH_CHECK(q->scalar_type() == et && q->dim() == 2 && q->stride(1) == 1 && q->size(0) == p.T && q_w.has_value() && q_w->scalar_type() == et && q_w->is_contiguous() &&
+                q_w->numel() == q->size(1), "query latent and its norm weight");
+    p.q = q->data_ptr(); p.ld_q = q->stride(0); p.q_w = q_w->data_ptr(); p.nq = (int)q->size(1);
+    out = torch::empty({p.T, p.nq}, q->options());
+    p.q_out = out->data_ptr();
+  }
+  TORCH_CHECK(oc::mla_prepare_launch(p, cur_stream()) == 0, "mla_prepare failed");
+  return out;
+}
+
+// mLSTM recurrence with head norm and output gate. chunk_meta (int32, one row per segment of the step's chunk list):
+// [chunk_req | chunk_t0 | chunk_long | long_req | long_chunk0 | long_n], counts given by `segments` as (offset, chunks, sequences).
+torch::Tensor mlstm(torch::Tensor x, torch::Tensor gates, torch::Tensor i_bias, torch::Tensor f_bias, torch::Tensor norm_w, double eps, double cap, int64_t H,
+                    int64_t D, int64_t V, torch::Tensor S, torch::Tensor n, torch::Tensor m, torch::Tensor qsl, torch::Tensor slots, torch::Tensor has_init,
+                    c10::optional<torch::Tensor> chunk_meta, std::vector<std::vector<int64_t>> segments, int64_t chunk_min_len, bool any_short) {
+  const auto et = x.scalar_type();
+  TORCH_CHECK(x.is_cuda() && (et == torch::kBFloat16 || et == torch::kFloat32) && x.dim() == 2 && x.stride(1) == 1 && x.size(1) == 2 * H * (D + V), "x must be [T, q | k | v | gate]");
+  TORCH_CHECK(gates.scalar_type() == torch::kFloat32 && gates.dim() == 2 && gates.size(0) == x.size(0) && gates.size(1) == 2 * H && gates.stride(1) == 1, "gates must be fp32 [T, 2H]");
+  for (auto* t : {&S, &n, &m, &i_bias, &f_bias}) TORCH_CHECK(t->is_cuda() && t->scalar_type() == torch::kFloat32 && t->is_contiguous(), "states and gate biases must be contiguous fp32");
+  TORCH_CHECK(S.dim() == 4 && S.size(1) == H && S.size(2) == D && S.size(3) == V && n.dim() == 3 && n.size(0) == S.size(0) && n.size(1) == H && n.size(2) == D &&
+              m.dim() == 2 && m.size(0) == S.size(0) && m.size(1) == H && i_bias.numel() == H && f_bias.numel() == H, "state shapes");
+  TORCH_CHECK(norm_w.scalar_type() == et && norm_w.is_contiguous() && norm_w.numel() == H * V, "norm weight");
+  TORCH_CHECK(qsl.scalar_type() == torch::kInt32 && slots.scalar_type() == torch::kInt32 && has_init.scalar_type() == torch::kInt32, "metadata must be int32");
+  const c10::cuda::CUDAGuard guard(x.device());
+  oc::MlstmParams p{};
+  p.T = (int)x.size(0); p.R = (int)slots.size(0); p.H = (int)H; p.D = (int)D; p.V = (int)V;
+  auto out = torch::empty({p.T, H * V}, x.options());
+  if (p.T == 0) return out;
+  p.x = x.data_ptr(); p.ld = x.stride(0); p.gates = gates.data_ptr<float>(); p.ld_g = gates.stride(0);
+  p.i_bias = i_bias.data_ptr<float>(); p.f_bias = f_bias.data_ptr<float>(); p.norm_w = norm_w.data_ptr();
+  p.eps = (float)eps; p.cap = (float)cap; p.scale = 1.f / std::sqrt((float)D);
+  p.S = S.data_ptr<float>(); p.n = n.data_ptr<float>(); p.m = m.data_ptr<float>(); p.out = out.data_ptr();
+  p.query_start_loc = qsl.data_ptr<int>(); p.state_slots = slots.data_ptr<int>(); p.has_initial_state = has_init.data_ptr<int>();
+  p.f32 = et == torch::kFloat32;
+  p.skip_min_len = segments.empty() ? 0 : (int)chunk_min_len;
+  auto st = cur_stream();
+  if (segments.empty() || any_short) {
+    const int rc = oc::mlstm_recurrent_launch(p, st);
+    TORCH_CHECK(rc == 0, "mlstm recurrence launch failed: ", rc, " (key and value sizes up to 512)");
+  }
+  if (segments.empty()) return out;
+  TORCH_CHECK(chunk_meta.has_value() && chunk_meta->scalar_type() == torch::kInt32 && chunk_meta->is_contiguous(), "chunk metadata must be int32");
+  int64_t most = 0;
+  for (auto& g : segments) {
+    TORCH_CHECK(g.size() == 3 && g[0] >= 0 && g[0] + 3 * (g[1] + g[2]) <= chunk_meta->numel(), "chunk metadata too small");
+    most = std::max(most, g[1]);
+  }
+  auto fopt = x.options().dtype(torch::kFloat32);
+  auto ws = torch::empty({most * H * (D * V + D + 3)}, fopt);
+  auto planes = torch::empty({most * H * 2 * D * V}, x.options().dtype(torch::kBFloat16));
+  p.ws_s = ws.data_ptr<float>();
+  p.ws_n = p.ws_s + most * H * D * V;
+  p.ws_g = p.ws_n + most * H * D;
+  p.ws_m = p.ws_g + most * H * 2;
+  p.ws_h = (__nv_bfloat16*)planes.data_ptr();
+  const bool rows16 = p.ld % 8 == 0 && ((uintptr_t)p.x & 15) == 0;
+  p.vec_qk = rows16 && D % 8 == 0;
+  p.vec_v = rows16 && D % 8 == 0 && V % 8 == 0;   // the value and gate columns start at 2 H D (+ H V)
+  for (auto& g : segments) {
+    const int* mp = chunk_meta->data_ptr<int>() + g[0];
+    p.chunk_req = mp; p.chunk_t0 = mp + g[1]; p.chunk_long = mp + 2 * g[1];
+    p.long_req = mp + 3 * g[1]; p.long_chunk0 = p.long_req + g[2]; p.long_n = p.long_chunk0 + g[2];
+    const int rc = oc::mlstm_chunk_launch(p, (int)g[1], (int)g[2], st);
+    TORCH_CHECK(rc == 0, "mlstm chunk launch failed: ", rc);
+  }
+  return out;
+}
+bool mlstm_chunkable(int64_t D, int64_t V) { return oc::mlstm_chunkable((int)D, (int)V); }
+
+torch::Tensor sigmoid_mul(torch::Tensor x, torch::Tensor gate) {
+  TORCH_CHECK(x.is_cuda() && (x.scalar_type() == torch::kBFloat16 || x.scalar_type() == torch::kFloat32) && gate.scalar_type() == x.scalar_type() && x.dim() == 2 &&
+              gate.sizes() == x.sizes() && x.stride(1) == 1 && gate.stride(1) == 1, "x and gate must be [T, n] of one type with unit inner stride");
+  const c10::cuda::CUDAGuard guard(x.device());
+  auto y = torch::empty({x.size(0), x.size(1)}, x.options());
+  TORCH_CHECK(oc::sigmoid_mul_launch(x.data_ptr(), x.stride(0), gate.data_ptr(), gate.stride(0), y.data_ptr(), (int)x.size(0), (int)x.size(1),
+                                     x.scalar_type() == torch::kFloat32, cur_stream()) == 0, "sigmoid_mul failed");
+  return y;
 }
 
 // Enqueues one small copy per translation unit's status word into `pinned` (int32, >= 16 entries, pinned host memory) on the current
@@ -864,6 +1015,12 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("read_status", &read_status);
   m.def("read_status_async", &read_status_async);
   m.def("mla_decode", &mla_decode);
+  m.def("mla_tensor_core_sizes", &mla_tensor_core_sizes);
+  m.def("mla_prepare", &mla_prepare);
+  m.def("mlstm", &mlstm);
+  m.def("mlstm_chunkable", &mlstm_chunkable);
+  m.def("sigmoid_mul", &sigmoid_mul);
+  m.def("fused_moe_f32", &fused_moe_f32);
   m.def("fused_moe", &fused_moe);
   m.def("fused_moe_a2a", &fused_moe_a2a);
   m.def("rejection_sample", &rejection_sample);

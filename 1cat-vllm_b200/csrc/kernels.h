@@ -45,6 +45,7 @@ struct StreamNorm {
   int kind, plus_one;
   const void *w, *b;            // null: ones / zeros
   float eps;
+  const void* alpha;            // dynamic tanh: the scalar inside
 };
 struct StreamJoinParams {
   const void* part;             // [T][H], pitch ld_part
@@ -54,6 +55,7 @@ struct StreamJoinParams {
   float* x_out;                 // [T][H], may be x_in
   StreamNorm post, next;
   const void *scale, *add;      // [H] or null
+  float mul;                    // number on the normalised, scaled part
   void* y;                      // [T][H] in the model's element type, or null (next.kind 0)
   void* copy_out;               // x' in the model's element type, pitch ld_copy, or null
   long long ld_copy;
@@ -139,12 +141,14 @@ struct SampleParams {
 int sample_launch(const SampleParams& p, cudaStream_t st);
 
 struct RouteParams {
-  const __nv_bfloat16* logits;  // [T][ld]
+  const void* logits;           // [T][ld] bf16 or fp32
+  int is_fp32;
   long long ld;
   const float* bias;            // e_score_correction_bias [E] or null
   float* topk_w;                // [T][k]
   int* topk_ids;                // [T][k]
   int T, E, k, n_group, topk_group, sigmoid, renormalize;
+  int whole_lanes;              // filled by the launcher: a group's scores lie in whole lanes of the warp
   float scaling;
 };
 int route_launch(const RouteParams& p, cudaStream_t st);
@@ -161,27 +165,73 @@ struct MoePlanParams {
   int4* work2;        // GEMM 2 items (stacked w2)
   int E, tn, n1, n2;  // local experts, token tile, 128-row tiles per expert in w13 / w2
 };
+// xs: rows of Hp >= H elements, zeros past H
 int moe_prepare_launch(const MoePlanParams& p, const int* ids, int n_pairs, int k, int e_off, int* slot_of, const void* x, long long ldx,
-                       void* xs, int H, cudaStream_t st);
+                       void* xs, int H, int Hp, int f32, cudaStream_t st);
+// fp32 grouped product over the work list: out[slot][n] = sum_k a[slot][k] w[expert][n][k]; silu: a = silu(x[k]) * x[K + k]
+int moe_gemm_f32_launch(const float* x, int ldx, const float* w, float* out, int N, int K, int silu, const int4* work, const int* work_count, int n_tiles,
+                        int num_sms, cudaStream_t st);
 int moe_plan_launch(const MoePlanParams& p, cudaStream_t st);
-int moe_combine_launch(const void* a2, const int* slot_of, const float* w, void* y, int T, int k, int H, cudaStream_t st);
+int moe_combine_launch(const void* a2, int lda, const int* slot_of, const float* w, void* y, int T, int k, int H, int f32, cudaStream_t st);
 unsigned int moe_read_status(bool clear);
 void moe_read_status_async(unsigned int* dst, cudaStream_t st);
 
 struct MlaParams {
-  const __nv_bfloat16* q_abs;   // [T][H][512] query with W_UK absorbed
-  const __nv_bfloat16* q_rope;  // [T][H][64]
-  const __nv_bfloat16* cache;   // [blocks][bs][576] latent | rope key
-  __nv_bfloat16* out;           // [T][H][512]
+  const void* q_abs;            // [T][H][kv_lora] query with W_UK absorbed, contiguous
+  const void* q_rope;           // [T][H][rope] with strides (elements)
+  long long qr_st, qr_sh;
+  const float* cos_sin;         // [positions][rope] (cos | sin): the kernel rotates q_rope; null: it is rotated already
+  int interleaved;              // rotary pairs (2i, 2i + 1) instead of (i, i + rope / 2)
+  const void* cache;            // [blocks][bs][kv_lora + rope_pad] latent | shared key part, zeros in the padding
+  void* out;                    // [T][H][kv_lora]
   const int* query_start_loc;
   const int* seq_lens;
   const int* block_table;
-  int bt_stride, R, T, H, kv_lora, rope, bs, bs_shift, max_q_len, splits;
+  int bt_stride, R, T, H, kv_lora, rope, rope_pad, bs, bs_shift, max_q_len, splits;
+  int fine;                     // softmax weights enter the value product as two bf16 terms
+  int f32;                      // element type of everything: fp32 instead of bf16
   float scale;
-  float* ws_o;                  // [splits][T][H][512]
+  float* ws_o;                  // [splits][T][H][kv_lora]
   float* ws_ml;                 // [splits][T][H][2]
 };
 int mla_decode_launch(const MlaParams& p, cudaStream_t st);
+bool mla_tensor_core_sizes(int kv_lora, int rope_pad);
+struct MlaPrepareParams {
+  const void *q, *kv;           // query latent [T][nq] or null; [T][lora + rope], pitches ld_q / ld_kv
+  long long ld_q, ld_kv;
+  const void *q_w, *kv_w;       // norm weights
+  float eps;
+  const int* positions;
+  const float* cos_sin;         // [positions][rope]
+  const int* slots;             // cache row per token, negative: none
+  void* q_out;                  // [T][nq]
+  void* cache;                  // rows of `width` elements: latent at 0, key part at lora_pad
+  int T, nq, lora, lora_pad, rope, width, interleaved, f32;
+};
+int mla_prepare_launch(const MlaPrepareParams& p, cudaStream_t st);
+struct MlstmParams {
+  const void* x;                // [T][ld] q [H D] | k [H D] | v [H V] | output gate [H V]
+  long long ld;
+  const float* gates;           // [T][ld_g] input | forget gate logits
+  long long ld_g;
+  const float *i_bias, *f_bias; // [H]
+  const void* norm_w;           // [H V]
+  float eps, cap, scale;        // scale: of the queries
+  float *S, *n, *m;             // [slots][H][D][V], [slots][H][D], [slots][H]
+  void* out;                    // [T][H V]
+  const int *query_start_loc, *state_slots, *has_initial_state;
+  int T, R, H, D, V, f32, skip_min_len;
+  // chunked form: one segment of the step's chunk list
+  const int *chunk_req, *chunk_t0, *chunk_long;      // per chunk: request, first token, entry of the sequence list
+  const int *long_req, *long_chunk0, *long_n;        // per sequence of the segment: request, first chunk, chunks
+  float *ws_s, *ws_n, *ws_g, *ws_m;                  // [chunks][H][D V], [chunks][H][D], [chunks][H][2], [chunks][H]
+  __nv_bfloat16* ws_h;                               // [chunks][H][2][D V] state ahead of the chunk in two terms
+  int vec_qk, vec_v;                                 // rows of q / k, and of v / the state planes, start on 16-byte boundaries
+};
+int mlstm_recurrent_launch(const MlstmParams& p, cudaStream_t st);
+bool mlstm_chunkable(int D, int V);
+int mlstm_chunk_launch(const MlstmParams& p, int num_chunks, int num_long, cudaStream_t st);
+int sigmoid_mul_launch(const void* x, long long ldx, const void* gate, long long ldg, void* y, int T, int N, int f32, cudaStream_t st);
 unsigned int mla_read_status(bool clear);
 void mla_read_status_async(unsigned int* dst, cudaStream_t st);
 

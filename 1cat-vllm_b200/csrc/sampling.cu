@@ -107,16 +107,21 @@ __global__ void accept_kernel(const RowStats* __restrict__ stats, const long lon
   o[n] = bonus[b];
 }
 
-// ---- routing: one warp per token, E <= 512 experts (E / 32 scores per lane)
-__global__ void route_kernel(const RouteParams p) {
+// ---- routing: one warp per token, E <= 512 experts (ceil(E / 32) scores per lane, scores past E never win)
+__global__ void __launch_bounds__(256) route_kernel(const RouteParams p) {
+  __shared__ float s_sel[8][512];
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (t >= p.T) return;
   const int lane = threadIdx.x & 31;
-  const int per = p.E / 32;  // host guarantees E % 32 == 0 and per <= 16
+  const int per = (p.E + 31) / 32;  // host guarantees per <= 16
   float sc[16], sel[16];
-  const __nv_bfloat16* x = p.logits + (size_t)t * p.ld;
   float mx = -INFINITY;
-  for (int i = 0; i < per; ++i) { sc[i] = __bfloat162float(x[lane * per + i]); mx = fmaxf(mx, sc[i]); }
+  for (int i = 0; i < per; ++i) {
+    const int e = lane * per + i;
+    const size_t at = (size_t)t * p.ld + e;
+    sc[i] = e >= p.E ? -INFINITY : p.is_fp32 ? reinterpret_cast<const float*>(p.logits)[at] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.logits)[at]);
+    mx = fmaxf(mx, sc[i]);
+  }
   if (p.sigmoid) {
     for (int i = 0; i < per; ++i) sc[i] = 1.f / (1.f + __expf(-sc[i]));
   } else {
@@ -126,8 +131,35 @@ __global__ void route_kernel(const RouteParams p) {
     sum = warp_sum(sum);
     for (int i = 0; i < per; ++i) sc[i] /= sum;
   }
-  for (int i = 0; i < per; ++i) sel[i] = sc[i] + (p.bias != nullptr ? p.bias[lane * per + i] : 0.f);
-  if (p.n_group > 1) {
+  for (int i = 0; i < per; ++i) sel[i] = lane * per + i < p.E ? sc[i] + (p.bias != nullptr ? p.bias[lane * per + i] : 0.f) : -INFINITY;
+  if (p.n_group > 1 && !p.whole_lanes) {
+    // groups that do not fill whole lanes: the same rule over a copy in shared memory, a lane per group
+    float* row = s_sel[threadIdx.x >> 5];
+    const int gsz = p.E / p.n_group;
+    for (int i = 0; i < per; ++i)
+      if (lane * per + i < p.E) row[lane * per + i] = sel[i];
+    __syncwarp();
+    float gs[16];   // n_group <= 512
+    for (int gi = 0, g = lane; g < p.n_group; ++gi, g += 32) {
+      float b1 = -INFINITY, b2 = -INFINITY;
+      for (int i = 0; i < gsz; ++i) {
+        const float v = row[g * gsz + i];
+        if (v > b1) { b2 = b1; b1 = v; } else if (v > b2) b2 = v;
+      }
+      gs[gi] = p.bias != nullptr ? b1 + (gsz > 1 ? b2 : 0.f) : b1;
+    }
+    __syncwarp();
+    for (int gi = 0, g = lane; g < p.n_group; ++gi, g += 32) row[g] = gs[gi];
+    __syncwarp();
+    for (int i = 0; i < per; ++i) {
+      if (lane * per + i >= p.E) continue;
+      const int g = (lane * per + i) / gsz;
+      int rank = 0;
+      for (int o = 0; o < p.n_group; ++o)
+        if (row[o] > row[g] || (row[o] == row[g] && o < g)) ++rank;
+      if (rank >= p.topk_group) sel[i] = -INFINITY;
+    }
+  } else if (p.n_group > 1) {
     // group score = sum of the two best biased scores in the group (max without bias); keep the topk_group best groups
     const int gsz = p.E / p.n_group;            // experts per group; a group spans gsz / per lanes
     const int lanes_per_group = gsz / per;      // host guarantees gsz % per == 0 and lanes_per_group is a power of two <= 32
@@ -188,14 +220,15 @@ int rejection_launch(const void* logits, int is_fp32, const long long* draft_ids
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
-int route_launch(const RouteParams& p, cudaStream_t st) {
+int route_launch(const RouteParams& q, cudaStream_t st) {
+  RouteParams p = q;
   if (p.T == 0) return 0;
-  if (p.E % 32 || p.E / 32 > 16 || p.k > 16 || p.k > p.E) return -1;
-  if (p.n_group > 1) {
-    const int per = p.E / 32, gsz = p.E / p.n_group;
-    if (p.E % p.n_group || gsz % per) return -1;
-    const int lpg = gsz / per;
-    if (lpg < 1 || (lpg & (lpg - 1)) || lpg > 32) return -1;
+  if (p.E < 1 || p.E > 512 || p.k < 1 || p.k > 16 || p.k > p.E || p.n_group < 1 || p.E % p.n_group) return -1;
+  if (p.n_group > 1 && p.k > p.E / p.n_group * p.topk_group) return -1;
+  p.whole_lanes = 0;
+  if (p.n_group > 1 && p.E % 32 == 0) {
+    const int per = p.E / 32, gsz = p.E / p.n_group, lpg = gsz / per;
+    p.whole_lanes = gsz % per == 0 && lpg >= 1 && (lpg & (lpg - 1)) == 0 && lpg <= 32;
   }
   route_kernel<<<(p.T + 7) / 8, 256, 0, st>>>(p);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;

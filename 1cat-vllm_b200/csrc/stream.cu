@@ -1,5 +1,5 @@
 // Kernels around the fp32 residual stream and the un-rotated paged cache.
-//   stream_join: x' = x + scale * post(part) (+ add), y = next(x'): a sub-block's output is normalised, scaled, added to the stream and the
+//   stream_join: x' = x + mul * scale * post(part) (+ add), y = next(x'): a sub-block's output is normalised, scaled, added to the stream and the
 //                sum normalised for the next sub-block in one pass; optionally x' also leaves in the model's element type.
 //   kv_insert:   key (and value) rows into their pages.
 #include <type_traits>
@@ -61,6 +61,21 @@ __global__ void __launch_bounds__(256) stream_join_kernel(const StreamJoinParams
     if (c < H) load_vec<PE, N>(part + c, v[i]);
   }
   auto normalise = [&](const StreamNorm& n) {
+    if (n.kind == 3) {   // dynamic tanh: no statistics
+      const float al = to_f<E>(*reinterpret_cast<const E*>(n.alpha));
+#pragma unroll
+      for (int i = 0; i < IT; ++i) {
+        const int c = (i * blockDim.x + threadIdx.x) * N;
+        if (c < H) {
+          float w[N], b[N];
+          load_vec<E, N>(reinterpret_cast<const E*>(n.w) + c, w);
+          load_vec<E, N>(reinterpret_cast<const E*>(n.b) + c, b);
+#pragma unroll
+          for (int j = 0; j < N; ++j) v[i][j] = fmaf(tanhf(al * v[i][j]), w[j], b[j]);
+        }
+      }
+      return;
+    }
     float mean = 0.f;
     if (n.kind == 2) {
       float s = 0.f;
@@ -109,6 +124,10 @@ __global__ void __launch_bounds__(256) stream_join_kernel(const StreamJoinParams
         load_vec<E, N>(reinterpret_cast<const E*>(p.scale) + c, a);
 #pragma unroll
         for (int j = 0; j < N; ++j) v[i][j] *= a[j];
+      }
+      if (p.mul != 1.f) {
+#pragma unroll
+        for (int j = 0; j < N; ++j) v[i][j] *= p.mul;
       }
       if (p.add != nullptr) {
         load_vec<E, N>(reinterpret_cast<const E*>(p.add) + c, a);
@@ -171,6 +190,8 @@ __global__ void __launch_bounds__(256) kv_insert_kernel(const KvInsertParams p) 
 
 int stream_join_launch(const StreamJoinParams& p, cudaStream_t st) {
   if (p.T == 0) return 0;
+  auto incomplete = [](const StreamNorm& n) { return n.kind == 3 && (n.w == nullptr || n.b == nullptr || n.alpha == nullptr); };
+  if (incomplete(p.post) || incomplete(p.next)) return -1;
   if (p.H < 1 || p.x_out == nullptr || (p.next.kind != 0 && p.y == nullptr) || (p.f32 && !p.part_f32)) return -1;
   // vectors of four elements when every row starts on a vector boundary
   const uintptr_t esz = p.f32 ? 4 : 2, psz = p.part_f32 ? 4 : 2;

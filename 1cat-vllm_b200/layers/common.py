@@ -55,9 +55,43 @@ class LayerNorm(nn.Module):
         getattr(self, pname).data.copy_(w)
 
 
+class DynamicTanh(nn.Module):
+    """``tanh(alpha * x) * w + b`` in the place of a norm: a learned scalar ``alpha``, no statistics of the row. Interface of ``RMSNorm``;
+    models with an fp32 residual stream run it inside the fused join kernel (``ops.stream_join``)."""
+
+    plain = True
+    gemma = False
+
+    def __init__(self, hidden: int, dtype=torch.float32, alpha: float = 0.5):
+        super().__init__()
+        self.hidden, self.eps = hidden, 0.0
+        self.weight = nn.Parameter(torch.ones(hidden, dtype=dtype), requires_grad=False)
+        self.bias = nn.Parameter(torch.zeros(hidden, dtype=dtype), requires_grad=False)
+        self.alpha = nn.Parameter(torch.full((1,), alpha, dtype=dtype), requires_grad=False)
+
+    def forward(self, x, residual: Optional[torch.Tensor] = None):
+        if residual is not None:
+            x = x + residual
+        return (torch.tanh(self.alpha.float() * x.float()) * self.weight.float() + self.bias.float()).to(x.dtype), x
+
+    def load_weight(self, pname, w, shard_id=None):
+        getattr(self, pname).data.copy_(w.reshape(getattr(self, pname).shape))
+
+
+def state_tensors(mixer) -> list:
+    """(shape of one slot, dtype or None for the model's) of every tensor of a state-slot mixer's per-sequence state. The usual pair of a
+    rolling convolution window and an fp32 recurrent state comes from ``state_shapes``; mixers with other states define ``state_tensors``."""
+    if hasattr(mixer, "state_tensors"):
+        return mixer.state_tensors()
+    conv, rec = mixer.state_shapes()
+    return [(tuple(conv), None), (tuple(rec), torch.float32)]
+
+
 def make_norm(cfg, hidden: Optional[int] = None) -> nn.Module:
     """The normalisation a model's blocks use: RMSNorm unless its configuration names the mean-and-variance form."""
     hidden = hidden or cfg.hidden_size
+    if cfg.norm_type == "dyt":
+        return DynamicTanh(hidden, cfg.dtype)
     if cfg.norm_type == "layernorm":
         return LayerNorm(hidden, cfg.rms_norm_eps, cfg.norm_affine, cfg.norm_bias, cfg.gemma_norm, cfg.dtype)
     return RMSNorm(hidden, cfg.rms_norm_eps, cfg.gemma_norm, cfg.dtype)

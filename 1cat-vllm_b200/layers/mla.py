@@ -7,19 +7,12 @@ from __future__ import annotations
 import torch
 import torch.nn as nn
 
+from onecat_vllm import ops
 from onecat_vllm.config import ModelConfig
 from onecat_vllm.layers.common import RMSNorm, get_rope
-from onecat_vllm.layers.linear import ColumnParallelLinear, ReplicatedLinear, RowParallelLinear
+from onecat_vllm.layers.linear import ColumnParallelLinear, LinearBase, ReplicatedLinear, RowParallelLinear
 from onecat_vllm.ops import ref
 from onecat_vllm.parallel.state import get_state
-
-
-def _rope_interleaved(x: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor) -> torch.Tensor:
-    """GPT-J style (pairs (2i, 2i+1)), as DeepSeek uses for the rope part."""
-    xf = x.float()
-    x1, x2 = xf[..., 0::2], xf[..., 1::2]
-    c, s = cos.unsqueeze(1), sin.unsqueeze(1)
-    return torch.stack([x1 * c - x2 * s, x2 * c + x1 * s], dim=-1).flatten(-2).to(x.dtype)
 
 
 class MLAAttention(nn.Module):
@@ -29,27 +22,54 @@ class MLAAttention(nn.Module):
         self.H = cfg.num_attention_heads // tp
         self.nope, self.rope_d, self.vd, self.lora = cfg.qk_nope_head_dim, cfg.qk_rope_head_dim, cfg.v_head_dim, cfg.kv_lora_rank
         self.q_lora = cfg.q_lora_rank
-        q, dt = cfg.quant, cfg.dtype
+        q, dt, Hg = cfg.quant, cfg.dtype, cfg.num_attention_heads
         qk = self.nope + self.rope_d
+        self.fused_in, self.gated, self.interleaved = cfg.mla_fused_in, cfg.attn_output_gate, not cfg.mla_rope_half
+        if Hg % tp:
+            raise ValueError(f"tensor_parallel_size={tp} does not divide the {Hg} heads of layer {layer_idx}")
+        if self.fused_in:
+            # query latent | key/value latent and shared key part | output gate: everything that reads the block's input, in one GEMM
+            sizes = [self.q_lora, self.lora + self.rope_d] + ([Hg * self.vd] if self.gated else [])
+            self.in_proj_dqkvg = LinearBase(cfg.hidden_size, sizes, "column", quant=q, prefix=prefix + ".in_proj_dqkvg", dtype=dt,
+                                            segment_tp=[1, 1, tp][: len(sizes)])
+        elif self.gated:
+            raise ValueError("the output gate of latent attention is part of the fused input projection")
         if self.q_lora:
-            self.q_a_proj = ReplicatedLinear(cfg.hidden_size, self.q_lora, quant=q, prefix=prefix + ".q_a_proj", dtype=dt)
+            if not self.fused_in:
+                self.q_a_proj = ReplicatedLinear(cfg.hidden_size, self.q_lora, quant=q, prefix=prefix + ".q_a_proj", dtype=dt)
             self.q_a_layernorm = RMSNorm(self.q_lora, cfg.rms_norm_eps, dtype=dt)
-            self.q_b_proj = ColumnParallelLinear(self.q_lora, cfg.num_attention_heads * qk, quant=q, prefix=prefix + ".q_b_proj", dtype=dt)
+            self.q_b_proj = ColumnParallelLinear(self.q_lora, Hg * qk, quant=q, prefix=prefix + ".q_b_proj", dtype=dt)
         else:
-            self.q_proj = ColumnParallelLinear(cfg.hidden_size, cfg.num_attention_heads * qk, quant=q, prefix=prefix + ".q_proj", dtype=dt)
-        self.kv_a_proj_with_mqa = ReplicatedLinear(cfg.hidden_size, self.lora + self.rope_d, quant=q, prefix=prefix + ".kv_a_proj_with_mqa", dtype=dt)
+            self.q_proj = ColumnParallelLinear(cfg.hidden_size, Hg * qk, quant=q, prefix=prefix + ".q_proj", dtype=dt)
+        if not self.fused_in:
+            self.kv_a_proj_with_mqa = ReplicatedLinear(cfg.hidden_size, self.lora + self.rope_d, quant=q, prefix=prefix + ".kv_a_proj_with_mqa", dtype=dt)
         self.kv_a_layernorm = RMSNorm(self.lora, cfg.rms_norm_eps, dtype=dt)
-        self.kv_b_proj = ColumnParallelLinear(self.lora, cfg.num_attention_heads * (self.nope + self.vd), quant=q, prefix=prefix + ".kv_b_proj", dtype=dt)
-        self.o_proj = RowParallelLinear(cfg.num_attention_heads * self.vd, cfg.hidden_size, quant=q, prefix=prefix + ".o_proj", dtype=dt)
+        self.kv_b_proj = ColumnParallelLinear(self.lora, Hg * (self.nope + self.vd), quant=q, prefix=prefix + ".kv_b_proj", dtype=dt)
+        self.o_proj = RowParallelLinear(Hg * self.vd, cfg.hidden_size, quant=q, prefix=prefix + ".o_proj", dtype=dt)
         self.rope = get_rope(self.rope_d, cfg.max_model_len, cfg.rope_theta, device, cfg.rope_scaling)
-        self.scale = qk ** -0.5
+        self.scale = cfg.attn_scale if cfg.attn_scale is not None else qk ** -0.5
         sc = cfg.rope_scaling or {}
-        if (sc.get("rope_type") or sc.get("type")) in ("yarn", "deepseek_yarn") and sc.get("mscale_all_dim"):
+        if cfg.attn_scale is None and (sc.get("rope_type") or sc.get("type")) in ("yarn", "deepseek_yarn") and sc.get("mscale_all_dim"):
             # DeepSeek yarn: the softmax scale carries mscale(factor, mscale_all_dim)^2 (reference: models/deepseek_v2.py:483-487)
             from onecat_vllm.ops.ref import yarn_mscale
             m = yarn_mscale(float(sc.get("factor", 1.0)), float(sc["mscale_all_dim"]))
             self.scale *= m * m
+        # fp32 residual streams come with fp32 softmax weights: the tensor-core kernels then carry them as two bf16 terms
+        self.fine_weights = cfg.residual_fp32
+        self.lora_pad, self.rope_pad = self.lora, self.rope_d
+        if torch.device(device).type == "cuda" and dt == torch.bfloat16:
+            from onecat_vllm.ops import cuda as K
+            self.lora_pad, self.rope_pad = K.mla_padded_sizes(self.lora, self.rope_d)
+        self.cache_width = self.lora_pad + self.rope_pad   # elements of a cached token: latent | shared key part, each padded for the kernel
         self._wuk = self._wuv = None
+
+    def load_weight(self, pname: str, w: torch.Tensor, shard=None) -> None:
+        """Key and value up-projections stored apart (``uk`` / ``uv``, rows head by head) take their places in ``kv_b_proj``."""
+        st = get_state()
+        n = {"uk": self.nope, "uv": self.vd}[pname]
+        o = 0 if pname == "uk" else self.nope
+        w = w.view(-1, n, self.lora)[st.tp_rank * self.H: (st.tp_rank + 1) * self.H]
+        self.kv_b_proj.weight.data.view(self.H, self.nope + self.vd, self.lora)[:, o:o + n].copy_(w)
 
     def process_weights_after_loading(self):
         """Runs before the child layers' own repacking (parents come first in ``modules()``): the absorbed ``W_UK`` / ``W_UV`` are
@@ -61,34 +81,38 @@ class MLAAttention(nn.Module):
     def _absorb(self, dtype):
         if self._wuk is None:
             w = self.kv_b_proj.method.dequantized_weight(self.kv_b_proj).to(dtype).view(self.H, self.nope + self.vd, self.lora)
+            w = torch.nn.functional.pad(w, (0, self.lora_pad - self.lora))   # zero columns: the padded latent is zero there as well
             self._wuk = w[:, : self.nope, :].contiguous()  # [H, nope, lora]
             self._wuv = w[:, self.nope:, :].contiguous()  # [H, v, lora]
         return self._wuk, self._wuv
 
     def forward(self, x, md, latent_cache):
-        T = x.shape[0]
-        if self.q_lora:
-            qa, _ = self.q_a_layernorm(self.q_a_proj(x))
-            q = self.q_b_proj(qa)
+        T, gate = x.shape[0], None
+        if self.fused_in:
+            y = self.in_proj_dqkvg(x)
+            n = self.q_lora + self.lora + self.rope_d
+            qa, kv = y[:, : self.q_lora], y[:, self.q_lora: n]
+            gate = y[:, n:] if self.gated else None
         else:
-            q = self.q_proj(x)
-        q = q.view(T, self.H, self.nope + self.rope_d)
-        kv = self.kv_a_proj_with_mqa(x)
-        c, _ = self.kv_a_layernorm(kv[:, : self.lora].contiguous())
-        cs = self.rope.cos_sin[md.positions.long()]
-        cos, sin = cs[:, : self.rope_d // 2], cs[:, self.rope_d // 2:]
-        k_pe = _rope_interleaved(kv[:, self.lora:].unsqueeze(1), cos, sin).squeeze(1)
-        q_pe = _rope_interleaved(q[..., self.nope:], cos, sin)
-        # insert without a data-dependent shape (no host synchronisation, so the step can be captured in a CUDA graph): tokens
-        # without a slot (-1, padding of a captured batch) are routed to slot 0 of block 0, the placeholder block nothing reads
-        sm = md.slot_mapping.long().clamp(min=0)
-        latent_cache.view(-1, latent_cache.shape[-1]).index_copy_(0, sm, torch.cat([c, k_pe], dim=-1).to(latent_cache.dtype))
-        wuk, wuv = self._absorb(x.dtype)
-        q_abs = torch.einsum("thn,hnl->thl", q[..., : self.nope], wuk)
-        if x.is_cuda:
+            qa, kv = self.q_a_proj(x) if self.q_lora else None, self.kv_a_proj_with_mqa(x)
+        # one kernel: both latent norms, the rotation of the shared key part and the cache insert (no data-dependent shape: the step can
+        # be captured in a CUDA graph; padding tokens have no slot)
+        qa = ops.mla_prepare(qa, kv, self.q_a_layernorm if self.q_lora else None, self.kv_a_layernorm, md.positions, self.rope.cos_sin, latent_cache,
+                             md.slot_mapping, self.lora, self.lora_pad, self.interleaved)
+        q = (self.q_b_proj(qa) if self.q_lora else self.q_proj(x)).view(T, self.H, self.nope + self.rope_d)
+        o = self._attend(q, md, latent_cache).reshape(T, self.H * self.vd)
+        return self.o_proj(ops.sigmoid_mul(o, gate) if gate is not None else o)
+
+    def _attend(self, q, md, latent_cache):
+        """Attention over the cached latents with the key up-projection moved to the query and the value one to the result."""
+        wuk, wuv = self._absorb(q.dtype)
+        if q.is_cuda:
             from onecat_vllm.ops import cuda as K
-            o_lat = K.mla_decode(q_abs, q_pe, latent_cache, md, self.scale, self.lora)
-        else:
-            o_lat = ref.mla_decode(q_abs, q_pe, latent_cache, md.block_table, md.query_start_loc, md.seq_lens, self.scale, self.lora)
-        o = torch.einsum("thl,hvl->thv", o_lat, wuv)
-        return self.o_proj(o.reshape(T, self.H * self.vd))
+            q_abs = K.per_head_matmul(q[..., : self.nope], wuk)
+            o_lat = K.mla_decode(q_abs, q[..., self.nope:], latent_cache, md, self.scale, self.lora_pad, self.rope.cos_sin, self.interleaved,
+                                 self.fine_weights)
+            return K.per_head_matmul(o_lat, wuv.transpose(1, 2))
+        q_abs = torch.einsum("thn,hnl->thl", q[..., : self.nope], wuk)
+        q_pe = ref.rope_rows(q[..., self.nope:], md.positions, self.rope.cos_sin, self.interleaved)
+        o_lat = ref.mla_decode(q_abs, q_pe, latent_cache, md.block_table, md.query_start_loc, md.seq_lens, self.scale, self.lora)
+        return torch.einsum("thl,hvl->thv", o_lat, wuv)

@@ -131,10 +131,10 @@ class SparseMoeBlock(nn.Module):
         super().__init__()
         self.cfg = cfg
         self.gate = ReplicatedLinear(cfg.hidden_size, cfg.num_experts, bias=cfg.router_linear_bias, quant=None, prefix=prefix + ".gate",
-                                     dtype=cfg.dtype)
+                                     dtype=cfg.dtype, out_dtype=torch.float32 if cfg.router_fp32 else None)
         self.experts = FusedMoE(cfg, prefix + ".experts")
         self.deepseek = cfg.scoring_func == "sigmoid" or cfg.n_group > 1 or cfg.router_bias
-        if self.deepseek:
+        if cfg.scoring_func == "sigmoid" or cfg.router_bias:   # softmax scores are grouped by their maximum, without a selection bias
             self.e_score_correction_bias = nn.Parameter(torch.zeros(cfg.num_experts, dtype=torch.float32), requires_grad=False)
         self.shared_expert: Optional[MLP] = None
         if cfg.shared_expert_intermediate_size > 0:
@@ -150,7 +150,7 @@ class SparseMoeBlock(nn.Module):
             from onecat_vllm.ops import cuda as K
             return K.route(logits, c, getattr(self, "e_score_correction_bias", None))
         if self.deepseek:
-            return ref.grouped_topk(logits, c.num_experts_per_tok, c.n_group, c.topk_group, self.e_score_correction_bias,
+            return ref.grouped_topk(logits, c.num_experts_per_tok, c.n_group, c.topk_group, getattr(self, "e_score_correction_bias", None),
                                     c.scoring_func, c.norm_topk_prob, c.routed_scaling_factor)
         return ref.topk_softmax(logits, c.num_experts_per_tok, c.norm_topk_prob)
 

@@ -80,6 +80,36 @@ def gabisun_name(name: str) -> str:
     return f"model.layers.{m.group(1)}." + (ours[: -len("weight")] + "bias" if m.group(3) else ours)
 
 
+# Sepirax checkpoints: ``l<i>.<name>``; the mixer's names depend on its kind
+_SEPIRAX_MIX = {"mla": {"dq": "self_attn.dq_proj.weight", "dkv": "self_attn.dkv_proj.weight", "g": "self_attn.g_proj.weight",
+                        "dq.norm": "self_attn.q_a_layernorm.weight", "dkv.norm": "self_attn.kv_a_layernorm.weight",
+                        "uq": "self_attn.q_b_proj.weight", "uk": "self_attn.uk", "uv": "self_attn.uv", "o": "self_attn.o_proj.weight"},
+                "mlstm": {**{n: f"linear_attn.in_proj_{n}.weight" for n in "qkvg"}, "i": "linear_attn.gate_i.weight", "f": "linear_attn.gate_f.weight",
+                          "i.b": "linear_attn.i_bias", "f.b": "linear_attn.f_bias", "norm": "linear_attn.norm_weight", "o": "linear_attn.out_proj.weight"}}
+_SEPIRAX_TOP = {"embed": "model.embed_tokens.weight", "head": "lm_head.weight", "final.norm": "model.norm.weight", "final.norm.b": "model.norm.bias",
+                "final.norm.alpha": "model.norm.alpha"}
+_SEPIRAX_NORM_RE = re.compile(r"norm([12])(\.b|\.alpha)?$")
+_SEPIRAX_EXPERT_RE = re.compile(r"mlp\.e(\d+)\.(gate|up|down)$")
+
+
+def sepirax_name(name: str, mixer_kind) -> str:
+    """Module parameter that a Sepirax checkpoint tensor belongs to (unknown names come back unchanged). ``mixer_kind(i)``: "mla" | "mlstm"."""
+    layer, _, rest = name.partition(".")
+    if name in _SEPIRAX_TOP or not re.fullmatch(r"l\d+", layer):
+        return _SEPIRAX_TOP.get(name, name)
+    base = f"model.layers.{layer[1:]}."
+    m = _SEPIRAX_NORM_RE.match(rest)
+    if m:
+        return base + ("input_layernorm" if m.group(1) == "1" else "post_attention_layernorm") + {".b": ".bias", ".alpha": ".alpha"}.get(m.group(2), ".weight")
+    m = _SEPIRAX_EXPERT_RE.match(rest)
+    if m:
+        return f"{base}mlp.experts.{m.group(1)}.{m.group(2)}_proj.weight"
+    if rest == "mlp.router":
+        return base + "mlp.gate.weight"
+    ours = _SEPIRAX_MIX[mixer_kind(int(layer[1:]))].get(rest[len("mix."):]) if rest.startswith("mix.") else None
+    return base + ours if ours else name
+
+
 _EXPERT_RE = re.compile(r"(.*\.mlp)\.experts\.(\d+)\.(gate_proj|up_proj|down_proj)\.(weight|weight_scale_inv|weight_scale|bias)$")
 
 
@@ -95,10 +125,13 @@ def load_weights(model: nn.Module, weights: Iterable[tuple[str, torch.Tensor]]) 
     vault = cfg is not None and cfg.architecture.startswith("VaultGemma")
     nemotron_h = cfg is not None and cfg.architecture.startswith("NemotronH")
     gabisun = cfg is not None and cfg.architecture == "Gabisun"
+    sepirax = cfg is not None and cfg.architecture == "Sepirax"
     loaded = set()
     for name, w in weights:
         if gabisun:
             name = gabisun_name(name)
+        elif sepirax:
+            name = sepirax_name(name, lambda i: "mlstm" if cfg.layer_type(i) == "mlstm" else "mla")
         if name.startswith("language_model."):
             name = name[len("language_model."):]
         elif name.startswith("model.language_model."):  # text tower of a multimodal checkpoint (Qwen3.5)
@@ -270,7 +303,7 @@ def dummy_init(model: nn.Module, seed: int = 0, std: float = 0.02) -> None:
     for name, p in model.named_parameters():
         g = gen(p.device)
         leaf = name.rsplit(".", 1)[-1]
-        if leaf in ("weight",) and name.endswith(("layernorm.weight", "norm.weight")) or leaf in ("q_norm", "k_norm", "norm_weight", "attn_layer_scale", "mlp_layer_scale"):
+        if leaf in ("weight",) and name.endswith(("layernorm.weight", "norm.weight")) or leaf in ("q_norm", "k_norm", "norm_weight", "attn_layer_scale", "mlp_layer_scale", "alpha"):
             continue  # keep constructor init (1, or 0 for Gemma-style)
         if p.dtype in (torch.float32, torch.float16, torch.bfloat16):
             if leaf in ("scales",):

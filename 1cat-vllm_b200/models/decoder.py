@@ -44,6 +44,10 @@ class DecoderLayer(nn.Module):
             self.self_attn = layer_class("MLAAttention", MLAAttention)(cfg, idx, prefix + ".self_attn", device)
         elif self.kind == "linear_attention":
             self.linear_attn = layer_class("GatedDeltaNet", GatedDeltaNet)(cfg, idx, prefix + ".linear_attn")
+        elif self.kind == "mlstm":
+            from onecat_vllm.layers.mlstm import MLSTM
+            self.linear_attn = layer_class("MLSTM", MLSTM)(cfg, idx, prefix + ".linear_attn")
+            self.kind = "linear_attention"   # a state-slot layer for the runner and the scheduler
         elif self.kind in ("mamba2", "mamba1", "short_conv", "ffn"):
             if self.kind == "ffn":
                 from onecat_vllm.layers.mlp import FeedForwardBlock as Mixer
@@ -107,8 +111,9 @@ class DecoderModel(nn.Module):
         self.norm = make_norm(cfg) if self.last_stage else PPMissingLayer()
         if cfg.residual_fp32 and (self.start != 0 or not self.last_stage):
             raise ValueError("models with an fp32 residual stream are served without pipeline parallelism")
-        if (cfg.residual_fp32 or cfg.layer_scale) and not (cfg.residual_fp32 and cfg.sandwich_norm) or cfg.loop is not None and not cfg.residual_fp32:
-            raise ValueError("the fp32 residual stream is served for blocks with norms on both sides; looped layers and layer scales need it")
+        if (cfg.layer_scale or cfg.loop is not None) and not cfg.residual_fp32 or cfg.residual_fp32 and (cfg.parallel_block or not cfg.pre_norm):
+            raise ValueError("the fp32 residual stream is served for blocks with norms ahead of (or on both sides of) the sub-blocks; looped layers "
+                             "and layer scales need it")
         if cfg.loop is not None:
             # ahead of every pass of the looped layers the stream x becomes loop_in([x ; x0]) + loop_step[pass], x0 being the embeddings
             self.loop_in = ReplicatedLinear(2 * cfg.hidden_size, cfg.hidden_size, quant=None, prefix="model.loop_in", dtype=cfg.dtype,
@@ -117,6 +122,11 @@ class DecoderModel(nn.Module):
         # EAGLE-3 drafting reads the residual stream at a few depths: layer indices to record, and what the last forward recorded
         self.aux_hidden_layers: tuple = ()
         self.last_aux: list = []
+
+    def embed(self, input_ids: torch.Tensor) -> torch.Tensor:
+        """Token embeddings as ``forward`` takes them in ``inputs_embeds`` for models whose stream starts from them unrounded."""
+        h = self.embed_tokens(input_ids)
+        return (h.float() * self.cfg.embed_scale).to(h.dtype) if self.cfg.residual_fp32 and self.cfg.embed_scale != 1.0 else h
 
     def local_layers(self):
         """(global index, layer) of the decoder layers this pipeline stage owns."""
@@ -139,6 +149,8 @@ class DecoderModel(nn.Module):
         if intermediate is None:
             if inputs_embeds is None:
                 h = self.embed_tokens(input_ids)
+                if cfg.residual_fp32:   # the stream starts from the scaled embeddings: the factor is applied in fp32
+                    return self._forward_stream(h, md, caches, return_prenorm, cfg.embed_scale)
                 if cfg.embed_scale != 1.0:
                     h = h * torch.tensor(cfg.embed_scale, dtype=h.dtype)  # the factor is rounded to the model dtype first, as in the checkpoint's code
             else:
@@ -188,37 +200,41 @@ class DecoderModel(nn.Module):
             return x, residual
         return x
 
-    def _forward_stream(self, h, md, caches, return_prenorm: bool = False):
-        """fp32 residual stream: ``x += scale * post_norm(sub-block(pre_norm(x)))``. One fused kernel joins a sub-block's output to the
-        stream and produces the next sub-block's input (``ops.stream_join``). Looped layers: the join ahead of a pass also leaves the
-        stream beside the embeddings as the input of the pass's entry projection, whose fp32 output becomes the new stream."""
-        runs, loop = self.cfg.layer_runs(), self.cfg.loop
+    def _forward_stream(self, h, md, caches, return_prenorm: bool = False, embed_scale: float = 1.0):
+        """fp32 residual stream: ``x += mult * scale * post_norm(sub-block(pre_norm(x)))``, post norms and layer scales where the model has
+        them. One fused kernel joins a sub-block's output to the stream and produces the next sub-block's input (``ops.stream_join``).
+        Looped layers: the join ahead of a pass also leaves the stream beside the embeddings as the input of the pass's entry projection,
+        whose fp32 output becomes the new stream."""
+        cfg = self.cfg
+        runs, loop, mult = cfg.layer_runs(), cfg.loop, cfg.residual_multiplier
         T, H = h.shape
         both = None
         if loop is not None:
             both = torch.empty(T, 2 * H, dtype=h.dtype, device=h.device)   # [stream ; embeddings]
             both[:, H:] = h
 
-        def join(part, x, post, scale, at):
+        def join(part, x, post, scale, at, mul):
             """Join, then the input of run ``at`` (past the last run: the final norm)."""
             part = reduce_only(part) if x is not None else part
             if at < len(runs) and loop is not None and runs[at][0] == loop[0] and runs[at][1] >= 0:
-                ops.stream_join(part, x, post, scale, None, copy_out=both[:, :H])
+                ops.stream_join(part, x, post, scale, None, copy_out=both[:, :H], mul=mul)
                 return ops.stream_join(self.loop_in(both), None, None, None, self.layers[loop[0]].input_layernorm, out_dtype=h.dtype,
                                        add=self.loop_step[runs[at][1]])
             return ops.stream_join(part, x, post, scale, self.layers[runs[at][0]].input_layernorm if at < len(runs) else self.norm,
-                                   out_dtype=h.dtype)
+                                   out_dtype=h.dtype, mul=mul)
 
-        y, x = join(h, None, None, None, 0)
+        y, x = join(h, None, None, None, 0, embed_scale)
         for r, (i, _) in enumerate(runs):
             layer = self.layers[i]
+            post1 = layer.post_attention_layernorm if cfg.sandwich_norm else None
+            scale1, scale2 = (layer.attn_layer_scale, layer.mlp_layer_scale) if cfg.layer_scale else (None, None)
             part = layer.mixer(y, md, caches[r])
             if layer.mlp is None:
-                y, x = join(part, x, layer.post_attention_layernorm, layer.attn_layer_scale, r + 1)
+                y, x = join(part, x, post1, scale1, r + 1, mult)
                 continue
-            y, x = ops.stream_join(reduce_only(part), x, layer.post_attention_layernorm, layer.attn_layer_scale, layer.pre_feedforward_layernorm,
-                                   out_dtype=h.dtype)
-            y, x = join(layer.mlp(y), x, layer.post_feedforward_layernorm, layer.mlp_layer_scale, r + 1)
+            y, x = ops.stream_join(reduce_only(part), x, post1, scale1,
+                                   layer.pre_feedforward_layernorm if cfg.sandwich_norm else layer.post_attention_layernorm, out_dtype=h.dtype, mul=mult)
+            y, x = join(layer.mlp(y), x, layer.post_feedforward_layernorm if cfg.sandwich_norm else None, scale2, r + 1, mult)
         return (y, x) if return_prenorm else y
 
     def _forward_post_norm(self, _x, residual, md, caches):
@@ -266,6 +282,9 @@ class CausalLM(nn.Module):
         (".qkv_proj", ".q_proj", 0), (".qkv_proj", ".k_proj", 1), (".qkv_proj", ".v_proj", 2),
         (".qkg_proj", ".q_proj", 0), (".qkg_proj", ".k_proj", 1), (".qkg_proj", ".g_proj", 2),
         (".gate_up_proj", ".gate_proj", 0), (".gate_up_proj", ".up_proj", 1),
+        (".in_proj_dqkvg", ".dq_proj", 0), (".in_proj_dqkvg", ".dkv_proj", 1), (".in_proj_dqkvg", ".g_proj", 2),
+        (".in_proj_qkvg", ".in_proj_q", 0), (".in_proj_qkvg", ".in_proj_k", 1), (".in_proj_qkvg", ".in_proj_v", 2), (".in_proj_qkvg", ".in_proj_g", 3),
+        (".gate_if", ".gate_i", 0), (".gate_if", ".gate_f", 1),
         (".in_proj_qkvz", ".in_proj_q", 0), (".in_proj_qkvz", ".in_proj_k", 1), (".in_proj_qkvz", ".in_proj_v", 2),
         (".in_proj_qkvz", ".in_proj_z", 3), (".in_proj_ba", ".in_proj_b", 0), (".in_proj_ba", ".in_proj_a", 1),
     ]
@@ -316,7 +335,7 @@ class CausalLM(nn.Module):
             e = self.model.embed_tokens
             logits = ParallelLMHead.compute_logits(e, hidden, torch.float32 if self.cfg.residual_fp32 else None)
         else:
-            logits = head.compute_logits(hidden)
+            logits = head.compute_logits(hidden, torch.float32 if self.cfg.residual_fp32 else None)
         c = self.cfg
         if c.logit_scale != 1.0:
             logits = logits * c.logit_scale

@@ -54,17 +54,42 @@ def kv_insert(k, kv_cache, slot_mapping, v=None):
 
 
 def _norm_spec(norm):
-    """(kind, weight, bias, eps, weight stored minus one) of a norm module: kind 1 RMS, 2 layer norm."""
+    """(kind, weight, bias, eps, weight stored minus one, alpha) of a norm module: kind 1 RMS, 2 layer norm, 3 dynamic tanh."""
     if norm is None:
         return None
-    return 2 if getattr(norm, "plain", False) else 1, norm.weight, getattr(norm, "bias", None), norm.eps, bool(norm.gemma)
+    alpha = getattr(norm, "alpha", None)
+    kind = 3 if alpha is not None else 2 if getattr(norm, "plain", False) else 1
+    return kind, norm.weight, getattr(norm, "bias", None), norm.eps, bool(norm.gemma), alpha
 
 
-def stream_join(part, x, post, scale, nxt, out_dtype=None, add=None, copy_out=None):
+def stream_join(part, x, post, scale, nxt, out_dtype=None, add=None, copy_out=None, mul=1.0):
     """Join a sub-block's output to the fp32 residual stream and normalise it for the next one, in one kernel:
-    ``x += scale * post(part) (+ add)``, ``y = nxt(x)``. ``post`` / ``nxt`` are norm modules or None. Returns (y, x); see ``ref.stream_join``."""
+    ``x += mul * scale * post(part) (+ add)``, ``y = nxt(x)``. ``post`` / ``nxt`` are norm modules or None, ``scale`` a vector and ``mul`` a
+    number. Returns (y, x); see ``ref.stream_join``."""
     f = ext().stream_join if part.is_cuda else ref.stream_join
-    return f(part, x, _norm_spec(post), scale, _norm_spec(nxt), out_dtype, add, copy_out)
+    return f(part, x, _norm_spec(post), scale, _norm_spec(nxt), out_dtype, add, copy_out, mul)
+
+
+def mla_prepare(q_latent, kv, q_norm, kv_norm, positions, cos_sin, cache, slot_mapping, lora, lora_pad, interleaved):
+    """Latent attention between its down- and up-projections: the normalised query latent comes back (None without one), the normalised
+    key/value latent and the rotated key part (``kv`` = [latent | key part]) go into the paged cache."""
+    f = ext().mla_prepare if kv.is_cuda else ref.mla_prepare
+    return f(q_latent, kv, q_norm.weight if q_norm is not None else None, kv_norm.weight, kv_norm.eps, positions, cos_sin, cache, slot_mapping, lora,
+             lora_pad, interleaved)
+
+
+def sigmoid_mul(x, gate):
+    """``x * sigmoid(gate)`` element by element, both ``[T, n]`` (the gate may be a column slice)."""
+    if x.is_cuda:
+        return ext().sigmoid_mul(x, gate)
+    return (x.float() * torch.sigmoid(gate.float())).to(x.dtype)
+
+
+def mlstm(qkvg, gates, i_bias, f_bias, norm_w, eps, cap, H, D, V, state, md):
+    """mLSTM recurrence with its head norm and output gate: ``qkvg`` ``[T, 2 H D + 2 H V]`` (q | k | v | output gate), ``gates`` fp32
+    ``[T, 2 H]`` (input | forget logits before bias and cap), ``state`` = (S, n, m) per slot, updated in place. Returns ``[T, H V]``."""
+    f = ext().mlstm if qkvg.is_cuda else ref.mlstm
+    return f(qkvg, gates, i_bias, f_bias, norm_w, eps, cap, H, D, V, state, md)
 
 
 def paged_attention(q, kv_cache, md, scale, out=None, window=0, softcap=0.0, sinks=None, keep=0, bias_table=None, gate=None):

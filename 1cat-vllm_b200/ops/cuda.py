@@ -409,15 +409,16 @@ def kv_insert(k, kv_cache, slot_mapping, v=None):
     _C.kv_insert(k, v, kv_cache, slot_mapping)
 
 
-def stream_join(part, x, post, scale, nxt, out_dtype=None, add=None, copy_out=None):
+def stream_join(part, x, post, scale, nxt, out_dtype=None, add=None, copy_out=None, mul=1.0):
     global _LAUNCHES
     _LAUNCHES += 1
     T, H = part.shape
     x_out = torch.empty(T, H, dtype=torch.float32, device=part.device) if x is None else x
     y = torch.empty(T, H, dtype=out_dtype, device=part.device) if nxt is not None else None
-    none = (0, None, None, 0.0, False)
-    _C.stream_join(part, x, x_out, *(post or none), scale, *(nxt or none), y, add, copy_out, (copy_out.dtype if y is None and copy_out is not None
-                   else out_dtype or part.dtype) == torch.float32)
+    none = (0, None, None, 0.0, False, None)
+    post, nxt = (tuple(n) + (None,) if len(n) == 5 else n for n in (post or none, nxt or none))
+    _C.stream_join(part, x, x_out, *post[:5], scale, *nxt[:5], y, add, copy_out, (copy_out.dtype if y is None and copy_out is not None
+                   else out_dtype or part.dtype) == torch.float32, mul, post[5], nxt[5])
     return y, x_out
 
 
@@ -639,8 +640,19 @@ def prepare_moe(moe) -> None:
     E, I2 = moe.w13.shape[0], moe.w13.shape[1]
     I = I2 // 2
     H = moe.w2.shape[1]
+    if moe.w13.dtype == torch.float32:
+        moe.kernel_state = dict(f32=True)   # engines that run in 32 bits: the weights as they are
+        return
+    if (I2 % 128 or H % 128 or I % 64) and moe.qmethod == "none":
+        # sizes that are no multiples of the kernel's tiles: zero rows and columns (a padded gate row gives silu(0) * 0)
+        Ip, Hp = -(-I // 64) * 64, -(-H // 128) * 128
+        pad = torch.nn.functional.pad
+        w13 = pad(moe.w13.data.view(E, 2, I, H), (0, Hp - H, 0, Ip - I)).reshape(E, 2 * Ip, Hp)
+        moe.w13 = torch.nn.Parameter(w13, requires_grad=False)
+        moe.w2 = torch.nn.Parameter(pad(moe.w2.data, (0, Ip - I, 0, Hp - H)), requires_grad=False)
+        I, I2, H = Ip, 2 * Ip, Hp
     if I2 % 128 or H % 128 or I % 64:
-        moe.kernel_state = None  # odd shapes take the device-side PyTorch path
+        moe.kernel_state = None  # odd shapes of packed experts take the device-side PyTorch path
         return
     perm = interleave_gate_up(I, moe.w13.device)
     q = moe.qmethod
@@ -673,9 +685,9 @@ def prepare_moe(moe) -> None:
 
 
 def route(logits, cfg, bias):
+    """Top-k experts and their weights from the router logits (bf16, or fp32 for routers that keep the accumulator's precision)."""
     global _LAUNCHES
-    E = logits.shape[1]
-    if E % 32 or E > 512 or cfg.num_experts_per_tok > 16:
+    if logits.shape[1] > 512 or cfg.num_experts_per_tok > 16:
         TORCH_STANDINS.add("route")
         if cfg.scoring_func == "sigmoid" or cfg.n_group > 1:
             return ref.grouped_topk(logits, cfg.num_experts_per_tok, cfg.n_group, cfg.topk_group, bias, cfg.scoring_func, cfg.norm_topk_prob,
@@ -683,7 +695,8 @@ def route(logits, cfg, bias):
         return ref.topk_softmax(logits, cfg.num_experts_per_tok, cfg.norm_topk_prob)
     _LAUNCHES += 1
     deepseek = cfg.scoring_func == "sigmoid" or cfg.n_group > 1
-    return _C.route(logits.to(torch.bfloat16), bias, cfg.num_experts_per_tok, cfg.n_group if deepseek else 1, cfg.topk_group if deepseek else 1,
+    return _C.route(logits if logits.dtype == torch.float32 else logits.to(torch.bfloat16), bias, cfg.num_experts_per_tok,
+                    cfg.n_group if deepseek else 1, cfg.topk_group if deepseek else 1,
                     cfg.scoring_func == "sigmoid", cfg.norm_topk_prob, cfg.routed_scaling_factor if deepseek else 1.0)
 
 
@@ -696,33 +709,127 @@ def fused_moe(moe, x, topk_w, topk_ids):
         return ref.fused_experts(x, w13, w2, topk_w, topk_ids, moe.e_off)
     ws = workspace(x.device)
     _LAUNCHES += 7
+    if ks.get("f32"):
+        return _C.fused_moe_f32(x.contiguous(), moe.w13.data, moe.w2.data, topk_w.contiguous().float(), topk_ids.contiguous().to(torch.int32), moe.e_off)
     if x.stride(-1) != 1 or (x.stride(0) * 2) % 16:
         x = x.contiguous()
     return _C.fused_moe(x, ks["w13"], ks["w2"], topk_w.contiguous().float(), topk_ids.contiguous().to(torch.int32), moe.E_local, moe.e_off,
                         ws.splitk, ws.counters, ks.get("wkind", 0), ks.get("w13_sz"), ks.get("w2_sz"), ks.get("I2", 0), ks.get("gk", 1))
 
 
-def mla_decode(q_abs, q_pe, latent_cache, md, scale, lora):
+# ----------------------------------------------------------------------------- latent attention
+MLA_WIDTHS = (64, 128, 192, 256, 384, 512)   # latents the tensor-core kernel has variants for
+
+
+def mla_padded_sizes(lora: int, rope: int) -> tuple[int, int]:
+    """(latent, key part) widths of a cached bf16 row: the next sizes of the tensor-core kernel (zeros in between), or the sizes as they are
+    when it has none."""
+    lp, rp = next((w for w in MLA_WIDTHS if w >= lora), 0), -(-rope // 16) * 16
+    return (lp, rp) if lp and _C.mla_tensor_core_sizes(lp, rp) else (lora, rope)
+
+
+def mla_prepare(q_latent, kv, q_w, kv_w, eps, positions, cos_sin, cache, slot_mapping, lora, lora_pad, interleaved):
+    global _LAUNCHES
+    _LAUNCHES += 1
+    if q_latent is not None and q_latent.stride(-1) != 1:
+        q_latent = q_latent.contiguous()
+    return _C.mla_prepare(q_latent, kv if kv.stride(-1) == 1 else kv.contiguous(), None if q_w is None else q_w.to(kv.dtype), kv_w.to(kv.dtype), eps,
+                          positions.to(torch.int32), cos_sin, cache, slot_mapping.to(torch.int32), lora, lora_pad, interleaved)
+
+
+def per_head_matmul(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """``x`` ``[T, H, a]`` (strided) times ``w`` ``[H, a, b]`` per head -> contiguous ``[T, H, b]`` (library batched product, written in place)."""
+    if x.dtype == torch.float32 and torch.backends.cuda.matmul.allow_tf32:
+        raise RuntimeError("fp32 models need torch.backends.cuda.matmul.allow_tf32 = False")
+    out = torch.empty(x.shape[0], x.shape[1], w.shape[2], dtype=x.dtype, device=x.device)
+    torch.bmm(x.transpose(0, 1), w, out=out.transpose(0, 1))
+    return out
+
+
+def plan_mla_splits(H: int, lora: int, query_lens: list, seq_lens: list, num_sms: int) -> int:
+    """KV splits of a latent-attention launch."""
+    mq = max(query_lens)
+    return choose_kv_splits(len(query_lens) * -(-mq * H // 16), max(seq_lens), num_sms)
+
+
+def mla_decode(q_abs, q_pe, latent_cache, md, scale, lora, cos_sin=None, interleaved=True, fine=False):
+    """Multi-query attention over the cached latents: ``q_abs`` ``[T, H, lora]``, ``q_pe`` ``[T, H, rope]`` (rotated by the kernel when
+    ``cos_sin`` is given). ``fine``: softmax weights in two bf16 terms."""
     global _LAUNCHES
     T, H, _ = q_abs.shape
-    if lora != 512 or q_pe.shape[-1] != 64 or q_abs.dtype != torch.bfloat16:
-        TORCH_STANDINS.add("mla_decode")
-        return ref.mla_decode(q_abs, q_pe, latent_cache, md.block_table, md.query_start_loc, md.seq_lens, scale, lora)
-    row_tiles = -(-md.max_query_len * H // 16)
     ws_o = ws_ml = None
-    if getattr(md, "static_ws", False) and getattr(md, "attn_plan", None) is not None and md.attn_plan[0][0] == "mla":
-        splits = md.attn_plan[1][2]  # captured decode graph: the split count is part of the graph's key, the workspace is static
+    splits = 1
+    if q_abs.dtype == torch.bfloat16 and _C.mla_tensor_core_sizes(lora, latent_cache.shape[-1] - lora):
+        static = getattr(md, "static_ws", False)
+        plan = getattr(md, "attn_plan", None)
+        if static and plan is not None and plan[0][0] == "mla":
+            splits = plan[1][2]  # captured decode graph: the split count is part of the graph's key
+        else:
+            splits = plan_mla_splits(H, lora, md.query_lens_cpu or [md.max_query_len] * md.num_reqs, md.seq_lens_cpu or [md.max_seq_len], _sms(q_abs.device))
         if splits > 1:
-            so, sm_ = workspace(q_abs.device).s_o, workspace(q_abs.device).s_ml
-            assert so.numel() >= splits * T * H * 512 and sm_.numel() >= splits * T * H * 2
-            ws_o, ws_ml = so, sm_
-    else:
-        splits = choose_kv_splits(md.num_reqs * row_tiles, max(md.seq_lens_cpu) if md.seq_lens_cpu else md.max_seq_len, _sms(q_abs.device))
-        if splits > 1:
-            ws_o, ws_ml = workspace(q_abs.device).attn(splits * T * H * 512, splits * T * H * 2)
+            w = workspace(q_abs.device)
+            ws_o, ws_ml = (w.attn_static if static else w.attn)(splits * T * H * lora, splits * T * H * 2)
     _LAUNCHES += 2 if splits > 1 else 1
-    return _C.mla_decode(q_abs.contiguous(), q_pe.contiguous(), latent_cache, md.query_start_loc, md.seq_lens, md.block_table, scale,
-                         md.max_query_len, splits, ws_o, ws_ml)
+    return _C.mla_decode(q_abs, q_pe, latent_cache, md.query_start_loc, md.seq_lens, md.block_table, scale, md.max_query_len, splits, ws_o, ws_ml, cos_sin,
+                         interleaved, fine)
+
+
+# ----------------------------------------------------------------------------- mLSTM
+MLSTM_CHUNK_MIN_LEN = 64           # portions of at least this many tokens take the chunked (tensor-core) kernels
+MLSTM_SEGMENT_BYTES = 64 << 20     # chunk states of a segment: what the L2 holds beside the step's activations
+
+
+def _mlstm_segments(md, H: int, D: int, V: int, device):
+    """(device tensor, [(offset, chunks, sequences)], whether short portions remain) of this step's chunk list, built once per step and
+    geometry from the host-side query lengths and cut into segments whose chunk states stay small."""
+    cache = md.__dict__.setdefault("_mlstm_segments", {})
+    if (H, D, V) in cache:
+        return cache[(H, D, V)]
+    qlens = getattr(md, "query_lens_cpu", None)
+    out = (None, [], True)
+    if qlens and max(qlens) >= MLSTM_CHUNK_MIN_LEN and not getattr(md, "is_uniform_decode", False) and _C.mlstm_chunkable(D, V):
+        chunks, t = [], 0
+        for r, n in enumerate(qlens):
+            if n >= MLSTM_CHUNK_MIN_LEN:
+                chunks += [(r, t + c) for c in range(0, n, 64)]
+            t += n
+        per = max(8, MLSTM_SEGMENT_BYTES // (8 * H * D * V))
+        flat, segs = [], []
+        for a in range(0, len(chunks), per):
+            part = chunks[a:a + per]
+            reqs, first, count, owner = [], [], [], []
+            for j, (r, _) in enumerate(part):
+                if not reqs or reqs[-1] != r:
+                    reqs.append(r)
+                    first.append(j)
+                    count.append(0)
+                count[-1] += 1
+                owner.append(len(reqs) - 1)
+            segs.append([len(flat), len(part), len(reqs)])
+            flat += [r for r, _ in part] + [t0 for _, t0 in part] + owner + reqs + first + count
+        host = torch.tensor(flat, dtype=torch.int32).pin_memory()
+        out = (host.to(device, non_blocking=True), segs, any(0 < n < MLSTM_CHUNK_MIN_LEN for n in qlens))
+        md.__dict__.setdefault("_mlstm_hosts", []).append(host)   # keep the pinned buffer alive until the copy has run
+    cache[(H, D, V)] = out
+    return out
+
+
+def mlstm(qkvg, gates, i_bias, f_bias, norm_w, eps, cap, H, D, V, state, md):
+    """Short portions (decoding included) run the recurrent kernel, portions of at least ``MLSTM_CHUNK_MIN_LEN`` tokens the chunked ones
+    (bf16); both include the head norm and the output gate."""
+    global _LAUNCHES
+    hi = md.has_initial_state if md.has_initial_state.dtype == torch.int32 else md.has_initial_state.to(torch.int32)
+    meta, segs, short = (None, [], True) if qkvg.dtype == torch.float32 else _mlstm_segments(md, H, D, V, qkvg.device)
+    _LAUNCHES += 3 * len(segs) + int(short or not segs)
+    S, n, m = state
+    return _C.mlstm(qkvg, gates, i_bias, f_bias, norm_w, eps, cap, H, D, V, S, n, m, md.query_start_loc, md.state_slots, hi, meta, segs,
+                    MLSTM_CHUNK_MIN_LEN, short)
+
+
+def sigmoid_mul(x, gate):
+    global _LAUNCHES
+    _LAUNCHES += 1
+    return _C.sigmoid_mul(x, gate)
 
 
 _REJ_STEP = [0]

@@ -33,12 +33,15 @@ def rms_norm(x: torch.Tensor, w: torch.Tensor, eps: float, residual: Optional[to
     return y.to(x.dtype), new_res
 
 
-def stream_join(part, x, post, scale, nxt, out_dtype=None, add=None, copy_out=None):
-    """fp32 residual stream: ``x' = x + scale * post(part) (+ add)``, ``y = nxt(x')``. ``x`` None starts a stream from ``part``; ``post`` /
-    ``nxt`` are (kind, weight, bias, eps, plus_one) with kind 1 RMS, 2 layer norm, or None; ``copy_out`` receives ``x'`` in its own dtype.
+def stream_join(part, x, post, scale, nxt, out_dtype=None, add=None, copy_out=None, mul=1.0):
+    """fp32 residual stream: ``x' = x + mul * scale * post(part) (+ add)``, ``y = nxt(x')``. ``x`` None starts a stream from ``part``;
+    ``post`` / ``nxt`` are (kind, weight, bias, eps, plus_one[, alpha]) with kind 1 RMS, 2 layer norm, 3 dynamic tanh
+    (``tanh(alpha x) w + b``), or None; ``copy_out`` receives ``x'`` in its own dtype.
     Everything is fp32; returns (y in ``out_dtype`` or None, x'), with ``x`` updated in place."""
     def norm(v, n):
-        kind, w, b, eps, plus = n
+        kind, w, b, eps, plus = n[:5]
+        if kind == 3:
+            return torch.tanh(n[5].float() * v) * w.float() + b.float()
         if kind == 2:
             v = v - v.mean(-1, keepdim=True)
         v = v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps)
@@ -50,6 +53,8 @@ def stream_join(part, x, post, scale, nxt, out_dtype=None, add=None, copy_out=No
         v = norm(v, post)
     if scale is not None:
         v = v * scale.float()
+    if mul != 1.0:
+        v = v * mul
     if add is not None:
         v = v + add.float()
     x = x.add_(v) if x is not None else v.clone()
@@ -109,9 +114,7 @@ def scaled_inv_freq(rotary_dim: int, theta: float, scaling: Optional[dict], devi
         if scaling.get("truncate", True):
             lo, hi = math.floor(lo), math.ceil(hi)
         lo, hi = max(lo, 0), min(hi, rotary_dim - 1)
-        if lo == hi:
-            hi += 0.001
-        ramp = ((torch.arange(rotary_dim // 2, dtype=torch.float32, device=device) - lo) / (hi - lo)).clamp(0, 1)
+        ramp = ((torch.arange(rotary_dim // 2, dtype=torch.float32, device=device) - lo) / max(hi - lo, 0.001)).clamp(0, 1)
         extrap = 1.0 - ramp
         out = inv / f * (1 - extrap) + inv * extrap
         if scaling.get("attention_factor") is not None:
@@ -294,6 +297,38 @@ def merge_attn_states(o1, lse1, o2, lse2):
     den = (w1 + w2).clamp_min(1e-30)
     o = (o1.float() * (w1 / den).unsqueeze(-1) + o2.float() * (w2 / den).unsqueeze(-1)).to(o1.dtype)
     return o, m + torch.log(den)
+
+
+def rope_interleaved(x: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor) -> torch.Tensor:
+    """Adjacent pairs (2i, 2i + 1) of ``x`` ``[T, heads, n]`` rotated; returns the input's dtype."""
+    xf = x.float()
+    x1, x2 = xf[..., 0::2], xf[..., 1::2]
+    c, s = cos.unsqueeze(1), sin.unsqueeze(1)
+    return torch.stack([x1 * c - x2 * s, x2 * c + x1 * s], dim=-1).flatten(-2).to(x.dtype)
+
+
+def rope_rows(x: torch.Tensor, positions, cos_sin, interleaved: bool) -> torch.Tensor:
+    """``x`` ``[T, heads, n]`` rotated over all n elements, pairs adjacent or (i, i + n/2)."""
+    n = x.shape[-1]
+    cs = cos_sin[positions.long()]
+    cos, sin = cs[:, : n // 2], cs[:, n // 2:]
+    return rope_interleaved(x, cos, sin) if interleaved else _rope_neox(x, cos, sin, n).to(x.dtype)
+
+
+def mla_prepare(q_latent, kv, q_w, kv_w, eps, positions, cos_sin, cache, slot_mapping, lora: int, lora_pad: int, interleaved: bool):
+    """Normalise the query latent (returned) and the key/value latent, rotate the shared key part, insert ``[latent | key part]`` into the
+    paged cache (rows without a slot go to the placeholder block 0). The cache may hold the key part at ``lora_pad`` >= ``lora``."""
+    c, _ = rms_norm(kv[:, :lora], kv_w, eps)
+    k_pe = rope_rows(kv[:, lora:].unsqueeze(1), positions, cos_sin, interleaved).squeeze(1)
+    rows = cache.view(-1, cache.shape[-1])
+    sm = slot_mapping.long().clamp(min=0)
+    if lora_pad != lora or rows.shape[1] != lora + k_pe.shape[1]:
+        new = torch.zeros(c.shape[0], rows.shape[1], dtype=cache.dtype, device=cache.device)
+        new[:, :lora], new[:, lora_pad: lora_pad + k_pe.shape[1]] = c.to(cache.dtype), k_pe.to(cache.dtype)
+    else:
+        new = torch.cat([c, k_pe], dim=-1).to(cache.dtype)
+    rows.index_copy_(0, sm, new)
+    return rms_norm(q_latent, q_w, eps)[0] if q_latent is not None else None
 
 
 def mla_decode(q_nope_abs, q_rope, latent_cache, block_table, query_start_loc, seq_lens, scale: float, kv_lora: int):
@@ -484,6 +519,45 @@ def gated_delta_rule(q, k, v, g, beta, state, query_start_loc, state_slots, has_
         if token_states is None or (b - a) > token_states.shape[1]:
             state[slot] = S.to(state.dtype)
     return out
+
+
+# ----------------------------------------------------------------------------- mLSTM
+def mlstm_gates(gates, i_bias, f_bias, cap: float):
+    """Log input gate and log forget gate ``[T, H]`` from the logits ``[T, 2H]``: both soft-capped, the forget gate through log-sigmoid."""
+    H = gates.shape[1] // 2
+    i = cap * torch.tanh((gates[:, :H].float() + i_bias.float()) / cap)
+    return i, F.logsigmoid(cap * torch.tanh((gates[:, H:].float() + f_bias.float()) / cap))
+
+
+def mlstm(qkvg, gates, i_bias, f_bias, norm_w, eps: float, cap: float, H: int, D: int, V: int, state, md):
+    """mLSTM over a variable-length batch, token by token, in fp32. With a running maximum m (0 before the first token):
+    ``m' = max(f + m, i)``; ``S' = e^(f + m - m') S + e^(i - m') k v^T``, n likewise with k alone;
+    ``o = S'^T q / (max(|n' q|, e^-m') + 1e-6)``. Each head's o is RMS-normalised, then scaled by ``norm_w`` and sigmoid(output gate)."""
+    S_all, n_all, m_all = state
+    T = qkvg.shape[0]
+    x = qkvg.float()
+    q = x[:, : H * D].view(T, H, D) * D ** -0.5
+    k = x[:, H * D: 2 * H * D].view(T, H, D)
+    v = x[:, 2 * H * D: 2 * H * D + H * V].view(T, H, V)
+    li, lf = mlstm_gates(gates, i_bias, f_bias, cap)
+    out = torch.zeros(T, H, V, device=x.device)
+    qsl, slots, init = md.query_start_loc.tolist(), md.state_slots.tolist(), md.has_initial_state.tolist()
+    for r in range(len(qsl) - 1):
+        if qsl[r + 1] <= qsl[r]:
+            continue
+        s = slots[r]
+        S, n, m = (t[s].clone() if init[r] else torch.zeros_like(t[s]) for t in (S_all, n_all, m_all))
+        for t in range(qsl[r], qsl[r + 1]):
+            new = torch.maximum(lf[t] + m, li[t])
+            keep, put = torch.exp(lf[t] + m - new).unsqueeze(-1), torch.exp(li[t] - new).unsqueeze(-1)
+            S = keep.unsqueeze(-1) * S + (put * k[t]).unsqueeze(-1) * v[t].unsqueeze(1)
+            n, m = keep * n + put * k[t], new
+            den = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
+            out[t] = torch.einsum("hd,hdv->hv", q[t], S) / den.unsqueeze(-1)
+        S_all[s], n_all[s], m_all[s] = S, n, m
+    y = out * torch.rsqrt(out.pow(2).mean(-1, keepdim=True) + eps)
+    y = y.reshape(T, H * V) * norm_w.float() * torch.sigmoid(x[:, 2 * H * D + H * V:])
+    return y.to(qkvg.dtype)
 
 
 # ----------------------------------------------------------------------------- MoE

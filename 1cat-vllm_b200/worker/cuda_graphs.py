@@ -43,17 +43,23 @@ class DecodeGraphs:
         attns = [l.self_attn for l in layers]
         self.own_plans = any(a.kv_shared or a.window_keep or a.bias_table is not None or (a.Hq, a.Hkv, a.D) != (attns[0].Hq, attns[0].Hkv, attns[0].D)
                              for a in attns)
+        mlas = [l.self_attn for l in mla]
+        self.own_plans = self.own_plans or bool(mla) and (bool(layers) or any((a.H, a.lora_pad) != (mlas[0].H, mlas[0].lora_pad) for a in mlas)) or not (layers or mla)
         self.max_span = 0   # the longest stretch of keys that a decode row of any layer walks (0: the whole context)
         if layers:
             a = layers[0].self_attn
             self.geom = (a.Hq, a.Hkv, a.D)
             K.workspace(runner.device).attn_static(32 * tmax * max(a.Hq * a.D for a in attns), 32 * tmax * 2 * max(a.Hq for a in attns))
+            for a in mlas:
+                K.workspace(runner.device).attn_static(32 * tmax * a.H * a.lora_pad, 32 * tmax * a.H * 2)
             spans = [K.attention_span(a.window, a.window_keep) for a in attns]
-            self.max_span = max(spans) if all(spans) else 0
+            self.max_span = max(spans) if all(spans) and not mla else 0
         elif mla:
-            a = mla[0].self_attn
-            self.geom = ("mla", a.H, 512)
-            K.workspace(runner.device).attn_static(32 * tmax * a.H * 512, 32 * tmax * a.H * 2)
+            self.geom = ("mla", mlas[0].H, mlas[0].lora_pad)
+            for a in mlas:
+                K.workspace(runner.device).attn_static(32 * tmax * a.H * a.lora_pad, 32 * tmax * a.H * 2)
+        else:
+            self.geom, self.max_span = ("state",), 1   # recurrent layers only: nothing depends on the context length
         # every mixer's decode path runs without host synchronisation on fixed addresses (attention, latent attention, Gated-DeltaNet
         # with its state slots; fused mixture-of-experts builds its work list on the device). What stays eager: experts that run the
         # per-expert loop (biased / clamped activations), pipeline stages, and anything without an attention geometry.
@@ -69,9 +75,9 @@ class DecodeGraphs:
         rp = self.sizes[bisect.bisect_left(self.sizes, R)]
         if self.own_plans:
             return rp, q, self._context_bucket(max_seq)
-        from onecat_vllm.ops.cuda import _sms, choose_decode_splits, choose_kv_splits
+        from onecat_vllm.ops.cuda import _sms, choose_decode_splits, plan_mla_splits
         if self.geom[0] == "mla":
-            want = choose_kv_splits(rp * (-(-q * self.geom[1] // 16)), max_seq, _sms(self.r.device))
+            want = plan_mla_splits(self.geom[1], self.geom[2], [q] * rp, [max_seq], _sms(self.r.device))
         else:
             want = choose_decode_splits(rp * self.geom[1], max_seq, _sms(self.r.device))
         s = 1  # bucketed to powers of two (rounding up keeps the grid sized for the live context)
@@ -98,7 +104,7 @@ class DecodeGraphs:
         if self.own_plans:
             md.seq_lens_cpu = [splits] * rp   # the context bucket; each layer's plan follows from it
         elif self.geom[0] == "mla":
-            md.attn_plan = (("mla", self.geom[1], 512), (q, 0, splits))
+            md.attn_plan = (self.geom, (q, 0, splits))
         else:
             Hq, Hkv, D = self.geom
             G = Hq // Hkv
@@ -113,6 +119,10 @@ class DecodeGraphs:
         r = self.r
         md = self._metadata(rp, q, splits)
         ids = r._view("ids", rp * q)
+        # the warm-up runs must not touch live requests (a recurrent state would advance once per run): they see a batch without tokens
+        live = r.d_pack.clone()
+        r.d_pack.zero_()
+        r._view("slot", r._seg["slot"]).fill_(-1)
         torch.cuda.synchronize()
         with torch.cuda.stream(self.stream):
             for _ in range(2):  # warm up allocator and lazy kernel attributes outside capture
@@ -123,6 +133,7 @@ class DecodeGraphs:
         n0 = K.launches()
         with torch.cuda.graph(g, pool=self.pool, stream=self.stream):
             out = r.model(ids, md, r.kv_caches)
+        r.d_pack.copy_(live)
         if self.pool is None:
             self.pool = g.pool()
         self.graphs[key] = (g, out, K.launches() - n0)  # kernels of ours inside one replay

@@ -20,6 +20,7 @@ import torch
 from onecat_vllm.config import VllmConfig
 from onecat_vllm.core.kv_cache_utils import KVCacheConfig, KVCacheSpec
 from onecat_vllm.core.sched_output import ModelRunnerOutput, SchedulerOutput
+from onecat_vllm.layers.common import state_tensors
 from onecat_vllm.logger import init_logger
 from onecat_vllm.ops import ref as ref_ops
 from onecat_vllm.parallel import state as ps
@@ -188,12 +189,11 @@ class ModelRunner:
         asz = torch.empty(0, dtype=self._attn_kv_dtype()).element_size()
         for name, layer in self.model.model.cache_layers():
             if layer.kind == "linear_attention":
-                (cd, kw), (hv, k, v) = layer.linear_attn.state_shapes()
-                nspec = self.num_spec + 1
-                specs[name] = KVCacheSpec("mamba", self.block_size, 0, 0, 0,
-                                                    state_bytes=(cd * kw * esz + hv * k * v * 4))
+                nbytes = sum(int(np.prod(shape)) * (esz if dt is None else torch.empty(0, dtype=dt).element_size())
+                             for shape, dt in state_tensors(layer.linear_attn))
+                specs[name] = KVCacheSpec("mamba", self.block_size, 0, 0, 0, state_bytes=nbytes)
             elif layer.kind == "mla":
-                specs[name] = KVCacheSpec("mla", self.block_size, 1, mc.kv_lora_rank + mc.qk_rope_head_dim, esz)
+                specs[name] = KVCacheSpec("mla", self.block_size, 1, layer.self_attn.cache_width, esz)
             else:
                 a = layer.self_attn
                 specs[name] = KVCacheSpec("full", self.block_size, a.Hkv, a.D, asz, tensors=1 if a.kv_shared else 2)
@@ -202,7 +202,7 @@ class ModelRunner:
         if self.mtp is not None:
             a = self.mtp.layer.self_attn
             if self.mc.use_mla:
-                specs["mtp.0"] = KVCacheSpec("mla", self.block_size, 1, mc.kv_lora_rank + mc.qk_rope_head_dim, esz)
+                specs["mtp.0"] = KVCacheSpec("mla", self.block_size, 1, a.cache_width, esz)
             else:
                 specs["mtp.0"] = KVCacheSpec("full", self.block_size, a.Hkv, mc.head_dim, asz)
         return specs
@@ -245,10 +245,8 @@ class ModelRunner:
         for name, layer in self.model.model.cache_layers():
             spec = kvc.layer_specs[name]
             if spec.kind == "mamba":
-                (cd, kw), (hv, k, v) = layer.linear_attn.state_shapes()
-                slots = kvc.num_state_slots
-                self.kv_caches.append((torch.zeros(slots, cd, kw, dtype=dt, device=dev),
-                                       torch.zeros(slots, hv, k, v, dtype=torch.float32, device=dev)))
+                self.kv_caches.append(tuple(torch.zeros(kvc.num_state_slots, *shape, dtype=sdt or dt, device=dev)
+                                            for shape, sdt in state_tensors(layer.linear_attn)))
             else:
                 self.kv_caches.append(alloc(spec))
         if self.mtp is not None:
@@ -854,7 +852,7 @@ class ModelRunner:
             c0 = st.num_computed_tokens
             if st.prompt_embeds is not None and c0 < st.num_prompt_tokens:
                 if emb is None:
-                    emb = self.model.model.embed_tokens(ids)
+                    emb = self.model.model.embed(ids)
                 n = min(q, st.num_prompt_tokens - c0)
                 emb[o:o + n] = st.prompt_embeds[c0:c0 + n]
             for f in st.mm_features or ():
@@ -862,7 +860,7 @@ class ModelRunner:
                 if lo >= hi:
                     continue
                 if emb is None:
-                    emb = self.model.model.embed_tokens(ids)
+                    emb = self.model.model.embed(ids)
                 emb[o + lo - c0: o + hi - c0] = self.encoder_cache[f.mm_hash][lo - f.offset: hi - f.offset]
             o += q
         return emb
@@ -1110,10 +1108,9 @@ class ModelRunner:
         dt = self._kv_dtype()
         for _, layer in self.model.model.cache_layers():
             if layer.kind == "linear_attention":
-                (cd, kw), (hv, k, v) = layer.linear_attn.state_shapes()
-                out.append((torch.zeros(1, cd, kw, dtype=dt, device=self.device), torch.zeros(1, hv, k, v, dtype=torch.float32, device=self.device)))
+                out.append(tuple(torch.zeros(1, *shape, dtype=sdt or dt, device=self.device) for shape, sdt in state_tensors(layer.linear_attn)))
             elif layer.kind == "mla":
-                out.append(torch.zeros(1, self.block_size, self.mc.kv_lora_rank + self.mc.qk_rope_head_dim, dtype=dt, device=self.device))
+                out.append(torch.zeros(1, self.block_size, layer.self_attn.cache_width, dtype=dt, device=self.device))
             else:
                 a = layer.self_attn
                 out.append(torch.zeros(1, 1 if a.kv_shared else 2, a.Hkv, self.block_size, a.D, dtype=dt, device=self.device))
