@@ -877,6 +877,8 @@ class VllmConfig:
         if m.residual_fp32 and (p.pipeline_parallel_size > 1 or self.speculative_config.method in ("mtp", "eagle", "eagle3")):
             raise ValueError(f"{m.architecture}: models with an fp32 residual stream are served without pipeline parallelism and without draft heads "
                              "that read the target's hidden states")
+        if m.layer_types and "mlstm" in m.layer_types and self.speculative_config.enabled:
+            raise ValueError(f"{m.architecture}: speculative decoding is not served for mLSTM layers (their states are not recorded per token)")
         if p.pipeline_parallel_size > 1:
             if p.pipeline_parallel_size > m.num_hidden_layers:
                 raise ValueError("pipeline_parallel_size exceeds the number of decoder layers")
