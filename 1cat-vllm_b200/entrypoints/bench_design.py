@@ -1,9 +1,15 @@
-"""Prefill and decode throughput of the Gabisun design beside the closest models of equal size, and its kernels beside theirs.
+"""Prefill and decode throughput of a design beside the closest models of equal size, and its kernels beside theirs.
 
-``python bench.py --design gabisun`` prints one JSON line per size. Random weights and token ids. The models share width, heads, head
-size, window, layer runs, vocabulary and tied embeddings: Starcoder2 (layer norms, ungated GELU feed-forward of the same width; its norms
-are PyTorch operations) and Mistral (every step fused; RMS norms, a gated feed-forward of 2/3 the width, so the same number of weights).
-Model throughput is device time of engine steps (CUDA events); kernels are timed alone with the L2 flushed before every launch."""
+``python bench.py --design gabisun|sepirax`` prints one JSON line per size. Random weights and token ids. Model throughput is device time
+of engine steps (CUDA events); kernels are timed alone with the L2 flushed before every launch.
+
+Gabisun: the models share width, heads, head size, window, layer runs, vocabulary and tied embeddings: Starcoder2 (layer norms, ungated
+GELU feed-forward of the same width; its norms are PyTorch operations) and Mistral (every step fused; RMS norms, a gated feed-forward of
+2/3 the width, so the same number of weights).
+
+Sepirax: beside DeepSeek-V2 (every layer latent attention with the same heads, latents and grouped softmax experts) and Qwen3-Next (Gated-
+DeltaNet in the place of the mLSTM layers with the same number of heads and states of 128 x 128, softmax attention in the place of latent
+attention, the same experts without groups)."""
 from __future__ import annotations
 
 import gc
@@ -148,6 +154,140 @@ def kernel_rows(s: dict, iters: int) -> list[dict]:
     gemm("logits", "gabisun, fp32 output", VOCAB, W, out_dtype=torch.float32)
     gemm("logits", "bf16 output", VOCAB, W)
     return rows
+
+
+SEPIRAX_SIZES = {
+    # width, layers (mLSTM and latent attention in turn), heads of both, latent attention (dim, rot, vdim, kv rank, q rank), state (dim, vdim), experts
+    "w2048": dict(width=2048, layers=12, heads=16, dim=128, rot=64, vdim=128, kv=512, q=768, sdim=128, svdim=128, experts=64, top=6, groups=8, keep=3, ff=512),
+    "w4096": dict(width=4096, layers=8, heads=32, dim=128, rot=64, vdim=128, kv=512, q=1536, sdim=128, svdim=128, experts=32, top=4, groups=4, keep=2, ff=1024),
+    "w2048s": dict(width=2048, layers=12, heads=32, dim=64, rot=32, vdim=64, kv=256, q=512, sdim=64, svdim=64, experts=16, top=4, groups=4, keep=2, ff=1024),
+}
+
+
+def sepirax_config(s: dict) -> dict:
+    mlp = dict(kind="moe", expert=dict(ff=s["ff"]), router=dict(experts=s["experts"], top=s["top"], groups=dict(count=s["groups"], keep=s["keep"])))
+    mem = dict(type="mlstm", mlp=mlp, mixer=dict(heads=s["heads"], dim=s["sdim"], vdim=s["svdim"], gate_cap=15.0))
+    att = dict(type="latent_attention", mlp=mlp, mixer=dict(heads=s["heads"], dim=s["dim"], rot_dim=s["rot"], vdim=s["vdim"], kv_rank=s["kv"], q_rank=s["q"],
+               scale=(s["dim"] + s["rot"]) ** -0.5, rot=dict(base=10000.0, dims=s["rot"], scaling=dict(factor=4.0, fast=32.0, slow=1.0, original=4096))))
+    return dict(architecture="Sepirax", width=s["width"], vocab=VOCAB, norm=dict(eps=1e-5), residual_mult=0.5, logit_softcap=30.0,
+                embedding=dict(scale=s["width"] ** 0.5), layers=[mem, att] * (s["layers"] // 2))
+
+
+def sepirax_like(s: dict, arch: str) -> dict:
+    cfg = dict(architectures=[arch], hidden_size=s["width"], num_hidden_layers=s["layers"], num_attention_heads=s["heads"], vocab_size=VOCAB,
+               max_position_embeddings=32768, rope_theta=10000.0, rms_norm_eps=1e-5, tie_word_embeddings=False, intermediate_size=s["ff"],
+               moe_intermediate_size=s["ff"], num_experts_per_tok=s["top"], norm_topk_prob=True)
+    if arch.startswith("Deepseek"):
+        return dict(cfg, num_key_value_heads=s["heads"], q_lora_rank=s["q"], kv_lora_rank=s["kv"], qk_nope_head_dim=s["dim"], qk_rope_head_dim=s["rot"],
+                    v_head_dim=s["vdim"], n_routed_experts=s["experts"], n_shared_experts=0, n_group=s["groups"], topk_group=s["keep"], scoring_func="softmax",
+                    first_k_dense_replace=0, routed_scaling_factor=1.0)
+    return dict(cfg, num_key_value_heads=max(s["heads"] // 4, 1), head_dim=128, num_experts=s["experts"], shared_expert_intermediate_size=0,
+                linear_num_key_heads=s["heads"], linear_num_value_heads=s["heads"], linear_key_head_dim=128, linear_value_head_dim=128,
+                linear_conv_kernel_dim=4, full_attention_interval=2, attn_output_gate=True, partial_rotary_factor=0.25)
+
+
+def sepirax_kernels(s: dict, iters: int) -> list[dict]:
+    """Each kernel of the design beside the like kernel of the closest models. Bytes and FLOPs are the algorithm's: what a kernel must read
+    and write once, and the products of latent attention in the form that needs fewest of them for its case."""
+    from types import SimpleNamespace
+    from onecat_vllm.ops import cuda as K
+    from onecat_vllm.ops.microbench import _peaks, timeit
+    pk, rows = _peaks(), []
+    W, H, L, R, E, top = s["width"], s["heads"], s["kv"], s["rot"], s["experts"], s["top"]
+    b = lambda *sh: torch.randn(*sh, device="cuda").bfloat16()
+    f32 = lambda *sh: torch.randn(*sh, device="cuda")
+
+    def row(kernel, case, who, fn, flops=0.0, nbytes=0.0):
+        ms = timeit(fn, iters)
+        t = max(flops / pk["bf16_tflops"] / 1e9, nbytes / pk["hbm_gbs"] / 1e6)
+        rows.append(dict(kernel=kernel, case=case, model=who, us=ms * 1e3, roofline_us=t * 1e3, frac_of_roofline=t / ms))
+
+    lp, rp = K.mla_padded_sizes(L, R)
+    table = f32(2 * PREFILL, R)
+    for case, n, q, S in (("prefill", 1, PREFILL, PREFILL), ("decode", DECODE_REQS, 1, DECODE_CTX)):
+        md, nblk = _meta(n, q, S)
+        cache, T = b(nblk, 16, lp + rp) * 0.3, n * q
+        cache[..., L:lp] = 0
+        cache[..., lp + R:] = 0
+        pairs = n * sum(range(S - q + 1, S + 1))
+        q_abs, q_pe = b(T, H, lp), b(T, H, R)
+        if case == "decode":
+            fl, by = 2.0 * H * pairs * (2 * L + R), 2.0 * (n * S * (L + R) + T * H * (2 * L + R))
+        else:
+            fl, by = 2.0 * H * pairs * (s["dim"] + R + s["vdim"]), 2.0 * (S * (L + R) + T * H * (s["dim"] + R + s["vdim"]))
+        for who, rest in (("sepirax (rotates q, two-term weights)", (table, False, True)), ("deepseek", (table, True, False))):
+            row("latent attention", case, who, lambda: K.mla_decode(q_abs, q_pe, cache, md, 0.1, lp, *rest), fl, by)
+        del cache
+    for case, n, q in (("prefill", 1, PREFILL), ("decode", DECODE_REQS, 1)):
+        T = n * q
+        md, _ = _meta(n, q, q)
+        md.state_slots = torch.arange(n, device="cuda", dtype=torch.int32)
+        md.has_initial_state = torch.ones(n, device="cuda", dtype=torch.int32)
+        md.is_uniform_decode = case == "decode"
+        for D, V in {(s["sdim"], s["svdim"]), (128, 128)}:
+            st = (f32(n, H, D, V), f32(n, H, D), f32(n, H))
+            x, g, bi, nw = b(T, 2 * H * (D + V)), f32(T, 2 * H), f32(H), b(H * V)
+            cost = lambda D, V: (4.0 * T * H * (D * V + 32 * (D + V)), 2.0 * T * H * (2 * D + 3 * V) + 8.0 * n * H * D * V)
+            row("recurrence", case, f"sepirax mLSTM {D}x{V}, head norm and gate included", lambda: K.mlstm(x, g, bi, bi, nw, 1e-5, 15.0, H, D, V, st, md), *cost(D, V))
+        D = V = 128
+        conv, st = b(n, 3 * H * D, 3), f32(n, H, D, V)
+        x, a, cw, al, z, nw = b(T, 3 * H * D), b(T, H), b(3 * H * D, 4), f32(H), b(T, H * V), b(V)
+        row("recurrence", case, "qwen3-next Gated-DeltaNet 128x128 with convolution, head norm and gate", lambda: K.rms_norm_gated(
+            K.gdn_forward(x, a, a, cw, al, al, conv, st, md, H, H, D, V).reshape(T, H * V), z, nw, 1e-5, H), *cost(D, V))
+    for T in (PREFILL, DECODE_REQS):
+        part, x32, w, res, al = b(T, W), f32(T, W), b(W), b(T, W), b(1)
+        row("norm", T, "sepirax join", lambda: K.stream_join(part, x32, None, None, (3, w, w, 0.0, False, al), torch.bfloat16, mul=0.5), nbytes=12.0 * T * W)
+        row("norm", T, "add + rms norm", lambda: K.rms_norm(part, w, 1e-5, res, False), nbytes=8.0 * T * W)
+        slot = torch.arange(T, device="cuda", dtype=torch.int32)
+        down = b(T, s["q"] + L + R + H * s["vdim"])
+        cache, wq, wk = b(T // 16 + 1, 16, lp + rp), b(s["q"]), b(L)
+        row("latent norms + rope + insert", T, "sepirax", lambda: K.mla_prepare(down[:, : s["q"]], down[:, s["q"]: s["q"] + L + R], wq, wk, 1e-5, slot, table, cache, slot, L, lp,
+                                                                               False), nbytes=4.0 * T * (s["q"] + L + R))
+        G = max(H // 4, 1)
+        kk, c2, cs = b(T, (H + 2 * G) * 128), b(T // 16 + 1, 2, G, 16, 128), torch.ones(T, 128, device="cuda")
+        row("latent norms + rope + insert", T, "rope + insert (qwen3-next)", lambda: K.rope_and_cache(
+            kk[:, : H * 128].view(T, H, 128), kk[:, H * 128: (H + G) * 128].view(T, G, 128), kk[:, (H + G) * 128:].view(T, G, 128), slot, cs, c2, slot, 128, None, None,
+            1e-5, False), nbytes=4.0 * T * (H + 2 * G) * 128)
+        o, gate = b(T, H * s["vdim"]), down[:, s["q"] + L + R:]
+        row("output gate", T, "sepirax", lambda: K.sigmoid_mul(o, gate), nbytes=6.0 * T * H * s["vdim"])
+        row("output gate", T, "qwen3-next (PyTorch)", lambda: o * torch.sigmoid(gate.float()).to(o.dtype), nbytes=6.0 * T * H * s["vdim"])
+        rc = SimpleNamespace(num_experts_per_tok=top, n_group=s["groups"], topk_group=s["keep"], scoring_func="softmax", norm_topk_prob=True, routed_scaling_factor=1.0)
+        z = f32(T, E)
+        zb = z.bfloat16()
+        row("router", T, "sepirax (fp32 logits)", lambda: K.route(z, rc, None), nbytes=T * (4.0 * E + 8.0 * top))
+        row("router", T, "deepseek (bf16 logits)", lambda: K.route(zb, rc, None), nbytes=T * (2.0 * E + 8.0 * top))
+
+        def gemm(name, who, N, Kd, **kw):
+            wt, xx = (torch.randn(N, Kd, device="cuda") * 0.02).bfloat16(), b(T, Kd)
+            out = torch.empty(T, -(-N // 8) * 8, dtype=kw.get("out_dtype", torch.bfloat16), device="cuda")[:, :N]
+            row(f"gemm {name}", T, who, lambda: K._gemm(xx, wt, None, None, out, None, N, N, N, 0, K.EPI_STORE, 1), flops=2.0 * T * N * Kd,
+                nbytes=2.0 * (N * Kd + T * Kd) + out.element_size() * T * N)
+        gemm("latent projections", "sepirax dq|dkv|gate", s["q"] + L + R + H * s["vdim"], W)
+        gemm("latent projections", "deepseek q_a", s["q"], W)
+        gemm("mixer input", "sepirax q|k|v|gate", 2 * H * (s["sdim"] + s["svdim"]), W)
+        gemm("mixer input", "qwen3-next q|k|v|z", 4 * H * 128, W)
+        gemm("gates", "sepirax input|forget, fp32 output", 2 * H, W, out_dtype=torch.float32)
+        gemm("gates", "qwen3-next b|a", 2 * H, W)
+        gemm("router logits", "sepirax, fp32 output", E, W, out_dtype=torch.float32)
+        gemm("router logits", "deepseek", E, W)
+    return rows
+
+
+def run_sepirax(steps: int, warmup: int, sizes=None, kernels: bool = True, clock_sampler=None) -> None:
+    for name, s in SEPIRAX_SIZES.items():
+        if sizes and name not in sizes:
+            continue
+        clocks = clock_sampler() if clock_sampler else None
+        models = {"Sepirax": sepirax_config(s), "DeepSeek-V2": sepirax_like(s, "DeepseekV2ForCausalLM"), "Qwen3-Next": sepirax_like(s, "Qwen3NextForCausalLM")}
+        res = {"design": "sepirax", "size": name, "dims": s, "dtype": "bf16", "data": "synthetic: random token ids and weights",
+               "workload": f"prefill: one {PREFILL}-token prompt a step; decode: {DECODE_REQS} requests at a context of about {DECODE_CTX}",
+               "l2": "model steps stream weights and caches larger than L2; kernels: L2 flushed before every launch",
+               "models": {k: model_throughput(c, steps, warmup) for k, c in models.items()}}
+        if kernels:
+            res["kernels"] = sepirax_kernels(s, max(5, steps // 6))
+        if clocks is not None:
+            res["clocks"] = clocks.stop()
+        print(json.dumps(res), flush=True)
 
 
 def run(steps: int, warmup: int, sizes=None, kernels: bool = True, clock_sampler=None) -> None:
