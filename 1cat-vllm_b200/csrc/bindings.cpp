@@ -768,7 +768,7 @@ torch::Tensor fused_moe_a2a(torch::Tensor x, torch::Tensor w13, torch::Tensor w2
 
 torch::Tensor mla_decode(torch::Tensor q_abs, torch::Tensor q_rope, torch::Tensor cache, torch::Tensor qsl, torch::Tensor seq_lens,
                          torch::Tensor block_table, double scale, int64_t max_q_len, int64_t splits, c10::optional<torch::Tensor> ws_o,
-                         c10::optional<torch::Tensor> ws_ml, c10::optional<torch::Tensor> cos_sin, bool interleaved, bool fine) {
+                         c10::optional<torch::Tensor> ws_ml, c10::optional<torch::Tensor> cos_sin, bool interleaved, bool fine, int64_t skip_min_len) {
   const auto et = q_abs.scalar_type();
   TORCH_CHECK(q_abs.is_cuda() && (et == torch::kBFloat16 || et == torch::kFloat32) && q_rope.scalar_type() == et && cache.scalar_type() == et, "bf16 or fp32 throughout");
   TORCH_CHECK(q_abs.is_contiguous() && cache.is_contiguous() && cache.dim() == 3 && q_rope.dim() == 3 && q_rope.stride(2) == 1, "q and cache layouts");
@@ -787,6 +787,7 @@ torch::Tensor mla_decode(torch::Tensor q_abs, torch::Tensor q_rope, torch::Tenso
   }
   p.interleaved = interleaved ? 1 : 0;
   p.fine = fine ? 1 : 0;
+  p.skip_min_len = (int)skip_min_len;
   p.cache = cache.data_ptr(); p.out = out.data_ptr();
   p.query_start_loc = qsl.data_ptr<int>(); p.seq_lens = seq_lens.data_ptr<int>(); p.block_table = block_table.data_ptr<int>();
   p.bt_stride = (int)block_table.stride(0); p.R = (int)seq_lens.size(0);
@@ -804,6 +805,58 @@ torch::Tensor mla_decode(torch::Tensor q_abs, torch::Tensor q_rope, torch::Tenso
 }
 
 bool mla_tensor_core_sizes(int64_t kv_lora, int64_t rope_pad) { return oc::mla_tensor_core_sizes((int)kv_lora, (int)rope_pad); }
+
+// Expanded-form prefill, first half: the contexts of the listed requests gathered from their pages and the query rows in whole chunks.
+// meta (int32): [request index | first gathered row] per listed request. Returns {latents [rows, lora_pad], key parts, queries}.
+std::vector<torch::Tensor> mla_prefill_inputs(torch::Tensor q, torch::Tensor cache, torch::Tensor qsl, torch::Tensor block_table, torch::Tensor positions,
+                                              torch::Tensor meta, int64_t num_long, int64_t rows, int64_t nope, int64_t lora_pad, torch::Tensor cos_sin,
+                                              bool interleaved) {
+  check_bf16(q, "q");
+  check_bf16(cache, "latent cache");
+  TORCH_CHECK(q.dim() == 3 && q.stride(2) == 1 && q.stride(1) == q.size(2) && cache.is_contiguous() && cache.dim() == 3, "q must be [T, H, nope + rope] with whole heads side by side");
+  TORCH_CHECK(meta.scalar_type() == torch::kInt32 && meta.numel() >= 2 * num_long && num_long > 0 && rows > 0, "prefill metadata");
+  TORCH_CHECK(block_table.scalar_type() == torch::kInt32 && positions.scalar_type() == torch::kInt32 && positions.numel() >= q.size(0), "metadata must be int32");
+  const c10::cuda::CUDAGuard guard(q.device());
+  oc::MlaPrefillParams p{};
+  p.T = (int)q.size(0); p.H = (int)q.size(1); p.nope = (int)nope; p.rope = (int)(q.size(2) - nope);
+  p.lora_pad = (int)lora_pad; p.rope_pad = (int)(cache.size(2) - lora_pad); p.bs = (int)cache.size(1);
+  TORCH_CHECK(p.rope >= 2 && p.rope_pad >= p.rope && cos_sin.scalar_type() == torch::kFloat32 && cos_sin.is_contiguous() && cos_sin.size(1) == p.rope, "rotary sizes");
+  p.NC = (p.nope + 63) / 64; p.RC = (p.rope + 63) / 64;
+  p.rows = (int)rows; p.num_long = (int)num_long; p.interleaved = interleaved ? 1 : 0;
+  TORCH_CHECK(p.rope_pad <= p.RC * 64, "the cached key part is wider than its chunks");
+  auto lat = torch::empty({rows, lora_pad}, q.options()), rot = torch::empty({rows, (int64_t)p.RC * 64}, q.options());
+  auto qo = torch::empty({p.T, p.H, (int64_t)(p.NC + p.RC) * 64}, q.options());
+  p.q = (const __nv_bfloat16*)q.data_ptr(); p.q_st = q.stride(0); p.q_out = (__nv_bfloat16*)qo.data_ptr();
+  p.cache = (const __nv_bfloat16*)cache.data_ptr(); p.lat = (__nv_bfloat16*)lat.data_ptr(); p.rot = (__nv_bfloat16*)rot.data_ptr();
+  p.query_start_loc = qsl.data_ptr<int>(); p.block_table = block_table.data_ptr<int>(); p.bt_stride = (int)block_table.stride(0);
+  p.positions = positions.data_ptr<int>(); p.cos_sin = cos_sin.data_ptr<float>();
+  p.long_req = meta.data_ptr<int>(); p.long_ctx = p.long_req + num_long;
+  TORCH_CHECK(oc::mla_prefill_inputs_launch(p, cur_stream()) == 0, "latent prefill inputs failed");
+  return {lat, rot, qo};
+}
+
+// Second half: causal attention of the listed requests' new tokens; rows of other requests in `out` [T, H, vd] stay as they are.
+void mla_prefill(torch::Tensor q, torch::Tensor kv, torch::Tensor rot, torch::Tensor out, torch::Tensor qsl, torch::Tensor seq_lens, torch::Tensor meta,
+                 int64_t num_long, int64_t num_q_tiles, int64_t nope, int64_t rope, double scale, bool fine) {
+  for (auto* t : {&q, &kv, &rot, &out}) {
+    check_bf16(*t, "prefill operands");
+    TORCH_CHECK(t->is_contiguous(), "prefill operands must be contiguous");
+  }
+  const c10::cuda::CUDAGuard guard(q.device());
+  oc::MlaPrefillParams p{};
+  p.T = (int)q.size(0); p.H = (int)q.size(1); p.nope = (int)nope; p.rope = (int)rope; p.vd = (int)out.size(2);
+  p.NC = (p.nope + 63) / 64; p.RC = (p.rope + 63) / 64;
+  p.rows = (int)kv.size(0); p.num_long = (int)num_long; p.num_q_tiles = (int)num_q_tiles; p.scale = (float)scale; p.fine = fine ? 1 : 0;
+  TORCH_CHECK(q.dim() == 3 && q.size(2) == (p.NC + p.RC) * 64 && kv.size(1) == (int64_t)p.H * (p.NC + (p.vd + 63) / 64) * 64 && rot.size(0) == p.rows && rot.size(1) == p.RC * 64 &&
+              out.size(0) == p.T && out.size(1) == p.H, "prefill operand shapes");
+  TORCH_CHECK(meta.scalar_type() == torch::kInt32 && meta.numel() >= 2 * num_long && qsl.scalar_type() == torch::kInt32 && seq_lens.scalar_type() == torch::kInt32, "metadata must be int32");
+  p.q_out = (__nv_bfloat16*)q.data_ptr(); p.kv = (const __nv_bfloat16*)kv.data_ptr(); p.rot = (__nv_bfloat16*)rot.data_ptr(); p.out = (__nv_bfloat16*)out.data_ptr();
+  p.query_start_loc = qsl.data_ptr<int>(); p.seq_lens = seq_lens.data_ptr<int>();
+  p.long_req = meta.data_ptr<int>(); p.long_ctx = p.long_req + num_long;
+  const int rc = oc::mla_prefill_launch(p, cur_stream());
+  TORCH_CHECK(rc == 0, "latent prefill launch failed: ", rc);
+}
+bool mla_prefill_sizes(int64_t nope, int64_t rope, int64_t vd) { return oc::mla_prefill_sizes((int)nope, (int)rope, (int)vd); }
 
 // Latent norms, rotation of the shared key part, cache insert; returns the normalised query latent when there is one.
 c10::optional<torch::Tensor> mla_prepare(c10::optional<torch::Tensor> q, torch::Tensor kv, c10::optional<torch::Tensor> q_w, torch::Tensor kv_w, double eps,
@@ -920,11 +973,12 @@ void read_status_async(torch::Tensor pinned) {
   oc::mla_read_status_async(p + 7, st);
   oc::moe_read_status_async(p + 8, st);
   oc::sampling_read_status_async(p + 9, st);
+  oc::mla_prefill_read_status_async(p + 10, st);
 }
 
 int64_t read_status(bool clear) {
   return (int64_t)(oc::gemm_read_status(clear) | oc::elementwise_read_status(clear) | oc::attention_read_status(clear) | oc::attention_tc_read_status(clear) |
-                   oc::comm_read_status(clear) | oc::gdn_read_status(clear) | oc::sampling_read_status(clear) | oc::moe_read_status(clear) | oc::mla_read_status(clear) | oc::ep_read_status(clear));
+                   oc::comm_read_status(clear) | oc::gdn_read_status(clear) | oc::sampling_read_status(clear) | oc::moe_read_status(clear) | oc::mla_read_status(clear) | oc::mla_prefill_read_status(clear) | oc::ep_read_status(clear));
 }
 
 // ---- symmetric slab + peer-memory reductions
@@ -1017,6 +1071,9 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("mla_decode", &mla_decode);
   m.def("mla_tensor_core_sizes", &mla_tensor_core_sizes);
   m.def("mla_prepare", &mla_prepare);
+  m.def("mla_prefill_inputs", &mla_prefill_inputs);
+  m.def("mla_prefill", &mla_prefill);
+  m.def("mla_prefill_sizes", &mla_prefill_sizes);
   m.def("mlstm", &mlstm);
   m.def("mlstm_chunkable", &mlstm_chunkable);
   m.def("sigmoid_mul", &sigmoid_mul);

@@ -188,6 +188,7 @@ struct MlaParams {
   const int* seq_lens;
   const int* block_table;
   int bt_stride, R, T, H, kv_lora, rope, rope_pad, bs, bs_shift, max_q_len, splits;
+  int skip_min_len;             // > 0: requests with at least this many new tokens are left to the prefill kernel
   int fine;                     // softmax weights enter the value product as two bf16 terms
   int f32;                      // element type of everything: fp32 instead of bf16
   float scale;
@@ -196,6 +197,26 @@ struct MlaParams {
 };
 int mla_decode_launch(const MlaParams& p, cudaStream_t st);
 bool mla_tensor_core_sizes(int kv_lora, int rope_pad);
+// Prefill in the expanded form: gathered latents -> per-head keys and values (a GEMM in between) -> causal attention.
+struct MlaPrefillParams {
+  const __nv_bfloat16* cache;   // [blocks][bs][lora_pad + rope_pad]
+  __nv_bfloat16 *lat, *rot;     // [rows][lora_pad], [rows][RC * 64]: the contexts of the listed requests, one after another
+  const __nv_bfloat16* q;       // [T][q_st] rows of H x (nope + rope)
+  long long q_st;
+  __nv_bfloat16* q_out;         // [T][H][(NC + RC) * 64]
+  const __nv_bfloat16* kv;      // [rows][H][(NC + VC) * 64] keys | values
+  __nv_bfloat16* out;           // [T][H][vd]
+  const int *query_start_loc, *seq_lens, *block_table, *positions;
+  const int *long_req, *long_ctx;   // per listed request: its index, its first row in the gathered buffers
+  const float* cos_sin;
+  int bt_stride, bs, T, H, rows, num_long, num_q_tiles, lora_pad, rope_pad, nope, rope, vd, NC, RC, interleaved, fine;
+  float scale;
+};
+bool mla_prefill_sizes(int nope, int rope, int vd);
+int mla_prefill_inputs_launch(const MlaPrefillParams& p, cudaStream_t st);   // gather + query rows
+int mla_prefill_launch(const MlaPrefillParams& p, cudaStream_t st);
+unsigned int mla_prefill_read_status(bool clear);
+void mla_prefill_read_status_async(unsigned int* dst, cudaStream_t st);
 struct MlaPrepareParams {
   const void *q, *kv;           // query latent [T][nq] or null; [T][lora + rope], pitches ld_q / ld_kv
   long long ld_q, ld_kv;

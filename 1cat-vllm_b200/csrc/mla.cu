@@ -69,7 +69,7 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g_ = lane >> 2, tg = lane & 3;
   const int r = blockIdx.y, rt = blockIdx.x, split = blockIdx.z;
   const int qs = p.query_start_loc[r], qlen = p.query_start_loc[r + 1] - qs, S = p.seq_lens[r];
-  if (qlen <= 0 || S <= 0) return;
+  if (qlen <= 0 || S <= 0 || (p.skip_min_len > 0 && qlen >= p.skip_min_len)) return;
   const int total_rows = qlen * p.H;         // row = token * H + head
   const int row0 = rt * ROWS;
   if (row0 >= total_rows) return;
@@ -263,7 +263,7 @@ __global__ void __launch_bounds__(128) mla_plain_kernel(const MlaParams p) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int r = blockIdx.y, row0 = blockIdx.x * PR;
   const int qs = p.query_start_loc[r], qlen = p.query_start_loc[r + 1] - qs, S = p.seq_lens[r];
-  if (qlen <= 0 || S <= 0 || row0 >= qlen * p.H) return;
+  if (qlen <= 0 || S <= 0 || row0 >= qlen * p.H || (p.skip_min_len > 0 && qlen >= p.skip_min_len)) return;
   const int nrows = min(PR, qlen * p.H - row0), ctx0 = S - qlen;
   const int kv_end = min(S, ctx0 + (row0 + nrows - 1) / p.H + 1);
   const int* bt = p.block_table + (size_t)r * p.bt_stride;

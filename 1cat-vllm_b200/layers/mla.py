@@ -57,11 +57,13 @@ class MLAAttention(nn.Module):
         # fp32 residual streams come with fp32 softmax weights: the tensor-core kernels then carry them as two bf16 terms
         self.fine_weights = cfg.residual_fp32
         self.lora_pad, self.rope_pad = self.lora, self.rope_d
+        self.prefill_sizes = False   # the expanded prefill kernel has a variant for this layer
         if torch.device(device).type == "cuda" and dt == torch.bfloat16:
             from onecat_vllm.ops import cuda as K
             self.lora_pad, self.rope_pad = K.mla_padded_sizes(self.lora, self.rope_d)
+            self.prefill_sizes = self.scale > 0 and self.lora_pad % 8 == 0 and self.rope_pad % 8 == 0
         self.cache_width = self.lora_pad + self.rope_pad   # elements of a cached token: latent | shared key part, each padded for the kernel
-        self._wuk = self._wuv = None
+        self._wuk = self._wuv = self._wkv = None
 
     def load_weight(self, pname: str, w: torch.Tensor, shard=None) -> None:
         """Key and value up-projections stored apart (``uk`` / ``uv``, rows head by head) take their places in ``kv_b_proj``."""
@@ -75,7 +77,7 @@ class MLAAttention(nn.Module):
         """Runs before the child layers' own repacking (parents come first in ``modules()``): the absorbed ``W_UK`` / ``W_UV`` are
         taken from ``kv_b_proj`` while its checkpoint tensors still exist — a quantised ``kv_b_proj`` is packed for the GEMM
         afterwards and can no longer be dequantised on the host side."""
-        self._wuk = self._wuv = None
+        self._wuk = self._wuv = self._wkv = None
         self._absorb(self.kv_b_proj.compute_dtype)
 
     def _absorb(self, dtype):
@@ -103,15 +105,36 @@ class MLAAttention(nn.Module):
         o = self._attend(q, md, latent_cache).reshape(T, self.H * self.vd)
         return self.o_proj(ops.sigmoid_mul(o, gate) if gate is not None else o)
 
+    def _expand(self, lat: torch.Tensor) -> torch.Tensor:
+        """Latents ``[rows, lora_pad]`` -> keys and values head by head, both padded to 64 columns."""
+        if self.nope % 64 == 0 and self.vd % 64 == 0 and self.lora_pad == self.lora:
+            return self.kv_b_proj(lat)
+        from onecat_vllm.ops import cuda as K
+        if self._wkv is None:
+            wuk, wuv = self._absorb(lat.dtype)
+            pad = lambda w: torch.nn.functional.pad(w, (0, 0, 0, -w.shape[1] % 64))
+            self._wkv = torch.cat([pad(wuk), pad(wuv)], 1).reshape(-1, self.lora_pad).contiguous()
+        return K.gemm_bf16(lat, self._wkv)
+
     def _attend(self, q, md, latent_cache):
-        """Attention over the cached latents with the key up-projection moved to the query and the value one to the result."""
+        """Attention over the cached latents. Single tokens and short portions: the key up-projection is moved to the query and the value one
+        to the result. Longer portions on the GPU (bf16): keys and values of the context are expanded and attended to per head."""
         wuk, wuv = self._absorb(q.dtype)
         if q.is_cuda:
             from onecat_vllm.ops import cuda as K
-            q_abs = K.per_head_matmul(q[..., : self.nope], wuk)
-            o_lat = K.mla_decode(q_abs, q[..., self.nope:], latent_cache, md, self.scale, self.lora_pad, self.rope.cos_sin, self.interleaved,
-                                 self.fine_weights)
-            return K.per_head_matmul(o_lat, wuv.transpose(1, 2))
+            plan = K.mla_prefill_plan(md, self.H, self.nope, self.rope_d, self.vd, self.lora_pad, q.device) if self.prefill_sizes else None
+            o = None
+            if plan is None or plan[-1]:
+                q_abs = K.per_head_matmul(q[..., : self.nope], wuk)
+                o_lat = K.mla_decode(q_abs, q[..., self.nope:], latent_cache, md, self.scale, self.lora_pad, self.rope.cos_sin, self.interleaved,
+                                     self.fine_weights, 0 if plan is None else K.MLA_PREFILL_MIN_LEN)
+                o = K.per_head_matmul(o_lat, wuv.transpose(1, 2))
+            if plan is not None:
+                if o is None:
+                    o = torch.empty(q.shape[0], self.H, self.vd, dtype=q.dtype, device=q.device)
+                K.mla_prefill(plan, q, latent_cache, md, self._expand, o, self.nope, self.rope_d, self.lora_pad, self.scale, self.rope.cos_sin,
+                              self.interleaved, self.fine_weights)
+            return o
         q_abs = torch.einsum("thn,hnl->thl", q[..., : self.nope], wuk)
         q_pe = ref.rope_rows(q[..., self.nope:], md.positions, self.rope.cos_sin, self.interleaved)
         o_lat = ref.mla_decode(q_abs, q_pe, latent_cache, md.block_table, md.query_start_loc, md.seq_lens, self.scale, self.lora)

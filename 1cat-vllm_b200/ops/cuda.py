@@ -752,26 +752,71 @@ def plan_mla_splits(H: int, lora: int, query_lens: list, seq_lens: list, num_sms
     return choose_kv_splits(len(query_lens) * -(-mq * H // 16), max(seq_lens), num_sms)
 
 
-def mla_decode(q_abs, q_pe, latent_cache, md, scale, lora, cos_sin=None, interleaved=True, fine=False):
+def mla_decode(q_abs, q_pe, latent_cache, md, scale, lora, cos_sin=None, interleaved=True, fine=False, skip_min_len=0):
     """Multi-query attention over the cached latents: ``q_abs`` ``[T, H, lora]``, ``q_pe`` ``[T, H, rope]`` (rotated by the kernel when
-    ``cos_sin`` is given). ``fine``: softmax weights in two bf16 terms."""
+    ``cos_sin`` is given). ``fine``: softmax weights in two bf16 terms. ``skip_min_len``: requests with at least that many new tokens are
+    left out (their rows of the result hold nothing)."""
     global _LAUNCHES
     T, H, _ = q_abs.shape
     ws_o = ws_ml = None
     splits = 1
+    ql, sl = md.query_lens_cpu or [md.max_query_len] * md.num_reqs, md.seq_lens_cpu or [md.max_seq_len]
+    if skip_min_len:
+        keep = [(q, s) for q, s in zip(ql, sl) if 0 < q < skip_min_len]
+        ql, sl = [q for q, _ in keep], [s for _, s in keep]
     if q_abs.dtype == torch.bfloat16 and _C.mla_tensor_core_sizes(lora, latent_cache.shape[-1] - lora):
         static = getattr(md, "static_ws", False)
         plan = getattr(md, "attn_plan", None)
         if static and plan is not None and plan[0][0] == "mla":
             splits = plan[1][2]  # captured decode graph: the split count is part of the graph's key
         else:
-            splits = plan_mla_splits(H, lora, md.query_lens_cpu or [md.max_query_len] * md.num_reqs, md.seq_lens_cpu or [md.max_seq_len], _sms(q_abs.device))
+            splits = plan_mla_splits(H, lora, ql, sl, _sms(q_abs.device))
         if splits > 1:
             w = workspace(q_abs.device)
             ws_o, ws_ml = (w.attn_static if static else w.attn)(splits * T * H * lora, splits * T * H * 2)
     _LAUNCHES += 2 if splits > 1 else 1
-    return _C.mla_decode(q_abs, q_pe, latent_cache, md.query_start_loc, md.seq_lens, md.block_table, scale, md.max_query_len, splits, ws_o, ws_ml, cos_sin,
-                         interleaved, fine)
+    return _C.mla_decode(q_abs, q_pe, latent_cache, md.query_start_loc, md.seq_lens, md.block_table, scale, max(ql), splits, ws_o, ws_ml, cos_sin,
+                         interleaved, fine, skip_min_len)
+
+
+MLA_PREFILL_MIN_LEN = 64           # portions of at least this many tokens attend in the expanded form
+MLA_PREFILL_BYTES = 4 << 30        # most memory of a step's expanded keys and values; beyond it the absorbed form runs
+
+
+def mla_prefill_plan(md, H: int, nope: int, rope: int, vd: int, lora_pad: int, device):
+    """(metadata, requests, context rows, query tiles, whether shorter portions remain) of the requests that attend in the expanded form in
+    this step, or None; built once per step from the host-side lengths."""
+    cache = md.__dict__.setdefault("_mla_prefill", {})
+    key = (H, nope, rope, vd, lora_pad)
+    if key in cache:
+        return cache[key]
+    ql, sl = getattr(md, "query_lens_cpu", None), getattr(md, "seq_lens_cpu", None)
+    out = None
+    if ql and sl and max(ql) >= MLA_PREFILL_MIN_LEN and not getattr(md, "is_uniform_decode", False) and _C.mla_prefill_sizes(nope, rope, vd):
+        reqs = [r for r, n in enumerate(ql) if n >= MLA_PREFILL_MIN_LEN]
+        rows = sum(sl[r] for r in reqs)
+        chunks = lambda n: -(-n // 64) * 64
+        if rows * (H * (chunks(nope) + chunks(vd)) + chunks(rope) + lora_pad) * 2 <= MLA_PREFILL_BYTES:
+            start, at = [], 0
+            for r in reqs:
+                start.append(at)
+                at += sl[r]
+            host = torch.tensor(reqs + start, dtype=torch.int32).pin_memory()
+            md.__dict__.setdefault("_mla_hosts", []).append(host)   # keep the pinned buffer alive until the copy has run
+            out = (host.to(device, non_blocking=True), len(reqs), rows, sum(-(-ql[r] // 128) for r in reqs), any(0 < n < MLA_PREFILL_MIN_LEN for n in ql))
+    cache[key] = out
+    return out
+
+
+def mla_prefill(plan, q, latent_cache, md, expand, out, nope, rope, lora_pad, scale, cos_sin, interleaved, fine):
+    """Causal attention of the planned requests in the expanded form, into their rows of ``out`` ``[T, H, vd]``. ``expand(latents)`` is the
+    per-head up-projection ``[rows, H * (keys | values)]`` with both parts padded to 64 columns."""
+    global _LAUNCHES
+    meta, n, rows, tiles, _ = plan
+    _LAUNCHES += 3
+    lat, rot, qp = _C.mla_prefill_inputs(q, latent_cache, md.query_start_loc, md.block_table, md.positions, meta, n, rows, nope, lora_pad, cos_sin, interleaved)
+    _C.mla_prefill(qp, expand(lat), rot, out, md.query_start_loc, md.seq_lens, meta, n, tiles, nope, rope, scale, fine)
+    return out
 
 
 # ----------------------------------------------------------------------------- mLSTM

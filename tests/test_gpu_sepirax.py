@@ -94,6 +94,49 @@ def test_latent_attention_kernels(H, lora, rope, fine, lens, dtype):
         o += n
 
 
+@pytest.mark.parametrize("fine", [True, False])
+@pytest.mark.parametrize("H,nope,rope,vd,lora", [(4, 128, 64, 128, 512), (3, 32, 32, 32, 64), (5, 20, 6, 10, 36), (2, 64, 16, 100, 200), (2, 48, 70, 64, 130), (1, 100, 2, 128, 64)])
+@pytest.mark.parametrize("lens", [[(200, 200), (1, 400), (3, 77), (64, 300), (130, 1000)], [(128, 128)], [(65, 65), (257, 513)], [(64, 64), (63, 63), (600, 601)]])
+def test_expanded_prefill_kernel(H, nope, rope, vd, lora, lens, fine):
+    """Portions of at least 64 tokens in the expanded form; the other requests' rows stay as they are."""
+    from onecat_vllm.ops import cuda as K
+    from onecat_vllm.ops import ref
+    g = torch.Generator().manual_seed(nope + vd)
+    dt = torch.bfloat16
+    lat = [torch.randn(s, lora + rope, generator=g).to(dt) for _, s in lens]
+    T = sum(n for n, _ in lens)
+    lp, rp = K.mla_padded_sizes(lora, rope)
+    cache, bt = latent_cache(lat, (lora, lp), lp + rp, dt)
+    q = torch.randn(T, H, nope + rope, generator=g).to(dt)
+    wk, wv = (torch.randn(H, n, lora, generator=g).mul(lora ** -0.5).to(dt) for n in (nope, vd))
+    pad = lambda w: torch.nn.functional.pad(w, (0, lp - lora, 0, -w.shape[1] % 64))
+    wkv = torch.cat([pad(wk), pad(wv)], 1).reshape(-1, lp).to(DEV)
+    md = Meta(lens, bt)
+    md.positions = torch.cat([torch.arange(s - n, s) for n, s in lens]).to(torch.int32).to(DEV)
+    table = ref.build_cos_sin_cache(rope, 2048, 300.0, DEV)
+    scale = 1.3 * (nope + rope) ** -0.5
+    out = torch.full((T, H, vd), 7.0, dtype=dt, device=DEV)
+    plan = K.mla_prefill_plan(md, H, nope, rope, vd, lp, torch.device(DEV))
+    assert plan[1] == sum(n >= 64 for n, _ in lens) and plan[-1] == any(n < 64 for n, _ in lens)
+    K.mla_prefill(plan, q.to(DEV), cache, md, lambda x: K.gemm_bf16(x, wkv), out, nope, rope, lp, scale, table, False, fine)
+    assert K.check_status() == 0
+    got, o = out.cpu().double(), 0
+    for (n, s), x in zip(lens, lat):
+        if n < 64:
+            assert (got[o:o + n] == 7.0).all()
+        else:
+            pos = torch.arange(s - n, s)
+            c = x[:, :lora].double()
+            k, v = (torch.einsum("sl,hnl->hsn", c, w.double()).to(dt).double() for w in (wk, wv))
+            qq = q[o:o + n].double().permute(1, 0, 2)
+            qr = O.rotate(qq[..., nope:], pos, dict(dims=rope, base=300.0)).to(dt).double()
+            sc = (qq[..., :nope] @ k.transpose(1, 2) + qr @ x[:, lora:].double().T) * scale
+            sc = sc.masked_fill(torch.arange(s).view(1, 1, -1) > pos.view(1, -1, 1), -math.inf)
+            want = (torch.softmax(sc, -1) @ v).permute(1, 0, 2)
+            assert (got[o:o + n] - want).abs().max() < (0.02 if fine else 0.03), (n, s)
+        o += n
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_one_latent_stands_out_everywhere(dtype):
     """A query that matches exactly one cached key, at page and tile borders, at the start and far away: found when it is visible, decoded
