@@ -2,7 +2,7 @@
 // folded into the query ("absorbed" form) and W_UV applied by the caller to the result.
 //   scores = [q_nope_abs | q_rope] . [latent | k_rope]^T   (512 + 64 wide for DeepSeek)       out = softmax(scores) . latent   (512 wide)
 // All heads of a token share the same keys, so heads are the rows of the tile: a CTA owns 16 (head, query-token) rows of one request
-// and one split of its context. Its four warps each compute the full 16 x 64 score tile (cheap next to the memory traffic) but own
+// and one split of its context. Its four warps each score a quarter of a tile's 64 keys, exchange the scores through shared memory and own
 // a different quarter of the output columns, so the accumulator stays in registers. The key tile is loaded once into
 // shared memory and serves as K (all columns) and as V (the latent ones): the latent is read from HBM exactly once per CTA.
 // Split-KV partials are merged by mla_combine_kernel. bf16 mma.sync.m16n8k16, fp32 softmax state in the exp2 domain.
@@ -62,6 +62,7 @@ __device__ __forceinline__ float rotated(const E* x, int j, int n, const float* 
 template <int DV, bool FINE>
 __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p) {
   constexpr int NB = DV / 32;                // output blocks of 8 columns per warp
+  __shared__ __align__(16) float sS[ROWS][KEYS + 8];
   extern __shared__ __align__(128) uint8_t smem[];
   const int DK = DV + p.rope_pad, PK = DV + ((p.rope_pad + 63) & ~63), CHK = DK / 8;
   uint8_t* sQ = smem;                        // [16][PK]
@@ -88,13 +89,13 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p) {
   const __nv_bfloat16* cache = reinterpret_cast<const __nv_bfloat16*>(p.cache);
   auto load_tile = [&](int tile, int buf) {
     uint8_t* dk = sK + (size_t)buf * KEYS * PK * 2;
-    for (int idx = threadIdx.x; idx < KEYS * CHK; idx += 128) {
-      const int row = idx / CHK, ch = idx % CHK, key = tile * KEYS + row;
+    for (int row = warp; row < KEYS; row += 4) {   // a warp copies whole rows
+      const int key = tile * KEYS + row;
       if (key < kv_end) {
-        const int blk = bt[key >> p.bs_shift];
-        cp16(dk + koff(row, ch, PK), cache + ((size_t)blk * p.bs + (key & (p.bs - 1))) * DK + ch * 8);
+        const __nv_bfloat16* src = cache + ((size_t)bt[key >> p.bs_shift] * p.bs + (key & (p.bs - 1))) * DK;
+        for (int ch = lane; ch < CHK; ch += 32) cp16(dk + koff(row, ch, PK), src + ch * 8);
       } else {
-        *reinterpret_cast<uint4*>(dk + koff(row, ch, PK)) = make_uint4(0, 0, 0, 0);
+        for (int ch = lane; ch < CHK; ch += 32) *reinterpret_cast<uint4*>(dk + koff(row, ch, PK)) = make_uint4(0, 0, 0, 0);
       }
     }
   };
@@ -129,20 +130,43 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p) {
     if (tile + 1 < hi) load_tile(tile + 1, buf ^ 1);
     asm volatile("cp.async.commit_group;" ::: "memory");
     const uint32_t kb = smem_u32(sK + (size_t)buf * KEYS * PK * 2), qb = smem_u32(sQ);
+    {
+      // scores of this warp's 16 keys (two accumulator sets, so that products of even and odd steps do not wait for each other)
+      float sc4[2][2][4];
+#pragma unroll
+      for (int e = 0; e < 2; ++e)
+#pragma unroll
+        for (int n = 0; n < 2; ++n) sc4[e][n][0] = sc4[e][n][1] = sc4[e][n][2] = sc4[e][n][3] = 0.f;
+      const int steps = DK / 16;
+#pragma unroll 2
+      for (int kk = 0; kk < steps; kk += 2) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          if (kk + e >= steps) break;
+          uint32_t a[4], b[4];
+          ldsm4(a, qb + koff(lane & 15, (kk + e) * 2 + (lane >> 4), PK));
+          ldsm4(b, kb + koff(warp * 16 + (lane & 7) + ((lane >> 4) << 3), (kk + e) * 2 + ((lane >> 3) & 1), PK));
+          mma16816(sc4[e][0], a, b[0], b[1]);
+          mma16816(sc4[e][1], a, b[2], b[3]);
+        }
+      }
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int h = 0; h < 2; ++h)
+          *reinterpret_cast<float2*>(&sS[g_ + h * 8][warp * 16 + n * 8 + tg * 2]) =
+              make_float2(sc4[0][n][h * 2] + sc4[1][n][h * 2], sc4[0][n][h * 2 + 1] + sc4[1][n][h * 2 + 1]);
+    }
+    __syncthreads();   // the tile's scores are complete; every warp takes all of them
     float s[8][4];
 #pragma unroll
-    for (int n = 0; n < 8; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
-    for (int kk = 0; kk < DK / 16; ++kk) {
-      uint32_t a[4];
-      ldsm4(a, qb + koff(lane & 15, kk * 2 + (lane >> 4), PK));
+    for (int n = 0; n < 8; ++n)
 #pragma unroll
-      for (int n2 = 0; n2 < 4; ++n2) {
-        uint32_t b[4];
-        ldsm4(b, kb + koff(n2 * 16 + (lane & 7) + ((lane >> 4) << 3), kk * 2 + ((lane >> 3) & 1), PK));
-        mma16816(s[n2 * 2], a, b[0], b[1]);
-        mma16816(s[n2 * 2 + 1], a, b[2], b[3]);
+      for (int h = 0; h < 2; ++h) {
+        const float2 v = *reinterpret_cast<const float2*>(&sS[g_ + h * 8][n * 8 + tg * 2]);
+        s[n][h * 2] = v.x;
+        s[n][h * 2 + 1] = v.y;
       }
-    }
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
       const int gr = row0 + g_ + h * 8;
@@ -377,11 +401,11 @@ __global__ void __launch_bounds__(128) mla_prepare_kernel(const MlaPrepareParams
 template <int DV, bool FINE>
 int decode_go(const MlaParams& p, cudaStream_t st) {
   const int PK = DV + ((p.rope_pad + 63) & ~63), smem = (ROWS + 2 * KEYS) * PK * 2;
-  if (smem > 227 * 1024) return -1;
+  if (smem > 220 * 1024) return -1;
   static bool configured_dev[kMaxDevices] = {};
   bool& configured = configured_dev[current_device_slot()];  // the limit is an attribute of (kernel, device)
   if (!configured) {
-    if (cudaFuncSetAttribute(mla_decode_kernel<DV, FINE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess) return -4;
+    if (cudaFuncSetAttribute(mla_decode_kernel<DV, FINE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024) != cudaSuccess) return -4;
     configured = true;
   }
   mla_decode_kernel<DV, FINE><<<dim3((p.max_q_len * p.H + ROWS - 1) / ROWS, p.R, p.splits), 128, smem, st>>>(p);
@@ -417,7 +441,7 @@ int plain_e(const MlaParams& p, cudaStream_t st) {
 
 bool mla_tensor_core_sizes(int kv_lora, int rope_pad) {
   const bool dv = kv_lora == 64 || kv_lora == 128 || kv_lora == 192 || kv_lora == 256 || kv_lora == 384 || kv_lora == 512;
-  return dv && rope_pad >= 16 && rope_pad % 16 == 0 && (ROWS + 2 * KEYS) * (kv_lora + ((rope_pad + 63) & ~63)) * 2 <= 227 * 1024;
+  return dv && rope_pad >= 16 && rope_pad % 16 == 0 && (ROWS + 2 * KEYS) * (kv_lora + ((rope_pad + 63) & ~63)) * 2 <= 220 * 1024;
 }
 
 int mla_decode_launch(const MlaParams& p, cudaStream_t st) {

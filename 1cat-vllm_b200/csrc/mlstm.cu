@@ -15,7 +15,7 @@
 //   scan kernel:   m' = max(F_C + m, mloc), S' = e^(F_C + m - m') S + e^(mloc - m') dS                        (elements in parallel)
 //   output kernel: num_t = e^(m0 - M_t) S0^T q_t + sum_{s<=t} e^(b_s - M_t) (q_t . k_s) v_s, den likewise, norm, gate
 // Products run on bf16 mma.sync; whatever is 32-bit by definition (S0, the weights) enters them as two bf16 terms (the rounded value and
-// what rounding took from it). The chunk states stay in L2: the host cuts the chunk list into segments of bounded size.
+// what rounding took from it). The host cuts the chunk list into segments, which bounds the memory of the chunk states.
 #include <type_traits>
 
 #include "common.cuh"
@@ -47,7 +47,7 @@ constexpr int RV = 64;    // state columns per CTA
 
 // HK: state rows per thread; a column is split over four lanes (lane = column + 8 * part, part p holds rows p * HK ..).
 template <typename E, int HK>
-__global__ void __launch_bounds__(256) mlstm_recurrent_kernel(const MlstmParams p) {
+__global__ void __launch_bounds__(256, HK <= 32 ? 3 : HK <= 64 ? 2 : 1) mlstm_recurrent_kernel(const MlstmParams p) {
   constexpr int KP = 4 * HK, NH = HK / 8;
   __shared__ __align__(16) float sq[RCH][KP], sk[RCH][KP];
   __shared__ float sv[RCH][RV], so[RCH][RV], si[RCH], sf[RCH], part_ss[2][RCH];
@@ -142,11 +142,12 @@ __global__ void __launch_bounds__(256) mlstm_recurrent_kernel(const MlstmParams 
       }
     }
   }
+  int pitch = V;
+  asm volatile("" : "+r"(pitch));   // the addresses are formed anew: keeping those of the loads would take two registers a row
+  float* Sw = Sg + (size_t)part * HK * pitch + col;
 #pragma unroll
-  for (int j = 0; j < HK; ++j) {
-    const int row = part * HK + j;
-    if (own && row < D) Sg[(size_t)row * V + col] = S[j];
-  }
+  for (int j = 0; j < HK; ++j)
+    if (own && part * HK + j < D) Sw[(size_t)j * pitch] = S[j];
   if (nz > 1) cluster_sync_all();   // the old n and m have been read, and nobody still reads this CTA's shared memory
   if (blockIdx.z == 0 && warp == 0) {
 #pragma unroll
@@ -193,6 +194,11 @@ __device__ __forceinline__ uint32_t bkn_addr(uint32_t base, int pitch, int k0, i
   return base + (uint32_t)(((k0 + (lane & 7) + ((lane >> 3) & 1) * 8) * pitch + n0 + (lane >> 4) * 8) * 2);
 }
 
+__device__ __forceinline__ void cp16(void* smem, const void* g) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(smem)), "l"(g) : "memory");
+}
+__device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+
 // rows x cols bf16 tile from global (row pitch ld) into shared memory (pitch `pitch`), zeros outside [vr) x [vc); pc: columns to fill
 __device__ __forceinline__ void load_tile(__nv_bfloat16* dst, int pitch, const __nv_bfloat16* src, long long ld, int rows, int pc, int vr, int vc, bool vec,
                                           int tid, int nt) {
@@ -200,9 +206,8 @@ __device__ __forceinline__ void load_tile(__nv_bfloat16* dst, int pitch, const _
     const int per = pc / 8;
     for (int e = tid; e < rows * per; e += nt) {
       const int i = e / per, s = (e - i * per) * 8;
-      uint4 v = make_uint4(0, 0, 0, 0);
-      if (i < vr && s < vc) v = *reinterpret_cast<const uint4*>(src + (size_t)i * ld + s);
-      *reinterpret_cast<uint4*>(dst + i * pitch + s) = v;
+      if (i < vr && s < vc) cp16(dst + i * pitch + s, src + (size_t)i * ld + s);   // the caller waits for the copies
+      else *reinterpret_cast<uint4*>(dst + i * pitch + s) = make_uint4(0, 0, 0, 0);
     }
   } else {
     for (int e = tid; e < rows * pc; e += nt) {
@@ -270,13 +275,15 @@ __global__ void __launch_bounds__(128) mlstm_chunk_kernel(const MlstmParams p) {
     }
   }
   load_tile(kt, PD, x + (size_t)H * D + (size_t)h * D, p.ld, C, Dp, n, D, p.vec_qk, tid, 128);
+  load_tile(vl, PV, x + 2 * (size_t)H * D + (size_t)h * V + c0, p.ld, C, KV, n, min(KV, V - c0), p.vec_v, tid, 128);
+  cp_wait();
   __syncthreads();
-  for (int e = tid; e < C * KV; e += 128) {   // weighted value rows as two terms
-    const int i = e / KV, c = e - i * KV;
-    const float v = i < n && c0 + c < V ? sw[i] * __bfloat162float(x[(size_t)i * p.ld + 2 * (size_t)H * D + (size_t)h * V + c0 + c]) : 0.f;
-    const __nv_bfloat16 hi = __float2bfloat16(v);
-    vh[i * PV + c] = hi;
-    vl[i * PV + c] = __float2bfloat16(v - __bfloat162float(hi));
+  for (int e = tid; e < C * KV / 2; e += 128) {   // weighted value rows as two terms, pairs of columns
+    const int i = e / (KV / 2), c = (e - i * (KV / 2)) * 2;
+    const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(vl + i * PV + c));
+    const float a = sw[i] * v.x, b = sw[i] * v.y;
+    *reinterpret_cast<uint32_t*>(vh + i * PV + c) = pack2(a, b);
+    *reinterpret_cast<uint32_t*>(vl + i * PV + c) = pack2(a - rounded(a), b - rounded(b));
   }
   if (blockIdx.z == 0)
     for (int d = tid; d < D; d += 128) {
@@ -403,7 +410,7 @@ __global__ void __launch_bounds__(256) mlstm_scan_kernel(const MlstmParams p) {
 __host__ __device__ __forceinline__ size_t out_smem(int D, int V) {
   const int Dp = (D + 15) & ~15, PD = Dp + 8;
   size_t kb = (size_t)C * PD * 2, pb = (size_t)2 * Dp * PS * 2;
-  return (size_t)C * PD * 2 + (kb > pb ? kb : pb) + (size_t)C * PS * 2 + (size_t)C * (((V + NS - 1) / NS) * NS + 4) * 4;
+  return (size_t)C * PD * 2 + (kb > pb ? kb : pb) + (size_t)C * PS * 2 + (size_t)C * (((V + NS - 1) / NS) * NS + 4) * 4;   // the last part holds n first
 }
 
 // grid (chunks of the segment, H), 128 threads; warp w owns tokens 16 w .. 16 w + 15.
@@ -435,14 +442,25 @@ __global__ void __launch_bounds__(128) mlstm_output_kernel(const MlstmParams p) 
   }
   load_tile(qt, PD, x + (size_t)h * D, p.ld, C, Dp, n, D, p.vec_qk, tid, 128);
   load_tile(kt, PD, x + (size_t)H * D + (size_t)h * D, p.ld, C, Dp, n, D, p.vec_qk, tid, 128);
+  for (int d = tid; d < Dp; d += 128) so[d] = d < D ? p.ws_n[((size_t)ci * H + h) * D + d] : 0.f;   // n ahead of the chunk
+  cp_wait();
   __syncthreads();
   {
     const int row = tid >> 1, half = tid & 1;
-    const float* n0 = p.ws_n + ((size_t)ci * H + h) * D;
-    float a = 0.f;
-    for (int d = half; d < D; d += 2) a = fmaf(__bfloat162float(qt[row * PD + d]), n0[d], a);
-    a += __shfl_xor_sync(0xffffffffu, a, 1);
-    if (half == 0) snq[row] = a;
+    float a[2] = {0.f, 0.f};
+    for (int d = half * 8; d < Dp; d += 16) {
+      const uint4 raw = *reinterpret_cast<const uint4*>(qt + row * PD + d);
+      const __nv_bfloat162* q2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float2 q = __bfloat1622float2(q2[e]);
+        a[0] = fmaf(q.x, so[d + 2 * e], a[0]);
+        a[1] = fmaf(q.y, so[d + 2 * e + 1], a[1]);
+      }
+    }
+    a[0] += a[1];
+    a[0] += __shfl_xor_sync(0xffffffffu, a[0], 1);
+    if (half == 0) snq[row] = a[0];
   }
   __syncthreads();
   const uint32_t sq = smem_u32(qt), sk = smem_u32(kt), sv = smem_u32(vt);
@@ -505,6 +523,7 @@ __global__ void __launch_bounds__(128) mlstm_output_kernel(const MlstmParams p) 
     load_tile(kt, PS, plane + c0, V, Dp, NS, D, vc, p.vec_v, tid, 128);
     load_tile(kt + Dp * PS, PS, plane + DV + c0, V, Dp, NS, D, vc, p.vec_v, tid, 128);
     load_tile(vt, PS, x + 2 * (size_t)H * D + (size_t)h * V + c0, p.ld, C, NS, n, vc, p.vec_v, tid, 128);
+    cp_wait();
     __syncthreads();
     float in[4][4], out[4][4];
 #pragma unroll
@@ -555,18 +574,28 @@ __global__ void __launch_bounds__(128) mlstm_output_kernel(const MlstmParams p) 
   __syncwarp();
   const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(p.norm_w) + (size_t)h * V;
   __nv_bfloat16* y = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)tc * H * V + (size_t)h * V;
-  for (int i = r0; i < min(r0 + 16, n); ++i) {
-    const __nv_bfloat16* gate = x + (size_t)i * p.ld + 2 * (size_t)H * D + (size_t)H * V + (size_t)h * V;
-    if (p.vec_v && (V & 1) == 0) {
-      for (int c = lane * 2; c < V; c += 64) {
-        const float2 o = *reinterpret_cast<const float2*>(so + i * PO + c);
-        const float2 wg = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(w + c)), gg = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gate + c));
-        *reinterpret_cast<uint32_t*>(y + (size_t)i * H * V + c) = pack2(o.x * sinv[i] * wg.x * sigmoid(gg.x), o.y * sinv[i] * wg.y * sigmoid(gg.y));
+  const __nv_bfloat16* gate = x + 2 * (size_t)H * D + (size_t)H * V + (size_t)h * V;
+  const int rows = min(16, n - r0);
+  if (p.vec_v && (V & 1) == 0) {
+    for (int c = lane * 2; c < V; c += 64) {
+      const float2 wg = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(w + c));
+      for (int i0 = 0; i0 < rows; i0 += 8) {   // the gates of eight rows are in flight together
+        uint32_t gr[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) gr[e] = i0 + e < rows ? *reinterpret_cast<const uint32_t*>(gate + (size_t)(r0 + i0 + e) * p.ld + c) : 0u;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          const int i = r0 + i0 + e;
+          if (i0 + e >= rows) continue;
+          const float2 o = *reinterpret_cast<const float2*>(so + i * PO + c), gg = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gr[e]));
+          *reinterpret_cast<uint32_t*>(y + (size_t)i * H * V + c) = pack2(o.x * sinv[i] * wg.x * sigmoid(gg.x), o.y * sinv[i] * wg.y * sigmoid(gg.y));
+        }
       }
-    } else {
-      for (int c = lane; c < V; c += 32)
-        y[(size_t)i * H * V + c] = __float2bfloat16(so[i * PO + c] * sinv[i] * __bfloat162float(w[c]) * sigmoid(__bfloat162float(gate[c])));
     }
+  } else {
+    for (int i = r0; i < r0 + rows; ++i)
+      for (int c = lane; c < V; c += 32)
+        y[(size_t)i * H * V + c] = __float2bfloat16(so[i * PO + c] * sinv[i] * __bfloat162float(w[c]) * sigmoid(__bfloat162float(gate[(size_t)i * p.ld + c])));
   }
 }
 
@@ -623,7 +652,7 @@ int mlstm_recurrent_launch(const MlstmParams& p, cudaStream_t st) {
   return p.f32 ? recurrent_e<float>(p, st) : recurrent_e<__nv_bfloat16>(p, st);
 }
 
-bool mlstm_chunkable(int D, int V) { return D >= 1 && D <= 512 && V >= 1 && V <= 512 && out_smem(D, V) <= 200 * 1024; }
+bool mlstm_chunkable(int D, int V) { return D >= 1 && D <= 512 && V >= 1 && V <= 512 && out_smem(D, V) <= 220 * 1024; }
 
 int mlstm_chunk_launch(const MlstmParams& p, int num_chunks, int num_long, cudaStream_t st) {
   if (num_chunks == 0 || num_long == 0) return 0;
@@ -631,8 +660,8 @@ int mlstm_chunk_launch(const MlstmParams& p, int num_chunks, int num_long, cudaS
   static bool configured_dev[kMaxDevices] = {};
   bool& configured = configured_dev[current_device_slot()];
   if (!configured) {
-    if (cudaFuncSetAttribute(mlstm_chunk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess) return -4;
-    if (cudaFuncSetAttribute(mlstm_output_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess) return -4;
+    if (cudaFuncSetAttribute(mlstm_chunk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024) != cudaSuccess) return -4;
+    if (cudaFuncSetAttribute(mlstm_output_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024) != cudaSuccess) return -4;
     configured = true;
   }
   const int Dp = (p.D + 15) & ~15;

@@ -215,6 +215,15 @@ def sepirax_kernels(s: dict, iters: int) -> list[dict]:
             fl, by = 2.0 * H * pairs * (2 * L + R), 2.0 * (n * S * (L + R) + T * H * (2 * L + R))
         else:
             fl, by = 2.0 * H * pairs * (s["dim"] + R + s["vdim"]), 2.0 * (S * (L + R) + T * H * (s["dim"] + R + s["vdim"]))
+        if case == "prefill":
+            # what the engine runs for prompts: latents gathered and expanded, then tcgen05 attention (deepseek: the same with plain weights)
+            wkv = b(H * (-(-s["dim"] // 64) * 64 + -(-s["vdim"] // 64) * 64), lp) * 0.05
+            md.positions = torch.arange(S, device="cuda", dtype=torch.int32)
+            plan = K.mla_prefill_plan(md, H, s["dim"], R, s["vdim"], lp, torch.device("cuda"))
+            qq, out = b(T, H, s["dim"] + R), b(T, H, s["vdim"])
+            for who, inter, fine in (("sepirax, two-term weights", False, True), ("deepseek", True, False)):
+                row("latent attention", case, who, lambda: K.mla_prefill(plan, qq, cache, md, lambda x: K.gemm_bf16(x, wkv), out, s["dim"], R, lp, 0.1, table, inter, fine), fl, by)
+            continue
         for who, rest in (("sepirax (rotates q, two-term weights)", (table, False, True)), ("deepseek", (table, True, False))):
             row("latent attention", case, who, lambda: K.mla_decode(q_abs, q_pe, cache, md, 0.1, lp, *rest), fl, by)
         del cache

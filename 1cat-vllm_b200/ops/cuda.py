@@ -747,9 +747,9 @@ def per_head_matmul(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
 
 
 def plan_mla_splits(H: int, lora: int, query_lens: list, seq_lens: list, num_sms: int) -> int:
-    """KV splits of a latent-attention launch."""
-    mq = max(query_lens)
-    return choose_kv_splits(len(query_lens) * -(-mq * H // 16), max(seq_lens), num_sms)
+    """KV splits of a latent-attention launch: as many CTAs fit an SM as two key tiles and the queries leave room for."""
+    per_sm = max(1, min(4, (227 << 10) // ((16 + 2 * 64) * (lora + 64) * 2 + 6144)))
+    return choose_decode_splits(len(query_lens) * -(-max(query_lens) * H // 16), max(seq_lens), num_sms, per_sm)
 
 
 def mla_decode(q_abs, q_pe, latent_cache, md, scale, lora, cos_sin=None, interleaved=True, fine=False, skip_min_len=0):
@@ -821,7 +821,7 @@ def mla_prefill(plan, q, latent_cache, md, expand, out, nope, rope, lora_pad, sc
 
 # ----------------------------------------------------------------------------- mLSTM
 MLSTM_CHUNK_MIN_LEN = 64           # portions of at least this many tokens take the chunked (tensor-core) kernels
-MLSTM_SEGMENT_BYTES = 64 << 20     # chunk states of a segment: what the L2 holds beside the step's activations
+MLSTM_SEGMENT_BYTES = 256 << 20    # chunk states of a segment (measured: smaller ones pay in half-filled waves what they save in traffic)
 
 
 def _mlstm_segments(md, H: int, D: int, V: int, device):
