@@ -241,7 +241,7 @@ mla_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       xch[half * TQ + row] = raw;
       pair_sync();
       if (!ok || *abort_flag) { ok = false; return; }
-      // the scale may be negative in no model: scaling commutes with the maximum
+      // the scale is positive (the launcher checks): it commutes with the maximum
       const float mx = fmaxf(m, fmaxf(raw, xch[(half ^ 1) * TQ + row]) * sl2);
       const float m_use = (mx == -INFINITY) ? 0.f : mx;
       alpha[j & 1] = (m == -INFINITY) ? 0.f : ex2(m - m_use);
@@ -356,32 +356,37 @@ __global__ void __launch_bounds__(256) mla_gather_kernel(const MlaPrefillParams 
   for (int c = lane; c < p.RC * 8; c += 32) rot[c] = c < p.rope_pad / 8 ? src[p.lora_pad / 8 + c] : make_uint4(0, 0, 0, 0);
 }
 
-// Query rows [unrotated | rotated] in whole chunks. Two elements per thread.
+// Query rows [unrotated | rotated] in whole chunks: one warp per (token, head), two elements per lane and step.
 __global__ void __launch_bounds__(256) mla_query_kernel(const MlaPrefillParams p) {
-  const int QP = (p.NC + p.RC) * 64, per = QP / 2;
-  const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
-  if (i >= (long long)p.T * p.H * per) return;
-  const int j = (int)(i % per) * 2;
-  const long long th = i / per;
-  const int t = (int)(th / p.H);
-  const __nv_bfloat16* q = p.q + (size_t)t * p.q_st + (size_t)(th % p.H) * (p.nope + p.rope);
-  float v[2];
-#pragma unroll
-  for (int e = 0; e < 2; ++e) {
-    const int c = j + e, k = c - p.NC * 64;
-    v[e] = 0.f;
-    if (k < 0) {
-      if (c < p.nope) v[e] = __bfloat162float(q[c]);
-    } else if (k < p.rope) {
-      const int hf = p.rope / 2, a = p.interleaved ? k >> 1 : (k < hf ? k : k - hf);
-      const bool second = p.interleaved ? (k & 1) : k >= hf;
-      const float* cs = p.cos_sin + (size_t)p.positions[t] * p.rope;
-      const __nv_bfloat16* x = q + p.nope;
-      const float u = __bfloat162float(x[p.interleaved ? 2 * a : a]), w = __bfloat162float(x[p.interleaved ? 2 * a + 1 : a + hf]), cc = cs[a], ss = cs[hf + a];
-      v[e] = second ? w * cc + u * ss : u * cc - w * ss;
-    }
+  const int row = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= p.T * p.H) return;
+  const int t = row / p.H, N = p.NC * 64, QP = N + p.RC * 64, hf = p.rope / 2;
+  const __nv_bfloat16* q = p.q + (size_t)t * p.q_st + (size_t)(row - t * p.H) * (p.nope + p.rope);
+  const __nv_bfloat16* x = q + p.nope;
+  const float* cs = p.cos_sin + (size_t)p.positions[t] * p.rope;
+  __nv_bfloat162* dst = reinterpret_cast<__nv_bfloat162*>(p.q_out + (size_t)row * QP);
+  const __nv_bfloat16 zero = __float2bfloat16(0.f);
+  for (int j = lane; j < N / 2; j += 32) {
+    __nv_bfloat162 v;
+    v.x = 2 * j < p.nope ? q[2 * j] : zero;
+    v.y = 2 * j + 1 < p.nope ? q[2 * j + 1] : zero;
+    dst[j] = v;
   }
-  *reinterpret_cast<__nv_bfloat162*>(p.q_out + (size_t)th * QP + j) = __floats2bfloat162_rn(v[0], v[1]);
+  for (int j = lane; j < p.RC * 32; j += 32) {
+    float v[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int k = 2 * j + e;
+      v[e] = 0.f;
+      if (k < p.rope) {
+        const int a = p.interleaved ? k >> 1 : (k < hf ? k : k - hf);
+        const bool second = p.interleaved ? (k & 1) : k >= hf;
+        const float u = __bfloat162float(x[p.interleaved ? 2 * a : a]), w = __bfloat162float(x[p.interleaved ? 2 * a + 1 : a + hf]), cc = cs[a], ss = cs[hf + a];
+        v[e] = second ? w * cc + u * ss : u * cc - w * ss;
+      }
+    }
+    dst[N / 2 + j] = __floats2bfloat162_rn(v[0], v[1]);
+  }
 }
 
 typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
@@ -441,8 +446,7 @@ int mla_prefill_inputs_launch(const MlaPrefillParams& p, cudaStream_t st) {
   if (p.rows <= 0 || p.T <= 0 || p.num_long <= 0) return 0;
   if (p.lora_pad % 8 || p.rope_pad % 8 || ((uintptr_t)p.cache & 15)) return -1;
   mla_gather_kernel<<<(p.rows + 7) / 8, 256, 0, st>>>(p);
-  const long long n = (long long)p.T * p.H * (p.NC + p.RC) * 32;
-  mla_query_kernel<<<(unsigned)((n + 255) / 256), 256, 0, st>>>(p);
+  mla_query_kernel<<<(p.T * p.H + 7) / 8, 256, 0, st>>>(p);
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
 }
 
