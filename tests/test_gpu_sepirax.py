@@ -62,7 +62,7 @@ LENS = [[(200, 200), (1, 400), (3, 77), (64, 300), (1, 1)], [(1, 1500), (1, 16),
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("H,lora,rope,fine", [(8, 64, 32, True), (5, 40, 6, True), (16, 512, 64, True), (16, 512, 64, False), (3, 200, 24, True), (7, 130, 64, False),
+@pytest.mark.parametrize("H,lora,rope,fine", [(6, 64, 48, True), (5, 40, 6, True), (16, 512, 64, True), (16, 512, 64, False), (3, 200, 24, True), (7, 130, 64, False),
                                               (32, 320, 96, True), (1, 12, 2, True), (4, 600, 16, True)])
 @pytest.mark.parametrize("lens", LENS)
 def test_latent_attention_kernels(H, lora, rope, fine, lens, dtype):
@@ -95,7 +95,7 @@ def test_latent_attention_kernels(H, lora, rope, fine, lens, dtype):
 
 
 @pytest.mark.parametrize("fine", [True, False])
-@pytest.mark.parametrize("H,nope,rope,vd,lora", [(4, 128, 64, 128, 512), (3, 32, 32, 32, 64), (5, 20, 6, 10, 36), (2, 64, 16, 100, 200), (2, 48, 70, 64, 130), (1, 100, 2, 128, 64)])
+@pytest.mark.parametrize("H,nope,rope,vd,lora", [(4, 128, 64, 128, 512), (3, 32, 48, 32, 64), (5, 20, 6, 10, 36), (2, 64, 16, 100, 200), (2, 48, 70, 64, 130), (1, 100, 2, 128, 64)])
 @pytest.mark.parametrize("lens", [[(200, 200), (1, 400), (3, 77), (64, 300), (130, 1000)], [(128, 128)], [(65, 65), (257, 513)], [(64, 64), (63, 63), (600, 601)]])
 def test_expanded_prefill_kernel(H, nope, rope, vd, lora, lens, fine):
     """Portions of at least 64 tokens in the expanded form; the other requests' rows stay as they are."""
@@ -159,7 +159,7 @@ def test_one_latent_stands_out_everywhere(dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("nq,lora,rope,interleaved", [(96, 64, 32, False), (30, 36, 6, False), (0, 512, 64, True), (1536, 512, 64, True)])
+@pytest.mark.parametrize("nq,lora,rope,interleaved", [(80, 64, 48, False), (30, 36, 6, False), (0, 512, 64, True), (1536, 512, 64, True)])
 def test_latent_prepare_kernel(nq, lora, rope, interleaved, dtype):
     from onecat_vllm import ops
     from onecat_vllm.layers.common import RMSNorm
@@ -210,7 +210,7 @@ def mlstm_want(x, gates, bi, bf, nw, eps, cap, H, D, V, state):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("H,D,V", [(4, 48, 64), (3, 20, 72), (2, 128, 128), (1, 256, 512), (2, 9, 21), (1, 130, 200), (1, 512, 64), (2, 64, 300)])
+@pytest.mark.parametrize("H,D,V", [(4, 56, 64), (3, 20, 72), (2, 128, 128), (1, 256, 512), (2, 9, 21), (1, 130, 200), (1, 512, 64), (2, 64, 300)])
 def test_mlstm_kernels(H, D, V, dtype, monkeypatch):
     """Prompts, portions and single tokens in one batch over shuffled slots, then the same sequences go on: outputs and states equal the
     token-by-token float64 recurrence of each sequence alone."""
@@ -282,7 +282,7 @@ def test_sigmoid_mul_kernel(T, n, off, dtype):
     assert torch.allclose(got, x.double() * torch.sigmoid(z[:, off: off + n].double()), atol=1e-6, rtol=5e-3 if dtype == torch.bfloat16 else 1e-6)
 
 
-@pytest.mark.parametrize("H", [4096, 320, 100, 77])
+@pytest.mark.parametrize("H", [4096, 336, 100, 77])
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_dynamic_tanh_join_kernel(H, dtype):
     from onecat_vllm import ops
@@ -299,7 +299,7 @@ def test_dynamic_tanh_join_kernel(H, dtype):
     assert torch.allclose(y.cpu().double(), O.dynamic_tanh(want, al, w, b), atol=1e-5 if dtype == torch.float32 else 0.03, rtol=1e-2 if dtype == torch.bfloat16 else 0)
 
 
-@pytest.mark.parametrize("E,top,count,keep", [(8, 4, 4, 3), (12, 3, 4, 1), (6, 2, 3, 2), (7, 2, 7, 3), (5, 5, 1, 1), (64, 6, 8, 3), (256, 8, 8, 4), (40, 6, 8, 3), (500, 16, 50, 7)])
+@pytest.mark.parametrize("E,top,count,keep", [(10, 4, 5, 3), (12, 3, 4, 1), (6, 2, 3, 2), (7, 2, 7, 3), (5, 5, 1, 1), (64, 6, 8, 3), (256, 8, 8, 4), (40, 6, 8, 3), (500, 16, 50, 7)])
 def test_router_kernel(E, top, count, keep):
     from types import SimpleNamespace
     from onecat_vllm.ops import cuda as K
@@ -312,7 +312,7 @@ def test_router_kernel(E, top, count, keep):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("T,E,top,H,I", [(1, 8, 4, 320, 64), (37, 5, 2, 100, 20), (300, 12, 3, 128, 96), (70, 4, 4, 77, 33), (513, 16, 4, 512, 256)])
+@pytest.mark.parametrize("T,E,top,H,I", [(1, 10, 4, 336, 48), (37, 5, 2, 100, 20), (300, 12, 3, 128, 96), (70, 4, 4, 77, 33), (513, 16, 4, 512, 256)])
 def test_experts_of_any_size(T, E, top, H, I, dtype):
     from onecat_vllm.config import ModelConfig
     from onecat_vllm.layers.moe import FusedMoE

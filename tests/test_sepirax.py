@@ -62,7 +62,7 @@ def test_dynamic_tanh_and_scaled_join():
     assert torch.allclose(n(part)[0].double(), norm(part.double()), atol=1e-6)
 
 
-@pytest.mark.parametrize("dims,base,factor,original,fast,slow", [(32, 10000.0, 4.0, 2048, 32.0, 1.0), (8, 50.0, 2.0, 64, 8.0, 0.5), (6, 1000.0, 1.0, 100, 3.0, 2.0),
+@pytest.mark.parametrize("dims,base,factor,original,fast,slow", [(32, 20000.0, 5.0, 1024, 16.0, 1.0), (8, 50.0, 2.0, 64, 8.0, 0.5), (6, 1000.0, 1.0, 100, 3.0, 2.0),
                                                                  (64, 500000.0, 16.0, 8192, 32.0, 1.0), (4, 10.0, 3.0, 1000000, 4.0, 1.0), (16, 1e6, 2.5, 4, 3.0, 2.0)])
 def test_yarn_table(dims, base, factor, original, fast, slow):
     sc = dict(factor=factor, original=original, fast=fast, slow=slow)
@@ -107,7 +107,7 @@ def test_latents_go_into_their_pages(lora, lora_pad, width):
     assert not rows[[i for i in range(32) if i not in used]].any() and not rows[:, lora_pad + rope:].any()
 
 
-@pytest.mark.parametrize("E,top,count,keep", [(8, 4, 4, 3), (8, 8, 1, 1), (12, 3, 4, 1), (6, 2, 3, 2), (7, 2, 7, 3), (5, 1, 1, 1), (64, 6, 8, 8)])
+@pytest.mark.parametrize("E,top,count,keep", [(10, 4, 5, 3), (8, 8, 1, 1), (12, 3, 4, 1), (6, 2, 3, 2), (7, 2, 7, 3), (5, 1, 1, 1), (64, 6, 8, 8)])
 def test_router(E, top, count, keep):
     z = torch.randn(40, E, generator=torch.Generator().manual_seed(E)) * 2
     w, ids = ref.grouped_topk(z, top, count, keep, None, "softmax", True)
