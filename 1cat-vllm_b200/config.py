@@ -154,6 +154,50 @@ def _sepirax_fields(hf: dict) -> dict:
                 num_experts=max((o.get("num_experts", 0) for o in over), default=0), layer_overrides=tuple(over), **top)
 
 
+def _lodevik_fields(hf: dict) -> dict:
+    """``ModelConfig`` fields of a Lodevik config.json: a list of layers, each with latent attention (sink, one output gate per head) or
+    differential attention inside chunks as its mixer and an optional gated feed-forward; RMS norms and layer scales on the sub-blocks'
+    outputs only, an fp32 residual stream that starts from token and bigram embeddings, tied embeddings."""
+    over = []
+    for i, l in enumerate(hf["layers"]):
+        m, mlp = l["mixer"], l.get("mlp")
+        rot = m.get("rot") or dict(base=10000.0, dims=0)
+        if int(rot["dims"]) % 2:
+            raise ValueError(f"Lodevik layer {i}: {rot['dims']} rotated dimensions are not pairs")
+        if mlp is not None and mlp.get("kind", "dense") != "dense":
+            raise ValueError(f"Lodevik layer {i}: feed-forward {mlp.get('kind')!r} is not known")
+        o: dict[str, Any] = dict(mixer_only_layers=mlp is None, intermediate_size=int(mlp["ff"]) if mlp else 0, num_attention_heads=int(m["heads"]),
+                                 attn_scale=float(m["scale"]), rope_theta=float(rot["base"]))
+        if l["type"] == "latent_attention":
+            if int(rot["dims"]) != int(m["rot_dim"]):
+                raise ValueError(f"Lodevik layer {i}: the rotated part has {m['rot_dim']} dimensions, rot.dims is {rot['dims']}")
+            o.update(use_mla=True, num_key_value_heads=int(m["heads"]), kv_lora_rank=int(m["kv_rank"]), qk_nope_head_dim=int(m["dim"]),
+                     qk_rope_head_dim=int(m["rot_dim"]), v_head_dim=int(m["vdim"]), attn_sinks=True, attn_head_gate=True, attn_diff=None,
+                     attn_chunk=0, qk_norm=False, attn_softcap=0.0)
+        elif l["type"] == "attention":
+            if int(rot["dims"]) > int(m["dim"]):
+                raise ValueError(f"Lodevik layer {i}: {rot['dims']} rotated dimensions of {m['dim']}")
+            if m["heads"] % m["kv_heads"]:
+                raise ValueError(f"Lodevik layer {i}: {m['kv_heads']} key/value heads do not divide {m['heads']} heads")
+            mask = m.get("mask")
+            o.update(use_mla=False, num_key_value_heads=int(m["kv_heads"]), head_dim=int(m["dim"]), v_head_dim=int(m["vdim"]),
+                     rotary_dims=int(rot["dims"]), attn_diff=float(m["diff"]), attn_chunk=int(mask["size"]) if mask else 0, qk_norm=True,
+                     attn_softcap=float(m.get("softcap") or 0.0), attn_sinks=False, attn_head_gate=False)
+        else:
+            raise ValueError(f"Lodevik layer {i}: mixer {l['type']!r} is not known")
+        over.append(o)
+    emb = hf["embedding"]
+    big = emb.get("bigram")
+    first = next((o for o in over if o["use_mla"]), over[0])
+    top = {k: first[k] for k in ("use_mla", "num_attention_heads", "num_key_value_heads", "head_dim", "v_head_dim", "kv_lora_rank", "qk_nope_head_dim",
+                                 "qk_rope_head_dim") if k in first}
+    return dict(architecture="Lodevik", vocab_size=int(hf["vocab"]), hidden_size=int(hf["width"]), num_hidden_layers=len(over),
+                rms_norm_eps=float(hf["norm"]["eps"]), pre_norm=False, sandwich_norm=True, layer_scale=True, residual_fp32=True,
+                embed_scale=float(emb["scale"]), bigram=(int(big["buckets"]), int(big["mul_prev"]), int(big["mul_cur"])) if big else None,
+                hidden_act="gelu_tanh", tie_word_embeddings=True, logit_scale=float(hf["logit_scale"]), mla_fused_in=True,
+                intermediate_size=max(o["intermediate_size"] for o in over), layer_overrides=tuple(over), **top)
+
+
 @dataclass
 class ModelConfig:
     """Architecture description, normalised from an HF ``config.json`` (or a dict for synthetic models).
@@ -183,6 +227,7 @@ class ModelConfig:
     attn_output_gate: bool = False  # gated attention: o * sigmoid(gate)
     # Gemma / GLM / Granite family switches
     hidden_act: str = "silu"  # silu | gelu_tanh (GeGLU)
+    bigram: Optional[tuple] = None  # (buckets, mul_prev, mul_cur): a learned row per hashed (previous token, token) joins the token embedding
     embed_scale: float = 1.0  # token embeddings are multiplied by this (Gemma: sqrt(hidden); Granite: embedding_multiplier)
     sandwich_norm: bool = False  # each sub-block's output is normalised before it joins the residual (Gemma2/3, GLM-4)
     attn_scale: Optional[float] = None  # softmax scale when it is not head_dim ** -0.5
@@ -216,6 +261,11 @@ class ModelConfig:
     qk_norm_full: bool = False  # q / k RMSNorm over the whole projection instead of per head (OLMo-2 / OLMo-3)
     # values of single layers that differ from the model's: per layer a dict of ModelConfig fields (``for_layer`` applies it)
     layer_overrides: tuple = ()
+    attn_chunk: int = 0  # > 0: attention stays inside chunks of this many positions, counted from the start of the sequence
+    # differential attention: two attention maps per head over the same values; the head's output is the first map's minus lambda times the
+    # second's, normalised. The number is the constant part of lambda.
+    attn_diff: Optional[float] = None
+    rotary_dims: Optional[int] = None  # rotated dimensions of a head when they are given as a number instead of a fraction
     attn_window_keep: int = 0  # sliding-window layers: the first tokens of a sequence stay visible to every later position
     attn_kv_shared: bool = False  # the values are the projected keys: no value projection, one cached tensor per layer
     attn_head_gate: bool = False  # each head's output is multiplied by sigmoid(g_proj(x)) of that head before the output projection
@@ -337,7 +387,8 @@ class ModelConfig:
     def release_window(self) -> tuple[int, int]:
         """(window, kept first tokens) outside of which no layer reads a sequence's K/V; (0, 0) when some layer reads all of it."""
         cfgs = [self.for_layer(i) for i in range(self.num_hidden_layers)]
-        w = [c.layer_window(i) for i, c in enumerate(cfgs)]
+        # a chunk never reaches further back than a window of its size
+        w = [0 if c.use_mla else c.attn_chunk or c.layer_window(i) for i, c in enumerate(cfgs)]
         return (max(w), max(c.attn_window_keep for c in cfgs)) if w and all(w) else (0, 0)
 
     def is_moe_layer(self, i: int) -> bool:
@@ -345,6 +396,8 @@ class ModelConfig:
 
     @property
     def rotary_dim(self) -> int:
+        if self.rotary_dims is not None and not self.use_mla:
+            return self.rotary_dims
         d = self.qk_rope_head_dim if self.use_mla else self.head_dim
         return int(d * self.partial_rotary_factor) if not self.use_mla else d
 
@@ -369,6 +422,8 @@ class ModelConfig:
             return cls(**{**_gabisun_fields(hf), **over})
         if hf.get("architecture") == "Sepirax" or "Sepirax" in (hf.get("architectures") or ()):
             return cls(**{**_sepirax_fields(hf), **over})
+        if hf.get("architecture") == "Lodevik" or "Lodevik" in (hf.get("architectures") or ()):
+            return cls(**{**_lodevik_fields(hf), **over})
         mm_ids = {m: int(hf[k]) for m, k in (("image", "image_token_id"), ("video", "video_token_id"), ("audio", "audio_token_id")) if hf.get(k) is not None}
         if mm_ids:
             over.setdefault("mm_token_ids", mm_ids)

@@ -18,6 +18,12 @@
 // both products read it), one output gate per head. The softmax weights enter the value product as two bf16 terms (p and the rest of
 // p after rounding), so that they keep about 16 bits of mantissa. In a decode tile of at most eight rows the second terms ride in the
 // unused rows 8..15 of the same operand and cost no extra product.
+// Chunks (EXT): a query sees the keys of its own chunk of the sequence; tiles before the chunk of a CTA's first row are skipped.
+// Differential attention (DIFF, an extended variant): a head has two maps over the same values. A cached key row holds both maps' keys side
+// by side and a query row belongs to one map. Prefill: warps 0 and 1 own the first map's rows, warps 2 and 3 the same rows of the
+// second map, each multiplying its half of the key columns; the second map's output crosses over in shared memory. Decode: rows (head, map)
+// lie next to one another with zeros in the other map's half (the tile has rows to spare), and the merge of the warps or splits takes
+// the difference. Either way the difference, the head norm and the scale are part of the epilogue.
 // (reference: flash-attention-v100/kernel/fused_mha_forward_paged.cu:364, flash_decode_paged.cu:667,831,1301;
 //  v1/attention/backends/flash_attn_v100.py:2216 for the math)
 #include <cuda_fp8.h>
@@ -83,17 +89,46 @@ __device__ __forceinline__ float head_gate(const AttnParams& p, size_t tok, int 
   return 1.f / (1.f + __expf(-__bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.gate)[tok * p.gate_st + head])));
 }
 
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// tanh for soft caps in fp32: an odd polynomial (the series up to x^11, 3e-8 off at 0.4) near zero, (1 - e^-2x) / (1 + e^-2x) elsewhere
+constexpr float kTanhSmall = 0.4f;
+__device__ __forceinline__ float tanh_small(float x) {
+  const float y = x * x;
+  return x * fmaf(y, fmaf(y, fmaf(y, fmaf(y, fmaf(y, -1382.f / 155925.f, 62.f / 2835.f), -17.f / 315.f), 2.f / 15.f), -1.f / 3.f), 1.f);
+}
+__device__ __forceinline__ float tanh_any(float x) {
+  const float e = ex2(-2.f * kLog2e * fabsf(x));
+  return fabsf(x) < kTanhSmall ? tanh_small(x) : copysignf(__fdividef(1.f - e, 1.f + e), x);
+}
+
+// columns c and c + 1 (c even) of an output row of n elements
+__device__ __forceinline__ void store_pair(__nv_bfloat16* dst, int c, int n, float x, float y) {
+  if ((n & 1) == 0) {
+    if (c < n) *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16(x, y);
+  } else {
+    if (c < n) dst[c] = __float2bfloat16(x);
+    if (c + 1 < n) dst[c + 1] = __float2bfloat16(y);
+  }
+}
+
 // CTAs per SM that the extended variants are compiled for (0: the compiler's choice)
-template <int D, int MODE, int MB, bool EXT>
+template <int D, int MODE, int MB, bool EXT, bool DIFF>
 constexpr int ext_min_ctas() {
   if (!EXT) return 0;
+  if (DIFF) return D == 64 ? 3 : D == 128 ? 2 : 0;
   if (D == 64) return MODE == 0 ? 4 : (MB == 1 ? 5 : 3);
   if (D == 128) return MODE == 0 ? 3 : (MB == 1 ? 4 : 2);
   return 0;
 }
 
-template <int D, int MODE, int MB, bool KV8, int ST = 3, bool EXT = false>
-__global__ void __launch_bounds__(128, ext_min_ctas<D, MODE, MB, EXT>()) attn_kernel(const AttnParams p) {
+template <int D, int MODE, int MB, bool KV8, int ST = 3, bool EXT = false, bool DIFF = false>
+__global__ void __launch_bounds__(128, ext_min_ctas<D, MODE, MB, EXT, DIFF>()) attn_kernel(const AttnParams p) {
+  static_assert(!DIFF || EXT, "differential attention is an extended variant");
+  constexpr bool BY_MAP = DIFF && MODE == 0;    // rows 0..31 are the first map's, 32..63 the same rows of the second map
   pdl_trigger();
   pdl_wait();
   constexpr int STAGES = ST;                    // K/V tiles in the cp.async ring (a fourth stage of byte tiles measured no faster)
@@ -147,12 +182,20 @@ __global__ void __launch_bounds__(128, ext_min_ctas<D, MODE, MB, EXT>()) attn_ke
   const int S = p.seq_lens[r];
   if (qlen <= 0 || S <= 0) return;
   const int ctx0 = S - qlen;
-  const int nrows = (tq1 - tq0) * G;
+  const int Gr = BY_MAP ? G / 2 : G;            // rows per token of a block of rows
+  const int nrows = (tq1 - tq0) * Gr;
+  auto row_tok = [&](int row) { return (BY_MAP ? row & 31 : row) / Gr; };
   const int kv_end = min(S, ctx0 + tq1);
   const int ntiles = (kv_end + kKeysPerTile - 1) / kKeysPerTile;
   // sliding window: the first row of the tile sees the earliest key, ctx0 + tq0 - window + 1
   const int wlo = p.window > 0 ? p.window : 0x3fffffff;
-  const int tile_first = p.window > 0 ? max(0, ctx0 + tq0 - p.window + 1) / kKeysPerTile : 0;
+  // earliest key that a position sees (kept tokens aside)
+  auto first_key = [&](int pos) {
+    int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+    if (EXT && p.chunk > 0) lo = max(lo, pos - pos % p.chunk);
+    return lo;
+  };
+  const int tile_first = first_key(ctx0 + tq0) / kKeysPerTile;
   int tile_lo = tile_first, tile_hi = ntiles;
   // kept first tokens: their tiles that lie wholly before the window are walked first (tile index - tile_shift for those)
   int keep_tiles = 0;
@@ -276,20 +319,22 @@ __global__ void __launch_bounds__(128, ext_min_ctas<D, MODE, MB, EXT>()) attn_ke
   const int g_ = lane >> 2, tg = lane & 3;
 
   // extended variants: what the rows of this thread need in every tile
-  int row_pos[MBW][2];
+  int row_pos[MBW][2], row_lo[MBW][2];
   const float* row_bias[MBW][2];
   float row_far[MBW][2];
-  int pos_lo = 0, pos_hi = 0;
+  int pos_lo = 0, pos_hi = 0, lo_hi = 0;
   const bool paired = EXT && MODE == 1 && MB == 1 && nrows <= 8;   // rows 8..15 carry the second terms of rows 0..7
   if constexpr (EXT) {
-    pos_lo = ctx0 + tq0 + row_base / G;
-    pos_hi = ctx0 + tq0 + (row_base + 16 * MBW - 1) / G;
+    pos_lo = ctx0 + tq0 + row_tok(row_base);
+    pos_hi = ctx0 + tq0 + row_tok(row_base + 16 * MBW - 1);
+    lo_hi = first_key(pos_hi);
 #pragma unroll
     for (int b = 0; b < MBW; ++b)
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
-        const int row = row_base + b * 16 + g_ + h * 8, tok = row / G;
+        const int row = row_base + b * 16 + g_ + h * 8, tok = row_tok(row);
         row_pos[b][h] = ctx0 + tq0 + tok;
+        row_lo[b][h] = first_key(row_pos[b][h]);
         row_bias[b][h] = p.bias != nullptr ? p.bias + (size_t)(hkv * G + row - tok * G) * p.bias_len : nullptr;
         row_far[b][h] = p.bias != nullptr ? __ldg(row_bias[b][h] + p.bias_len - 1) * kLog2e : 0.f;
       }
@@ -310,7 +355,11 @@ __global__ void __launch_bounds__(128, ext_min_ctas<D, MODE, MB, EXT>()) attn_ke
   for (int idx = threadIdx.x; idx < ROWS * CH; idx += 128) {
     int row = idx / CH, ch = idx % CH;
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (row < nrows) {
+    if constexpr (DIFF) {
+      const int rr = BY_MAP ? row & 31 : row, tok = tq0 + rr / Gr, gh = BY_MAP ? (rr % Gr) * 2 + (row >> 5) : rr % Gr;
+      if (rr < nrows && ch / (CH / 2) == (gh & 1))
+        v = *reinterpret_cast<const uint4*>(p.q + (size_t)(qs + tok) * p.q_st + (size_t)(hkv * G + gh) * p.q_sh + (ch % (CH / 2)) * 8);
+    } else if (row < nrows) {
       int tok = tq0 + row / G, gh = row % G;
       v = *reinterpret_cast<const uint4*>(p.q + (size_t)(qs + tok) * p.q_st + (size_t)(hkv * G + gh) * p.q_sh + ch * 8);
     }
@@ -375,19 +424,20 @@ __global__ void __launch_bounds__(128, ext_min_ctas<D, MODE, MB, EXT>()) attn_ke
     for (int b = 0; b < MBW; ++b)
 #pragma unroll
       for (int n = 0; n < NB2 * 2; ++n) s[b][n][0] = s[b][n][1] = s[b][n][2] = s[b][n][3] = 0.f;
+    const int ch0 = BY_MAP ? (warp >> 1) * (CH / 2) : 0;   // this warp's half of the key columns
 #pragma unroll
-    for (int kk = 0; kk < D / 16; ++kk) {
+    for (int kk = 0; kk < (BY_MAP ? D / 32 : D / 16); ++kk) {
       uint32_t a[MBW][4];
 #pragma unroll
       for (int b = 0; b < MBW; ++b) {
         int row = row_base + b * 16 + (lane & 15);
-        ldsm_x4(a[b], qb + sw_off<D>(row, kk * 2 + (lane >> 4)));
+        ldsm_x4(a[b], qb + sw_off<D>(row, ch0 + kk * 2 + (lane >> 4)));
       }
 #pragma unroll
       for (int n2 = 0; n2 < NB2; ++n2) {
         uint32_t bfr[4];
         int krow = key_base + n2 * 16 + (lane & 7) + ((lane >> 4) << 3);
-        ldsm_x4(bfr, kb + sw_off<D>(krow, kk * 2 + ((lane >> 3) & 1)));
+        ldsm_x4(bfr, kb + sw_off<D>(krow, ch0 + kk * 2 + ((lane >> 3) & 1)));
 #pragma unroll
         for (int b = 0; b < MBW; ++b) {
           mma_bf16(s[b][n2 * 2], a[b], bfr[0], bfr[1]);
@@ -401,7 +451,7 @@ __global__ void __launch_bounds__(128, ext_min_ctas<D, MODE, MB, EXT>()) attn_ke
     bool no_mask = false, far_bias = false;
     if constexpr (EXT) {
       const int k_hi = k0 + NB2 * 16 - 1;
-      no_mask = k_hi <= pos_lo && k_hi < kv_end && (k0 + wlo > pos_hi || k_hi < p.keep);
+      no_mask = k_hi <= pos_lo && k_hi < kv_end && (k0 >= lo_hi || k_hi < p.keep);
       far_bias = p.bias == nullptr || pos_lo - k_hi >= p.bias_len - 1;   // one value per row (0 without a bias)
     }
 #pragma unroll
@@ -426,13 +476,19 @@ __global__ void __launch_bounds__(128, ext_min_ctas<D, MODE, MB, EXT>()) attn_ke
           if (far_bias && !capped) {
             each([&](float v, int) { return fmaf(v, sc, far); });
           } else {
-            if (capped) each([&](float v, int) { return tanhf(v * sc) * sc_post; });
-            else each([&](float v, int) { return v * sc; });
+            if (capped) {
+              float top = 0.f;
+              each([&](float v, int) { top = fmaxf(top, fabsf(v)); return v; });
+              if (__any_sync(0xffffffffu, top * fabsf(sc) >= kTanhSmall)) each([&](float v, int) { return tanh_any(v * sc) * sc_post; });
+              else each([&](float v, int) { return tanh_small(v * sc) * sc_post; });
+            } else {
+              each([&](float v, int) { return v * sc; });
+            }
             if (far_bias) each([&](float v, int) { return v + far; });
             else each([&](float v, int key) { return fmaf(__ldg(row_bias[b][h] + min(max(qpos - key, 0), p.bias_len - 1)), kLog2e, v); });
           }
           if (!no_mask)
-            each([&](float v, int key) { return (key <= qpos && key < kv_end && (key + wlo > qpos || key < p.keep)) ? v : -INFINITY; });
+            each([&](float v, int key) { return (key <= qpos && key < kv_end && (key >= row_lo[b][h] || key < p.keep)) ? v : -INFINITY; });
         }
         float mx = -INFINITY;
 #pragma unroll
@@ -534,6 +590,44 @@ __global__ void __launch_bounds__(128, ext_min_ctas<D, MODE, MB, EXT>()) attn_ke
   }
   cp_async_wait<0>();
 
+  if constexpr (BY_MAP) {
+    // the second map's output crosses over to the warps of the first one: same rows, same registers
+    float inv[2];
+#pragma unroll
+    for (int h = 0; h < 2; ++h) inv[h] = lrow[0][h] > 0.f ? 1.f / lrow[0][h] : 0.f;
+    __syncthreads();   // everyone is done reading K/V tiles
+    float2* xch = reinterpret_cast<float2*>(sK) + (warp & 1) * (D / 8) * 2 * 32 + lane;
+    if (warp >= 2) {
+#pragma unroll
+      for (int i = 0; i < D / 8; ++i)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) xch[(i * 2 + h) * 32] = make_float2(o[0][i][h * 2] * inv[h], o[0][i][h * 2 + 1] * inv[h]);
+    }
+    __syncthreads();
+    if (warp >= 2) return;
+    const float lam = *p.lam;
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      float ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < D / 8; ++i) {
+        const float2 b = xch[(i * 2 + h) * 32];
+        const float x = o[0][i][h * 2] * inv[h] - lam * b.x, y = o[0][i][h * 2 + 1] * inv[h] - lam * b.y;
+        o[0][i][h * 2] = x;
+        o[0][i][h * 2 + 1] = y;
+        ss = fmaf(x, x, fmaf(y, y, ss));
+      }
+      ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+      ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+      const int row = row_base + g_ + h * 8;
+      if (row >= nrows) continue;
+      const float f = p.out_scale / sqrtf(ss / (float)p.vdim + p.eps);
+      __nv_bfloat16* dst = p.out + ((size_t)(qs + tq0 + row / Gr) * (p.Hq / 2) + hkv * Gr + row % Gr) * p.vdim;
+#pragma unroll
+      for (int i = 0; i < D / 8; ++i) store_pair(dst, i * 8 + tg * 2, p.vdim, o[0][i][h * 2] * f, o[0][i][h * 2 + 1] * f);
+    }
+    return;
+  }
   if (MODE == 0) {
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
@@ -581,6 +675,47 @@ __global__ void __launch_bounds__(128, ext_min_ctas<D, MODE, MB, EXT>()) attn_ke
       }
     }
   __syncthreads();
+  if constexpr (DIFF) {
+    if (p.splits == 1) {   // one warp per (token, head): rows 2 * pair and 2 * pair + 1 are its maps
+      const float lam = *p.lam;
+      for (int pair = warp; pair * 2 < nrows; pair += 4) {
+        float f[2][4];
+#pragma unroll
+        for (int m = 0; m < 2; ++m) {
+          float M = -INFINITY, L = 0.f;
+#pragma unroll
+          for (int w = 0; w < 4; ++w) M = fmaxf(M, mm[((size_t)w * ROWS + pair * 2 + m) * 2]);
+#pragma unroll
+          for (int w = 0; w < 4; ++w) {
+            const float* ml = mm + ((size_t)w * ROWS + pair * 2 + m) * 2;
+            f[m][w] = ml[0] == -INFINITY ? 0.f : exp2f(ml[0] - M);
+            L += ml[1] * f[m][w];
+          }
+          const float inv = L > 0.f ? (m == 0 ? 1.f : -lam) / L : 0.f;
+#pragma unroll
+          for (int w = 0; w < 4; ++w) f[m][w] *= inv;
+        }
+        float x[D / 32], ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < D / 32; ++i) {
+          x[i] = 0.f;
+#pragma unroll
+          for (int w = 0; w < 4; ++w) {
+            const float* src = mo + ((size_t)w * ROWS + pair * 2) * D + lane + 32 * i;
+            x[i] = fmaf(src[0], f[0][w], fmaf(src[D], f[1][w], x[i]));
+          }
+          ss = fmaf(x[i], x[i], ss);
+        }
+        const float g = p.out_scale / sqrtf(warp_sum(ss) / (float)p.vdim + p.eps);
+        const int tok = pair / (G / 2), gh = pair % (G / 2);
+        __nv_bfloat16* dst = p.out + ((size_t)(qs + tok) * (p.Hq / 2) + hkv * (G / 2) + gh) * p.vdim;
+#pragma unroll
+        for (int i = 0; i < D / 32; ++i)
+          if (lane + 32 * i < p.vdim) dst[lane + 32 * i] = __float2bfloat16(x[i] * g);
+      }
+      return;
+    }
+  }
   for (int idx = threadIdx.x; idx < nrows * (D / 4); idx += 128) {
     const int row = idx / (D / 4), c4 = (idx % (D / 4)) * 4;
     float M = -INFINITY;
@@ -645,7 +780,43 @@ __global__ void attn_combine_kernel(const AttnParams p) {
   if (p.lse != nullptr && lane == 0) p.lse[warp] = (M + log2f(L)) * 0.6931471805599453f;
 }
 
-template <int D, int MODE, int MB, bool KV8, int ST = 3, bool EXT = false>
+// the same for the two maps of a head: one warp per (token, head)
+template <int D>
+__global__ void diff_combine_kernel(const AttnParams p) {
+  pdl_trigger();
+  pdl_wait();
+  const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
+  const size_t rows = (size_t)p.T * p.Hq;
+  if ((size_t)warp * 2 >= rows) return;
+  const float lam = *p.lam;
+  float x[D / 32];
+#pragma unroll
+  for (int i = 0; i < D / 32; ++i) x[i] = 0.f;
+#pragma unroll
+  for (int m = 0; m < 2; ++m) {
+    const size_t row = (size_t)warp * 2 + m;
+    const float mine = lane < p.splits ? p.ws_ml[((size_t)lane * rows + row) * 2] : -INFINITY;   // at most 32 splits
+    const float M = warp_max(mine), f_mine = mine == -INFINITY ? 0.f : exp2f(mine - M);
+    const float L = warp_sum(lane < p.splits ? p.ws_ml[((size_t)lane * rows + row) * 2 + 1] * f_mine : 0.f);
+    const float inv = L > 0.f ? (m == 0 ? 1.f : -lam) / L : 0.f;
+    for (int s = 0; s < p.splits; ++s) {
+      const float f = __shfl_sync(0xffffffffu, f_mine, s) * inv;
+      if (f == 0.f) continue;
+      const float* src = p.ws_o + (s * rows + row) * D;
+#pragma unroll
+      for (int i = 0; i < D / 32; ++i) x[i] = fmaf(src[lane + 32 * i], f, x[i]);
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < D / 32; ++i) ss = fmaf(x[i], x[i], ss);
+  const float g = p.out_scale / sqrtf(warp_sum(ss) / (float)p.vdim + p.eps);
+#pragma unroll
+  for (int i = 0; i < D / 32; ++i)
+    if (lane + 32 * i < p.vdim) p.out[(size_t)warp * p.vdim + lane + 32 * i] = __float2bfloat16(x[i] * g);
+}
+
+template <int D, int MODE, int MB, bool KV8, int ST = 3, bool EXT = false, bool DIFF = false>
 int launch_one(const AttnParams& p, cudaStream_t st) {
   constexpr int ROWS = (MODE == 0) ? 64 : 16 * MB;
   const int smem_max = ROWS * D * 2 + (KV8 ? 2 * ST * kKeysPerTile * D + 2 * kKeysPerTile * D * 2 : 2 * ST * kKeysPerTile * D * 2);
@@ -657,15 +828,16 @@ int launch_one(const AttnParams& p, cudaStream_t st) {
   static int configured_dev[kMaxDevices] = {};
   int& configured = configured_dev[current_device_slot()];  // the limit is an attribute of (kernel, device)
   if (!configured) {
-    if (cudaFuncSetAttribute(attn_kernel<D, MODE, MB, KV8, ST, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_max) != cudaSuccess) return -4;
+    if (cudaFuncSetAttribute(attn_kernel<D, MODE, MB, KV8, ST, EXT, DIFF>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_max) != cudaSuccess) return -4;
     configured = 1;
   }
   dim3 grid(MODE == 0 ? p.num_q_tiles : p.R, p.Hkv, MODE == 0 ? 1 : p.splits);
   if (grid.x == 0) return 0;
-  launch_k(attn_kernel<D, MODE, MB, KV8, ST, EXT>, grid, dim3(128), (size_t)smem, st, true, p);
+  launch_k(attn_kernel<D, MODE, MB, KV8, ST, EXT, DIFF>, grid, dim3(128), (size_t)smem, st, true, p);
   if (MODE == 1 && p.splits > 1) {
     int rows = p.T * p.Hq;
-    launch_k(attn_combine_kernel<D>, dim3((rows * 32 + 255) / 256), dim3(256), 0, st, true, p);
+    if constexpr (DIFF) launch_k(diff_combine_kernel<D>, dim3((rows / 2 * 32 + 255) / 256), dim3(256), 0, st, true, p);
+    else launch_k(attn_combine_kernel<D>, dim3((rows * 32 + 255) / 256), dim3(256), 0, st, true, p);
   }
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
 }
@@ -677,7 +849,26 @@ int attention_launch(const AttnParams& p, int mode, cudaStream_t st) {
   const int G = p.Hq / p.Hkv;
   if (G > 64) return -1;
   const bool f8 = p.kv_fp8 != 0;
-  if (p.keep > 0 || p.kv_shared || p.bias != nullptr || p.gate != nullptr) {
+  if (p.maps == 2) {
+    if (f8 || p.keep > 0 || p.kv_shared || p.bias != nullptr || p.gate != nullptr || p.sinks != nullptr || p.lse != nullptr || p.lam == nullptr || G % 2 ||
+        p.vdim < 1 || p.vdim > p.D || p.splits > 32) return -8;
+    if (mode == 1) {
+      const int rows = p.short_q_len * G;
+      if (p.D == 64) {
+        if (rows <= 16) return launch_one<64, 1, 1, false, 3, true, true>(p, st);
+        if (rows <= 32) return launch_one<64, 1, 2, false, 3, true, true>(p, st);
+      } else if (p.D == 128) {
+        if (rows <= 16) return launch_one<128, 1, 1, false, 3, true, true>(p, st);
+        if (rows <= 32) return launch_one<128, 1, 2, false, 3, true, true>(p, st);
+      } else if (rows <= 16) {
+        return launch_one<256, 1, 1, false, 3, true, true>(p, st);
+      }
+      return -6;
+    }
+    return p.D == 64 ? launch_one<64, 0, 1, false, 3, true, true>(p, st) : p.D == 128 ? launch_one<128, 0, 1, false, 3, true, true>(p, st)
+                                                                                      : launch_one<256, 0, 1, false, 3, true, true>(p, st);
+  }
+  if (p.chunk > 0 || p.keep > 0 || p.kv_shared || p.bias != nullptr || p.gate != nullptr) {
     if (f8 || (p.bias != nullptr && p.bias_len < 1)) return -7;
     const int rows = p.short_q_len * G;
     if (mode == 1) {

@@ -35,7 +35,7 @@ void gemm(torch::Tensor x, c10::optional<torch::Tensor> w, c10::optional<torch::
   } else {
     check_bf16(out, "out");
   }
-  TORCH_CHECK(epi != oc::EPI_GELU_TANH || w.has_value(), "the GELU epilogue is for bf16 weights");
+  TORCH_CHECK((epi != oc::EPI_GELU_TANH && epi != oc::EPI_GELU_MUL) || w.has_value(), "the GELU epilogues are for bf16 weights");
   TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && out.dim() == 2 && out.stride(1) == 1, "x/out must be row-major 2-D");
   const c10::cuda::CUDAGuard guard(x.device());
   oc::GemmParams p{};
@@ -53,7 +53,7 @@ void gemm(torch::Tensor x, c10::optional<torch::Tensor> w, c10::optional<torch::
   p.out = f32_out ? nullptr : (__nv_bfloat16*)out.data_ptr();
   p.out_f32 = f32_out ? out.data_ptr<float>() : nullptr;
   p.ldo = (int)out.stride(0);
-  TORCH_CHECK(out.size(0) >= p.T && out.size(1) >= (epi == oc::EPI_SILU_MUL ? n_out : N), "out is too small");
+  TORCH_CHECK(out.size(0) >= p.T && out.size(1) >= (epi == oc::EPI_SILU_MUL || epi == oc::EPI_GELU_MUL ? n_out : N), "out is too small");
   p.bias = bias.has_value() ? (const __nv_bfloat16*)bias->data_ptr() : nullptr;
   p.ws = (float*)ws.data_ptr();
   p.ws_bytes = (size_t)ws.numel() * ws.element_size();
@@ -215,7 +215,7 @@ void paged_attention(torch::Tensor q, torch::Tensor kv_cache, torch::Tensor out,
                      torch::Tensor seq_lens, torch::Tensor block_table, double scale, int64_t mode, int64_t num_q_tiles, int64_t splits,
                      int64_t max_q_len, int64_t short_q_len, c10::optional<torch::Tensor> ws_o, c10::optional<torch::Tensor> ws_ml,
                      int64_t window, double softcap, c10::optional<torch::Tensor> sinks, double k_scale, double v_scale, int64_t keep,
-                     c10::optional<torch::Tensor> bias, c10::optional<torch::Tensor> gate) {
+                     c10::optional<torch::Tensor> bias, c10::optional<torch::Tensor> gate, int64_t chunk) {
   // mode 3: everything fp32 (attention_f32.cu)
   if (mode == 3) {
     TORCH_CHECK(q.is_cuda() && q.scalar_type() == torch::kFloat32 && kv_cache.scalar_type() == torch::kFloat32 && out.scalar_type() == torch::kFloat32,
@@ -283,7 +283,8 @@ void paged_attention(torch::Tensor q, torch::Tensor kv_cache, torch::Tensor out,
     p.gate = gate->data_ptr();
     p.gate_st = gate->stride(0);
   }
-  const bool extended = keep > 0 || p.kv_shared || p.bias != nullptr || p.gate != nullptr;
+  p.chunk = (int)chunk;
+  const bool extended = chunk > 0 || keep > 0 || p.kv_shared || p.bias != nullptr || p.gate != nullptr;
   TORCH_CHECK(mode != 2 || (window == 0 && softcap == 0.0 && !sinks.has_value() && !extended), "window / softcap / sinks and the like run on the mma.sync kernels");
   TORCH_CHECK(!(extended && p.kv_fp8), "an fp8 KV cache has no distance bias, kept tokens, output gate or shared keys and values");
   if (mode == 1 && splits > 1) {
@@ -295,8 +296,96 @@ void paged_attention(torch::Tensor q, torch::Tensor kv_cache, torch::Tensor out,
   }
   if (p.T == 0 || p.R == 0) return;
   // mode 0: mma.sync prefill, 1: decode / short verify queries, 2: tcgen05 prefill (D = 128, query tiles of 128 tokens), 3: fp32
-  int rc = mode == 3 ? oc::attention_f32_launch(p, cur_stream()) : mode == 2 ? oc::attention_prefill_tc_launch(p, kv_cache.size(0), cur_stream()) : oc::attention_launch(p, (int)mode, cur_stream());
+  int rc = mode == 3 ? oc::attention_f32_launch(p, false, cur_stream()) : mode == 2 ? oc::attention_prefill_tc_launch(p, kv_cache.size(0), cur_stream()) : oc::attention_launch(p, (int)mode, cur_stream());
   TORCH_CHECK(rc == 0, "attention launch failed with code ", rc);
+}
+
+// Differential attention: q [T, 2 H, D / 2] (head, map), cache rows of both maps' keys and of the values, out [T, H, vdim]. Modes as in
+// paged_attention without 2; mode 3 takes fp32, or bf16 rows of any width.
+void diff_attention(torch::Tensor q, torch::Tensor kv_cache, torch::Tensor out, torch::Tensor qsl, torch::Tensor seq_lens, torch::Tensor block_table,
+                    double scale, int64_t mode, int64_t num_q_tiles, int64_t splits, int64_t max_q_len, int64_t short_q_len,
+                    c10::optional<torch::Tensor> ws_o, c10::optional<torch::Tensor> ws_ml, double softcap, int64_t chunk, torch::Tensor lam,
+                    double out_scale, double eps) {
+  const auto et = q.scalar_type();
+  TORCH_CHECK(q.is_cuda() && (et == torch::kBFloat16 || (et == torch::kFloat32 && mode == 3)) && kv_cache.scalar_type() == et && out.scalar_type() == et,
+              "q, kv_cache and out must be bf16 (or fp32 in mode 3)");
+  TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && out.dim() == 3 && out.is_contiguous() && kv_cache.dim() == 5 && kv_cache.is_contiguous() && kv_cache.size(1) == 2,
+              "q, out and kv_cache must be contiguous");
+  TORCH_CHECK(q.size(2) * 2 == kv_cache.size(4) && q.size(0) == out.size(0) && q.size(1) == 2 * out.size(1) && out.size(2) <= kv_cache.size(4) &&
+              out.size(1) % kv_cache.size(2) == 0, "q / out / cache shapes do not match");
+  TORCH_CHECK(mode == 3 || (((uintptr_t)q.data_ptr() & 15) == 0 && q.size(2) % 8 == 0), "q must be 16-byte aligned");
+  TORCH_CHECK(qsl.scalar_type() == torch::kInt32 && seq_lens.scalar_type() == torch::kInt32 && block_table.scalar_type() == torch::kInt32, "metadata must be int32");
+  TORCH_CHECK(lam.is_cuda() && lam.scalar_type() == torch::kFloat32 && lam.numel() == 1, "lam must be one fp32 number on the device");
+  const c10::cuda::CUDAGuard guard(q.device());
+  oc::AttnParams p{};
+  p.q = (const __nv_bfloat16*)q.data_ptr(); p.q_st = q.stride(0); p.q_sh = q.stride(1);
+  p.kv_cache = (const __nv_bfloat16*)kv_cache.data_ptr();
+  p.out = (__nv_bfloat16*)out.data_ptr();
+  p.query_start_loc = qsl.data_ptr<int>(); p.seq_lens = seq_lens.data_ptr<int>(); p.block_table = block_table.data_ptr<int>();
+  p.bt_stride = (int)block_table.stride(0);
+  p.R = (int)seq_lens.size(0); p.T = (int)q.size(0); p.Hq = (int)q.size(1); p.Hkv = (int)kv_cache.size(2); p.D = (int)kv_cache.size(4); p.bs = (int)kv_cache.size(3);
+  while ((1 << p.bs_shift) < p.bs) ++p.bs_shift;
+  p.scale = (float)scale; p.num_q_tiles = (int)num_q_tiles; p.splits = (int)splits; p.max_q_len = (int)max_q_len; p.short_q_len = (int)short_q_len;
+  p.softcap = (float)softcap; p.k_scale = p.v_scale = 1.f; p.chunk = (int)chunk;
+  p.maps = 2; p.lam = lam.data_ptr<float>(); p.out_scale = (float)out_scale; p.eps = (float)eps; p.vdim = (int)out.size(2);
+  if (mode == 1 && splits > 1) {
+    TORCH_CHECK(ws_o.has_value() && ws_ml.has_value() && (size_t)ws_o->numel() >= (size_t)splits * p.T * p.Hq * p.D &&
+                (size_t)ws_ml->numel() >= (size_t)splits * p.T * p.Hq * 2, "split-KV workspace too small");
+    p.ws_o = ws_o->data_ptr<float>(); p.ws_ml = ws_ml->data_ptr<float>();
+  }
+  if (p.T == 0 || p.R == 0) return;
+  TORCH_CHECK(mode == 0 || mode == 1 || mode == 3, "mode must be 0, 1 or 3");
+  const int rc = mode == 3 ? oc::attention_f32_launch(p, et == torch::kBFloat16, cur_stream()) : oc::attention_launch(p, (int)mode, cur_stream());
+  TORCH_CHECK(rc == 0, "differential attention launch failed with code ", rc);
+}
+
+// Norm, rotation and cache insert ahead of diff_attention; returns the queries [T, 2 H, D / 2].
+torch::Tensor diff_prepare(torch::Tensor qkv, torch::Tensor q_w, torch::Tensor k_w, double eps, torch::Tensor positions, torch::Tensor cos_sin,
+                           torch::Tensor cache, torch::Tensor slots, int64_t H, int64_t G, int64_t dim, int64_t vdim, bool interleaved) {
+  const auto et = qkv.scalar_type();
+  TORCH_CHECK(qkv.is_cuda() && (et == torch::kBFloat16 || et == torch::kFloat32) && qkv.dim() == 2 && qkv.stride(1) == 1 && cache.scalar_type() == et &&
+              cache.is_contiguous() && cache.dim() == 5 && cache.size(1) == 2 && cache.size(2) == G, "qkv and cache must be bf16 or fp32 [blocks, 2, G, bs, D]");
+  TORCH_CHECK(qkv.size(1) == 2 * (H + G) * dim + G * vdim, "qkv must hold the queries, keys and values of all heads");
+  TORCH_CHECK(q_w.scalar_type() == et && k_w.scalar_type() == et && q_w.is_contiguous() && k_w.is_contiguous() && q_w.numel() == dim && k_w.numel() == dim, "norm weights");
+  TORCH_CHECK(positions.scalar_type() == torch::kInt32 && slots.scalar_type() == torch::kInt32 && positions.numel() >= qkv.size(0) && slots.numel() >= qkv.size(0),
+              "positions and slots must be int32 [T]");
+  TORCH_CHECK(cos_sin.scalar_type() == torch::kFloat32 && cos_sin.is_contiguous() && cos_sin.dim() == 2, "cos_sin must be fp32 [positions, rot]");
+  const c10::cuda::CUDAGuard guard(qkv.device());
+  oc::DiffPrepareParams p{};
+  p.x = qkv.data_ptr(); p.ld = qkv.stride(0); p.q_w = q_w.data_ptr(); p.k_w = k_w.data_ptr(); p.eps = (float)eps;
+  p.positions = positions.data_ptr<int>(); p.slots = slots.data_ptr<int>(); p.cos_sin = cos_sin.data_ptr<float>(); p.cache = cache.data_ptr();
+  p.T = (int)qkv.size(0); p.H = (int)H; p.G = (int)G; p.dim = (int)dim; p.vdim = (int)vdim; p.D = (int)cache.size(4); p.bs = (int)cache.size(3);
+  p.rot = (int)cos_sin.size(1); p.interleaved = interleaved ? 1 : 0; p.f32 = et == torch::kFloat32;
+  auto out = torch::empty({p.T, 2 * H, (int64_t)p.D / 2}, qkv.options());
+  p.q_out = out.data_ptr();
+  const int rc = oc::diff_prepare_launch(p, cur_stream());
+  TORCH_CHECK(rc == 0, "diff_prepare failed: ", rc, " (maps of up to 512 dimensions, an even number of them rotated)");
+  return out;
+}
+
+// x fp32 [T, H] (and y of the table's type, when given) from token and bigram embeddings; see EmbedParams.
+void embed_stream(torch::Tensor ids, torch::Tensor table, double scale, c10::optional<torch::Tensor> prev, c10::optional<torch::Tensor> bigram,
+                  int64_t mul_prev, int64_t mul_cur, torch::Tensor x, c10::optional<torch::Tensor> y, bool gathered) {
+  const auto et = table.scalar_type();
+  TORCH_CHECK(table.is_cuda() && (et == torch::kBFloat16 || et == torch::kFloat32) && table.dim() == 2 && table.is_contiguous(), "the table must be a contiguous bf16 or fp32 matrix");
+  TORCH_CHECK(ids.is_cuda() && ids.scalar_type() == torch::kInt32 && ids.is_contiguous(), "ids must be int32 [T]");
+  const int64_t T = ids.numel(), H = table.size(1);
+  TORCH_CHECK(x.scalar_type() == torch::kFloat32 && x.is_contiguous() && x.numel() == T * H && (!gathered || table.size(0) == T), "x must be fp32 [T, H]");
+  oc::EmbedParams p{};
+  p.table = table.data_ptr(); p.ids = ids.data_ptr<int>(); p.x = x.data_ptr<float>(); p.scale = (float)scale;
+  p.T = (int)T; p.H = (int)H; p.vocab = (int)table.size(0); p.gathered = gathered ? 1 : 0; p.f32 = et == torch::kFloat32;
+  if (y.has_value()) {
+    TORCH_CHECK(y->scalar_type() == et && y->is_contiguous() && y->numel() == T * H, "y must be [T, H] of the table's type");
+    p.y = y->data_ptr();
+  }
+  if (bigram.has_value()) {
+    TORCH_CHECK(bigram->scalar_type() == et && bigram->is_contiguous() && bigram->dim() == 2 && bigram->size(1) == H && bigram->size(0) >= 2, "the bigram table must be [buckets + 1, H]");
+    TORCH_CHECK(prev.has_value() && prev->scalar_type() == torch::kInt32 && prev->is_contiguous() && prev->numel() >= T, "prev must be int32 [T]");
+    p.bigram = bigram->data_ptr(); p.prev = prev->data_ptr<int>(); p.buckets = (int)bigram->size(0) - 1;
+    p.mul_prev = (int)mul_prev; p.mul_cur = (int)mul_cur;
+  }
+  const c10::cuda::CUDAGuard guard(table.device());
+  TORCH_CHECK(oc::embed_stream_launch(p, cur_stream()) == 0, "embed_stream failed");
 }
 
 // Key (and value) rows [T, H, D] into pages [blocks, 1 or 2, H, block_size, D] of the same element type.
@@ -766,9 +855,18 @@ torch::Tensor fused_moe_a2a(torch::Tensor x, torch::Tensor w13, torch::Tensor w2
   return y;
 }
 
+// sink logits [H] fp32 and per-head output gate [T, H] of the element type
+static void check_sink_gate(const c10::optional<torch::Tensor>& sinks, const c10::optional<torch::Tensor>& gate, c10::ScalarType et, int64_t T, int64_t H) {
+  TORCH_CHECK(!sinks.has_value() || (sinks->is_cuda() && sinks->scalar_type() == torch::kFloat32 && sinks->is_contiguous() && sinks->numel() == H),
+              "sinks must be a contiguous fp32 CUDA tensor with one entry per head");
+  TORCH_CHECK(!gate.has_value() || (gate->is_cuda() && gate->scalar_type() == et && gate->dim() == 2 && gate->size(0) == T && gate->size(1) == H && gate->stride(1) == 1),
+              "the gate must be [T, H] of the queries' type with unit inner stride");
+}
+
 torch::Tensor mla_decode(torch::Tensor q_abs, torch::Tensor q_rope, torch::Tensor cache, torch::Tensor qsl, torch::Tensor seq_lens,
                          torch::Tensor block_table, double scale, int64_t max_q_len, int64_t splits, c10::optional<torch::Tensor> ws_o,
-                         c10::optional<torch::Tensor> ws_ml, c10::optional<torch::Tensor> cos_sin, bool interleaved, bool fine, int64_t skip_min_len) {
+                         c10::optional<torch::Tensor> ws_ml, c10::optional<torch::Tensor> cos_sin, bool interleaved, bool fine, int64_t skip_min_len,
+                         c10::optional<torch::Tensor> sinks, c10::optional<torch::Tensor> gate) {
   const auto et = q_abs.scalar_type();
   TORCH_CHECK(q_abs.is_cuda() && (et == torch::kBFloat16 || et == torch::kFloat32) && q_rope.scalar_type() == et && cache.scalar_type() == et, "bf16 or fp32 throughout");
   TORCH_CHECK(q_abs.is_contiguous() && cache.is_contiguous() && cache.dim() == 3 && q_rope.dim() == 3 && q_rope.stride(2) == 1, "q and cache layouts");
@@ -794,6 +892,9 @@ torch::Tensor mla_decode(torch::Tensor q_abs, torch::Tensor q_rope, torch::Tenso
   p.bs = (int)cache.size(1); p.bs_shift = 0;
   while ((1 << p.bs_shift) < p.bs) ++p.bs_shift;
   p.max_q_len = (int)max_q_len; p.splits = (int)splits; p.scale = (float)scale;
+  check_sink_gate(sinks, gate, et, p.T, p.H);
+  if (sinks.has_value()) p.sinks = sinks->data_ptr<float>();
+  if (gate.has_value()) { p.gate = gate->data_ptr(); p.gate_st = gate->stride(0); }
   if (splits > 1) {
     TORCH_CHECK(ws_o.has_value() && ws_ml.has_value() && (size_t)ws_o->numel() >= (size_t)splits * p.T * p.H * p.kv_lora &&
                 (size_t)ws_ml->numel() >= (size_t)splits * p.T * p.H * 2, "split-KV workspace too small");
@@ -837,7 +938,8 @@ std::vector<torch::Tensor> mla_prefill_inputs(torch::Tensor q, torch::Tensor cac
 
 // Second half: causal attention of the listed requests' new tokens; rows of other requests in `out` [T, H, vd] stay as they are.
 void mla_prefill(torch::Tensor q, torch::Tensor kv, torch::Tensor rot, torch::Tensor out, torch::Tensor qsl, torch::Tensor seq_lens, torch::Tensor meta,
-                 int64_t num_long, int64_t num_q_tiles, int64_t nope, int64_t rope, double scale, bool fine) {
+                 int64_t num_long, int64_t num_q_tiles, int64_t nope, int64_t rope, double scale, bool fine, c10::optional<torch::Tensor> sinks,
+                 c10::optional<torch::Tensor> gate) {
   for (auto* t : {&q, &kv, &rot, &out}) {
     check_bf16(*t, "prefill operands");
     TORCH_CHECK(t->is_contiguous(), "prefill operands must be contiguous");
@@ -853,6 +955,9 @@ void mla_prefill(torch::Tensor q, torch::Tensor kv, torch::Tensor rot, torch::Te
   p.q_out = (__nv_bfloat16*)q.data_ptr(); p.kv = (const __nv_bfloat16*)kv.data_ptr(); p.rot = (__nv_bfloat16*)rot.data_ptr(); p.out = (__nv_bfloat16*)out.data_ptr();
   p.query_start_loc = qsl.data_ptr<int>(); p.seq_lens = seq_lens.data_ptr<int>();
   p.long_req = meta.data_ptr<int>(); p.long_ctx = p.long_req + num_long;
+  check_sink_gate(sinks, gate, torch::kBFloat16, p.T, p.H);
+  if (sinks.has_value()) p.sinks = sinks->data_ptr<float>();
+  if (gate.has_value()) { p.gate = (const __nv_bfloat16*)gate->data_ptr(); p.gate_st = gate->stride(0); }
   const int rc = oc::mla_prefill_launch(p, cur_stream());
   TORCH_CHECK(rc == 0, "latent prefill launch failed: ", rc);
 }
@@ -1060,8 +1165,11 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("paged_attention", &paged_attention, py::arg("q"), py::arg("kv_cache"), py::arg("out"), py::arg("lse"), py::arg("qsl"), py::arg("seq_lens"),
         py::arg("block_table"), py::arg("scale"), py::arg("mode"), py::arg("num_q_tiles"), py::arg("splits"), py::arg("max_q_len"), py::arg("short_q_len"),
         py::arg("ws_o"), py::arg("ws_ml"), py::arg("window"), py::arg("softcap"), py::arg("sinks"), py::arg("k_scale"), py::arg("v_scale"),
-        py::arg("keep") = 0, py::arg("bias") = py::none(), py::arg("gate") = py::none());
+        py::arg("keep") = 0, py::arg("bias") = py::none(), py::arg("gate") = py::none(), py::arg("chunk") = 0);
   m.def("kv_insert", &kv_insert);
+  m.def("diff_attention", &diff_attention);
+  m.def("diff_prepare", &diff_prepare);
+  m.def("embed_stream", &embed_stream);
   m.def("stream_join", &stream_join);
   m.def("gelu_tanh_f32", &gelu_tanh_f32);
   m.def("argmax", &argmax);

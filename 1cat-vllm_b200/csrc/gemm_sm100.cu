@@ -10,7 +10,7 @@
 //   * warp 0: producer (TMA tensor copies of X and of bf16 W)
 //     warp 1: TMEM allocation + single-thread tcgen05.mma issue
 //     warps 2-9 (4-bit only): 4-bit -> bf16 dequantisation straight into TMEM (tcgen05.st); the MMA reads operand A from there
-//     next four warps: epilogue (tcgen05.ld -> bf16 store | SiLU*mul | fp32 split-K partial + last-arriver reduction)
+//     next four warps: epilogue (tcgen05.ld -> bf16 store | act(gate)*up | fp32 split-K partial + last-arriver reduction)
 //     last warp (4-bit only): bulk copies of packed 4-bit tiles, running up to `pstages` tiles ahead of the operand stages
 //   * one ring of stages carries both operands of a k tile, with one full and one empty barrier per stage: measured on
 //     B200 the MMA-issuing thread is the critical path (a ready mbarrier wait, four tcgen05.mma and a tcgen05.commit cost it
@@ -31,6 +31,9 @@
 namespace oc {
 
 namespace {
+
+// tanh form of GELU: 0.5 z (1 + tanh(u)) = z / (1 + e^-2u), u = sqrt(2/pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float gelu_tanh(float z) { return z / (1.f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z))); }
 
 #ifdef ONECAT_GEMM_TRACE
 #define TRACE(slot) do { if (p.trace) p.trace[blockIdx.x * 16 + (slot)] = globaltimer_ns(); } while (0)
@@ -246,7 +249,7 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ 
   const int row = q * 32 + lane;       // weight row inside the tile
   const int et = threadIdx.x - R::kEpiThread0;    // 0..127 in the warps that run the epilogue
   uint32_t chunk_i = 0;
-  const bool silu = p.epi == EPI_SILU_MUL;
+  const bool gated = p.epi == EPI_SILU_MUL || p.epi == EPI_GELU_MUL;
   const uint32_t stg_u32 = smem_u32(smem + L.stage_off);
   // which of the rotating arrival buffers a tensor-parallel push goes to: a device word that the previous reduction kernel advances,
   // so it is read only after this thread has passed pdl_wait()
@@ -264,11 +267,12 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ 
   // tok_gstride 4); a[] are this thread's feature row, one value per staged token
   auto emit = [&](float (&a)[32], int rows, int tok0, int tok_gstride, int n_base, int t0, int t_end, float bias_v) {
     const uint32_t buf = stg_u32 + (chunk_i & 1u) * (32 * kStagePitch);
-    if (silu) {
+    if (gated) {
 #pragma unroll
       for (int j = 0; j < 32; ++j) {  // lanes 0-15 hold gate rows, lanes 16-31 the matching up rows
         const float other = __shfl_xor_sync(0xffffffffu, a[j], 16);
-        a[j] = a[j] / (1.f + __expf(-a[j])) * other;
+        if (WKIND == 0 && p.epi == EPI_GELU_MUL) a[j] = gelu_tanh(a[j]) * other;
+        else a[j] = a[j] / (1.f + __expf(-a[j])) * other;
       }
     } else if (bias_v != 0.f) {
 #pragma unroll
@@ -277,10 +281,7 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ 
     if constexpr (WKIND == 0) {
       if (p.epi == EPI_GELU_TANH) {
 #pragma unroll
-        for (int j = 0; j < 32; ++j) {  // 0.5 z (1 + tanh(u)) = z / (1 + e^-2u), u = sqrt(2/pi) (z + 0.044715 z^3)
-          const float z = a[j], u2 = 1.5957691216057308f * (z + 0.044715f * z * z * z);
-          a[j] = z / (1.f + __expf(-u2));
-        }
+        for (int j = 0; j < 32; ++j) a[j] = gelu_tanh(a[j]);
       }
       if (p.out_f32 != nullptr) {
         // a warp holds 32 neighbouring features of a token: its fp32 stores are whole 128-byte segments as they are
@@ -296,19 +297,19 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ 
       }
     }
     // feature pair (f, f + 1) of staged token j goes to the even lane, of token j + 1 to the odd lane
-    const uint32_t col_b = silu ? (uint32_t)(q * 16 + (lane & 14)) * 2u : (uint32_t)(q * 32 + (lane & 30)) * 2u;
+    const uint32_t col_b = gated ? (uint32_t)(q * 16 + (lane & 14)) * 2u : (uint32_t)(q * 32 + (lane & 30)) * 2u;
 #pragma unroll
     for (int j = 0; j < 32; j += 2) {
       const float send = (lane & 1) ? a[j] : a[j + 1];
       const float recv = __shfl_xor_sync(0xffffffffu, send, 1);
       const float lo = (lane & 1) ? recv : a[j], hi = (lane & 1) ? a[j + 1] : recv;
       __nv_bfloat162 pk = __floats2bfloat162_rn(lo, hi);
-      if (!silu || lane < 16)
+      if (!gated || lane < 16)
         asm volatile("st.shared.b32 [%0], %1;" ::"r"(buf + (uint32_t)(j + (lane & 1)) * kStagePitch + col_b), "r"(*reinterpret_cast<uint32_t*>(&pk)) : "memory");
     }
     asm volatile("bar.sync 1, 128;" ::: "memory");
-    const int vpr = silu ? 8 : 16;                       // 16-byte vectors per staged token row
-    const int nb = silu ? n_base / 2 : n_base, nlim = silu ? p.n_out : p.N;
+    const int vpr = gated ? 8 : 16;                       // 16-byte vectors per staged token row
+    const int nb = gated ? n_base / 2 : n_base, nlim = gated ? p.n_out : p.N;
     for (int v = et; v < rows * vpr; v += 128) {
       const int r = v / vpr, cv = v - r * vpr;
       const int t = t0 + tok0 + (r >> 2) * tok_gstride + (r & 3), n0 = nb + cv * 8;
@@ -349,7 +350,7 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ 
       n_base = it.w;
     }
     const int n = n_base + row;
-    const float bias_v = (!silu && p.bias != nullptr && n < p.N) ? __bfloat162float(p.bias[n]) : 0.f;
+    const float bias_v = (!gated && p.bias != nullptr && n < p.N) ? __bfloat162float(p.bias[n]) : 0.f;
     if (p.splits > 1 && p.cluster > 1) {
       // Split-K inside a thread-block cluster: the CTAs that share a tile are the cluster (rank = split index, one work item per
       // CTA). Each leaves its fp32 partial in its own shared memory ([token / 4][row][4], over the operand ring, which is idle once

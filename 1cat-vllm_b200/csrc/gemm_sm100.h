@@ -6,12 +6,12 @@
 
 namespace oc {
 
-enum { EPI_STORE = 0, EPI_SILU_MUL = 1, EPI_GELU_TANH = 2 };
+enum { EPI_STORE = 0, EPI_SILU_MUL = 1, EPI_GELU_TANH = 2, EPI_GELU_MUL = 3 };
 
 struct GemmParams {
   int T, N, K;        // tokens, logical output features, reduction length (multiple of 64)
   int n_rows;         // weight rows the kernel walks (N, or 2*n_out for the interleaved gate|up layout)
-  int n_out;          // output columns for EPI_SILU_MUL
+  int n_out;          // output columns for EPI_SILU_MUL / EPI_GELU_MUL
   int n_pad;          // padded weight rows (stride of the scale/zero table)
   int tn, num_t_tiles, num_n_tiles, splits, ktiles_per_split;
   int acc_stride;               // TMEM columns between the two accumulators

@@ -63,6 +63,16 @@ struct StreamJoinParams {
   int f32;                      // the model's element type (part, weights, y, copy_out): 1 fp32, 0 bf16
 };
 int stream_join_launch(const StreamJoinParams& p, cudaStream_t st);
+// Start of the stream: x = table[id] * scale (+ bigram[hash of (previous token, token)]), y = x in the model's element type.
+struct EmbedParams {
+  const void *table, *bigram;   // [vocab][H], [buckets + 1][H] or null
+  const int *ids, *prev;        // [T]; prev < 0: no previous token (the last row)
+  float* x;                     // [T][H]
+  void* y;                      // [T][H] or null
+  float scale;
+  int T, H, vocab, buckets, mul_prev, mul_cur, gathered, f32;   // gathered: the table's rows are the tokens' own
+};
+int embed_stream_launch(const EmbedParams& p, cudaStream_t st);
 int gelu_tanh_f32_launch(float* x, long long n, cudaStream_t st);  // in place
 
 int argmax_launch(const void* x, int is_fp32, long long* out, unsigned long long* packed, int B, int V, long long ld, cudaStream_t st);
@@ -101,15 +111,37 @@ struct AttnParams {
   int bias_len;
   const void* gate;           // [T][Hq] (row pitch gate_st, element type of q): outputs are multiplied by its sigmoid, or null
   long long gate_st;
+  int chunk;                  // > 0: only keys of the query's own chunk of that many positions are visible
+  // Differential attention (maps == 2): Hq counts (head, map) rows, q is [T][Hq][D / 2], a key row holds both maps side by side, out is
+  // [T][Hq / 2][vdim]: the first map's output minus *lam times the second's, divided by its root mean square over vdim, times out_scale.
+  int maps;
+  const float* lam;
+  float out_scale, eps;
+  int vdim;
 };
-// fp32 queries, cache and outputs (attention_f32.cu): q / kv_cache / out / gate point at floats, num_q_tiles counts tiles of 16
+// fp32 queries, cache and outputs (attention_f32.cu; bf16: differential attention only, with fp32 arithmetic): q / kv_cache / out / gate
+// point at floats, num_q_tiles counts tiles of 16
 // (token, query head of the group) rows over all requests; splits, short_q_len and the workspaces are not used.
-int attention_f32_launch(const AttnParams& p, cudaStream_t st);
+int attention_f32_launch(const AttnParams& p, bool bf16, cudaStream_t st);
 // mode 0: rows of a query tile are spread over warps (prefill / long queries); mode 1: keys are spread over warps
 // (decode and short verify queries, with split-KV + combine).
 int attention_launch(const AttnParams& p, int mode, cudaStream_t st);
 unsigned int attention_read_status(bool clear);
 void attention_read_status_async(unsigned int* dst, cudaStream_t st);
+// Differential attention ahead of its kernels: per (token, head, map) RMS norm and rotation of queries and keys, cache insert.
+struct DiffPrepareParams {
+  const void* x;              // [T][ld]: q [2 H dim] | k [2 G dim] | v [G vdim]
+  long long ld;
+  const void *q_w, *k_w;      // norm weights [dim]
+  float eps;
+  const int *positions, *slots;   // slots negative: nothing is inserted
+  const float* cos_sin;       // [positions][rot]
+  void* q_out;                // [T][2 H][D / 2], zeros past dim
+  void* cache;                // [blocks][2][G][bs][D]: key rows (map 1 | map 2), value rows, zeros in the padding
+  int T, H, G, dim, vdim, D, rot, bs, interleaved, f32;
+};
+int diff_prepare_launch(const DiffPrepareParams& p, cudaStream_t st);
+
 // tcgen05 prefill (attention_tc.cu): D == 128, 128-token query tiles; num_q_tiles counts those tiles.
 int attention_prefill_tc_launch(const AttnParams& p, long long num_blocks, cudaStream_t st);
 unsigned int attention_tc_read_status(bool clear);
@@ -194,6 +226,9 @@ struct MlaParams {
   float scale;
   float* ws_o;                  // [splits][T][H][kv_lora]
   float* ws_ml;                 // [splits][T][H][2]
+  const float* sinks;           // [H] logits that join the softmax denominator only, or null
+  const void* gate;             // [T][H] (row pitch gate_st): outputs are multiplied by its sigmoid, or null
+  long long gate_st;
 };
 int mla_decode_launch(const MlaParams& p, cudaStream_t st);
 bool mla_tensor_core_sizes(int kv_lora, int rope_pad);
@@ -211,6 +246,9 @@ struct MlaPrefillParams {
   const float* cos_sin;
   int bt_stride, bs, T, H, rows, num_long, num_q_tiles, lora_pad, rope_pad, nope, rope, vd, NC, RC, interleaved, fine;
   float scale;
+  const float* sinks;           // as in MlaParams
+  const __nv_bfloat16* gate;
+  long long gate_st;
 };
 bool mla_prefill_sizes(int nope, int rope, int vd);
 int mla_prefill_inputs_launch(const MlaPrefillParams& p, cudaStream_t st);   // gather + query rows

@@ -49,6 +49,12 @@ template <typename E> __device__ __forceinline__ void stf(E* p, float v);
 template <> __device__ __forceinline__ void stf<float>(float* p, float v) { *p = v; }
 template <> __device__ __forceinline__ void stf<__nv_bfloat16>(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
 
+// factor of the output gate of (token, head); 1 without a gate
+template <typename E>
+__device__ __forceinline__ float gate_of(const MlaParams& p, size_t tok, int head) {
+  return p.gate != nullptr ? 1.f / (1.f + expf(-ldf<E>(reinterpret_cast<const E*>(p.gate) + tok * p.gate_st + head))) : 1.f;
+}
+
 // Element j of a rotated row: pair and half from the layout, (cos | sin) row of the position in the table.
 template <typename E>
 __device__ __forceinline__ float rotated(const E* x, int j, int n, const float* cs, int interleaved) {
@@ -244,7 +250,8 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p) {
         wm[1] = l2[h];
       }
     } else {
-      const float inv = l2[h] > 0.f ? 1.f / l2[h] : 0.f;
+      const float den = l2[h] + (p.sinks != nullptr ? ex2(p.sinks[hd] * 1.4426950408889634f - m2[h]) : 0.f);
+      const float inv = den > 0.f ? gate_of<__nv_bfloat16>(p, qs + tok, hd) / den : 0.f;
       __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out) + orow * DV + warp * (DV / 4);
 #pragma unroll
       for (int i = 0; i < NB; ++i) *reinterpret_cast<uint32_t*>(dst + i * 8 + tg * 2) = pk(o[i][h * 2] * inv, o[i][h * 2 + 1] * inv);
@@ -261,7 +268,8 @@ __global__ void mla_combine_kernel(const MlaParams p) {
   const float M = warp_max(mine);
   const float f_mine = mine == -INFINITY ? 0.f : ex2(mine - M);
   const float L = warp_sum(lane < p.splits ? p.ws_ml[((size_t)lane * rows + warp) * 2 + 1] * f_mine : 0.f);
-  const float inv = L > 0.f ? 1.f / L : 0.f;
+  const float den = L + (p.sinks != nullptr ? ex2(p.sinks[warp % p.H] * 1.4426950408889634f - M) : 0.f);
+  const float inv = L > 0.f ? gate_of<__nv_bfloat16>(p, warp / p.H, warp % p.H) / den : 0.f;
   for (int c = lane * 2; c < DV; c += 64) {
     float x = 0.f, y = 0.f;
     for (int s = 0; s < p.splits; ++s) {
@@ -351,7 +359,14 @@ __global__ void __launch_bounds__(128) mla_plain_kernel(const MlaParams p) {
       }
     }
   }
-  if (lane == 0) { sl[warp * 2] = l[0]; sl[warp * 2 + 1] = l[1]; }
+  if (lane == 0) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {   // the factor of the row's output
+      const int gr = row0 + warp * 2 + i, hd = gr % p.H;
+      const float den = l[i] + (p.sinks != nullptr ? expf(p.sinks[hd] - m[i]) : 0.f);
+      sl[warp * 2 + i] = den > 0.f && warp * 2 + i < nrows ? gate_of<E>(p, qs + gr / p.H, hd) / den : 0.f;
+    }
+  }
   __syncthreads();
 #pragma unroll
   for (int c = 0; c < NC; ++c) {
@@ -361,7 +376,7 @@ __global__ void __launch_bounds__(128) mla_plain_kernel(const MlaParams p) {
     for (int i = 0; i < PR; ++i)
       if (i < nrows) {
         const int gr = row0 + i;
-        stf<E>(reinterpret_cast<E*>(p.out) + ((size_t)(qs + gr / p.H) * p.H + gr % p.H) * p.kv_lora + col, sl[i] > 0.f ? o[i][c] / sl[i] : 0.f);
+        stf<E>(reinterpret_cast<E*>(p.out) + ((size_t)(qs + gr / p.H) * p.H + gr % p.H) * p.kv_lora + col, o[i][c] * sl[i]);
       }
   }
 }

@@ -305,7 +305,9 @@ mla_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       l += xch[(half ^ 1) * TQ + row];
     }
     if (ok && !*abort_flag && tq < qlen) {
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      if (p.sinks != nullptr) l += ex2(p.sinks[h] * 1.4426950408889634f - m);
+      float inv = l > 0.f ? 1.f / l : 0.f;
+      if (p.gate != nullptr) inv *= 1.f / (1.f + __expf(-__bfloat162float(p.gate[(size_t)(qs + tq) * p.gate_st + h])));
       __nv_bfloat16* dst = p.out + ((size_t)(qs + tq) * p.H + h) * p.vd + half * HC;
       const int n = min(HC, p.vd - half * HC);
       if (p.vd % 8 == 0) {

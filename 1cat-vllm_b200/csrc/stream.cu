@@ -1,6 +1,7 @@
 // Kernels around the fp32 residual stream and the un-rotated paged cache.
 //   stream_join: x' = x + mul * scale * post(part) (+ add), y = next(x'): a sub-block's output is normalised, scaled, added to the stream and the
 //                sum normalised for the next sub-block in one pass; optionally x' also leaves in the model's element type.
+//   embed_stream: the stream's start from scaled token embeddings and hashed-bigram rows.
 //   kv_insert:   key (and value) rows into their pages.
 #include <type_traits>
 
@@ -168,6 +169,30 @@ int stream_join_n(const StreamJoinParams& p, cudaStream_t st) {
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
+template <typename E, int N>
+__global__ void __launch_bounds__(256) embed_stream_kernel(const EmbedParams p) {
+  pdl_trigger();
+  pdl_wait();
+  const size_t t = blockIdx.x;
+  const int id = p.ids[t];
+  const E* row = reinterpret_cast<const E*>(p.table) + (p.gathered ? t : (size_t)min(max(id, 0), p.vocab - 1)) * p.H;
+  const E* big = nullptr;
+  if (p.bigram != nullptr) {
+    const int prev = p.prev[t];
+    const long long h = prev < 0 ? p.buckets : ((long long)prev * p.mul_prev + (long long)id * p.mul_cur) % p.buckets;
+    big = reinterpret_cast<const E*>(p.bigram) + (h < 0 ? h + p.buckets : h) * p.H;
+  }
+  for (int c = threadIdx.x * N; c < p.H; c += blockDim.x * N) {
+    float v[N], b[N];
+    load_vec<E, N>(row + c, v);
+    if (big != nullptr) load_vec<E, N>(big + c, b);
+#pragma unroll
+    for (int j = 0; j < N; ++j) v[j] = big != nullptr ? fmaf(v[j], p.scale, b[j]) : v[j] * p.scale;
+    store_vec<float, N>(p.x + t * p.H + c, v);
+    if (p.y != nullptr) store_vec<E, N>(reinterpret_cast<E*>(p.y) + t * p.H + c, v);
+  }
+}
+
 template <typename W>
 __global__ void __launch_bounds__(256) kv_insert_kernel(const KvInsertParams p) {
   pdl_trigger();
@@ -202,6 +227,20 @@ int stream_join_launch(const StreamJoinParams& p, cudaStream_t st) {
   if (p.f32) return vec ? stream_join_n<float, float, 4>(p, st) : stream_join_n<float, float, 1>(p, st);
   if (p.part_f32) return vec ? stream_join_n<__nv_bfloat16, float, 4>(p, st) : stream_join_n<__nv_bfloat16, float, 1>(p, st);
   return vec ? stream_join_n<__nv_bfloat16, __nv_bfloat16, 4>(p, st) : stream_join_n<__nv_bfloat16, __nv_bfloat16, 1>(p, st);
+}
+
+int embed_stream_launch(const EmbedParams& p, cudaStream_t st) {
+  if (p.T == 0) return 0;
+  if (p.H < 1 || p.vocab < 1 || (p.bigram != nullptr && (p.prev == nullptr || p.buckets < 1))) return -1;
+  const uintptr_t a = p.f32 ? 16 : 8;
+  auto ok = [](const void* q, uintptr_t n) { return ((uintptr_t)q & (n - 1)) == 0; };
+  const bool vec = p.H % 4 == 0 && ok(p.table, a) && ok(p.bigram, a) && ok(p.x, 16) && ok(p.y, a);
+  int threads = ((vec ? (p.H + 3) / 4 : p.H) + 31) / 32 * 32;
+  if (threads > 256) threads = 256;
+  auto go = [&](auto kernel) { launch_k(kernel, dim3((unsigned)p.T), dim3((unsigned)threads), 0, st, true, p); };
+  if (p.f32) vec ? go(embed_stream_kernel<float, 4>) : go(embed_stream_kernel<float, 1>);
+  else vec ? go(embed_stream_kernel<__nv_bfloat16, 4>) : go(embed_stream_kernel<__nv_bfloat16, 1>);
+  return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
 int kv_insert_launch(const KvInsertParams& p, cudaStream_t st) {

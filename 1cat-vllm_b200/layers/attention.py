@@ -43,7 +43,7 @@ class Attention(nn.Module):
                                               q_mult=2 if self.gated else 1, bias=cfg.attention_bias, quant=cfg.quant,
                                               prefix=prefix + ".qkv_proj", dtype=cfg.dtype)
             self.Hq, self.Hkv = self.qkv_proj.num_heads, self.qkv_proj.num_kv_heads
-        self.window_keep = cfg.attn_window_keep
+        self.window_keep, self.chunk = cfg.attn_window_keep, cfg.attn_chunk
         self.rel_max, self.bias_table = cfg.attn_rel_max, None
         self.rel_bias = nn.Parameter(torch.zeros(cfg.attn_rel_buckets, self.Hq, dtype=torch.float32), requires_grad=False) \
             if cfg.attn_rel_buckets else None
@@ -116,7 +116,7 @@ class Attention(nn.Module):
         k = qkg[:, Hq * D: (Hq + Hkv) * D].view(T, Hkv, D)
         ops.kv_insert(k, kv_cache, md.slot_mapping)
         o = ops.paged_attention(q, kv_cache, md, self.scale, window=self.window, softcap=self.softcap, sinks=self.sinks, keep=self.window_keep,
-                                bias_table=self.bias_table, gate=qkg[:, (Hq + Hkv) * D:] if self.head_gate else None)
+                                bias_table=self.bias_table, chunk=self.chunk, gate=qkg[:, (Hq + Hkv) * D:] if self.head_gate else None)
         return self.o_proj(o.reshape(T, Hq * D))
 
     def forward(self, x: torch.Tensor, md, kv_cache: torch.Tensor) -> torch.Tensor:
@@ -151,7 +151,57 @@ class Attention(nn.Module):
                                self.q_norm if self.qk_norm else None, self.k_norm if self.qk_norm else None, self.eps, self.gemma,
                                mrope_section=mrope)
         o = ops.paged_attention(q, kv_cache, md, self.scale, window=self.window, softcap=self.softcap, sinks=self.sinks, keep=self.window_keep,
-                                bias_table=self.bias_table)
+                                bias_table=self.bias_table, chunk=self.chunk)
         if gate is not None:
             o = o * torch.sigmoid(gate.float()).to(o.dtype)
         return self.o_proj(o.reshape(T, Hq * D))
+
+
+class DifferentialAttention(nn.Module):
+    """Two attention maps per head over the same values: ``o = rms(a1 - lam a2) * (1 - diff)`` with a1, a2 the maps' outputs and one learned
+    ``lam`` per layer. Queries and keys are laid out head by head as (map 1, map 2), each map normalised and rotated by itself; scores may be
+    soft-capped, and attention may stay inside chunks of the sequence.
+
+    fused QKV GEMM -> per-map norm, rotation and cache insert (one kernel) -> paged attention with both maps of a head in one CTA, which takes
+    the difference and normalises it -> output projection. A cached key row holds both maps side by side."""
+
+    kv_shared, window, window_keep, bias_table = False, 0, 0, None   # what the runner and the graphs ask of an attention layer
+
+    def __init__(self, cfg: ModelConfig, layer_idx: int, prefix: str, device):
+        super().__init__()
+        tp = get_state().tp_size
+        H, G = cfg.num_attention_heads, cfg.num_key_value_heads
+        if H % tp or (G % tp and tp % G):
+            raise ValueError(f"tensor_parallel_size={tp} does not divide the heads of layer {layer_idx}")
+        self.dim, self.vdim = cfg.head_dim, cfg.v_head_dim or cfg.head_dim
+        self.qkv_proj = QKVParallelLinear(cfg.hidden_size, 2 * self.dim, H, G, v_dim=self.vdim, quant=cfg.quant, prefix=prefix + ".qkv_proj",
+                                          dtype=cfg.dtype)
+        self.H, self.Hkv = self.qkv_proj.num_heads, self.qkv_proj.num_kv_heads
+        self.Hq = 2 * self.H   # rows of the attention kernel: (head, map)
+        self.o_proj = RowParallelLinear(H * self.vdim, cfg.hidden_size, quant=cfg.quant, prefix=prefix + ".o_proj", dtype=cfg.dtype)
+        vec = lambda: nn.Parameter(torch.ones(self.dim, dtype=cfg.dtype), requires_grad=False)
+        self.q_norm, self.k_norm = vec(), vec()
+        self.lq1, self.lk1, self.lq2, self.lk2 = (nn.Parameter(torch.zeros(self.dim, dtype=torch.float32), requires_grad=False) for _ in range(4))
+        self.register_buffer("lam", torch.zeros(1, dtype=torch.float32), persistent=False)
+        self.diff, self.eps = cfg.attn_diff, cfg.rms_norm_eps
+        self.rope = get_rope(cfg.rotary_dim, cfg.max_model_len, cfg.rope_theta, device, cfg.rope_scaling)
+        self.scale = cfg.attn_scale if cfg.attn_scale is not None else cfg.head_dim ** -0.5
+        self.softcap, self.chunk = cfg.attn_softcap, cfg.attn_chunk
+        # width of a cached key (both maps) and value row: the next size of the tensor-core kernels
+        need = max(2 * self.dim, self.vdim + self.vdim % 2)
+        tc = torch.device(device).type == "cuda" and cfg.dtype == torch.bfloat16
+        self.D = next((d for d in (64, 128, 256) if d >= need), need) if tc else need
+        self.layer_idx = layer_idx
+
+    def load_weight(self, pname: str, w: torch.Tensor, shard_id=None) -> None:
+        getattr(self, pname).data.copy_(w)
+
+    def process_weights_after_loading(self) -> None:
+        lam = torch.exp((self.lq1.data * self.lk1.data).sum()) - torch.exp((self.lq2.data * self.lk2.data).sum()) + self.diff
+        self.lam.copy_(lam)
+
+    def forward(self, x: torch.Tensor, md, kv_cache: torch.Tensor) -> torch.Tensor:
+        q = ops.diff_prepare(self.qkv_proj(x), self.q_norm, self.k_norm, self.eps, md.positions, self.rope.cos_sin, kv_cache, md.slot_mapping, self.H,
+                             self.Hkv, self.dim, self.vdim)
+        o = ops.diff_attention(q, kv_cache, md, self.scale, self.lam, 1.0 - self.diff, self.eps, self.vdim, self.softcap, self.chunk)
+        return self.o_proj(o.reshape(x.shape[0], self.H * self.vdim))

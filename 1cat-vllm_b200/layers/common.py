@@ -148,6 +148,19 @@ class VocabParallelEmbedding(nn.Module):
         return reduce_only(out)
 
 
+class BigramEmbedding(nn.Module):
+    """A learned row per hashed pair (previous token, token), added to the token embedding where an fp32 residual stream starts. The table has
+    one more row than buckets, for tokens without a previous one; every TP rank holds all of it."""
+
+    def __init__(self, buckets: int, mul_prev: int, mul_cur: int, hidden: int, dtype=torch.float32):
+        super().__init__()
+        self.muls = (mul_prev, mul_cur)
+        self.weight = nn.Parameter(torch.zeros(buckets + 1, hidden, dtype=dtype), requires_grad=False)
+
+    def load_weight(self, pname, w, shard_id=None):
+        self.weight.data.copy_(w)
+
+
 class ParallelLMHead(VocabParallelEmbedding):
     """Vocab-sharded output projection; ``compute_logits`` gathers the shards."""
 

@@ -56,6 +56,8 @@ class LinearMethod:
             y = ref.silu_and_mul(y)
         elif layer.fuse_gelu_tanh:
             y = F.gelu(y, approximate="tanh")
+        elif layer.fuse_gelu_mul:
+            y = ref.gelu_tanh_and_mul(y)
         return y.to(layer.out_dtype) if layer.out_dtype is not None else y
 
 
@@ -271,12 +273,12 @@ class LinearBase(nn.Module):
     def __init__(self, in_features: int, output_sizes: list[int], parallel: str = "replicated", bias: bool = False,
                  quant: Optional[QuantConfig] = None, prefix: str = "", dtype: torch.dtype = torch.float32,
                  fuse_silu_mul: bool = False, segment_tp: Optional[list[int]] = None, fuse_gelu_tanh: bool = False,
-                 out_dtype: Optional[torch.dtype] = None) -> None:
+                 fuse_gelu_mul: bool = False, out_dtype: Optional[torch.dtype] = None) -> None:
         super().__init__()
         st = get_state()
         self.tp, self.tp_rank = st.tp_size, st.tp_rank
         self.parallel, self.prefix, self.compute_dtype = parallel, prefix, dtype
-        self.fuse_silu_mul, self.fuse_gelu_tanh = fuse_silu_mul, fuse_gelu_tanh
+        self.fuse_silu_mul, self.fuse_gelu_tanh, self.fuse_gelu_mul = fuse_silu_mul, fuse_gelu_tanh, fuse_gelu_mul
         self.out_dtype = out_dtype  # None: the input's dtype; fp32 keeps the accumulator's precision (dense weights only)
         self.in_features_global, self.output_sizes = in_features, list(output_sizes)
         # segment_tp[i]: over how many ranks segment i is split (kv heads may be replicated)
@@ -361,11 +363,11 @@ class MergedColumnParallelLinear(LinearBase):
 class QKVParallelLinear(LinearBase):
     """q|k|v stacked along the output; KV heads are replicated when there are fewer of them than TP ranks."""
 
-    def __init__(self, hidden, head_dim, num_heads, num_kv_heads, q_mult: int = 1, **kw):
+    def __init__(self, hidden, head_dim, num_heads, num_kv_heads, q_mult: int = 1, v_dim: Optional[int] = None, **kw):
         tp = get_state().tp_size
         kv_tp = min(tp, num_kv_heads)
         self.num_heads, self.num_kv_heads = num_heads // tp, max(num_kv_heads // tp, 1)
-        super().__init__(hidden, [num_heads * head_dim * q_mult, num_kv_heads * head_dim, num_kv_heads * head_dim], "column",
+        super().__init__(hidden, [num_heads * head_dim * q_mult, num_kv_heads * head_dim, num_kv_heads * (v_dim or head_dim)], "column",
                          segment_tp=[tp, kv_tp, kv_tp], **kw)
 
 

@@ -25,21 +25,25 @@ class MLAAttention(nn.Module):
         q, dt, Hg = cfg.quant, cfg.dtype, cfg.num_attention_heads
         qk = self.nope + self.rope_d
         self.fused_in, self.gated, self.interleaved = cfg.mla_fused_in, cfg.attn_output_gate, not cfg.mla_rope_half
+        self.head_gate = cfg.attn_head_gate   # one gate logit per head, applied inside the attention kernels
         if Hg % tp:
             raise ValueError(f"tensor_parallel_size={tp} does not divide the {Hg} heads of layer {layer_idx}")
         if self.fused_in:
-            # query latent | key/value latent and shared key part | output gate: everything that reads the block's input, in one GEMM
-            sizes = [self.q_lora, self.lora + self.rope_d] + ([Hg * self.vd] if self.gated else [])
+            # query latent (or the queries themselves) | key/value latent and shared key part | output gate, element by element or one
+            # logit per head: everything that reads the block's input, in one GEMM
+            if self.gated and self.head_gate:
+                raise ValueError("latent attention has an elementwise output gate or one per head, not both")
+            sizes = [self.q_lora or Hg * qk, self.lora + self.rope_d] + ([Hg * self.vd] if self.gated else [Hg] if self.head_gate else [])
             self.in_proj_dqkvg = LinearBase(cfg.hidden_size, sizes, "column", quant=q, prefix=prefix + ".in_proj_dqkvg", dtype=dt,
-                                            segment_tp=[1, 1, tp][: len(sizes)])
-        elif self.gated:
+                                            segment_tp=[1 if self.q_lora else tp, 1, tp][: len(sizes)])
+        elif self.gated or self.head_gate:
             raise ValueError("the output gate of latent attention is part of the fused input projection")
         if self.q_lora:
             if not self.fused_in:
                 self.q_a_proj = ReplicatedLinear(cfg.hidden_size, self.q_lora, quant=q, prefix=prefix + ".q_a_proj", dtype=dt)
             self.q_a_layernorm = RMSNorm(self.q_lora, cfg.rms_norm_eps, dtype=dt)
             self.q_b_proj = ColumnParallelLinear(self.q_lora, Hg * qk, quant=q, prefix=prefix + ".q_b_proj", dtype=dt)
-        else:
+        elif not self.fused_in:
             self.q_proj = ColumnParallelLinear(cfg.hidden_size, Hg * qk, quant=q, prefix=prefix + ".q_proj", dtype=dt)
         if not self.fused_in:
             self.kv_a_proj_with_mqa = ReplicatedLinear(cfg.hidden_size, self.lora + self.rope_d, quant=q, prefix=prefix + ".kv_a_proj_with_mqa", dtype=dt)
@@ -63,11 +67,16 @@ class MLAAttention(nn.Module):
             self.lora_pad, self.rope_pad = K.mla_padded_sizes(self.lora, self.rope_d)
             self.prefill_sizes = self.scale > 0 and self.lora_pad % 8 == 0 and self.rope_pad % 8 == 0
         self.cache_width = self.lora_pad + self.rope_pad   # elements of a cached token: latent | shared key part, each padded for the kernel
+        self.sinks = nn.Parameter(torch.zeros(self.H, dtype=torch.float32), requires_grad=False) if cfg.attn_sinks else None
         self._wuk = self._wuv = self._wkv = None
 
     def load_weight(self, pname: str, w: torch.Tensor, shard=None) -> None:
-        """Key and value up-projections stored apart (``uk`` / ``uv``, rows head by head) take their places in ``kv_b_proj``."""
+        """Key and value up-projections stored apart (``uk`` / ``uv``, rows head by head) take their places in ``kv_b_proj``; the sink logits
+        are sharded with the heads."""
         st = get_state()
+        if pname == "sinks":
+            self.sinks.data.copy_(w.narrow(0, st.tp_rank * self.H, self.H))
+            return
         n = {"uk": self.nope, "uv": self.vd}[pname]
         o = 0 if pname == "uk" else self.nope
         w = w.view(-1, n, self.lora)[st.tp_rank * self.H: (st.tp_rank + 1) * self.H]
@@ -89,21 +98,25 @@ class MLAAttention(nn.Module):
         return self._wuk, self._wuv
 
     def forward(self, x, md, latent_cache):
-        T, gate = x.shape[0], None
+        T, gate, q = x.shape[0], None, None
         if self.fused_in:
             y = self.in_proj_dqkvg(x)
-            n = self.q_lora + self.lora + self.rope_d
-            qa, kv = y[:, : self.q_lora], y[:, self.q_lora: n]
-            gate = y[:, n:] if self.gated else None
+            a = self.q_lora or self.H * (self.nope + self.rope_d)
+            n = a + self.lora + self.rope_d
+            qa, kv = y[:, :a], y[:, a: n]
+            gate = y[:, n:] if self.gated or self.head_gate else None
+            if not self.q_lora:
+                q, qa = qa, None
         else:
             qa, kv = self.q_a_proj(x) if self.q_lora else None, self.kv_a_proj_with_mqa(x)
         # one kernel: both latent norms, the rotation of the shared key part and the cache insert (no data-dependent shape: the step can
         # be captured in a CUDA graph; padding tokens have no slot)
         qa = ops.mla_prepare(qa, kv, self.q_a_layernorm if self.q_lora else None, self.kv_a_layernorm, md.positions, self.rope.cos_sin, latent_cache,
                              md.slot_mapping, self.lora, self.lora_pad, self.interleaved)
-        q = (self.q_b_proj(qa) if self.q_lora else self.q_proj(x)).view(T, self.H, self.nope + self.rope_d)
-        o = self._attend(q, md, latent_cache).reshape(T, self.H * self.vd)
-        return self.o_proj(ops.sigmoid_mul(o, gate) if gate is not None else o)
+        if q is None:
+            q = self.q_b_proj(qa) if self.q_lora else self.q_proj(x)
+        o = self._attend(q.view(T, self.H, self.nope + self.rope_d), md, latent_cache, gate if self.head_gate else None).reshape(T, self.H * self.vd)
+        return self.o_proj(ops.sigmoid_mul(o, gate) if self.gated else o)
 
     def _expand(self, lat: torch.Tensor) -> torch.Tensor:
         """Latents ``[rows, lora_pad]`` -> keys and values head by head, both padded to 64 columns."""
@@ -116,7 +129,7 @@ class MLAAttention(nn.Module):
             self._wkv = torch.cat([pad(wuk), pad(wuv)], 1).reshape(-1, self.lora_pad).contiguous()
         return K.gemm_bf16(lat, self._wkv)
 
-    def _attend(self, q, md, latent_cache):
+    def _attend(self, q, md, latent_cache, gate=None):
         """Attention over the cached latents. Single tokens and short portions: the key up-projection is moved to the query and the value one
         to the result. Longer portions on the GPU (bf16): keys and values of the context are expanded and attended to per head."""
         wuk, wuv = self._absorb(q.dtype)
@@ -127,15 +140,15 @@ class MLAAttention(nn.Module):
             if plan is None or plan[-1]:
                 q_abs = K.per_head_matmul(q[..., : self.nope], wuk)
                 o_lat = K.mla_decode(q_abs, q[..., self.nope:], latent_cache, md, self.scale, self.lora_pad, self.rope.cos_sin, self.interleaved,
-                                     self.fine_weights, 0 if plan is None else K.MLA_PREFILL_MIN_LEN)
+                                     self.fine_weights, 0 if plan is None else K.MLA_PREFILL_MIN_LEN, self.sinks, gate)
                 o = K.per_head_matmul(o_lat, wuv.transpose(1, 2))
             if plan is not None:
                 if o is None:
                     o = torch.empty(q.shape[0], self.H, self.vd, dtype=q.dtype, device=q.device)
                 K.mla_prefill(plan, q, latent_cache, md, self._expand, o, self.nope, self.rope_d, self.lora_pad, self.scale, self.rope.cos_sin,
-                              self.interleaved, self.fine_weights)
+                              self.interleaved, self.fine_weights, self.sinks, gate)
             return o
         q_abs = torch.einsum("thn,hnl->thl", q[..., : self.nope], wuk)
         q_pe = ref.rope_rows(q[..., self.nope:], md.positions, self.rope.cos_sin, self.interleaved)
-        o_lat = ref.mla_decode(q_abs, q_pe, latent_cache, md.block_table, md.query_start_loc, md.seq_lens, self.scale, self.lora)
+        o_lat = ref.mla_decode(q_abs, q_pe, latent_cache, md.block_table, md.query_start_loc, md.seq_lens, self.scale, self.lora, self.sinks, gate)
         return torch.einsum("thl,hvl->thv", o_lat, wuv)

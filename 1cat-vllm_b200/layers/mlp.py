@@ -1,4 +1,4 @@
-"""SwiGLU feed-forward: merged gate|up column-parallel GEMM with the SiLU·mul applied in its epilogue,
+"""Gated feed-forward: merged gate|up column-parallel GEMM with act(gate)·up (SiLU or the tanh form of GELU) applied in its epilogue,
 then the row-parallel down projection (reference: models/llama.py ``LlamaMLP``; layers/activation.py ``SiluAndMul``)."""
 from __future__ import annotations
 
@@ -10,13 +10,15 @@ from onecat_vllm.layers.linear import ColumnParallelLinear, MergedColumnParallel
 class MLP(nn.Module):
     def __init__(self, hidden: int, inter: int, quant, prefix: str, dtype, parallel: bool = True, fuse_act: bool = True, act: str = "silu",
                  bias: bool = False):
-        """``fuse_act=False`` (LoRA-enabled models) keeps gate|up as a plain GEMM so adapter deltas can be added before SiLU·mul.
-        ``act="gelu_tanh"`` (Gemma GeGLU) always takes the unfused form: the GEMM epilogue implements SiLU·mul only."""
+        """``fuse_act=False`` (LoRA-enabled models) keeps gate|up as a plain GEMM so adapter deltas can be added before the activation.
+        ``act="gelu_tanh"`` (GeGLU) is fused for dense weights; the packed-weight GEMM's epilogue implements SiLU·mul only."""
         super().__init__()
-        fuse_act = fuse_act and act == "silu" and not bias   # the fused epilogue has no bias input
+        # the fused epilogue has no bias input
+        fuse_act = fuse_act and not bias and (act == "silu" or act == "gelu_tanh" and (quant is None or quant.method == "none"))
         self.fuse_act, self.act = fuse_act, act
         self.gate_up_proj = MergedColumnParallelLinear(hidden, [inter, inter], bias=bias, quant=quant, prefix=prefix + ".gate_up_proj",
-                                                       dtype=dtype, fuse_silu_mul=fuse_act)
+                                                       dtype=dtype, fuse_silu_mul=fuse_act and act == "silu",
+                                                       fuse_gelu_mul=fuse_act and act == "gelu_tanh")
         self.down_proj = RowParallelLinear(inter, hidden, bias=bias, quant=quant, prefix=prefix + ".down_proj", dtype=dtype)
 
     def forward(self, x):

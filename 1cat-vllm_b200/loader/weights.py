@@ -110,6 +110,24 @@ def sepirax_name(name: str, mixer_kind) -> str:
     return base + ours if ours else name
 
 
+# Lodevik checkpoints: ``l<i>.<name>``
+_LODEVIK_NAMES = {"norm1": "post_attention_layernorm.weight", "norm2": "post_feedforward_layernorm.weight", "ls1": "attn_layer_scale",
+                  "ls2": "mlp_layer_scale", "mlp.gate": "mlp.gate_proj.weight", "mlp.up": "mlp.up_proj.weight", "mlp.down": "mlp.down_proj.weight",
+                  **{f"mix.{n}": f"self_attn.{n}_proj.weight" for n in ("q", "k", "v", "o", "dkv", "g")}, "mix.q.norm": "self_attn.q_norm",
+                  "mix.k.norm": "self_attn.k_norm", "mix.dkv.norm": "self_attn.kv_a_layernorm.weight", "mix.sink": "self_attn.sinks",
+                  **{f"mix.{n}": f"self_attn.{n}" for n in ("uk", "uv", "lq1", "lk1", "lq2", "lk2")}}
+_LODEVIK_TOP = {"embed": "model.embed_tokens.weight", "bigram": "model.bigram.weight", "final.norm": "model.norm.weight"}
+
+
+def lodevik_name(name: str) -> str:
+    """Module parameter that a Lodevik checkpoint tensor belongs to (unknown names come back unchanged)."""
+    m = re.match(r"l(\d+)\.(.+)$", name)
+    if m is None:
+        return _LODEVIK_TOP.get(name, name)
+    ours = _LODEVIK_NAMES.get(m.group(2))
+    return f"model.layers.{m.group(1)}.{ours}" if ours else name
+
+
 _EXPERT_RE = re.compile(r"(.*\.mlp)\.experts\.(\d+)\.(gate_proj|up_proj|down_proj)\.(weight|weight_scale_inv|weight_scale|bias)$")
 
 
@@ -126,12 +144,15 @@ def load_weights(model: nn.Module, weights: Iterable[tuple[str, torch.Tensor]]) 
     nemotron_h = cfg is not None and cfg.architecture.startswith("NemotronH")
     gabisun = cfg is not None and cfg.architecture == "Gabisun"
     sepirax = cfg is not None and cfg.architecture == "Sepirax"
+    lodevik = cfg is not None and cfg.architecture == "Lodevik"
     loaded = set()
     for name, w in weights:
         if gabisun:
             name = gabisun_name(name)
         elif sepirax:
             name = sepirax_name(name, lambda i: "mlstm" if cfg.layer_type(i) == "mlstm" else "mla")
+        elif lodevik:
+            name = lodevik_name(name)
         if name.startswith("language_model."):
             name = name[len("language_model."):]
         elif name.startswith("model.language_model."):  # text tower of a multimodal checkpoint (Qwen3.5)

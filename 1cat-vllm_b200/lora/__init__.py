@@ -163,8 +163,8 @@ class LoRAManager:
             layer = self.mods.get(target)
             if layer is None or not hasattr(layer, "local_output_sizes"):
                 continue  # a module this model does not have (or one on another pipeline stage)
-            if getattr(layer, "fuse_silu_mul", False):
-                raise ValueError("this model was built without enable_lora: its gate|up projection applies SiLU·mul in the GEMM epilogue")
+            if getattr(layer, "fuse_silu_mul", False) or getattr(layer, "fuse_gelu_mul", False):
+                raise ValueError("this model was built without enable_lora: its gate|up projection applies the activation in the GEMM epilogue")
             col0 = sum(layer.local_output_sizes[:sub])
             a, b = ab["a"], ab["b"]
             # tensor parallelism: a column-parallel layer keeps this rank's rows of B (its slice of the sub-projection's outputs); a

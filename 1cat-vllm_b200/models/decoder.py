@@ -15,8 +15,8 @@ import torch.nn as nn
 
 from onecat_vllm import ops
 from onecat_vllm.config import ModelConfig
-from onecat_vllm.layers.attention import Attention
-from onecat_vllm.layers.common import ParallelLMHead, RMSNorm, VocabParallelEmbedding, make_norm
+from onecat_vllm.layers.attention import Attention, DifferentialAttention
+from onecat_vllm.layers.common import BigramEmbedding, ParallelLMHead, RMSNorm, VocabParallelEmbedding, make_norm
 from onecat_vllm.layers.gdn import GatedDeltaNet
 from onecat_vllm.layers.linear import ReplicatedLinear
 from onecat_vllm.layers.mla import MLAAttention
@@ -60,14 +60,18 @@ class DecoderLayer(nn.Module):
             self.linear_attn = Mixer(cfg, idx, prefix + ".linear_attn")
             self.kind = "linear_attention"   # a state-slot layer like Gated-DeltaNet for the runner and the scheduler
             self.graph_safe = False          # its convolution and scan read batch geometry on the host
+        elif cfg.attn_diff is not None:
+            self.self_attn = layer_class("DifferentialAttention", DifferentialAttention)(cfg, idx, prefix + ".self_attn", device)
         else:
             self.self_attn = layer_class("Attention", Attention)(cfg, idx, prefix + ".self_attn", device)
         if cfg.layer_scale:
             scale = lambda: nn.Parameter(torch.ones(cfg.hidden_size, dtype=cfg.dtype), requires_grad=False)
             self.attn_layer_scale, self.mlp_layer_scale = scale(), None if cfg.mixer_only_layers else scale()
+        no_pre = cfg.residual_fp32 and not cfg.pre_norm   # the sub-blocks read the stream itself
         if cfg.mixer_only_layers:
             self.mlp = None
-            self.input_layernorm = make_norm(cfg)
+            if not no_pre:
+                self.input_layernorm = make_norm(cfg)
             if cfg.sandwich_norm:
                 self.post_attention_layernorm = make_norm(cfg)
             return
@@ -80,13 +84,15 @@ class DecoderLayer(nn.Module):
         else:
             self.mlp = layer_class("MLP", MLP)(cfg.hidden_size, cfg.intermediate_size, cfg.quant, prefix + ".mlp", cfg.dtype, fuse_act=not cfg.enable_lora,
                            act=cfg.hidden_act, bias=cfg.mlp_bias)
-        self.input_layernorm = make_norm(cfg)
+        if not no_pre:
+            self.input_layernorm = make_norm(cfg)
         if not cfg.parallel_block:
             self.post_attention_layernorm = make_norm(cfg)
         if cfg.sandwich_norm:
             # Gemma2/3 and GLM-4: post_attention_layernorm normalises the mixer's output, pre_feedforward_layernorm is the pre-norm of
             # the feed-forward, post_feedforward_layernorm normalises its output (GLM-4's names are mapped to these at load)
-            self.pre_feedforward_layernorm = make_norm(cfg)
+            if not no_pre:
+                self.pre_feedforward_layernorm = make_norm(cfg)
             self.post_feedforward_layernorm = make_norm(cfg)
 
     def mixer(self, x, md, cache):
@@ -111,9 +117,11 @@ class DecoderModel(nn.Module):
         self.norm = make_norm(cfg) if self.last_stage else PPMissingLayer()
         if cfg.residual_fp32 and (self.start != 0 or not self.last_stage):
             raise ValueError("models with an fp32 residual stream are served without pipeline parallelism")
-        if (cfg.layer_scale or cfg.loop is not None) and not cfg.residual_fp32 or cfg.residual_fp32 and (cfg.parallel_block or not cfg.pre_norm):
-            raise ValueError("the fp32 residual stream is served for blocks with norms ahead of (or on both sides of) the sub-blocks; looped layers "
-                             "and layer scales need it")
+        if (cfg.layer_scale or cfg.loop is not None or cfg.bigram) and not cfg.residual_fp32 or \
+                cfg.residual_fp32 and (cfg.parallel_block or not cfg.pre_norm and (cfg.loop is not None or not cfg.sandwich_norm)):
+            raise ValueError("the fp32 residual stream is served for blocks with norms ahead of, behind or on both sides of the sub-blocks; looped "
+                             "layers, layer scales and bigram embeddings need it")
+        self.bigram = BigramEmbedding(*cfg.bigram, cfg.hidden_size, cfg.dtype) if cfg.bigram else None
         if cfg.loop is not None:
             # ahead of every pass of the looped layers the stream x becomes loop_in([x ; x0]) + loop_step[pass], x0 being the embeddings
             self.loop_in = ReplicatedLinear(2 * cfg.hidden_size, cfg.hidden_size, quant=None, prefix="model.loop_in", dtype=cfg.dtype,
@@ -123,10 +131,18 @@ class DecoderModel(nn.Module):
         self.aux_hidden_layers: tuple = ()
         self.last_aux: list = []
 
-    def embed(self, input_ids: torch.Tensor) -> torch.Tensor:
+    def embed(self, input_ids: torch.Tensor, prev_ids: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Token embeddings as ``forward`` takes them in ``inputs_embeds`` for models whose stream starts from them unrounded."""
+        if self.bigram is not None:
+            return self._embed_stream(input_ids, prev_ids)[0]
         h = self.embed_tokens(input_ids)
         return (h.float() * self.cfg.embed_scale).to(h.dtype) if self.cfg.residual_fp32 and self.cfg.embed_scale != 1.0 else h
+
+    def _embed_stream(self, input_ids, prev_ids):
+        """(fp32 stream, the same in the model's type) of scaled token embeddings plus bigram rows."""
+        e, b = self.embed_tokens, self.bigram
+        table = e.weight if e.tp == 1 else e(input_ids)   # a sharded table: the tokens' rows, already gathered
+        return ops.embed_stream(input_ids, table, self.cfg.embed_scale, prev_ids, b.weight, b.muls, gathered=e.tp > 1)
 
     def local_layers(self):
         """(global index, layer) of the decoder layers this pipeline stage owns."""
@@ -147,6 +163,9 @@ class DecoderModel(nn.Module):
         layers = self.layers
         cfg = self.cfg
         if intermediate is None:
+            if inputs_embeds is None and self.bigram is not None:
+                x, y = self._embed_stream(input_ids, md.prev_ids)
+                return self._forward_stream(y, md, caches, return_prenorm, stream=x)
             if inputs_embeds is None:
                 h = self.embed_tokens(input_ids)
                 if cfg.residual_fp32:   # the stream starts from the scaled embeddings: the factor is applied in fp32
@@ -156,6 +175,8 @@ class DecoderModel(nn.Module):
             else:
                 h = inputs_embeds
             if cfg.residual_fp32:
+                if self.bigram is not None:
+                    return self._forward_stream(h.to(cfg.dtype), md, caches, return_prenorm, stream=h)
                 return self._forward_stream(h, md, caches, return_prenorm)
             x, residual = layers[self.start].input_layernorm(h, None)
             residual = h
@@ -200,9 +221,9 @@ class DecoderModel(nn.Module):
             return x, residual
         return x
 
-    def _forward_stream(self, h, md, caches, return_prenorm: bool = False, embed_scale: float = 1.0):
-        """fp32 residual stream: ``x += mult * scale * post_norm(sub-block(pre_norm(x)))``, post norms and layer scales where the model has
-        them. One fused kernel joins a sub-block's output to the stream and produces the next sub-block's input (``ops.stream_join``).
+    def _forward_stream(self, h, md, caches, return_prenorm: bool = False, embed_scale: float = 1.0, stream=None):
+        """fp32 residual stream: ``x += mult * scale * post_norm(sub-block(pre_norm(x)))``, pre and post norms and layer scales where the model
+        has them; ``stream``: the stream's start in fp32 when it is more than the embeddings ``h``. One fused kernel joins a sub-block's output to the stream and produces the next sub-block's input (``ops.stream_join``).
         Looped layers: the join ahead of a pass also leaves the stream beside the embeddings as the input of the pass's entry projection,
         whose fp32 output becomes the new stream."""
         cfg = self.cfg
@@ -213,9 +234,17 @@ class DecoderModel(nn.Module):
             both = torch.empty(T, 2 * H, dtype=h.dtype, device=h.device)   # [stream ; embeddings]
             both[:, H:] = h
 
+        def plain_join(part, x, post, scale, mul):
+            """Join without a norm behind it: the next sub-block reads the stream itself, rounded to the model's type."""
+            y = torch.empty(T, H, dtype=h.dtype, device=h.device) if h.dtype != torch.float32 else None
+            _, x = ops.stream_join(part, x, post, scale, None, out_dtype=h.dtype, copy_out=y, mul=mul)
+            return (x if y is None else y), x
+
         def join(part, x, post, scale, at, mul):
             """Join, then the input of run ``at`` (past the last run: the final norm)."""
             part = reduce_only(part) if x is not None else part
+            if not cfg.pre_norm and at < len(runs):
+                return plain_join(part, x, post, scale, mul)
             if at < len(runs) and loop is not None and runs[at][0] == loop[0] and runs[at][1] >= 0:
                 ops.stream_join(part, x, post, scale, None, copy_out=both[:, :H], mul=mul)
                 return ops.stream_join(self.loop_in(both), None, None, None, self.layers[loop[0]].input_layernorm, out_dtype=h.dtype,
@@ -223,7 +252,7 @@ class DecoderModel(nn.Module):
             return ops.stream_join(part, x, post, scale, self.layers[runs[at][0]].input_layernorm if at < len(runs) else self.norm,
                                    out_dtype=h.dtype, mul=mul)
 
-        y, x = join(h, None, None, None, 0, embed_scale)
+        y, x = (h, stream) if stream is not None and not cfg.pre_norm else join(h if stream is None else stream, None, None, None, 0, embed_scale)
         for r, (i, _) in enumerate(runs):
             layer = self.layers[i]
             post1 = layer.post_attention_layernorm if cfg.sandwich_norm else None
@@ -232,8 +261,12 @@ class DecoderModel(nn.Module):
             if layer.mlp is None:
                 y, x = join(part, x, post1, scale1, r + 1, mult)
                 continue
-            y, x = ops.stream_join(reduce_only(part), x, post1, scale1,
-                                   layer.pre_feedforward_layernorm if cfg.sandwich_norm else layer.post_attention_layernorm, out_dtype=h.dtype, mul=mult)
+            if not cfg.pre_norm:
+                y, x = plain_join(reduce_only(part), x, post1, scale1, mult)
+            else:
+                y, x = ops.stream_join(reduce_only(part), x, post1, scale1,
+                                       layer.pre_feedforward_layernorm if cfg.sandwich_norm else layer.post_attention_layernorm, out_dtype=h.dtype,
+                                       mul=mult)
             y, x = join(layer.mlp(y), x, layer.post_feedforward_layernorm if cfg.sandwich_norm else None, scale2, r + 1, mult)
         return (y, x) if return_prenorm else y
 
@@ -282,7 +315,7 @@ class CausalLM(nn.Module):
         (".qkv_proj", ".q_proj", 0), (".qkv_proj", ".k_proj", 1), (".qkv_proj", ".v_proj", 2),
         (".qkg_proj", ".q_proj", 0), (".qkg_proj", ".k_proj", 1), (".qkg_proj", ".g_proj", 2),
         (".gate_up_proj", ".gate_proj", 0), (".gate_up_proj", ".up_proj", 1),
-        (".in_proj_dqkvg", ".dq_proj", 0), (".in_proj_dqkvg", ".dkv_proj", 1), (".in_proj_dqkvg", ".g_proj", 2),
+        (".in_proj_dqkvg", ".dq_proj", 0), (".in_proj_dqkvg", ".q_proj", 0), (".in_proj_dqkvg", ".dkv_proj", 1), (".in_proj_dqkvg", ".g_proj", 2),
         (".in_proj_qkvg", ".in_proj_q", 0), (".in_proj_qkvg", ".in_proj_k", 1), (".in_proj_qkvg", ".in_proj_v", 2), (".in_proj_qkvg", ".in_proj_g", 3),
         (".gate_if", ".gate_i", 0), (".gate_if", ".gate_f", 1),
         (".in_proj_qkvz", ".in_proj_q", 0), (".in_proj_qkvz", ".in_proj_k", 1), (".in_proj_qkvz", ".in_proj_v", 2),

@@ -85,6 +85,28 @@ def sigmoid_mul(x, gate):
     return (x.float() * torch.sigmoid(gate.float())).to(x.dtype)
 
 
+def embed_stream(ids, table, scale, prev=None, bigram=None, muls=(0, 0), out_dtype=None, gathered=False):
+    """Scaled token embeddings plus hashed-bigram rows as the start of an fp32 residual stream; returns (stream, stream in ``out_dtype``).
+    See ``ref.embed_stream``."""
+    f = ext().embed_stream if table.is_cuda else ref.embed_stream
+    return f(ids, table, scale, prev, bigram, muls, out_dtype or table.dtype, gathered)
+
+
+def diff_prepare(qkv, q_norm, k_norm, eps, positions, cos_sin, kv_cache, slot_mapping, heads, kv_heads, dim, vdim, interleaved=True):
+    """Norm, rotation and cache insert of differential attention's queries, keys and values in one kernel; returns the queries. See
+    ``ref.diff_prepare``."""
+    f = ext().diff_prepare if qkv.is_cuda else ref.diff_prepare
+    return f(qkv, q_norm, k_norm, eps, positions, cos_sin, kv_cache, slot_mapping, heads, kv_heads, dim, vdim, interleaved)
+
+
+def diff_attention(q, kv_cache, md, scale, lam, out_scale, eps, vdim, softcap=0.0, chunk=0):
+    """Differential attention of the step ``md``: two softmax maps per head over the same values, their difference, the head norm. See
+    ``ref.diff_attention``."""
+    if q.is_cuda:
+        return ext().diff_attention(q, kv_cache, md, scale, lam, out_scale, eps, vdim, softcap, chunk)
+    return ref.diff_attention(q, kv_cache, md.block_table, md.query_start_loc, md.seq_lens, scale, lam, out_scale, eps, vdim, softcap, chunk)
+
+
 def mlstm(qkvg, gates, i_bias, f_bias, norm_w, eps, cap, H, D, V, state, md):
     """mLSTM recurrence with its head norm and output gate: ``qkvg`` ``[T, 2 H D + 2 H V]`` (q | k | v | output gate), ``gates`` fp32
     ``[T, 2 H]`` (input | forget logits before bias and cap), ``state`` = (S, n, m) per slot, updated in place. Returns ``[T, H V]``."""
@@ -92,19 +114,21 @@ def mlstm(qkvg, gates, i_bias, f_bias, norm_w, eps, cap, H, D, V, state, md):
     return f(qkvg, gates, i_bias, f_bias, norm_w, eps, cap, H, D, V, state, md)
 
 
-def paged_attention(q, kv_cache, md, scale, out=None, window=0, softcap=0.0, sinks=None, keep=0, bias_table=None, gate=None):
+def paged_attention(q, kv_cache, md, scale, out=None, window=0, softcap=0.0, sinks=None, keep=0, bias_table=None, gate=None,
+                    chunk=0):
     """``md`` is the step's AttentionMetadata. ``window``: sliding window in tokens (0 = full causal); ``softcap``: tanh soft-capping
     of the scaled scores (0 = off); ``sinks``: fp32 ``[Hq]`` sink logits that join the softmax denominator; ``keep``: first tokens visible
-    outside the window; ``bias_table``: fp32 ``[Hq, n]`` added by distance; ``gate``: ``[T, Hq]`` logits of the per-head output gate."""
+    outside the window; ``bias_table``: fp32 ``[Hq, n]`` added by distance; ``gate``: ``[T, Hq]`` logits of the per-head output gate;
+    ``chunk``: only keys of the query's own chunk of that many positions are visible."""
     if q.is_cuda:
         return ext().paged_attention(q, kv_cache, md, scale, out, window=window, softcap=softcap, sinks=sinks, keep=keep, bias_table=bias_table,
-                                     gate=gate)
+                                     gate=gate, chunk=chunk)
     from onecat_vllm import envs
-    extended = keep or bias_table is not None or gate is not None or kv_cache.shape[1] == 1   # not in the native CPU kernel
+    extended = keep or bias_table is not None or gate is not None or kv_cache.shape[1] == 1 or chunk   # not in the native CPU kernel
     if envs.ONECAT_CPU_ATTENTION == "native" and not extended and kv_cache.dtype in (torch.float32, torch.bfloat16) and q.dtype in (torch.float32, torch.bfloat16):
         return cpu_paged_attention(q, kv_cache, md.block_table, md.query_start_loc, md.seq_lens, scale, out, window=window, softcap=softcap, sinks=sinks)
     return ref.paged_attention(q, kv_cache, md.block_table, md.query_start_loc, md.seq_lens, scale, out, window=window, softcap=softcap,
-                               sinks=sinks, keep=keep, bias_table=bias_table, gate=gate)
+                               sinks=sinks, keep=keep, bias_table=bias_table, gate=gate, chunk=chunk)
 
 
 def cpu_paged_attention(q, kv_cache, block_table, query_start_loc, seq_lens, scale, out=None, return_lse=False, window=0, softcap=0.0, sinks=None,

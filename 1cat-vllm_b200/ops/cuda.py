@@ -18,7 +18,7 @@ except ImportError as e:  # pragma: no cover
     raise ImportError("the CUDA extension onecat_vllm.ops._C is not built; run `python -c 'import __graft_entry__ as g; g.build()'` "
                       f"or `python 1cat-vllm_b200/ops/build.py` ({e})") from e
 
-EPI_STORE, EPI_SILU_MUL, EPI_GELU_TANH = 0, 1, 2
+EPI_STORE, EPI_SILU_MUL, EPI_GELU_TANH, EPI_GELU_MUL = 0, 1, 2, 3
 TORCH_STANDINS: set = set()  # names of ops that ran as device-side PyTorch code in this process
 _LAUNCHES = 0  # launches of our own kernels (for bench accounting)
 _LIB_GEMM = os.environ.get("ONECAT_GEMM_BACKEND", "tcgen05") == "library"  # debug switch only
@@ -130,13 +130,20 @@ def prepare_w4(layer, q: torch.Tensor, z: torch.Tensor, s: torch.Tensor, group: 
 def prepare_bf16(layer) -> None:
     w = layer.weight.data
     n_rows, epi, n_out = w.shape[0], EPI_STORE, w.shape[0]
-    if layer.fuse_silu_mul:
+    gelu_mul = getattr(layer, "fuse_gelu_mul", False)
+    if layer.fuse_silu_mul or gelu_mul:
+        n = n_rows // 2
+        if n % 16:   # the epilogue pairs 16 gate rows with 16 up rows: zero rows make up the last block (their outputs are cut off)
+            w = torch.nn.functional.pad(w.view(2, n, -1), (0, 0, 0, -n % 16)).reshape(-1, w.shape[1])
+            n_rows = w.shape[0]
         w = w[interleave_gate_up(n_rows // 2, w.device)].contiguous()
         layer.weight.data = w
-        epi, n_out = EPI_SILU_MUL, n_rows // 2
+        epi, n_out = EPI_GELU_MUL if gelu_mul else EPI_SILU_MUL, n_rows // 2
     elif getattr(layer, "fuse_gelu_tanh", False):
         epi = EPI_GELU_TANH
     layer.kernel_state = dict(kind="bf16", n_rows=n_rows, n_out=n_out, epi=epi, K=w.shape[1])
+    if epi in (EPI_SILU_MUL, EPI_GELU_MUL) and n != n_out:
+        layer.kernel_state["n_cut"] = n
     if w.shape[1] % 64:   # the GEMM walks whole 64-wide k tiles: zero columns in a copy that only the kernel reads
         layer.kernel_state["w_pad"] = torch.nn.functional.pad(w, (0, -w.shape[1] % 64)).contiguous()
 
@@ -330,6 +337,8 @@ def _linear_f32(layer, x: torch.Tensor) -> torch.Tensor:
     if getattr(layer, "fuse_gelu_tanh", False):
         _LAUNCHES += 1
         _C.gelu_tanh_f32(y)
+    if getattr(layer, "fuse_gelu_mul", False):
+        return ref.gelu_tanh_and_mul(y)
     return y
 
 
@@ -360,11 +369,15 @@ def linear(layer, x: torch.Tensor, out: Optional[torch.Tensor] = None, push=None
         y = torch.nn.functional.linear(x, layer.weight if w is None else w, bias)
         if ks["epi"] == EPI_SILU_MUL:  # rows are interleaved in blocks of 16
             y = y.view(T, -1, 2, 16)
-            return (torch.nn.functional.silu(y[:, :, 0].float()) * y[:, :, 1].float()).to(x.dtype).reshape(T, -1)
+            return (torch.nn.functional.silu(y[:, :, 0].float()) * y[:, :, 1].float()).to(x.dtype).reshape(T, -1)[:, : ks.get("n_cut")]
+        if ks["epi"] == EPI_GELU_MUL:
+            y = y.view(T, -1, 2, 16)
+            return (torch.nn.functional.gelu(y[:, :, 0].float(), approximate="tanh") * y[:, :, 1].float()).to(x.dtype).reshape(T, -1)[:, : ks.get("n_cut")]
         if ks["epi"] == EPI_GELU_TANH:
             y = torch.nn.functional.gelu(y, approximate="tanh")
         return y.to(out.dtype)
-    return _gemm(x, layer.weight if w is None else w, None, None, out, bias, ks["n_rows"], ks["n_rows"], ks["n_out"], 0, ks["epi"], 1, push=push)
+    y = _gemm(x, layer.weight if w is None else w, None, None, out, bias, ks["n_rows"], ks["n_rows"], ks["n_out"], 0, ks["epi"], 1, push=push)
+    return y[:, : ks["n_cut"]] if "n_cut" in ks else y
 
 
 # ----------------------------------------------------------------------------- elementwise
@@ -420,6 +433,23 @@ def stream_join(part, x, post, scale, nxt, out_dtype=None, add=None, copy_out=No
     _C.stream_join(part, x, x_out, *post[:5], scale, *nxt[:5], y, add, copy_out, (copy_out.dtype if y is None and copy_out is not None
                    else out_dtype or part.dtype) == torch.float32, mul, post[5], nxt[5])
     return y, x_out
+
+
+def embed_stream(ids, table, scale, prev, bigram, muls, out_dtype, gathered=False):
+    global _LAUNCHES
+    _LAUNCHES += 1
+    T, H = ids.shape[0], table.shape[1]
+    x = torch.empty(T, H, dtype=torch.float32, device=table.device)
+    y = torch.empty(T, H, dtype=out_dtype, device=table.device) if out_dtype != torch.float32 else None
+    _C.embed_stream(ids.to(torch.int32).contiguous(), table, scale, prev, bigram, muls[0], muls[1], x, y, gathered)
+    return x, (x if y is None else y)
+
+
+def diff_prepare(qkv, q_norm, k_norm, eps, positions, cos_sin, kv_cache, slot_mapping, heads, kv_heads, dim, vdim, interleaved):
+    global _LAUNCHES
+    _LAUNCHES += 1
+    return _C.diff_prepare(qkv if qkv.stride(-1) == 1 else qkv.contiguous(), q_norm, k_norm, eps, positions, cos_sin, kv_cache, slot_mapping, heads,
+                           kv_heads, dim, vdim, interleaved)
 
 
 def sample(logits, temperature, top_k=None, top_p=None, min_p=None, generators=None, kept=None):
@@ -512,13 +542,13 @@ def plan_attention(query_lens: list, seq_lens: list, Hq: int, Hkv: int, D: int, 
 
 
 def attention_span(window: int, keep: int) -> int:
-    """Most keys that the decode kernel walks for a sliding-window layer, in whole 64-key tiles; 0: the whole context."""
+    """Most keys that the decode kernel walks for a sliding-window (or chunked) layer, in whole 64-key tiles; 0: the whole context."""
     return 64 * (-(-window // 64) + 1 + -(-keep // 64)) if window else 0
 
 
-def paged_attention(q, kv_cache, md, scale, out=None, lse=None, window=0, softcap=0.0, sinks=None, keep=0, bias_table=None, gate=None):
+def paged_attention(q, kv_cache, md, scale, out=None, lse=None, window=0, softcap=0.0, sinks=None, keep=0, bias_table=None, gate=None, chunk=0):
     """``window`` (tokens, 0 = full), ``softcap`` (0 = off), ``sinks`` (fp32 ``[Hq]``), ``keep`` (first tokens visible outside the window),
-    ``bias_table`` (fp32 ``[Hq, n]`` by distance), ``gate`` (``[T, Hq]`` logits) and a cache with one tensor per page select the mma.sync
+    ``bias_table`` (fp32 ``[Hq, n]`` by distance), ``gate`` (``[T, Hq]`` logits), ``chunk`` (positions, 0 = off) and a cache with one tensor per page select the mma.sync
     kernels; the tcgen05 prefill kernel serves plain causal attention with D = 128. fp32 queries run the fp32 kernel."""
     global _LAUNCHES
     T, Hq, D = q.shape
@@ -529,11 +559,11 @@ def paged_attention(q, kv_cache, md, scale, out=None, lse=None, window=0, softca
         G = Hq // Hkv
         tiles = sum(-(-n * G // 16) for n in md.query_lens_cpu)
         _C.paged_attention(q, kv_cache, out, lse, md.query_start_loc, md.seq_lens, md.block_table, scale, 3, tiles, 1, md.max_query_len, 0, None, None,
-                           window, softcap, sinks, 1.0, 1.0, keep, bias_table, gate)
+                           window, softcap, sinks, 1.0, 1.0, keep, bias_table, gate, chunk)
         _LAUNCHES += 1
         return out
-    extended = keep > 0 or bias_table is not None or gate is not None or kv_cache.shape[1] == 1
-    key = (Hq, Hkv, D, attention_span(window, keep)) if extended else (Hq, Hkv, D)
+    extended = keep > 0 or bias_table is not None or gate is not None or kv_cache.shape[1] == 1 or chunk > 0
+    key = (Hq, Hkv, D, attention_span(min(window, chunk) if window and chunk else window or chunk, keep)) if extended else (Hq, Hkv, D)
     plan = getattr(md, "attn_plan", None)
     if plan is None or plan[0] != key:
         plan = (key, plan_attention(md.query_lens_cpu, md.seq_lens_cpu, Hq, Hkv, D, _sms(q.device), span=key[3] if extended else 0,
@@ -547,7 +577,7 @@ def paged_attention(q, kv_cache, md, scale, out=None, lse=None, window=0, softca
         ws_o, ws_ml = (w.attn_static if getattr(md, "static_ws", False) else w.attn)(splits * T * Hq * D, splits * T * Hq * 2)
     if n_short:
         _C.paged_attention(q, kv_cache, out, lse, md.query_start_loc, md.seq_lens, md.block_table, scale, 1, 0, splits,
-                           md.max_query_len, short, ws_o, ws_ml, window, softcap, sinks, 1.0, 1.0, keep, bias_table, gate)
+                           md.max_query_len, short, ws_o, ws_ml, window, softcap, sinks, 1.0, 1.0, keep, bias_table, gate, chunk)
         _LAUNCHES += 2 if splits > 1 else 1
     if tiles:
         if (D == 128 and q.stride(1) == D and _ATTN_PREFILL_TC and not window and not softcap and sinks is None and not extended
@@ -558,7 +588,38 @@ def paged_attention(q, kv_cache, md, scale, out=None, lse=None, window=0, softca
                                md.max_query_len, short, None, None, 0, 0.0, None, 1.0, 1.0)
         else:
             _C.paged_attention(q, kv_cache, out, lse, md.query_start_loc, md.seq_lens, md.block_table, scale, 0, tiles, 1,
-                               md.max_query_len, short, None, None, window, softcap, sinks, 1.0, 1.0, keep, bias_table, gate)
+                               md.max_query_len, short, None, None, window, softcap, sinks, 1.0, 1.0, keep, bias_table, gate, chunk)
+        _LAUNCHES += 1
+    return out
+
+
+def diff_attention(q, kv_cache, md, scale, lam, out_scale, eps, vdim, softcap, chunk):
+    """Both maps of a head are rows of one tile, so decoding and prefill each are one launch (and a combine where the context is split) that
+    ends with the difference and the head norm. Rows of the tensor-core kernels: 64, 128 or 256 wide; others, and fp32, run the plain kernel."""
+    global _LAUNCHES
+    T, rows, _ = q.shape
+    G, D = kv_cache.shape[2], kv_cache.shape[4]
+    out = torch.empty(T, rows // 2, vdim, dtype=q.dtype, device=q.device)
+    common = (md.query_start_loc, md.seq_lens, md.block_table, scale)
+    if q.dtype == torch.float32 or D not in (64, 128, 256) or rows // G > 64:
+        tiles = sum(-(-n * (rows // G) // 16) for n in md.query_lens_cpu)
+        _C.diff_attention(q, kv_cache, out, *common, 3, tiles, 1, md.max_query_len, 0, None, None, softcap, chunk, lam, out_scale, eps)
+        _LAUNCHES += 1
+        return out
+    key = ("diff", rows, G, D, chunk)
+    plans = md.__dict__.setdefault("_diff_plans", {})
+    if key not in plans:
+        plans[key] = plan_attention(md.query_lens_cpu, md.seq_lens_cpu, rows, G, D, _sms(q.device), span=attention_span(chunk, 0))
+    short, tiles, splits = plans[key]
+    if any(0 < n <= short for n in md.query_lens_cpu):
+        ws_o = ws_ml = None
+        if splits > 1:
+            w = workspace(q.device)
+            ws_o, ws_ml = (w.attn_static if getattr(md, "static_ws", False) else w.attn)(splits * T * rows * D, splits * T * rows * 2)
+        _C.diff_attention(q, kv_cache, out, *common, 1, 0, splits, md.max_query_len, short, ws_o, ws_ml, softcap, chunk, lam, out_scale, eps)
+        _LAUNCHES += 2 if splits > 1 else 1
+    if tiles:
+        _C.diff_attention(q, kv_cache, out, *common, 0, tiles, 1, md.max_query_len, short, None, None, softcap, chunk, lam, out_scale, eps)
         _LAUNCHES += 1
     return out
 
@@ -752,10 +813,11 @@ def plan_mla_splits(H: int, lora: int, query_lens: list, seq_lens: list, num_sms
     return choose_decode_splits(len(query_lens) * -(-max(query_lens) * H // 16), max(seq_lens), num_sms, per_sm)
 
 
-def mla_decode(q_abs, q_pe, latent_cache, md, scale, lora, cos_sin=None, interleaved=True, fine=False, skip_min_len=0):
+def mla_decode(q_abs, q_pe, latent_cache, md, scale, lora, cos_sin=None, interleaved=True, fine=False, skip_min_len=0, sinks=None, gate=None):
     """Multi-query attention over the cached latents: ``q_abs`` ``[T, H, lora]``, ``q_pe`` ``[T, H, rope]`` (rotated by the kernel when
     ``cos_sin`` is given). ``fine``: softmax weights in two bf16 terms. ``skip_min_len``: requests with at least that many new tokens are
-    left out (their rows of the result hold nothing)."""
+    left out (their rows of the result hold nothing). ``sinks`` fp32 ``[H]`` join the softmax denominator; ``gate`` ``[T, H]``: logits of a
+    per-head output gate."""
     global _LAUNCHES
     T, H, _ = q_abs.shape
     ws_o = ws_ml = None
@@ -776,7 +838,7 @@ def mla_decode(q_abs, q_pe, latent_cache, md, scale, lora, cos_sin=None, interle
             ws_o, ws_ml = (w.attn_static if static else w.attn)(splits * T * H * lora, splits * T * H * 2)
     _LAUNCHES += 2 if splits > 1 else 1
     return _C.mla_decode(q_abs, q_pe, latent_cache, md.query_start_loc, md.seq_lens, md.block_table, scale, max(ql), splits, ws_o, ws_ml, cos_sin,
-                         interleaved, fine, skip_min_len)
+                         interleaved, fine, skip_min_len, sinks, gate)
 
 
 MLA_PREFILL_MIN_LEN = 64           # portions of at least this many tokens attend in the expanded form
@@ -808,14 +870,14 @@ def mla_prefill_plan(md, H: int, nope: int, rope: int, vd: int, lora_pad: int, d
     return out
 
 
-def mla_prefill(plan, q, latent_cache, md, expand, out, nope, rope, lora_pad, scale, cos_sin, interleaved, fine):
+def mla_prefill(plan, q, latent_cache, md, expand, out, nope, rope, lora_pad, scale, cos_sin, interleaved, fine, sinks=None, gate=None):
     """Causal attention of the planned requests in the expanded form, into their rows of ``out`` ``[T, H, vd]``. ``expand(latents)`` is the
     per-head up-projection ``[rows, H * (keys | values)]`` with both parts padded to 64 columns."""
     global _LAUNCHES
     meta, n, rows, tiles, _ = plan
     _LAUNCHES += 3
     lat, rot, qp = _C.mla_prefill_inputs(q, latent_cache, md.query_start_loc, md.block_table, md.positions, meta, n, rows, nope, lora_pad, cos_sin, interleaved)
-    _C.mla_prefill(qp, expand(lat), rot, out, md.query_start_loc, md.seq_lens, meta, n, tiles, nope, rope, scale, fine)
+    _C.mla_prefill(qp, expand(lat), rot, out, md.query_start_loc, md.seq_lens, meta, n, tiles, nope, rope, scale, fine, sinks, gate)
     return out
 
 

@@ -236,7 +236,7 @@ def distance_buckets(buckets: int, max_dist: int) -> list[int]:
 def paged_attention(q, kv_cache, block_table, query_start_loc, seq_lens, scale: float,
                     out: Optional[torch.Tensor] = None, return_lse: bool = False, window: int = 0, softcap: float = 0.0,
                     sinks: Optional[torch.Tensor] = None, keep: int = 0, bias_table: Optional[torch.Tensor] = None,
-                    gate: Optional[torch.Tensor] = None):
+                    gate: Optional[torch.Tensor] = None, chunk: int = 0):
     """Causal varlen attention over a paged cache. Request r owns query rows
     ``query_start_loc[r]:query_start_loc[r+1]`` which are the LAST rows of its ``seq_lens[r]``-token context
     (so decode, chunked prefill with prefix and multi-token verify are the same call).
@@ -244,7 +244,8 @@ def paged_attention(q, kv_cache, block_table, query_start_loc, seq_lens, scale: 
     (reference: Gemma2/3, GPT-OSS, Mistral sliding attention); ``softcap`` > 0: scores become cap·tanh(score/cap) (Gemma2);
     ``sinks`` ``[Hq]``: one extra logit per head that takes probability mass but contributes no value (GPT-OSS). ``keep``: keys at
     positions below it stay visible outside the window. ``bias_table`` ``[Hq, n]``: added to the scaled score by distance, distances past
-    the end take the last entry. ``gate`` ``[T, Hq]``: outputs are multiplied by its sigmoid. A cache with one tensor per page
+    the end take the last entry. ``gate`` ``[T, Hq]``: outputs are multiplied by its sigmoid. ``chunk`` > 0: only keys of the query's own
+    chunk of that many positions are visible. A cache with one tensor per page
     (``[blocks, 1, ...]``) serves as keys and values."""
     T, Hq, D = q.shape
     Hkv, bs = kv_cache.shape[2], kv_cache.shape[3]
@@ -276,6 +277,8 @@ def paged_attention(q, kv_cache, block_table, query_start_loc, seq_lens, scale: 
         s = s.masked_fill(kpos > qpos, -float("inf"))
         if window > 0:
             s = s.masked_fill((kpos <= qpos - window) & (kpos >= keep), -float("inf"))
+        if chunk > 0:
+            s = s.masked_fill((kpos // chunk != qpos // chunk) & (kpos >= keep), -float("inf"))
         l = torch.logsumexp(s, dim=-1)
         if sinks is not None:
             l = torch.logaddexp(l, sinks.float().view(Hkv, g, 1).expand_as(l))
@@ -286,6 +289,51 @@ def paged_attention(q, kv_cache, block_table, query_start_loc, seq_lens, scale: 
         o[q0:q1] = oo.to(o.dtype)
         lse[q0:q1] = l.reshape(Hq, nq).t()
     return (o, lse) if return_lse else o
+
+
+def diff_prepare(qkv, q_norm, k_norm, eps: float, positions, cos_sin, kv_cache, slot_mapping, heads: int, kv_heads: int, dim: int, vdim: int,
+                 interleaved: bool):
+    """Between the projections and differential attention: ``qkv`` ``[T, 2 heads dim + 2 kv_heads dim + kv_heads vdim]``, queries and keys head
+    by head as (map 1, map 2). Every map of every head is RMS-normalised, rotated over the first ``cos_sin.shape[1]`` dimensions and padded
+    with zeros to half of the cache's row width D; key rows (map 1 | map 2) and value rows go into their pages ``[blocks, 2, kv_heads, bs, D]``
+    (rows without a slot into the placeholder block 0). Returns the queries ``[T, 2 heads, D / 2]``."""
+    T, D, rot = qkv.shape[0], kv_cache.shape[4], cos_sin.shape[1]
+    q, k, v = qkv.split([2 * heads * dim, 2 * kv_heads * dim, kv_heads * vdim], 1)
+
+    def finish(x, w):
+        x = x.reshape(T, -1, dim).float()
+        x = x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+        if rot:
+            x = torch.cat([rope_rows(x[..., :rot], positions, cos_sin, interleaved), x[..., rot:]], -1)
+        return F.pad(x, (0, D // 2 - dim)).to(kv_cache.dtype)
+    slot = slot_mapping.long().clamp(min=0)
+    b, o = slot // kv_cache.shape[3], slot % kv_cache.shape[3]
+    kv_cache[b, 0, :, o] = finish(k, k_norm).reshape(T, kv_heads, D)
+    kv_cache[b, 1, :, o] = F.pad(v.reshape(T, kv_heads, vdim), (0, D - vdim)).to(kv_cache.dtype)
+    return finish(q, q_norm)
+
+
+def diff_attention(q, kv_cache, block_table, query_start_loc, seq_lens, scale: float, lam, out_scale: float, eps: float, vdim: int,
+                   softcap: float = 0.0, chunk: int = 0):
+    """Differential attention over a paged cache of ``diff_prepare``: ``rms(a1 - lam a2) * out_scale`` with a1, a2 the outputs of a head's two
+    maps over the same values. ``q`` ``[T, 2 heads, D / 2]``, ``lam`` one number in a tensor; returns ``[T, heads, vdim]``."""
+    T, maps, half = q.shape
+    wide = torch.zeros(T, maps, 2 * half, dtype=torch.float32, device=q.device)   # a map's queries see its half of the key rows
+    wide[:, 0::2, :half], wide[:, 1::2, half:] = q[:, 0::2].float(), q[:, 1::2].float()
+    a = paged_attention(wide, kv_cache, block_table, query_start_loc, seq_lens, scale, softcap=softcap, chunk=chunk)[..., :vdim]
+    o = a[:, 0::2] - lam.float() * a[:, 1::2]
+    return (o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * out_scale).to(q.dtype)
+
+
+def embed_stream(ids, table, scale: float, prev=None, bigram=None, muls=(0, 0), out_dtype=None, gathered: bool = False):
+    """Start of an fp32 residual stream: ``table[id] * scale``, plus the row of ``bigram`` (last row: no previous token) that (previous token,
+    token) hash to. ``prev`` < 0: none. ``gathered``: ``table`` holds the tokens' own rows. Returns (the stream, the stream in ``out_dtype``)."""
+    x = (table if gathered else F.embedding(ids.long(), table)).float() * scale
+    if bigram is not None:
+        n = bigram.shape[0] - 1
+        row = torch.where(prev < 0, n, (prev.long() * muls[0] + ids.long() * muls[1]) % n)
+        x = x + F.embedding(row, bigram).float()
+    return x, x.to(out_dtype)
 
 
 def merge_attn_states(o1, lse1, o2, lse2):
@@ -331,10 +379,11 @@ def mla_prepare(q_latent, kv, q_w, kv_w, eps, positions, cos_sin, cache, slot_ma
     return rms_norm(q_latent, q_w, eps)[0] if q_latent is not None else None
 
 
-def mla_decode(q_nope_abs, q_rope, latent_cache, block_table, query_start_loc, seq_lens, scale: float, kv_lora: int):
+def mla_decode(q_nope_abs, q_rope, latent_cache, block_table, query_start_loc, seq_lens, scale: float, kv_lora: int, sinks=None, gate=None):
     """MLA decode as MQA over the latent cache (reference: csrc/cpu/mla_decode.cpp; layers/attention/mla_attention.py
     ``forward_mqa``). q_nope_abs ``[T,H,kv_lora]`` (W_UK absorbed), q_rope ``[T,H,rope]``, cache
-    ``[blocks, bs, kv_lora+rope]``. Returns ``[T,H,kv_lora]`` (to be multiplied by W_UV)."""
+    ``[blocks, bs, kv_lora+rope]``. ``sinks`` ``[H]``: logits that join the softmax denominator only; ``gate`` ``[T,H]``: outputs are
+    multiplied by its sigmoid. Returns ``[T,H,kv_lora]`` (to be multiplied by W_UV)."""
     T, H, _ = q_nope_abs.shape
     bs = latent_cache.shape[1]
     out = torch.empty(T, H, kv_lora, dtype=q_nope_abs.dtype, device=q_nope_abs.device)
@@ -350,8 +399,13 @@ def mla_decode(q_nope_abs, q_rope, latent_cache, block_table, query_start_loc, s
         s = torch.einsum("qhd,kd->hqk", qcat[q0:q1], kv) * scale
         qpos = torch.arange(S - nq, S, device=kv.device).view(1, nq, 1)
         s = s.masked_fill(torch.arange(S, device=kv.device).view(1, 1, S) > qpos, -float("inf"))
-        p = torch.softmax(s, dim=-1)
-        out[q0:q1] = torch.einsum("hqk,kd->qhd", p, kv[:, :kv_lora]).to(out.dtype)
+        l = torch.logsumexp(s, dim=-1, keepdim=True)
+        if sinks is not None:
+            l = torch.logaddexp(l, sinks.float().view(H, 1, 1).expand_as(l))
+        o = torch.einsum("hqk,kd->qhd", torch.exp(s - l), kv[:, :kv_lora])
+        if gate is not None:
+            o = o * torch.sigmoid(gate[q0:q1].float()).unsqueeze(-1)
+        out[q0:q1] = o.to(out.dtype)
     return out
 
 

@@ -30,3 +30,4 @@ class AttentionMetadata:
     is_uniform_decode: bool = False
     uniform_query_len: int = 1
     mrope_positions: Optional[torch.Tensor] = None  # int32 [3, T] (temporal, height, width) for models with rotary sections
+    prev_ids: Optional[torch.Tensor] = None  # int32 [T] token ahead of each one in its sequence, -1: none (models with bigram embeddings)

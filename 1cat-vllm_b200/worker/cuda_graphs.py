@@ -41,7 +41,7 @@ class DecodeGraphs:
         # against one latent "head" of 512
         self.geom = None
         attns = [l.self_attn for l in layers]
-        self.own_plans = any(a.kv_shared or a.window_keep or a.bias_table is not None or (a.Hq, a.Hkv, a.D) != (attns[0].Hq, attns[0].Hkv, attns[0].D)
+        self.own_plans = any(getattr(a, "chunk", 0) or getattr(a, "diff", None) is not None or a.kv_shared or a.window_keep or a.bias_table is not None or (a.Hq, a.Hkv, a.D) != (attns[0].Hq, attns[0].Hkv, attns[0].D)
                              for a in attns)
         mlas = [l.self_attn for l in mla]
         self.own_plans = self.own_plans or bool(mla) and (bool(layers) or any((a.H, a.lora_pad) != (mlas[0].H, mlas[0].lora_pad) for a in mlas)) or not (layers or mla)
@@ -52,7 +52,7 @@ class DecodeGraphs:
             K.workspace(runner.device).attn_static(32 * tmax * max(a.Hq * a.D for a in attns), 32 * tmax * 2 * max(a.Hq for a in attns))
             for a in mlas:
                 K.workspace(runner.device).attn_static(32 * tmax * a.H * a.lora_pad, 32 * tmax * a.H * 2)
-            spans = [K.attention_span(a.window, a.window_keep) for a in attns]
+            spans = [K.attention_span(a.window or getattr(a, "chunk", 0), a.window_keep) for a in attns]
             self.max_span = max(spans) if all(spans) and not mla else 0
         elif mla:
             self.geom = ("mla", mlas[0].H, mlas[0].lora_pad)
@@ -101,6 +101,8 @@ class DecodeGraphs:
                                uniform_query_len=q)
         if r._seg["pos3"]:
             md.mrope_positions = r._view("pos3", 3 * r._tcap).view(3, r._tcap)[:, :T]
+        if r._seg["prev"]:
+            md.prev_ids = r._view("prev", T)
         if self.own_plans:
             md.seq_lens_cpu = [splits] * rp   # the context bucket; each layer's plan follows from it
         elif self.geom[0] == "mla":

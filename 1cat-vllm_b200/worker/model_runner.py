@@ -145,7 +145,7 @@ class ModelRunner:
             dcfg.max_model_len = self.mc.max_model_len
             if dcfg.vocab_size != self.mc.vocab_size:
                 raise ValueError(f"the draft model's vocabulary ({dcfg.vocab_size}) differs from the target's ({self.mc.vocab_size})")
-            if dcfg.is_hybrid or dcfg.use_mla:
+            if dcfg.is_hybrid or dcfg.use_mla or dcfg.bigram or any(o.get("attn_diff") is not None for o in dcfg.layer_overrides):
                 raise ValueError("the draft model must be a plain attention decoder (its K/V pages live under the target's block ids)")
             self.draft = load_model(dcfg, self.device)
         if self.spec.method == "eagle3":
@@ -218,8 +218,9 @@ class ModelRunner:
         if cd in ("auto", "bfloat16", "bf16"):
             return self.mc.dtype
         if cd in ("fp8", "fp8_e4m3"):
-            if self.mc.attn_kv_shared or self.mc.attn_rel_buckets or any(o.get("attn_window_keep") for o in self.mc.layer_overrides):
-                raise ValueError("an fp8 KV cache is not served for attention with shared keys and values, a distance bias or kept first tokens")
+            if self.mc.attn_kv_shared or self.mc.attn_rel_buckets or any(o.get("attn_window_keep") or o.get("attn_diff") is not None
+                                                                         for o in self.mc.layer_overrides):
+                raise ValueError("an fp8 KV cache is not served for differential attention, shared keys and values, a distance bias or kept first tokens")
             return torch.float8_e4m3fn
         raise ValueError(f"kv cache dtype {cd!r} is not supported (auto | fp8 | fp8_e4m3)")
 
@@ -274,7 +275,8 @@ class ModelRunner:
         # one packed int32 staging area: ids | positions | slot_mapping | qsl | seq_lens | state_slots | has_init | logit_idx
         # pdst | psrc: where last step's sampled tokens (still on the device) go in this step's ids (async scheduling)
         self._seg = {"ids": T, "pos": T, "slot": T, "qsl": R + 1, "seq": R, "sslot": R, "hinit": R, "lidx": T, "pdst": R, "psrc": R,
-                     "pos3": 3 * T if getattr(self.mc, "mrope_section", None) else 0}  # [3, T] rotary positions (models with rotary sections)
+                     "pos3": 3 * T if getattr(self.mc, "mrope_section", None) else 0,  # [3, T] rotary positions (models with rotary sections)
+                     "prev": T if self.mc.bigram else 0}  # token ahead of each one (models with bigram embeddings)
         self._tcap = T
         total = sum(self._seg.values())
         self.h_pack = host(total, torch.int32)
@@ -368,6 +370,7 @@ class ModelRunner:
         psrc = npk[o["psrc"][0]: o["psrc"][0] + R]
         n_patch = 0
         pos3 = npk[o["pos3"][0]: o["pos3"][0] + 3 * self._tcap].reshape(3, self._tcap) if self._seg["pos3"] else None
+        prev = npk[o["prev"][0]: o["prev"][0] + T] if self._seg["prev"] else None
         if self._h2d_done is not None:
             self._h2d_done.synchronize()   # the previous step's copy out of this staging area has finished (it has, long ago)
         for r, rid in enumerate(req_ids):
@@ -405,6 +408,11 @@ class ModelRunner:
                 b = np.asarray(bl[b0:nb], dtype=np.int32)
                 p = pos[t:t + n]
                 slot[t:t + n] = b[p // bs - b0] * bs + p % bs
+            if prev is not None:
+                # a token in flight is only ever the last one of its sequence: the one ahead of it is known. Nothing precedes a first token,
+                # nor the first one behind a prompt that was given as vectors.
+                prev[t + 1:t + n] = ids[t:t + n - 1]
+                prev[t] = known[start - 1] if start > 0 and (st.prompt_embeds is None or start != st.num_prompt_tokens) else -1
             # block-table row: a request that kept its row only appends the blocks it gained (its list is append-only)
             if bt_owner[r] is st and bt_written[r] <= nb:
                 w = bt_written[r]
@@ -453,6 +461,8 @@ class ModelRunner:
         npk[o["pos"][0] + T: o["pos"][0] + tp] = 0
         if self._seg["pos3"]:
             npk[o["pos3"][0]: o["pos3"][0] + 3 * self._tcap].reshape(3, self._tcap)[:, T:tp] = 0
+        if self._seg["prev"]:
+            npk[o["prev"][0] + T: o["prev"][0] + tp] = -1
         npk[o["slot"][0] + T: o["slot"][0] + tp] = -1
         npk[o["qsl"][0] + R + 1: o["qsl"][0] + rp + 1] = T
         npk[o["seq"][0] + R: o["seq"][0] + rp] = 0
@@ -485,7 +495,8 @@ class ModelRunner:
             positions=self._view("pos", T), max_query_len=max_q, max_seq_len=max_s, state_slots=self._view("sslot", R),
             has_initial_state=self._view("hinit", R), query_lens_cpu=query_lens, seq_lens_cpu=seq_lens,
             is_uniform_decode=(max_q == min(query_lens)) and max_q <= 1 + self.num_spec, uniform_query_len=max_q,
-            mrope_positions=self._view("pos3", 3 * self._tcap).view(3, self._tcap)[:, :T] if self._seg["pos3"] else None)
+            mrope_positions=self._view("pos3", 3 * self._tcap).view(3, self._tcap)[:, :T] if self._seg["pos3"] else None,
+            prev_ids=self._view("prev", T) if self._seg["prev"] else None)
 
     def _sampling_metadata(self, req_ids: list, rows: list[int]) -> SamplingMetadata:
         """One entry per *sampling request* (requests contributing logits rows this step)."""
@@ -847,12 +858,13 @@ class ModelRunner:
         if not self.pp.is_first_pp:
             return None
         emb, o = None, 0
+        prev = self._view("prev", ids.shape[0]) if self._seg["prev"] else None
         for rid, q in zip(req_ids, query_lens):
             st = self.requests[rid]
             c0 = st.num_computed_tokens
             if st.prompt_embeds is not None and c0 < st.num_prompt_tokens:
                 if emb is None:
-                    emb = self.model.model.embed(ids)
+                    emb = self.model.model.embed(ids, prev)
                 n = min(q, st.num_prompt_tokens - c0)
                 emb[o:o + n] = st.prompt_embeds[c0:c0 + n]
             for f in st.mm_features or ():
@@ -860,7 +872,7 @@ class ModelRunner:
                 if lo >= hi:
                     continue
                 if emb is None:
-                    emb = self.model.model.embed(ids)
+                    emb = self.model.model.embed(ids, prev)
                 emb[o + lo - c0: o + hi - c0] = self.encoder_cache[f.mm_hash][lo - f.offset: hi - f.offset]
             o += q
         return emb
@@ -1092,7 +1104,7 @@ class ModelRunner:
                                torch.full((T,), -1, dtype=torch.int32, device=self.device),
                                torch.zeros(T, dtype=torch.int32, device=self.device), int(seq.max()), int(seq.max()),
                                torch.zeros(R, dtype=torch.int32, device=self.device), torch.zeros(R, dtype=torch.int32, device=self.device),
-                               seq.tolist(), seq.tolist())
+                               seq.tolist(), seq.tolist(), prev_ids=torch.full((T,), -1, dtype=torch.int32, device=self.device) if self.mc.bigram else None)
         ids = torch.zeros(T, dtype=torch.int32, device=self.device)
         caches = self.kv_caches if self.kv_caches else self._tiny_caches()
         inter = None
