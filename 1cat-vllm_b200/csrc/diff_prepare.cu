@@ -1,7 +1,6 @@
 // Differential attention, between the QKV projection and the attention kernel: every map of every query and key head is RMS-normalised
 // and rotated in fp32, queries leave padded for the kernel, keys (both maps of a head side by side) and values go into their pages.
-// One warp per (token, head, map) or (token, value head); a lane holds the pairs lane, lane + 32, ... of its row, so both elements of a
-// rotated pair are in one thread.
+// A lane holds the pairs lane, lane + 32, ... of a row, so both elements of a rotated pair are in one thread.
 #include "common.cuh"
 #include "kernels.h"
 
@@ -20,25 +19,26 @@ __device__ __forceinline__ float2 ld2(const __nv_bfloat16* p) { return __bfloat1
 __device__ __forceinline__ void st2(float* p, float2 v) { *reinterpret_cast<float2*>(p) = v; }
 __device__ __forceinline__ void st2(__nv_bfloat16* p, float2 v) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v.x, v.y); }
 
-// NP: pairs per lane. VEC: rows have an even number of elements and start on pairs.
+// A warp takes kRows neighbouring (head, map) rows of one token - all their loads are in flight before the first reduction - or one value row.
+// NP: pairs per lane and row. VEC: rows have an even number of elements and start on pairs.
+constexpr int kRows = 4;
 template <typename E, int NP, bool VEC>
 __global__ void __launch_bounds__(256) diff_prepare_kernel(const DiffPrepareParams p) {
   pdl_trigger();
   pdl_wait();
-  const int units = 2 * p.H + 3 * p.G, lane = threadIdx.x & 31;
-  const long long wid = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
-  const int t = (int)(wid / units), u = (int)(wid - (long long)t * units);
+  const int maps = 2 * (p.H + p.G), groups = (maps + kRows - 1) / kRows, units = groups + p.G, lane = threadIdx.x & 31;
+  const unsigned wid = blockIdx.x * 8 + (threadIdx.x >> 5);
+  const int t = (int)(wid / (unsigned)units), unit = (int)(wid - (unsigned)t * units);
   if (t >= p.T) return;
   const E* x = reinterpret_cast<const E*>(p.x) + (size_t)t * p.ld;
-  const int kv = u - 2 * p.H, hd = p.D / 2;
-  const int slot = kv >= 0 ? p.slots[t] : 0;
-  if (slot < 0) return;
+  const int hd = p.D / 2, slot = p.slots[t];
   auto cache_row = [&](int which, int g) {
     return reinterpret_cast<E*>(p.cache) + ((((size_t)(slot / p.bs) * 2 + which) * p.G + g) * p.bs + slot % p.bs) * p.D;
   };
-  if (kv >= 2 * p.G) {
-    const int g = kv - 2 * p.G;
-    const E* v = x + (size_t)2 * (p.H + p.G) * p.dim + (size_t)g * p.vdim;
+  if (unit >= groups) {
+    if (slot < 0) return;
+    const int g = unit - groups;
+    const E* v = x + (size_t)maps * p.dim + (size_t)g * p.vdim;
     E* dst = cache_row(1, g);
     if (VEC) {
       for (int c = lane * 2; c < p.D; c += 64) st2(dst + c, c < p.vdim ? ld2(v + c) : make_float2(0.f, 0.f));
@@ -47,56 +47,77 @@ __global__ void __launch_bounds__(256) diff_prepare_kernel(const DiffPreparePara
     }
     return;
   }
-  x += (size_t)u * p.dim;   // queries and keys follow one another
-  const E* w = reinterpret_cast<const E*>(kv < 0 ? p.q_w : p.k_w);
-  E* dst = kv < 0 ? reinterpret_cast<E*>(p.q_out) + ((size_t)t * 2 * p.H + u) * hd : cache_row(0, kv >> 1) + (kv & 1) * hd;
-  const int half = p.rot / 2, pairs = (p.dim + 1) / 2;
+  const int u0 = unit * kRows, half = p.rot / 2, pairs = (p.dim + 1) / 2;
   // elements of pair i: neighbours, or (i, i + rot / 2) inside the rotated part of the half-split layout
   const bool split = !VEC || !p.interleaved;
   auto first = [&](int i) { return p.interleaved || i >= half ? 2 * i : i; };
   auto second = [&](int i) { return p.interleaved || i >= half ? 2 * i + 1 : i + half; };
-  float2 v[NP];
-  float ss = 0.f;
+  float2 v[kRows][NP], cs[NP];
 #pragma unroll
-  for (int k = 0; k < NP; ++k) {
-    const int i = lane + 32 * k;
-    v[k] = make_float2(0.f, 0.f);
-    if (i < pairs) {
-      if (split) {
-        v[k].x = ld1<E>(x + first(i));
-        if (second(i) < p.dim) v[k].y = ld1<E>(x + second(i));
-      } else {
-        v[k] = ld2(x + 2 * i);
+  for (int r = 0; r < kRows; ++r)   // queries and keys follow one another
+#pragma unroll
+    for (int k = 0; k < NP; ++k) {
+      const int i = lane + 32 * k;
+      const E* row = x + (size_t)(u0 + r) * p.dim;
+      v[r][k] = make_float2(0.f, 0.f);
+      if (i < pairs && u0 + r < maps) {
+        if (split) {
+          v[r][k].x = ld1<E>(row + first(i));
+          if (second(i) < p.dim) v[r][k].y = ld1<E>(row + second(i));
+        } else {
+          v[r][k] = ld2(row + 2 * i);
+        }
       }
     }
-    ss = fmaf(v[k].x, v[k].x, fmaf(v[k].y, v[k].y, ss));
-  }
-  const float inv = 1.f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);
-  const float* cs = p.cos_sin + (size_t)p.positions[t] * p.rot;
+  const float* angles = p.cos_sin + (size_t)p.positions[t] * p.rot;
 #pragma unroll
   for (int k = 0; k < NP; ++k) {
     const int i = lane + 32 * k;
-    if (i >= pairs) continue;
-    const int e0 = first(i), e1 = second(i);
-    float a = v[k].x * inv * ld1<E>(w + e0), b = e1 < p.dim ? v[k].y * inv * ld1<E>(w + e1) : 0.f;
-    if (i < half) {
-      const float c = cs[i], s = cs[half + i], a0 = a;
-      a = a0 * c - b * s;
-      b = b * c + a0 * s;
-    }
-    if (split) {
-      st1<E>(dst + e0, a);
-      if (e1 < p.dim) st1<E>(dst + e1, b);
-    } else {
-      st2(dst + 2 * i, make_float2(a, b));
-    }
+    cs[k] = i < half ? make_float2(angles[i], angles[half + i]) : make_float2(1.f, 0.f);
   }
-  for (int c = p.dim + lane; c < hd; c += 32) st1<E>(dst + c, 0.f);
+  float ss[kRows];
+#pragma unroll
+  for (int r = 0; r < kRows; ++r) {
+    ss[r] = 0.f;
+#pragma unroll
+    for (int k = 0; k < NP; ++k) ss[r] = fmaf(v[r][k].x, v[r][k].x, fmaf(v[r][k].y, v[r][k].y, ss[r]));
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+    for (int r = 0; r < kRows; ++r) ss[r] += __shfl_xor_sync(0xffffffffu, ss[r], o);
+#pragma unroll
+  for (int r = 0; r < kRows; ++r) {
+    const int u = u0 + r, kv = u - 2 * p.H;
+    if (u >= maps || (kv >= 0 && slot < 0)) continue;
+    const E* w = reinterpret_cast<const E*>(kv < 0 ? p.q_w : p.k_w);
+    E* dst = kv < 0 ? reinterpret_cast<E*>(p.q_out) + ((size_t)t * 2 * p.H + u) * hd : cache_row(0, kv >> 1) + (kv & 1) * hd;
+    const float inv = 1.f / sqrtf(ss[r] / (float)p.dim + p.eps);
+#pragma unroll
+    for (int k = 0; k < NP; ++k) {
+      const int i = lane + 32 * k;
+      if (i >= pairs) continue;
+      const int e0 = first(i), e1 = second(i);
+      float2 wv;
+      if (split) wv = make_float2(ld1<E>(w + e0), e1 < p.dim ? ld1<E>(w + e1) : 0.f);
+      else wv = make_float2(ld1<E>(w + 2 * i), ld1<E>(w + 2 * i + 1));
+      const float a0 = v[r][k].x * inv * wv.x, b0 = v[r][k].y * inv * wv.y;
+      const float a = i < half ? a0 * cs[k].x - b0 * cs[k].y : a0, b = i < half ? b0 * cs[k].x + a0 * cs[k].y : b0;
+      if (split) {
+        st1<E>(dst + e0, a);
+        if (e1 < p.dim) st1<E>(dst + e1, b);
+      } else {
+        st2(dst + 2 * i, make_float2(a, b));
+      }
+    }
+    for (int c = p.dim + lane; c < hd; c += 32) st1<E>(dst + c, 0.f);
+  }
 }
 
 template <typename E>
 int prepare_e(const DiffPrepareParams& p, cudaStream_t st) {
-  const long long warps = (long long)p.T * (2 * p.H + 3 * p.G);
+  const long long warps = (long long)p.T * ((2 * (p.H + p.G) + kRows - 1) / kRows + p.G);
+  if (warps >= (1ll << 31)) return -1;
   const uintptr_t pair = 2 * sizeof(E);
   auto ok = [&](const void* q) { return ((uintptr_t)q & (pair - 1)) == 0; };
   const bool vec = p.dim % 2 == 0 && p.vdim % 2 == 0 && p.D % 4 == 0 && p.ld % 2 == 0 && ok(p.x) && ok(p.q_out) && ok(p.cache);

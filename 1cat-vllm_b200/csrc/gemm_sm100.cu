@@ -32,8 +32,11 @@ namespace oc {
 
 namespace {
 
-// tanh form of GELU: 0.5 z (1 + tanh(u)) = z / (1 + e^-2u), u = sqrt(2/pi) (z + 0.044715 z^3)
-__device__ __forceinline__ float gelu_tanh(float z) { return z / (1.f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z))); }
+// tanh form of GELU: 0.5 z (1 + tanh(u)) = z / (1 + 2^(-2u log2 e)), u = sqrt(2/pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float gelu_tanh(float z) {
+  constexpr float c = -1.5957691216057308f * 1.4426950408889634f;
+  return z / (1.f + exp2f(z * fmaf(z * z, 0.044715f * c, c)));
+}
 
 #ifdef ONECAT_GEMM_TRACE
 #define TRACE(slot) do { if (p.trace) p.trace[blockIdx.x * 16 + (slot)] = globaltimer_ns(); } while (0)
@@ -267,12 +270,14 @@ gemm_wx_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ 
   // tok_gstride 4); a[] are this thread's feature row, one value per staged token
   auto emit = [&](float (&a)[32], int rows, int tok0, int tok_gstride, int n_base, int t0, int t_end, float bias_v) {
     const uint32_t buf = stg_u32 + (chunk_i & 1u) * (32 * kStagePitch);
-    if (gated) {
+    if (WKIND == 0 && p.epi == EPI_GELU_MUL) {
+#pragma unroll
+      for (int j = 0; j < 32; ++j) a[j] = gelu_tanh(a[j]) * __shfl_xor_sync(0xffffffffu, a[j], 16);
+    } else if (gated) {
 #pragma unroll
       for (int j = 0; j < 32; ++j) {  // lanes 0-15 hold gate rows, lanes 16-31 the matching up rows
         const float other = __shfl_xor_sync(0xffffffffu, a[j], 16);
-        if (WKIND == 0 && p.epi == EPI_GELU_MUL) a[j] = gelu_tanh(a[j]) * other;
-        else a[j] = a[j] / (1.f + __expf(-a[j])) * other;
+        a[j] = a[j] / (1.f + __expf(-a[j])) * other;
       }
     } else if (bias_v != 0.f) {
 #pragma unroll

@@ -1,6 +1,6 @@
 """Prefill and decode throughput of a design beside the closest models of equal size, and its kernels beside theirs.
 
-``python bench.py --design gabisun|sepirax`` prints one JSON line per size. Random weights and token ids. Model throughput is device time
+``python bench.py --design gabisun|sepirax|lodevik`` prints one JSON line per size. Random weights and token ids. Model throughput is device time
 of engine steps (CUDA events); kernels are timed alone with the L2 flushed before every launch.
 
 Gabisun: the models share width, heads, head size, window, layer runs, vocabulary and tied embeddings: Starcoder2 (layer norms, ungated
@@ -9,7 +9,11 @@ GELU feed-forward of the same width; its norms are PyTorch operations) and Mistr
 
 Sepirax: beside DeepSeek-V2 (every layer latent attention with the same heads, latents and grouped softmax experts) and Qwen3-Next (Gated-
 DeltaNet in the place of the mLSTM layers with the same number of heads and states of 128 x 128, softmax attention in the place of latent
-attention, the same experts without groups)."""
+attention, the same experts without groups).
+
+Lodevik: beside Gemma-2 (soft-capped attention with one map of the same number of columns, a window of the chunk's size in every other layer,
+full attention in the rest, gated GELU, norms ahead of and behind the sub-blocks) and a dense DeepSeek-V2 (every layer latent attention with
+the same heads and latents, gated SiLU)."""
 from __future__ import annotations
 
 import gc
@@ -280,6 +284,141 @@ def sepirax_kernels(s: dict, iters: int) -> list[dict]:
         gemm("router logits", "sepirax, fp32 output", E, W, out_dtype=torch.float32)
         gemm("router logits", "deepseek", E, W)
     return rows
+
+
+LODEVIK_SIZES = {
+    # width, layers (differential and latent attention in turn), heads of both, differential attention (kv heads, dim, vdim, rot, chunk), latent
+    # attention (dim, rot, vdim, kv rank), feed-forward
+    "w2048": dict(width=2048, layers=12, heads=16, kv=4, dim=64, vdim=128, rot=32, chunk=1024, ldim=128, lrot=64, lvdim=128, lora=512, ff=6144),
+    "w4096": dict(width=4096, layers=8, heads=32, kv=8, dim=64, vdim=128, rot=64, chunk=4096, ldim=128, lrot=64, lvdim=128, lora=512, ff=12288),
+    "w2048s": dict(width=2048, layers=12, heads=32, kv=8, dim=32, vdim=64, rot=16, chunk=512, ldim=64, lrot=32, lvdim=64, lora=256, ff=6144),
+}
+
+
+def lodevik_config(s: dict) -> dict:
+    mlp = dict(kind="dense", ff=s["ff"])
+    dif = dict(type="attention", mlp=mlp, mixer=dict(heads=s["heads"], kv_heads=s["kv"], dim=s["dim"], vdim=s["vdim"], diff=0.4, scale=s["dim"] ** -0.5, softcap=30.0,
+               rot=dict(base=10000.0, dims=s["rot"]), mask=dict(size=s["chunk"])))
+    lat = dict(type="latent_attention", mlp=mlp, mixer=dict(heads=s["heads"], dim=s["ldim"], rot_dim=s["lrot"], vdim=s["lvdim"], kv_rank=s["lora"],
+               scale=(s["ldim"] + s["lrot"]) ** -0.5, rot=dict(base=500000.0, dims=s["lrot"])))
+    return dict(architecture="Lodevik", width=s["width"], vocab=VOCAB, norm=dict(eps=1e-5), logit_scale=0.5, layers=[dif, lat] * (s["layers"] // 2),
+                embedding=dict(scale=s["width"] ** 0.5, bigram=dict(buckets=65521, mul_prev=7919, mul_cur=104729)))
+
+
+def lodevik_like(s: dict, arch: str) -> dict:
+    cfg = dict(architectures=[arch], hidden_size=s["width"], num_hidden_layers=s["layers"], num_attention_heads=s["heads"], vocab_size=VOCAB,
+               max_position_embeddings=32768, rope_theta=10000.0, rms_norm_eps=1e-5, tie_word_embeddings=True, intermediate_size=s["ff"])
+    if arch.startswith("Deepseek"):
+        return dict(cfg, num_key_value_heads=s["heads"], kv_lora_rank=s["lora"], qk_nope_head_dim=s["ldim"], qk_rope_head_dim=s["lrot"], v_head_dim=s["lvdim"])
+    return dict(cfg, num_key_value_heads=s["kv"], head_dim=2 * s["dim"], query_pre_attn_scalar=2 * s["dim"], attn_logit_softcapping=30.0,
+                final_logit_softcapping=None, hidden_activation="gelu_pytorch_tanh", sliding_window=s["chunk"],
+                layer_types=["sliding_attention", "full_attention"] * (s["layers"] // 2))
+
+
+def lodevik_kernels(s: dict, iters: int) -> list[dict]:
+    """Each kernel of the design beside the like kernel of the closest models. Bytes and FLOPs are the algorithm's: visible pairs of queries and
+    keys, what a kernel must read and write once, and the products of latent attention in the form that needs fewest of them for its case."""
+    from onecat_vllm.ops import cuda as K
+    from onecat_vllm.ops.microbench import _peaks, timeit
+    pk, rows = _peaks(), []
+    W, H, G, D, V, c, L, R = s["width"], s["heads"], s["kv"], s["dim"], s["vdim"], s["chunk"], s["lora"], s["lrot"]
+    b = lambda *sh: torch.randn(*sh, device="cuda").bfloat16()
+    f32 = lambda *sh: torch.randn(*sh, device="cuda")
+
+    def row(kernel, case, who, fn, flops=0.0, nbytes=0.0):
+        ms = timeit(fn, iters)
+        t = max(flops / pk["bf16_tflops"] / 1e9, nbytes / pk["hbm_gbs"] / 1e6)
+        rows.append(dict(kernel=kernel, case=case, model=who, us=ms * 1e3, roofline_us=t * 1e3, frac_of_roofline=t / ms))
+
+    lam, sink, wide = torch.full((1,), 0.5, device="cuda"), f32(H), 2 * D
+    for case, n, q, S in (("prefill", 1, PREFILL, PREFILL), ("decode", DECODE_REQS, 1, DECODE_CTX)):
+        T = n * q
+        md, nblk = _meta(n, q, S)
+        cache = b(nblk, 2, G, 16, wide) * 0.5
+        near = lambda seen: (n * sum(seen(i) for i in range(S - q, S)), n * (seen(S - 1) if q == 1 else S))
+        qq, x, out = b(T, 2 * H, D), b(T, H, wide), torch.empty(T, H, wide, dtype=torch.bfloat16, device="cuda")
+        pairs, keys = near(lambda i: i % c + 1)
+        row("attention", case, "lodevik, chunks", lambda: K.diff_attention(qq, cache, md, D ** -0.5, lam, 0.6, 1e-5, V, 30.0, c), 4.0 * H * (D + V) * pairs,
+            2.0 * (keys * G * (wide + V) + T * H * (wide + V)))
+        pairs, keys = near(lambda i: min(i + 1, c))
+        row("attention", case, "gemma-2, window and soft cap", lambda: K.paged_attention(x, cache, md, wide ** -0.5, out=out, window=c, softcap=30.0),
+            4.0 * H * wide * pairs, 2.0 * (keys * G * 2 * wide + 2 * T * H * wide))
+        pairs, keys = near(lambda i: i + 1)
+        md.attn_plan = None
+        row("attention", case, "gemma-2, full with soft cap", lambda: K.paged_attention(x, cache, md, wide ** -0.5, out=out, softcap=30.0),
+            4.0 * H * wide * pairs, 2.0 * (keys * G * 2 * wide + 2 * T * H * wide))
+        del cache
+    lp, rp = K.mla_padded_sizes(L, R)
+    table = f32(2 * PREFILL, R)
+    for case, n, q, S in (("prefill", 1, PREFILL, PREFILL), ("decode", DECODE_REQS, 1, DECODE_CTX)):
+        md, nblk = _meta(n, q, S)
+        cache, T, pairs, gate = b(nblk, 16, lp + rp) * 0.3, n * q, n * sum(range(S - q + 1, S + 1)), b(n * q, H)
+        if case == "prefill":
+            wkv = b(H * (-(-s["ldim"] // 64) * 64 + -(-s["lvdim"] // 64) * 64), lp) * 0.05
+            md.positions = torch.arange(S, device="cuda", dtype=torch.int32)
+            plan = K.mla_prefill_plan(md, H, s["ldim"], R, s["lvdim"], lp, torch.device("cuda"))
+            qq, out = b(T, H, s["ldim"] + R), b(T, H, s["lvdim"])
+            fl, by = 2.0 * H * pairs * (s["ldim"] + R + s["lvdim"]), 2.0 * (S * (L + R) + T * H * (s["ldim"] + R + s["lvdim"]))
+            for who, rest in (("lodevik, two-term weights, sink and gate", (True, sink, gate)), ("deepseek", (False, None, None))):
+                row("latent attention", case, who, lambda: K.mla_prefill(plan, qq, cache, md, lambda x: K.gemm_bf16(x, wkv), out, s["ldim"], R, lp, 0.1, table,
+                                                                         True, *rest), fl, by)
+            continue
+        q_abs, q_pe = b(T, H, lp), b(T, H, R)
+        fl, by = 2.0 * H * pairs * (2 * L + R), 2.0 * (n * S * (L + R) + T * H * (2 * L + R))
+        for who, rest in (("lodevik, two-term weights, sink and gate", (True, 0, sink, gate)), ("deepseek", (False,))):
+            row("latent attention", case, who, lambda: K.mla_decode(q_abs, q_pe, cache, md, 0.1, lp, table, True, *rest), fl, by)
+        del cache
+    for T in (PREFILL, DECODE_REQS):
+        part, x32, w, res, y = b(T, W), f32(T, W), b(W), b(T, W), b(T, W)
+        row("norm", T, "lodevik join", lambda: K.stream_join(part, x32, (1, w, None, 1e-5, False), w, None, torch.bfloat16, copy_out=y), nbytes=12.0 * T * W)
+        row("norm", T, "add + rms norm", lambda: K.rms_norm(part, w, 1e-5, res, False), nbytes=8.0 * T * W)
+        ids, prev = (torch.randint(0, VOCAB, (T,), device="cuda", dtype=torch.int32) for _ in range(2))
+        emb, big = b(VOCAB, W), b(65522, W)
+        row("embedding", T, "lodevik, token and bigram rows", lambda: K.embed_stream(ids, emb, 3.0, prev, big, (7919, 104729), torch.bfloat16), nbytes=10.0 * T * W)
+        row("embedding", T, "gemma-2 (PyTorch)", lambda: torch.nn.functional.embedding(ids, emb) * 3.0, nbytes=4.0 * T * W)
+        slot = torch.arange(T, device="cuda", dtype=torch.int32)
+        kk, cc, cs, nw = b(T, H * wide + G * (wide + V)), b(T // 16 + 1, 2, G, 16, wide), torch.ones(T, s["rot"], device="cuda"), b(D)
+        row("norms + rope + insert", T, "lodevik", lambda: K.diff_prepare(kk, nw, nw, 1e-5, slot, cs, cc, slot, H, G, D, V, True), nbytes=4.0 * T * (H * wide + G * (wide + V)))
+        k2, cs2, nw2 = b(T, (H + 2 * G) * wide), torch.ones(T, wide, device="cuda"), b(wide)
+        row("norms + rope + insert", T, "qwen3", lambda: K.rope_and_cache(k2[:, : H * wide].view(T, H, wide), k2[:, H * wide: (H + G) * wide].view(T, G, wide),
+            k2[:, (H + G) * wide:].view(T, G, wide), slot, cs2, cc, slot, wide, nw2, nw2, 1e-5, False), nbytes=4.0 * T * (H + 2 * G) * wide)
+        n_in = H * (s["ldim"] + R) + L + R + H
+        down, lc, wk = b(T, -(-n_in // 8) * 8), b(T // 16 + 1, 16, lp + rp), b(L)
+        row("latent norm + rope + insert", T, "lodevik and deepseek", lambda: K.mla_prepare(None, down[:, H * (s["ldim"] + R): n_in - H], None, wk, 1e-5, slot, table, lc,
+                                                                                             slot, L, lp, True), nbytes=4.0 * T * (L + R))
+
+        def gemm(name, who, N, Kd, **kw):
+            wt, xx = (torch.randn(N, Kd, device="cuda") * 0.02).bfloat16(), b(T, Kd)
+            epi = kw.get("epi", K.EPI_STORE)
+            no = N if epi == K.EPI_STORE else N // 2
+            out = torch.empty(T, -(-no // 8) * 8, dtype=kw.get("out_dtype", torch.bfloat16), device="cuda")[:, :no]
+            row(f"gemm {name}", T, who, lambda: K._gemm(xx, wt, None, None, out, None, N, N, no, 0, epi, 1), flops=2.0 * T * N * Kd,
+                nbytes=2.0 * (N * Kd + T * Kd) + out.element_size() * T * no)
+        gemm("projections", "lodevik q|k|v", H * wide + G * (wide + V), W)
+        gemm("projections", "lodevik latent q|dkv|gate", n_in, W)
+        gemm("projections", "deepseek q", H * (s["ldim"] + R), W)
+        gemm("gate|up", "lodevik, GELU epilogue", 2 * s["ff"], W, epi=K.EPI_GELU_MUL)
+        gemm("gate|up", "SiLU epilogue", 2 * s["ff"], W, epi=K.EPI_SILU_MUL)
+    gemm("logits", "lodevik, fp32 output", VOCAB, W, out_dtype=torch.float32)
+    gemm("logits", "bf16 output", VOCAB, W)
+    return rows
+
+
+def run_lodevik(steps: int, warmup: int, sizes=None, kernels: bool = True, clock_sampler=None) -> None:
+    for name, s in LODEVIK_SIZES.items():
+        if sizes and name not in sizes:
+            continue
+        clocks = clock_sampler() if clock_sampler else None
+        models = {"Lodevik": lodevik_config(s), "Gemma-2": lodevik_like(s, "Gemma2ForCausalLM"), "DeepSeek-V2 (dense)": lodevik_like(s, "DeepseekV2ForCausalLM")}
+        res = {"design": "lodevik", "size": name, "dims": s, "dtype": "bf16", "data": "synthetic: random token ids and weights",
+               "workload": f"prefill: one {PREFILL}-token prompt a step; decode: {DECODE_REQS} requests at a context of about {DECODE_CTX}",
+               "l2": "model steps stream weights and caches larger than L2; kernels: L2 flushed before every launch",
+               "models": {k: model_throughput(m, steps, warmup) for k, m in models.items()}}
+        if kernels:
+            res["kernels"] = lodevik_kernels(s, max(5, steps // 6))
+        if clocks is not None:
+            res["clocks"] = clocks.stop()
+        print(json.dumps(res), flush=True)
 
 
 def run_sepirax(steps: int, warmup: int, sizes=None, kernels: bool = True, clock_sampler=None) -> None:
