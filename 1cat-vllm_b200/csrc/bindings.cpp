@@ -301,7 +301,7 @@ void paged_attention(torch::Tensor q, torch::Tensor kv_cache, torch::Tensor out,
 }
 
 // Differential attention: q [T, 2 H, D / 2] (head, map), cache rows of both maps' keys and of the values, out [T, H, vdim]. Modes as in
-// paged_attention without 2; mode 3 takes fp32, or bf16 rows of any width.
+// paged_attention (2: soft-capped scores, D = 64 or 128); mode 3 takes fp32, or bf16 rows of any width.
 void diff_attention(torch::Tensor q, torch::Tensor kv_cache, torch::Tensor out, torch::Tensor qsl, torch::Tensor seq_lens, torch::Tensor block_table,
                     double scale, int64_t mode, int64_t num_q_tiles, int64_t splits, int64_t max_q_len, int64_t short_q_len,
                     c10::optional<torch::Tensor> ws_o, c10::optional<torch::Tensor> ws_ml, double softcap, int64_t chunk, torch::Tensor lam,
@@ -334,8 +334,7 @@ void diff_attention(torch::Tensor q, torch::Tensor kv_cache, torch::Tensor out, 
     p.ws_o = ws_o->data_ptr<float>(); p.ws_ml = ws_ml->data_ptr<float>();
   }
   if (p.T == 0 || p.R == 0) return;
-  TORCH_CHECK(mode == 0 || mode == 1 || mode == 3, "mode must be 0, 1 or 3");
-  const int rc = mode == 3 ? oc::attention_f32_launch(p, et == torch::kBFloat16, cur_stream()) : oc::attention_launch(p, (int)mode, cur_stream());
+  const int rc = mode == 2 ? oc::diff_prefill_tc_launch(p, kv_cache.size(0), cur_stream()) : mode == 3 ? oc::attention_f32_launch(p, et == torch::kBFloat16, cur_stream()) : oc::attention_launch(p, (int)mode, cur_stream());
   TORCH_CHECK(rc == 0, "differential attention launch failed with code ", rc);
 }
 
@@ -1079,11 +1078,12 @@ void read_status_async(torch::Tensor pinned) {
   oc::moe_read_status_async(p + 8, st);
   oc::sampling_read_status_async(p + 9, st);
   oc::mla_prefill_read_status_async(p + 10, st);
+  oc::diff_prefill_read_status_async(p + 11, st);
 }
 
 int64_t read_status(bool clear) {
   return (int64_t)(oc::gemm_read_status(clear) | oc::elementwise_read_status(clear) | oc::attention_read_status(clear) | oc::attention_tc_read_status(clear) |
-                   oc::comm_read_status(clear) | oc::gdn_read_status(clear) | oc::sampling_read_status(clear) | oc::moe_read_status(clear) | oc::mla_read_status(clear) | oc::mla_prefill_read_status(clear) | oc::ep_read_status(clear));
+                   oc::comm_read_status(clear) | oc::gdn_read_status(clear) | oc::sampling_read_status(clear) | oc::moe_read_status(clear) | oc::mla_read_status(clear) | oc::mla_prefill_read_status(clear) | oc::diff_prefill_read_status(clear) | oc::ep_read_status(clear));
 }
 
 // ---- symmetric slab + peer-memory reductions
@@ -1169,6 +1169,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("kv_insert", &kv_insert);
   m.def("diff_attention", &diff_attention);
   m.def("diff_prepare", &diff_prepare);
+  m.def("diff_prefill_tc_sizes", [](int64_t D, double softcap) { return oc::diff_prefill_tc_sizes((int)D, (float)softcap); });
   m.def("embed_stream", &embed_stream);
   m.def("stream_join", &stream_join);
   m.def("gelu_tanh_f32", &gelu_tanh_f32);

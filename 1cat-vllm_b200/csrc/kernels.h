@@ -141,6 +141,12 @@ struct DiffPrepareParams {
   int T, H, G, dim, vdim, D, rot, bs, interleaved, f32;
 };
 int diff_prepare_launch(const DiffPrepareParams& p, cudaStream_t st);
+// tcgen05 prefill of differential attention (diff_prefill_tc.cu): requests with more than short_q_len new tokens, num_q_tiles counts their
+// 128-token tiles; q contiguous.
+bool diff_prefill_tc_sizes(int D, float softcap);
+int diff_prefill_tc_launch(const AttnParams& p, long long num_blocks, cudaStream_t st);
+unsigned int diff_prefill_read_status(bool clear);
+void diff_prefill_read_status_async(unsigned int* dst, cudaStream_t st);
 
 // tcgen05 prefill (attention_tc.cu): D == 128, 128-token query tiles; num_q_tiles counts those tiles.
 int attention_prefill_tc_launch(const AttnParams& p, long long num_blocks, cudaStream_t st);

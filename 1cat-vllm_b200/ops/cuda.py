@@ -593,9 +593,13 @@ def paged_attention(q, kv_cache, md, scale, out=None, lse=None, window=0, softca
     return out
 
 
+DIFF_PREFILL_MIN_LEN = 64          # a step with a portion of at least this many tokens runs its portions on tcgen05
+
+
 def diff_attention(q, kv_cache, md, scale, lam, out_scale, eps, vdim, softcap, chunk):
     """Both maps of a head are rows of one tile, so decoding and prefill each are one launch (and a combine where the context is split) that
-    ends with the difference and the head norm. Rows of the tensor-core kernels: 64, 128 or 256 wide; others, and fp32, run the plain kernel."""
+    ends with the difference and the head norm. Rows of the tensor-core kernels: 64, 128 or 256 wide; others, and fp32, run the plain kernel.
+    Prompts with soft-capped scores (rows of 64 or 128) run on tcgen05."""
     global _LAUNCHES
     T, rows, _ = q.shape
     G, D = kv_cache.shape[2], kv_cache.shape[4]
@@ -618,7 +622,11 @@ def diff_attention(q, kv_cache, md, scale, lam, out_scale, eps, vdim, softcap, c
             ws_o, ws_ml = (w.attn_static if getattr(md, "static_ws", False) else w.attn)(splits * T * rows * D, splits * T * rows * 2)
         _C.diff_attention(q, kv_cache, out, *common, 1, 0, splits, md.max_query_len, short, ws_o, ws_ml, softcap, chunk, lam, out_scale, eps)
         _LAUNCHES += 2 if splits > 1 else 1
-    if tiles:
+    if tiles and max(md.query_lens_cpu) >= DIFF_PREFILL_MIN_LEN and _C.diff_prefill_tc_sizes(D, softcap):
+        tiles = sum(-(-n // 128) for n in md.query_lens_cpu if n > short)
+        _C.diff_attention(q, kv_cache, out, *common, 2, tiles, 1, md.max_query_len, short, None, None, softcap, chunk, lam, out_scale, eps)
+        _LAUNCHES += 1
+    elif tiles:
         _C.diff_attention(q, kv_cache, out, *common, 0, tiles, 1, md.max_query_len, short, None, None, softcap, chunk, lam, out_scale, eps)
         _LAUNCHES += 1
     return out
