@@ -128,6 +128,55 @@ def test_one_key_stands_out_at_page_tile_and_chunk_edges(m, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("Hq,Hkv,D", [(4, 2, 64), (6, 1, 128), (3, 3, 256)])
+@pytest.mark.parametrize("cap,chunk,window", [(0.0, 100, 0), (3.0, 77, 0), (9.0, 200, 50)])
+def test_chunks_and_soft_cap_of_ordinary_attention(Hq, Hkv, D, cap, chunk, window, dtype):
+    """The chunk mask is an option of ordinary attention as well; with a window the nearer edge counts."""
+    from onecat_vllm.ops import cuda as K
+    g, bs = torch.Generator().manual_seed(D + chunk), 16
+    for lens in LENS[:3]:
+        bt, n = pages(lens, bs, D)
+        ks, vs = ([torch.randn(s, Hkv, D, generator=g).to(dtype) for _, s in lens] for _ in range(2))
+        cache = torch.full((n, 2, Hkv, bs, D), 3.0, dtype=dtype)
+        for r, (k, v) in enumerate(zip(ks, vs)):
+            pos = torch.arange(k.shape[0])
+            cache[bt[r].long()[pos // bs], :, :, pos % bs] = torch.stack([k, v], 1)
+        q = torch.randn(sum(a for a, _ in lens), Hq, D, generator=g).to(dtype)
+        got = K.paged_attention(q.to(DEV), cache.to(DEV), Meta(lens, bt.to(DEV)), 1.3 * D ** -0.5, chunk=chunk, softcap=cap, window=window).cpu().double()
+        o = 0
+        for (a, s), k, v in zip(lens, ks, vs):
+            i = torch.arange(s)
+            ok = O.sees(s, chunk) & (i.view(1, -1) > i.view(-1, 1) - window if window else torch.ones(s, s, dtype=torch.bool))
+            for h in range(Hq):
+                sc = (q[o:o + a, h].double() @ k[:, h * Hkv // Hq].double().T) * 1.3 * D ** -0.5
+                sc = cap * torch.tanh(sc / cap) if cap else sc
+                want = O.weights(sc.unsqueeze(0), ok[s - a:])[0] @ v[:, h * Hkv // Hq].double()
+                assert (got[o:o + a, h] - want).abs().max() < (0.02 if dtype == torch.bfloat16 else 3e-5), (a, s, h)
+            o += a
+
+
+def test_both_prefill_kernels_agree():
+    """The tcgen05 form (long portions) and the mma.sync form of one prompt: beyond the output's rounding they agree; scores well past the cap."""
+    from onecat_vllm.ops import cuda as K
+    g, bs, H, G, dim, U = torch.Generator().manual_seed(8), 32, 6, 2, 64, 128
+    lens = [(300, 700), (257, 257)]
+    bt, n = pages(lens, bs, 1)
+    ks, vs = [torch.randn(s, G, 2, dim, generator=g).bfloat16() for _, s in lens], [torch.randn(s, G, U, generator=g).bfloat16() for _, s in lens]
+    cache = diff_cache(ks, vs, bt, n, G, 128, torch.bfloat16, bs)
+    q = (torch.randn(557, 2 * H, dim, generator=g) * 4).bfloat16().to(DEV)
+    for cap, chunk in ((20.0, 200), (55.0, 0), (0.5, 64)):
+        outs = []
+        for least in (64, 10 ** 9):
+            old, K.DIFF_PREFILL_MIN_LEN = K.DIFF_PREFILL_MIN_LEN, least
+            try:
+                outs.append(K.diff_attention(q, cache, Meta(lens, bt.to(DEV)), 1.0, torch.tensor([0.5], device=DEV), 0.6, 1e-5, U, cap, chunk).float().cpu())
+            finally:
+                K.DIFF_PREFILL_MIN_LEN = old
+        assert K.check_status() == 0 and outs[0].isfinite().all()
+        assert (outs[0] - outs[1]).abs().mean() < 1e-3 and (outs[0] - outs[1]).abs().max() < 0.1
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("H,G,dim,vdim,rot,interleaved", [(4, 4, 24, 40, 8, True), (6, 2, 64, 128, 64, True), (3, 1, 9, 15, 4, True), (2, 2, 100, 256, 30, False),
                                                           (2, 1, 140, 300, 10, True), (5, 5, 33, 64, 0, True), (4, 2, 31, 40, 6, False)])
 def test_prepare_kernel(H, G, dim, vdim, rot, interleaved, dtype):
