@@ -20,7 +20,7 @@
 // unused rows 8..15 of the same operand and cost no extra product.
 // Chunks (EXT): a query sees the keys of its own chunk of the sequence; tiles before the chunk of a CTA's first row are skipped.
 // Differential attention (DIFF, an extended variant): a head has two maps over the same values. A cached key row holds both maps' keys side
-// by side and a query row belongs to one map. Prefill: warps 0 and 1 own the first map's rows, warps 2 and 3 the same rows of the
+// by side and a query row belongs to one map. (Prompts with soft-capped scores run diff_prefill_tc.cu instead.) Prefill: warps 0 and 1 own the first map's rows, warps 2 and 3 the same rows of the
 // second map, each multiplying its half of the key columns; the second map's output crosses over in shared memory. Decode: rows (head, map)
 // lie next to one another with zeros in the other map's half (the tile has rows to spare), and the merge of the warps or splits takes
 // the difference. Either way the difference, the head norm and the scale are part of the epilogue.
