@@ -198,6 +198,68 @@ def _lodevik_fields(hf: dict) -> dict:
                 intermediate_size=max(o["intermediate_size"] for o in over), layer_overrides=tuple(over), **top)
 
 
+def checkpoint_shapes(path: str) -> dict:
+    """Tensor name -> shape of a folder's safetensors files (headers only)."""
+    import glob
+
+    from safetensors import safe_open
+    out = {}
+    for f in sorted(glob.glob(os.path.join(path, "*.safetensors"))):
+        with safe_open(f, framework="pt", device="cpu") as sf:
+            out.update((k, tuple(sf.get_slice(k).get_shape())) for k in sf.keys())
+    return out
+
+
+def _nalasun_fields(hf: dict, shapes: Optional[dict] = None) -> dict:
+    """``ModelConfig`` fields of a Nalasun config.json: a list of layers, each with talking-heads attention (values are the unnormalised keys), a
+    delta rule with one decay per key channel or a Mamba-2 mixer, and an optional mixture of sigmoid-scored experts with a shared one; a short
+    convolution on every mixer's input, RMS norms ahead of the sub-blocks, an fp32 residual stream, learned positions, tied embeddings. The ranks
+    of the delta rule's decay and gate are those of a checkpoint's tensors (``shapes``); without one, the head sizes."""
+    shapes = shapes or {}
+    over, types = [], []
+    for i, l in enumerate(hf["layers"]):
+        m, mlp, kind = l["mixer"], l.get("mlp"), l["type"]
+        o: dict[str, Any] = dict(mixer_only_layers=mlp is None, num_attention_heads=int(m["heads"]))
+        if kind in ("attention", "channel_delta") and int(m["heads"]) % int(m["kv_heads"]):
+            raise ValueError(f"Nalasun layer {i}: {m['kv_heads']} key heads do not divide {m['heads']} heads")
+        if kind == "attention":
+            if int(m.get("vdim", m["dim"])) != int(m["dim"]):
+                raise ValueError(f"Nalasun layer {i}: the values are the keys, so vdim must equal dim")
+            t = m.get("q_temp")
+            o.update(num_key_value_heads=int(m["kv_heads"]), head_dim=int(m["dim"]), attn_scale=float(m["scale"]),
+                     attn_temperature=(float(t["coef"]), int(t["every"])) if t else None)
+            types.append("full_attention")
+        elif kind == "channel_delta":
+            o.update(num_key_value_heads=int(m["kv_heads"]), linear_num_key_heads=int(m["kv_heads"]), linear_num_value_heads=int(m["heads"]),
+                     linear_key_head_dim=int(m["dim"]), linear_value_head_dim=int(m["vdim"]), linear_conv_kernel_dim=int(m["conv"]),
+                     linear_decay_rank=shapes.get(f"l{i}.mix.a1", (int(m["dim"]),))[0], linear_gate_rank=shapes.get(f"l{i}.mix.g1", (int(m["vdim"]),))[0])
+            types.append("channel_delta")
+        elif kind == "mamba2":
+            if int(m["heads"]) % int(m["groups"]) or int(m["heads"]) * int(m["vdim"]) % int(m["norm_groups"]):
+                raise ValueError(f"Nalasun layer {i}: {m['groups']} groups and {m['norm_groups']} norm groups do not divide {m['heads']} heads of {m['vdim']}")
+            o.update(num_key_value_heads=int(m["heads"]), mamba_n_heads=int(m["heads"]), mamba_d_head=int(m["vdim"]), mamba_n_groups=int(m["groups"]),
+                     mamba_d_state=int(m["state"]), mamba_d_conv=int(m["conv"]), mamba_norm_groups=int(m["norm_groups"]))
+            types.append("mamba2")
+        else:
+            raise ValueError(f"Nalasun layer {i}: mixer {kind!r} is not known")
+        if mlp is not None:
+            if mlp.get("kind", "moe") != "moe":
+                raise ValueError(f"Nalasun layer {i}: feed-forward {mlp.get('kind')!r} is not known")
+            r = mlp["router"]
+            if int(r["top"]) > int(r["experts"]):
+                raise ValueError(f"Nalasun layer {i}: {r['experts']} experts cannot give each token {r['top']}")
+            o.update(num_experts=int(r["experts"]), num_experts_per_tok=int(r["top"]), routed_scaling_factor=float(r["scale"]),
+                     moe_intermediate_size=int(mlp["expert"]["ff"]), shared_expert_intermediate_size=int(mlp["shared"]["ff"]) if mlp.get("shared") else 0)
+        over.append(o)
+    first = next((o for o, t in zip(over, types) if t == "full_attention"), over[0])
+    top = {k: first[k] for k in ("num_attention_heads", "num_key_value_heads", "head_dim") if k in first}
+    return dict(architecture="Nalasun", vocab_size=int(hf["vocab"]), hidden_size=int(hf["width"]), num_hidden_layers=len(over),
+                rms_norm_eps=float(hf["norm"]["eps"]), residual_fp32=True, tie_word_embeddings=True, position_rows=int(hf["max_positions"]),
+                max_position_embeddings=int(hf["max_positions"]), input_conv=int(hf["canon"]["taps"]), layer_types=types, attn_kv_shared=True,
+                attn_talk=True, attn_log_bias=True, qk_norm_full=True, attention_bias=True, scoring_func="sigmoid", norm_topk_prob=False,
+                router_fp32=True, num_experts=max((o.get("num_experts", 0) for o in over), default=0), layer_overrides=tuple(over), **top)
+
+
 @dataclass
 class ModelConfig:
     """Architecture description, normalised from an HF ``config.json`` (or a dict for synthetic models).
@@ -268,6 +330,11 @@ class ModelConfig:
     rotary_dims: Optional[int] = None  # rotated dimensions of a head when they are given as a number instead of a fraction
     attn_window_keep: int = 0  # sliding-window layers: the first tokens of a sequence stay visible to every later position
     attn_kv_shared: bool = False  # the values are the projected keys: no value projection, one cached tensor per layer
+    attn_talk: bool = False  # the softmax weights of all heads are mixed by a learned matrix before they meet the values (talking heads)
+    attn_log_bias: bool = False  # r1 * ln(1 + r2 * distance) is taken off the scores, two learned numbers per head
+    attn_temperature: Optional[tuple] = None  # (coef, every): queries are multiplied by 1 + coef * ln(floor((position + 1) / every) + 1)
+    position_rows: int = 0  # > 0: a learned vector per position is added to the token embedding; the longest sequence has that many tokens
+    input_conv: int = 0  # > 0: taps of a causal convolution per channel that is added to what every mixer reads
     attn_head_gate: bool = False  # each head's output is multiplied by sigmoid(g_proj(x)) of that head before the output projection
     attn_rel_buckets: int = 0  # > 0: a learned bias per (distance bucket, head) is added to the scores; a checkpoint's table sets the row count
     attn_rel_max: int = 0  # distance at which the last bucket begins
@@ -277,7 +344,7 @@ class ModelConfig:
     loop: Optional[tuple] = None  # (start, stop, times): layers start..stop-1 run ``times`` times in a row with the same weights
     num_labels: int = 0  # > 0: a *ForSequenceClassification checkpoint (a ``score`` head on the pooled state instead of an LM head)
     # hybrid (Gated-DeltaNet)
-    layer_types: Optional[list[str]] = None  # "full_attention" | "linear_attention" (Gated-DeltaNet) | "mamba2" | "mamba1" | "short_conv" | "mlstm"
+    layer_types: Optional[list[str]] = None  # "full_attention" | "linear_attention" (Gated-DeltaNet) | "mamba2" | "mamba1" | "short_conv" | "mlstm" | "channel_delta"
     # Mamba-2 mixers (Bamba, Mamba2): heads x head size = inner width; B / C groups of the state size; conv kernel
     mamba_n_heads: int = 0
     mamba_d_head: int = 64
@@ -297,6 +364,8 @@ class ModelConfig:
     linear_key_head_dim: int = 128
     linear_value_head_dim: int = 128
     linear_conv_kernel_dim: int = 4
+    linear_decay_rank: int = 0  # channel_delta: widths of the low-rank projections to the decays and to the output gate
+    linear_gate_rank: int = 0
     # mLSTM mixers: matrix memory [key size, value size] per head, exponential gates whose logits are soft-capped
     mlstm_heads: int = 0
     mlstm_key_dim: int = 0
@@ -358,7 +427,8 @@ class ModelConfig:
     # ---- derived
     @property
     def is_hybrid(self) -> bool:
-        return bool(self.layer_types) and any(t in ("linear_attention", "mamba2", "mamba1", "short_conv", "mlstm") for t in self.layer_types)
+        return self.input_conv > 0 or bool(self.layer_types) and any(t in ("linear_attention", "mamba2", "mamba1", "short_conv", "mlstm", "channel_delta")
+                                                                    for t in self.layer_types)
 
     @property
     def is_moe(self) -> bool:
@@ -424,6 +494,8 @@ class ModelConfig:
             return cls(**{**_sepirax_fields(hf), **over})
         if hf.get("architecture") == "Lodevik" or "Lodevik" in (hf.get("architectures") or ()):
             return cls(**{**_lodevik_fields(hf), **over})
+        if hf.get("architecture") == "Nalasun" or "Nalasun" in (hf.get("architectures") or ()):
+            return cls(**{**_nalasun_fields(hf, checkpoint_shapes(over["model"]) if os.path.isdir(str(over.get("model"))) else None), **over})
         mm_ids = {m: int(hf[k]) for m, k in (("image", "image_token_id"), ("video", "video_token_id"), ("audio", "audio_token_id")) if hf.get(k) is not None}
         if mm_ids:
             over.setdefault("mm_token_ids", mm_ids)
@@ -1021,6 +1093,8 @@ class EngineArgs:
             elif mc.quant.method != self.quantization.replace("_marlin", ""):
                 raise ValueError(f"quantization={self.quantization} does not match the checkpoint's {mc.quant.method}")
         mc.max_model_len = self.max_model_len or min(mc.max_position_embeddings, 32768)
+        if mc.position_rows:   # there is no vector for later positions
+            mc.max_model_len = min(mc.max_model_len, mc.position_rows)
         if mc.index_topk and mc.max_model_len > mc.index_topk:
             # DeepSeek-V3.2 attends to the index_topk keys its lightning indexer selects; up to that many tokens this equals dense
             # attention, which is what runs here. Longer contexts would silently change the model's outputs, so they are refused.

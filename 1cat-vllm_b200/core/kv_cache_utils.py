@@ -127,13 +127,14 @@ class KVCacheSpec:
     dtype_bytes: int
     state_bytes: int = 0  # mamba: bytes of recurrent + conv state per sequence
     tensors: int = 2  # full: cached tensors per page, keys and values (1: the values are the keys)
+    token_bytes: int = 0  # full: bytes per token beside the pages (a factor of the token's scores)
 
     @property
     def page_size_bytes(self) -> int:
         if self.kind == "mamba":
             return self.state_bytes
         coef = 1 if self.kind == "mla" else self.tensors
-        return coef * self.block_size * self.num_kv_heads * self.head_size * self.dtype_bytes
+        return self.block_size * (coef * self.num_kv_heads * self.head_size * self.dtype_bytes + self.token_bytes)
 
 
 @dataclass

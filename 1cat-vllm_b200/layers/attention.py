@@ -157,6 +157,58 @@ class Attention(nn.Module):
         return self.o_proj(o.reshape(T, Hq * D))
 
 
+class TalkingAttention(nn.Module):
+    """Attention whose values are its unnormalised keys and whose heads' softmax weights are mixed by a learned matrix before they meet the values
+    (talking heads). Queries and keys are normalised over the whole projection, queries take a temperature that grows with the position, and
+    ``r1 ln(1 + r2 distance)`` is taken off the scores.
+
+    One cached row per token serves as key and value: the key norm's weight moves into the queries, its factor is one number per token that is
+    cached beside the pages and multiplies the scores. fused q|k GEMM -> norm, temperature and cache insert (one kernel) -> attention in two
+    passes (the mix needs normalised weights, so the first pass leaves every head's maximum and sum) -> output projection."""
+
+    kv_shared, token_scale, window, window_keep, bias_table = True, True, 0, 0, None   # what the runner and the graphs ask of an attention layer
+
+    def __init__(self, cfg: ModelConfig, layer_idx: int, prefix: str, device):
+        super().__init__()
+        if get_state().tp_size > 1:
+            raise ValueError("talking-heads attention (norms over the whole projection, weights mixed over all heads) is served with tensor_parallel_size=1")
+        if not (cfg.attn_kv_shared and cfg.qk_norm_full and cfg.attn_log_bias) or cfg.attn_softcap or cfg.attn_sinks or cfg.layer_window(layer_idx) or \
+                cfg.attn_chunk:
+            raise ValueError("talking-heads attention is served with shared keys and values, norms over the whole projection and the logarithmic "
+                             "distance bias, over the whole context")
+        self.Hq, self.Hkv, self.dim = cfg.num_attention_heads, cfg.num_key_value_heads, cfg.head_dim
+        self.qkg_proj = QKGParallelLinear(cfg.hidden_size, self.dim, self.Hq, self.Hkv, bias=cfg.attention_bias, quant=cfg.quant,
+                                          prefix=prefix + ".qkg_proj", dtype=cfg.dtype)
+        self.o_proj = RowParallelLinear(self.Hq * self.dim, cfg.hidden_size, bias=cfg.attn_o_bias, quant=cfg.quant, prefix=prefix + ".o_proj",
+                                        dtype=cfg.dtype)
+        ones = lambda n, dt: nn.Parameter(torch.ones(n, dtype=dt), requires_grad=False)
+        self.q_norm, self.k_norm = ones(self.Hq * self.dim, cfg.dtype), ones(self.Hkv * self.dim, cfg.dtype)
+        self.r1, self.r2 = ones(self.Hq, torch.float32), ones(self.Hq, torch.float32)
+        self.talk = nn.Parameter(torch.eye(self.Hq, dtype=cfg.dtype), requires_grad=False)
+        self.register_buffer("q_gain", torch.ones(self.Hq * self.dim, dtype=torch.float32), persistent=False)
+        self.register_buffer("bias", torch.zeros(2, self.Hq, dtype=torch.float32), persistent=False)
+        self.scale = cfg.attn_scale if cfg.attn_scale is not None else self.dim ** -0.5
+        self.temperature, self.eps = cfg.attn_temperature, cfg.rms_norm_eps
+        tc = torch.device(device).type == "cuda" and cfg.dtype == torch.bfloat16
+        self.D = ops.ext().talk_row(self.Hq, self.Hkv, self.dim) if tc else self.dim   # width of a cached row
+        self.layer_idx = layer_idx
+
+    def load_weight(self, pname: str, w: torch.Tensor, shard_id=None) -> None:
+        getattr(self, pname).data.copy_(w)
+
+    def process_weights_after_loading(self) -> None:
+        k = self.k_norm.data.float().view(self.Hkv, 1, self.dim).expand(-1, self.Hq // self.Hkv, -1).reshape(-1)
+        self.q_gain.copy_(self.q_norm.data.float() * k * self.scale)
+        self.bias.copy_(torch.stack([self.r1.data, self.r2.data]))
+
+    def forward(self, x: torch.Tensor, md, kv_cache) -> torch.Tensor:
+        pages, k_scale = kv_cache
+        q = ops.talk_prepare(self.qkg_proj(x), self.q_gain, self.eps, self.temperature, md.positions, pages, k_scale, md.slot_mapping, self.Hq, self.Hkv,
+                             self.dim)
+        o = ops.talk_attention(q, pages, k_scale, md, self.bias, self.talk)
+        return self.o_proj(o.reshape(x.shape[0], self.Hq * self.dim))
+
+
 class DifferentialAttention(nn.Module):
     """Two attention maps per head over the same values: ``o = rms(a1 - lam a2) * (1 - diff)`` with a1, a2 the maps' outputs and one learned
     ``lam`` per layer. Queries and keys are laid out head by head as (map 1, map 2), each map normalised and rotated by itself; scores may be

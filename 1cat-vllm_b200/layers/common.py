@@ -161,6 +161,17 @@ class BigramEmbedding(nn.Module):
         self.weight.data.copy_(w)
 
 
+class PositionEmbedding(nn.Module):
+    """A learned row per position, added to the token embedding where an fp32 residual stream starts; every TP rank holds all of it."""
+
+    def __init__(self, rows: int, hidden: int, dtype=torch.float32):
+        super().__init__()
+        self.weight = nn.Parameter(torch.zeros(rows, hidden, dtype=dtype), requires_grad=False)
+
+    def load_weight(self, pname, w, shard_id=None):
+        self.weight.data.copy_(w)
+
+
 class ParallelLMHead(VocabParallelEmbedding):
     """Vocab-sharded output projection; ``compute_logits`` gathers the shards."""
 

@@ -5,17 +5,16 @@ x → in_proj → [z | xBC | dt];  xBC → depthwise causal conv (bias, SiLU) wi
 dt = softplus(dt + dt_bias) clamped to the time-step limits, A = -exp(A_log);  h_t = exp(dt A) h_{t-1} + dt x ⊗ B,
 y = h C + D x;  y → RMSNorm(y * SiLU(z)) over groups of the inner width → out_proj.
 
-The convolution and the scan run as PyTorch operations on every device (the chunked form of ``ops.ref.mamba2_scan``); there is no
-CUDA kernel for this mixer, and it is served with tensor_parallel_size = 1 and without speculative decoding."""
+Convolution, recurrence and gated norm are kernels on a GPU (``ops.causal_conv``, ``ops.mamba2``, ``ops.gated_norm``); the mixer is served with
+tensor_parallel_size = 1 and without speculative decoding."""
 from __future__ import annotations
 
 import torch
 import torch.nn as nn
-import torch.nn.functional as F
 
+from onecat_vllm import ops
 from onecat_vllm.config import ModelConfig
 from onecat_vllm.layers.linear import ReplicatedLinear
-from onecat_vllm.ops import ref
 from onecat_vllm.parallel.state import get_state
 
 
@@ -48,29 +47,16 @@ class Mamba2Mixer(nn.Module):
         p = getattr(self, pname)
         p.data.copy_(w.reshape(p.shape).to(p.dtype))
 
-    def state_shapes(self):
-        return (self.conv_dim, self.kw - 1), (self.H, self.P, self.N)
+    def state_tensors(self):
+        return [(ops.conv_state_shape(self.conv_dim, self.kw), None), ((self.H, self.N, self.P), torch.float32)]
 
     def forward(self, x: torch.Tensor, md, state) -> torch.Tensor:
-        """``state`` = (conv_state [slots, conv_dim, kw-1], ssm_state fp32 [slots, H, P, N])."""
+        """``state`` = (convolution inputs [slots, kw-1, conv_dim], S fp32 [slots, H, N, P])."""
         if getattr(md, "gdn_record", None) is not None:
             raise ValueError("speculative decoding is not served for Mamba-2 layers (their states are not recorded per token)")
         conv_state, ssm_state = state
-        T = x.shape[0]
         zxbcdt = self.in_proj(x)
-        z, xbc, dt = zxbcdt[:, : self.d_inner], zxbcdt[:, self.d_inner: self.d_inner + self.conv_dim], zxbcdt[:, self.d_inner + self.conv_dim:]
-        xbc = ref.causal_conv1d(xbc.contiguous(), self.conv_weight, self.conv_bias, conv_state, md.query_start_loc, md.state_slots,
-                                md.has_initial_state)
-        xs = xbc[:, : self.d_inner].reshape(T, self.H, self.P)
-        B = xbc[:, self.d_inner: self.d_inner + self.G * self.N].reshape(T, self.G, self.N)
-        C = xbc[:, self.d_inner + self.G * self.N:].reshape(T, self.G, self.N)
-        dt = F.softplus(dt.float() + self.dt_bias)
-        if self.dt_limit[0] > 0.0 or self.dt_limit[1] != float("inf"):
-            dt = dt.clamp(self.dt_limit[0], self.dt_limit[1])
-        y = ref.mamba2_scan(xs, dt, -torch.exp(self.A_log), B, C, self.D, ssm_state, md.query_start_loc, md.state_slots, md.has_initial_state)
-        y = y.reshape(T, self.d_inner) * F.silu(z.float())
-        g = self.norm_groups
-        yg = y.view(T, g, self.d_inner // g)
-        y = (yg * torch.rsqrt(yg.pow(2).mean(-1, keepdim=True) + self.eps)).view(T, self.d_inner)
-        y = (y.to(x.dtype) * self.norm_weight)
-        return self.out_proj(y)
+        n, c = self.d_inner, self.conv_dim
+        xbc = ops.causal_conv(zxbcdt[:, n: n + c], self.conv_weight, self.conv_bias, conv_state, md, silu=True)
+        y = ops.mamba2(xbc, zxbcdt[:, n + c:], self.A_log, self.dt_bias, self.D, ssm_state, md, self.H, self.G, self.N, self.P, self.dt_limit)
+        return self.out_proj(ops.gated_norm(y, zxbcdt[:, :n], self.norm_weight, self.eps, self.norm_groups, gate_first=True))

@@ -9,10 +9,38 @@ from __future__ import annotations
 import torch
 import torch.nn as nn
 
+from onecat_vllm import ops
 from onecat_vllm.config import ModelConfig
 from onecat_vllm.layers.linear import ReplicatedLinear
 from onecat_vllm.ops import ref
 from onecat_vllm.parallel.state import get_state
+
+
+class InputConv(nn.Module):
+    """``h + conv(h)`` ahead of a mixer: a causal convolution over time on every channel, no activation. It owns a state slot of its own (the last
+    ``taps - 1`` inputs), beside the state or the pages of the mixer behind it."""
+
+    kind = "linear_attention"   # a state-slot owner for the runner
+
+    def __init__(self, hidden: int, taps: int, dtype):
+        super().__init__()
+        self.H, self.taps = hidden, taps
+        self.weight = nn.Parameter(torch.zeros(hidden, taps, dtype=dtype), requires_grad=False)
+
+    @property
+    def linear_attn(self):
+        return self
+
+    def load_weight(self, pname: str, w: torch.Tensor, shard=None) -> None:
+        self.weight.data.copy_(w.reshape(self.weight.shape))
+
+    def state_tensors(self):
+        return [(ops.conv_state_shape(self.H, self.taps), None)]
+
+    def forward(self, x: torch.Tensor, md, state) -> torch.Tensor:
+        if getattr(md, "gdn_record", None) is not None:
+            raise ValueError("speculative decoding is not served for input convolutions (their state is not recorded per token)")
+        return ops.causal_conv(x, self.weight, None, state[0], md, silu=False, residual=True)
 
 
 class ShortConv(nn.Module):

@@ -128,6 +128,35 @@ def lodevik_name(name: str) -> str:
     return f"model.layers.{m.group(1)}.{ours}" if ours else name
 
 
+# Nalasun checkpoints: ``l<i>.<name>``; the mixer's names depend on its kind
+_NALASUN_LAYER = {"norm1": "input_layernorm.weight", "norm2": "post_attention_layernorm.weight", "canon1": "input_conv.weight",
+                  "mlp.router": "mlp.gate.weight", **{f"mlp.shared.{n}": f"mlp.shared_expert.{n}_proj.weight" for n in ("gate", "up", "down")}}
+_NALASUN_MIX = {"full_attention": {"q": "self_attn.q_proj.weight", "k": "self_attn.k_proj.weight", "q.b": "self_attn.q_proj.bias",
+                                   "k.b": "self_attn.k_proj.bias", "q.norm": "self_attn.q_norm", "k.norm": "self_attn.k_norm", "r1": "self_attn.r1",
+                                   "r2": "self_attn.r2", "talk": "self_attn.talk", "o": "self_attn.o_proj.weight"},
+                "channel_delta": {**{n: f"linear_attn.in_proj_{n}.weight" for n in ("q", "k", "v", "b", "a1", "g1")},
+                                  **{f"{n}.conv": f"linear_attn.conv_{n}" for n in "qkv"}, "a2": "linear_attn.a_proj.weight",
+                                  "g2": "linear_attn.g_proj.weight", "A_log": "linear_attn.A_log", "dt_bias": "linear_attn.dt_bias",
+                                  "norm": "linear_attn.norm_weight", "o": "linear_attn.out_proj.weight"},
+                "mamba2": {"in": "linear_attn.in_proj.weight", "conv": "linear_attn.conv_weight", "conv.b": "linear_attn.conv_bias",
+                           "dt_bias": "linear_attn.dt_bias", "A_log": "linear_attn.A_log", "D": "linear_attn.D", "norm": "linear_attn.norm_weight",
+                           "o": "linear_attn.out_proj.weight"}}
+_NALASUN_TOP = {"embed": "model.embed_tokens.weight", "pos": "model.positions.weight", "final.norm": "model.norm.weight"}
+
+
+def nalasun_name(name: str, mixer_kind) -> str:
+    """Module parameter that a Nalasun checkpoint tensor belongs to (unknown names come back unchanged). ``mixer_kind(i)``: the layer's type."""
+    m = re.match(r"l(\d+)\.(.+)$", name)
+    if m is None:
+        return _NALASUN_TOP.get(name, name)
+    base, rest = f"model.layers.{m.group(1)}.", m.group(2)
+    e = _SEPIRAX_EXPERT_RE.match(rest)
+    if e:
+        return f"{base}mlp.experts.{e.group(1)}.{e.group(2)}_proj.weight"
+    ours = _NALASUN_MIX[mixer_kind(int(m.group(1)))].get(rest[len("mix."):]) if rest.startswith("mix.") else _NALASUN_LAYER.get(rest)
+    return base + ours if ours else name
+
+
 _EXPERT_RE = re.compile(r"(.*\.mlp)\.experts\.(\d+)\.(gate_proj|up_proj|down_proj)\.(weight|weight_scale_inv|weight_scale|bias)$")
 
 
@@ -145,6 +174,7 @@ def load_weights(model: nn.Module, weights: Iterable[tuple[str, torch.Tensor]]) 
     gabisun = cfg is not None and cfg.architecture == "Gabisun"
     sepirax = cfg is not None and cfg.architecture == "Sepirax"
     lodevik = cfg is not None and cfg.architecture == "Lodevik"
+    nalasun = cfg is not None and cfg.architecture == "Nalasun"
     loaded = set()
     for name, w in weights:
         if gabisun:
@@ -153,6 +183,8 @@ def load_weights(model: nn.Module, weights: Iterable[tuple[str, torch.Tensor]]) 
             name = sepirax_name(name, lambda i: "mlstm" if cfg.layer_type(i) == "mlstm" else "mla")
         elif lodevik:
             name = lodevik_name(name)
+        elif nalasun:
+            name = nalasun_name(name, cfg.layer_type)
         if name.startswith("language_model."):
             name = name[len("language_model."):]
         elif name.startswith("model.language_model."):  # text tower of a multimodal checkpoint (Qwen3.5)
@@ -324,7 +356,7 @@ def dummy_init(model: nn.Module, seed: int = 0, std: float = 0.02) -> None:
     for name, p in model.named_parameters():
         g = gen(p.device)
         leaf = name.rsplit(".", 1)[-1]
-        if leaf in ("weight",) and name.endswith(("layernorm.weight", "norm.weight")) or leaf in ("q_norm", "k_norm", "norm_weight", "attn_layer_scale", "mlp_layer_scale", "alpha"):
+        if leaf in ("weight",) and name.endswith(("layernorm.weight", "norm.weight")) or leaf in ("q_norm", "k_norm", "norm_weight", "attn_layer_scale", "mlp_layer_scale", "alpha", "talk", "r1", "r2"):
             continue  # keep constructor init (1, or 0 for Gemma-style)
         if p.dtype in (torch.float32, torch.float16, torch.bfloat16):
             if leaf in ("scales",):

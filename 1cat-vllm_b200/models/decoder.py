@@ -15,8 +15,8 @@ import torch.nn as nn
 
 from onecat_vllm import ops
 from onecat_vllm.config import ModelConfig
-from onecat_vllm.layers.attention import Attention, DifferentialAttention
-from onecat_vllm.layers.common import BigramEmbedding, ParallelLMHead, RMSNorm, VocabParallelEmbedding, make_norm
+from onecat_vllm.layers.attention import Attention, DifferentialAttention, TalkingAttention
+from onecat_vllm.layers.common import BigramEmbedding, ParallelLMHead, PositionEmbedding, RMSNorm, VocabParallelEmbedding, make_norm
 from onecat_vllm.layers.gdn import GatedDeltaNet
 from onecat_vllm.layers.linear import ReplicatedLinear
 from onecat_vllm.layers.mla import MLAAttention
@@ -48,11 +48,16 @@ class DecoderLayer(nn.Module):
             from onecat_vllm.layers.mlstm import MLSTM
             self.linear_attn = layer_class("MLSTM", MLSTM)(cfg, idx, prefix + ".linear_attn")
             self.kind = "linear_attention"   # a state-slot layer for the runner and the scheduler
-        elif self.kind in ("mamba2", "mamba1", "short_conv", "ffn"):
+        elif self.kind in ("channel_delta", "mamba2"):
+            if self.kind == "mamba2":
+                from onecat_vllm.layers.mamba2 import Mamba2Mixer as Mixer
+            else:
+                from onecat_vllm.layers.channel_delta import ChannelDelta as Mixer
+            self.linear_attn = Mixer(cfg, idx, prefix + ".linear_attn")
+            self.kind = "linear_attention"
+        elif self.kind in ("mamba1", "short_conv", "ffn"):
             if self.kind == "ffn":
                 from onecat_vllm.layers.mlp import FeedForwardBlock as Mixer
-            elif self.kind == "mamba2":
-                from onecat_vllm.layers.mamba2 import Mamba2Mixer as Mixer
             elif self.kind == "mamba1":
                 from onecat_vllm.layers.mamba1 import Mamba1Mixer as Mixer
             else:
@@ -60,10 +65,16 @@ class DecoderLayer(nn.Module):
             self.linear_attn = Mixer(cfg, idx, prefix + ".linear_attn")
             self.kind = "linear_attention"   # a state-slot layer like Gated-DeltaNet for the runner and the scheduler
             self.graph_safe = False          # its convolution and scan read batch geometry on the host
+        elif cfg.attn_talk:
+            self.self_attn = layer_class("TalkingAttention", TalkingAttention)(cfg, idx, prefix + ".self_attn", device)
         elif cfg.attn_diff is not None:
             self.self_attn = layer_class("DifferentialAttention", DifferentialAttention)(cfg, idx, prefix + ".self_attn", device)
         else:
             self.self_attn = layer_class("Attention", Attention)(cfg, idx, prefix + ".self_attn", device)
+        self.input_conv = None
+        if cfg.input_conv:
+            from onecat_vllm.layers.short_conv import InputConv
+            self.input_conv = InputConv(cfg.hidden_size, cfg.input_conv, cfg.dtype)
         if cfg.layer_scale:
             scale = lambda: nn.Parameter(torch.ones(cfg.hidden_size, dtype=cfg.dtype), requires_grad=False)
             self.attn_layer_scale, self.mlp_layer_scale = scale(), None if cfg.mixer_only_layers else scale()
@@ -117,11 +128,12 @@ class DecoderModel(nn.Module):
         self.norm = make_norm(cfg) if self.last_stage else PPMissingLayer()
         if cfg.residual_fp32 and (self.start != 0 or not self.last_stage):
             raise ValueError("models with an fp32 residual stream are served without pipeline parallelism")
-        if (cfg.layer_scale or cfg.loop is not None or cfg.bigram) and not cfg.residual_fp32 or \
+        if (cfg.layer_scale or cfg.loop is not None or cfg.bigram or cfg.position_rows or cfg.input_conv) and not cfg.residual_fp32 or \
                 cfg.residual_fp32 and (cfg.parallel_block or not cfg.pre_norm and (cfg.loop is not None or not cfg.sandwich_norm)):
             raise ValueError("the fp32 residual stream is served for blocks with norms ahead of, behind or on both sides of the sub-blocks; looped "
-                             "layers, layer scales and bigram embeddings need it")
+                             "layers, layer scales, bigram and position embeddings and input convolutions need it")
         self.bigram = BigramEmbedding(*cfg.bigram, cfg.hidden_size, cfg.dtype) if cfg.bigram else None
+        self.positions = PositionEmbedding(cfg.position_rows, cfg.hidden_size, cfg.dtype) if cfg.position_rows else None
         if cfg.loop is not None:
             # ahead of every pass of the looped layers the stream x becomes loop_in([x ; x0]) + loop_step[pass], x0 being the embeddings
             self.loop_in = ReplicatedLinear(2 * cfg.hidden_size, cfg.hidden_size, quant=None, prefix="model.loop_in", dtype=cfg.dtype,
@@ -150,10 +162,16 @@ class DecoderModel(nn.Module):
 
     def cache_layers(self):
         """(name, layer) of everything on this stage that owns a cache or a state, in execution order: the layers, with one entry per
-        pass for looped ones (every pass has its own K/V). KV caches are indexed in this order."""
-        if self.cfg.loop is None:
-            return [(f"layers.{i}", layer) for i, layer in self.local_layers()]
-        return [(f"layers.{i}" if t < 0 else f"layers.{i}.{t}", self.layers[i]) for i, t in self.cfg.layer_runs()]
+        pass for looped ones (every pass has its own K/V); a layer's input convolution comes ahead of its mixer. KV caches are indexed in this
+        order."""
+        runs = [(i, -1) for i, _ in self.local_layers()] if self.cfg.loop is None else self.cfg.layer_runs()
+        out = []
+        for i, t in runs:
+            name, layer = f"layers.{i}" if t < 0 else f"layers.{i}.{t}", self.layers[i]
+            if layer.input_conv is not None:
+                out.append((name + ".input_conv", layer.input_conv))
+            out.append((name, layer))
+        return out
 
     def forward(self, input_ids: torch.Tensor, md, caches: list, inputs_embeds: Optional[torch.Tensor] = None,
                 return_prenorm: bool = False, intermediate: Optional[tuple] = None):
@@ -163,6 +181,13 @@ class DecoderModel(nn.Module):
         layers = self.layers
         cfg = self.cfg
         if intermediate is None:
+            if self.positions is not None:   # prompts given as vectors take the positions' rows as well
+                given = inputs_embeds is not None
+                e = self.embed_tokens
+                whole = not given and e.tp == 1
+                table = inputs_embeds.to(cfg.dtype).contiguous() if given else e.weight if whole else e(input_ids)
+                x, _ = ops.embed_stream(input_ids, table, cfg.embed_scale, gathered=not whole, rows=self.positions.weight, positions=md.positions)
+                return self._forward_stream(x, md, caches, return_prenorm)
             if inputs_embeds is None and self.bigram is not None:
                 x, y = self._embed_stream(input_ids, md.prev_ids)
                 return self._forward_stream(y, md, caches, return_prenorm, stream=x)
@@ -229,15 +254,16 @@ class DecoderModel(nn.Module):
         cfg = self.cfg
         runs, loop, mult = cfg.layer_runs(), cfg.loop, cfg.residual_multiplier
         T, H = h.shape
+        caches = iter(caches)
         both = None
         if loop is not None:
-            both = torch.empty(T, 2 * H, dtype=h.dtype, device=h.device)   # [stream ; embeddings]
+            both = torch.empty(T, 2 * H, dtype=cfg.dtype, device=h.device)   # [stream ; embeddings]
             both[:, H:] = h
 
         def plain_join(part, x, post, scale, mul):
             """Join without a norm behind it: the next sub-block reads the stream itself, rounded to the model's type."""
-            y = torch.empty(T, H, dtype=h.dtype, device=h.device) if h.dtype != torch.float32 else None
-            _, x = ops.stream_join(part, x, post, scale, None, out_dtype=h.dtype, copy_out=y, mul=mul)
+            y = torch.empty(T, H, dtype=cfg.dtype, device=h.device) if cfg.dtype != torch.float32 else None
+            _, x = ops.stream_join(part, x, post, scale, None, out_dtype=cfg.dtype, copy_out=y, mul=mul)
             return (x if y is None else y), x
 
         def join(part, x, post, scale, at, mul):
@@ -247,17 +273,19 @@ class DecoderModel(nn.Module):
                 return plain_join(part, x, post, scale, mul)
             if at < len(runs) and loop is not None and runs[at][0] == loop[0] and runs[at][1] >= 0:
                 ops.stream_join(part, x, post, scale, None, copy_out=both[:, :H], mul=mul)
-                return ops.stream_join(self.loop_in(both), None, None, None, self.layers[loop[0]].input_layernorm, out_dtype=h.dtype,
+                return ops.stream_join(self.loop_in(both), None, None, None, self.layers[loop[0]].input_layernorm, out_dtype=cfg.dtype,
                                        add=self.loop_step[runs[at][1]])
             return ops.stream_join(part, x, post, scale, self.layers[runs[at][0]].input_layernorm if at < len(runs) else self.norm,
-                                   out_dtype=h.dtype, mul=mul)
+                                   out_dtype=cfg.dtype, mul=mul)
 
         y, x = (h, stream) if stream is not None and not cfg.pre_norm else join(h if stream is None else stream, None, None, None, 0, embed_scale)
         for r, (i, _) in enumerate(runs):
             layer = self.layers[i]
             post1 = layer.post_attention_layernorm if cfg.sandwich_norm else None
             scale1, scale2 = (layer.attn_layer_scale, layer.mlp_layer_scale) if cfg.layer_scale else (None, None)
-            part = layer.mixer(y, md, caches[r])
+            if layer.input_conv is not None:
+                y = layer.input_conv(y, md, next(caches))
+            part = layer.mixer(y, md, next(caches))
             if layer.mlp is None:
                 y, x = join(part, x, post1, scale1, r + 1, mult)
                 continue
@@ -265,7 +293,7 @@ class DecoderModel(nn.Module):
                 y, x = plain_join(reduce_only(part), x, post1, scale1, mult)
             else:
                 y, x = ops.stream_join(reduce_only(part), x, post1, scale1,
-                                       layer.pre_feedforward_layernorm if cfg.sandwich_norm else layer.post_attention_layernorm, out_dtype=h.dtype,
+                                       layer.pre_feedforward_layernorm if cfg.sandwich_norm else layer.post_attention_layernorm, out_dtype=cfg.dtype,
                                        mul=mult)
             y, x = join(layer.mlp(y), x, layer.post_feedforward_layernorm if cfg.sandwich_norm else None, scale2, r + 1, mult)
         return (y, x) if return_prenorm else y
@@ -317,6 +345,7 @@ class CausalLM(nn.Module):
         (".gate_up_proj", ".gate_proj", 0), (".gate_up_proj", ".up_proj", 1),
         (".in_proj_dqkvg", ".dq_proj", 0), (".in_proj_dqkvg", ".q_proj", 0), (".in_proj_dqkvg", ".dkv_proj", 1), (".in_proj_dqkvg", ".g_proj", 2),
         (".in_proj_qkvg", ".in_proj_q", 0), (".in_proj_qkvg", ".in_proj_k", 1), (".in_proj_qkvg", ".in_proj_v", 2), (".in_proj_qkvg", ".in_proj_g", 3),
+        *((".in_proj", f".in_proj_{n}", i) for i, n in enumerate(("q", "k", "v", "a1", "g1", "b"))),
         (".gate_if", ".gate_i", 0), (".gate_if", ".gate_f", 1),
         (".in_proj_qkvz", ".in_proj_q", 0), (".in_proj_qkvz", ".in_proj_k", 1), (".in_proj_qkvz", ".in_proj_v", 2),
         (".in_proj_qkvz", ".in_proj_z", 3), (".in_proj_ba", ".in_proj_b", 0), (".in_proj_ba", ".in_proj_a", 1),

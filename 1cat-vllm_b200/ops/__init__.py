@@ -85,11 +85,11 @@ def sigmoid_mul(x, gate):
     return (x.float() * torch.sigmoid(gate.float())).to(x.dtype)
 
 
-def embed_stream(ids, table, scale, prev=None, bigram=None, muls=(0, 0), out_dtype=None, gathered=False):
-    """Scaled token embeddings plus hashed-bigram rows as the start of an fp32 residual stream; returns (stream, stream in ``out_dtype``).
+def embed_stream(ids, table, scale, prev=None, bigram=None, muls=(0, 0), out_dtype=None, gathered=False, rows=None, positions=None):
+    """Scaled token embeddings plus hashed-bigram rows or learned position rows as the start of an fp32 residual stream; returns (stream, stream in ``out_dtype``).
     See ``ref.embed_stream``."""
     f = ext().embed_stream if table.is_cuda else ref.embed_stream
-    return f(ids, table, scale, prev, bigram, muls, out_dtype or table.dtype, gathered)
+    return f(ids, table, scale, prev, bigram, muls, out_dtype or table.dtype, gathered, rows, positions)
 
 
 def diff_prepare(qkv, q_norm, k_norm, eps, positions, cos_sin, kv_cache, slot_mapping, heads, kv_heads, dim, vdim, interleaved=True):
@@ -105,6 +105,47 @@ def diff_attention(q, kv_cache, md, scale, lam, out_scale, eps, vdim, softcap=0.
     if q.is_cuda:
         return ext().diff_attention(q, kv_cache, md, scale, lam, out_scale, eps, vdim, softcap, chunk)
     return ref.diff_attention(q, kv_cache, md.block_table, md.query_start_loc, md.seq_lens, scale, lam, out_scale, eps, vdim, softcap, chunk)
+
+
+def talk_prepare(qk, q_gain, eps, temperature, positions, pages, k_scale, slot_mapping, heads, kv_heads, dim):
+    """Norm and temperature of talking-heads attention's queries, cache insert of its keys in one kernel; returns the queries. See
+    ``ref.talk_prepare``."""
+    f = ext().talk_prepare if qk.is_cuda else ref.talk_prepare
+    return f(qk, q_gain, eps, temperature, positions, pages, k_scale, slot_mapping, heads, kv_heads, dim)
+
+
+def talk_attention(q, pages, k_scale, md, bias, mix):
+    """Talking-heads attention of the step ``md``; see ``ref.talk_attention``."""
+    if q.is_cuda:
+        return ext().talk_attention(q, pages, k_scale, md, bias, mix)
+    return ref.talk_attention(q, pages, k_scale, md.block_table, md.query_start_loc, md.seq_lens, bias, mix)
+
+
+conv_state_shape = ref.conv_state_shape   # one slot of ``causal_conv``'s state
+
+
+def causal_conv(x, weight, bias, state, md, silu=False, residual=False):
+    """Causal convolution per channel over the step's portions with a rolling state; see ``ref.causal_conv``."""
+    f = ext().causal_conv if x.is_cuda else ref.causal_conv
+    return f(x, weight, bias, state, md, silu, residual)
+
+
+def channel_delta(qkv, a, b, A_log, dt_bias, state, md, Hk, H, D, V):
+    """Gated delta rule with one decay per key channel; see ``ref.channel_delta``."""
+    f = ext().channel_delta if qkv.is_cuda else ref.channel_delta
+    return f(qkv, a, b, A_log, dt_bias, state, md, Hk, H, D, V)
+
+
+def mamba2(xbc, dt, A_log, dt_bias, D, state, md, H, G, N, V, dt_limit=(0.0, float("inf"))):
+    """Mamba-2 state space; see ``ref.mamba2``."""
+    f = ext().mamba2 if xbc.is_cuda else ref.mamba2
+    return f(xbc, dt, A_log, dt_bias, D, state, md, H, G, N, V, dt_limit)
+
+
+def gated_norm(x, gate, w, eps, groups, gate_first):
+    """RMS norm in equal parts with a gate ahead of it (SiLU) or behind it (sigmoid); see ``ref.gated_norm``."""
+    f = ext().gated_norm if x.is_cuda else ref.gated_norm
+    return f(x, gate, w, eps, groups, gate_first)
 
 
 def mlstm(qkvg, gates, i_bias, f_bias, norm_w, eps, cap, H, D, V, state, md):

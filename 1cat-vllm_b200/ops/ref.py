@@ -291,6 +291,48 @@ def paged_attention(q, kv_cache, block_table, query_start_loc, seq_lens, scale: 
     return (o, lse) if return_lse else o
 
 
+def talk_prepare(qk, q_gain, eps: float, temperature, positions, pages, k_scale, slot_mapping, heads: int, kv_heads: int, dim: int):
+    """Between the projections and talking-heads attention: ``qk`` ``[T, heads dim | kv_heads dim]``. Queries are RMS-normalised over the whole row,
+    multiplied by ``q_gain`` fp32 ``[heads dim]`` (norm weights of queries and keys and the score's scale) and by the temperature ``(coef, every)``
+    of their position. Keys are cached as projected (they are the values) in ``pages`` ``[blocks, 1, kv_heads, bs, dim]``, their rows' RMS factor
+    beside them in ``k_scale`` fp32 ``[blocks, bs]``. Returns the queries ``[T, heads, dim]``."""
+    T, bs = qk.shape[0], pages.shape[3]
+    q, k = qk[:, : heads * dim].float(), qk[:, heads * dim:]
+    q = q * torch.rsqrt(q.pow(2).mean(-1, keepdim=True) + eps) * q_gain
+    if temperature is not None:
+        coef, every = temperature
+        steps = torch.div(positions.long() + 1, every, rounding_mode="floor").float()
+        q = q * (1.0 + coef * torch.log(steps + 1.0)).unsqueeze(-1)
+    kv_insert(k.reshape(T, kv_heads, dim), pages, slot_mapping)
+    ok = slot_mapping >= 0
+    sm = slot_mapping[ok].long()
+    k_scale[sm // bs, sm % bs] = torch.rsqrt(k.float().pow(2).mean(-1) + eps)[ok]
+    return q.view(T, heads, dim).to(qk.dtype)
+
+
+def talk_attention(q, pages, k_scale, block_table, query_start_loc, seq_lens, bias, mix):
+    """Talking-heads attention over keys that are the values: scores ``(q . k) * k_scale - r1 ln(1 + r2 distance)`` (``bias`` fp32 ``[2, heads]``),
+    softmax per head, weights of all heads mixed by ``mix`` ``[heads, heads]`` (to, from), each head's mixed weights applied to its own key head.
+    q ``[T, heads, dim]`` -> ``[T, heads, dim]``."""
+    T, H, D = q.shape
+    G, bs = pages.shape[2], pages.shape[3]
+    out = torch.empty_like(q)
+    qsl, sl = query_start_loc.tolist(), seq_lens.tolist()
+    for r, S in enumerate(sl):
+        a, n = qsl[r], qsl[r + 1] - qsl[r]
+        if n == 0:
+            continue
+        blocks = block_table[r, : -(-S // bs)].long()
+        k = pages[blocks, 0].float().permute(1, 0, 2, 3).reshape(G, -1, D)[:, :S].repeat_interleave(H // G, dim=0)
+        s = torch.einsum("qhd,hkd->hqk", q[a:a + n].float(), k) * k_scale[blocks].reshape(-1)[:S]
+        dist = torch.arange(S - n, S, device=q.device).view(-1, 1) - torch.arange(S, device=q.device).view(1, -1)
+        s = s - bias[0].view(H, 1, 1) * torch.log(1.0 + bias[1].view(H, 1, 1) * dist.clamp(min=0))
+        p = torch.softmax(s.masked_fill(dist < 0, -float("inf")), -1)
+        p = torch.einsum("hg,gqk->hqk", mix.float(), p)
+        out[a:a + n] = torch.einsum("hqk,hkd->qhd", p, k).to(q.dtype)
+    return out
+
+
 def diff_prepare(qkv, q_norm, k_norm, eps: float, positions, cos_sin, kv_cache, slot_mapping, heads: int, kv_heads: int, dim: int, vdim: int,
                  interleaved: bool):
     """Between the projections and differential attention: ``qkv`` ``[T, 2 heads dim + 2 kv_heads dim + kv_heads vdim]``, queries and keys head
@@ -325,14 +367,16 @@ def diff_attention(q, kv_cache, block_table, query_start_loc, seq_lens, scale: f
     return (o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * out_scale).to(q.dtype)
 
 
-def embed_stream(ids, table, scale: float, prev=None, bigram=None, muls=(0, 0), out_dtype=None, gathered: bool = False):
+def embed_stream(ids, table, scale: float, prev=None, bigram=None, muls=(0, 0), out_dtype=None, gathered: bool = False, rows=None, positions=None):
     """Start of an fp32 residual stream: ``table[id] * scale``, plus the row of ``bigram`` (last row: no previous token) that (previous token,
-    token) hash to. ``prev`` < 0: none. ``gathered``: ``table`` holds the tokens' own rows. Returns (the stream, the stream in ``out_dtype``)."""
+    token) hash to. ``prev`` < 0: none. ``rows``: a learned vector per position. ``gathered``: ``table`` holds the tokens' own rows. Returns (the stream, the stream in ``out_dtype``)."""
     x = (table if gathered else F.embedding(ids.long(), table)).float() * scale
     if bigram is not None:
         n = bigram.shape[0] - 1
         row = torch.where(prev < 0, n, (prev.long() * muls[0] + ids.long() * muls[1]) % n)
         x = x + F.embedding(row, bigram).float()
+    if rows is not None:
+        x = x + F.embedding(positions.long(), rows).float()
     return x, x.to(out_dtype)
 
 
@@ -543,7 +587,7 @@ def gated_delta_rule(q, k, v, g, beta, state, query_start_loc, state_slots, has_
                      use_qk_l2norm: bool = True, token_states: Optional[torch.Tensor] = None):
     """Sequential gated delta rule, fp32 state ``[slots, Hv, K, V]`` updated in place:
     ``S <- e^g S + k (x) ((v - (e^g S)^T k) beta)``, ``o = S^T q * scale``. q,k ``[T,Hk,K]``, v ``[T,Hv,V]``,
-    g,beta ``[T,Hv]``. This token-by-token form is the oracle for both the chunked prefill and the
+    beta ``[T,Hv]``, g ``[T,Hv]`` or one decay per key channel ``[T,Hv,K]``. This token-by-token form is the oracle for both the chunked prefill and the
     recurrent decode kernels."""
     T, Hk, K = q.shape
     Hv, V = v.shape[1], v.shape[2]
@@ -563,7 +607,7 @@ def gated_delta_rule(q, k, v, g, beta, state, query_start_loc, state_slots, has_
         slot = int(state_slots[r])
         S = state[slot].float().clone() if bool(has_initial_state[r]) else torch.zeros(Hv, K, V, device=v.device)
         for t in range(a, b):
-            S = S * torch.exp(g[t].float()).view(Hv, 1, 1)
+            S = S * torch.exp(g[t].float()).view(Hv, -1, 1)
             kv = torch.einsum("hk,hkv->hv", kf[t], S)
             delta = (v[t].float() - kv) * beta[t].float().view(Hv, 1)
             S = S + torch.einsum("hk,hv->hkv", kf[t], delta)
@@ -573,6 +617,68 @@ def gated_delta_rule(q, k, v, g, beta, state, query_start_loc, state_slots, has_
         if token_states is None or (b - a) > token_states.shape[1]:
             state[slot] = S.to(state.dtype)
     return out
+
+
+# ----------------------------------------------------------------------------- short convolutions, matrix-state recurrences
+def conv_state_shape(channels: int, taps: int) -> tuple:
+    return max(taps - 1, 1), channels
+
+
+def causal_conv(x, weight, bias, state, md, silu: bool = False, residual: bool = False):
+    """Causal convolution over time per channel, ``weight`` ``[C, taps]`` (last tap: the current token), over a variable-length batch; SiLU or
+    ``x +`` on top. ``state`` ``[slots, taps - 1, C]`` holds the inputs ahead of each portion and is updated in place."""
+    T, C = x.shape
+    m = weight.shape[1] - 1
+    out = torch.empty(T, C, dtype=x.dtype, device=x.device)
+    qsl = md.query_start_loc.tolist()
+    for r in range(len(qsl) - 1):
+        a, b = qsl[r], qsl[r + 1]
+        if a == b:
+            continue
+        s = int(md.state_slots[r])
+        prev = state[s, :m].float() if bool(md.has_initial_state[r]) else torch.zeros(m, C, device=x.device)
+        seq = torch.cat([prev, x[a:b].float()])
+        y = (seq.unfold(0, m + 1, 1) * weight.float()).sum(-1)
+        if bias is not None:
+            y = y + bias.float()
+        y = F.silu(y) if silu else y
+        out[a:b] = (x[a:b].float() + y if residual else y).to(x.dtype)
+        if m:
+            state[s, :m] = seq[-m:].to(state.dtype)
+    return out
+
+
+def channel_delta(qkv, a, b, A_log, dt_bias, state, md, Hk: int, H: int, D: int, V: int):
+    """Gated delta rule with one decay per (head, key channel). ``qkv`` ``[T, Hk D | Hk D | H V]`` after the short convolutions, ``a`` ``[T, H D]``
+    decay logits, ``b`` ``[T, H]`` step logits, ``state`` fp32 ``[slots, H, D, V]``. Returns ``[T, H V]``."""
+    T = qkv.shape[0]
+    q, k, v = qkv.split([Hk * D, Hk * D, H * V], -1)
+    g = -torch.exp(A_log.float()).view(1, H, 1) * F.softplus(a.float() + dt_bias.float()).view(T, H, D)
+    o = gated_delta_rule(q.reshape(T, Hk, D), k.reshape(T, Hk, D), v.reshape(T, H, V), g, torch.sigmoid(b.float()), state, md.query_start_loc,
+                         md.state_slots, md.has_initial_state)
+    return o.reshape(T, H * V)
+
+
+def mamba2(xbc, dt, A_log, dt_bias, D, state, md, H: int, G: int, N: int, V: int, dt_limit=(0.0, float("inf"))):
+    """Mamba-2 state space of a step: ``xbc`` ``[T, H V | G N | G N]`` after the convolution, ``dt`` ``[T, H]`` step logits, ``state`` fp32
+    ``[slots, H, N, V]``. Returns ``[T, H V]``, the skip ``D x`` included."""
+    T = xbc.shape[0]
+    x, B, C = xbc.split([H * V, G * N, G * N], -1)
+    step = F.softplus(dt.float() + dt_bias.float()).clamp(dt_limit[0], dt_limit[1])
+    y = mamba2_scan(x.reshape(T, H, V), step, -torch.exp(A_log.float()), B.reshape(T, G, N), C.reshape(T, G, N), D, state.transpose(2, 3),
+                    md.query_start_loc, md.state_slots, md.has_initial_state)
+    return y.reshape(T, H * V).to(xbc.dtype)
+
+
+def gated_norm(x, gate, w, eps: float, groups: int, gate_first: bool):
+    """RMS norm of ``x`` ``[T, n]`` in ``groups`` equal parts with a gate: ``norm(x * silu(gate)) * w`` (``gate_first``) or
+    ``norm(x) * w * sigmoid(gate)``. ``w``: ``[n]``, or one part's, shared by all."""
+    T, n = x.shape
+    v = x.float() * F.silu(gate.float()) if gate_first else x.float()
+    v = v.reshape(T, groups, n // groups)
+    v = v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps) * w.float().view(-1, n // groups)
+    v = v.reshape(T, n)
+    return (v if gate_first else v * torch.sigmoid(gate.float())).to(x.dtype)
 
 
 # ----------------------------------------------------------------------------- mLSTM

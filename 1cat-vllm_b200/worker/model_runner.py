@@ -196,7 +196,8 @@ class ModelRunner:
                 specs[name] = KVCacheSpec("mla", self.block_size, 1, layer.self_attn.cache_width, esz)
             else:
                 a = layer.self_attn
-                specs[name] = KVCacheSpec("full", self.block_size, a.Hkv, a.D, asz, tensors=1 if a.kv_shared else 2)
+                specs[name] = KVCacheSpec("full", self.block_size, a.Hkv, a.D, asz, tensors=1 if a.kv_shared else 2,
+                                          token_bytes=4 if getattr(a, "token_scale", False) else 0)
         for i, layer in (self.draft.model.local_layers() if self.draft is not None else ()):
             specs[f"draft.{i}"] = KVCacheSpec("full", self.block_size, layer.self_attn.Hkv, self.draft.cfg.head_dim, asz)
         if self.mtp is not None:
@@ -240,7 +241,8 @@ class ModelRunner:
                 return None
             if spec.kind == "mla":
                 return torch.zeros(nb, bs, spec.head_size, dtype=dt, device=dev)
-            return torch.zeros(nb, spec.tensors, spec.num_kv_heads, bs, spec.head_size, dtype=self._attn_kv_dtype(), device=dev)
+            pages = torch.zeros(nb, spec.tensors, spec.num_kv_heads, bs, spec.head_size, dtype=self._attn_kv_dtype(), device=dev)
+            return (pages, torch.zeros(nb, bs, dtype=torch.float32, device=dev)) if spec.token_bytes else pages
 
         self.kv_caches = []
         for name, layer in self.model.model.cache_layers():
