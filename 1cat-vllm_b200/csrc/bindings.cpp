@@ -364,7 +364,8 @@ torch::Tensor diff_prepare(torch::Tensor qkv, torch::Tensor q_w, torch::Tensor k
 
 // x fp32 [T, H] (and y of the table's type, when given) from token and bigram embeddings; see EmbedParams.
 void embed_stream(torch::Tensor ids, torch::Tensor table, double scale, c10::optional<torch::Tensor> prev, c10::optional<torch::Tensor> bigram,
-                  int64_t mul_prev, int64_t mul_cur, torch::Tensor x, c10::optional<torch::Tensor> y, bool gathered) {
+                  int64_t mul_prev, int64_t mul_cur, torch::Tensor x, c10::optional<torch::Tensor> y, bool gathered,
+                  c10::optional<torch::Tensor> rows, c10::optional<torch::Tensor> positions) {
   const auto et = table.scalar_type();
   TORCH_CHECK(table.is_cuda() && (et == torch::kBFloat16 || et == torch::kFloat32) && table.dim() == 2 && table.is_contiguous(), "the table must be a contiguous bf16 or fp32 matrix");
   TORCH_CHECK(ids.is_cuda() && ids.scalar_type() == torch::kInt32 && ids.is_contiguous(), "ids must be int32 [T]");
@@ -382,6 +383,11 @@ void embed_stream(torch::Tensor ids, torch::Tensor table, double scale, c10::opt
     TORCH_CHECK(prev.has_value() && prev->scalar_type() == torch::kInt32 && prev->is_contiguous() && prev->numel() >= T, "prev must be int32 [T]");
     p.bigram = bigram->data_ptr(); p.prev = prev->data_ptr<int>(); p.buckets = (int)bigram->size(0) - 1;
     p.mul_prev = (int)mul_prev; p.mul_cur = (int)mul_cur;
+  }
+  if (rows.has_value()) {
+    TORCH_CHECK(rows->scalar_type() == et && rows->is_contiguous() && rows->dim() == 2 && rows->size(1) == H, "position rows must be [rows, H]");
+    TORCH_CHECK(positions.has_value() && positions->scalar_type() == torch::kInt32 && positions->is_contiguous() && positions->numel() >= T, "positions must be int32 [T]");
+    p.rows = rows->data_ptr(); p.positions = positions->data_ptr<int>(); p.num_rows = (int)rows->size(0);
   }
   const c10::cuda::CUDAGuard guard(table.device());
   TORCH_CHECK(oc::embed_stream_launch(p, cur_stream()) == 0, "embed_stream failed");
@@ -1051,6 +1057,130 @@ torch::Tensor mlstm(torch::Tensor x, torch::Tensor gates, torch::Tensor i_bias, 
 }
 bool mlstm_chunkable(int64_t D, int64_t V) { return oc::mlstm_chunkable((int)D, (int)V); }
 
+static void check_step(const torch::Tensor& qsl, const torch::Tensor& slots, const torch::Tensor& has_init) {
+  for (auto* t : {&qsl, &slots, &has_init}) TORCH_CHECK(t->is_cuda() && t->scalar_type() == torch::kInt32 && t->is_contiguous(), "step metadata must be int32");
+  TORCH_CHECK(qsl.numel() == slots.numel() + 1 && has_init.numel() >= slots.numel(), "step metadata sizes");
+}
+
+torch::Tensor causal_conv(torch::Tensor x, torch::Tensor w, c10::optional<torch::Tensor> bias, torch::Tensor state, torch::Tensor qsl, torch::Tensor slots,
+                          torch::Tensor has_init, bool silu, bool residual) {
+  const auto et = x.scalar_type();
+  TORCH_CHECK(x.is_cuda() && (et == torch::kBFloat16 || et == torch::kFloat32) && x.dim() == 2 && x.stride(1) == 1, "x must be [T, C] with unit inner stride");
+  const int64_t T = x.size(0), C = x.size(1);
+  TORCH_CHECK(w.scalar_type() == et && w.is_contiguous() && w.dim() == 2 && w.size(0) == C, "weights must be [C, taps]");
+  const int64_t taps = w.size(1);
+  TORCH_CHECK(state.scalar_type() == et && state.is_contiguous() && state.dim() == 3 && state.size(1) == std::max<int64_t>(taps - 1, 1) && state.size(2) == C, "state must be [slots, taps - 1, C]");
+  if (bias.has_value()) TORCH_CHECK(bias->scalar_type() == et && bias->is_contiguous() && bias->numel() == C, "bias must be [C]");
+  check_step(qsl, slots, has_init);
+  const c10::cuda::CUDAGuard guard(x.device());
+  auto y = torch::empty({T, C}, x.options());
+  oc::CausalConvParams p{};
+  p.x = x.data_ptr(); p.ldx = x.stride(0); p.w = w.data_ptr(); p.bias = bias.has_value() ? bias->data_ptr() : nullptr;
+  p.y = y.data_ptr(); p.state = state.data_ptr();
+  p.query_start_loc = qsl.data_ptr<int>(); p.state_slots = slots.data_ptr<int>(); p.has_initial_state = has_init.data_ptr<int>();
+  p.T = (int)T; p.R = (int)slots.numel(); p.C = (int)C; p.taps = (int)taps; p.silu = silu; p.residual = residual; p.f32 = et == torch::kFloat32;
+  const int rc = oc::causal_conv_launch(p, cur_stream());
+  TORCH_CHECK(rc == 0, "causal_conv failed: ", rc, " (up to 16 taps)");
+  return y;
+}
+
+// q | k | v (channel delta) or x | B | C (Mamba-2, a absent) side by side in `x`.
+torch::Tensor recurrence(torch::Tensor x, c10::optional<torch::Tensor> a, torch::Tensor b, torch::Tensor A_log, torch::Tensor dt_bias,
+                         c10::optional<torch::Tensor> skip, torch::Tensor state, torch::Tensor qsl, torch::Tensor slots, torch::Tensor has_init, int64_t Hk, int64_t H,
+                         int64_t D, int64_t V, double dt_min, double dt_max, int64_t skip_min_len, c10::optional<torch::Tensor> out_) {
+  const auto et = x.scalar_type();
+  const bool delta = a.has_value();
+  TORCH_CHECK(x.is_cuda() && (et == torch::kBFloat16 || et == torch::kFloat32) && x.dim() == 2 && x.stride(1) == 1 && x.size(1) == 2 * Hk * D + H * V, "inputs must be [T, 2 Hk D + H V]");
+  const int64_t T = x.size(0);
+  TORCH_CHECK(b.scalar_type() == et && b.dim() == 2 && b.size(0) == T && b.size(1) == H && b.stride(1) == 1, "step logits must be [T, H]");
+  for (auto* t : {&state, &A_log, &dt_bias}) TORCH_CHECK(t->is_cuda() && t->scalar_type() == torch::kFloat32 && t->is_contiguous(), "states, A_log and dt_bias must be contiguous fp32");
+  TORCH_CHECK(state.dim() == 4 && state.size(1) == H && state.size(2) == D && state.size(3) == V && A_log.numel() == H && dt_bias.numel() == (delta ? H * D : H), "state shapes");
+  if (delta) { TORCH_CHECK(a->scalar_type() == torch::kFloat32 && a->dim() == 2 && a->size(0) == T && a->size(1) == H * D && a->stride(1) == 1, "decay logits must be fp32 [T, H D]"); }
+  else { TORCH_CHECK(skip.has_value() && skip->scalar_type() == torch::kFloat32 && skip->is_contiguous() && skip->numel() == H, "skip must be fp32 [H]"); }
+  check_step(qsl, slots, has_init);
+  const c10::cuda::CUDAGuard guard(x.device());
+  auto out = out_.has_value() ? *out_ : torch::empty({T, H * V}, x.options());
+  TORCH_CHECK(out.scalar_type() == et && out.is_contiguous() && out.numel() == T * H * V, "out must be [T, H V]");
+  oc::RecurrenceParams p{};
+  const char* base = (const char*)x.data_ptr();
+  const int64_t es = x.element_size();
+  if (delta) { p.q = base; p.k = base + Hk * D * es; p.v = base + 2 * Hk * D * es; }
+  else { p.v = base; p.k = base + H * V * es; p.q = base + (H * V + Hk * D) * es; }
+  p.ld = x.stride(0);
+  if (delta) { p.a = a->data_ptr<float>(); p.ld_a = a->stride(0); }
+  else p.skip = skip->data_ptr<float>();
+  p.b = b.data_ptr(); p.ld_b = b.stride(0); p.A_log = A_log.data_ptr<float>(); p.dt_bias = dt_bias.data_ptr<float>();
+  p.dt_min = (float)dt_min; p.dt_max = (float)dt_max; p.scale = 1.f / std::sqrt((float)D);
+  p.state = state.data_ptr<float>(); p.out = out.data_ptr();
+  p.query_start_loc = qsl.data_ptr<int>(); p.state_slots = slots.data_ptr<int>(); p.has_initial_state = has_init.data_ptr<int>();
+  p.T = (int)T; p.R = (int)slots.numel(); p.Hk = (int)Hk; p.H = (int)H; p.D = (int)D; p.V = (int)V; p.delta = delta; p.f32 = et == torch::kFloat32;
+  p.skip_min_len = (int)skip_min_len;
+  const int rc = oc::recurrence_launch(p, cur_stream());
+  TORCH_CHECK(rc == 0, "recurrence failed: ", rc, " (key sizes up to 256)");
+  return out;
+}
+
+torch::Tensor gated_norm(torch::Tensor x, torch::Tensor gate, torch::Tensor w, double eps, int64_t groups, bool gate_first) {
+  const auto et = x.scalar_type();
+  TORCH_CHECK(x.is_cuda() && (et == torch::kBFloat16 || et == torch::kFloat32) && x.dim() == 2 && x.stride(1) == 1, "x must be [T, n] with unit inner stride");
+  TORCH_CHECK(gate.scalar_type() == et && gate.sizes() == x.sizes() && gate.stride(1) == 1, "the gate must match x");
+  TORCH_CHECK(w.scalar_type() == et && w.is_contiguous() && groups > 0 && x.size(1) % groups == 0 && (w.numel() == x.size(1) || w.numel() * groups == x.size(1)), "norm weight");
+  const c10::cuda::CUDAGuard guard(x.device());
+  auto y = torch::empty({x.size(0), x.size(1)}, x.options());
+  oc::GatedNormParams p{};
+  p.x = x.data_ptr(); p.gate = gate.data_ptr(); p.w = w.data_ptr(); p.ld_x = x.stride(0); p.ld_g = gate.stride(0); p.y = y.data_ptr(); p.eps = (float)eps;
+  p.T = (int)x.size(0); p.n = (int)x.size(1); p.groups = (int)groups; p.w_shared = w.numel() != x.size(1); p.gate_first = gate_first; p.f32 = et == torch::kFloat32;
+  TORCH_CHECK(oc::gated_norm_launch(p, cur_stream()) == 0, "gated_norm failed");
+  return y;
+}
+
+torch::Tensor talk_prepare(torch::Tensor qk, torch::Tensor gain, double eps, double coef, int64_t every, torch::Tensor positions, torch::Tensor pages,
+                           torch::Tensor k_scale, torch::Tensor slots, int64_t H, int64_t G, int64_t dim, int64_t group_rows) {
+  const auto et = qk.scalar_type();
+  TORCH_CHECK(qk.is_cuda() && (et == torch::kBFloat16 || et == torch::kFloat32) && qk.dim() == 2 && qk.stride(1) == 1 && qk.size(1) == (H + G) * dim, "q|k must be [T, (H + G) dim]");
+  const int64_t T = qk.size(0), row = pages.size(4), bs = pages.size(3);
+  TORCH_CHECK(pages.scalar_type() == et && pages.is_contiguous() && pages.dim() == 5 && pages.size(1) == 1 && pages.size(2) == G && row >= dim, "pages must be [blocks, 1, G, bs, row]");
+  TORCH_CHECK(k_scale.scalar_type() == torch::kFloat32 && k_scale.is_contiguous() && k_scale.numel() == pages.size(0) * bs, "key factors must be fp32 [blocks, bs]");
+  TORCH_CHECK(gain.scalar_type() == torch::kFloat32 && gain.is_contiguous() && gain.numel() == H * dim && group_rows * G >= H, "gain must be fp32 [H dim]");
+  for (auto* t : {&positions, &slots}) TORCH_CHECK(t->scalar_type() == torch::kInt32 && t->is_contiguous() && t->numel() >= T, "positions and slots must be int32 [T]");
+  const c10::cuda::CUDAGuard guard(qk.device());
+  auto q = torch::empty({T, G * group_rows, row}, qk.options());
+  oc::TalkPrepareParams p{};
+  p.qk = qk.data_ptr(); p.ld = qk.stride(0); p.gain = gain.data_ptr<float>(); p.eps = (float)eps; p.coef = (float)coef; p.every = (int)every;
+  p.positions = positions.data_ptr<int>(); p.slots = slots.data_ptr<int>(); p.q_out = q.data_ptr(); p.pages = pages.data_ptr(); p.k_scale = k_scale.data_ptr<float>();
+  p.T = (int)T; p.H = (int)H; p.G = (int)G; p.dim = (int)dim; p.group_rows = (int)group_rows; p.row = (int)row; p.bs = (int)bs; p.f32 = et == torch::kFloat32;
+  TORCH_CHECK(oc::talk_prepare_launch(p, cur_stream()) == 0, "talk_prepare failed");
+  return q;
+}
+
+static oc::TalkParams talk_params(const torch::Tensor& q, const torch::Tensor& pages, const torch::Tensor& k_scale, const torch::Tensor& bias, const torch::Tensor& mix,
+                                  const torch::Tensor& out, const torch::Tensor& qsl, const torch::Tensor& seq_lens, const torch::Tensor& bt, int64_t H, int64_t dim) {
+  const auto et = q.scalar_type();
+  const int64_t G = pages.size(2), row = pages.size(4);
+  TORCH_CHECK(q.is_cuda() && q.is_contiguous() && q.dim() == 3 && q.size(2) == row && q.size(1) % G == 0 && q.size(1) >= H && H % G == 0, "q must be [T, G group_rows, row]");
+  TORCH_CHECK(pages.scalar_type() == et && pages.is_contiguous() && pages.dim() == 5 && pages.size(1) == 1, "pages must be [blocks, 1, G, bs, row]");
+  TORCH_CHECK(k_scale.scalar_type() == torch::kFloat32 && k_scale.is_contiguous() && bias.scalar_type() == torch::kFloat32 && bias.is_contiguous() && bias.numel() == 2 * H, "key factors and bias must be fp32");
+  TORCH_CHECK(mix.scalar_type() == et && mix.is_contiguous() && mix.numel() == H * H, "mix must be [H, H]");
+  TORCH_CHECK(out.scalar_type() == et && out.is_contiguous() && out.numel() == q.size(0) * H * dim, "out must be [T, H, dim]");
+  TORCH_CHECK(qsl.scalar_type() == torch::kInt32 && seq_lens.scalar_type() == torch::kInt32 && bt.scalar_type() == torch::kInt32 && bt.stride(1) == 1 &&
+              bt.size(0) >= seq_lens.numel() && qsl.numel() == seq_lens.numel() + 1, "step metadata must be int32");
+  oc::TalkParams p{};
+  p.q = q.data_ptr(); p.pages = pages.data_ptr(); p.mix = mix.data_ptr(); p.k_scale = k_scale.data_ptr<float>(); p.bias = bias.data_ptr<float>();
+  p.out = out.data_ptr(); p.query_start_loc = qsl.data_ptr<int>(); p.seq_lens = seq_lens.data_ptr<int>(); p.block_table = bt.data_ptr<int>();
+  p.bt_stride = (int)bt.stride(0); p.T = (int)q.size(0); p.R = (int)seq_lens.numel(); p.H = (int)H; p.G = (int)G; p.dim = (int)dim;
+  p.group_rows = (int)(q.size(1) / G); p.row = (int)row; p.bs = (int)pages.size(3); p.f32 = et == torch::kFloat32;
+  return p;
+}
+
+void talk_plain(torch::Tensor q, torch::Tensor pages, torch::Tensor k_scale, torch::Tensor bias, torch::Tensor mix, torch::Tensor out, torch::Tensor qsl,
+                torch::Tensor seq_lens, torch::Tensor bt, int64_t H, int64_t dim) {
+  auto p = talk_params(q, pages, k_scale, bias, mix, out, qsl, seq_lens, bt, H, dim);
+  TORCH_CHECK(p.row == p.dim && p.group_rows * p.G == p.H, "the plain kernel takes unpadded rows");
+  const c10::cuda::CUDAGuard guard(q.device());
+  const int rc = oc::talk_plain_launch(p, cur_stream());
+  TORCH_CHECK(rc == 0, "talk_plain failed: ", rc);
+}
+
 torch::Tensor sigmoid_mul(torch::Tensor x, torch::Tensor gate) {
   TORCH_CHECK(x.is_cuda() && (x.scalar_type() == torch::kBFloat16 || x.scalar_type() == torch::kFloat32) && gate.scalar_type() == x.scalar_type() && x.dim() == 2 &&
               gate.sizes() == x.sizes() && x.stride(1) == 1 && gate.stride(1) == 1, "x and gate must be [T, n] of one type with unit inner stride");
@@ -1186,6 +1316,11 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("mlstm", &mlstm);
   m.def("mlstm_chunkable", &mlstm_chunkable);
   m.def("sigmoid_mul", &sigmoid_mul);
+  m.def("causal_conv", &causal_conv);
+  m.def("recurrence", &recurrence);
+  m.def("gated_norm", &gated_norm);
+  m.def("talk_prepare", &talk_prepare);
+  m.def("talk_plain", &talk_plain);
   m.def("fused_moe_f32", &fused_moe_f32);
   m.def("fused_moe", &fused_moe);
   m.def("fused_moe_a2a", &fused_moe_a2a);

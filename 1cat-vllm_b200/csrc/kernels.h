@@ -71,6 +71,9 @@ struct EmbedParams {
   void* y;                      // [T][H] or null
   float scale;
   int T, H, vocab, buckets, mul_prev, mul_cur, gathered, f32;   // gathered: the table's rows are the tokens' own
+  const void* rows;             // [num_rows][H] learned position rows or null
+  const int* positions;         // [T]
+  int num_rows;
 };
 int embed_stream_launch(const EmbedParams& p, cudaStream_t st);
 int gelu_tanh_f32_launch(float* x, long long n, cudaStream_t st);  // in place
@@ -362,5 +365,63 @@ int gdn_conv_commit_launch(const GdnConvParams& p, cudaStream_t st);
 int gdn_recurrent_launch(const GdnParams& p, cudaStream_t st);
 unsigned int gdn_read_status(bool clear);
 void gdn_read_status_async(unsigned int* dst, cudaStream_t st);
+
+struct CausalConvParams {
+  const void* x;                // [T][C], row pitch ldx
+  long long ldx;
+  const void *w, *bias;         // [C][taps], [C] or null
+  void* y;                      // [T][C]
+  void* state;                  // [slots][max(taps - 1, 1)][C], updated in place
+  const int *query_start_loc, *state_slots, *has_initial_state;
+  int T, R, C, taps, silu, residual, f32;
+};
+int causal_conv_launch(const CausalConvParams& p, cudaStream_t st);
+
+// Recurrences with a matrix state (recurrence.cu). channel delta: q, k [Hk D], v [H V], a decay logits, b step logits; Mamba-2 (delta = 0): q = C and
+// k = B [Hk D] (Hk groups, D the state size), v = x [H V], b the dt logits.
+struct RecurrenceParams {
+  const void *q, *k, *v;        // rows of a common pitch ld
+  long long ld;
+  const float* a;               // [T][H D], pitch ld_a
+  long long ld_a;
+  const void* b;                // [T][H], pitch ld_b
+  long long ld_b;
+  const float *A_log, *dt_bias, *skip;   // [H]; [H D] (delta) or [H]; [H]
+  float dt_min, dt_max, scale;
+  float* state;                 // [slots][H][D][V]
+  void* out;                    // [T][H V]
+  const int *query_start_loc, *state_slots, *has_initial_state;
+  int T, R, Hk, H, D, V, delta, f32, skip_min_len;
+};
+int recurrence_launch(const RecurrenceParams& p, cudaStream_t st);
+struct GatedNormParams {
+  const void *x, *gate, *w;     // [T][n], [T][n], [n] or one part's
+  long long ld_x, ld_g;
+  void* y;                      // [T][n]
+  float eps;
+  int T, n, groups, w_shared, gate_first, f32;
+};
+int gated_norm_launch(const GatedNormParams& p, cudaStream_t st);
+
+struct TalkPrepareParams {
+  const void* qk;               // [T][H dim | G dim], pitch ld
+  long long ld;
+  const float* gain;            // [H dim]
+  float eps, coef;
+  int every;                    // 0: no temperature
+  const int *positions, *slots;
+  void *q_out, *pages;          // [T][G][group_rows][row]; [blocks][G][bs][row]
+  float* k_scale;               // [blocks][bs]
+  int T, H, G, dim, group_rows, row, bs, f32;
+};
+int talk_prepare_launch(const TalkPrepareParams& p, cudaStream_t st);
+struct TalkParams {
+  const void *q, *pages, *mix;  // as talk_prepare leaves them; [H][H] (to, from)
+  const float *k_scale, *bias;  // [blocks][bs]; [2][H]: r1, r2
+  void* out;                    // [T][H][dim]
+  const int *query_start_loc, *seq_lens, *block_table;
+  int bt_stride, T, R, H, G, dim, group_rows, row, bs, f32;
+};
+int talk_plain_launch(const TalkParams& p, cudaStream_t st);
 
 }  // namespace oc

@@ -1,7 +1,7 @@
 // Kernels around the fp32 residual stream and the un-rotated paged cache.
 //   stream_join: x' = x + mul * scale * post(part) (+ add), y = next(x'): a sub-block's output is normalised, scaled, added to the stream and the
 //                sum normalised for the next sub-block in one pass; optionally x' also leaves in the model's element type.
-//   embed_stream: the stream's start from scaled token embeddings and hashed-bigram rows.
+//   embed_stream: the stream's start from scaled token embeddings and hashed-bigram rows or learned position rows.
 //   kv_insert:   key (and value) rows into their pages.
 #include <type_traits>
 
@@ -188,6 +188,11 @@ __global__ void __launch_bounds__(256) embed_stream_kernel(const EmbedParams p) 
     if (big != nullptr) load_vec<E, N>(big + c, b);
 #pragma unroll
     for (int j = 0; j < N; ++j) v[j] = big != nullptr ? fmaf(v[j], p.scale, b[j]) : v[j] * p.scale;
+    if (p.rows != nullptr) {
+      load_vec<E, N>(reinterpret_cast<const E*>(p.rows) + (size_t)min(max(p.positions[t], 0), p.num_rows - 1) * p.H + c, b);
+#pragma unroll
+      for (int j = 0; j < N; ++j) v[j] += b[j];
+    }
     store_vec<float, N>(p.x + t * p.H + c, v);
     if (p.y != nullptr) store_vec<E, N>(reinterpret_cast<E*>(p.y) + t * p.H + c, v);
   }
@@ -231,10 +236,11 @@ int stream_join_launch(const StreamJoinParams& p, cudaStream_t st) {
 
 int embed_stream_launch(const EmbedParams& p, cudaStream_t st) {
   if (p.T == 0) return 0;
-  if (p.H < 1 || p.vocab < 1 || (p.bigram != nullptr && (p.prev == nullptr || p.buckets < 1))) return -1;
+  if (p.H < 1 || p.vocab < 1 || (p.bigram != nullptr && (p.prev == nullptr || p.buckets < 1)) ||
+      (p.rows != nullptr && (p.positions == nullptr || p.num_rows < 1))) return -1;
   const uintptr_t a = p.f32 ? 16 : 8;
   auto ok = [](const void* q, uintptr_t n) { return ((uintptr_t)q & (n - 1)) == 0; };
-  const bool vec = p.H % 4 == 0 && ok(p.table, a) && ok(p.bigram, a) && ok(p.x, 16) && ok(p.y, a);
+  const bool vec = p.H % 4 == 0 && ok(p.table, a) && ok(p.bigram, a) && ok(p.rows, a) && ok(p.x, 16) && ok(p.y, a);
   int threads = ((vec ? (p.H + 3) / 4 : p.H) + 31) / 32 * 32;
   if (threads > 256) threads = 256;
   auto go = [&](auto kernel) { launch_k(kernel, dim3((unsigned)p.T), dim3((unsigned)threads), 0, st, true, p); };

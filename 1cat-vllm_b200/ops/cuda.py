@@ -435,13 +435,14 @@ def stream_join(part, x, post, scale, nxt, out_dtype=None, add=None, copy_out=No
     return y, x_out
 
 
-def embed_stream(ids, table, scale, prev, bigram, muls, out_dtype, gathered=False):
+def embed_stream(ids, table, scale, prev, bigram, muls, out_dtype, gathered=False, rows=None, positions=None):
     global _LAUNCHES
     _LAUNCHES += 1
     T, H = ids.shape[0], table.shape[1]
     x = torch.empty(T, H, dtype=torch.float32, device=table.device)
-    y = torch.empty(T, H, dtype=out_dtype, device=table.device) if out_dtype != torch.float32 else None
-    _C.embed_stream(ids.to(torch.int32).contiguous(), table, scale, prev, bigram, muls[0], muls[1], x, y, gathered)
+    y = torch.empty(T, H, dtype=out_dtype, device=table.device) if out_dtype != torch.float32 and rows is None else None
+    _C.embed_stream(ids.to(torch.int32).contiguous(), table, scale, prev, bigram, muls[0], muls[1], x, y, gathered, rows,
+                    positions)
     return x, (x if y is None else y)
 
 
@@ -939,6 +940,59 @@ def mlstm(qkvg, gates, i_bias, f_bias, norm_w, eps, cap, H, D, V, state, md):
     S, n, m = state
     return _C.mlstm(qkvg, gates, i_bias, f_bias, norm_w, eps, cap, H, D, V, S, n, m, md.query_start_loc, md.state_slots, hi, meta, segs,
                     MLSTM_CHUNK_MIN_LEN, short)
+
+
+# ----------------------------------------------------------------------------- short convolutions, matrix-state recurrences
+def _int32(t):
+    return t if t.dtype == torch.int32 else t.to(torch.int32)
+
+
+def causal_conv(x, weight, bias, state, md, silu=False, residual=False):
+    global _LAUNCHES
+    _LAUNCHES += 1
+    return _C.causal_conv(x, weight, bias, state, md.query_start_loc, md.state_slots, _int32(md.has_initial_state), silu, residual)
+
+
+def channel_delta(qkv, a, b, A_log, dt_bias, state, md, Hk, H, D, V):
+    global _LAUNCHES
+    _LAUNCHES += 1
+    return _C.recurrence(qkv, a, b, A_log, dt_bias, None, state, md.query_start_loc, md.state_slots, _int32(md.has_initial_state), Hk, H, D, V, 0.0,
+                         float("inf"), 0, None)
+
+
+def mamba2(xbc, dt, A_log, dt_bias, D, state, md, H, G, N, V, dt_limit):
+    global _LAUNCHES
+    _LAUNCHES += 1
+    return _C.recurrence(xbc, None, dt, A_log, dt_bias, D, state, md.query_start_loc, md.state_slots, _int32(md.has_initial_state), G, H, N, V,
+                         dt_limit[0], dt_limit[1], 0, None)
+
+
+def gated_norm(x, gate, w, eps, groups, gate_first):
+    global _LAUNCHES
+    _LAUNCHES += 1
+    return _C.gated_norm(x, gate, w, eps, groups, gate_first)
+
+
+# ----------------------------------------------------------------------------- talking-heads attention
+def talk_row(H: int, G: int, dim: int) -> int:
+    """Width of a cached bf16 row."""
+    return dim
+
+
+def talk_prepare(qk, q_gain, eps, temperature, positions, pages, k_scale, slot_mapping, heads, kv_heads, dim):
+    global _LAUNCHES
+    _LAUNCHES += 1
+    coef, every = temperature or (0.0, 0)
+    return _C.talk_prepare(qk, q_gain, eps, coef, every, _int32(positions), pages, k_scale, _int32(slot_mapping), heads, kv_heads, dim, heads // kv_heads)
+
+
+def talk_attention(q, pages, k_scale, md, bias, mix):
+    global _LAUNCHES
+    H, T = mix.shape[0], q.shape[0]
+    out = torch.empty(T, H, q.shape[2], dtype=q.dtype, device=q.device)
+    _LAUNCHES += 1
+    _C.talk_plain(q, pages, k_scale, bias, mix, out, md.query_start_loc, md.seq_lens, md.block_table, H, q.shape[2])
+    return out
 
 
 def sigmoid_mul(x, gate):
