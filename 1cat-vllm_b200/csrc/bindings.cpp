@@ -1087,7 +1087,8 @@ torch::Tensor causal_conv(torch::Tensor x, torch::Tensor w, c10::optional<torch:
 // q | k | v (channel delta) or x | B | C (Mamba-2, a absent) side by side in `x`.
 torch::Tensor recurrence(torch::Tensor x, c10::optional<torch::Tensor> a, torch::Tensor b, torch::Tensor A_log, torch::Tensor dt_bias,
                          c10::optional<torch::Tensor> skip, torch::Tensor state, torch::Tensor qsl, torch::Tensor slots, torch::Tensor has_init, int64_t Hk, int64_t H,
-                         int64_t D, int64_t V, double dt_min, double dt_max, int64_t skip_min_len, c10::optional<torch::Tensor> out_) {
+                         int64_t D, int64_t V, double dt_min, double dt_max, c10::optional<torch::Tensor> chunk_meta, std::vector<std::vector<int64_t>> segments,
+                         int64_t chunk_min_len, bool any_short) {
   const auto et = x.scalar_type();
   const bool delta = a.has_value();
   TORCH_CHECK(x.is_cuda() && (et == torch::kBFloat16 || et == torch::kFloat32) && x.dim() == 2 && x.stride(1) == 1 && x.size(1) == 2 * Hk * D + H * V, "inputs must be [T, 2 Hk D + H V]");
@@ -1099,8 +1100,7 @@ torch::Tensor recurrence(torch::Tensor x, c10::optional<torch::Tensor> a, torch:
   else { TORCH_CHECK(skip.has_value() && skip->scalar_type() == torch::kFloat32 && skip->is_contiguous() && skip->numel() == H, "skip must be fp32 [H]"); }
   check_step(qsl, slots, has_init);
   const c10::cuda::CUDAGuard guard(x.device());
-  auto out = out_.has_value() ? *out_ : torch::empty({T, H * V}, x.options());
-  TORCH_CHECK(out.scalar_type() == et && out.is_contiguous() && out.numel() == T * H * V, "out must be [T, H V]");
+  auto out = torch::empty({T, H * V}, x.options());
   oc::RecurrenceParams p{};
   const char* base = (const char*)x.data_ptr();
   const int64_t es = x.element_size();
@@ -1114,9 +1114,36 @@ torch::Tensor recurrence(torch::Tensor x, c10::optional<torch::Tensor> a, torch:
   p.state = state.data_ptr<float>(); p.out = out.data_ptr();
   p.query_start_loc = qsl.data_ptr<int>(); p.state_slots = slots.data_ptr<int>(); p.has_initial_state = has_init.data_ptr<int>();
   p.T = (int)T; p.R = (int)slots.numel(); p.Hk = (int)Hk; p.H = (int)H; p.D = (int)D; p.V = (int)V; p.delta = delta; p.f32 = et == torch::kFloat32;
-  p.skip_min_len = (int)skip_min_len;
-  const int rc = oc::recurrence_launch(p, cur_stream());
-  TORCH_CHECK(rc == 0, "recurrence failed: ", rc, " (key sizes up to 256)");
+  p.skip_min_len = segments.empty() ? 0 : (int)chunk_min_len;
+  if (segments.empty() || any_short) {
+    const int rc = oc::recurrence_launch(p, cur_stream());
+    TORCH_CHECK(rc == 0, "recurrence failed: ", rc, " (key sizes up to 256)");
+  }
+  if (segments.empty()) return out;
+  TORCH_CHECK(et == torch::kBFloat16 && chunk_meta.has_value() && chunk_meta->scalar_type() == torch::kInt32 && chunk_meta->is_contiguous(), "chunk metadata must be int32, inputs bf16");
+  int64_t most = 0;
+  for (auto& g : segments) {
+    TORCH_CHECK(g.size() == 3 && g[0] >= 0 && g[0] + 3 * (g[1] + g[2]) <= chunk_meta->numel(), "chunk metadata too small");
+    most = std::max(most, g[1]);
+  }
+  oc::DeltaChunkParams c{};
+  c.q = (const __nv_bfloat16*)p.q; c.k = (const __nv_bfloat16*)p.k; c.v = (const __nv_bfloat16*)p.v; c.ld = p.ld; c.a = p.a; c.ld_a = p.ld_a;
+  c.b = (const __nv_bfloat16*)p.b; c.ld_b = p.ld_b; c.A_log = p.A_log; c.dt_bias = p.dt_bias; c.skip = p.skip; c.dt_min = p.dt_min; c.dt_max = p.dt_max;
+  c.scale = p.scale; c.state = p.state; c.out = (__nv_bfloat16*)p.out; c.query_start_loc = p.query_start_loc; c.state_slots = p.state_slots;
+  c.has_initial_state = p.has_initial_state; c.Hk = p.Hk; c.H = p.H; c.D = p.D; c.V = p.V; c.Vp = (p.V + 31) / 32 * 32;
+  c.vec = p.ld % 8 == 0 && D % 8 == 0 && V % 8 == 0 && ((uintptr_t)base & 15) == 0;
+  torch::Tensor ws;
+  if (delta) {
+    ws = torch::empty({most * H * (int64_t)oc::delta_chunk_elems((int)D, c.Vp)}, x.options());
+    c.ws = (__nv_bfloat16*)ws.data_ptr();
+  }
+  for (auto& g : segments) {
+    const int* mp = chunk_meta->data_ptr<int>() + g[0];
+    c.chunk_req = mp; c.chunk_t0 = mp + g[1];
+    c.long_req = mp + 3 * g[1]; c.long_chunk0 = c.long_req + g[2]; c.long_n = c.long_chunk0 + g[2];
+    const int rc = delta ? oc::delta_chunk_launch(c, (int)g[1], (int)g[2], cur_stream()) : oc::ssd_chunk_launch(c, (int)g[2], cur_stream());
+    TORCH_CHECK(rc == 0, "chunked recurrence failed: ", rc);
+  }
   return out;
 }
 
@@ -1318,6 +1345,8 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("sigmoid_mul", &sigmoid_mul);
   m.def("causal_conv", &causal_conv);
   m.def("recurrence", &recurrence);
+  m.def("recurrence_chunkable", [](int64_t D, int64_t V) { return oc::recurrence_chunkable((int)D, (int)V); });
+  m.def("delta_chunk_bytes", [](int64_t D, int64_t V) { return (int64_t)oc::delta_chunk_elems((int)D, (int)((V + 31) / 32 * 32)) * 2; });
   m.def("gated_norm", &gated_norm);
   m.def("talk_prepare", &talk_prepare);
   m.def("talk_plain", &talk_plain);

@@ -394,6 +394,27 @@ struct RecurrenceParams {
   int T, R, Hk, H, D, V, delta, f32, skip_min_len;
 };
 int recurrence_launch(const RecurrenceParams& p, cudaStream_t st);
+// Chunked forms for bf16 portions of at least 64 tokens (recurrence_chunk.cu); the recurrent kernel skips those (skip_min_len).
+struct DeltaChunkParams {
+  const __nv_bfloat16 *q, *k, *v;
+  long long ld;
+  const float* a;
+  long long ld_a;
+  const __nv_bfloat16* b;
+  long long ld_b;
+  const float *A_log, *dt_bias, *skip;
+  float dt_min, dt_max, scale;
+  float* state;
+  __nv_bfloat16* out;
+  const int *query_start_loc, *state_slots, *has_initial_state;
+  const int *chunk_req, *chunk_t0, *long_req, *long_chunk0, *long_n;   // one segment of the step's chunk list, see MlstmParams
+  __nv_bfloat16* ws;            // delta: [chunks][H] x delta_chunk_elems
+  int Hk, H, D, V, Vp, vec;     // Vp: V rounded up to 32; vec: every row of q, k, v starts on a 16-byte boundary
+};
+bool recurrence_chunkable(int D, int V);
+size_t delta_chunk_elems(int D, int Vp);
+int delta_chunk_launch(const DeltaChunkParams& p, int chunks, int longs, cudaStream_t st);
+int ssd_chunk_launch(const DeltaChunkParams& p, int longs, cudaStream_t st);
 struct GatedNormParams {
   const void *x, *gate, *w;     // [T][n], [T][n], [n] or one part's
   long long ld_x, ld_g;

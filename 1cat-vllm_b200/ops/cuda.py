@@ -891,25 +891,24 @@ def mla_prefill(plan, q, latent_cache, md, expand, out, nope, rope, lora_pad, sc
 
 
 # ----------------------------------------------------------------------------- mLSTM
-MLSTM_CHUNK_MIN_LEN = 64           # portions of at least this many tokens take the chunked (tensor-core) kernels
-MLSTM_SEGMENT_BYTES = 256 << 20    # chunk states of a segment (measured: smaller ones pay in half-filled waves what they save in traffic)
+CHUNK_MIN_LEN = 64                 # portions of at least this many tokens take the chunked (tensor-core) kernels
+CHUNK_SEGMENT_BYTES = 256 << 20    # what a segment keeps per chunk (measured: smaller ones pay in half-filled waves what they save in traffic)
 
 
-def _mlstm_segments(md, H: int, D: int, V: int, device):
-    """(device tensor, [(offset, chunks, sequences)], whether short portions remain) of this step's chunk list, built once per step and
-    geometry from the host-side query lengths and cut into segments whose chunk states stay small."""
-    cache = md.__dict__.setdefault("_mlstm_segments", {})
-    if (H, D, V) in cache:
-        return cache[(H, D, V)]
+def _chunk_segments(md, per: int, device):
+    """(device tensor, [(offset, chunks, sequences)], whether short portions remain) of this step's list of 64-token chunks, built once per step
+    from the host-side query lengths and cut into segments of ``per`` chunks, which bounds the memory of what is kept per chunk."""
+    cache = md.__dict__.setdefault("_chunk_segments", {})
+    if per in cache:
+        return cache[per]
     qlens = getattr(md, "query_lens_cpu", None)
     out = (None, [], True)
-    if qlens and max(qlens) >= MLSTM_CHUNK_MIN_LEN and not getattr(md, "is_uniform_decode", False) and _C.mlstm_chunkable(D, V):
+    if qlens and max(qlens) >= CHUNK_MIN_LEN and not getattr(md, "is_uniform_decode", False):
         chunks, t = [], 0
         for r, n in enumerate(qlens):
-            if n >= MLSTM_CHUNK_MIN_LEN:
+            if n >= CHUNK_MIN_LEN:
                 chunks += [(r, t + c) for c in range(0, n, 64)]
             t += n
-        per = max(8, MLSTM_SEGMENT_BYTES // (8 * H * D * V))
         flat, segs = [], []
         for a in range(0, len(chunks), per):
             part = chunks[a:a + per]
@@ -924,22 +923,23 @@ def _mlstm_segments(md, H: int, D: int, V: int, device):
             segs.append([len(flat), len(part), len(reqs)])
             flat += [r for r, _ in part] + [t0 for _, t0 in part] + owner + reqs + first + count
         host = torch.tensor(flat, dtype=torch.int32).pin_memory()
-        out = (host.to(device, non_blocking=True), segs, any(0 < n < MLSTM_CHUNK_MIN_LEN for n in qlens))
-        md.__dict__.setdefault("_mlstm_hosts", []).append(host)   # keep the pinned buffer alive until the copy has run
-    cache[(H, D, V)] = out
+        out = (host.to(device, non_blocking=True), segs, any(0 < n < CHUNK_MIN_LEN for n in qlens))
+        md.__dict__.setdefault("_chunk_hosts", []).append(host)   # keep the pinned buffer alive until the copy has run
+    cache[per] = out
     return out
 
 
 def mlstm(qkvg, gates, i_bias, f_bias, norm_w, eps, cap, H, D, V, state, md):
-    """Short portions (decoding included) run the recurrent kernel, portions of at least ``MLSTM_CHUNK_MIN_LEN`` tokens the chunked ones
+    """Short portions (decoding included) run the recurrent kernel, portions of at least ``CHUNK_MIN_LEN`` tokens the chunked ones
     (bf16); both include the head norm and the output gate."""
     global _LAUNCHES
     hi = md.has_initial_state if md.has_initial_state.dtype == torch.int32 else md.has_initial_state.to(torch.int32)
-    meta, segs, short = (None, [], True) if qkvg.dtype == torch.float32 else _mlstm_segments(md, H, D, V, qkvg.device)
+    meta, segs, short = (None, [], True) if qkvg.dtype == torch.float32 or not _C.mlstm_chunkable(D, V) else \
+        _chunk_segments(md, max(8, CHUNK_SEGMENT_BYTES // (8 * H * D * V)), qkvg.device)
     _LAUNCHES += 3 * len(segs) + int(short or not segs)
     S, n, m = state
     return _C.mlstm(qkvg, gates, i_bias, f_bias, norm_w, eps, cap, H, D, V, S, n, m, md.query_start_loc, md.state_slots, hi, meta, segs,
-                    MLSTM_CHUNK_MIN_LEN, short)
+                    CHUNK_MIN_LEN, short)
 
 
 # ----------------------------------------------------------------------------- short convolutions, matrix-state recurrences
@@ -954,17 +954,22 @@ def causal_conv(x, weight, bias, state, md, silu=False, residual=False):
 
 
 def channel_delta(qkv, a, b, A_log, dt_bias, state, md, Hk, H, D, V):
+    """Short portions (decoding included) run the recurrent kernel, portions of at least ``CHUNK_MIN_LEN`` tokens the chunked ones (bf16)."""
     global _LAUNCHES
-    _LAUNCHES += 1
+    meta, segs, short = (None, [], True) if qkv.dtype == torch.float32 or not _C.recurrence_chunkable(D, V) else \
+        _chunk_segments(md, max(8, CHUNK_SEGMENT_BYTES // (H * _C.delta_chunk_bytes(D, V))), qkv.device)
+    _LAUNCHES += 2 * len(segs) + int(short or not segs)
     return _C.recurrence(qkv, a, b, A_log, dt_bias, None, state, md.query_start_loc, md.state_slots, _int32(md.has_initial_state), Hk, H, D, V, 0.0,
-                         float("inf"), 0, None)
+                         float("inf"), meta, segs, CHUNK_MIN_LEN, short)
 
 
 def mamba2(xbc, dt, A_log, dt_bias, D, state, md, H, G, N, V, dt_limit):
+    """As ``channel_delta``; the chunked kernel keeps nothing per chunk, so its list is one segment."""
     global _LAUNCHES
-    _LAUNCHES += 1
+    meta, segs, short = (None, [], True) if xbc.dtype == torch.float32 or not _C.recurrence_chunkable(N, V) else _chunk_segments(md, 1 << 30, xbc.device)
+    _LAUNCHES += len(segs) + int(short or not segs)
     return _C.recurrence(xbc, None, dt, A_log, dt_bias, D, state, md.query_start_loc, md.state_slots, _int32(md.has_initial_state), G, H, N, V,
-                         dt_limit[0], dt_limit[1], 0, None)
+                         dt_limit[0], dt_limit[1], meta, segs, CHUNK_MIN_LEN, short)
 
 
 def gated_norm(x, gate, w, eps, groups, gate_first):

@@ -1,0 +1,160 @@
+"""Nalasun's kernels on a B200: each against a plain float64 computation, then the engine (paged cache, state slots, CUDA graphs, mixed batches) in
+bf16 and fp32 against the float64 restatement."""
+import pytest
+import torch
+
+import nalasun_oracle as O
+
+pytestmark = pytest.mark.gpu
+DEV = "cuda"
+DTYPES = [torch.bfloat16, torch.float32]
+
+
+class Meta:
+    """Metadata of a batch of (new tokens, context length) requests; ``bt`` [R, pages]."""
+
+    def __init__(self, lens, bt=None, slots=None):
+        q = [a for a, _ in lens]
+        i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=DEV)
+        self.query_start_loc = torch.tensor([0] + q, dtype=torch.int32).cumsum(0, dtype=torch.int32).to(DEV)
+        self.query_lens_cpu, self.seq_lens_cpu, self.num_reqs = q, [s for _, s in lens], len(q)
+        self.seq_lens, self.block_table = i32(self.seq_lens_cpu), bt
+        self.max_query_len, self.max_seq_len = max(q), max(self.seq_lens_cpu)
+        self.positions = torch.cat([torch.arange(s - n, s) for n, s in lens]).to(torch.int32).to(DEV)
+        self.state_slots, self.has_initial_state = i32(slots or list(range(len(q)))), i32([int(s > n) for n, s in lens])
+
+
+def portions(plan, slots, run):
+    """``plan``: steps of token counts per sequence. ``run(md, who, ranges)`` gets one step's metadata and (first, last) of every sequence in it and
+    returns the rows of the step; comes back with the rows of every sequence."""
+    n = len(slots)
+    done, got = [0] * n, [[] for _ in range(n)]
+    for step in plan:
+        who = [a for a in range(n) if step[a]]
+        md = Meta([(step[a], done[a] + step[a]) for a in who], slots=[slots[a] for a in who])
+        y, o = run(md, who, [(done[a], done[a] + step[a]) for a in who]), 0
+        for a in who:
+            got[a].append(y[o:o + step[a]].cpu())
+            o += step[a]
+            done[a] += step[a]
+    return [torch.cat(x) for x in got]
+
+
+PLAN = [[700, 1, 63, 64, 0], [1, 65, 1, 2, 130], [64, 1, 1, 128, 7], [3, 200, 0, 0, 1]]
+SLOTS = [4, 0, 6, 2, 5]
+TOTAL = [sum(s[a] for s in PLAN) for a in range(5)]
+
+
+def rel(got, want):
+    return ((got.double() - want).abs().max() / want.abs().max()).item()
+
+
+# ------------------------------------------------------------------------------------------------ short convolutions
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("C,taps,bias,silu,residual", [(192, 4, False, False, True), (256, 4, True, True, False), (77, 3, True, True, False),
+                                                       (64, 2, False, True, True), (40, 1, True, False, False), (24, 7, False, True, False),
+                                                       (4104, 4, False, False, True), (96, 3, False, False, True)])
+def test_causal_convolution(C, taps, bias, silu, residual, dtype):
+    from onecat_vllm import ops
+    g = torch.Generator().manual_seed(C + taps)
+    plan = PLAN + [[2, 1, 2, 1, 3], [1, 2, 1, 3, 1], [2500, 0, 2, 0, 5]]
+    total = [sum(s[a] for s in plan) for a in range(5)]
+    full = [torch.randn(n, C + 16, generator=g).to(dtype) for n in total]
+    w, b = torch.randn(C, taps, generator=g).to(dtype), torch.randn(C, generator=g).to(dtype) if bias else None
+    state = torch.randn(7, *ops.conv_state_shape(C, taps), generator=g).to(dtype).to(DEV)   # what earlier owners of the slots left
+    spare = state[1].clone()
+
+    def run(md, who, ranges):
+        x = torch.cat([full[a][i:j] for a, (i, j) in zip(who, ranges)]).to(DEV)[:, 8: 8 + C]   # a column slice
+        return ops.causal_conv(x, w.to(DEV), None if b is None else b.to(DEV), state, md, silu, residual)
+    got = portions(plan, SLOTS, run)
+    assert torch.equal(state[1], spare)
+    for a in range(5):
+        x = full[a][:, 8: 8 + C].double()
+        y = O.causal_conv(x, w.double(), None if b is None else b.double())
+        y = O.silu(y) if silu else y
+        assert rel(got[a], x + y if residual else y) < (6e-3 if dtype == torch.bfloat16 else 1e-6)
+
+
+# ------------------------------------------------------------------------------------------------ matrix-state recurrences
+def delta_case(g, n, Hk, H, D, V, dtype, strong):
+    qkv = torch.randn(n, 2 * Hk * D + H * V + 8, generator=g).to(dtype)
+    a = torch.randn(n, H * D, generator=g) * (4.0 if strong else 1.0) - (0.0 if strong else 3.0)
+    return qkv, a, torch.randn(n, H, generator=g).to(dtype)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("Hk,H,D,V,strong", [(4, 4, 64, 32, False), (2, 6, 128, 128, False), (1, 2, 32, 64, True), (3, 3, 20, 72, True), (2, 2, 100, 40, False),
+                                             (1, 1, 256, 48, False), (2, 4, 9, 21, True), (1, 3, 128, 200, True), (2, 2, 16, 33, False)])
+def test_channel_delta_kernels(Hk, H, D, V, strong, dtype, monkeypatch):
+    """Prompts, portions and single tokens in one batch over shuffled slots, then the same sequences go on: outputs and states equal the
+    token-by-token float64 recurrence of each sequence alone. ``strong``: decays that forget within a token or two beside some near one."""
+    from onecat_vllm import ops
+    from onecat_vllm.ops import cuda as K
+    monkeypatch.setattr(K, "CHUNK_SEGMENT_BYTES", 8 * H * K._C.delta_chunk_bytes(D, V) if D <= 128 else 1)   # several segments a step
+    g = torch.Generator().manual_seed(D + V)
+    A_log, dt_bias = torch.rand(H, generator=g) * 2 - (1.0 if not strong else 0.0), torch.randn(H * D, generator=g)
+    full = [delta_case(g, n, Hk, H, D, V, dtype, strong) for n in TOTAL]
+    state = torch.randn(7, H, D, V, generator=g).to(DEV)
+    spare = state[1].clone()
+
+    def run(md, who, ranges):
+        qkv, a, b = (torch.cat([full[x][k][i:j] for x, (i, j) in zip(who, ranges)]).to(DEV) for k in range(3))
+        return ops.channel_delta(qkv[:, : 2 * Hk * D + H * V], a, b, A_log.to(DEV), dt_bias.to(DEV), state, md, Hk, H, D, V)
+    got = portions(PLAN, SLOTS, run)
+    assert torch.equal(state[1], spare)
+    own = [h // (H // Hk) for h in range(H)]
+    for x in range(5):
+        qkv, a, b = full[x]
+        n = qkv.shape[0]
+        q, k, v = qkv[:, : 2 * Hk * D + H * V].double().split([Hk * D, Hk * D, H * V], 1)
+        gate = torch.exp(-torch.exp(A_log.double()).view(1, H, 1) * O.softplus(a.double() + dt_bias.double()).view(n, H, D))
+        want = O.delta_steps(O.unit(q.view(n, Hk, D))[:, own] * D ** -0.5, O.unit(k.view(n, Hk, D))[:, own], v.view(n, H, V), gate,
+                             torch.sigmoid(b.double())).reshape(n, H * V)
+        assert rel(got[x], want) < (6e-3 if dtype == torch.bfloat16 else 2e-5), (x, rel(got[x], want))
+        err = (got[x].double() - want).abs().mean() / want.abs().mean()
+        assert err < (3e-3 if dtype == torch.bfloat16 else 2e-6), (x, err)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("G,H,N,V,limit", [(2, 4, 32, 32, (0.0, float("inf"))), (1, 8, 128, 64, (0.0, float("inf"))), (3, 3, 20, 72, (0.05, 0.9)),
+                                           (2, 4, 9, 21, (0.0, float("inf"))), (1, 2, 256, 40, (0.0, float("inf"))), (4, 4, 64, 100, (0.0, 0.5))])
+def test_mamba2_kernels(G, H, N, V, limit, dtype):
+    from onecat_vllm import ops
+    g = torch.Generator().manual_seed(N + V)
+    A_log, dt_bias, skip = torch.rand(H, generator=g) * 3 - 2, torch.randn(H, generator=g) - 1, torch.randn(H, generator=g)
+    full = [(torch.randn(n, H * V + 2 * G * N, generator=g).mul(0.7).to(dtype), torch.randn(n, H + 3, generator=g).to(dtype)) for n in TOTAL]
+    state = torch.randn(7, H, N, V, generator=g).to(DEV)
+    spare = state[1].clone()
+
+    def run(md, who, ranges):
+        xbc, dt = (torch.cat([full[x][k][i:j] for x, (i, j) in zip(who, ranges)]).to(DEV) for k in range(2))
+        return ops.mamba2(xbc, dt[:, 3:], A_log.to(DEV), dt_bias.to(DEV), skip.to(DEV), state, md, H, G, N, V, limit)
+    got = portions(PLAN, SLOTS, run)
+    assert torch.equal(state[1], spare)
+    own = [h // (H // G) for h in range(H)]
+    for a in range(5):
+        xbc, dt = full[a]
+        n = xbc.shape[0]
+        x, B, Cc = xbc.double().split([H * V, G * N, G * N], 1)
+        want = O.ssm_steps(x.reshape(n, H, V), B.reshape(n, G, N)[:, own], Cc.reshape(n, G, N)[:, own],
+                           O.softplus(dt[:, 3:].double() + dt_bias.double()).clamp(*limit), A_log.double(), skip.double()).reshape(n, H * V)
+        assert rel(got[a], want) < (6e-3 if dtype == torch.bfloat16 else 2e-5), (a, rel(got[a], want))
+        err = (got[a].double() - want).abs().mean() / want.abs().mean()
+        assert err < (3e-3 if dtype == torch.bfloat16 else 2e-6), (a, err)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("T,n,groups,shared", [(33, 128, 4, True), (5, 4096, 2, False), (64, 300, 3, False), (7, 21, 1, True), (129, 2048, 16, True), (3, 8192, 1, False)])
+@pytest.mark.parametrize("gate_first", [True, False])
+def test_gated_norm(T, n, groups, shared, gate_first, dtype):
+    from onecat_vllm import ops
+    g = torch.Generator().manual_seed(n)
+    x, z = (torch.randn(T, n + 8, generator=g).to(dtype) for _ in range(2))
+    w = torch.randn(n // groups if shared else n, generator=g).to(dtype)
+    got = ops.gated_norm(x.to(DEV)[:, :n], z.to(DEV)[:, 8:], w.to(DEV), 1e-3, groups, gate_first).cpu()
+    v, zz = x[:, :n].double(), z[:, 8:].double()
+    v = v * O.silu(zz) if gate_first else v
+    v = O.rms(v.view(T, groups, -1), 1e-3) * w.double().view(-1, n // groups)
+    want = v.reshape(T, n) if gate_first else v.reshape(T, n) * torch.sigmoid(zz)
+    assert rel(got, want) < (6e-3 if dtype == torch.bfloat16 else 2e-6)

@@ -216,7 +216,7 @@ def test_mlstm_kernels(H, D, V, dtype, monkeypatch):
     token-by-token float64 recurrence of each sequence alone."""
     from onecat_vllm import ops
     from onecat_vllm.ops import cuda as K
-    monkeypatch.setattr(K, "MLSTM_SEGMENT_BYTES", 8 * 8 * H * D * V)   # several segments a step
+    monkeypatch.setattr(K, "CHUNK_SEGMENT_BYTES", 8 * 8 * H * D * V)   # several segments a step
     g = torch.Generator().manual_seed(D + V)
     eps, cap = 1e-5, 9.0
     # how many tokens each of five sequences brings, step by step
@@ -259,14 +259,14 @@ def test_mlstm_chunks_and_recurrence_agree():
     x, gates, bi, bf, nw = mlstm_inputs(g, T, H, D, V, torch.bfloat16)
     outs, states = [], []
     for least in (64, 10 ** 9):
-        old, K.MLSTM_CHUNK_MIN_LEN = K.MLSTM_CHUNK_MIN_LEN, least
+        old, K.CHUNK_MIN_LEN = K.CHUNK_MIN_LEN, least
         try:
             state = tuple(torch.zeros(2, *s, device=DEV) for s in ((H, D, V), (H, D), (H,)))
             md = Meta([(T, T)], slots=[1], init=[0])
             outs.append(ops.mlstm(x.to(DEV), gates.to(DEV), bi.to(DEV), bf.to(DEV), nw.to(DEV), 1e-5, 9.0, H, D, V, state, md).float().cpu())
             states.append([t[1].cpu() for t in state])
         finally:
-            K.MLSTM_CHUNK_MIN_LEN = old
+            K.CHUNK_MIN_LEN = old
     assert (outs[0] - outs[1]).abs().mean() < 1e-3
     assert all((a - b).abs().max() <= 1e-4 * b.abs().max() for a, b in zip(*states))
 
