@@ -1208,6 +1208,30 @@ void talk_plain(torch::Tensor q, torch::Tensor pages, torch::Tensor k_scale, tor
   TORCH_CHECK(rc == 0, "talk_plain failed: ", rc);
 }
 
+// (cached row, query rows per key head, tokens per block of the two passes, longest portion of the single-token variant); empty: plain kernel
+std::vector<int64_t> talk_sizes(int64_t H, int64_t G, int64_t dim) {
+  oc::TalkSizes s;
+  if (!oc::talk_tc_sizes((int)H, (int)G, (int)dim, &s)) return {};
+  return {s.row, s.group_rows, s.stats_tokens, s.mix_tokens, s.short_len};
+}
+
+void talk_tc(torch::Tensor q, torch::Tensor pages, torch::Tensor k_scale, torch::Tensor bias, torch::Tensor mix, torch::Tensor out, torch::Tensor qsl,
+             torch::Tensor seq_lens, torch::Tensor bt, int64_t H, int64_t dim, bool dec, int64_t short_len, int64_t splits, int64_t mix_splits, int64_t stats_tiles,
+             int64_t mix_tiles, torch::Tensor ws_ml, c10::optional<torch::Tensor> ws_o) {
+  oc::TalkTcParams p{};
+  p.t = talk_params(q, pages, k_scale, bias, mix, out, qsl, seq_lens, bt, H, dim);
+  const int64_t T = p.t.T;
+  TORCH_CHECK(!p.t.f32 && ((uintptr_t)p.t.q & 15) == 0 && ((uintptr_t)p.t.pages & 15) == 0, "bf16 rows on 16-byte boundaries");
+  TORCH_CHECK(ws_ml.scalar_type() == torch::kFloat32 && ws_ml.numel() >= splits * T * H * 2, "workspace of the sums");
+  if (mix_splits > 1) TORCH_CHECK(ws_o.has_value() && ws_o->scalar_type() == torch::kFloat32 && ws_o->numel() >= mix_splits * T * H * dim, "workspace of the outputs");
+  p.ws_ml = ws_ml.data_ptr<float>();
+  p.ws_o = mix_splits > 1 ? ws_o->data_ptr<float>() : nullptr;
+  p.splits = (int)splits; p.mix_splits = (int)mix_splits; p.stats_tiles = (int)stats_tiles; p.mix_tiles = (int)mix_tiles; p.short_len = (int)short_len;
+  const c10::cuda::CUDAGuard guard(q.device());
+  const int rc = oc::talk_tc_launch(p, dec, cur_stream());
+  TORCH_CHECK(rc == 0, "talk_tc failed: ", rc);
+}
+
 torch::Tensor sigmoid_mul(torch::Tensor x, torch::Tensor gate) {
   TORCH_CHECK(x.is_cuda() && (x.scalar_type() == torch::kBFloat16 || x.scalar_type() == torch::kFloat32) && gate.scalar_type() == x.scalar_type() && x.dim() == 2 &&
               gate.sizes() == x.sizes() && x.stride(1) == 1 && gate.stride(1) == 1, "x and gate must be [T, n] of one type with unit inner stride");
@@ -1350,6 +1374,8 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gated_norm", &gated_norm);
   m.def("talk_prepare", &talk_prepare);
   m.def("talk_plain", &talk_plain);
+  m.def("talk_sizes", &talk_sizes);
+  m.def("talk_tc", &talk_tc);
   m.def("fused_moe_f32", &fused_moe_f32);
   m.def("fused_moe", &fused_moe);
   m.def("fused_moe_a2a", &fused_moe_a2a);

@@ -444,5 +444,16 @@ struct TalkParams {
   int bt_stride, T, R, H, G, dim, group_rows, row, bs, f32;
 };
 int talk_plain_launch(const TalkParams& p, cudaStream_t st);
+// Tensor-core form (talk_tc.cu): cached rows and query rows padded as TalkSizes says; single tokens (dec) and longer portions are launched apart.
+struct TalkSizes { int row, group_rows, stats_tokens, mix_tokens, short_len; };   // tokens per block of either pass; longest portion of the dec variant
+bool talk_tc_sizes(int H, int G, int dim, TalkSizes* s);
+struct TalkTcParams {
+  TalkParams t;
+  float* ws_ml;                 // [splits][T][H][2] maximum (log2 domain) and sum
+  float* ws_o;                  // [mix_splits][T][H][dim], when there is more than one
+  int splits, mix_splits, stats_tiles, mix_tiles, short_len;
+  int kt;                       // keys per tile of the second pass, set by the launcher
+};
+int talk_tc_launch(const TalkTcParams& p, bool dec, cudaStream_t st);
 
 }  // namespace oc

@@ -205,7 +205,7 @@ class TalkingAttention(nn.Module):
         pages, k_scale = kv_cache
         q = ops.talk_prepare(self.qkg_proj(x), self.q_gain, self.eps, self.temperature, md.positions, pages, k_scale, md.slot_mapping, self.Hq, self.Hkv,
                              self.dim)
-        o = ops.talk_attention(q, pages, k_scale, md, self.bias, self.talk)
+        o = ops.talk_attention(q, pages, k_scale, md, self.bias, self.talk, self.dim)
         return self.o_proj(o.reshape(x.shape[0], self.Hq * self.dim))
 
 

@@ -114,10 +114,10 @@ def talk_prepare(qk, q_gain, eps, temperature, positions, pages, k_scale, slot_m
     return f(qk, q_gain, eps, temperature, positions, pages, k_scale, slot_mapping, heads, kv_heads, dim)
 
 
-def talk_attention(q, pages, k_scale, md, bias, mix):
-    """Talking-heads attention of the step ``md``; see ``ref.talk_attention``."""
+def talk_attention(q, pages, k_scale, md, bias, mix, dim):
+    """Talking-heads attention of the step ``md`` with heads of ``dim`` columns; see ``ref.talk_attention``."""
     if q.is_cuda:
-        return ext().talk_attention(q, pages, k_scale, md, bias, mix)
+        return ext().talk_attention(q, pages, k_scale, md, bias, mix, dim)
     return ref.talk_attention(q, pages, k_scale, md.block_table, md.query_start_loc, md.seq_lens, bias, mix)
 
 

@@ -158,3 +158,126 @@ def test_gated_norm(T, n, groups, shared, gate_first, dtype):
     v = O.rms(v.view(T, groups, -1), 1e-3) * w.double().view(-1, n // groups)
     want = v.reshape(T, n) if gate_first else v.reshape(T, n) * torch.sigmoid(zz)
     assert rel(got, want) < (6e-3 if dtype == torch.bfloat16 else 2e-6)
+
+
+# ------------------------------------------------------------------------------------------------ talking-heads attention
+def pages(lens, bs, seed):
+    """Block table [R, pages] of shuffled pages, their number."""
+    nbs = [-(-s // bs) for _, s in lens]
+    perm = torch.randperm(sum(nbs) + 4, generator=torch.Generator().manual_seed(seed)).tolist()
+    bt = torch.zeros(len(lens), max(nbs), dtype=torch.int32)
+    for r, n in enumerate(nbs):
+        bt[r, :n] = torch.tensor([perm.pop() for _ in range(n)])
+    return bt, sum(nbs) + 4
+
+
+LENS = [[(200, 200), (1, 400), (3, 77), (64, 300), (1, 1)], [(1, 1500), (1, 16), (1, 17), (1, 640)], [(2, 2), (33, 65), (130, 513)], [(1, 129)] * 40,
+        [(300, 1100)]]
+
+
+def attend(q, k, f, bias, mix):
+    """q [n, H, D] (the last rows of the sequence), k [S, G, D], f [S] -> [n, H, D], all float64."""
+    n, H, _ = q.shape
+    S, G, _ = k.shape
+    kk = k[:, [h // (H // G) for h in range(H)]]
+    s = torch.einsum("ihd,jhd->hij", q, kk) * f - O.distance_penalty(S, bias[0], bias[1])[:, S - n:]
+    s = s.masked_fill(torch.arange(S).view(1, -1) > torch.arange(S - n, S).view(-1, 1), -float("inf"))
+    return torch.einsum("hij,jhd->ihd", O.talk(torch.softmax(s, -1), mix), kk)
+
+
+def talk_case(g, lens, H, G, dim, dtype, bs=16, sharp=1.0):
+    """The step's q|k rows, the cache with everything ahead of them, and what the kernels need beside them."""
+    from onecat_vllm import ops
+    from onecat_vllm.ops import cuda as K
+    row = K.talk_row(H, G, dim) if dtype == torch.bfloat16 else dim
+    bt, n = pages(lens, bs, len(lens) + H)
+    cache, fac = torch.full((n, 1, G, bs, row), 3.0, dtype=dtype, device=DEV), torch.full((n, bs), 9.0, device=DEV)   # what earlier owners left
+    seqs = [torch.randn(s, (H + G) * dim, generator=g).to(dtype) for _, s in lens]
+    gain = (torch.randn(H * dim, generator=g) * 0.3 + 1.0) * sharp * 2 * dim ** -0.5
+    bias = torch.stack([torch.rand(H, generator=g) * 0.8 + 0.1, torch.rand(H, generator=g) * 2 + 0.05])
+    mix = (torch.eye(H) * 0.6 + torch.randn(H, H, generator=g) * 0.4).to(dtype)
+
+    def insert(rows, md, a, b):   # positions a .. b - 1 of every request
+        slot = torch.cat([bt[r].long()[torch.arange(i, j) // bs] * bs + torch.arange(i, j) % bs for r, (i, j) in enumerate(zip(a, b))])
+        return ops.talk_prepare(rows.to(DEV), gain.to(DEV), 1e-4, (0.3, 50), md.positions, cache, fac, slot.to(torch.int32).to(DEV), H, G, dim)
+    ahead = [s - q for q, s in lens]
+    if any(ahead):
+        insert(torch.cat([x[:n] for x, n in zip(seqs, ahead)]), Meta([(n, n) for n in ahead if n]), [0] * len(lens), ahead)
+    md = Meta(lens, bt.to(DEV))
+    q = insert(torch.cat([x[n:] for x, n in zip(seqs, ahead)]), md, ahead, [s for _, s in lens])
+    return md, q, cache, fac, seqs, gain, bias, mix
+
+
+SIZES = [(8, 2, 64), (16, 4, 128), (32, 8, 128), (6, 3, 40), (4, 4, 64), (12, 2, 96), (16, 1, 128), (5, 5, 20), (7, 1, 33), (1, 1, 64), (24, 8, 64), (18, 1, 32),
+         (2, 1, 128), (16, 16, 128), (3, 1, 200), (33, 1, 16), (40, 8, 16)]
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,G,dim", SIZES)
+def test_talking_heads_kernels(H, G, dim, dtype):
+    """Prompts, portions and single tokens in one batch over shuffled pages against float64 on the same cached numbers."""
+    from onecat_vllm import ops
+    from onecat_vllm.ops import cuda as K
+    g = torch.Generator().manual_seed(H * dim + G)
+    for lens in LENS:
+        md, q, cache, fac, seqs, gain, bias, mix = talk_case(g, lens, H, G, dim, dtype)
+        rows = q.view(q.shape[0], G, -1, q.shape[2])[:, :, : H // G, :dim].reshape(-1, H, dim).cpu().double()
+        got = ops.talk_attention(q, cache, fac, md, bias.to(DEV), mix.to(DEV), dim).cpu().double()
+        assert K.check_status() == 0
+        o, seen = 0, set()
+        for (n, s), x in zip(lens, seqs):
+            k = x[:, H * dim:].double()
+            want_q = O.rms(x[s - n:, : H * dim].double(), 1e-4) * gain.double() * O.temperature(s, 0.3, 50)[s - n:].view(-1, 1)
+            assert rel(rows[o:o + n].reshape(n, -1), want_q) < (5e-3 if dtype == torch.bfloat16 else 1e-6)
+            if (n, s) not in seen or o == 0:
+                f = 1 / torch.sqrt((k * k).mean(-1) + 1e-4)
+                want = attend(rows[o:o + n], k.view(s, G, dim), f, bias.double(), mix.double())
+                assert rel(got[o:o + n], want) < (5e-3 if dtype == torch.bfloat16 else 1e-5), (n, s, rel(got[o:o + n], want))
+            seen.add((n, s))
+            o += n
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,G,dim", [(8, 2, 64), (6, 3, 40), (16, 1, 128)])
+def test_one_key_stands_out_at_page_and_tile_edges(H, G, dim, dtype):
+    """One head's query fits one far key, whose value is large: heads read it through the mix, in a prompt and decoded alone."""
+    from onecat_vllm import ops
+    g = torch.Generator().manual_seed(dim)
+    S = 700
+    for at in (0, 15, 16, 31, 32, 63, 64, 127, 128, 511, 698):
+        for lens in ([(40, S)], [(1, S)]):
+            md, q, cache, fac, seqs, gain, bias, mix = talk_case(g, lens, H, G, dim, dtype)
+            k = seqs[0][:, H * dim:].double().view(S, G, dim)
+            rows = q.view(q.shape[0], G, -1, q.shape[2])
+            h = H - 1
+            rows[:, G - 1, (H // G) - 1, :dim] = (k[at, G - 1] * 20 * dim ** -0.5).to(dtype).to(DEV)
+            f = 1 / torch.sqrt((k.reshape(S, -1) ** 2).mean(-1) + 1e-4)
+            qq = rows[:, :, : H // G, :dim].reshape(-1, H, dim).cpu().double()
+            want = attend(qq, k, f, bias.double() * 0.1, mix.double())
+            got = ops.talk_attention(q, cache, fac, md, bias.to(DEV) * 0.1, mix.to(DEV), dim).cpu()
+            assert rel(got, want) < (5e-3 if dtype == torch.bfloat16 else 1e-5), (at, lens)
+            assert (want[-1, h] - k[at, G - 1] * mix[h, h].double()).abs().max() < 3 * want[-1].abs().max()
+
+
+def test_portions_do_not_depend_on_splits(monkeypatch):
+    from onecat_vllm import ops
+    from onecat_vllm.ops import cuda as K
+    g = torch.Generator().manual_seed(3)
+    md, q, cache, fac, _, _, bias, mix = talk_case(g, [(1, 900), (37, 1300), (1, 33)], 16, 4, 64, torch.bfloat16)
+    outs = []
+    for n in (1, 2, 5, 16):
+        monkeypatch.setattr(K, "plan_talk", lambda *a, n=n: (1, [(True, n, n, 0, 0), (False, n, n, 10, 40)]))
+        md.__dict__.pop("_talk_plans", None)
+        outs.append(ops.talk_attention(q, cache, fac, md, bias.to(DEV), mix.to(DEV), 64).float())
+    assert all(torch.isfinite(o).all() and (o - outs[0]).abs().max() < 0.02 * outs[0].abs().max() for o in outs)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,rows", [(192, 50), (100, 7), (77, 3), (2048, 300)])
+def test_embedding_with_positions(H, rows, dtype):
+    from onecat_vllm import ops
+    g = torch.Generator().manual_seed(H)
+    table, pos = torch.randn(90, H, generator=g).to(dtype), torch.randn(rows, H, generator=g).to(dtype)
+    ids, p = torch.randint(0, 90, (41,), generator=g), torch.randint(0, rows, (41,), generator=g)
+    x, _ = ops.embed_stream(ids.int().to(DEV), table.to(DEV), 1.0, rows=pos.to(DEV), positions=p.int().to(DEV))
+    assert x.dtype == torch.float32 and (x.cpu().double() - table[ids].double() - pos[p].double()).abs().max() < 1e-6
