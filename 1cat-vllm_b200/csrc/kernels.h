@@ -452,7 +452,7 @@ struct TalkTcParams {
   float* ws_ml;                 // [splits][T][H][2] maximum (log2 domain) and sum
   float* ws_o;                  // [mix_splits][T][H][dim], when there is more than one
   int splits, mix_splits, stats_tiles, mix_tiles, short_len;
-  int kt;                       // keys per tile of the second pass, set by the launcher
+  int kt_shift, bs_shift;       // keys per tile of the second pass and tokens per page, as powers of two; set by the launcher
 };
 int talk_tc_launch(const TalkTcParams& p, bool dec, cudaStream_t st);
 

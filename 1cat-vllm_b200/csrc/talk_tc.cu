@@ -79,7 +79,7 @@ __global__ void __launch_bounds__(128) talk_stats_kernel(const TalkTcParams p) {
   pdl_trigger();
   pdl_wait();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3, g = blockIdx.y, split = blockIdx.z;
-  const int hp = p.t.group_rows, share = p.t.H / p.t.G, per = DEC ? 1 : ROWS / hp;
+  const int hp = p.t.group_rows, share = p.t.H / p.t.G, per = DEC ? 1 : ROWS / hp, bs = p.bs_shift, bsm = p.t.bs - 1;
   if (tid == 0) s_w = locate(p, blockIdx.x, per, DEC);
   __syncthreads();
   const Where w = s_w;
@@ -101,11 +101,11 @@ __global__ void __launch_bounds__(128) talk_stats_kernel(const TalkTcParams p) {
         const int kr = e / (DP / 8), c = e % (DP / 8) * 8, key = tile * SK + kr;
         const bool live = key < keys;
         const int at = live ? key : 0;
-        cp_async16(smem_u32(sk + (st * SK + kr) * PD + c), pages + (((size_t)bt[at / p.t.bs] * p.t.G + g) * p.t.bs + at % p.t.bs) * DP + c, live ? 16 : 0);
+        cp_async16(smem_u32(sk + (st * SK + kr) * PD + c), pages + ((((size_t)bt[at >> bs] * p.t.G + g) << bs) + (at & bsm)) * DP + c, live ? 16 : 0);
       }
       if (tid < SK) {
         const int key = tile * SK + tid, at = key < keys ? key : 0;
-        cp_async4(smem_u32(sf + st * SK + tid), p.t.k_scale + (size_t)bt[at / p.t.bs] * p.t.bs + at % p.t.bs, key < keys ? 4 : 0);
+        cp_async4(smem_u32(sf + st * SK + tid), p.t.k_scale + ((size_t)bt[at >> bs] << bs) + (at & bsm), key < keys ? 4 : 0);
       }
     }
     cp_async_commit();
@@ -114,14 +114,14 @@ __global__ void __launch_bounds__(128) talk_stats_kernel(const TalkTcParams p) {
   fetch(first + 1);
   const int row0 = DEC ? 0 : warp * 16;
   float r1[2], r2[2], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-  int pos[2];
+  float pos[2];
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int row = row0 + g8 + 8 * i, h = row % hp, tok = row / hp;
     const bool live = h < share && tok < w.ntok;
     r1[i] = live ? p.t.bias[g * share + h] : 0.f;
     r2[i] = live ? p.t.bias[p.t.H + g * share + h] : 0.f;
-    pos[i] = live ? w.ctx0 + w.tok0 + tok : -1;
+    pos[i] = live ? (float)(w.ctx0 + w.tok0 + tok) : -1.f;
   }
   const uint32_t aq = smem_u32(sq);
   for (int tile = first; tile < last; ++tile) {
@@ -148,15 +148,21 @@ __global__ void __launch_bounds__(128) talk_stats_kernel(const TalkTcParams p) {
       }
     }
     float nm[2] = {m[0], m[1]};
+    const int kr0 = (DEC ? warp * 16 : 0) + 2 * t4;
+    const float k0 = (float)(tile * SK + kr0);
+    const float d0[2] = {pos[0] - k0, pos[1] - k0};   // distance to this lane's first key
 #pragma unroll
-    for (int t = 0; t < NB; ++t)
+    for (int t = 0; t < NB; ++t) {
+      const float2 f = *reinterpret_cast<const float2*>(sf + st * SK + kr0 + t * 8);
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int i = e >> 1, kr = (DEC ? warp * 16 : 0) + t * 8 + 2 * t4 + (e & 1), key = tile * SK + kr;
-        const float s = acc[t][e] * (sf[st * SK + kr] * kLog2e) - r1[i] * lg2(fmaf(r2[i], (float)(pos[i] - key), 1.f));
-        acc[t][e] = key <= pos[i] ? s : -INFINITY;
+        const int i = e >> 1;
+        const float d = d0[i] - (float)(t * 8 + (e & 1));
+        const float s = fmaf(acc[t][e], ((e & 1) ? f.y : f.x) * kLog2e, -r1[i] * lg2(fmaf(r2[i], d, 1.f)));
+        acc[t][e] = d >= 0.f ? s : -INFINITY;
         nm[i] = fmaxf(nm[i], acc[t][e]);
       }
+    }
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       const float base = nm[i] == -INFINITY ? 0.f : nm[i];
@@ -231,7 +237,7 @@ __host__ __device__ inline MixGeom mix_geom(int G, int hp, int pd, int nqb, int 
   m.p = (size_t)nqb * kt * m.pp;
   m.w = (size_t)G * m.rgp * m.pw;
   m.t = (size_t)8 * m.nt * m.pp;
-  m.f = (size_t)2 * kt + nqb * 8 * m.nt + 16 * m.nt + 32;
+  m.f = (size_t)2 * kt + nqb * 8 * m.nt + 16 * m.nt + 32 + 4 * ((size_t)m.nt * (kt / 16) * nqb + (size_t)m.nte * (kt / 16) * nqb);
   return m;
 }
 inline size_t mix_smem(const MixGeom& m, bool pack) { return (2 * m.k + m.q + 2 * m.p + (pack ? 1 : 2) * m.w + m.t) * 2 + m.f * 4; }
@@ -246,7 +252,7 @@ __global__ void __launch_bounds__(MT) talk_mix_kernel(const TalkTcParams p) {
   pdl_trigger();
   pdl_wait();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3, split = blockIdx.y;
-  const int H = p.t.H, G = p.t.G, hp = p.t.group_rows, share = H / G, KT = p.kt;
+  const int H = p.t.H, G = p.t.G, hp = p.t.group_rows, share = H / G, kts = p.kt_shift, KT = 1 << kts, bs = p.bs_shift, bsm = p.t.bs - 1;
   const MixGeom m = mix_geom(G, hp, PD, NQB, KT);
   const bool pack = m.rg < 16;
   const int cols = 8 * m.nt, per = DEC ? 1 : NQB * m.qb;
@@ -263,7 +269,8 @@ __global__ void __launch_bounds__(MT) talk_mix_kernel(const TalkTcParams p) {
   float* slse = sf + 2 * KT;                                   // [NQB][cols]
   float* sr1 = slse + NQB * cols;                              // [cols]
   float* sr2 = sr1 + cols;
-  int* spos = reinterpret_cast<int*>(sr2 + cols);              // [NQB * qb]
+  float* spos = sr2 + cols;                                    // [NQB * qb]
+  int4* units = reinterpret_cast<int4*>(spos + 32);            // what the warps do, for the scores and then for the mix
 
   const int* bt = p.t.block_table + (size_t)w.req * p.t.bt_stride;
   const int keys = w.ctx0 + w.tok0 + w.ntok, tiles = (keys + KT - 1) / KT;
@@ -279,15 +286,16 @@ __global__ void __launch_bounds__(MT) talk_mix_kernel(const TalkTcParams p) {
   auto fetch = [&](int tile) {
     if (tile < last) {
       const int st = tile & 1;
+      const uint32_t dst = smem_u32(sk + st * m.k);
       for (int e = tid; e < G * KT * (DP / 8); e += MT) {
-        const int c = e % (DP / 8) * 8, kr = e / (DP / 8) % KT, g = e / (DP / 8 * KT), key = tile * KT + kr;
+        const int c = e % (DP / 8) * 8, row = e / (DP / 8), kr = row & (KT - 1), g = row >> kts, key = tile * KT + kr;
         const bool live = key < keys;
         const int at = live ? key : 0;
-        cp_async16(smem_u32(sk + st * m.k + (size_t)(g * KT + kr) * PD + c), pages + (((size_t)bt[at / p.t.bs] * G + g) * p.t.bs + at % p.t.bs) * DP + c, live ? 16 : 0);
+        cp_async16(dst + (uint32_t)((row * PD + c) * 2), pages + ((((size_t)bt[at >> bs] * G + g) << bs) + (at & bsm)) * DP + c, live ? 16 : 0);
       }
-      for (int kr = tid; kr < KT; kr += MT) {
-        const int key = tile * KT + kr, at = key < keys ? key : 0;
-        cp_async4(smem_u32(sf + st * KT + kr), p.t.k_scale + (size_t)bt[at / p.t.bs] * p.t.bs + at % p.t.bs, key < keys ? 4 : 0);
+      if (tid < KT) {
+        const int key = tile * KT + tid, at = key < keys ? key : 0;
+        cp_async4(smem_u32(sf + st * KT + tid), p.t.k_scale + ((size_t)bt[at >> bs] << bs) + (at & bsm), key < keys ? 4 : 0);
       }
     }
     cp_async_commit();
@@ -299,7 +307,7 @@ __global__ void __launch_bounds__(MT) talk_mix_kernel(const TalkTcParams p) {
     return h < share ? g * share + h : -1;
   };
   auto token_of = [&](int c) { return hp <= 8 ? c / hp : 0; };
-  for (int i = tid; i < NQB * m.qb; i += MT) spos[i] = i < w.ntok ? w.ctx0 + w.tok0 + i : -1;
+  for (int i = tid; i < NQB * m.qb; i += MT) spos[i] = i < w.ntok ? (float)(w.ctx0 + w.tok0 + i) : -1.f;
   for (int i = tid; i < cols; i += MT) {
     const int h = head_of(i);
     sr1[i] = h >= 0 ? p.t.bias[h] : 0.f;
@@ -329,6 +337,16 @@ __global__ void __launch_bounds__(MT) talk_mix_kernel(const TalkTcParams p) {
     }
     stt[i] = __float2bfloat16(v);
   }
+  const int mts = KT / 16, nu1 = m.nt * mts * (NQB / QPU), nu2 = mts * NQB * (m.nte / NPU);
+  for (int u = tid; u < nu1; u += MT) {   // byte offsets of the key rows and query rows, row in the tile, column, query block
+    const int t = u % m.nt, mt = u / m.nt % mts, qb = u / (m.nt * mts) * QPU, g = t / m.tg, part = t % m.tg;
+    units[u] = make_int4((g * KT + mt * 16) * PD * 2, (g * m.rg + (qb * m.tg + part) * 8) * PD * 2, mt * 16 | t << 16, qb);
+  }
+  for (int u = tid; u < nu2; u += MT) {   // offset of the weights, first column tile, offsets of the stores of its tiles (-1: none)
+    const int mt = u % mts, qb = u / mts % NQB, n0 = u / (mts * NQB) * NPU;
+    auto out = [&](int t) { return t < m.nt ? (((t / m.tg) * m.rgp + (qb * m.tg + t % m.tg) * 8) * m.pw + mt * 16) * 2 : -1; };
+    units[nu1 + u] = make_int4((qb * KT + mt * 16) * m.pp * 2, min(n0, m.nt - 1), out(n0), NPU == 2 ? out(n0 + 1) : -1);
+  }
   if (m.nte != m.nt)   // the columns that round the mix's inner dimension up
     for (int i = tid; i < 2 * NQB * KT * 8; i += MT) sp[(size_t)(i >> 3) * m.pp + cols + (i & 7)] = __float2bfloat16(0.f);
 
@@ -340,111 +358,117 @@ __global__ void __launch_bounds__(MT) talk_mix_kernel(const TalkTcParams p) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[a][t][e] = 0.f;
   const int mtiles = m.rgp / 16, pieces = G * mtiles * DC, piece0 = warp * ACC;
+  uint32_t woff[ACC], koff[ACC];   // byte offsets of a piece's rows of the mixed weights and of its key columns, this lane's address included
+#pragma unroll
+  for (int a = 0; a < ACC; ++a) {
+    const int gm = min(piece0 + a, pieces - 1) / DC, c = min(piece0 + a, pieces - 1) % DC, g = gm / mtiles;
+    woff[a] = a_addr((uint32_t)(g * m.rgp * m.pw * 2), m.pw, gm % mtiles * 16, 0, lane);
+    koff[a] = bkn_addr((uint32_t)(g * KT * PD * 2), PD, 0, c * 16, lane);
+  }
+  const uint32_t aw = smem_u32(sw), aq = smem_u32(sq), ap = smem_u32(sp), plane_p = (uint32_t)(m.p * 2), plane_w = (uint32_t)(m.w * 2);
+  const uint32_t lane_a = a_addr(0, PD, 0, 0, lane), lane_p = a_addr(0, m.pp, 0, 0, lane);
+  // columns of a pair of query blocks, one block above the other
+  const uint32_t lane_q = (uint32_t)((((QPU == 2 ? (lane >> 4) * m.tg * 8 : 0) + (lane & 7)) * PD + ((lane >> 3) & 1) * 8) * 2);
+  const uint32_t lane_t = (uint32_t)(((lane & 7) * m.pp + ((lane >> 3) & 1) * 8) * 2), next_t = NPU == 2 && lane >= 16 ? (uint32_t)(8 * m.pp * 2) : 0;
+  const uint32_t lane_w = (uint32_t)(((lane & 7) * m.pw + ((lane >> 3) & 1) * 8) * 2) + (lane >= 16 ? (pack ? (uint32_t)(8 * m.pw * 2) : plane_w) : 0);
+  const int tk0 = token_of(2 * t4), tk1 = token_of(2 * t4 + 1);
 
   for (int tile = first; tile < last; ++tile) {
     const int st = tile & 1;
     cp_async_wait<0>();
     __syncthreads();   // the tile is there, and every warp is done with the previous one
     fetch(tile + 1);
-    const __nv_bfloat16* kt = sk + st * m.k;
+    const uint32_t ak = smem_u32(sk + st * m.k);
+    const float key0 = (float)(tile * KT);
     // ---- scores and weights
-    for (int u = warp; u < m.nt * (KT / 16) * (NQB / QPU); u += MT / 32) {
-      const int t = u % m.nt, mt = u / m.nt % (KT / 16), qb0 = u / (m.nt * (KT / 16)) * QPU, g = t / m.tg, part = t % m.tg;
-      const uint32_t ak = smem_u32(kt + (size_t)g * KT * PD), aq = smem_u32(sq + (size_t)g * m.rg * PD);
+    for (int u = warp; u < nu1; u += MT / 32) {
+      const int4 un = units[u];
+      const int mt16 = un.z & 0xffff, col = (un.z >> 16) * 8 + 2 * t4;
+      const uint32_t ka = ak + un.x + lane_a, qa = aq + un.y + lane_q;
       float s[QPU][4];
 #pragma unroll
       for (int i = 0; i < QPU; ++i)
 #pragma unroll
         for (int e = 0; e < 4; ++e) s[i][e] = 0.f;
-      const int qrow = ((qb0 + (QPU == 2 ? lane >> 4 : 0)) * m.tg + part) * 8 + (lane & 7);
-      const uint32_t qa = aq + (uint32_t)((qrow * PD + ((lane >> 3) & 1) * 8) * 2);
 #pragma unroll
       for (int ks = 0; ks < DP / 16; ++ks) {
         uint32_t a[4], b[4];
-        ldsm_x4(a, a_addr(ak, PD, mt * 16, ks * 16, lane));
+        ldsm_x4(a, ka + ks * 32);
         if (QPU == 2) ldsm_x4(b, qa + ks * 32);
         else ldsm_x2(b[0], b[1], qa + ks * 32);
 #pragma unroll
         for (int i = 0; i < QPU; ++i) mma16816(s[i], a, b[2 * i], b[2 * i + 1]);
       }
-      const int col = t * 8 + 2 * t4, kr = mt * 16 + g8;
-      const float f0 = sf[st * KT + kr] * kLog2e, f1 = sf[st * KT + kr + 8] * kLog2e;
-      const float ra[2] = {sr1[col], sr1[col + 1]}, rb[2] = {sr2[col], sr2[col + 1]};
+      const int kr = mt16 + g8;
+      const float f[2] = {sf[st * KT + kr] * kLog2e, sf[st * KT + kr + 8] * kLog2e};
+      const float2 ra = *reinterpret_cast<const float2*>(sr1 + col), rb = *reinterpret_cast<const float2*>(sr2 + col);
+      const float key = key0 + (float)kr;
 #pragma unroll
       for (int i = 0; i < QPU; ++i) {
-        const int qb = qb0 + i;
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int key = tile * KT + kr + 8 * (e >> 1), ps = spos[qb * m.qb + token_of(2 * t4 + (e & 1))];
-          const float x = s[i][e] * (e < 2 ? f0 : f1) - ra[e & 1] * lg2(fmaf(rb[e & 1], (float)(ps - key), 1.f)) - slse[qb * cols + col + (e & 1)];
-          s[i][e] = key <= ps ? ex2(x) : 0.f;
-        }
+        const int qb = un.w + i;
+        const float d0 = spos[qb * m.qb + tk0] - key, d1 = spos[qb * m.qb + tk1] - key;
+        const float2 lse = *reinterpret_cast<const float2*>(slse + qb * cols + col);
+        const uint32_t dst = ap + (uint32_t)(((qb * KT + kr) * m.pp + col) * 2);
 #pragma unroll
         for (int hh = 0; hh < 2; ++hh) {
+          const float e0 = d0 - 8.f * hh, e1 = d1 - 8.f * hh;
+          const float x0 = fmaf(s[i][2 * hh], f[hh], -fmaf(ra.x, lg2(fmaf(rb.x, e0, 1.f)), lse.x));
+          const float x1 = fmaf(s[i][2 * hh + 1], f[hh], -fmaf(ra.y, lg2(fmaf(rb.y, e1, 1.f)), lse.y));
           uint32_t hi, lo;
-          split2(s[i][2 * hh], s[i][2 * hh + 1], hi, lo);
-          __nv_bfloat16* d = sp + (size_t)(qb * KT + kr + 8 * hh) * m.pp + col;
-          *reinterpret_cast<uint32_t*>(d) = hi;
-          *reinterpret_cast<uint32_t*>(d + m.p) = lo;
+          split2(e0 >= 0.f ? ex2(x0) : 0.f, e1 >= 0.f ? ex2(x1) : 0.f, hi, lo);
+          const uint32_t at = dst + (uint32_t)(hh * 8 * m.pp * 2);
+          asm volatile("st.shared.b32 [%0], %1;" ::"r"(at), "r"(hi) : "memory");
+          asm volatile("st.shared.b32 [%0], %1;" ::"r"(at + plane_p), "r"(lo) : "memory");
         }
       }
     }
     __syncthreads();   // the weights are there
     // ---- mix over the heads, transposed into rows of the value product
-    for (int u = warp; u < (KT / 16) * NQB * (m.nte / NPU); u += MT / 32) {
-      const int mt = u % (KT / 16), qb = u / (KT / 16) % NQB, n0 = u / (KT / 16 * NQB) * NPU;
-      if (n0 >= m.nt) continue;
-      const uint32_t ph = smem_u32(sp + (size_t)qb * KT * m.pp), pl = ph + (uint32_t)(m.p * 2), tt = smem_u32(stt);
+    for (int u = warp; u < nu2; u += MT / 32) {
+      const int4 un = units[nu1 + u];
+      if (un.z < 0) continue;
+      const uint32_t pa = ap + un.x + lane_p, ta = smem_u32(stt) + (uint32_t)(un.y * 8 * m.pp * 2) + lane_t + (un.w >= 0 ? next_t : 0);
       float x[NPU][4];
 #pragma unroll
       for (int i = 0; i < NPU; ++i)
 #pragma unroll
         for (int e = 0; e < 4; ++e) x[i][e] = 0.f;
-      const int trow = min(n0 * 8 + (NPU == 2 ? (lane >> 4) * 8 : 0), (m.nt - 1) * 8) + (lane & 7);
-      const uint32_t ta = tt + (uint32_t)((trow * m.pp + ((lane >> 3) & 1) * 8) * 2);
+#pragma unroll 4
       for (int ks = 0; ks < m.nte / 2; ++ks) {
         uint32_t a0[4], a1[4], b[4];
-        ldsm_x4(a0, a_addr(ph, m.pp, mt * 16, ks * 16, lane));
-        ldsm_x4(a1, a_addr(pl, m.pp, mt * 16, ks * 16, lane));
+        ldsm_x4(a0, pa + ks * 32);
+        ldsm_x4(a1, pa + plane_p + ks * 32);
         if (NPU == 2) ldsm_x4(b, ta + ks * 32);
         else ldsm_x2(b[0], b[1], ta + ks * 32);
 #pragma unroll
-        for (int i = 0; i < NPU; ++i) {
-          mma16816(x[i], a0, b[2 * i], b[2 * i + 1]);
-          mma16816(x[i], a1, b[2 * i], b[2 * i + 1]);
-        }
+        for (int i = 0; i < NPU; ++i) mma16816(x[i], a0, b[2 * i], b[2 * i + 1]);
+#pragma unroll
+        for (int i = 0; i < NPU; ++i) mma16816(x[i], a1, b[2 * i], b[2 * i + 1]);
       }
 #pragma unroll
       for (int i = 0; i < NPU; ++i) {
-        const int t = n0 + i;
-        if (t >= m.nt) break;
+        const int off = i ? un.w : un.z;
+        if (off < 0) break;
         uint32_t h0, l0, h1, l1;
         split2(x[i][0], x[i][1], h0, l0);
         split2(x[i][2], x[i][3], h1, l1);
-        const int row = (qb * m.tg + t % m.tg) * 8 + (lane & 7);
-        __nv_bfloat16* d = sw + (size_t)((t / m.tg) * m.rgp + row) * m.pw + mt * 16 + ((lane >> 3) & 1) * 8;
-        if (lane >= 16) d += pack ? (size_t)8 * m.pw : m.w;
-        stsm_x4_t(smem_u32(d), h0, h1, l0, l1);
+        stsm_x4_t(aw + off + lane_w, h0, h1, l0, l1);
       }
     }
     __syncthreads();
     // ---- values
-    for (int ks = 0; ks < KT / 16; ++ks) {
+#pragma unroll 2
+    for (int ks = 0; ks < mts; ++ks) {
       uint32_t a0[4], a1[4];
-      int have = -1;
 #pragma unroll
       for (int a = 0; a < ACC; ++a) {
-        const int piece = piece0 + a;
-        if (piece >= pieces) break;
-        const int gm = piece / DC, c = piece % DC, g = gm / mtiles, r0 = gm % mtiles * 16;
-        if (gm != have) {
-          const uint32_t wa = smem_u32(sw + (size_t)g * m.rgp * m.pw);
-          ldsm_x4(a0, a_addr(wa, m.pw, r0, ks * 16, lane));
-          if (!pack) ldsm_x4(a1, a_addr(wa + (uint32_t)(m.w * 2), m.pw, r0, ks * 16, lane));
-          have = gm;
+        if (piece0 + a >= pieces) break;
+        if (a == 0 || woff[a] != woff[a - 1]) {
+          ldsm_x4(a0, aw + woff[a] + ks * 32);
+          if (!pack) ldsm_x4(a1, aw + plane_w + woff[a] + ks * 32);
         }
         uint32_t b[4];
-        ldsm_x4_t(b, bkn_addr(smem_u32(kt + (size_t)g * KT * PD), PD, ks * 16, c * 16, lane));
+        ldsm_x4_t(b, ak + koff[a] + (uint32_t)(ks * 16 * PD * 2));
         mma16816(acc[a][0], a0, b[0], b[1]);
         mma16816(acc[a][1], a0, b[2], b[3]);
         if (!pack) {
@@ -556,7 +580,7 @@ int mix_go(const TalkTcParams& p, int blocks, cudaStream_t st) {
     if (allow(talk_mix_kernel<DP, NQB, ACC>)) return -4;
     configured = true;
   }
-  const MixGeom m = mix_geom(p.t.G, p.t.group_rows, DP + 8, NQB, p.kt);
+  const MixGeom m = mix_geom(p.t.G, p.t.group_rows, DP + 8, NQB, 1 << p.kt_shift);
   launch_k(talk_mix_kernel<DP, NQB, ACC>, dim3((unsigned)blocks, (unsigned)p.mix_splits), dim3(MT), mix_smem(m, m.rg < 16), st, true, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
 }
@@ -565,8 +589,10 @@ template <int DP>
 int run(TalkTcParams p, bool dec, cudaStream_t st) {
   const int hp = p.t.group_rows, nqb = dec ? 1 : prefill_blocks(p.t.G, hp, DP);
   int acc;
-  p.kt = mix_tile(p.t.G, hp, DP, nqb, acc);
-  if (p.kt == 0) return -3;
+  const int kt = mix_tile(p.t.G, hp, DP, nqb, acc);
+  if (kt == 0) return -3;
+  p.kt_shift = __builtin_ctz((unsigned)kt);
+  p.bs_shift = __builtin_ctz((unsigned)p.t.bs);
   int rc = dec ? stats_go<DP, true>(p, p.t.R, st) : stats_go<DP, false>(p, p.stats_tiles, st);
   if (rc) return rc;
   const int blocks = dec ? p.t.R : p.mix_tiles;
@@ -601,7 +627,7 @@ bool talk_tc_sizes(int H, int G, int dim, TalkSizes* s) {
 int talk_tc_launch(const TalkTcParams& p, bool dec, cudaStream_t st) {
   TalkSizes s;
   if (p.t.T == 0) return 0;
-  if (!talk_tc_sizes(p.t.H, p.t.G, p.t.dim, &s) || s.row != p.t.row || s.group_rows != p.t.group_rows || p.t.f32 || p.splits < 1 || p.mix_splits < 1 ||
+  if (!talk_tc_sizes(p.t.H, p.t.G, p.t.dim, &s) || s.row != p.t.row || s.group_rows != p.t.group_rows || p.t.f32 || (p.t.bs & (p.t.bs - 1)) || p.splits < 1 || p.mix_splits < 1 ||
       p.short_len != s.short_len || (dec && s.short_len == 0) || p.ws_ml == nullptr || (p.mix_splits > 1 && p.ws_o == nullptr)) return -1;
   return p.t.row == 64 ? run<64>(p, dec, st) : run<128>(p, dec, st);
 }

@@ -1,6 +1,6 @@
 """Prefill and decode throughput of a design beside the closest models of equal size, and its kernels beside theirs.
 
-``python bench.py --design gabisun|sepirax|lodevik`` prints one JSON line per size. Random weights and token ids. Model throughput is device time
+``python bench.py --design gabisun|sepirax|lodevik|nalasun`` prints one JSON line per size. Random weights and token ids. Model throughput is device time
 of engine steps (CUDA events); kernels are timed alone with the L2 flushed before every launch.
 
 Gabisun: the models share width, heads, head size, window, layer runs, vocabulary and tied embeddings: Starcoder2 (layer norms, ungated
@@ -13,7 +13,11 @@ attention, the same experts without groups).
 
 Lodevik: beside Gemma-2 (soft-capped attention with one map of the same number of columns, a window of the chunk's size in every other layer,
 full attention in the rest, gated GELU, norms ahead of and behind the sub-blocks) and a dense DeepSeek-V2 (every layer latent attention with
-the same heads and latents, gated SiLU)."""
+the same heads and latents, gated SiLU).
+
+Nalasun (talking-heads attention, channel delta rule and Mamba-2 in turn): beside Qwen3-Next (Gated-DeltaNet in two of three layers, softmax
+attention with the same heads in the third, the same experts and shared expert) and Granite 4 hybrid (Mamba-2 in two of three layers, softmax attention in
+the third, the same experts and shared expert). Kernels of the attention layers also beside Gabisun's, whose values are its keys as well."""
 from __future__ import annotations
 
 import gc
@@ -402,6 +406,164 @@ def lodevik_kernels(s: dict, iters: int) -> list[dict]:
     gemm("logits", "lodevik, fp32 output", VOCAB, W, out_dtype=torch.float32)
     gemm("logits", "bf16 output", VOCAB, W)
     return rows
+
+
+NALASUN_SIZES = {
+    # width, layers (attention, channel delta, Mamba-2 in turn), attention (heads, kv heads, dim), delta rule (heads, dim), Mamba-2 (heads, vdim, state,
+    # groups), experts (count, chosen, width, shared width)
+    "w2048": dict(width=2048, layers=12, heads=16, kv=4, dim=128, dheads=16, ddim=128, mheads=64, mdim=64, state=128, groups=1, experts=64, top=6, ff=512, shared=1024),
+    "w4096": dict(width=4096, layers=9, heads=32, kv=8, dim=128, dheads=32, ddim=128, mheads=128, mdim=64, state=128, groups=8, experts=64, top=4, ff=1024, shared=2048),
+    "w2048s": dict(width=2048, layers=12, heads=32, kv=8, dim=64, dheads=32, ddim=64, mheads=32, mdim=64, state=64, groups=2, experts=64, top=6, ff=512, shared=1024),
+}
+
+
+def nalasun_config(s: dict) -> dict:
+    mlp = dict(kind="moe", expert=dict(ff=s["ff"]), shared=dict(ff=s["shared"]), router=dict(experts=s["experts"], top=s["top"], scale=2.0))
+    att = dict(type="attention", mlp=mlp, mixer=dict(heads=s["heads"], kv_heads=s["kv"], dim=s["dim"], vdim=s["dim"], scale=s["dim"] ** -0.5, q_temp=dict(coef=0.1, every=4096)))
+    dlt = dict(type="channel_delta", mlp=mlp, mixer=dict(heads=s["dheads"], kv_heads=s["dheads"], dim=s["ddim"], vdim=s["ddim"], conv=4))
+    ssm = dict(type="mamba2", mlp=mlp, mixer=dict(heads=s["mheads"], vdim=s["mdim"], state=s["state"], groups=s["groups"], norm_groups=s["groups"], conv=4))
+    return dict(architecture="Nalasun", width=s["width"], vocab=VOCAB, max_positions=2 * PREFILL, norm=dict(eps=1e-5), canon=dict(taps=4),
+                layers=[att, dlt, ssm] * (s["layers"] // 3))
+
+
+def nalasun_like(s: dict, arch: str) -> dict:
+    cfg = dict(architectures=[arch], hidden_size=s["width"], num_hidden_layers=s["layers"], num_attention_heads=s["heads"], num_key_value_heads=s["kv"],
+               head_dim=s["dim"], vocab_size=VOCAB, max_position_embeddings=32768, rope_theta=10000.0, rms_norm_eps=1e-5, tie_word_embeddings=True,
+               num_experts_per_tok=s["top"])
+    if arch.startswith("Granite"):
+        return dict(cfg, layer_types=["attention", "mamba", "mamba"] * (s["layers"] // 3), mamba_n_heads=s["mheads"], mamba_d_head=s["mdim"], mamba_d_state=s["state"],
+                    mamba_n_groups=s["groups"], mamba_d_conv=4, mamba_expand=s["mheads"] * s["mdim"] / s["width"], intermediate_size=s["ff"],
+                    shared_intermediate_size=s["shared"], num_local_experts=s["experts"], attention_multiplier=s["dim"] ** -0.5, embedding_multiplier=1.0,
+                    residual_multiplier=1.0, logits_scaling=1.0, position_embedding_type="nope")
+    return dict(cfg, intermediate_size=s["ff"], moe_intermediate_size=s["ff"], norm_topk_prob=True, num_experts=s["experts"],
+                shared_expert_intermediate_size=s["shared"], linear_num_key_heads=s["dheads"], linear_num_value_heads=s["dheads"], linear_key_head_dim=128,
+                linear_value_head_dim=128, linear_conv_kernel_dim=4, full_attention_interval=3, attn_output_gate=True, partial_rotary_factor=0.25)
+
+
+def nalasun_kernels(s: dict, iters: int) -> list[dict]:
+    """Each kernel of the design beside the like kernel of the closest models. Bytes and FLOPs are the algorithm's: every input read and every output
+    written once, and for attention the score, mix and value products over the visible pairs."""
+    from types import SimpleNamespace
+    from onecat_vllm.ops import cuda as K
+    from onecat_vllm.ops import ref
+    from onecat_vllm.ops.microbench import _peaks, timeit
+    pk, rows = _peaks(), []
+    W, H, G, D, E, top = s["width"], s["heads"], s["kv"], s["dim"], s["experts"], s["top"]
+    b = lambda *sh: torch.randn(*sh, device="cuda").bfloat16()
+    f32 = lambda *sh: torch.randn(*sh, device="cuda")
+
+    def row(kernel, case, who, fn, flops=0.0, nbytes=0.0, n=iters):
+        ms = timeit(fn, n)
+        t = max(flops / pk["bf16_tflops"] / 1e9, nbytes / pk["hbm_gbs"] / 1e6)
+        rows.append(dict(kernel=kernel, case=case, model=who, us=ms * 1e3, roofline_us=t * 1e3, frac_of_roofline=t / ms))
+
+    wide, (_, hp, *_) = K.talk_row(H, G, D), K._C.talk_sizes(H, G, D)
+    for case, n, q, S in (("prefill", 1, PREFILL, PREFILL), ("decode", DECODE_REQS, 1, DECODE_CTX)):
+        T = n * q
+        md, nblk = _meta(n, q, S)
+        md.is_uniform_decode = case == "decode"
+        pairs = n * sum(range(S - q + 1, S + 1))
+        cache, fac, qq, bias, mix = b(nblk, 1, G, 16, wide) * 0.5, torch.ones(nblk, 16, device="cuda"), b(T, G * hp, wide) * 0.1, torch.rand(2, H, device="cuda"), b(H, H) * 0.2
+        cost = lambda mixed, tensors: (2.0 * H * pairs * (2 * D + (H if mixed else 0)), 2.0 * (n * S * G * D * tensors + 2 * T * H * D))
+        row("attention", case, "nalasun, shared keys, mixed heads", lambda: K.talk_attention(qq, cache, fac, md, bias, mix, D), *cost(True, 1))
+        x, out, table = b(T, H, D), torch.empty(T, H, D, dtype=torch.bfloat16, device="cuda"), f32(H, BIAS_MAX + 1)
+        row("attention", case, "gabisun, shared keys, distance bias", lambda: K.paged_attention(x, cache, md, D ** -0.5, out=out, bias_table=table), *cost(False, 1))
+        del cache
+        md.attn_plan = None
+        kv = b(nblk, 2, G, 16, D) * 0.5
+        row("attention", case, "qwen3-next, plain", lambda: K.paged_attention(x, kv, md, D ** -0.5, out=out), *cost(False, 2))
+        del kv
+    for case, n, q in (("prefill", 1, PREFILL), ("decode", DECODE_REQS, 1)):
+        T = n * q
+        md, _ = _meta(n, q, q)
+        md.state_slots = torch.arange(n, device="cuda", dtype=torch.int32)
+        md.has_initial_state = torch.ones(n, device="cuda", dtype=torch.int32)
+        md.is_uniform_decode = case == "decode"
+        cx, cw, cs = b(T, W), b(W, 4), b(n, 3, W)
+        row("input convolution", case, "nalasun", lambda: K.causal_conv(cx, cw, None, cs, md, False, True), nbytes=4.0 * T * W + 12.0 * n * W)
+        # matrix states: the products of the chunked form with 64 tokens (two with the state, one inside the chunk), or the state's traffic
+        cost = lambda h, d, v, extra: (4.0 * T * h * (d * v + 32 * (d + v)), 2.0 * T * h * (2 * d + 3 * v) + extra + 8.0 * n * h * d * v)
+        h, d = s["dheads"], s["ddim"]
+        x, a, st, wt, gate, nw, conv = b(T, 3 * h * d + h), f32(T, h * d), f32(n, h, d, d), b(3 * h * d, 4), b(T, h * d), b(d), b(n, 3, 3 * h * d)
+        al, dtb = f32(h), f32(h * d)
+
+        def delta():
+            y = K.causal_conv(x[:, : 3 * h * d], wt, None, conv, md, True, False)
+            return K.gated_norm(K.channel_delta(y, a, x[:, 3 * h * d:], al, dtb, st, md, h, h, d, d), gate, nw, 1e-5, h, False)
+        row("recurrence", case, f"nalasun channel delta {d}x{d} with convolution, head norm and gate", delta, *cost(h, d, d, 4.0 * T * h * d))
+        y = K.causal_conv(x[:, : 3 * h * d], wt, None, conv, md, True, False)
+        row("recurrence", case, f"nalasun channel delta {d}x{d} alone", lambda: K.channel_delta(y, a, x[:, 3 * h * d:], al, dtb, st, md, h, h, d, d), *cost(h, d, d, 4.0 * T * h * d))
+        gc_, gs, gx, ga, gw, gz, gn = b(n, 3 * h * 128, 3), f32(n, h, 128, 128), b(T, 3 * h * 128), b(T, h), b(3 * h * 128, 4), b(T, h * 128), b(128)
+        row("recurrence", case, "qwen3-next Gated-DeltaNet 128x128 with convolution, head norm and gate", lambda: K.rms_norm_gated(
+            K.gdn_forward(gx, ga, ga, gw, al, al, gc_, gs, md, h, h, 128, 128).reshape(T, h * 128), gz, gn, 1e-5, h), *cost(h, 128, 128, 0.0))
+        mh, mv, N, mg = s["mheads"], s["mdim"], s["state"], s["groups"]
+        inner, ch = mh * mv, mh * mv + 2 * mg * N
+        mx, mw, mb, mc, ms, mn = b(T, inner + ch + mh), b(ch, 4), b(ch), b(n, 3, ch), f32(n, mh, N, mv), b(inner)
+        mal, mdt, msk = f32(mh), f32(mh), f32(mh)
+        mcost = (4.0 * T * mh * (N * mv + 32 * mv) + 4.0 * T * mg * 32 * N, 2.0 * T * (3 * inner + 2 * mg * N) + 8.0 * n * mh * N * mv)
+
+        def ssm():
+            y = K.causal_conv(mx[:, inner: inner + ch], mw, mb, mc, md, True, False)
+            return K.gated_norm(K.mamba2(y, mx[:, inner + ch:], mal, mdt, msk, ms, md, mh, mg, N, mv, (0.0, float("inf"))), mx[:, :inner], mn, 1e-5, mg, True)
+        row("recurrence", case, f"nalasun Mamba-2 {N}x{mv} x {mh} with convolution, gate and norm", ssm, *mcost)
+        my = K.causal_conv(mx[:, inner: inner + ch], mw, mb, mc, md, True, False)
+        row("recurrence", case, f"nalasun Mamba-2 {N}x{mv} x {mh} alone", lambda: K.mamba2(my, mx[:, inner + ch:], mal, mdt, msk, ms, md, mh, mg, N, mv, (0.0, float("inf"))), *mcost)
+        row("recurrence", case, f"Mamba-2 {N}x{mv} x {mh} alone as PyTorch operations", lambda: ref.mamba2(my, mx[:, inner + ch:], mal, mdt, msk, ms, md, mh, mg, N, mv), *mcost, n=3)
+        go = b(T, h * d)
+        row("gated norm", case, "nalasun, sigmoid gate", lambda: K.gated_norm(go, gate, nw, 1e-5, h, False), nbytes=6.0 * T * h * d)
+        row("gated norm", case, "nalasun, SiLU gate ahead", lambda: K.gated_norm(mx[:, :inner], mx[:, inner: 2 * inner], mn, 1e-5, mg, True), nbytes=6.0 * T * inner)
+        row("gated norm", case, "qwen3-next", lambda: K.rms_norm_gated(gz, gx[:, : h * 128], gn, 1e-5, h), nbytes=6.0 * T * h * 128)
+    for T in (PREFILL, DECODE_REQS):
+        part, x32, w, res = b(T, W), f32(T, W), b(W), b(T, W)
+        row("norm", T, "nalasun join", lambda: K.stream_join(part, x32, None, None, (1, w, None, 1e-5, False), torch.bfloat16), nbytes=12.0 * T * W)
+        row("norm", T, "add + rms norm", lambda: K.rms_norm(part, w, 1e-5, res, False), nbytes=8.0 * T * W)
+        slot = torch.arange(T, device="cuda", dtype=torch.int32)
+        ids, emb, pos = torch.randint(0, VOCAB, (T,), device="cuda", dtype=torch.int32), b(VOCAB, W), b(2 * PREFILL, W)
+        row("embedding", T, "nalasun, token and position rows", lambda: K.embed_stream(ids, emb, 1.0, None, None, (0, 0), torch.bfloat16, rows=pos, positions=slot), nbytes=8.0 * T * W)
+        row("embedding", T, "qwen3-next (PyTorch)", lambda: torch.nn.functional.embedding(ids, emb), nbytes=4.0 * T * W)
+        qk, gain, cache, fac = b(T, (H + G) * D), f32(H * D), b(T // 16 + 1, 1, G, 16, wide), f32(T // 16 + 1, 16)
+        row("norms + insert", T, "nalasun", lambda: K.talk_prepare(qk, gain, 1e-5, (0.1, 4096), slot, cache, fac, slot, H, G, D), nbytes=4.0 * T * (H + G) * D)
+        k2, c2, cs2, nw2 = b(T, (H + 2 * G) * D), b(T // 16 + 1, 2, G, 16, D), torch.ones(T, D, device="cuda"), b(D)
+        row("norms + insert", T, "qwen3", lambda: K.rope_and_cache(k2[:, : H * D].view(T, H, D), k2[:, H * D: (H + G) * D].view(T, G, D), k2[:, (H + G) * D:].view(T, G, D),
+                                                                 slot, cs2, c2, slot, D, nw2, nw2, 1e-5, False), nbytes=4.0 * T * (H + 2 * G) * D)
+        rc = SimpleNamespace(num_experts_per_tok=top, n_group=1, topk_group=1, scoring_func="sigmoid", norm_topk_prob=False, routed_scaling_factor=2.0)
+        z, zero = f32(T, E), torch.zeros(E, device="cuda")
+        row("router", T, "nalasun (sigmoid, fp32 logits)", lambda: K.route(z, rc, zero), nbytes=T * (4.0 * E + 8.0 * top))
+        rq, zb = SimpleNamespace(num_experts_per_tok=top, n_group=1, topk_group=1, scoring_func="softmax", norm_topk_prob=True, routed_scaling_factor=1.0), z.bfloat16()
+        row("router", T, "qwen3-next (softmax, bf16 logits)", lambda: K.route(zb, rq, None), nbytes=T * (2.0 * E + 8.0 * top))
+
+        def gemm(name, who, N, Kd, **kw):
+            wt, xx = (torch.randn(N, Kd, device="cuda") * 0.02).bfloat16(), b(T, Kd)
+            out = torch.empty(T, -(-N // 8) * 8, dtype=kw.get("out_dtype", torch.bfloat16), device="cuda")[:, :N]
+            row(f"gemm {name}", T, who, lambda: K._gemm(xx, wt, None, None, out, None, N, N, N, 0, K.EPI_STORE, 1), flops=2.0 * T * N * Kd,
+                nbytes=2.0 * (N * Kd + T * Kd) + out.element_size() * T * N)
+        h, d = s["dheads"], s["ddim"]
+        gemm("mixer input", "nalasun q|k", (H + G) * D, W)
+        gemm("mixer input", "nalasun delta q|k|v|a|g|b", 3 * h * d + 2 * d + h, W)
+        gemm("mixer input", "nalasun Mamba-2", 2 * s["mheads"] * s["mdim"] + 2 * s["groups"] * s["state"] + s["mheads"], W)
+        gemm("mixer input", "qwen3-next q|k|v|z", 4 * h * 128, W)
+        gemm("low rank", "nalasun decays, fp32 output", h * d, d, out_dtype=torch.float32)
+        gemm("low rank", "nalasun gate", h * d, d)
+        gemm("router logits", "nalasun, fp32 output", E, W, out_dtype=torch.float32)
+        gemm("router logits", "qwen3-next", E, W)
+    return rows
+
+
+def run_nalasun(steps: int, warmup: int, sizes=None, kernels: bool = True, clock_sampler=None) -> None:
+    for name, s in NALASUN_SIZES.items():
+        if sizes and name not in sizes:
+            continue
+        clocks = clock_sampler() if clock_sampler else None
+        models = {"Nalasun": nalasun_config(s), "Qwen3-Next": nalasun_like(s, "Qwen3NextForCausalLM"), "Granite 4 hybrid": nalasun_like(s, "GraniteMoeHybridForCausalLM")}
+        res = {"design": "nalasun", "size": name, "dims": s, "dtype": "bf16", "data": "synthetic: random token ids and weights",
+               "workload": f"prefill: one {PREFILL}-token prompt a step; decode: {DECODE_REQS} requests at a context of about {DECODE_CTX}",
+               "l2": "model steps stream weights and caches larger than L2; kernels: L2 flushed before every launch",
+               "models": {k: model_throughput(m, steps, warmup) for k, m in models.items()}}
+        if kernels:
+            res["kernels"] = nalasun_kernels(s, max(5, steps // 6))
+        if clocks is not None:
+            res["clocks"] = clocks.stop()
+        print(json.dumps(res), flush=True)
 
 
 def run_lodevik(steps: int, warmup: int, sizes=None, kernels: bool = True, clock_sampler=None) -> None:

@@ -248,12 +248,13 @@ def main() -> None:
     ap.add_argument("--eager", action="store_true")
     ap.add_argument("--no-full", action="store_true", help="skip the full-workload pass (4 x concurrency requests, ramp-up and tail) after the timed steps")
     ap.add_argument("--no-async", action="store_true", help="plain schedule-run-update order instead of async scheduling (one step kept in flight)")
-    ap.add_argument("--design", default=None, choices=["gabisun", "sepirax", "lodevik"], help="instead of the headline workload: throughput of this design beside like models of equal size")
+    ap.add_argument("--design", default=None, choices=["gabisun", "sepirax", "lodevik", "nalasun"], help="instead of the headline workload: throughput of this design beside like models of equal size")
     ap.add_argument("--design-size", nargs="*", default=None, help="with --design: only these sizes")
     args = ap.parse_args()
     if args.design:
         from onecat_vllm.entrypoints import bench_design
-        run = {"gabisun": bench_design.run, "sepirax": bench_design.run_sepirax, "lodevik": bench_design.run_lodevik}[args.design]
+        run = {"gabisun": bench_design.run, "sepirax": bench_design.run_sepirax, "lodevik": bench_design.run_lodevik,
+               "nalasun": bench_design.run_nalasun}[args.design]
         run(args.steps, max(args.warmup, 3), args.design_size, clock_sampler=lambda: ClockSampler(0))
         return
     if args.impl == "reference":
