@@ -1162,20 +1162,20 @@ torch::Tensor gated_norm(torch::Tensor x, torch::Tensor gate, torch::Tensor w, d
 }
 
 torch::Tensor talk_prepare(torch::Tensor qk, torch::Tensor gain, double eps, double coef, int64_t every, torch::Tensor positions, torch::Tensor pages,
-                           torch::Tensor k_scale, torch::Tensor slots, int64_t H, int64_t G, int64_t dim, int64_t group_rows) {
+                           torch::Tensor k_scale, torch::Tensor slots, int64_t H, int64_t G, int64_t dim) {
   const auto et = qk.scalar_type();
   TORCH_CHECK(qk.is_cuda() && (et == torch::kBFloat16 || et == torch::kFloat32) && qk.dim() == 2 && qk.stride(1) == 1 && qk.size(1) == (H + G) * dim, "q|k must be [T, (H + G) dim]");
   const int64_t T = qk.size(0), row = pages.size(4), bs = pages.size(3);
   TORCH_CHECK(pages.scalar_type() == et && pages.is_contiguous() && pages.dim() == 5 && pages.size(1) == 1 && pages.size(2) == G && row >= dim, "pages must be [blocks, 1, G, bs, row]");
   TORCH_CHECK(k_scale.scalar_type() == torch::kFloat32 && k_scale.is_contiguous() && k_scale.numel() == pages.size(0) * bs, "key factors must be fp32 [blocks, bs]");
-  TORCH_CHECK(gain.scalar_type() == torch::kFloat32 && gain.is_contiguous() && gain.numel() == H * dim && group_rows * G >= H, "gain must be fp32 [H dim]");
+  TORCH_CHECK(gain.scalar_type() == torch::kFloat32 && gain.is_contiguous() && gain.numel() == H * dim, "gain must be fp32 [H dim]");
   for (auto* t : {&positions, &slots}) TORCH_CHECK(t->scalar_type() == torch::kInt32 && t->is_contiguous() && t->numel() >= T, "positions and slots must be int32 [T]");
   const c10::cuda::CUDAGuard guard(qk.device());
-  auto q = torch::empty({T, G * group_rows, row}, qk.options());
+  auto q = torch::empty({T, H, row}, qk.options());
   oc::TalkPrepareParams p{};
   p.qk = qk.data_ptr(); p.ld = qk.stride(0); p.gain = gain.data_ptr<float>(); p.eps = (float)eps; p.coef = (float)coef; p.every = (int)every;
   p.positions = positions.data_ptr<int>(); p.slots = slots.data_ptr<int>(); p.q_out = q.data_ptr(); p.pages = pages.data_ptr(); p.k_scale = k_scale.data_ptr<float>();
-  p.T = (int)T; p.H = (int)H; p.G = (int)G; p.dim = (int)dim; p.group_rows = (int)group_rows; p.row = (int)row; p.bs = (int)bs; p.f32 = et == torch::kFloat32;
+  p.T = (int)T; p.H = (int)H; p.G = (int)G; p.dim = (int)dim; p.row = (int)row; p.bs = (int)bs; p.f32 = et == torch::kFloat32;
   TORCH_CHECK(oc::talk_prepare_launch(p, cur_stream()) == 0, "talk_prepare failed");
   return q;
 }
@@ -1184,7 +1184,7 @@ static oc::TalkParams talk_params(const torch::Tensor& q, const torch::Tensor& p
                                   const torch::Tensor& out, const torch::Tensor& qsl, const torch::Tensor& seq_lens, const torch::Tensor& bt, int64_t H, int64_t dim) {
   const auto et = q.scalar_type();
   const int64_t G = pages.size(2), row = pages.size(4);
-  TORCH_CHECK(q.is_cuda() && q.is_contiguous() && q.dim() == 3 && q.size(2) == row && q.size(1) % G == 0 && q.size(1) >= H && H % G == 0, "q must be [T, G group_rows, row]");
+  TORCH_CHECK(q.is_cuda() && q.is_contiguous() && q.dim() == 3 && q.size(2) == row && q.size(1) == H && H % G == 0, "q must be [T, H, row]");
   TORCH_CHECK(pages.scalar_type() == et && pages.is_contiguous() && pages.dim() == 5 && pages.size(1) == 1, "pages must be [blocks, 1, G, bs, row]");
   TORCH_CHECK(k_scale.scalar_type() == torch::kFloat32 && k_scale.is_contiguous() && bias.scalar_type() == torch::kFloat32 && bias.is_contiguous() && bias.numel() == 2 * H, "key factors and bias must be fp32");
   TORCH_CHECK(mix.scalar_type() == et && mix.is_contiguous() && mix.numel() == H * H, "mix must be [H, H]");
@@ -1195,41 +1195,50 @@ static oc::TalkParams talk_params(const torch::Tensor& q, const torch::Tensor& p
   p.q = q.data_ptr(); p.pages = pages.data_ptr(); p.mix = mix.data_ptr(); p.k_scale = k_scale.data_ptr<float>(); p.bias = bias.data_ptr<float>();
   p.out = out.data_ptr(); p.query_start_loc = qsl.data_ptr<int>(); p.seq_lens = seq_lens.data_ptr<int>(); p.block_table = bt.data_ptr<int>();
   p.bt_stride = (int)bt.stride(0); p.T = (int)q.size(0); p.R = (int)seq_lens.numel(); p.H = (int)H; p.G = (int)G; p.dim = (int)dim;
-  p.group_rows = (int)(q.size(1) / G); p.row = (int)row; p.bs = (int)pages.size(3); p.f32 = et == torch::kFloat32;
+  p.row = (int)row; p.bs = (int)pages.size(3); p.f32 = et == torch::kFloat32;
   return p;
 }
 
 void talk_plain(torch::Tensor q, torch::Tensor pages, torch::Tensor k_scale, torch::Tensor bias, torch::Tensor mix, torch::Tensor out, torch::Tensor qsl,
                 torch::Tensor seq_lens, torch::Tensor bt, int64_t H, int64_t dim) {
   auto p = talk_params(q, pages, k_scale, bias, mix, out, qsl, seq_lens, bt, H, dim);
-  TORCH_CHECK(p.row == p.dim && p.group_rows * p.G == p.H, "the plain kernel takes unpadded rows");
+  TORCH_CHECK(p.row == p.dim, "the plain kernel takes unpadded rows");
   const c10::cuda::CUDAGuard guard(q.device());
   const int rc = oc::talk_plain_launch(p, cur_stream());
   TORCH_CHECK(rc == 0, "talk_plain failed: ", rc);
 }
 
-// (cached row, query rows per key head, tokens per block of the two passes, longest portion of the single-token variant); empty: plain kernel
-std::vector<int64_t> talk_sizes(int64_t H, int64_t G, int64_t dim) {
-  oc::TalkSizes s;
-  if (!oc::talk_tc_sizes((int)H, (int)G, (int)dim, &s)) return {};
-  return {s.row, s.group_rows, s.stats_tokens, s.mix_tokens, s.short_len};
-}
-
-void talk_tc(torch::Tensor q, torch::Tensor pages, torch::Tensor k_scale, torch::Tensor bias, torch::Tensor mix, torch::Tensor out, torch::Tensor qsl,
-             torch::Tensor seq_lens, torch::Tensor bt, int64_t H, int64_t dim, bool dec, int64_t short_len, int64_t splits, int64_t mix_splits, int64_t stats_tiles,
-             int64_t mix_tiles, torch::Tensor ws_ml, c10::optional<torch::Tensor> ws_o) {
+static oc::TalkTcParams talk_tc_params(const torch::Tensor& q, const torch::Tensor& pages, const torch::Tensor& k_scale, const torch::Tensor& bias,
+                                       const torch::Tensor& mix, const torch::Tensor& out, const torch::Tensor& qsl, const torch::Tensor& seq_lens, const torch::Tensor& bt,
+                                       int64_t H, int64_t dim, int64_t rows, const torch::Tensor& ws_ml, const torch::Tensor& ws_o) {
   oc::TalkTcParams p{};
   p.t = talk_params(q, pages, k_scale, bias, mix, out, qsl, seq_lens, bt, H, dim);
-  const int64_t T = p.t.T;
   TORCH_CHECK(!p.t.f32 && ((uintptr_t)p.t.q & 15) == 0 && ((uintptr_t)p.t.pages & 15) == 0, "bf16 rows on 16-byte boundaries");
-  TORCH_CHECK(ws_ml.scalar_type() == torch::kFloat32 && ws_ml.numel() >= splits * T * H * 2, "workspace of the sums");
-  if (mix_splits > 1) TORCH_CHECK(ws_o.has_value() && ws_o->scalar_type() == torch::kFloat32 && ws_o->numel() >= mix_splits * T * H * dim, "workspace of the outputs");
+  TORCH_CHECK(ws_ml.scalar_type() == torch::kFloat32 && ws_ml.numel() >= rows * H * 2, "workspace of the sums");
+  TORCH_CHECK(ws_o.scalar_type() == torch::kFloat32 && ws_o.numel() >= rows * H * pages.size(2) * pages.size(4), "workspace of the results");
   p.ws_ml = ws_ml.data_ptr<float>();
-  p.ws_o = mix_splits > 1 ? ws_o->data_ptr<float>() : nullptr;
-  p.splits = (int)splits; p.mix_splits = (int)mix_splits; p.stats_tiles = (int)stats_tiles; p.mix_tiles = (int)mix_tiles; p.short_len = (int)short_len;
+  p.ws_o = ws_o.data_ptr<float>();
+  p.min_len = 2;
+  return p;
+}
+
+void talk_decode(torch::Tensor q, torch::Tensor pages, torch::Tensor k_scale, torch::Tensor bias, torch::Tensor mix, torch::Tensor out, torch::Tensor qsl,
+                 torch::Tensor seq_lens, torch::Tensor bt, int64_t H, int64_t dim, int64_t splits, torch::Tensor ws_ml, torch::Tensor ws_o) {
+  auto p = talk_tc_params(q, pages, k_scale, bias, mix, out, qsl, seq_lens, bt, H, dim, splits * seq_lens.numel(), ws_ml, ws_o);
+  p.splits = (int)splits;
   const c10::cuda::CUDAGuard guard(q.device());
-  const int rc = oc::talk_tc_launch(p, dec, cur_stream());
-  TORCH_CHECK(rc == 0, "talk_tc failed: ", rc);
+  const int rc = oc::talk_decode_launch(p, cur_stream());
+  TORCH_CHECK(rc == 0, "talk_decode failed: ", rc);
+}
+
+// tiles: 128-token tiles over the portions of at least two tokens
+void talk_prefill(torch::Tensor q, torch::Tensor pages, torch::Tensor k_scale, torch::Tensor bias, torch::Tensor mix, torch::Tensor out, torch::Tensor qsl,
+                  torch::Tensor seq_lens, torch::Tensor bt, int64_t H, int64_t dim, int64_t tiles, int64_t segment, torch::Tensor ws_ml, torch::Tensor ws_o) {
+  auto p = talk_tc_params(q, pages, k_scale, bias, mix, out, qsl, seq_lens, bt, H, dim, std::min(tiles, segment) * 128, ws_ml, ws_o);
+  p.splits = 1;
+  const c10::cuda::CUDAGuard guard(q.device());
+  const int rc = oc::talk_prefill_launch(p, (int)tiles, (int)segment, pages.size(0), cur_stream());
+  TORCH_CHECK(rc == 0, "talk_prefill failed: ", rc);
 }
 
 torch::Tensor sigmoid_mul(torch::Tensor x, torch::Tensor gate) {
@@ -1260,11 +1269,12 @@ void read_status_async(torch::Tensor pinned) {
   oc::sampling_read_status_async(p + 9, st);
   oc::mla_prefill_read_status_async(p + 10, st);
   oc::diff_prefill_read_status_async(p + 11, st);
+  oc::talk_prefill_read_status_async(p + 12, st);
 }
 
 int64_t read_status(bool clear) {
   return (int64_t)(oc::gemm_read_status(clear) | oc::elementwise_read_status(clear) | oc::attention_read_status(clear) | oc::attention_tc_read_status(clear) |
-                   oc::comm_read_status(clear) | oc::gdn_read_status(clear) | oc::sampling_read_status(clear) | oc::moe_read_status(clear) | oc::mla_read_status(clear) | oc::mla_prefill_read_status(clear) | oc::diff_prefill_read_status(clear) | oc::ep_read_status(clear));
+                   oc::comm_read_status(clear) | oc::gdn_read_status(clear) | oc::sampling_read_status(clear) | oc::moe_read_status(clear) | oc::mla_read_status(clear) | oc::mla_prefill_read_status(clear) | oc::diff_prefill_read_status(clear) | oc::talk_prefill_read_status(clear) | oc::ep_read_status(clear));
 }
 
 // ---- symmetric slab + peer-memory reductions
@@ -1374,8 +1384,9 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gated_norm", &gated_norm);
   m.def("talk_prepare", &talk_prepare);
   m.def("talk_plain", &talk_plain);
-  m.def("talk_sizes", &talk_sizes);
-  m.def("talk_tc", &talk_tc);
+  m.def("talk_tc_row", [](int64_t H, int64_t G, int64_t dim) { return (int64_t)oc::talk_tc_row((int)H, (int)G, (int)dim); });
+  m.def("talk_decode", &talk_decode);
+  m.def("talk_prefill", &talk_prefill);
   m.def("fused_moe_f32", &fused_moe_f32);
   m.def("fused_moe", &fused_moe);
   m.def("fused_moe_a2a", &fused_moe_a2a);

@@ -431,9 +431,9 @@ struct TalkPrepareParams {
   float eps, coef;
   int every;                    // 0: no temperature
   const int *positions, *slots;
-  void *q_out, *pages;          // [T][G][group_rows][row]; [blocks][G][bs][row]
+  void *q_out, *pages;          // [T][H][row]; [blocks][G][bs][row]
   float* k_scale;               // [blocks][bs]
-  int T, H, G, dim, group_rows, row, bs, f32;
+  int T, H, G, dim, row, bs, f32;
 };
 int talk_prepare_launch(const TalkPrepareParams& p, cudaStream_t st);
 struct TalkParams {
@@ -441,19 +441,23 @@ struct TalkParams {
   const float *k_scale, *bias;  // [blocks][bs]; [2][H]: r1, r2
   void* out;                    // [T][H][dim]
   const int *query_start_loc, *seq_lens, *block_table;
-  int bt_stride, T, R, H, G, dim, group_rows, row, bs, f32;
+  int bt_stride, T, R, H, G, dim, row, bs, f32;
 };
 int talk_plain_launch(const TalkParams& p, cudaStream_t st);
-// Tensor-core form (talk_tc.cu): cached rows and query rows padded as TalkSizes says; single tokens (dec) and longer portions are launched apart.
-struct TalkSizes { int row, group_rows, stats_tokens, mix_tokens, short_len; };   // tokens per block of either pass; longest portion of the dec variant
-bool talk_tc_sizes(int H, int G, int dim, TalkSizes* s);
+// Tensor-core forms: single tokens (talk_decode.cu) and portions of at least min_len tokens (talk_prefill_tc.cu), launched apart.
+int talk_tc_row(int H, int G, int dim);   // width of a query row and of a cached row, zeros behind dim; 0: only the plain kernel takes the sizes
 struct TalkTcParams {
   TalkParams t;
-  float* ws_ml;                 // [splits][T][H][2] maximum (log2 domain) and sum
-  float* ws_o;                  // [mix_splits][T][H][dim], when there is more than one
-  int splits, mix_splits, stats_tiles, mix_tiles, short_len;
-  int kt_shift, bs_shift;       // keys per tile of the second pass and tokens per page, as powers of two; set by the launcher
+  float* ws_ml;                 // [rows][H][2] reference (log2 domain) and sum; rows: [splits][R] (single tokens), or tokens of a segment's tiles
+  float* ws_o;                  // [rows][H][G row] unnormalised results over the rows of all key heads
+  int splits, min_len;
+  int tile0, bs_shift;          // set by the launchers
 };
-int talk_tc_launch(const TalkTcParams& p, bool dec, cudaStream_t st);
+int talk_decode_launch(const TalkTcParams& p, cudaStream_t st);
+int talk_join_launch(const TalkTcParams& p, bool dec, int rows, cudaStream_t st);
+// tiles: 128-token tiles over the portions; `segment` of them at a time go through the workspace
+int talk_prefill_launch(const TalkTcParams& p, int tiles, int segment, long long num_blocks, cudaStream_t st);
+unsigned int talk_prefill_read_status(bool clear);
+void talk_prefill_read_status_async(unsigned int* dst, cudaStream_t st);
 
 }  // namespace oc

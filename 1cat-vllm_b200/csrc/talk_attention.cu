@@ -35,7 +35,7 @@ __global__ void __launch_bounds__(256) talk_prepare_kernel(const TalkPreparePara
   pdl_trigger();
   pdl_wait();
   const size_t t = blockIdx.x;
-  const int nq = p.H * p.dim, nk = p.G * p.dim, share = p.H / p.G;
+  const int nq = p.H * p.dim, nk = p.G * p.dim;
   const E* q = reinterpret_cast<const E*>(p.qk) + t * p.ld;
   const E* k = q + nq;
   float qq = 0.f, kk = 0.f;
@@ -52,13 +52,12 @@ __global__ void __launch_bounds__(256) talk_prepare_kernel(const TalkPreparePara
   kk = block_total(square(k, nk), red);
   float f = 1.f / sqrtf(qq / (float)nq + p.eps);
   if (p.every > 0) f *= 1.f + p.coef * logf((float)((p.positions[t] + 1) / p.every) + 1.f);
-  // queries: [token][key head][rows of the group, padded][columns, padded]
-  E* qo = reinterpret_cast<E*>(p.q_out) + t * p.G * p.group_rows * p.row;
+  E* qo = reinterpret_cast<E*>(p.q_out) + t * p.H * p.row;
   const int per = p.row / N;
-  for (int i = threadIdx.x; i < p.G * p.group_rows * per; i += blockDim.x) {
-    const int d = i % per * N, hr = i / per, hh = hr % p.group_rows, head = hr / p.group_rows * share + hh;
+  for (int i = threadIdx.x; i < p.H * per; i += blockDim.x) {
+    const int d = i % per * N, head = i / per;
     Vec o;
-    if (hh < share && d < p.dim) {
+    if (d < p.dim) {
       const Vec v = *reinterpret_cast<const Vec*>(q + head * p.dim + d);
 #pragma unroll
       for (int j = 0; j < N; ++j) o.e[j] = from_f<E>(to_f<E>(v.e[j]) * f * p.gain[head * p.dim + d + j]);
@@ -66,7 +65,7 @@ __global__ void __launch_bounds__(256) talk_prepare_kernel(const TalkPreparePara
 #pragma unroll
       for (int j = 0; j < N; ++j) o.e[j] = from_f<E>(0.f);
     }
-    *reinterpret_cast<Vec*>(qo + (size_t)hr * p.row + d) = o;
+    *reinterpret_cast<Vec*>(qo + (size_t)head * p.row + d) = o;
   }
   const int slot = p.slots[t];
   if (slot < 0) return;
@@ -207,7 +206,7 @@ int plain_go(const TalkParams& p, cudaStream_t st) {
 
 int talk_prepare_launch(const TalkPrepareParams& p, cudaStream_t st) {
   if (p.T == 0) return 0;
-  if (p.H < 1 || p.G < 1 || p.H % p.G || p.row < p.dim || p.group_rows < p.H / p.G || p.bs < 1) return -1;
+  if (p.H < 1 || p.G < 1 || p.H % p.G || p.row < p.dim || p.bs < 1) return -1;
   const int n = p.f32 ? 4 : 8;
   auto ok = [&](const void* q) { return ((uintptr_t)q & 15) == 0; };
   const bool vec = p.dim % n == 0 && p.row % n == 0 && p.ld % n == 0 && ok(p.qk) && ok(p.q_out) && ok(p.pages);

@@ -457,13 +457,13 @@ def nalasun_kernels(s: dict, iters: int) -> list[dict]:
         t = max(flops / pk["bf16_tflops"] / 1e9, nbytes / pk["hbm_gbs"] / 1e6)
         rows.append(dict(kernel=kernel, case=case, model=who, us=ms * 1e3, roofline_us=t * 1e3, frac_of_roofline=t / ms))
 
-    wide, (_, hp, *_) = K.talk_row(H, G, D), K._C.talk_sizes(H, G, D)
+    wide = K.talk_row(H, G, D)
     for case, n, q, S in (("prefill", 1, PREFILL, PREFILL), ("decode", DECODE_REQS, 1, DECODE_CTX)):
         T = n * q
         md, nblk = _meta(n, q, S)
         md.is_uniform_decode = case == "decode"
         pairs = n * sum(range(S - q + 1, S + 1))
-        cache, fac, qq, bias, mix = b(nblk, 1, G, 16, wide) * 0.5, torch.ones(nblk, 16, device="cuda"), b(T, G * hp, wide) * 0.1, torch.rand(2, H, device="cuda"), b(H, H) * 0.2
+        cache, fac, qq, bias, mix = b(nblk, 1, G, 16, wide) * 0.5, torch.ones(nblk, 16, device="cuda"), b(T, H, wide) * 0.1, torch.rand(2, H, device="cuda"), b(H, H) * 0.2
         cost = lambda mixed, tensors: (2.0 * H * pairs * (2 * D + (H if mixed else 0)), 2.0 * (n * S * G * D * tensors + 2 * T * H * D))
         row("attention", case, "nalasun, shared keys, mixed heads", lambda: K.talk_attention(qq, cache, fac, md, bias, mix, D), *cost(True, 1))
         x, out, table = b(T, H, D), torch.empty(T, H, D, dtype=torch.bfloat16, device="cuda"), f32(H, BIAS_MAX + 1)

@@ -17,7 +17,7 @@ OUT = os.path.join(HERE, "_C.so")
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "--use_fast_math",
               "-Xcompiler", "-fPIC", "-Xptxas", "-v"] + (["-DONECAT_GEMM_TRACE"] if os.environ.get("ONECAT_GEMM_TRACE") else [])
 # units whose results are fp32: without the approximate division, square root and exponentials
-PRECISE = ("attention_f32.cu", "causal_conv.cu", "diff_prepare.cu", "mla.cu", "mlstm.cu", "moe.cu", "recurrence.cu", "recurrence_chunk.cu", "stream.cu", "talk_attention.cu")
+PRECISE = ("attention_f32.cu", "causal_conv.cu", "diff_prepare.cu", "mla.cu", "mlstm.cu", "moe.cu", "recurrence.cu", "recurrence_chunk.cu", "stream.cu", "talk_attention.cu", "talk_decode.cu")
 # --use_fast_math only affects __expf/exp2f-style intrinsics used in softmax/SiLU epilogues; accumulation stays fp32
 
 

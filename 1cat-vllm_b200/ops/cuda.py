@@ -979,63 +979,61 @@ def gated_norm(x, gate, w, eps, groups, gate_first):
 
 
 # ----------------------------------------------------------------------------- talking-heads attention
-TALK_WS_BYTES = 512 << 20   # most memory of a step's partial outputs
+TALK_WS_BYTES = 256 << 20   # partial results of a prompt's tiles that are in memory at a time
+TALK_ROWS = 592             # partial rows of single tokens (requests times key splits), four per SM
 
 
 def talk_row(H: int, G: int, dim: int) -> int:
     """Width of a cached bf16 row: padded for the tensor-core kernels, or as it is where only the plain kernel serves the sizes."""
-    s = _C.talk_sizes(H, G, dim)
-    return s[0] if s else dim
+    return _C.talk_tc_row(H, G, dim) or dim
+
+
+def talk_workspace(H: int, G: int, D: int, tokens: int) -> tuple[int, int]:
+    """Most elements of the partial results and of the sums that decode steps of up to ``tokens`` requests need."""
+    rows = max(tokens, TALK_ROWS)
+    return rows * H * G * D, rows * H * 2
 
 
 def talk_prepare(qk, q_gain, eps, temperature, positions, pages, k_scale, slot_mapping, heads, kv_heads, dim):
     global _LAUNCHES
     _LAUNCHES += 1
     coef, every = temperature or (0.0, 0)
-    s = _C.talk_sizes(heads, kv_heads, dim) if qk.dtype == torch.bfloat16 else None
-    return _C.talk_prepare(qk, q_gain, eps, coef, every, _int32(positions), pages, k_scale, _int32(slot_mapping), heads, kv_heads, dim,
-                           s[1] if s else heads // kv_heads)
+    return _C.talk_prepare(qk, q_gain, eps, coef, every, _int32(positions), pages, k_scale, _int32(slot_mapping), heads, kv_heads, dim)
 
 
-def plan_talk(md, H: int, G: int, dim: int, sizes, num_sms: int):
-    """(single tokens?, splits of either pass, blocks of either pass) of the launches of a step."""
-    _, hp, st_tok, mix_tok, short = sizes
-    ql, sl = md.query_lens_cpu, md.seq_lens_cpu
-    out = []
-    n_short = sum(1 for q in ql if 0 < q <= short)
-    if n_short:
-        longest = max(s for q, s in zip(ql, sl) if 0 < q <= short)
-        out.append((True, choose_decode_splits(n_short * G, longest, num_sms, 4), choose_decode_splits(n_short, longest, num_sms, 1), 0, 0))
-    longs = [(q, s) for q, s in zip(ql, sl) if q > short]
-    if longs:
-        st, mx, longest = sum(-(-q // st_tok) for q, _ in longs), sum(-(-q // mix_tok) for q, _ in longs), max(s for _, s in longs)
-        parts = lambda blocks, most: max(1, min(most, -(-longest // 256), num_sms // max(blocks, 1)))
-        room = max(1, TALK_WS_BYTES // (4 * sum(ql) * H * dim))
-        out.append((False, parts(st * G, 16), min(parts(mx, 16), room), st, mx))
-    return short, out
+def plan_talk(query_lens: list, seq_lens: list, num_sms: int) -> tuple[int, int]:
+    """(key splits of the single tokens, 0 without any; 128-token tiles of the longer portions)."""
+    longest = max((s for q, s in zip(query_lens, seq_lens) if q == 1), default=0)
+    splits = max(1, min(choose_decode_splits(query_lens.count(1), longest, num_sms, 1), TALK_ROWS // len(query_lens))) if longest else 0
+    return splits, sum(-(-q // 128) for q in query_lens if q > 1)
 
 
 def talk_attention(q, pages, k_scale, md, bias, mix, dim):
-    """Talking-heads attention: tensor-core kernels for the sizes they take (single tokens and longer portions in launches of their own), the
-    plain kernel otherwise and for fp32."""
+    """Talking-heads attention: single tokens and longer portions run tensor-core kernels of their own for the sizes they take; the plain kernel
+    serves the rest and fp32."""
     global _LAUNCHES
-    H, T, G = mix.shape[0], q.shape[0], pages.shape[2]
+    T, H, row = q.shape
+    G = pages.shape[2]
     out = torch.empty(T, H, dim, dtype=q.dtype, device=q.device)
-    sizes = _C.talk_sizes(H, G, dim) if q.dtype == torch.bfloat16 else None
-    if not sizes:
+    args = (q, pages, k_scale, bias, mix, out, md.query_start_loc, md.seq_lens, md.block_table, H, dim)
+    if q.dtype != torch.bfloat16 or not _C.talk_tc_row(H, G, dim):
         _LAUNCHES += 1
-        _C.talk_plain(q, pages, k_scale, bias, mix, out, md.query_start_loc, md.seq_lens, md.block_table, H, dim)
+        _C.talk_plain(*args)
         return out
-    cache = md.__dict__.setdefault("_talk_plans", {})
-    if (H, G, dim) not in cache:
-        cache[(H, G, dim)] = plan_talk(md, H, G, dim, sizes, _sms(q.device))
-    short, launches = cache[(H, G, dim)]
+    plan = md.__dict__.get("_talk_plan")
+    if plan is None:
+        plan = md.__dict__["_talk_plan"] = plan_talk(md.query_lens_cpu, md.seq_lens_cpu, _sms(q.device))
+    splits, tiles = plan
     w = workspace(q.device)
-    for dec, splits, mix_splits, st_tiles, mix_tiles in launches:
-        ws_o, ws_ml = (w.attn_static if getattr(md, "static_ws", False) else w.attn)(mix_splits * T * H * dim if mix_splits > 1 else 1, splits * T * H * 2)
-        _C.talk_tc(q, pages, k_scale, bias, mix, out, md.query_start_loc, md.seq_lens, md.block_table, H, dim, dec, short, splits, mix_splits, st_tiles,
-                   mix_tiles, ws_ml, ws_o)
-        _LAUNCHES += 3 if mix_splits > 1 else 2
+    if splits:
+        ws_o, ws_ml = (w.attn_static if getattr(md, "static_ws", False) else w.attn)(splits * md.num_reqs * H * G * row, splits * md.num_reqs * H * 2)
+        _C.talk_decode(*args, splits, ws_ml, ws_o)
+        _LAUNCHES += 2
+    if tiles:
+        segment = min(tiles, max(1, TALK_WS_BYTES // (4 * 128 * H * G * row)))
+        ws_o, ws_ml = w.attn(segment * 128 * H * G * row, segment * 128 * H * 2)
+        _C.talk_prefill(*args, tiles, segment, ws_ml, ws_o)
+        _LAUNCHES += 2 * -(-tiles // segment)
     return out
 
 

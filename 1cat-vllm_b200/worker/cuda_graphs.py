@@ -52,6 +52,9 @@ class DecodeGraphs:
             K.workspace(runner.device).attn_static(32 * tmax * max(a.Hq * a.D for a in attns), 32 * tmax * 2 * max(a.Hq for a in attns))
             for a in mlas:
                 K.workspace(runner.device).attn_static(32 * tmax * a.H * a.lora_pad, 32 * tmax * a.H * 2)
+            for a in attns:
+                if getattr(a, "token_scale", False):
+                    K.workspace(runner.device).attn_static(*K.talk_workspace(a.Hq, a.Hkv, a.D, tmax))
             spans = [K.attention_span(a.window or getattr(a, "chunk", 0), a.window_keep) for a in attns]
             self.max_span = max(spans) if all(spans) and not mla else 0
         elif mla:
