@@ -71,6 +71,7 @@ __global__ void __launch_bounds__(MT) talk_decode_kernel(const TalkTcParams p) {
   float* ss = reinterpret_cast<float*>(sp + 2 * m.p);          // [nt * 8][ps] scores
   float* sf = ss + m.s;                                        // [2][KT]
   float* sal = sf + 2 * KT;                                    // [rows] what the tile scales earlier results by
+  int* moved = reinterpret_cast<int*>(sal + m.rows);           // last tile that scales anything
   const int keys = p.t.seq_lens[r], tiles = (keys + KT - 1) / KT;
   const int each = (tiles + p.splits - 1) / p.splits, first = split * each, last = min(tiles, first + each);
   const int* bt = p.t.block_table + (size_t)r * p.t.bt_stride;
@@ -83,6 +84,7 @@ __global__ void __launch_bounds__(MT) talk_decode_kernel(const TalkTcParams p) {
   }
   for (int i = tid; i < (int)(2 * m.p); i += MT) sp[i] = __float2bfloat16(0.f);
   for (int i = tid; i < m.rows; i += MT) sal[i] = 1.f;
+  if (tid == 0) *moved = -1;
   auto fetch = [&](int tile) {
     if (tile < last) {
       constexpr int RPI = MT / (DP / 8);   // rows of the tile that the threads copy at a time
@@ -119,7 +121,7 @@ __global__ void __launch_bounds__(MT) talk_decode_kernel(const TalkTcParams p) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) acc[a][b][t][e] = 0.f;
   const int col0 = warp * NTC * 16;   // this warp's columns of all key heads' rows
-  // heads warp, warp + 16, ...: running maximum, this lane's part of the sum
+  // heads warp, warp + 16, ...: reference of the exponents (it moves when a score exceeds it by 2^8), this lane's part of the sum
   constexpr int HW = MH;
   float mx[HW], l[HW], r1[HW], r2[HW];
   int srow[HW];
@@ -144,27 +146,33 @@ __global__ void __launch_bounds__(MT) talk_decode_kernel(const TalkTcParams p) {
     for (int u = warp; u < m.nt * MTS; u += WARPS) {
       const int t = u / MTS, mt = u % MTS, g = t / m.tg;
       const uint32_t ka = ak + (uint32_t)((g * KT + mt * 16) * PD * 2) + lane_k, qa = aq + (uint32_t)(t * 8 * PD * 2) + lane_q;
-      float s[4] = {0.f, 0.f, 0.f, 0.f}, s2[4] = {0.f, 0.f, 0.f, 0.f};
+      float sa[4][4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sa[i][e] = 0.f;
 #pragma unroll
       for (int ks = 0; ks < DP / 16; ++ks) {
         uint32_t a[4], b0, b1;
         ldsm_x4(a, ka + ks * 32);
         ldsm_x2(b0, b1, qa + ks * 32);
-        if (ks & 1) mma16816(s2, a, b0, b1);
-        else mma16816(s, a, b0, b1);
+        mma16816(sa[ks & 3], a, b0, b1);
       }
+      float s[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[e] = (sa[0][e] + sa[1][e]) + (sa[2][e] + sa[3][e]);
       float* d = ss + (size_t)(t * 8 + 2 * t4) * m.ps + mt * 16 + g8;
-      d[0] = s[0] + s2[0];
-      d[m.ps] = s[1] + s2[1];
-      d[8] = s[2] + s2[2];
-      d[m.ps + 8] = s[3] + s2[3];
+      d[0] = s[0];
+      d[m.ps] = s[1];
+      d[8] = s[2];
+      d[m.ps + 8] = s[3];
     }
     __syncthreads();   // the scores are there
 #pragma unroll
     for (int i = 0; i < HW; ++i) {
       const int h = warp + i * WARPS;
       if (h >= H) break;
-      float x[KL], top = mx[i];
+      float x[KL], top = -INFINITY;
 #pragma unroll
       for (int k = 0; k < KL; ++k) {
         const int kr = lane + 32 * k;
@@ -173,14 +181,22 @@ __global__ void __launch_bounds__(MT) talk_decode_kernel(const TalkTcParams p) {
         if (kr < KT && d >= 0.f) x[k] = fmaf(ss[(size_t)srow[i] * m.ps + kr], sf[st * KT + kr] * kLog2e, -r1[i] * lg2(fmaf(r2[i], d, 1.f)));
         top = fmaxf(top, x[k]);
       }
-      top = warp_max(top);
-      const float al = ex2(mx[i] - top);   // a tile of a split holds at least one key, so the maximum is a number
-      float sum = l[i] * al;
+      float sum = l[i];
+      if (__any_sync(0xffffffffu, top > mx[i] + 8.f)) {
+        top = fmaxf(warp_max(top), mx[i]);
+        const float al = ex2(mx[i] - top);
+        sum *= al;
+        mx[i] = top;
+        if (lane == 0) {
+          sal[h] = al;
+          *moved = tile;
+        }
+      } else if (lane == 0) sal[h] = 1.f;
 #pragma unroll
       for (int k = 0; k < KL; ++k) {
         const int kr = lane + 32 * k;
         if (kr < KT) {
-          const float w = ex2(x[k] - top);
+          const float w = ex2(x[k] - mx[i]);   // a tile of a split holds at least one key, so the reference is a number
           const __nv_bfloat16 hi = __float2bfloat16(w);
           sum += w;
           sp[h * m.pp + kr] = hi;
@@ -188,21 +204,21 @@ __global__ void __launch_bounds__(MT) talk_decode_kernel(const TalkTcParams p) {
         }
       }
       l[i] = sum;
-      mx[i] = top;
-      if (lane == 0) sal[h] = al;
     }
     __syncthreads();   // weights and factors are there
     if (col0 < GD) {
+if (*moved == tile) {
 #pragma unroll
-      for (int a = 0; a < MH; ++a) {
-        const float f0 = sal[a * 16 + g8], f1 = sal[a * 16 + g8 + 8];
+        for (int a = 0; a < MH; ++a) {
+          const float f0 = sal[a * 16 + g8], f1 = sal[a * 16 + g8 + 8];
 #pragma unroll
-        for (int b = 0; b < NTC; ++b)
+          for (int b = 0; b < NTC; ++b)
 #pragma unroll
-          for (int t = 0; t < 2; ++t) {
-            acc[a][b][t][0] *= f0; acc[a][b][t][1] *= f0;
-            acc[a][b][t][2] *= f1; acc[a][b][t][3] *= f1;
-          }
+            for (int t = 0; t < 2; ++t) {
+              acc[a][b][t][0] *= f0; acc[a][b][t][1] *= f0;
+              acc[a][b][t][2] *= f1; acc[a][b][t][3] *= f1;
+            }
+        }
       }
 #pragma unroll
       for (int ks = 0; ks < MTS; ++ks) {
@@ -222,6 +238,9 @@ __global__ void __launch_bounds__(MT) talk_decode_kernel(const TalkTcParams p) {
           for (int a = 0; a < MH; ++a) {
             mma16816(acc[a][b][0], hi[a], v[0], v[1]);
             mma16816(acc[a][b][1], hi[a], v[2], v[3]);
+          }
+#pragma unroll
+          for (int a = 0; a < MH; ++a) {
             mma16816(acc[a][b][0], lo[a], v[0], v[1]);
             mma16816(acc[a][b][1], lo[a], v[2], v[3]);
           }
@@ -252,15 +271,17 @@ __global__ void __launch_bounds__(MT) talk_decode_kernel(const TalkTcParams p) {
         }
 }
 
-// One CTA per row of the partial results: rows are requests (dec), or the tokens of the tiles tile0, tile0 + 1, ... of 128 over the longer portions.
-constexpr int kJoinHeads = 8, kJoinThreads = 256;
+// One CTA per row of the partial results and block of columns; rows are requests (dec), or the tokens of the tiles tile0, tile0 + 1, ... of 128 over
+// the longer portions. A thread owns a column of one key head's rows and up to eight of the heads that read it.
+constexpr int kJoinHeads = 8, kJoinThreads = 128;
 
 template <bool DEC>
 __global__ void __launch_bounds__(kJoinThreads) talk_join_kernel(const TalkTcParams p) {
-  extern __shared__ float jm[];
+  extern __shared__ __align__(16) float jm[];
   const int H = p.t.H, G = p.t.G, share = H / G, dim = p.t.dim, DP = p.t.row, GD = G * DP, splits = DEC ? p.splits : 1;
-  float* st = jm;            // [H][H] mix
-  float* sc = jm + H * H;    // [splits][H] factors
+  const int blocks = (share + kJoinHeads - 1) / kJoinHeads, wide = G * blocks * kJoinHeads;
+  float* st = jm;             // [from][key head, block, eight heads] mix
+  float* sc = jm + H * wide;  // [splits][H] factors
   __shared__ int s_tok;
   pdl_trigger();
   pdl_wait();
@@ -303,27 +324,47 @@ __global__ void __launch_bounds__(kJoinThreads) talk_join_kernel(const TalkTcPar
       sc[s * H + g] = x == -INFINITY ? 0.f : ex2(x - m) / sum;
     }
   }
-  for (int i = threadIdx.x; i < H * H; i += kJoinThreads) st[i] = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.t.mix)[i]);
+  for (int i = threadIdx.x; i < H * wide; i += kJoinThreads) {
+    const int from = i / wide, a = i % wide / (blocks * kJoinHeads), k = i % (blocks * kJoinHeads);
+    st[i] = k < share ? __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p.t.mix)[(a * share + k) * H + from]) : 0.f;
+  }
   __syncthreads();
   const float* o = p.ws_o + row * H * GD;
   __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.t.out) + (size_t)tok * H * dim;
-  for (int i = threadIdx.x; i < G * dim; i += kJoinThreads) {
+  const int step = gridDim.y * kJoinThreads;
+  for (int i = blockIdx.y * kJoinThreads + threadIdx.x; i < G * dim; i += step) {
     const int a = i / dim, d = i % dim;
-    for (int h0 = 0; h0 < share; h0 += kJoinHeads) {
+    const float* src = o + a * DP + d;
+    for (int blk = 0; blk < blocks; ++blk) {
+      const float* w = st + (a * blocks + blk) * kJoinHeads;
       float acc[kJoinHeads];
 #pragma unroll
       for (int k = 0; k < kJoinHeads; ++k) acc[k] = 0.f;
-#pragma unroll 4
-      for (int g = 0; g < H; ++g) {
-        float x = 0.f;
-        for (int s = 0; s < splits; ++s) x = fmaf(sc[s * H + g], o[(s * plane * H + g) * GD + a * DP + d], x);
+      auto add = [&](int g, float x) {
+        const float4 t0 = *reinterpret_cast<const float4*>(w + g * wide), t1 = *reinterpret_cast<const float4*>(w + g * wide + 4);
+        acc[0] = fmaf(t0.x, x, acc[0]); acc[1] = fmaf(t0.y, x, acc[1]); acc[2] = fmaf(t0.z, x, acc[2]); acc[3] = fmaf(t0.w, x, acc[3]);
+        acc[4] = fmaf(t1.x, x, acc[4]); acc[5] = fmaf(t1.y, x, acc[5]); acc[6] = fmaf(t1.z, x, acc[6]); acc[7] = fmaf(t1.w, x, acc[7]);
+      };
+      int g = 0;
+      for (; g + 8 <= H; g += 8) {   // eight loads in flight
+        float x[8];
 #pragma unroll
-        for (int k = 0; k < kJoinHeads; ++k)
-          if (h0 + k < share) acc[k] = fmaf(st[(a * share + h0 + k) * H + g], x, acc[k]);
+        for (int k = 0; k < 8; ++k) x[k] = sc[g + k] * src[(size_t)(g + k) * GD];
+        for (int s = 1; s < splits; ++s) {
+#pragma unroll
+          for (int k = 0; k < 8; ++k) x[k] = fmaf(sc[s * H + g + k], src[(s * plane * H + g + k) * GD], x[k]);
+        }
+#pragma unroll
+        for (int k = 0; k < 8; ++k) add(g + k, x[k]);
+      }
+      for (; g < H; ++g) {
+        float x = 0.f;
+        for (int s = 0; s < splits; ++s) x = fmaf(sc[s * H + g], src[(s * plane * H + g) * GD], x);
+        add(g, x);
       }
 #pragma unroll
       for (int k = 0; k < kJoinHeads; ++k)
-        if (h0 + k < share) out[(a * share + h0 + k) * dim + d] = __float2bfloat16(acc[k]);
+        if (blk * kJoinHeads + k < share) out[(a * share + blk * kJoinHeads + k) * dim + d] = __float2bfloat16(acc[k]);
     }
   }
 }
@@ -391,10 +432,20 @@ int talk_decode_launch(const TalkTcParams& p_, cudaStream_t st) {
 }
 
 int talk_join_launch(const TalkTcParams& p, bool dec, int rows, cudaStream_t st) {
-  const size_t smem = ((size_t)p.t.H * p.t.H + (size_t)(dec ? p.splits : 1) * p.t.H) * 4;
-  if (smem > 48 * 1024) return -6;
-  if (dec) launch_k(talk_join_kernel<true>, dim3((unsigned)rows), dim3(kJoinThreads), smem, st, true, p);
-  else launch_k(talk_join_kernel<false>, dim3((unsigned)rows), dim3(kJoinThreads), smem, st, true, p);
+  const int share = p.t.H / p.t.G, wide = p.t.G * ((share + kJoinHeads - 1) / kJoinHeads) * kJoinHeads;
+  const size_t smem = ((size_t)p.t.H * wide + (size_t)(dec ? p.splits : 1) * p.t.H) * 4;
+  static bool configured_dev[kMaxDevices] = {};
+  bool& configured = configured_dev[current_device_slot()];
+  if (!configured) {   // up to 64 key heads of one head each: 64 x 512 numbers
+    if (cudaFuncSetAttribute(talk_join_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) != cudaSuccess ||
+        cudaFuncSetAttribute(talk_join_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) != cudaSuccess) return -4;
+    configured = true;
+  }
+  if (smem > 160 * 1024) return -6;
+  const int cols = (p.t.G * p.t.dim + kJoinThreads - 1) / kJoinThreads;
+  const dim3 grid((unsigned)rows, (unsigned)(dec ? cols : (cols + 3) / 4));   // few rows: more blocks of columns
+  if (dec) launch_k(talk_join_kernel<true>, grid, dim3(kJoinThreads), smem, st, true, p);
+  else launch_k(talk_join_kernel<false>, grid, dim3(kJoinThreads), smem, st, true, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
 }
 

@@ -21,7 +21,7 @@ constexpr int TQ = 128, TK = 128;
 constexpr int kChunk = 128 * 128;          // bytes of one 64-column chunk of a 128-row operand tile
 constexpr int kSlots = 5, kSlot = 2 * kChunk, kThreads = 576;
 constexpr uint32_t kColS = 0, kColO = 256;
-constexpr float kLog2e = 1.4426950408889634f, kSlack = 8.f;
+constexpr float kLog2e = 1.4426950408889634f, kSlack = 8.f, kNear = 1.f / 16.f;
 
 __device__ __forceinline__ float ex2(float x) {
   float y;
@@ -32,6 +32,34 @@ __device__ __forceinline__ float lg2(float x) {
   float y;
   asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+
+// two fp32 numbers in a register pair
+typedef unsigned long long f2;
+__device__ __forceinline__ f2 pair(float a, float b) {
+  f2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ float2 unpair(f2 v) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+  return r;
+}
+__device__ __forceinline__ f2 fma2(f2 a, f2 b, f2 c) {
+  f2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ f2 mul2(f2 a, f2 b) {
+  f2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ f2 add2(f2 a, f2 b) {
+  f2 r;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
 }
 
 // MN-major operand B: 64 columns x 8 keys form a 1024-byte swizzle atom; the next 8 keys are 1024 bytes on, the next 64 columns a chunk on.
@@ -234,18 +262,22 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const int tq = tq0 + row, pos = ctx0 + tq;
     const float r1 = p.t.bias[h], r2 = p.t.bias[H + h];
     float* f = s_f + (warp - 2) * 32;
-    auto factor = [&](int j) {   // of this lane's key of the j-th tile from the end
-      const int key = (ntiles - 1 - j) * TK + part * 32 + lane;
-      return j < ntiles && key < S ? p.t.k_scale[((size_t)bt[key >> bs] << bs) + (key & (p.t.bs - 1))] * kLog2e : 0.f;
-    };
-    float m = -INFINITY, l = 0.f, fk = factor(0);
+    // page of this lane's key in the j-th tile from the end, and the key's factor: loaded two tiles and one tile ahead, so that nobody waits
+    auto key_of = [&](int j) { return (ntiles - 1 - j) * TK + part * 32 + lane; };
+    auto page = [&](int j) { return j < ntiles && key_of(j) < S ? bt[key_of(j) >> bs] : -1; };
+    auto factor = [&](int j, int pg) { return pg >= 0 ? p.t.k_scale[((size_t)pg << bs) + (key_of(j) & (p.t.bs - 1))] : 0.f; };
+    auto both = [](float x) { return pair(x, x); };
+    f2 l = 0ull;
+    float m = -INFINITY, fk = factor(0, page(0));
+    int pg = page(1);
     bool ok = ntiles > 0;
     for (int j = 0; j < ntiles; ++j) {
       const int k0 = (ntiles - 1 - j) * TK + part * 32;
       const bool all = __all_sync(0xffffffffu, k0 + 31 <= pos), none = __all_sync(0xffffffffu, k0 > pos);
-      f[lane] = fk;
+      f[lane] = fk * kLog2e;
       __syncwarp();
-      fk = factor(j + 1);
+      fk = factor(j + 1, pg);
+      pg = page(j + 2);
       if (ok) ok = mbar_wait(&s_full[j & 1], (j >> 1) & 1, abort_flag);
       ok = __all_sync(0xffffffffu, ok);
       const uint32_t s_addr = lane_addr + kColS + (j & 1) * TK + part * 32;
@@ -255,19 +287,50 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         tc_fence_after();
         tmem_ld_32x32(s_addr, v);
         tmem_ld_wait();
-        const float d0 = (float)(pos - k0), a0 = fmaf(r2, d0, 1.f);
+        // r1 log2(1 + r2 d) over the 32 keys, d = d0 - i. Away from the row's own position a series around the middle key takes the place of the
+        // logarithms: with u = r2 (d - dm) / (1 + r2 dm) it ends at u^4, whose successor is below 2^-22 for |u| <= 1/16.
+        const float d0 = (float)(pos - k0), am = fmaf(r2, d0 - 15.5f, 1.f), inv = __fdividef(1.f, am), g = -r2 * inv;
+        if (__all_sync(0xffffffffu, fabsf(g) * 15.5f <= kNear && am > 0.f)) {
+          const float c = -r1 * kLog2e * g;
+          const f2 c0 = both(-r1 * lg2(am)), c1 = both(c), c2 = both(c * g * -0.5f), c3 = both(c * g * g * (1.f / 3.f)), c4 = both(c * g * g * g * -0.25f);
 #pragma unroll
-        for (int i = 0; i < 32; i += 4) {
-          const float4 ff = *reinterpret_cast<const float4*>(f + i);
-          const float fi[4] = {ff.x, ff.y, ff.z, ff.w};
+          for (int i = 0; i < 32; i += 4) {
+            const ulonglong2 ff = *reinterpret_cast<const ulonglong2*>(f + i);
 #pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            float s = fmaf(__uint_as_float(v[i + e]), fi[e], -r1 * lg2(fmaf(r2, -(float)(i + e), a0)));
-            if (!all) s = k0 + i + e <= pos ? s : -INFINITY;
-            v[i + e] = __float_as_uint(s);
-            top = fmaxf(top, s);
+            for (int e = 0; e < 4; e += 2) {
+              const f2 x = pair((float)(i + e) - 15.5f, (float)(i + e) - 14.5f);
+              const f2 bias = fma2(x, fma2(x, fma2(x, fma2(x, c4, c3), c2), c1), c0);
+              const float2 t = unpair(fma2(pair(__uint_as_float(v[i + e]), __uint_as_float(v[i + e + 1])), e ? ff.y : ff.x, bias));
+              v[i + e] = __float_as_uint(t.x);
+              v[i + e + 1] = __float_as_uint(t.y);
+            }
+          }
+        } else {
+          const f2 a0 = both(fmaf(r2, d0, 1.f)), step = both(-r2), factor1 = both(-r1);
+#pragma unroll
+          for (int i = 0; i < 32; i += 4) {
+            const ulonglong2 ff = *reinterpret_cast<const ulonglong2*>(f + i);
+#pragma unroll
+            for (int e = 0; e < 4; e += 2) {
+              const float2 t = unpair(fma2(step, pair((float)(i + e), (float)(i + e + 1)), a0));
+              const float2 y = unpair(fma2(factor1, pair(lg2(t.x), lg2(t.y)), mul2(pair(__uint_as_float(v[i + e]), __uint_as_float(v[i + e + 1])), e ? ff.y : ff.x)));
+              v[i + e] = __float_as_uint(y.x);
+              v[i + e + 1] = __float_as_uint(y.y);
+            }
           }
         }
+        if (!all) {
+          const int seen = pos - k0;
+#pragma unroll
+          for (int i = 0; i < 32; ++i) v[i] = i <= seen ? v[i] : 0xff800000u;
+        }
+        float top2 = -INFINITY;
+#pragma unroll
+        for (int i = 0; i < 32; i += 4) {
+          top = fmaxf(top, fmaxf(__uint_as_float(v[i]), __uint_as_float(v[i + 1])));
+          top2 = fmaxf(top2, fmaxf(__uint_as_float(v[i + 2]), __uint_as_float(v[i + 3])));
+        }
+        top = fmaxf(top, top2);
       }
       // does any row of the quarter have to move its reference?
       if (quarter_any(q4, top > m + kSlack)) {
@@ -276,7 +339,7 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         const float nm = fmaxf(fmaxf(fmaxf(s_x[row], s_x[TQ + row]), fmaxf(s_x[2 * TQ + row], s_x[3 * TQ + row])), m);
         const float al = nm == -INFINITY ? 1.f : ex2(m - nm);
         m = nm;
-        l *= al;
+        l = mul2(l, both(al));
         if (j > 0) {
           if (ok) ok = mbar_wait(&o_done[(j - 1) & 1], ((j - 1) >> 1) & 1, abort_flag);   // every earlier product is complete, none is issued before these weights
           ok = __all_sync(0xffffffffu, ok);
@@ -301,17 +364,23 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 #pragma unroll
           for (int i = 0; i < 32; ++i) out[i] = 0u;
         } else {
-          const float base = m == -INFINITY ? 0.f : m;
+          const f2 base = both(m == -INFINITY ? 0.f : -m), minus = both(-1.f);
+          f2 l2 = 0ull;
 #pragma unroll
           for (int i = 0; i < 32; i += 2) {
-            const float w0 = ex2(__uint_as_float(v[i]) - base), w1 = ex2(__uint_as_float(v[i + 1]) - base);
-            l += w0 + w1;
-            __nv_bfloat162 b = __floats2bfloat162_rn(w0, w1);
+            const float2 x = unpair(add2(pair(__uint_as_float(v[i]), __uint_as_float(v[i + 1])), base));
+            const f2 w = pair(ex2(x.x), ex2(x.y));
+            if (i & 2) l2 = add2(l2, w);
+            else l = add2(l, w);
+            const float2 wf = unpair(w);
+            __nv_bfloat162 b = __floats2bfloat162_rn(wf.x, wf.y);
             const uint32_t bits = *reinterpret_cast<uint32_t*>(&b);
-            __nv_bfloat162 e = __floats2bfloat162_rn(w0 - __uint_as_float(bits << 16), w1 - __uint_as_float(bits & 0xffff0000u));
+            const float2 d = unpair(fma2(pair(__uint_as_float(bits << 16), __uint_as_float(bits & 0xffff0000u)), minus, w));
+            __nv_bfloat162 e = __floats2bfloat162_rn(d.x, d.y);
             out[i >> 1] = bits;
             out[16 + (i >> 1)] = *reinterpret_cast<uint32_t*>(&e);
           }
+          l = add2(l, l2);
         }
         tmem_st_32x32(s_addr, out);
         tmem_st_wait();
@@ -321,7 +390,8 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       }
     }
     quarter_sync(q4);   // s_x has been read
-    s_x[part * TQ + row] = l;
+    const float2 lsum = unpair(l);
+    s_x[part * TQ + row] = lsum.x + lsum.y;
     quarter_sync(q4);
     if (ok) ok = mbar_wait(&o_done[(ntiles - 1) & 1], ((ntiles - 1) >> 1) & 1, abort_flag);
     ok = __all_sync(0xffffffffu, ok);
