@@ -6,8 +6,9 @@
 //   P = 2^(s - m)   sixteen warps, four threads per query row (32 keys each). The reference m of a row only moves when a score exceeds it by 2^8:
 //                   then the row's results in TMEM are rescaled. The distance bias makes the newest keys' scores the largest as a rule, so after
 //                   the first tile this is rare. P replaces S in its columns as two bf16 terms, the rounded weight and what rounding took from it.
-//   O += P V        operand A from TMEM, V (the same cached rows, 128 columns at a time) as an MN-major operand, accumulated in TMEM
-// Key and value tiles share one ring of 32 KB slots, filled in the order in which the MMA warp uses them. O leaves unnormalised in fp32, with m
+//   O += P V        operand A from TMEM, V (the same cached rows, 256 columns) as an MN-major operand, accumulated in TMEM
+// Key and value tiles share one ring of 16 KB slots (64 columns of 128 keys, or 256 columns of 32 values), filled in the order in which the MMA
+// warp uses them. The MMA warp looks after the slots of a product while the product ahead of it runs. O leaves unnormalised in fp32, with m
 // and the row's sum beside it.
 // Roles: warp 0 TMA producer, warp 1 MMA issue, warps 2-17 softmax and epilogue. Every mbarrier wait is bounded; on expiry the CTA raises the
 // status word and tears down. The softmax warps also meet at named barriers, which have no time-out: they pass all of them whatever happened.
@@ -19,7 +20,7 @@ namespace {
 
 constexpr int TQ = 128, TK = 128;
 constexpr int kChunk = 128 * 128;          // bytes of one 64-column chunk of a 128-row operand tile
-constexpr int kSlots = 5, kSlot = 2 * kChunk, kThreads = 576;
+constexpr int kSlots = 10, kSlot = kChunk, kVChunk = 32 * 128, kThreads = 576;   // kVChunk: 64 columns of 32 values
 constexpr uint32_t kColS = 0, kColO = 256;
 constexpr float kLog2e = 1.4426950408889634f, kSlack = 8.f, kNear = 1.f / 16.f;
 
@@ -62,11 +63,11 @@ __device__ __forceinline__ f2 add2(f2 a, f2 b) {
   return r;
 }
 
-// MN-major operand B: 64 columns x 8 keys form a 1024-byte swizzle atom; the next 8 keys are 1024 bytes on, the next 64 columns a chunk on.
+// MN-major operand B: 64 columns x 8 keys form a 1024-byte swizzle atom; the next 8 keys are 1024 bytes on, the next 64 columns 32 keys on.
 __device__ __forceinline__ uint64_t desc_mn(uint32_t smem_addr) {
   uint64_t d = 0;
   d |= (uint64_t)((smem_addr & 0x3FFFF) >> 4);
-  d |= (uint64_t)((kChunk >> 4) & 0x3FFF) << 16;
+  d |= (uint64_t)((kVChunk >> 4) & 0x3FFF) << 16;
   d |= (uint64_t)(1024 >> 4) << 32;
   d |= (uint64_t)1 << 46;
   d |= (uint64_t)2 << 61;
@@ -163,10 +164,9 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     ntiles = (min(S, ctx0 + min(tq0 + TQ, qlen)) + TK - 1) / TK;   // up to the last key that the tile's last row sees
   }
   const int* bt = p.t.block_table + (size_t)max(r, 0) * p.t.bt_stride;
-  const int vhalves = (vchunks + 1) / 2;
 
   if (warp == 0) {
-    // ------------------------------------------------------------------ producer: K(0), then K(j + 1) and the value tiles of j
+    // ------------------------------------------------------------------ producer: K(0), then K(j + 1) and the values of j
     if (ntiles > 0) {
       if (lane == 0) {
         mbar_expect_tx(q_full, NC * kChunk);
@@ -174,83 +174,91 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 #pragma unroll
         for (int c = 0; c < NC; ++c) tma_load_2d(sQ + c * kChunk, &tmQ, h * DP + c * 64, qs + tq0, q_full);
       }
-      Ring st;
+      int at = 0;   // slots handed out so far
       bool ok = true;
-      const int part = lane & 7, sub = lane >> 3;   // 16 keys of the tile; chunk of the slot
-      auto load = [&](int j, int c0, int chunks) {  // chunks c0 .. of all key heads' columns, keys of the j-th tile from the end
-        if (!ok) return;
-        const int key0 = (ntiles - 1 - j) * TK + part * 16;
-        int page = 0, off = 0;   // keys past the sequence read the null block
-        if (key0 < S) {
-          page = bt[key0 >> bs];
-          off = key0 & (p.t.bs - 1);
-        }
-        if (lane == 0) {
-          ok = mbar_wait(&empty[st.idx], st.phase ^ 1, abort_flag);
-          if (ok) mbar_expect_tx(&full[st.idx], chunks * kChunk);
-        }
-        ok = __shfl_sync(0xffffffffu, (int)ok, 0) != 0;
-        if (!ok) return;
-        if (sub < chunks) {
-          const int c = c0 + sub;
-          tma_load_2d(ring + st.idx * kSlot + sub * kChunk + part * 2048, &tmK, (c % NC) * 64, ((page * G + c / NC) << bs) + off, &full[st.idx]);
-        }
-        st.advance(kSlots);
+      const int sub = lane >> 3, box = lane & 7;   // eight lanes fill a slot with boxes of 16 rows x 64 columns
+      auto row_of = [&](int key0, int g) {         // keys past the sequence read the null block
+        return key0 < S ? ((bt[key0 >> bs] * G + g) << bs) + (key0 & (p.t.bs - 1)) : g << bs;
       };
-      load(0, hk * NC, NC);
-      for (int j = 0; j < ntiles; ++j) {
-        if (j + 1 < ntiles) load(j + 1, hk * NC, NC);
-        for (int v = 0; v < vhalves; ++v) load(j, chunk0 + 2 * v, min(2, vchunks - 2 * v));
+      auto take = [&](int slots, int bytes) {      // lane groups 0 .. slots - 1 wait for their slots; returns this lane's
+        const int n = at + sub, s = n % kSlots;
+        if (ok && sub < slots && box == 0) {
+          ok = mbar_wait(&empty[s], ((n / kSlots) & 1) ^ 1, abort_flag);
+          if (ok) mbar_expect_tx(&full[s], bytes);
+        }
+        ok = __all_sync(0xffffffffu, ok);
+        at += slots;
+        return s;
+      };
+      auto load_k = [&](int j) {
+        const int key0 = (ntiles - 1 - j) * TK + box * 16, s = take(NC, kChunk);
+        if (ok && sub < NC) tma_load_2d(ring + s * kSlot + box * 2048, &tmK, sub * 64, row_of(key0, hk), &full[s]);
+      };
+      auto load_v = [&](int j) {                   // slot: 32 keys; box: 16 of them and one of the chunks
+        const int key0 = (ntiles - 1 - j) * TK + sub * 32 + (box & 1) * 16, s = take(4, vchunks * kVChunk), c = chunk0 + (box >> 1);
+        if (ok && (box >> 1) < vchunks)
+          tma_load_2d(ring + s * kSlot + (box >> 1) * kVChunk + (box & 1) * 2048, &tmK, (c % NC) * 64, row_of(key0, c / NC), &full[s]);
+      };
+      load_k(0);
+      for (int j = 0; j < ntiles && ok; ++j) {
+        if (j + 1 < ntiles) load_k(j + 1);
+        load_v(j);
       }
     }
   } else if (warp == 1) {
     // ------------------------------------------------------------------ MMA issue, in the same order
     if (lane == 0 && ntiles > 0) {
-      const uint32_t idesc_qk = umma_idesc_bf16(TQ, TK);
-      const uint32_t q_addr = smem_u32(sQ), ring_addr = smem_u32(ring);
-      Ring st;
-      bool ok = mbar_wait(q_full, 0, abort_flag);
-      auto issue_qk = [&](int j) {
-        ok = mbar_wait(&full[st.idx], st.phase, abort_flag);
-        if (!ok) return;
+      const uint32_t idesc_qk = umma_idesc_bf16(TQ, TK), idesc_pv = umma_idesc_bf16(TQ, vchunks * 64) | (1u << 16);   // operand B (V) is MN-major
+      // Descriptors are a constant beside the address in 16-byte units, so one thread issues the products with an addition for each.
+      const uint64_t dq = umma_desc_sw128(smem_u32(sQ)), dk0 = umma_desc_sw128(smem_u32(ring)), dv0 = desc_mn(smem_u32(ring));
+      int at = 0;   // slots used so far
+      auto wait_slots = [&](int n) {
+        bool good = true;
+        for (int i = 0; i < n && good; ++i) good = mbar_wait(&full[(at + i) % kSlots], ((at + i) / kSlots) & 1, abort_flag);
+        return good;
+      };
+      auto issue_qk = [&](int j) {   // its slots have been waited for
         tc_fence_after();
-        const uint32_t k_base = ring_addr + st.idx * kSlot;
+        const uint32_t d = tmem_base + kColS + (j & 1) * TK;
 #pragma unroll
-        for (int i = 0; i < DP / 16; ++i) {
-          const int c = (i >> 2) * kChunk;
-          umma_bf16(tmem_base + kColS + (j & 1) * TK, umma_desc_sw128(q_addr + c) + (uint64_t)((i & 3) * 2),
-                    umma_desc_sw128(k_base + c) + (uint64_t)((i & 3) * 2), idesc_qk, i ? 1u : 0u);
+        for (int c = 0; c < NC; ++c) {
+          const int s = (at + c) % kSlots;
+          const uint64_t dk = dk0 + (uint64_t)(s * (kSlot >> 4)), da = dq + (uint64_t)(c * (kChunk >> 4));
+#pragma unroll
+          for (int i = 0; i < 4; ++i) umma_bf16(d, da + (uint64_t)(i * 2), dk + (uint64_t)(i * 2), idesc_qk, (c | i) ? 1u : 0u);
+          umma_commit(&empty[s]);
         }
         umma_commit(&s_full[j & 1]);
-        umma_commit(&empty[st.idx]);
-        st.advance(kSlots);
+        at += NC;
       };
+      bool ok = mbar_wait(q_full, 0, abort_flag) && wait_slots(NC);
       if (ok) issue_qk(0);
+      if (ok && ntiles > 1) ok = wait_slots(NC);
       for (int j = 0; j < ntiles && ok; ++j) {
         if (j + 1 < ntiles) {
           // the buffer holds the weights of tile j - 1: their product must be complete
           if (j > 0) ok = mbar_wait(&o_done[(j - 1) & 1], ((j - 1) >> 1) & 1, abort_flag);
-          if (ok) issue_qk(j + 1);
-        }
-        if (ok) ok = mbar_wait(&p_ready[j & 1], (j >> 1) & 1, abort_flag);
-        for (int v = 0; v < vhalves && ok; ++v) {
-          ok = mbar_wait(&full[st.idx], st.phase, abort_flag);
           if (!ok) break;
-          tc_fence_after();
-          const uint32_t idesc_pv = umma_idesc_bf16(TQ, min(2, vchunks - 2 * v) * 64) | (1u << 16);   // operand B (V) is MN-major
-          const uint32_t v_base = ring_addr + st.idx * kSlot;
-#pragma unroll
-          for (int i = 0; i < TK / 16; ++i) {
-            // 16 keys per MMA: 8 TMEM columns of P (32 keys take 32 columns: 16 of first terms, 16 of second ones), 2048 bytes of V
-            const uint64_t db = desc_mn(v_base + i * 2048);
-            const uint32_t a = tmem_base + kColS + (j & 1) * TK + (i >> 1) * 32 + (i & 1) * 8;
-            umma_bf16_ts(tmem_base + kColO + v * 128, a, db, idesc_pv, (i | j) ? 1u : 0u);
-            umma_bf16_ts(tmem_base + kColO + v * 128, a + 16, db, idesc_pv, 1u);
-          }
-          umma_commit(&empty[st.idx]);
-          st.advance(kSlots);
+          issue_qk(j + 1);
         }
-        if (ok) umma_commit(&o_done[j & 1]);
+        ok = wait_slots(4) && mbar_wait(&p_ready[j & 1], (j >> 1) & 1, abort_flag);
+        if (!ok) break;
+        tc_fence_after();
+        const uint32_t a = tmem_base + kColS + (j & 1) * TK, d = tmem_base + kColO;
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {   // 32 keys: 32 TMEM columns of P (16 of first terms, 16 of second ones), one slot of V
+          const int s = (at + q) % kSlots;
+          const uint64_t dv = dv0 + (uint64_t)(s * (kSlot >> 4));
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            umma_bf16_ts(d, a + q * 32 + i * 8, dv + (uint64_t)(i * 128), idesc_pv, (q | i) ? 1u : (j ? 1u : 0u));
+            umma_bf16_ts(d, a + q * 32 + i * 8 + 16, dv + (uint64_t)(i * 128), idesc_pv, 1u);
+          }
+          umma_commit(&empty[s]);
+        }
+        umma_commit(&o_done[j & 1]);
+        at += 4;
+        if (j + 2 < ntiles) ok = wait_slots(NC);
       }
     }
   } else {
