@@ -26,7 +26,7 @@ class ChannelDelta(nn.Module):
         self.C, self.kw, self.eps = sum(self.sizes), cfg.linear_conv_kernel_dim, cfg.rms_norm_eps
         self.ranks = (cfg.linear_decay_rank or self.D, cfg.linear_gate_rank or self.V)
         kw = dict(quant=None, dtype=cfg.dtype)
-        self.in_proj = LinearBase(cfg.hidden_size, self.sizes + [*self.ranks, self.H], "replicated", prefix=prefix + ".in_proj", **kw)
+        self.in_proj_qkvagb = LinearBase(cfg.hidden_size, self.sizes + [*self.ranks, self.H], "replicated", prefix=prefix + ".in_proj_qkvagb", **kw)
         self.a_proj = ReplicatedLinear(self.ranks[0], self.H * self.D, prefix=prefix + ".a_proj", out_dtype=torch.float32, **kw)
         self.g_proj = ReplicatedLinear(self.ranks[1], self.H * self.V, prefix=prefix + ".g_proj", **kw)
         self.conv_weight = nn.Parameter(torch.zeros(self.C, self.kw, dtype=cfg.dtype), requires_grad=False)
@@ -52,7 +52,7 @@ class ChannelDelta(nn.Module):
         """``state`` = (convolution inputs [slots, taps - 1, C], S fp32 [slots, H, D, V])."""
         if getattr(md, "gdn_record", None) is not None:
             raise ValueError("speculative decoding is not served for delta-rule layers with decays per channel (their states are not recorded per token)")
-        y = self.in_proj(x)
+        y = self.in_proj_qkvagb(x)
         C, (ra, rg) = self.C, self.ranks
         qkv = ops.causal_conv(y[:, :C], self.conv_weight, None, state[0], md, silu=True)
         a = self.a_proj(y[:, C: C + ra])

@@ -345,7 +345,7 @@ class CausalLM(nn.Module):
         (".gate_up_proj", ".gate_proj", 0), (".gate_up_proj", ".up_proj", 1),
         (".in_proj_dqkvg", ".dq_proj", 0), (".in_proj_dqkvg", ".q_proj", 0), (".in_proj_dqkvg", ".dkv_proj", 1), (".in_proj_dqkvg", ".g_proj", 2),
         (".in_proj_qkvg", ".in_proj_q", 0), (".in_proj_qkvg", ".in_proj_k", 1), (".in_proj_qkvg", ".in_proj_v", 2), (".in_proj_qkvg", ".in_proj_g", 3),
-        *((".in_proj", f".in_proj_{n}", i) for i, n in enumerate(("q", "k", "v", "a1", "g1", "b"))),
+        *((".in_proj_qkvagb", f".in_proj_{n}", i) for i, n in enumerate(("q", "k", "v", "a1", "g1", "b"))),
         (".gate_if", ".gate_i", 0), (".gate_if", ".gate_f", 1),
         (".in_proj_qkvz", ".in_proj_q", 0), (".in_proj_qkvz", ".in_proj_k", 1), (".in_proj_qkvz", ".in_proj_v", 2),
         (".in_proj_qkvz", ".in_proj_z", 3), (".in_proj_ba", ".in_proj_b", 0), (".in_proj_ba", ".in_proj_a", 1),
