@@ -102,7 +102,7 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   uint8_t* sQ = smem;
   uint8_t* ring = smem + NC * kChunk;
   uint64_t* q_full = reinterpret_cast<uint64_t*>(smem + kEnd);   // [1]
-  uint64_t* full = q_full + 1;         // [kSlots]
+  uint64_t* full = q_full + 1;         // [kSlots] the slots of a tile have arrived: the barrier of the first one
   uint64_t* empty = full + kSlots;     // [kSlots]
   uint64_t* s_full = empty + kSlots;   // [2] scores of a tile are complete
   uint64_t* p_ready = s_full + 2;      // [2] weights written over the scores
@@ -180,24 +180,25 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       auto row_of = [&](int key0, int g) {         // keys past the sequence read the null block
         return key0 < S ? ((bt[key0 >> bs] * G + g) << bs) + (key0 & (p.t.bs - 1)) : g << bs;
       };
+      uint64_t* arrived = nullptr;                 // barrier of the tile
       auto take = [&](int slots, int bytes) {      // lane groups 0 .. slots - 1 wait for their slots; returns this lane's
         const int n = at + sub, s = n % kSlots;
-        if (ok && sub < slots && box == 0) {
-          ok = mbar_wait(&empty[s], ((n / kSlots) & 1) ^ 1, abort_flag);
-          if (ok) mbar_expect_tx(&full[s], bytes);
-        }
+        if (ok && sub < slots && box == 0) ok = mbar_wait(&empty[s], ((n / kSlots) & 1) ^ 1, abort_flag);
         ok = __all_sync(0xffffffffu, ok);
+        arrived = &full[at % kSlots];
+        if (ok && lane == 0) mbar_expect_tx(arrived, slots * bytes);
+        __syncwarp();
         at += slots;
         return s;
       };
       auto load_k = [&](int j) {
         const int key0 = (ntiles - 1 - j) * TK + box * 16, s = take(NC, kChunk);
-        if (ok && sub < NC) tma_load_2d(ring + s * kSlot + box * 2048, &tmK, sub * 64, row_of(key0, hk), &full[s]);
+        if (ok && sub < NC) tma_load_2d(ring + s * kSlot + box * 2048, &tmK, sub * 64, row_of(key0, hk), arrived);
       };
       auto load_v = [&](int j) {                   // slot: 32 keys; box: 16 of them and one of the chunks
         const int key0 = (ntiles - 1 - j) * TK + sub * 32 + (box & 1) * 16, s = take(4, vchunks * kVChunk), c = chunk0 + (box >> 1);
         if (ok && (box >> 1) < vchunks)
-          tma_load_2d(ring + s * kSlot + (box >> 1) * kVChunk + (box & 1) * 2048, &tmK, (c % NC) * 64, row_of(key0, c / NC), &full[s]);
+          tma_load_2d(ring + s * kSlot + (box >> 1) * kVChunk + (box & 1) * 2048, &tmK, (c % NC) * 64, row_of(key0, c / NC), arrived);
       };
       load_k(0);
       for (int j = 0; j < ntiles && ok; ++j) {
@@ -207,14 +208,19 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     }
   } else if (warp == 1) {
     // ------------------------------------------------------------------ MMA issue, in the same order
-    if (lane == 0 && ntiles > 0) {
+    // The whole warp walks the loop (descriptors stay in uniform registers), one elected lane issues.
+    if (ntiles > 0) {
+      const bool leader = elect_one();
       const uint32_t idesc_qk = umma_idesc_bf16(TQ, TK), idesc_pv = umma_idesc_bf16(TQ, vchunks * 64) | (1u << 16);   // operand B (V) is MN-major
       // Descriptors are a constant beside the address in 16-byte units, so one thread issues the products with an addition for each.
       const uint64_t dq = umma_desc_sw128(smem_u32(sQ)), dk0 = umma_desc_sw128(smem_u32(ring)), dv0 = desc_mn(smem_u32(ring));
+      // Barrier of the tile whose first slot is number n. A slot is the first of a tile in some rounds of the ring only, so its phase is counted apart.
       int at = 0;   // slots used so far
-      auto wait_slots = [&](int n) {
-        bool good = true;
-        for (int i = 0; i < n && good; ++i) good = mbar_wait(&full[(at + i) % kSlots], ((at + i) / kSlots) & 1, abort_flag);
+      uint32_t phases = 0;
+      auto wait_tile = [&]() {
+        const int s = at % kSlots;
+        const bool good = mbar_wait(&full[s], (phases >> s) & 1u, abort_flag);
+        phases ^= 1u << s;
         return good;
       };
       auto issue_qk = [&](int j) {   // its slots have been waited for
@@ -224,16 +230,19 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         for (int c = 0; c < NC; ++c) {
           const int s = (at + c) % kSlots;
           const uint64_t dk = dk0 + (uint64_t)(s * (kSlot >> 4)), da = dq + (uint64_t)(c * (kChunk >> 4));
+          if (leader) {
 #pragma unroll
-          for (int i = 0; i < 4; ++i) umma_bf16(d, da + (uint64_t)(i * 2), dk + (uint64_t)(i * 2), idesc_qk, (c | i) ? 1u : 0u);
-          umma_commit(&empty[s]);
+            for (int i = 0; i < 4; ++i) umma_bf16(d, da + (uint64_t)(i * 2), dk + (uint64_t)(i * 2), idesc_qk, (c | i) ? 1u : 0u);
+            umma_commit(&empty[s]);
+          }
         }
-        umma_commit(&s_full[j & 1]);
+        if (leader) umma_commit(&s_full[j & 1]);
+        __syncwarp();
         at += NC;
       };
-      bool ok = mbar_wait(q_full, 0, abort_flag) && wait_slots(NC);
+      bool ok = mbar_wait(q_full, 0, abort_flag) && wait_tile();
       if (ok) issue_qk(0);
-      if (ok && ntiles > 1) ok = wait_slots(NC);
+      if (ok && ntiles > 1) ok = wait_tile();
       for (int j = 0; j < ntiles && ok; ++j) {
         if (j + 1 < ntiles) {
           // the buffer holds the weights of tile j - 1: their product must be complete
@@ -241,7 +250,7 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           if (!ok) break;
           issue_qk(j + 1);
         }
-        ok = wait_slots(4) && mbar_wait(&p_ready[j & 1], (j >> 1) & 1, abort_flag);
+        ok = wait_tile() && mbar_wait(&p_ready[j & 1], (j >> 1) & 1, abort_flag);
         if (!ok) break;
         tc_fence_after();
         const uint32_t a = tmem_base + kColS + (j & 1) * TK, d = tmem_base + kColO;
@@ -249,16 +258,19 @@ talk_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         for (int q = 0; q < 4; ++q) {   // 32 keys: 32 TMEM columns of P (16 of first terms, 16 of second ones), one slot of V
           const int s = (at + q) % kSlots;
           const uint64_t dv = dv0 + (uint64_t)(s * (kSlot >> 4));
+          if (leader) {
 #pragma unroll
-          for (int i = 0; i < 2; ++i) {
-            umma_bf16_ts(d, a + q * 32 + i * 8, dv + (uint64_t)(i * 128), idesc_pv, (q | i) ? 1u : (j ? 1u : 0u));
-            umma_bf16_ts(d, a + q * 32 + i * 8 + 16, dv + (uint64_t)(i * 128), idesc_pv, 1u);
+            for (int i = 0; i < 2; ++i) {
+              umma_bf16_ts(d, a + q * 32 + i * 8, dv + (uint64_t)(i * 128), idesc_pv, (q | i) ? 1u : (j ? 1u : 0u));
+              umma_bf16_ts(d, a + q * 32 + i * 8 + 16, dv + (uint64_t)(i * 128), idesc_pv, 1u);
+            }
+            umma_commit(&empty[s]);
           }
-          umma_commit(&empty[s]);
         }
-        umma_commit(&o_done[j & 1]);
+        if (leader) umma_commit(&o_done[j & 1]);
+        __syncwarp();
         at += 4;
-        if (j + 2 < ntiles) ok = wait_slots(NC);
+        if (j + 2 < ntiles) ok = wait_tile();
       }
     }
   } else {
