@@ -738,7 +738,7 @@ def grouped_topk(logits, k: int, n_group: int, topk_group: int, bias=None, scori
     sb = s + bias.float() if bias is not None else s
     T, E = s.shape
     gs = sb.view(T, n_group, E // n_group)
-    group_score = gs.topk(2, dim=-1)[0].sum(-1) if bias is not None else gs.max(-1)[0]
+    group_score = gs.topk(min(2, gs.shape[-1]), dim=-1)[0].sum(-1) if bias is not None else gs.max(-1)[0]
     gi = group_score.topk(topk_group, dim=-1)[1]
     mask = torch.zeros(T, n_group, device=s.device, dtype=torch.bool).scatter_(1, gi, True)
     masked = sb.masked_fill(~mask.unsqueeze(-1).expand(T, n_group, E // n_group).reshape(T, E), -float("inf"))

@@ -3,11 +3,15 @@ bf16 and fp32 against the float64 restatement."""
 import pytest
 import torch
 
+import nalasun_models as M
 import nalasun_oracle as O
+from gabisun_models import error, replay, tokens
 
 pytestmark = pytest.mark.gpu
 DEV = "cuda"
 DTYPES = [torch.bfloat16, torch.float32]
+# differences of the logits in units of their spread: bf16 products against float64, and true fp32 against float64
+TOL = {"bfloat16": 0.08, "float32": 1e-4}
 
 
 class Meta:
@@ -306,3 +310,90 @@ def test_embedding_with_positions(H, rows, dtype):
     ids, p = torch.randint(0, 90, (41,), generator=g), torch.randint(0, rows, (41,), generator=g)
     x, _ = ops.embed_stream(ids.int().to(DEV), table.to(DEV), 1.0, rows=pos.to(DEV), positions=p.int().to(DEV))
     assert x.dtype == torch.float32 and (x.cpu().double() - table[ids].double() - pos[p].double()).abs().max() < 1e-6
+
+
+@pytest.mark.parametrize("E,top,scale", [(12, 3, 1.5), (1, 1, 0.5), (64, 6, 2.0), (5, 5, 1.0)])
+def test_sigmoid_router(E, top, scale):
+    from types import SimpleNamespace
+    from onecat_vllm.ops import cuda as K
+    g = torch.Generator().manual_seed(E)
+    h, router = torch.randn(77, 24, generator=g), torch.randn(E, 24, generator=g) * 0.3
+    c = SimpleNamespace(num_experts_per_tok=top, n_group=1, topk_group=1, scoring_func="sigmoid", norm_topk_prob=False, routed_scaling_factor=scale)
+    w, ids = K.route((h @ router.T).to(DEV), c, torch.zeros(E, device=DEV))
+    got = torch.zeros(77, E).scatter_(1, ids.cpu().long(), w.cpu().float())
+    assert (got.double() - O.route(h.double(), router.double(), top, scale)).abs().max() < 1e-5
+
+
+# ------------------------------------------------------------------------------------------------ the engine
+@pytest.fixture(scope="module")
+def models(tmp_path_factory):
+    out = {}
+    for name, cfg in M.CONFIGS.items():
+        w = M.make_weights(cfg, len(name), M.RANKS[name], sharp=1.2)
+        out[name] = (cfg, w, M.save(cfg, w, tmp_path_factory.mktemp(name)))
+    return out
+
+
+def engine(path, dtype, max_tokens, **kw):
+    from onecat_vllm.engine.replay import TraceReplay
+    return TraceReplay(path, dtype, max_tokens, device="cuda", **kw)
+
+
+CASES = [(n, d) for n in M.CONFIGS for d in ("bfloat16", "float32") if not (n == "routed" and d == "bfloat16")]
+
+
+@pytest.mark.parametrize("name,dtype", CASES)
+def test_prompts_portions_and_decoding(models, name, dtype):
+    cfg, w, path = models[name]
+    toks = tokens(cfg, 330, 1)
+    want = O.forward(cfg, w, toks)[0]
+    run = engine(path, dtype, 336)
+    for sizes in ([330], [1] * 40 + [290], [2] * 20 + [100, 3, 130, 1, 1, 55], [250] + [1] * 80, [64, 64, 64, 64, 64, 10], [37] * 9):
+        got = replay(run, {"a": toks}, [[("a", n)] for n in sizes])["a"]
+        assert error(got, want) < TOL[dtype], (sizes[:4], error(got, want))
+    graphs = run.core.executor.worker.runner.graphs
+    if dtype == "bfloat16":
+        assert graphs.eligible and graphs.hits > 0   # single tokens ran as CUDA graphs
+    run.close()
+
+
+@pytest.mark.parametrize("name,dtype", [(n, d) for n, d in CASES if n in ("mixed", "wide", "states", "routed")])
+def test_mixed_batches_reuse_pages_and_slots(models, name, dtype):
+    cfg, w, path = models[name]
+    seqs = {f"r{i}": tokens(cfg, n, 10 + i) for i, n in enumerate((130, 1, 47, 64, 16, 99, 33, 130))}
+    run = engine(path, dtype, 336)
+    steps = [[("r0", 40), ("r1", 1), ("r2", 2)], [("r2", 1), ("r3", 63)], [("r0", 1), ("r3", 1), ("r2", 44), ("r4", 3)], [("r4", 1), ("r0", 17)],
+             [("r5", 50), ("r4", 12), ("r0", 1)]] + [[("r0", 2), ("r5", 3)]] * 15 + [[("r0", 99), ("r5", 99), ("r6", 5)], [("r6", 28), ("r7", 2)]] + \
+            [[("r7", 1)]] * 60 + [[("r7", 68)]]
+    got = replay(run, seqs, steps)
+    for k, t in seqs.items():
+        assert error(got[k], O.forward(cfg, w, t)[0]) < TOL[dtype], k
+    run.close()
+
+
+@pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
+def test_long_decoding(tmp_path, dtype):
+    """Decoding across several context buckets: every new bucket captures its graphs in the middle of live sequences, whose states must not move."""
+    cfg, ranks = M.config(64, 50, [M.attn(4, 2, 16, M.moe(2, 2, 24, 16), 0.3, 90), M.delta(2, 1, 16, 24, None), M.mamba(2, 16, 24, 1, 2, M.moe(1, 1, 20, 16))], positions=1200)
+    w = M.make_weights(cfg, 5, ranks, sharp=1.1)
+    run = engine(M.save(cfg, w, tmp_path), dtype, 2048)
+    seqs = {"a": tokens(cfg, 1100), "b": tokens(cfg, 700, 1)}
+    got = replay(run, seqs, [[("a", 400)], [("b", 5)]] + [[("a", 1), ("b", 1)]] * 695 + [[("a", 1)]] * 5)
+    for k, t in seqs.items():
+        assert error(got[k], O.forward(cfg, w, t)[0]) < TOL[dtype], k
+    run.close()
+
+
+@pytest.mark.parametrize("dtype,name", [("float32", "mixed"), ("float32", "odd"), ("float32", "routed"), ("bfloat16", "wide"), ("bfloat16", "states"), ("bfloat16", "heads")])
+def test_greedy_generation_through_the_scheduler(models, name, dtype):
+    """fp32: token for token. bf16: every chosen token's exact logit is within rounding of the best one along the engine's own path."""
+    from onecat_vllm import LLM, SamplingParams
+    cfg, w, path = models[name]
+    llm = LLM(model=path, dtype=dtype, device="cuda", max_model_len=256, max_num_batched_tokens=96, max_num_seqs=4, kv_cache_memory_bytes=64 << 20)
+    prompts = [tokens(cfg, n, 30 + n) for n in (50, 3, 1, 140, 41)]
+    outs = llm.generate([{"prompt_token_ids": p} for p in prompts], SamplingParams(temperature=0.0, max_tokens=24, ignore_eos=True, detokenize=False))
+    for p, o in zip(prompts, outs):
+        ids = list(o.outputs[0].token_ids)
+        lg = O.forward(cfg, w, p + ids)[0][len(p) - 1:-1]
+        gap = lg.max(-1).values - lg[torch.arange(len(ids)), ids]
+        assert gap.max() <= (0 if dtype == "float32" else 4 * TOL[dtype] * lg.std()), gap.max()
