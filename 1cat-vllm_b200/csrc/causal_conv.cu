@@ -31,7 +31,7 @@ __device__ __forceinline__ void store_vec(E* p, const float (&v)[N]) {
   *reinterpret_cast<Vec<E, N>*>(p) = t;
 }
 
-constexpr int kMaxTaps = 16;
+constexpr int kMaxTaps = 16, kTile = 8;   // most taps; tokens per tile of a long step
 
 // TAPS 0: any number of taps up to kMaxTaps
 template <typename E, int N, int TAPS>
@@ -53,11 +53,20 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(const CausalConvParams
   const E* x = reinterpret_cast<const E*>(p.x) + c;
   E* state = reinterpret_cast<E*>(p.state) + c;
   float w[KT][N], b[N], h[KT][N];   // h[j]: the input j + 1 tokens back
+  E wt[N * KT];   // [channel][tap]: a few vector loads where the taps are whole vectors
+  if constexpr (TAPS == 4 && N > 1) {
+#pragma unroll
+    for (int i = 0; i < TAPS; ++i) *reinterpret_cast<Vec<E, N>*>(wt + i * N) = *reinterpret_cast<const Vec<E, N>*>(reinterpret_cast<const E*>(p.w) + (size_t)c * 4 + i * N);
+  } else {
+#pragma unroll
+    for (int e = 0; e < N * KT; ++e)
+      if (e < N * taps) wt[e] = reinterpret_cast<const E*>(p.w)[(size_t)c * taps + e];
+  }
 #pragma unroll
   for (int j = 0; j < KT; ++j)
     if (j < taps) {
 #pragma unroll
-      for (int e = 0; e < N; ++e) w[j][e] = to_f<E>(reinterpret_cast<const E*>(p.w)[(size_t)(c + e) * taps + j]);
+      for (int e = 0; e < N; ++e) w[j][e] = to_f<E>(wt[e * taps + j]);
     }
 #pragma unroll
   for (int e = 0; e < N; ++e) b[e] = 0.f;
@@ -79,6 +88,28 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(const CausalConvParams
         }
       }
   };
+  // A whole tile inside a portion, away from its first tokens: all rows are loaded before the first one is used.
+  if constexpr (TAPS > 0 && N > 1) {
+    if (start - t0 >= m && stop <= t1 && stop - start == kTile) {
+      Vec<E, N> raw[kTile + TAPS - 1];
+#pragma unroll
+      for (int i = 0; i < kTile + TAPS - 1; ++i) raw[i] = *reinterpret_cast<const Vec<E, N>*>(x + (size_t)(start - (TAPS - 1) + i) * p.ldx);
+#pragma unroll
+      for (int i = 0; i < kTile; ++i) {
+        float y[N];
+#pragma unroll
+        for (int e = 0; e < N; ++e) {
+          y[e] = b[e];
+#pragma unroll
+          for (int j = 0; j < TAPS; ++j) y[e] = fmaf(w[j][e], to_f<E>(raw[i + j].e[e]), y[e]);
+          if (p.silu) y[e] = y[e] * (p.f32 ? 1.f / (1.f + expf(-y[e])) : __fdividef(1.f, 1.f + __expf(-y[e])));
+          if (p.residual) y[e] += to_f<E>(raw[i + TAPS - 1].e[e]);
+        }
+        store_vec<E, N>(reinterpret_cast<E*>(p.y) + (size_t)(start + i) * p.C + c, y);
+      }
+      return;
+    }
+  }
   int t = start;
   if (t > t0 && t - t0 < m) t = min(t1, t0 + m);   // these belong to the thread of the portion's first token
   bool fresh = true;
@@ -158,7 +189,7 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(const CausalConvParams
 
 template <typename E, int N>
 int go(const CausalConvParams& p, cudaStream_t st) {
-  const int threads = 128, tile = p.T <= 2048 ? 1 : 8;
+  const int threads = 128, tile = p.T <= 2048 ? 1 : kTile;
   const dim3 grid((unsigned)((p.C / N + threads - 1) / threads), (unsigned)((p.T + tile - 1) / tile));
   auto run = [&](auto kernel) { launch_k(kernel, grid, dim3(threads), 0, st, true, p, tile); };
   if (p.taps == 4) run(causal_conv_kernel<E, N, 4>);
@@ -175,7 +206,7 @@ int causal_conv_launch(const CausalConvParams& p, cudaStream_t st) {
   if (p.taps < 1 || p.taps > kMaxTaps || p.C < 1 || p.R < 1) return -1;
   const int n = p.f32 ? 4 : 8;
   auto ok = [&](const void* q) { return ((uintptr_t)q & 15) == 0; };
-  const bool vec = p.taps >= 2 && p.taps <= 4 && p.C % n == 0 && p.ldx % n == 0 && ok(p.x) && ok(p.y) && ok(p.state) && ok(p.bias);
+  const bool vec = p.taps >= 2 && p.taps <= 4 && p.C % n == 0 && p.ldx % n == 0 && ok(p.x) && ok(p.y) && ok(p.state) && ok(p.bias) && ok(p.w);
   if (p.f32) return vec ? go<float, 4>(p, st) : go<float, 1>(p, st);
   return vec ? go<__nv_bfloat16, 8>(p, st) : go<__nv_bfloat16, 1>(p, st);
 }

@@ -23,7 +23,7 @@ constexpr int VC = 32, NP = 4, THREADS = VC * NP;
 
 // RT: rows of a column per lane (D up to 4 * RT)
 template <typename E, bool DELTA, int RT>
-__global__ void __launch_bounds__(THREADS) recurrent_kernel(const RecurrenceParams p) {
+__global__ void __launch_bounds__(THREADS, RT == 64 ? 2 : RT == 32 ? 6 : 8) recurrent_kernel(const RecurrenceParams p) {
   constexpr int DP = RT * NP, CH = RT == 64 ? 8 : 16;
   __shared__ __align__(16) float sq[CH][DP], sk[CH][DP];
   __shared__ __align__(16) float sg[DELTA ? CH : 1][DP];
@@ -39,10 +39,14 @@ __global__ void __launch_bounds__(THREADS) recurrent_kernel(const RecurrencePara
   float* Sg = p.state + ((size_t)p.state_slots[r] * p.H + h) * D * V;
   const bool init = p.has_initial_state[r] != 0, mine = col < V;
   float S[RT];
+  const bool whole = D == DP && c0 + VC <= V;   // no padding in this CTA's rows and columns
+  float* mineg = Sg + (size_t)part * RT * V + col;
+  if (whole && init) {
 #pragma unroll
-  for (int k = 0; k < RT; ++k) {
-    const int row = part * RT + k;
-    S[k] = init && mine && row < D ? Sg[(size_t)row * V + col] : 0.f;
+    for (int k = 0; k < RT; ++k) S[k] = mineg[(size_t)k * V];
+  } else {
+#pragma unroll
+    for (int k = 0; k < RT; ++k) S[k] = init && mine && part * RT + k < D ? mineg[(size_t)k * V] : 0.f;
   }
   const float nega = -expf(p.A_log[h]);
   const float skip = DELTA ? 0.f : p.skip[h], dt_bias = DELTA ? 0.f : p.dt_bias[h];
@@ -126,10 +130,15 @@ __global__ void __launch_bounds__(THREADS) recurrent_kernel(const RecurrencePara
       if (part == 0 && mine) reinterpret_cast<E*>(p.out)[((size_t)(tc + i) * p.H + h) * V + col] = from_f<E>(y);
     }
   }
+  int W = V;   // opaque: the rows' addresses are computed again rather than kept in registers since the loads
+  asm volatile("" : "+r"(W));
+  if (whole) {
 #pragma unroll
-  for (int k = 0; k < RT; ++k) {
-    const int row = part * RT + k;
-    if (mine && row < D) Sg[(size_t)row * V + col] = S[k];
+    for (int k = 0; k < RT; ++k) mineg[(size_t)k * W] = S[k];
+  } else {
+#pragma unroll
+    for (int k = 0; k < RT; ++k)
+      if (mine && part * RT + k < D) mineg[(size_t)k * W] = S[k];
   }
 }
 
@@ -145,66 +154,95 @@ int recurrent_go(const RecurrenceParams& p, cudaStream_t st) {
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
-// One warp per (token, part) for parts up to 1024 elements, a CTA of four warps otherwise; the row is read twice (the second time from L1).
-template <typename E, int N, bool WIDE>
-__global__ void __launch_bounds__(128) gated_norm_kernel(const GatedNormParams p) {
-  __shared__ float red[4];
+// LANES lanes own a part of a row and keep it in registers: IT vectors of N elements each. Parts of at least LANES == 32 vectors take a warp, wide
+// ones (LANES == 256) a CTA; parts that are wider still are read twice.
+template <typename E> __device__ __forceinline__ float sigmoid(float x);
+template <> __device__ __forceinline__ float sigmoid<float>(float x) { return 1.f / (1.f + expf(-x)); }
+template <> __device__ __forceinline__ float sigmoid<__nv_bfloat16>(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
+
+template <typename E, int N, int LANES, int IT>
+__global__ void __launch_bounds__(256) gated_norm_kernel(const GatedNormParams p) {
+  struct alignas(sizeof(E) * N) Vec { E e[N]; };
+  __shared__ float red[8];
   pdl_trigger();
   pdl_wait();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const long long item = WIDE ? blockIdx.x : (long long)blockIdx.x * 4 + warp;
-  if (!WIDE && item >= (long long)p.T * p.groups) return;
-  const size_t t = item / p.groups;
-  const int g = (int)(item % p.groups), n = p.n / p.groups, first = (WIDE ? threadIdx.x : lane) * N, step = (WIDE ? 128 : 32) * N;
+  const int lane = threadIdx.x % LANES, n = p.n / p.groups;
+  const long long item = (long long)blockIdx.x * (256 / LANES) + threadIdx.x / LANES;
+  const bool live = item < (long long)p.T * p.groups;
+  const size_t t = live ? item / p.groups : 0;
+  const int g = live ? (int)(item % p.groups) : 0;
   const E* x = reinterpret_cast<const E*>(p.x) + t * p.ld_x + (size_t)g * n;
   const E* z = reinterpret_cast<const E*>(p.gate) + t * p.ld_g + (size_t)g * n;
   const E* w = reinterpret_cast<const E*>(p.w) + (p.w_shared ? 0 : (size_t)g * n);
-  auto ld = [&](const E* q, float (&v)[N]) {
-    struct alignas(sizeof(E) * N) Vec { E e[N]; };
-    const Vec raw = *reinterpret_cast<const Vec*>(q);
-#pragma unroll
-    for (int j = 0; j < N; ++j) v[j] = to_f<E>(raw.e[j]);
-  };
-  auto value = [&](int c, float (&v)[N], float (&s)[N]) {   // what is normalised, and the sigmoid of the gate
-    ld(x + c, v);
-    ld(z + c, s);
+  E* y = reinterpret_cast<E*>(p.y) + t * p.n + (size_t)g * n;
+  float v[IT][N], s[IT][N], ss = 0.f;
+  auto value = [&](int c, float (&a)[N], float (&b)[N]) {   // what is normalised, and the factor behind the norm
+    const Vec vx = *reinterpret_cast<const Vec*>(x + c), vz = *reinterpret_cast<const Vec*>(z + c);
 #pragma unroll
     for (int j = 0; j < N; ++j) {
-      const float sg = 1.f / (1.f + expf(-s[j]));
-      if (p.gate_first) v[j] *= s[j] * sg;
-      s[j] = sg;
+      const float q = to_f<E>(vz.e[j]), sg = sigmoid<E>(q);
+      a[j] = to_f<E>(vx.e[j]) * (p.gate_first ? q * sg : 1.f);
+      b[j] = p.gate_first ? 1.f : sg;
     }
   };
-  float v[N], s[N], ss = 0.f;
-  for (int c = first; c < n; c += step) {
-    if (p.gate_first) value(c, v, s);
-    else ld(x + c, v);
+  auto total = [&](float a) {
 #pragma unroll
-    for (int j = 0; j < N; ++j) ss = fmaf(v[j], v[j], ss);
-  }
-  ss = warp_sum(ss);
-  if (WIDE) {
-    if (lane == 0) red[warp] = ss;
-    __syncthreads();
-    ss = (red[0] + red[1]) + (red[2] + red[3]);
-  }
-  const float inv = 1.f / sqrtf(ss / (float)n + p.eps);
-  for (int c = first; c < n; c += step) {
-    float wv[N];
-    value(c, v, s);
-    ld(w + c, wv);
-    struct alignas(sizeof(E) * N) Vec { E e[N]; } o;
+    for (int o = (LANES < 32 ? LANES : 32) / 2; o > 0; o >>= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
+    if (LANES > 32) {
+      if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = a;
+      __syncthreads();
+      a = 0.f;
 #pragma unroll
-    for (int j = 0; j < N; ++j) o.e[j] = from_f<E>(v[j] * inv * wv[j] * (p.gate_first ? 1.f : s[j]));
-    *reinterpret_cast<Vec*>(reinterpret_cast<E*>(p.y) + t * p.n + (size_t)g * n + c) = o;
+      for (int i = 0; i < 8; ++i) a += red[i];
+    }
+    return a;
+  };
+  auto write = [&](int c, const float (&a)[N], const float (&b)[N], float inv) {
+    const Vec vw = *reinterpret_cast<const Vec*>(w + c);
+    Vec o;
+#pragma unroll
+    for (int j = 0; j < N; ++j) o.e[j] = from_f<E>(a[j] * inv * to_f<E>(vw.e[j]) * b[j]);
+    *reinterpret_cast<Vec*>(y + c) = o;
+  };
+#pragma unroll
+  for (int i = 0; i < IT; ++i) {
+    const int c = (i * LANES + lane) * N;
+    if (live && c < n) {
+      value(c, v[i], s[i]);
+#pragma unroll
+      for (int j = 0; j < N; ++j) ss = fmaf(v[i][j], v[i][j], ss);
+    }
+  }
+  float a[N], b[N];
+  for (int c = (IT * LANES + lane) * N; live && c < n; c += LANES * N) {
+    value(c, a, b);
+#pragma unroll
+    for (int j = 0; j < N; ++j) ss = fmaf(a[j], a[j], ss);
+  }
+  const float inv = 1.f / sqrtf(total(ss) / (float)n + p.eps);
+  if (!live) return;
+#pragma unroll
+  for (int i = 0; i < IT; ++i) {
+    const int c = (i * LANES + lane) * N;
+    if (c < n) write(c, v[i], s[i], inv);
+  }
+  for (int c = (IT * LANES + lane) * N; c < n; c += LANES * N) {
+    value(c, a, b);
+    write(c, a, b, inv);
   }
 }
 
 template <typename E, int N>
 int gated_norm_go(const GatedNormParams& p, cudaStream_t st) {
   const long long items = (long long)p.T * p.groups;
-  if (p.n / p.groups > 1024) launch_k(gated_norm_kernel<E, N, true>, dim3((unsigned)items), dim3(128), 0, st, true, p);
-  else launch_k(gated_norm_kernel<E, N, false>, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, st, true, p);
+  const int vecs = (p.n / p.groups + N - 1) / N;
+  auto run = [&](auto kernel, int lanes) { launch_k(kernel, dim3((unsigned)((items * lanes + 255) / 256)), dim3(256), 0, st, true, p); };
+  if (vecs <= 8) run(gated_norm_kernel<E, N, 8, 1>, 8);
+  else if (vecs <= 16) run(gated_norm_kernel<E, N, 16, 1>, 16);
+  else if (vecs <= 32) run(gated_norm_kernel<E, N, 32, 1>, 32);
+  else if (vecs <= 64) run(gated_norm_kernel<E, N, 32, 2>, 32);
+  else if (vecs <= 128) run(gated_norm_kernel<E, N, 32, 4>, 32);
+  else run(gated_norm_kernel<E, N, 256, 2>, 256);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
 
@@ -221,11 +259,11 @@ int gated_norm_launch(const GatedNormParams& p, cudaStream_t st) {
   if (p.T == 0) return 0;
   if (p.groups < 1 || p.n % p.groups) return -1;
   const int n = p.n / p.groups;
-  const uintptr_t a = p.f32 ? 16 : 8;
-  auto ok = [&](const void* q) { return ((uintptr_t)q & (a - 1)) == 0; };
-  const bool vec = n % 4 == 0 && p.ld_x % 4 == 0 && p.ld_g % 4 == 0 && ok(p.x) && ok(p.gate) && ok(p.w) && ok(p.y);
+  const int v = p.f32 ? 4 : 8;   // elements of a 16-byte vector
+  auto ok = [&](const void* q) { return ((uintptr_t)q & 15) == 0; };
+  const bool vec = n % v == 0 && p.n % v == 0 && p.ld_x % v == 0 && p.ld_g % v == 0 && ok(p.x) && ok(p.gate) && ok(p.w) && ok(p.y);
   if (p.f32) return vec ? gated_norm_go<float, 4>(p, st) : gated_norm_go<float, 1>(p, st);
-  return vec ? gated_norm_go<__nv_bfloat16, 4>(p, st) : gated_norm_go<__nv_bfloat16, 1>(p, st);
+  return vec ? gated_norm_go<__nv_bfloat16, 8>(p, st) : gated_norm_go<__nv_bfloat16, 1>(p, st);
 }
 
 }  // namespace oc

@@ -18,17 +18,33 @@
 namespace oc {
 namespace {
 
-constexpr int C = 64, VT = 32, THREADS = 256;
+constexpr int C = 64, VT = 32, THREADS = 256, PREP = 512;   // tokens per chunk, state columns per CTA, threads of a scan and of delta_prepare
 constexpr int P64 = 72, PV = 40;          // pitches of [*][64] and [*][32] tiles
 constexpr float kLog2e = 1.4426950408889634f;
 
 __device__ __forceinline__ float softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
+// 2^x for exponents that are not positive (2 ulp)
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 __device__ __forceinline__ float bf(const __nv_bfloat16 v) { return __bfloat162float(v); }
 
+// two neighbouring outputs, as far as `left` columns go
+__device__ __forceinline__ void put2(__nv_bfloat16* dst, float a, float b, int left) {
+  if (left >= 2 && ((uintptr_t)dst & 3) == 0) *reinterpret_cast<uint32_t*>(dst) = pack2(a, b);
+  else {
+    if (left >= 1) dst[0] = __float2bfloat16(a);
+    if (left >= 2) dst[1] = __float2bfloat16(b);
+  }
+}
+
 // rows of `width` bf16 columns (zeros from `cols` on and from row `n` on) into a tile of pitch `pitch`
+template <int N>
 __device__ __forceinline__ void fetch_rows(__nv_bfloat16* dst, int pitch, const __nv_bfloat16* src, long long ld, int n, int cols, int width, bool vec) {
   const int segs = width / 8;
-  for (int e = threadIdx.x; e < C * segs; e += THREADS) {
+  for (int e = threadIdx.x; e < C * segs; e += N) {
     const int row = e / segs, c = e % segs * 8;
     __nv_bfloat16* d = dst + row * pitch + c;
     const int live = row < n ? min(8, cols - c) : 0;
@@ -63,11 +79,11 @@ struct PrepSmem {
     float A[C][C + 1];
     __nv_bfloat16 tb[2][C][P64];
   };
-  float rq[C], rk[C], beta[C];
+  float rq[C], rk[C], pd[C], beta[C];   // factors of the unit vectors; diagonal of P; step sizes
 };
 
 template <int DP>
-__global__ void __launch_bounds__(THREADS) delta_prepare_kernel(const DeltaChunkParams p) {
+__global__ void __launch_bounds__(PREP) delta_prepare_kernel(const DeltaChunkParams p) {
   using SM = PrepSmem<DP>;
   using W_ = Ws<DP>;
   constexpr int PD = SM::PD;
@@ -77,39 +93,58 @@ __global__ void __launch_bounds__(THREADS) delta_prepare_kernel(const DeltaChunk
   pdl_wait();
   const int ci = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3;
   const int r = p.chunk_req[ci], tc = p.chunk_t0[ci], n = min(C, p.query_start_loc[r + 1] - tc), D = p.D, hk = h / (p.H / p.Hk);
-  fetch_rows(&s.q[0][0], PD, p.q + (size_t)tc * p.ld + (size_t)hk * D, p.ld, n, D, DP, p.vec);
-  fetch_rows(&s.k[0][0], PD, p.k + (size_t)tc * p.ld + (size_t)hk * D, p.ld, n, D, DP, p.vec);
+  fetch_rows<PREP>(&s.q[0][0], PD, p.q + (size_t)tc * p.ld + (size_t)hk * D, p.ld, n, D, DP, p.vec);
+  fetch_rows<PREP>(&s.k[0][0], PD, p.k + (size_t)tc * p.ld + (size_t)hk * D, p.ld, n, D, DP, p.vec);
   cp_async_commit();
   const float nega = -expf(p.A_log[h]) * kLog2e;
-  for (int e = tid; e < C * DP; e += THREADS) {
+  for (int e = tid; e < C * DP; e += PREP) {
     const int i = e / DP, d = e % DP;
     s.G[i][d] = i < n && d < D ? nega * softplus(p.a[(size_t)(tc + i) * p.ld_a + (size_t)h * D + d] + p.dt_bias[(size_t)h * D + d]) : 0.f;
   }
   if (tid < C) s.beta[tid] = tid < n ? 1.f / (1.f + expf(-bf(p.b[(size_t)(tc + tid) * p.ld_b + h]))) : 0.f;
   cp_async_wait<0>();
   __syncthreads();
-  if (tid < DP) {
-    float x = 0.f;
-#pragma unroll 8
-    for (int i = 0; i < C; ++i) {
-      x += s.G[i][tid];
-      s.G[i][tid] = x;
-    }
+  constexpr int SEG = PREP / DP < 16 ? PREP / DP : 16, PER = C / SEG;   // a channel's running sum in SEG parts
+  if (tid < DP * SEG) {
+    const int d = tid % DP, i0 = tid / DP * PER;
+    float x[PER];
+#pragma unroll
+    for (int i = 0; i < PER; ++i) x[i] = s.G[i0 + i][d];
+#pragma unroll
+    for (int i = 1; i < PER; ++i) x[i] += x[i - 1];
+#pragma unroll
+    for (int i = 0; i < PER; ++i) s.G[i0 + i][d] = x[i];
   }
-  for (int i = warp; i < C; i += THREADS / 32) {
-    float q2 = 0.f, k2 = 0.f;
+  for (int i = warp; i < C; i += PREP / 32) {
+    float q2 = 0.f, k2 = 0.f, qk = 0.f;
 #pragma unroll
     for (int d = lane; d < DP; d += 32) {
       const float a = bf(s.q[i][d]), b = bf(s.k[i][d]);
       q2 = fmaf(a, a, q2);
       k2 = fmaf(b, b, k2);
+      qk = fmaf(a, b, qk);
     }
     q2 = warp_sum(q2);
     k2 = warp_sum(k2);
+    qk = warp_sum(qk);
     if (lane == 0) {
-      s.rq[i] = 1.f / sqrtf(q2 + 1e-6f) * p.scale;
-      s.rk[i] = 1.f / sqrtf(k2 + 1e-6f);
+      const float fq = 1.f / sqrtf(q2 + 1e-6f) * p.scale, fk = 1.f / sqrtf(k2 + 1e-6f);
+      s.rq[i] = fq;
+      s.rk[i] = fk;
+      s.pd[i] = qk * fq * fk;
     }
+  }
+  __syncthreads();
+  if (tid < DP * (SEG - 1)) {   // what the parts ahead add; a part's own last row is left to the end, the others read it
+    const int d = tid % DP, part = tid / DP + 1;
+    float add = 0.f;
+    for (int k = 0; k < part; ++k) add += s.G[(k + 1) * PER - 1][d];
+    float x[PER];
+#pragma unroll
+    for (int i = 0; i < PER; ++i) x[i] = s.G[part * PER + i][d] + add;
+    asm volatile("bar.sync 1, %0;" ::"n"(DP * (SEG - 1)) : "memory");
+#pragma unroll
+    for (int i = 0; i < PER; ++i) s.G[part * PER + i][d] = x[i];
   }
   __syncthreads();
   __nv_bfloat16* ws = p.ws + ((size_t)ci * p.H + h) * W_::elems(p.Vp);
@@ -118,20 +153,20 @@ __global__ void __launch_bounds__(THREADS) delta_prepare_kernel(const DeltaChunk
     ws[W_::p + (size_t)i * C + j] = hi;
     ws[W_::p + C * C + (size_t)i * C + j] = __float2bfloat16(v - bf(hi));
   };
-  // blocks above the diagonal, and A and P inside the diagonal blocks: one thread per pair
-  for (int e = tid; e < C * C; e += THREADS) {
+  // what is not below the diagonal, then A and P inside the diagonal blocks: one thread per pair
+  for (int e = tid; e < C * C; e += PREP) {
     const int i = e >> 6, j = e & 63;
-    if ((j >> 4) > (i >> 4) || ((j >> 4) == (i >> 4) && j > i)) {
+    if (j >= i) {
       s.A[i][j] = 0.f;
-      put_p(i, j, 0.f);
+      put_p(i, j, j == i ? s.pd[i] : 0.f);
     }
   }
-  for (int e = tid; e < 4 * 136; e += THREADS) {
-    const int blk = e & 3;
-    int x = e >> 2, i = (int)((sqrtf(8.f * (float)x + 1.f) - 1.f) * 0.5f);
-    if ((i + 1) * (i + 2) / 2 <= x) ++i;
-    if (i * (i + 1) / 2 > x) --i;
-    const int j = blk * 16 + x - i * (i + 1) / 2;
+  if (tid < 4 * 120) {
+    const int blk = tid & 3, x = tid >> 2;   // x = i (i - 1) / 2 + j for 0 <= j < i < 16
+    int i = (int)((1.f + sqrtf(8.f * (float)x + 1.f)) * 0.5f);
+    if (i * (i + 1) / 2 <= x) ++i;
+    if (i * (i - 1) / 2 > x) --i;
+    const int j = blk * 16 + x - i * (i - 1) / 2;
     i += blk * 16;
     float kk = 0.f, qk = 0.f;
 #pragma unroll 4
@@ -140,11 +175,11 @@ __global__ void __launch_bounds__(THREADS) delta_prepare_kernel(const DeltaChunk
       const uint2 a = *reinterpret_cast<const uint2*>(&s.k[i][d]), b = *reinterpret_cast<const uint2*>(&s.q[i][d]), c = *reinterpret_cast<const uint2*>(&s.k[j][d]);
       auto f2 = [](uint32_t v) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v)); };
       const float2 a0 = f2(a.x), a1 = f2(a.y), b0 = f2(b.x), b1 = f2(b.y), c0 = f2(c.x), c1 = f2(c.y);
-      const float e0 = c0.x * exp2f(gi.x - gj.x), e1 = c0.y * exp2f(gi.y - gj.y), e2 = c1.x * exp2f(gi.z - gj.z), e3 = c1.y * exp2f(gi.w - gj.w);
+      const float e0 = c0.x * ex2(gi.x - gj.x), e1 = c0.y * ex2(gi.y - gj.y), e2 = c1.x * ex2(gi.z - gj.z), e3 = c1.y * ex2(gi.w - gj.w);
       kk = fmaf(a0.x, e0, fmaf(a0.y, e1, fmaf(a1.x, e2, fmaf(a1.y, e3, kk))));
       qk = fmaf(b0.x, e0, fmaf(b0.y, e1, fmaf(b1.x, e2, fmaf(b1.y, e3, qk))));
     }
-    s.A[i][j] = j < i ? s.beta[i] * s.rk[i] * s.rk[j] * kk : 0.f;
+    s.A[i][j] = s.beta[i] * s.rk[i] * s.rk[j] * kk;
     put_p(i, j, s.rq[i] * s.rk[j] * qk);
   }
   // between blocks: rows of block I decayed from its first token on, earlier keys decayed up to it
@@ -159,14 +194,14 @@ __global__ void __launch_bounds__(THREADS) delta_prepare_kernel(const DeltaChunk
       *reinterpret_cast<uint32_t*>(hi) = a;
       *reinterpret_cast<uint32_t*>(lo) = b;
     };
-    for (int e = tid; e < (16 * I + 16) * (DP / 2); e += THREADS) {
+    for (int e = tid; e < (16 * I + 16) * (DP / 2); e += PREP) {
       const int row = e / (DP / 2), d = e % (DP / 2) * 2;
       if (row < 16 * I) {
-        const float e0 = exp2f(ref[d] - s.G[row][d]), e1 = exp2f(ref[d + 1] - s.G[row][d + 1]);
+        const float e0 = ex2(ref[d] - s.G[row][d]), e1 = ex2(ref[d + 1] - s.G[row][d + 1]);
         planes(&s.f.kj[0][row][d], &s.f.kj[1][row][d], *reinterpret_cast<const uint32_t*>(&s.k[row][d]), e0, e1);
       } else {
         const int i = row - 16 * I;
-        const float e0 = exp2f(s.G[row][d] - ref[d]), e1 = exp2f(s.G[row][d + 1] - ref[d + 1]);
+        const float e0 = ex2(s.G[row][d] - ref[d]), e1 = ex2(s.G[row][d + 1] - ref[d + 1]);
         planes(&s.f.ki[0][i][d], &s.f.ki[1][i][d], *reinterpret_cast<const uint32_t*>(&s.k[row][d]), e0, e1);
         planes(&s.f.qi[0][i][d], &s.f.qi[1][i][d], *reinterpret_cast<const uint32_t*>(&s.q[row][d]), e0, e1);
       }
@@ -177,7 +212,7 @@ __global__ void __launch_bounds__(THREADS) delta_prepare_kernel(const DeltaChunk
       const int n0 = (warp >> 1) * 16;
       const uint32_t ah = smem_u32(isq ? &s.f.qi[0][0][0] : &s.f.ki[0][0][0]), al = smem_u32(isq ? &s.f.qi[1][0][0] : &s.f.ki[1][0][0]);
       const uint32_t bh = smem_u32(&s.f.kj[0][0][0]), bl = smem_u32(&s.f.kj[1][0][0]);
-      float acc[2][4] = {};
+      float acc3[3][2][4] = {};   // the three products of the planes, apart: a chain of dependent products each
 #pragma unroll
       for (int ks = 0; ks < DP / 16; ++ks) {
         uint32_t a0[4], a1[4], b0[4], b1[4];
@@ -187,41 +222,42 @@ __global__ void __launch_bounds__(THREADS) delta_prepare_kernel(const DeltaChunk
         ldsm_x4(b1, bnk_addr(bl, PD, n0, ks * 16, lane));
 #pragma unroll
         for (int t = 0; t < 2; ++t) {
-          mma16816(acc[t], a0, b0[2 * t], b0[2 * t + 1]);
-          mma16816(acc[t], a0, b1[2 * t], b1[2 * t + 1]);
-          mma16816(acc[t], a1, b0[2 * t], b0[2 * t + 1]);
+          mma16816(acc3[0][t], a0, b0[2 * t], b0[2 * t + 1]);
+          mma16816(acc3[1][t], a0, b1[2 * t], b1[2 * t + 1]);
+          mma16816(acc3[2][t], a1, b0[2 * t], b0[2 * t + 1]);
         }
       }
 #pragma unroll
       for (int t = 0; t < 2; ++t)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
+          const float sum = acc3[0][t][e] + (acc3[1][t][e] + acc3[2][t][e]);
           const int i = 16 * I + g8 + 8 * (e >> 1), j = n0 + 8 * t + 2 * t4 + (e & 1);
-          if (isq) put_p(i, j, s.rq[i] * s.rk[j] * acc[t][e]);
-          else s.A[i][j] = s.beta[i] * s.rk[i] * s.rk[j] * acc[t][e];
+          if (isq) put_p(i, j, s.rq[i] * s.rk[j] * sum);
+          else s.A[i][j] = s.beta[i] * s.rk[i] * s.rk[j] * sum;
         }
     }
   }
   __syncthreads();
   // decayed queries and keys for the products with the state
-  for (int e = tid; e < C * (DP / 2); e += THREADS) {
+  for (int e = tid; e < C * (DP / 2); e += PREP) {
     const int i = e / (DP / 2), d = e % (DP / 2) * 2;
     const float2 q = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&s.q[i][d])), k = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&s.k[i][d]));
     const float g0 = s.G[i][d], g1 = s.G[i][d + 1];
     uint32_t a, b;
-    split2(q.x * s.rq[i] * exp2f(g0), q.y * s.rq[i] * exp2f(g1), a, b);
+    split2(q.x * s.rq[i] * ex2(g0), q.y * s.rq[i] * ex2(g1), a, b);
     *reinterpret_cast<uint32_t*>(ws + W_::q + (size_t)i * DP + d) = a;
     *reinterpret_cast<uint32_t*>(ws + W_::q + W_::tile + (size_t)i * DP + d) = b;
-    split2(k.x * s.rk[i] * exp2f(s.G[C - 1][d] - g0), k.y * s.rk[i] * exp2f(s.G[C - 1][d + 1] - g1), a, b);
+    split2(k.x * s.rk[i] * ex2(s.G[C - 1][d] - g0), k.y * s.rk[i] * ex2(s.G[C - 1][d + 1] - g1), a, b);
     *reinterpret_cast<uint32_t*>(ws + W_::k + (size_t)i * DP + d) = a;
     *reinterpret_cast<uint32_t*>(ws + W_::k + W_::tile + (size_t)i * DP + d) = b;
   }
   float* wsU = reinterpret_cast<float*>(ws + W_::u);
-  if (tid < DP) wsU[(size_t)C * p.Vp + tid] = exp2f(s.G[C - 1][tid]);
+  if (tid < DP) wsU[(size_t)C * p.Vp + tid] = ex2(s.G[C - 1][tid]);
   // T = (I + A)^-1 in fp32: diagonal blocks by forward substitution, then the block sub-diagonals T_ij = -T_ii sum_{j <= k < i} A_ik T_kj
   {
     float (*T)[C + 1] = s.t.T;
-    for (int e = tid; e < C * C; e += THREADS) T[e >> 6][e & 63] = 0.f;
+    for (int e = tid; e < C * C; e += PREP) T[e >> 6][e & 63] = 0.f;
     __syncthreads();
     if (tid < C) {
       const int b0 = (tid >> 4) * 16, c = tid & 15;
@@ -240,14 +276,14 @@ __global__ void __launch_bounds__(THREADS) delta_prepare_kernel(const DeltaChunk
     __syncthreads();
 #pragma unroll 1
     for (int d = 1; d < 4; ++d) {
-      for (int o = tid; o < (4 - d) * 256; o += THREADS) {
+      for (int o = tid; o < (4 - d) * 256; o += PREP) {
         const int blk = o >> 8, rr = (o >> 4) & 15, c = o & 15, i0 = (blk + d) * 16, j0 = blk * 16;
         float acc = 0.f;
         for (int k = j0; k < i0; ++k) acc = fmaf(s.A[i0 + rr][k], T[k][j0 + c], acc);
         s.t.M[blk][rr][c] = acc;
       }
       __syncthreads();
-      for (int o = tid; o < (4 - d) * 256; o += THREADS) {
+      for (int o = tid; o < (4 - d) * 256; o += PREP) {
         const int blk = o >> 8, rr = (o >> 4) & 15, c = o & 15, i0 = (blk + d) * 16, j0 = blk * 16;
         float acc = 0.f;
 #pragma unroll
@@ -256,7 +292,7 @@ __global__ void __launch_bounds__(THREADS) delta_prepare_kernel(const DeltaChunk
       }
       __syncthreads();
     }
-    for (int e = tid; e < C * C / 2; e += THREADS) {   // A is no longer needed
+    for (int e = tid; e < C * C / 2; e += PREP) {   // A is no longer needed
       const int i = e >> 5, j = (e & 31) * 2;
       uint32_t a, b;
       split2(T[i][j], T[i][j + 1], a, b);
@@ -265,21 +301,21 @@ __global__ void __launch_bounds__(THREADS) delta_prepare_kernel(const DeltaChunk
     }
   }
   // W = T (beta rk 2^G K), then U = T (beta V) in tiles of DP columns
-  const int mt = warp & 3, half = warp >> 2;
+  const int mt = warp & 3, part = warp >> 2;   // 16 rows; DP / 4 columns
   const uint32_t th = smem_u32(&s.tb[0][0][0]), tl = smem_u32(&s.tb[1][0][0]), bh = smem_u32(&s.b[0][0][0]), bl = smem_u32(&s.b[1][0][0]);
   const int vtiles = (p.Vp + DP - 1) / DP;
 #pragma unroll 1
   for (int job = 0; job <= vtiles; ++job) {
     __syncthreads();   // the tile's storage is free
     const int c0 = (job - 1) * DP;
-    for (int e = tid; e < C * (DP / 2); e += THREADS) {
+    for (int e = tid; e < C * (DP / 2); e += PREP) {
       const int i = e / (DP / 2), d = e % (DP / 2) * 2;
       float x = 0.f, y = 0.f;
       if (job == 0) {
         const float2 k = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&s.k[i][d]));
         const float f = s.beta[i] * s.rk[i];
-        x = k.x * f * exp2f(s.G[i][d]);
-        y = k.y * f * exp2f(s.G[i][d + 1]);
+        x = k.x * f * ex2(s.G[i][d]);
+        y = k.y * f * ex2(s.G[i][d + 1]);
       } else if (i < n) {
         const __nv_bfloat16* v = p.v + (size_t)(tc + i) * p.ld + (size_t)h * p.V + c0 + d;
         if (c0 + d < p.V) x = s.beta[i] * bf(v[0]);
@@ -291,9 +327,10 @@ __global__ void __launch_bounds__(THREADS) delta_prepare_kernel(const DeltaChunk
       *reinterpret_cast<uint32_t*>(&s.b[1][i][d]) = b;
     }
     __syncthreads();
-    float acc[DP / 16][4];
+    constexpr int NT = DP / 32;   // tiles of eight columns; DP = 32 has one, loaded with a neighbour that is not used
+    float acc[NT][4];
 #pragma unroll
-    for (int t = 0; t < DP / 16; ++t)
+    for (int t = 0; t < NT; ++t)
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[t][e] = 0.f;
     for (int ks = 0; ks <= mt; ++ks) {   // T is lower triangular
@@ -301,12 +338,12 @@ __global__ void __launch_bounds__(THREADS) delta_prepare_kernel(const DeltaChunk
       ldsm_x4(a0, a_addr(th, P64, mt * 16, ks * 16, lane));
       ldsm_x4(a1, a_addr(tl, P64, mt * 16, ks * 16, lane));
 #pragma unroll
-      for (int np = 0; np < DP / 32; ++np) {
+      for (int np = 0; np < (NT + 1) / 2; ++np) {
         uint32_t b0[4], b1[4];
-        ldsm_x4_t(b0, bkn_addr(bh, PD, ks * 16, half * (DP / 2) + np * 16, lane));
-        ldsm_x4_t(b1, bkn_addr(bl, PD, ks * 16, half * (DP / 2) + np * 16, lane));
+        ldsm_x4_t(b0, bkn_addr(bh, PD, ks * 16, part * (DP / 4) + np * 16, lane));
+        ldsm_x4_t(b1, bkn_addr(bl, PD, ks * 16, part * (DP / 4) + np * 16, lane));
 #pragma unroll
-        for (int t = 0; t < 2; ++t) {
+        for (int t = 0; t < (NT < 2 ? 1 : 2); ++t) {
           mma16816(acc[2 * np + t], a0, b0[2 * t], b0[2 * t + 1]);
           mma16816(acc[2 * np + t], a0, b1[2 * t], b1[2 * t + 1]);
           mma16816(acc[2 * np + t], a1, b0[2 * t], b0[2 * t + 1]);
@@ -314,10 +351,10 @@ __global__ void __launch_bounds__(THREADS) delta_prepare_kernel(const DeltaChunk
       }
     }
 #pragma unroll
-    for (int t = 0; t < DP / 16; ++t)
+    for (int t = 0; t < NT; ++t)
 #pragma unroll
       for (int hh = 0; hh < 2; ++hh) {
-        const int i = mt * 16 + g8 + 8 * hh, d = half * (DP / 2) + t * 8 + t4 * 2;
+        const int i = mt * 16 + g8 + 8 * hh, d = part * (DP / 4) + t * 8 + t4 * 2;
         if (job == 0) {
           uint32_t a, b;
           split2(acc[t][2 * hh], acc[t][2 * hh + 1], a, b);
@@ -396,6 +433,8 @@ __global__ void __launch_bounds__(THREADS) delta_scan_kernel(const DeltaChunkPar
   const uint32_t kh = smem_u32(&s.k[0][0][0]), kl = smem_u32(&s.k[1][0][0]), ph = smem_u32(&s.p[0][0][0]), pl = smem_u32(&s.p[1][0][0]);
   const uint32_t sh = smem_u32(&s.st[0][0][0]), sl = smem_u32(&s.st[1][0][0]), nhh = smem_u32(&s.nv[0][0][0]), nl = smem_u32(&s.nv[1][0][0]);
   auto product = [&](float (&acc)[2][4], uint32_t ah, uint32_t al, int pitch, uint32_t bh, uint32_t bl, int steps) {
+    float m1[2][4] = {}, m2[2][4] = {};   // the three products of the planes, apart: a chain of dependent products each
+#pragma unroll 4
     for (int ks = 0; ks < steps; ++ks) {
       uint32_t a0[4], a1[4], b0[4], b1[4];
       ldsm_x4(a0, a_addr(ah, pitch, mt * 16, ks * 16, lane));
@@ -405,10 +444,14 @@ __global__ void __launch_bounds__(THREADS) delta_scan_kernel(const DeltaChunkPar
 #pragma unroll
       for (int t = 0; t < 2; ++t) {
         mma16816(acc[t], a0, b0[2 * t], b0[2 * t + 1]);
-        mma16816(acc[t], a0, b1[2 * t], b1[2 * t + 1]);
-        mma16816(acc[t], a1, b0[2 * t], b0[2 * t + 1]);
+        mma16816(m1[t], a0, b1[2 * t], b1[2 * t + 1]);
+        mma16816(m2[t], a1, b0[2 * t], b0[2 * t + 1]);
       }
     }
+#pragma unroll
+    for (int t = 0; t < 2; ++t)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[t][e] += m1[t][e] + m2[t][e];
   };
   for (int c = 0; c < nch; ++c) {
     const bool more = c + 1 < nch;
@@ -450,9 +493,9 @@ __global__ void __launch_bounds__(THREADS) delta_scan_kernel(const DeltaChunkPar
 #pragma unroll
       for (int t = 0; t < 2; ++t)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int tok = tbase + c * C + mt * 16 + g8 + 8 * (e >> 1), col = v0 + nh + t * 8 + t4 * 2 + (e & 1);
-          if (tok < t1 && col < V) p.out[((size_t)tok * p.H + h) * V + col] = __float2bfloat16(acc[t][e]);
+        for (int hh = 0; hh < 2; ++hh) {
+          const int tok = tbase + c * C + mt * 16 + g8 + 8 * hh, col = v0 + nh + t * 8 + t4 * 2;
+          if (tok < t1) put2(p.out + ((size_t)tok * p.H + h) * V + col, acc[t][2 * hh], acc[t][2 * hh + 1], V - col);
         }
     }
     cp_async_wait<1>();
@@ -528,20 +571,28 @@ __global__ void __launch_bounds__(THREADS) ssd_chunk_kernel(const DeltaChunkPara
       const int row = sm_t * 16 + g8 + 8 * (e >> 1), col = v0 + sc + t * 8 + t4 * 2 + (e & 1);
       S[t][e] = owner && init && row < D && col < V ? Sg[(size_t)row * V + col] : 0.f;
     }
+  float z[2] = {0.f, 0.f};   // warp 0: step logits of the next chunk, loaded a chunk ahead
+  auto logits = [&](int c) {
+    const int tc = t0 + c * C;
+#pragma unroll
+    for (int j = 0; j < 2; ++j) z[j] = tc + lane + 32 * j < t1 ? bf(p.b[(size_t)(tc + lane + 32 * j) * p.ld_b + h]) : 0.f;
+  };
+  if (warp == 0) logits(0);
   auto fetch = [&](int c) {
     const int b = c & 1, tc = t0 + c * C, n = min(C, t1 - tc);
-    fetch_rows(&s.c[b][0][0], PD, p.q + (size_t)tc * p.ld + (size_t)hk * D, p.ld, n, D, DP, p.vec);
-    fetch_rows(&s.b[b][0][0], PD, p.k + (size_t)tc * p.ld + (size_t)hk * D, p.ld, n, D, DP, p.vec);
-    fetch_rows(&s.x[b][0][0], PV, p.v + (size_t)tc * p.ld + (size_t)h * V + v0, p.ld, n, V - v0, VT, p.vec);
+    fetch_rows<THREADS>(&s.c[b][0][0], PD, p.q + (size_t)tc * p.ld + (size_t)hk * D, p.ld, n, D, DP, p.vec);
+    fetch_rows<THREADS>(&s.b[b][0][0], PD, p.k + (size_t)tc * p.ld + (size_t)hk * D, p.ld, n, D, DP, p.vec);
+    fetch_rows<THREADS>(&s.x[b][0][0], PV, p.v + (size_t)tc * p.ld + (size_t)h * V + v0, p.ld, n, V - v0, VT, p.vec);
     cp_async_commit();
     if (warp == 0) {   // step sizes, and the running sum of the decays' logarithms
       float a[2], g[2];
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         const int i = lane + 32 * j;
-        a[j] = i < n ? fminf(fmaxf(softplus(bf(p.b[(size_t)(tc + i) * p.ld_b + h]) + dt_bias), p.dt_min), p.dt_max) : 0.f;
+        a[j] = i < n ? fminf(fmaxf(softplus(z[j] + dt_bias), p.dt_min), p.dt_max) : 0.f;
         g[j] = nega * a[j];
       }
+      logits(c + 1);
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
         const float x = __shfl_up_sync(0xffffffffu, g[0], o), y = __shfl_up_sync(0xffffffffu, g[1], o);
@@ -596,8 +647,8 @@ __global__ void __launch_bounds__(THREADS) ssd_chunk_kernel(const DeltaChunkPara
 #pragma unroll
         for (int hh = 0; hh < 2; ++hh) {
           const int i = mt * 16 + g8 + 8 * hh, j = nh * 32 + t * 8 + t4 * 2;
-          const float v0_ = j <= i ? acc[t][2 * hh] * exp2f(G[i] - G[j]) * dt[j] : 0.f;
-          const float v1_ = j + 1 <= i ? acc[t][2 * hh + 1] * exp2f(G[i] - G[j + 1]) * dt[j + 1] : 0.f;
+          const float v0_ = j <= i ? acc[t][2 * hh] * ex2(G[i] - G[j]) * dt[j] : 0.f;
+          const float v1_ = j + 1 <= i ? acc[t][2 * hh + 1] * ex2(G[i] - G[j + 1]) * dt[j + 1] : 0.f;
           uint32_t u, w;
           split2(v0_, v1_, u, w);
           *reinterpret_cast<uint32_t*>(&s.p[0][i][j]) = u;
@@ -607,7 +658,7 @@ __global__ void __launch_bounds__(THREADS) ssd_chunk_kernel(const DeltaChunkPara
     for (int e = tid; e < C * (VT / 2); e += THREADS) {   // what a token leaves in the state at the chunk's end
       const int i = e / (VT / 2), d = e % (VT / 2) * 2;
       const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&s.x[b][i][d]));
-      const float f = exp2f(G[C - 1] - G[i]) * dt[i];
+      const float f = ex2(G[C - 1] - G[i]) * dt[i];
       uint32_t u, w;
       split2(x.x * f, x.y * f, u, w);
       *reinterpret_cast<uint32_t*>(&s.xs[0][i][d]) = u;
@@ -615,7 +666,7 @@ __global__ void __launch_bounds__(THREADS) ssd_chunk_kernel(const DeltaChunkPara
     }
     __syncthreads();
     {
-      float acc[2][4] = {};
+      float acc[2][4] = {}, low[2][4] = {};
 #pragma unroll
       for (int ks = 0; ks < DP / 16; ++ks) {
         uint32_t a[4], x[4], y[4];
@@ -625,10 +676,17 @@ __global__ void __launch_bounds__(THREADS) ssd_chunk_kernel(const DeltaChunkPara
 #pragma unroll
         for (int t = 0; t < 2; ++t) {
           mma16816(acc[t], a, x[2 * t], x[2 * t + 1]);
-          mma16816(acc[t], a, y[2 * t], y[2 * t + 1]);
+          mma16816(low[t], a, y[2 * t], y[2 * t + 1]);
         }
       }
-      const float ga = exp2f(G[mt * 16 + g8]), gb = exp2f(G[mt * 16 + g8 + 8]);
+#pragma unroll
+      for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          acc[t][e] += low[t][e];
+          low[t][e] = 0.f;
+        }
+      const float ga = ex2(G[mt * 16 + g8]), gb = ex2(G[mt * 16 + g8 + 8]);
 #pragma unroll
       for (int t = 0; t < 2; ++t) {
         acc[t][0] *= ga; acc[t][1] *= ga; acc[t][2] *= gb; acc[t][3] *= gb;
@@ -641,19 +699,22 @@ __global__ void __launch_bounds__(THREADS) ssd_chunk_kernel(const DeltaChunkPara
 #pragma unroll
         for (int t = 0; t < 2; ++t) {
           mma16816(acc[t], a0, x[2 * t], x[2 * t + 1]);
-          mma16816(acc[t], a1, x[2 * t], x[2 * t + 1]);
+          mma16816(low[t], a1, x[2 * t], x[2 * t + 1]);
         }
       }
 #pragma unroll
       for (int t = 0; t < 2; ++t)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int i = mt * 16 + g8 + 8 * (e >> 1), cc = nh * 16 + t * 8 + t4 * 2 + (e & 1), tok = t0 + c * C + i;
-          if (tok < t1 && v0 + cc < V) p.out[((size_t)tok * p.H + h) * V + v0 + cc] = __float2bfloat16(fmaf(skip, bf(s.x[b][i][cc]), acc[t][e]));
+        for (int hh = 0; hh < 2; ++hh) {
+          const int i = mt * 16 + g8 + 8 * hh, cc = nh * 16 + t * 8 + t4 * 2, tok = t0 + c * C + i;
+          if (tok >= t1) continue;
+          const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&s.x[b][i][cc]));
+          put2(p.out + ((size_t)tok * p.H + h) * V + v0 + cc, fmaf(skip, x.x, acc[t][2 * hh] + low[t][2 * hh]),
+               fmaf(skip, x.y, acc[t][2 * hh + 1] + low[t][2 * hh + 1]), V - v0 - cc);
         }
     }
     if (owner) {
-      const float gc = exp2f(G[C - 1]);
+      const float gc = ex2(G[C - 1]);
 #pragma unroll
       for (int t = 0; t < NC; ++t)
 #pragma unroll
@@ -700,7 +761,7 @@ int delta_go(const DeltaChunkParams& p, int chunks, int longs, cudaStream_t st) 
     if (prepare(delta_prepare_kernel<DP>, sizeof(PrepSmem<DP>)) || prepare(delta_scan_kernel<DP>, sizeof(ScanSmem<DP>))) return -4;
     configured = true;
   }
-  launch_k(delta_prepare_kernel<DP>, dim3((unsigned)chunks, (unsigned)p.H), dim3(THREADS), sizeof(PrepSmem<DP>), st, true, p);
+  launch_k(delta_prepare_kernel<DP>, dim3((unsigned)chunks, (unsigned)p.H), dim3(PREP), sizeof(PrepSmem<DP>), st, true, p);
   launch_k(delta_scan_kernel<DP>, dim3((unsigned)longs, (unsigned)p.H, (unsigned)(p.Vp / VT)), dim3(THREADS), sizeof(ScanSmem<DP>), st, true, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
