@@ -97,9 +97,16 @@ __global__ void __launch_bounds__(PREP) delta_prepare_kernel(const DeltaChunkPar
   fetch_rows<PREP>(&s.k[0][0], PD, p.k + (size_t)tc * p.ld + (size_t)hk * D, p.ld, n, D, DP, p.vec);
   cp_async_commit();
   const float nega = -expf(p.A_log[h]) * kLog2e;
-  for (int e = tid; e < C * DP; e += PREP) {
-    const int i = e / DP, d = e % DP;
-    s.G[i][d] = i < n && d < D ? nega * softplus(p.a[(size_t)(tc + i) * p.ld_a + (size_t)h * D + d] + p.dt_bias[(size_t)h * D + d]) : 0.f;
+  {   // all loads of a thread are in flight before the first is used; a thread keeps its channel
+    constexpr int N = C * DP / PREP, STEP = PREP / DP;
+    const int i0 = tid / DP, d = tid % DP;
+    const float* a = p.a + (size_t)tc * p.ld_a + (size_t)h * D + d;
+    float x[N];
+#pragma unroll
+    for (int k = 0; k < N; ++k) x[k] = d < D && i0 + k * STEP < n ? __ldg(a + (size_t)(i0 + k * STEP) * p.ld_a) : 0.f;
+    const float bias = d < D ? p.dt_bias[(size_t)h * D + d] : 0.f;
+#pragma unroll
+    for (int k = 0; k < N; ++k) s.G[i0 + k * STEP][d] = d < D && i0 + k * STEP < n ? nega * softplus(x[k] + bias) : 0.f;
   }
   if (tid < C) s.beta[tid] = tid < n ? 1.f / (1.f + expf(-bf(p.b[(size_t)(tc + tid) * p.ld_b + h]))) : 0.f;
   cp_async_wait<0>();
@@ -161,8 +168,8 @@ __global__ void __launch_bounds__(PREP) delta_prepare_kernel(const DeltaChunkPar
       put_p(i, j, j == i ? s.pd[i] : 0.f);
     }
   }
-  if (tid < 4 * 120) {
-    const int blk = tid & 3, x = tid >> 2;   // x = i (i - 1) / 2 + j for 0 <= j < i < 16
+  if ((tid & 127) < 120) {   // four warps to a block: lanes read neighbouring rows
+    const int blk = tid >> 7, x = tid & 127;   // x = i (i - 1) / 2 + j for 0 <= j < i < 16
     int i = (int)((1.f + sqrtf(8.f * (float)x + 1.f)) * 0.5f);
     if (i * (i + 1) / 2 <= x) ++i;
     if (i * (i - 1) / 2 > x) --i;
@@ -197,11 +204,13 @@ __global__ void __launch_bounds__(PREP) delta_prepare_kernel(const DeltaChunkPar
     for (int e = tid; e < (16 * I + 16) * (DP / 2); e += PREP) {
       const int row = e / (DP / 2), d = e % (DP / 2) * 2;
       if (row < 16 * I) {
-        const float e0 = ex2(ref[d] - s.G[row][d]), e1 = ex2(ref[d + 1] - s.G[row][d + 1]);
+        const float2 rf = *reinterpret_cast<const float2*>(ref + d), gr = *reinterpret_cast<const float2*>(&s.G[row][d]);
+        const float e0 = ex2(rf.x - gr.x), e1 = ex2(rf.y - gr.y);
         planes(&s.f.kj[0][row][d], &s.f.kj[1][row][d], *reinterpret_cast<const uint32_t*>(&s.k[row][d]), e0, e1);
       } else {
         const int i = row - 16 * I;
-        const float e0 = ex2(s.G[row][d] - ref[d]), e1 = ex2(s.G[row][d + 1] - ref[d + 1]);
+        const float2 rf = *reinterpret_cast<const float2*>(ref + d), gr = *reinterpret_cast<const float2*>(&s.G[row][d]);
+        const float e0 = ex2(gr.x - rf.x), e1 = ex2(gr.y - rf.y);
         planes(&s.f.ki[0][i][d], &s.f.ki[1][i][d], *reinterpret_cast<const uint32_t*>(&s.k[row][d]), e0, e1);
         planes(&s.f.qi[0][i][d], &s.f.qi[1][i][d], *reinterpret_cast<const uint32_t*>(&s.q[row][d]), e0, e1);
       }
@@ -243,12 +252,12 @@ __global__ void __launch_bounds__(PREP) delta_prepare_kernel(const DeltaChunkPar
   for (int e = tid; e < C * (DP / 2); e += PREP) {
     const int i = e / (DP / 2), d = e % (DP / 2) * 2;
     const float2 q = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&s.q[i][d])), k = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&s.k[i][d]));
-    const float g0 = s.G[i][d], g1 = s.G[i][d + 1];
+    const float2 g = *reinterpret_cast<const float2*>(&s.G[i][d]), end = *reinterpret_cast<const float2*>(&s.G[C - 1][d]);
     uint32_t a, b;
-    split2(q.x * s.rq[i] * ex2(g0), q.y * s.rq[i] * ex2(g1), a, b);
+    split2(q.x * s.rq[i] * ex2(g.x), q.y * s.rq[i] * ex2(g.y), a, b);
     *reinterpret_cast<uint32_t*>(ws + W_::q + (size_t)i * DP + d) = a;
     *reinterpret_cast<uint32_t*>(ws + W_::q + W_::tile + (size_t)i * DP + d) = b;
-    split2(k.x * s.rk[i] * ex2(s.G[C - 1][d] - g0), k.y * s.rk[i] * ex2(s.G[C - 1][d + 1] - g1), a, b);
+    split2(k.x * s.rk[i] * ex2(end.x - g.x), k.y * s.rk[i] * ex2(end.y - g.y), a, b);
     *reinterpret_cast<uint32_t*>(ws + W_::k + (size_t)i * DP + d) = a;
     *reinterpret_cast<uint32_t*>(ws + W_::k + W_::tile + (size_t)i * DP + d) = b;
   }
@@ -308,23 +317,33 @@ __global__ void __launch_bounds__(PREP) delta_prepare_kernel(const DeltaChunkPar
   for (int job = 0; job <= vtiles; ++job) {
     __syncthreads();   // the tile's storage is free
     const int c0 = (job - 1) * DP;
-    for (int e = tid; e < C * (DP / 2); e += PREP) {
-      const int i = e / (DP / 2), d = e % (DP / 2) * 2;
-      float x = 0.f, y = 0.f;
-      if (job == 0) {
-        const float2 k = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&s.k[i][d]));
-        const float f = s.beta[i] * s.rk[i];
-        x = k.x * f * ex2(s.G[i][d]);
-        y = k.y * f * ex2(s.G[i][d + 1]);
-      } else if (i < n) {
-        const __nv_bfloat16* v = p.v + (size_t)(tc + i) * p.ld + (size_t)h * p.V + c0 + d;
-        if (c0 + d < p.V) x = s.beta[i] * bf(v[0]);
-        if (c0 + d + 1 < p.V) y = s.beta[i] * bf(v[1]);
-      }
+    constexpr int N = C * DP / 2 / PREP, STEP = PREP * 2 / DP;
+    const int r0 = tid / (DP / 2), d = tid % (DP / 2) * 2;
+    auto put = [&](int i, float x, float y) {
       uint32_t a, b;
       split2(x, y, a, b);
       *reinterpret_cast<uint32_t*>(&s.b[0][i][d]) = a;
       *reinterpret_cast<uint32_t*>(&s.b[1][i][d]) = b;
+    };
+    if (job == 0) {
+#pragma unroll
+      for (int e = 0; e < N; ++e) {
+        const int i = r0 + e * STEP;
+        const float2 k = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&s.k[i][d])), g = *reinterpret_cast<const float2*>(&s.G[i][d]);
+        const float f = s.beta[i] * s.rk[i];
+        put(i, k.x * f * ex2(g.x), k.y * f * ex2(g.y));
+      }
+    } else {
+      float x[N][2];
+#pragma unroll
+      for (int e = 0; e < N; ++e) {
+        const int i = r0 + e * STEP;
+        const __nv_bfloat16* v = p.v + (size_t)(tc + i) * p.ld + (size_t)h * p.V + c0 + d;
+        x[e][0] = i < n && c0 + d < p.V ? bf(__ldg(v)) : 0.f;
+        x[e][1] = i < n && c0 + d + 1 < p.V ? bf(__ldg(v + 1)) : 0.f;
+      }
+#pragma unroll
+      for (int e = 0; e < N; ++e) put(r0 + e * STEP, s.beta[r0 + e * STEP] * x[e][0], s.beta[r0 + e * STEP] * x[e][1]);
     }
     __syncthreads();
     constexpr int NT = DP / 32;   // tiles of eight columns; DP = 32 has one, loaded with a neighbour that is not used
