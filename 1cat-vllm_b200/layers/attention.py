@@ -163,8 +163,9 @@ class TalkingAttention(nn.Module):
     ``r1 ln(1 + r2 distance)`` is taken off the scores.
 
     One cached row per token serves as key and value: the key norm's weight moves into the queries, its factor is one number per token that is
-    cached beside the pages and multiplies the scores. fused q|k GEMM -> norm, temperature and cache insert (one kernel) -> attention in two
-    passes (the mix needs normalised weights, so the first pass leaves every head's maximum and sum) -> output projection."""
+    cached beside the pages and multiplies the scores. fused q|k GEMM -> norm, temperature and cache insert (one kernel) -> attention in one walk
+    over the keys (the mix is linear: every head keeps its weighted sums over the rows of all key heads, and the normalised sums are mixed
+    afterwards) -> output projection."""
 
     kv_shared, token_scale, window, window_keep, bias_table = True, True, 0, 0, None   # what the runner and the graphs ask of an attention layer
 
