@@ -47,8 +47,8 @@ class Mamba2Mixer(nn.Module):
         p = getattr(self, pname)
         p.data.copy_(w.reshape(p.shape).to(p.dtype))
 
-    def state_tensors(self):
-        return [(ops.conv_state_shape(self.conv_dim, self.kw), None), ((self.H, self.N, self.P), torch.float32)]
+    def state_shapes(self):
+        return ops.conv_state_shape(self.conv_dim, self.kw), (self.H, self.N, self.P)
 
     def forward(self, x: torch.Tensor, md, state) -> torch.Tensor:
         """``state`` = (convolution inputs [slots, kw-1, conv_dim], S fp32 [slots, H, N, P])."""
